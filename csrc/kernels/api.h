@@ -5,6 +5,8 @@
 #pragma once
 #include <cuda.h>
 #include <stdint.h>
+#include "attn_maps.h"
+#include "proj_src.h"
 
 namespace nkb {
 int encode_tmap_bf16_2d(CUtensorMap* m, const void* ptr, uint64_t inner, uint64_t outer, uint64_t ld_elems,
@@ -53,10 +55,11 @@ void nkb_set_pdl(int enabled);
 int nkb_gemm_bf16(const void* A, const void* B, void* out, int rows, int cols, int k, long long lda, long long ldb,
                   long long ldo, int transpose_out, int out_fp32, int splits, long long split_stride, int gated,
                   int gate_off, const void* bias, int bias_on_rows, const void* residual, int block_n, int max_ctas,
-                  int weights_operand, int ctas_per_sm, void* stream);
+                  int weights_operand, int ctas_per_sm, int act, void* stream);
 int nkb_gemm_effective_splits(int k, int splits);
 int nkb_gemm_bf16_2cta(const void* A, const void* B, void* out, int m, int n, int k, long long lda, long long ldb,
-                       long long ldo, const void* bias, const void* residual, int gated, int gate_off, void* stream);
+                       long long ldo, const void* bias, const void* residual, int gated, int gate_off, int act,
+                       void* stream);
 int nkb_gemm_bf16_push(const void* weights, const void* x, int features, int tokens, int k, long long ldw,
                        long long ldx, long long ldo, int splits, const void* bias, int block_n, void* const* peer_out,
                        void* const* peer_flag, int n_peers, int rank, void* done_counter, void* mc_out, void* mc_flag,
@@ -151,4 +154,39 @@ int nkb_flash_attn_prefill(const void* q, const void* k_cache, const void* v_cac
                            int total_q, int max_q_len, int nq, int nkv, int head_dim, int block_size, int num_blocks,
                            int max_blocks_per_seq, float scale, int causal, int window, const float* sinks,
                            void* stream);
+
+// layers with an fp32 residual stream (gated_residual.cu)
+int nkb_gated_residual(const float* x_in, const int* ids, const void* table, int table_bf16, int vocab, float scale,
+                       int branches, const NkbProj* y, const NkbProj* g, const float* const* gbias, const float* add_row,
+                       const float* add_mat, float* x_out, int norms, const float* const* w, void* const* out,
+                       int out_bf16, int rows, int width, int groups, float eps, void* stream);
+int nkb_gated_act(const NkbProj* gate, const NkbProj* up, void* out, int out_bf16, int rows, int inter, int kind,
+                  void* stream);
+// CUDA-core GEMM for 32-bit models and untileable sizes (gemm_simt.cu)
+int nkb_gemm_simt(const void* x, int x_bf16, const void* w, int w_bf16, void* out, int out_bf16, int m, int n, int k,
+                  long long ldx, long long ldw, long long ldo, void* stream);
+// gated linear recurrence (recurrent.cu)
+int nkb_hgrn2_scan(const NkbProj* q, const NkbProj* f, const NkbProj* v, const float* f_bias, const float* lower,
+                   float* state, const int* slot_ids, const int* q_start, const int* q_lens, const int* context_lens,
+                   void* out, int out_bf16, int batch, int tokens, int heads, int dim, int vdim, const float* norm_w,
+                   float eps, void* stream);
+int nkb_hgrn2_step(const NkbProj* q, const NkbProj* f, const NkbProj* v, const float* f_bias, const float* lower,
+                   float* state, const int* slot_ids, const int* context_lens, void* out, int out_bf16, int batch,
+                   int heads, int dim, int vdim, const float* norm_w, float eps, void* stream);
+// attention with several score maps over shared values (attn_maps.cu, attn_maps_prefill.cu)
+int nkb_maps_append(const NkbMapsArgs* a, const NkbProj* q, const NkbProj* k, const NkbProj* v, const float* cos_sin,
+                    int rot_dims, int max_pos, const int* positions, const int* slots, void* q_out, void* k_cache,
+                    void* v_cache, int bf16, int tokens, int block_size, void* stream);
+int nkb_maps_attn_simple(const NkbMapsArgs* a, const void* q, const void* k_cache, const void* v_cache,
+                         const int* block_table, const int* q_start, const int* q_lens, const int* context_lens,
+                         void* out, int bf16, int batch, int total_q, int block_size, int max_blocks_per_seq,
+                         void* stream);
+long long nkb_maps_decode_scratch_floats(const NkbMapsArgs* a, int batch, int num_splits);
+int nkb_maps_attn_decode(const NkbMapsArgs* a, const void* q, const void* k_cache, const void* v_cache,
+                         const int* block_table, const int* context_lens, void* out, float* scratch, int batch,
+                         int block_size, int num_blocks, int max_blocks_per_seq, int num_splits, void* stream);
+int nkb_maps_attn_prefill(const NkbMapsArgs* a, const void* q, const void* k_cache, const void* v_cache,
+                          const int* block_table, const int* q_start, const int* q_lens, const int* context_lens,
+                          void* out, int batch, int total_q, int max_q_len, int block_size, int num_blocks,
+                          int max_blocks_per_seq, void* stream);
 }

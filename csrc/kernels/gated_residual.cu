@@ -1,0 +1,254 @@
+// The elementwise ends of a layer whose residual stream stays in fp32:
+//
+//   embedding        x = table[id] * scale
+//   gated residual   x <- x + sum_i sigmoid(gate_i + gate_bias_i) * branch_i   (+ a per-model vector) (+ a
+//                    per-token matrix, both used ahead of a repeated block of layers)
+//   group norms      out_j = w_j * x / sqrt(mean over the element's group of x^2 + eps), up to two weightings
+//                    of one normalised row (layers whose two sublayers read the same residual)
+//
+// in one launch per layer: a CTA owns a token row, keeps it in shared memory between the sum and the norm, and
+// takes the branches and gates as split-K partial sums, bf16 or fp32 (proj_src.h).  Also here: the gated
+// activation act(gate) * up over the same forms.
+#include "common.cuh"
+#include "proj_src.cuh"
+#include "api.h"
+
+namespace nkb {
+
+constexpr int kGrMaxGroups = 1024;
+
+struct GatedResidualParams {
+  const float* x_in;              // fp32 rows, or nullptr with ids / table
+  const int* ids;
+  const void* table;              // [vocab, width], bf16 or fp32
+  float scale;
+  int vocab, table_bf16;
+  int branches;
+  NkbProj y[2], g[2];
+  const float* gbias[2];
+  const float* add_row;           // [width] or nullptr
+  const float* add_mat;           // [tokens, width] fp32 or nullptr
+  float* x_out;                   // may be nullptr
+  int norms;
+  const float* w[2];
+  void* out[2];
+  int width, groups;
+  float eps;
+};
+
+template <int V>
+struct VecF {
+  float v[V];
+};
+
+template <int V, typename OutT>
+__global__ void __launch_bounds__(256) gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
+  extern __shared__ float row_s[];                 // [width] then [groups]
+  __shared__ float red[8];
+  float* inv_s = row_s + p.width;
+  const long long t = blockIdx.x;
+  const int nv = p.width / V;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  griddep_wait();
+  griddep_launch();
+  const int id = p.ids ? min(max(p.ids[t], 0), p.vocab - 1) : 0;
+  for (int i = threadIdx.x; i < nv; i += blockDim.x) {
+    const int c = i * V;
+    float a[V];
+    if (p.x_in) {
+      if constexpr (V == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(p.x_in + t * p.width + c);
+        a[0] = x.x; a[1] = x.y; a[2] = x.z; a[3] = x.w;
+      } else {
+        a[0] = p.x_in[t * p.width + c];
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        const long long o = (long long)id * p.width + c + j;
+        a[j] = p.scale * (p.table_bf16 ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.table)[o])
+                                       : reinterpret_cast<const float*>(p.table)[o]);
+      }
+    }
+    float s[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) s[j] = 0.f;
+#pragma unroll
+    for (int b = 0; b < 2; ++b) {
+      if (b < p.branches) {
+        float y[V], g[V];
+        if constexpr (V == 4) {
+          const float4 yy = proj_load4(p.y[b], t, c), gg = proj_load4(p.g[b], t, c);
+          const float4 bb = *reinterpret_cast<const float4*>(p.gbias[b] + c);
+          y[0] = yy.x; y[1] = yy.y; y[2] = yy.z; y[3] = yy.w;
+          g[0] = gg.x + bb.x; g[1] = gg.y + bb.y; g[2] = gg.z + bb.z; g[3] = gg.w + bb.w;
+        } else {
+          y[0] = proj_load(p.y[b], t, c);
+          g[0] = proj_load(p.g[b], t, c) + p.gbias[b][c];
+        }
+#pragma unroll
+        for (int j = 0; j < V; ++j) s[j] += y[j] * sigmoid_f(g[j]);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      a[j] += s[j];
+      if (p.add_mat) a[j] += p.add_mat[t * p.width + c + j];
+      if (p.add_row) a[j] += p.add_row[c + j];
+      row_s[c + j] = a[j];
+    }
+    if (p.x_out) {
+      if constexpr (V == 4)
+        *reinterpret_cast<float4*>(p.x_out + t * p.width + c) = make_float4(a[0], a[1], a[2], a[3]);
+      else
+        p.x_out[t * p.width + c] = a[0];
+    }
+  }
+  if (p.norms == 0) return;
+  __syncthreads();
+  const int gsz = p.width / p.groups;
+  if (p.groups <= nw) {
+    // nw / groups warps share a group
+    const int wpg = nw / p.groups, g = warp / wpg, sub = warp % wpg;
+    float ss = 0.f;
+    if (g < p.groups)
+      for (int i = sub * 32 + lane; i < gsz; i += wpg * 32) {
+        const float v = row_s[g * gsz + i];
+        ss += v * v;
+      }
+    ss = warp_sum(ss);
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    if (int(threadIdx.x) < p.groups) {
+      float tot = 0.f;
+      for (int i = 0; i < wpg; ++i) tot += red[threadIdx.x * wpg + i];
+      inv_s[threadIdx.x] = 1.f / sqrtf(tot / float(gsz) + p.eps);
+    }
+  } else {
+    for (int g = warp; g < p.groups; g += nw) {
+      float ss = 0.f;
+      for (int i = lane; i < gsz; i += 32) {
+        const float v = row_s[g * gsz + i];
+        ss += v * v;
+      }
+      ss = warp_sum(ss);
+      if (lane == 0) inv_s[g] = 1.f / sqrtf(ss / float(gsz) + p.eps);
+    }
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < nv; i += blockDim.x) {
+    const int c = i * V;
+    const float inv = inv_s[c / gsz];              // V > 1 only when a group is a multiple of V
+    float a[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) a[j] = row_s[c + j] * inv;
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+      if (n < p.norms) {
+        OutT* o = reinterpret_cast<OutT*>(p.out[n]) + t * p.width + c;
+        if constexpr (V == 4 && sizeof(OutT) == 2) {
+          const float4 w = *reinterpret_cast<const float4*>(p.w[n] + c);
+          *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16x2(a[0] * w.x, a[1] * w.y), pack_bf16x2(a[2] * w.z, a[3] * w.w));
+        } else {
+#pragma unroll
+          for (int j = 0; j < V; ++j) o[j] = cast_out<OutT>(a[j] * p.w[n][c + j]);
+        }
+      }
+    }
+  }
+}
+
+// kind 0: SiLU, 1: GELU in its tanh form, written with the exponential: (1 + tanh u) / 2 = 1 / (1 + exp(-2 u))
+__device__ __forceinline__ float gate_act(float z, int kind) {
+  if (kind == 0) return z / (1.f + expf(-z));
+  return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
+
+template <int V, typename OutT>
+__global__ void __launch_bounds__(256) gated_act_kernel(const __grid_constant__ NkbProj gate,
+                                                        const __grid_constant__ NkbProj up, OutT* __restrict__ out,
+                                                        int rows, int inter, int kind) {
+  const int nv = inter / V;
+  const long long n = (long long)rows * nv;
+  griddep_wait();
+  griddep_launch();
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / nv;
+    const int c = int(i % nv) * V;
+    float g[V], u[V];
+    if constexpr (V == 4) {
+      const float4 a = proj_load4(gate, r, c), b = proj_load4(up, r, c);
+      g[0] = a.x; g[1] = a.y; g[2] = a.z; g[3] = a.w;
+      u[0] = b.x; u[1] = b.y; u[2] = b.z; u[3] = b.w;
+    } else {
+      g[0] = proj_load(gate, r, c);
+      u[0] = proj_load(up, r, c);
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) g[j] = gate_act(g[j], kind) * u[j];
+    OutT* o = out + r * inter + c;
+    if constexpr (V == 4 && sizeof(OutT) == 2) {
+      *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16x2(g[0], g[1]), pack_bf16x2(g[2], g[3]));
+    } else {
+#pragma unroll
+      for (int j = 0; j < V; ++j) o[j] = cast_out<OutT>(g[j]);
+    }
+  }
+}
+
+}  // namespace nkb
+
+using namespace nkb;
+
+static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+extern "C" int nkb_gated_residual(const float* x_in, const int* ids, const void* table, int table_bf16, int vocab,
+                                  float scale, int branches, const NkbProj* y, const NkbProj* g,
+                                  const float* const* gbias, const float* add_row, const float* add_mat, float* x_out,
+                                  int norms, const float* const* w, void* const* out, int out_bf16, int rows, int width,
+                                  int groups, float eps, void* stream) {
+  if (rows <= 0) return 0;
+  if (width <= 0 || width > 12000 || groups < 1 || groups > kGrMaxGroups || width % groups) return -2;
+  if (branches < 0 || branches > 2 || norms < 0 || norms > 2 || (!x_in && (!ids || !table || vocab < 1))) return -2;
+  GatedResidualParams p{};
+  p.x_in = x_in; p.ids = ids; p.table = table; p.scale = scale; p.vocab = vocab; p.table_bf16 = table_bf16;
+  p.branches = branches; p.norms = norms;
+  bool vec = width % 4 == 0 && (width / groups) % 4 == 0 && (!x_in || aligned16(x_in)) && (!x_out || aligned16(x_out));
+  for (int b = 0; b < branches; ++b) {
+    p.y[b] = y[b]; p.g[b] = g[b]; p.gbias[b] = gbias[b];
+    vec = vec && proj_vec4_ok(y[b]) && proj_vec4_ok(g[b]) && aligned16(gbias[b]);
+  }
+  for (int n = 0; n < norms; ++n) {
+    p.w[n] = w[n]; p.out[n] = out[n];
+    vec = vec && aligned16(w[n]) && aligned16(out[n]);
+  }
+  p.add_row = add_row; p.add_mat = add_mat; p.x_out = x_out;
+  p.width = width; p.groups = groups; p.eps = eps;
+  const size_t smem = size_t(width + groups) * sizeof(float);
+  const int threads = (vec ? width / 4 : width) > 128 ? 256 : 128;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (smem > 48 * 1024) return -2;
+  if (vec)
+    return out_bf16 ? launch_pdl(gated_residual_kernel<4, __nv_bfloat16>, dim3(rows), dim3(threads), smem, s, p)
+                    : launch_pdl(gated_residual_kernel<4, float>, dim3(rows), dim3(threads), smem, s, p);
+  return out_bf16 ? launch_pdl(gated_residual_kernel<1, __nv_bfloat16>, dim3(rows), dim3(threads), smem, s, p)
+                  : launch_pdl(gated_residual_kernel<1, float>, dim3(rows), dim3(threads), smem, s, p);
+}
+
+extern "C" int nkb_gated_act(const NkbProj* gate, const NkbProj* up, void* out, int out_bf16, int rows, int inter,
+                             int kind, void* stream) {
+  if (rows <= 0 || inter <= 0) return 0;
+  if (kind < 0 || kind > 1) return -2;
+  const bool vec = inter % 4 == 0 && proj_vec4_ok(*gate) && proj_vec4_ok(*up) && aligned16(out);
+  const long long n = (long long)rows * (vec ? inter / 4 : inter);
+  const int blocks = int((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (out_bf16) {
+    auto* o = reinterpret_cast<__nv_bfloat16*>(out);
+    return vec ? launch_pdl(gated_act_kernel<4, __nv_bfloat16>, dim3(blocks), dim3(256), 0, s, *gate, *up, o, rows, inter, kind)
+               : launch_pdl(gated_act_kernel<1, __nv_bfloat16>, dim3(blocks), dim3(256), 0, s, *gate, *up, o, rows, inter, kind);
+  }
+  auto* o = reinterpret_cast<float*>(out);
+  return vec ? launch_pdl(gated_act_kernel<4, float>, dim3(blocks), dim3(256), 0, s, *gate, *up, o, rows, inter, kind)
+             : launch_pdl(gated_act_kernel<1, float>, dim3(blocks), dim3(256), 0, s, *gate, *up, o, rows, inter, kind);
+}

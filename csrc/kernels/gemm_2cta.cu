@@ -32,6 +32,7 @@ struct Gemm2Args {            // <= 128 bytes (see GemmArgs)
   int group_m;                // row tiles that share one sweep over the column tiles (L2 reuse)
   int gated;                  // B holds [gate; up] rows: the pair's first CTA loads gate rows, the second up rows
   int gate_off;               // row offset of the up half in B
+  int act;                    // gated: 0 = SiLU, 1 = GELU (tanh form)
   long long ldo;
   void* out;
   const __nv_bfloat16* bias;
@@ -196,9 +197,15 @@ gemm2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CU
           }
           const int cbase = gcol0 + c;
           if (row >= args.m || cbase >= args.n) continue;
+          if (args.act) {
 #pragma unroll
-          for (int j = 0; j < 32; ++j)
-            v[j] = __float_as_uint(silu_f(__uint_as_float(v[j])) * __uint_as_float(u[j]));
+            for (int j = 0; j < 32; ++j)
+              v[j] = __float_as_uint(gelu_tanh_f(__uint_as_float(v[j])) * __uint_as_float(u[j]));
+          } else {
+#pragma unroll
+            for (int j = 0; j < 32; ++j)
+              v[j] = __float_as_uint(silu_f(__uint_as_float(v[j])) * __uint_as_float(u[j]));
+          }
           const long long off = (long long)row * args.ldo + cbase;
           if (cbase + 32 <= args.n && ((off & 7) == 0)) {
             uint4* p = reinterpret_cast<uint4*>(out_h + off);
@@ -301,7 +308,8 @@ extern "C" int nkb_gemm_2cta_pairs() { return g_pairs_last; }
 // silu(A gate^T) * (A up^T); bias / residual are not applied in that mode.
 extern "C" int nkb_gemm_bf16_2cta(const void* A, const void* B, void* out, int m, int n, int k, long long lda,
                                   long long ldb, long long ldo, const void* bias, const void* residual, int gated,
-                                  int gate_off, void* stream) {
+                                  int gate_off, int act, void* stream) {
+  if (act < 0 || act > 1) return -2;
   if (!status_word() && nkb_init() != 0) return -1;
   if (m <= 0 || n <= 0 || k <= 0) return -2;
   if ((k & 7) || (lda & 7) || (ldb & 7)) return -2;
@@ -312,6 +320,7 @@ extern "C" int nkb_gemm_bf16_2cta(const void* A, const void* B, void* out, int m
   a.tiles_n = gated ? (n + 127) / 128 : (n + 255) / 256;
   a.gated = gated ? 1 : 0;
   a.gate_off = gate_off;
+  a.act = act;
   if (gated && (bias || residual)) return -2;
   a.kb_total = (k + kBlockK - 1) / kBlockK;
   a.bias_on_cols = 1;

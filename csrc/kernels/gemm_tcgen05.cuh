@@ -103,6 +103,10 @@ __device__ __forceinline__ WorkItem decode_work(const GemmArgs& a, const GroupAr
 }
 
 __device__ __forceinline__ float silu_f(float g) { return g / (1.f + __expf(-g)); }
+// tanh-form GELU with the exponential: (1 + tanh(w)) / 2 = 1 / (1 + exp(-2 w))
+__device__ __forceinline__ float gelu_tanh_f(float g) {
+  return g / (1.f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g)));
+}
 
 // GROUPED selects the per-expert variant (3-D weight map, group offsets / tile list, expert
 // biases and the clamped activation); the plain variant compiles none of that.
@@ -499,7 +503,8 @@ __device__ __forceinline__ bool gemm_bf16_body(const CUtensorMap& tmA, const CUt
               tmem_ld_32x16(t0 + BN + c, u);
               tmem_ld_wait();
 #pragma unroll
-              for (int j = 0; j < 16; ++j) x[j] = silu_f(__uint_as_float(g[j])) * __uint_as_float(u[j]);
+              for (int j = 0; j < 16; ++j)
+                x[j] = (args.act ? gelu_tanh_f(__uint_as_float(g[j])) : silu_f(__uint_as_float(g[j]))) * __uint_as_float(u[j]);
             } else {
               uint32_t v[16];
               tmem_ld_32x16(t0 + c, v);
@@ -576,6 +581,10 @@ __device__ __forceinline__ bool gemm_bf16_body(const CUtensorMap& tmA, const CUt
 #pragma unroll
             for (int j = 0; j < 32; ++j)
               v[j] = __float_as_uint(silu_f(__uint_as_float(v[j]) + bias_r) * (__uint_as_float(u[j]) + bias_u));
+          } else if (args.act) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j)
+              v[j] = __float_as_uint(gelu_tanh_f(__uint_as_float(v[j])) * __uint_as_float(u[j]));
           } else {
 #pragma unroll
             for (int j = 0; j < 32; ++j)

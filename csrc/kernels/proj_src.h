@@ -1,0 +1,13 @@
+// Where a kernel finds one slice of a projection's result.  The layers of a mixed decoder hand their
+// projections on in three forms: fp32 split-K partial sums [splits][tokens][ld] (decode-sized batches), a
+// bf16 matrix [tokens][ld] (prefill-sized ones) or an fp32 matrix (32-bit models, the same as one split).
+// `ptr` already points at the slice's first column.
+#pragma once
+
+struct NkbProj {
+  const void* ptr;
+  long long ld;             // elements between two tokens
+  long long split_stride;   // elements between two partial sums (fp32 only)
+  int splits;               // 1 for finished values
+  int bf16;                 // 1 = bf16 values, 0 = fp32
+};

@@ -5,13 +5,66 @@ Llama-style (tests/kernels/llama_decoder_dynamo.py, qwen3_embedding), Qwen3 MoE
 (examples/models/qwen3/config.py:12-46) and gpt-oss
 (examples/models/gpt_oss/config.py:14-68: alternating sliding-window layers,
 attention sinks, biases, clamped SwiGLU, YaRN RoPE).
+
+Decoders whose layers differ from one another (`models/hybrid.py`) list them in
+`ModelConfig.layers`, one `LayerSpec` with its mixer's sizes per layer; the
+uniform fields above (heads, head_dim, intermediate_size) are then unused.
 """
 
 from __future__ import annotations
 
 import math
 from dataclasses import dataclass, field, replace
-from typing import List, Optional
+from typing import List, Optional, Tuple, Union
+
+
+@dataclass(frozen=True)
+class RopeSpec:
+    """Rotary embedding of the first `dims` dimensions of a head, YaRN-scaled when factor is given."""
+    base: float = 10000.0
+    dims: int = 0
+    factor: Optional[float] = None
+    original: float = 0.0
+    fast: float = 32.0
+    slow: float = 1.0
+
+
+@dataclass(frozen=True)
+class MapsAttentionSpec:
+    """Differential attention: two score maps of size `dim` per head over values of size `vdim`."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    diff: float                      # constant part of the second map's weight
+    rope: RopeSpec = RopeSpec()
+    softcap: float = 0.0             # <= 0: scores are not capped
+    kind = "attention"
+
+
+@dataclass(frozen=True)
+class RecurrenceSpec:
+    """HGRN2 linear recurrence: `dim` gated channels by `vdim` values per head."""
+    heads: int
+    dim: int
+    vdim: int
+    kind = "hgrn2"
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: Union[MapsAttentionSpec, RecurrenceSpec]
+    ff: int = 0                      # 0: no feed-forward
+    act: str = "gelu_tanh"
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers [start, stop) run `times` times in a row with the same weights."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass
@@ -49,6 +102,11 @@ class ModelConfig:
     rope_beta_fast: float = 32.0
     rope_beta_slow: float = 1.0
     block_size: int = 32
+    # layer-by-layer description (models/hybrid.py)
+    layers: Optional[List[LayerSpec]] = None
+    loop: Optional[LoopSpec] = None
+    embedding_scale: float = 1.0
+    norm_groups: int = 1
 
     @property
     def q_size(self) -> int:
@@ -85,8 +143,26 @@ class ModelConfig:
             top_k=max(1, self.top_k // n) if self.is_moe else 0,      # same (token, expert) pairs per rank
             vocab_size=self.vocab_size // n)
 
+    def layer_runs(self) -> List[Tuple[int, int]]:
+        """(layer, pass) in execution order for a layer-by-layer configuration; pass is -1 outside the loop."""
+        n = len(self.layers)
+        lp = self.loop or LoopSpec(n, n, 1)
+        return ([(i, -1) for i in range(lp.start)]
+                + [(i, t) for t in range(lp.times) for i in range(lp.start, lp.stop)]
+                + [(i, -1) for i in range(lp.stop, n)])
+
     def param_count(self) -> int:
         h = self.hidden_size
+        if self.layers is not None:
+            n = 2 * self.vocab_size * h + h + (self.loop.times * h if self.loop else 0)
+            for l in self.layers:
+                m = l.mixer
+                if m.kind == "hgrn2":
+                    n += h * m.heads * (2 * m.dim + 2 * m.vdim) + 2 * m.heads * m.dim + m.vdim
+                else:
+                    n += h * (2 * m.dim * (m.heads + m.kv_heads) + m.vdim * (m.heads + m.kv_heads)) + 4 * m.dim
+                n += h + h * h + h + ((3 * l.ff + h + 2) * h if l.ff else 0)
+            return n
         attn = h * (self.q_size + 2 * self.kv_size) + self.q_size * h
         if self.is_moe:
             ffn = self.num_experts * 3 * h * self.moe_intermediate_size + h * self.num_experts
@@ -140,6 +216,73 @@ def tiny(**kw) -> ModelConfig:
     """Small dense config for unit tests and the smoke run."""
     base = dict(name="tiny", vocab_size=512, hidden_size=256, num_layers=2, num_heads=4, num_kv_heads=2,
                 head_dim=64, intermediate_size=512, max_position=512)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+def rope_frequencies(rope: RopeSpec):
+    """(frequencies [dims / 2], cos / sin multiplier) of a `RopeSpec`.  With a factor, the frequencies are blended
+    between base^(-2i/dims) and the same divided by the factor over the pairs whose wavelengths lie between
+    original / fast and original / slow tokens (bounds rounded outwards to whole pairs)."""
+    import torch
+
+    i = torch.arange(rope.dims // 2, dtype=torch.float64)
+    freq = rope.base ** (-2.0 * i / max(rope.dims, 1))
+    if rope.factor is None:
+        return freq, 1.0
+
+    def pair_of(turns):          # pair index whose angle makes `turns` full turns over the original length
+        return rope.dims * math.log(rope.original / (2 * math.pi * turns)) / (2 * math.log(rope.base))
+
+    lo = max(math.floor(pair_of(rope.fast)), 0)
+    hi = min(math.ceil(pair_of(rope.slow)), rope.dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+    return freq / rope.factor * ramp + freq * (1 - ramp), 0.1 * math.log(rope.factor) + 1.0
+
+
+def tolenex_config(raw: dict, **kw) -> ModelConfig:
+    """`ModelConfig` of a Tolenex config.json."""
+    layers = []
+    for l in raw["layers"]:
+        m, mlp = l["mixer"], l.get("mlp")
+        if l["type"] == "hgrn2":
+            mixer = RecurrenceSpec(m["heads"], m["dim"], m["vdim"])
+        elif l["type"] == "attention":
+            r = m["rot"]
+            sc = r.get("scaling") or {}
+            mixer = MapsAttentionSpec(
+                m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["scale"], m["diff"],
+                RopeSpec(r["base"], r["dims"], sc.get("factor"), sc.get("original", 0), sc.get("fast", 32.0),
+                         sc.get("slow", 1.0)), m.get("softcap") or 0.0)
+        else:
+            raise ValueError(f"unknown layer type {l['type']!r}")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise ValueError(f"unknown feed-forward kind {mlp['kind']!r}")
+        layers.append(LayerSpec(mixer, mlp["ff"] if mlp is not None else 0))
+    lp = raw.get("loop")
+    base = dict(name="tolenex", vocab_size=raw["vocab"], hidden_size=raw["width"], num_layers=len(layers),
+                rms_eps=raw["norm"]["eps"], norm_groups=raw["norm"]["groups"], layers=layers,
+                loop=LoopSpec(lp["start"], lp["stop"], lp["times"]) if lp else None,
+                embedding_scale=raw["embedding"]["scale"], max_position=0)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+def tolenex_shape(width: int, *, layers: int, heads: int, kv_heads: int, ff: int, vocab: int = 32000,
+                  dim: int = 64, vdim: int = 128, recurrent_every: int = 2, loop: Optional[LoopSpec] = None,
+                  groups: int = 4, **kw) -> ModelConfig:
+    """A Tolenex configuration of regular shape: every `recurrent_every`-th layer is an attention layer, the
+    others are recurrences whose heads are vdim by vdim."""
+    rope = RopeSpec(500000.0, dim, 4.0, 8192, 32.0, 1.0)
+    specs = []
+    for i in range(layers):
+        if i % recurrent_every == recurrent_every - 1:
+            mixer = MapsAttentionSpec(heads, kv_heads, dim, vdim, dim ** -0.5, 0.5, rope, 30.0)
+        else:
+            mixer = RecurrenceSpec(heads, vdim, vdim)
+        specs.append(LayerSpec(mixer, ff))
+    base = dict(name="tolenex", vocab_size=vocab, hidden_size=width, num_layers=layers, rms_eps=1e-5,
+                norm_groups=groups, layers=specs, loop=loop, embedding_scale=1.0, max_position=0)
     base.update(kw)
     return ModelConfig(**base)
 

@@ -9,13 +9,18 @@ Full blocks are content-addressed by the hash of their token ids chained with
 the hash of the preceding block, so sequences with a common prompt prefix share
 the blocks (reference-counted; a freed block stays findable until it is
 recycled, least recently freed first).
+
+Layers may also differ: `PagedKVCache.for_layers` takes one `KVLayer` (keys and
+values of any sizes, paged) or `StateLayer` (a fixed-size recurrent state per
+batch row, fp32) per layer.  A state belongs to a whole sequence, not to a block
+of tokens, so a cache with state layers never shares prefixes.
 """
 
 from __future__ import annotations
 
 from collections import OrderedDict
 from dataclasses import dataclass, field
-from typing import Dict, List, Optional, Sequence, Tuple
+from typing import Dict, List, Optional, Sequence, Tuple, Union
 
 import torch
 
@@ -145,24 +150,56 @@ class BlockAllocator:
             self.release_block(b)
 
 
+@dataclass(frozen=True)
+class KVLayer:
+    """Paged keys [block, kv_heads, 32, k_dim] and values [block, kv_heads, 32, v_dim]."""
+    kv_heads: int
+    k_dim: int
+    v_dim: int
+
+
+@dataclass(frozen=True)
+class StateLayer:
+    """Recurrent state of `shape` per batch row, fp32.  The slot of a sequence is its batch row; kernels start a
+    sequence whose first token is at position 0 from zero, so a slot needs no clearing between sequences."""
+    shape: Tuple[int, ...]
+
+
 class PagedKVCache:
-    """Per-layer K/V block pools plus the batch-level device tables the kernels read."""
+    """Per-layer K/V block pools and recurrent states plus the batch-level device tables the kernels read."""
 
     def __init__(self, num_layers: int, num_kv_heads: int, head_dim: int, num_blocks: int, max_batch: int,
                  max_blocks_per_seq: int, device, dtype=torch.bfloat16, enable_prefix_sharing: bool = True):
-        self.num_layers = num_layers
         self.num_kv_heads = num_kv_heads
         self.head_dim = head_dim
+        self._setup([KVLayer(num_kv_heads, head_dim, head_dim)] * num_layers, num_blocks, max_batch,
+                    max_blocks_per_seq, device, dtype, enable_prefix_sharing)
+
+    @classmethod
+    def for_layers(cls, layers: Sequence[Union[KVLayer, StateLayer]], num_blocks: int, max_batch: int,
+                   max_blocks_per_seq: int, device, dtype=torch.bfloat16,
+                   enable_prefix_sharing: bool = True) -> "PagedKVCache":
+        self = cls.__new__(cls)
+        self._setup(list(layers), num_blocks, max_batch, max_blocks_per_seq, device, dtype, enable_prefix_sharing)
+        return self
+
+    def _setup(self, layers, num_blocks, max_batch, max_blocks_per_seq, device, dtype, enable_prefix_sharing) -> None:
+        self.layers = layers
+        self.num_layers = len(layers)
         self.block_size = BLOCK_SIZE
         self.num_blocks = num_blocks
         self.max_batch = max_batch
         self.max_blocks_per_seq = max_blocks_per_seq
         self.device = torch.device(device)
-        shape = (num_blocks, num_kv_heads, BLOCK_SIZE, head_dim)
+        self.has_state = any(isinstance(l, StateLayer) for l in layers)
         # zero-filled: masked positions are multiplied by probability 0 and must be finite
-        self.k = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
-        self.v = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
-        self.allocator = BlockAllocator(num_blocks, BLOCK_SIZE, enable_prefix_sharing)
+        pool = lambda heads, dim: torch.zeros((num_blocks, heads, BLOCK_SIZE, dim), dtype=dtype, device=device)
+        kv = [isinstance(l, KVLayer) for l in layers]
+        self.k = [pool(l.kv_heads, l.k_dim) if on else None for l, on in zip(layers, kv)]
+        self.v = [pool(l.kv_heads, l.v_dim) if on else None for l, on in zip(layers, kv)]
+        self.state = [None if on else torch.zeros((max_batch, *l.shape), dtype=torch.float32, device=device)
+                      for l, on in zip(layers, kv)]
+        self.allocator = BlockAllocator(num_blocks, BLOCK_SIZE, enable_prefix_sharing and not self.has_state)
         self.block_table = torch.zeros((max_batch, max_blocks_per_seq), dtype=torch.int32, device=device)
         pin = self.device.type == "cuda"
         self._table_host = torch.zeros((max_batch, max_blocks_per_seq), dtype=torch.int32, pin_memory=pin)
@@ -171,10 +208,13 @@ class PagedKVCache:
         self._next_id = 0
 
     def bytes(self) -> int:
-        per = self.k[0].numel() * self.k[0].element_size()
-        return 2 * per * self.num_layers
+        return sum(t.numel() * t.element_size() for t in (*self.k, *self.v, *self.state) if t is not None)
 
     # -- admission / growth / release
+    def open_sequence(self) -> SequenceState:
+        """A sequence without tokens yet: a batch row (and state slot) now, blocks as it grows."""
+        return self.add_sequence([])
+
     def add_sequence(self, tokens: Sequence[int]) -> SequenceState:
         if not self._free_slots:
             raise OutOfBlocks("batch table full")

@@ -154,6 +154,46 @@ def random_weights(cfg: ModelConfig, rank: int = 0, world: int = 1, device="cpu"
     return out
 
 
+def hybrid_weight_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
+    """Name -> shape of every tensor of a layer-by-layer configuration (models/hybrid.py), matrices [out, in]."""
+    W, V = cfg.hidden_size, cfg.vocab_size
+    out: Dict[str, tuple] = {"embed": (V, W), "head": (V, W), "final.norm": (W,)}
+    if cfg.loop:
+        out["loop.step"] = (cfg.loop.times, W)
+    for i, layer in enumerate(cfg.layers):
+        p, m = f"l{i}.", layer.mixer
+        shapes = {"norm1": (W,), "rg1": (W, W), "rg1.b": (W,), "mix.o": (W, m.heads * m.vdim)}
+        if m.kind == "hgrn2":
+            c = m.heads * m.dim
+            shapes.update({"mix.q": (c, W), "mix.f": (c, W), "mix.f.b": (c,), "mix.lower": (c,),
+                           "mix.v": (m.heads * m.vdim, W), "mix.norm": (m.vdim,)})
+        else:
+            shapes.update({"mix.q": (2 * m.heads * m.dim, W), "mix.k": (2 * m.kv_heads * m.dim, W),
+                           "mix.v": (m.kv_heads * m.vdim, W)})
+            shapes.update({f"mix.{n}": (m.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
+        if layer.ff:
+            shapes.update({"norm2": (W,), "mlp.gate": (layer.ff, W), "mlp.up": (layer.ff, W),
+                           "mlp.down": (W, layer.ff), "rg2": (W, W), "rg2.b": (W,)})
+        out.update({p + k: v for k, v in shapes.items()})
+    return out
+
+
+def hybrid_random_weights(cfg: ModelConfig, device="cpu", seed: int = 0, std: float = 0.02,
+                          dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
+    """Random-init weights of a layer-by-layer configuration: N(0, std), norm weights 1, lower bounds of the
+    forget gates uniform in [0, 0.9)."""
+    out: Dict[str, torch.Tensor] = {}
+    for n, (name, shape) in enumerate(hybrid_weight_shapes(cfg).items()):
+        if name.endswith(("norm1", "norm2", ".norm")):
+            out[name] = torch.ones(shape, dtype=dtype, device=device)
+        elif name.endswith(".lower"):
+            g = torch.Generator(device=device).manual_seed(seed * 100003 + n)
+            out[name] = (0.9 * torch.rand(shape, generator=g, device=device)).to(dtype)
+        else:
+            out[name] = _normal(shape, std, seed * 100003 + n, device, dtype)
+    return out
+
+
 def save_shard(weights: Dict[str, torch.Tensor], directory: str, rank: int) -> str:
     """Write ``shard_{rank}.safetensors`` (same file naming as the reference converter)."""
     from safetensors.torch import save_file

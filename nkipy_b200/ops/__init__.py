@@ -29,6 +29,7 @@ from ._lib import KernelLibraryError, device_status, raise_on_device_error
 __all__ = [
     "linear", "decode_linear", "qkv_rope_append", "reduce_partials", "rmsnorm", "add_rmsnorm", "silu_mul", "embedding", "rope_kv_append",
     "argmax", "sample", "decode_advance", "router_topk", "moe_dispatch", "grouped_linear", "moe_combine", "paged_attn_decode", "flash_attn_prefill", "rope_table",
+    "MapsSpec", "Proj", "gated_act", "gated_residual", "hgrn2", "maps_append", "maps_attention",
     "KernelLibraryError", "device_status", "raise_on_device_error", "native_available", "launch_count",
     "reset_launch_count",
 ]
@@ -101,12 +102,16 @@ def linear(
     max_ctas: int = 0,
     weights_static: bool = True,
     ctas_per_sm: Optional[int] = None,
+    act: str = "silu",
+    fp32_out: bool = False,
 ) -> torch.Tensor:
     """``y = x @ w.T`` with optional fused epilogue.
 
-    x: [M, K] bf16 (row stride may exceed K), w: [N, K] bf16.
+    x: [M, K] bf16 (row stride may exceed K), w: [N, K] bf16; both fp32 for a model that runs in 32-bit, whose
+           products (and those of operands without a 16-byte row pitch) run on the CUDA cores (gemm_simt.cu).
     gated: w is ``[2*I, K]`` holding gate rows then up rows; returns
-           ``silu(x @ gate.T) * (x @ up.T)`` of shape [M, I].
+           ``act(x @ gate.T) * (x @ up.T)`` of shape [M, I], act "silu" or "gelu_tanh".
+    fp32_out: finished values in fp32 instead of bf16 (not with gated).
     splits > 1: split-K; returns fp32 partial sums ``[S, M, N]`` (S may be smaller
            than requested) for a fused reduction (`add_rmsnorm`, `rope_kv_append`,
            `reduce_partials`).  bias is added to partial 0.
@@ -125,7 +130,7 @@ def linear(
         xf, wf = x.float(), w.float()
         if gated:
             g, u = xf @ wf[:N].T, xf @ wf[N:].T
-            y = torch.nn.functional.silu(g) * u
+            y = mixers.ACTIVATIONS[act][1](g) * u
         else:
             y = xf @ wf.T
         if bias is not None:
@@ -134,15 +139,21 @@ def linear(
             return y.unsqueeze(0)
         if residual is not None:
             y = y + residual.float()
-        y = y.to(torch.bfloat16)
+        y = y.to(torch.float32 if fp32_out or x.dtype == torch.float32 else torch.bfloat16)
         if out is not None:
             out.copy_(y)
             return out
         return y
     global _launches
-    _check_bf16(x, w, bias, residual)
     if x.stride(1) != 1 or w.stride(1) != 1:
         raise ValueError("linear needs K-contiguous operands")
+    if x.dtype == torch.float32 or (K | x.stride(0) | w.stride(0)) & 7:
+        if bias is not None or residual is not None or out is not None:
+            raise ValueError("the CUDA-core GEMM has no bias, residual or out argument")
+        return mixers.linear_simt(x, w, gated=gated, act=act, fp32_out=fp32_out or splits > 1)
+    _check_bf16(x, w, bias, residual)
+    if fp32_out and gated:
+        raise ValueError("fp32_out is for plain products")
     if swap is None:
         swap = M <= 128
     L = _lib.lib()
@@ -157,15 +168,16 @@ def linear(
     else:
         eff = 1
         if out is None:
-            out = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+            out = torch.empty((M, N), dtype=torch.float32 if fp32_out else torch.bfloat16, device=x.device)
         out_view = out
-        out_fp32, split_stride = 0, 0
+        out_fp32, split_stride = 1 if fp32_out else 0, 0
     ldo = out_view.stride(-2) if out_view.dim() >= 2 else N
-    if (not swap and splits <= 1 and M >= 512 and N >= 256 and _USE_2CTA and (ldo & 7) == 0
+    if (not swap and splits <= 1 and not fp32_out and M >= 512 and N >= 256 and _USE_2CTA and (ldo & 7) == 0
             and not (gated and (bias is not None or residual is not None))):
         # prefill-sized: CTA pairs on 256 x 256 tiles (csrc/kernels/gemm_2cta.cu)
         rc = L.nkb_gemm_bf16_2cta(x.data_ptr(), w.data_ptr(), out_view.data_ptr(), M, N, K, x.stride(0), w.stride(0),
-                                  ldo, _ptr(bias), _ptr(residual), 1 if gated else 0, N if gated else 0, _stream())
+                                  ldo, _ptr(bias), _ptr(residual), 1 if gated else 0, N if gated else 0,
+                                  mixers.ACTIVATIONS[act][0], _stream())
         if rc != -5:
             _lib.check(rc, "nkb_gemm_bf16_2cta")
             _launches += 1
@@ -186,7 +198,7 @@ def linear(
         a.data_ptr(), b.data_ptr(), out_view.data_ptr(), rows, cols, K, lda, ldb, ldo, transpose_out, out_fp32,
         eff if splits > 1 else 1, split_stride, gate_mode, N if gated else 0, _ptr(bias), bias_on_rows,
         _ptr(residual), block_n, max_ctas, (0 if swap else 1) if weights_static else -1,
-        (2 if (swap and not gated) else 1) if ctas_per_sm is None else ctas_per_sm, _stream(),
+        (2 if (swap and not gated) else 1) if ctas_per_sm is None else ctas_per_sm, mixers.ACTIVATIONS[act][0], _stream(),
     )
     _lib.check(rc, "nkb_gemm_bf16")
     _launches += 1
@@ -1097,3 +1109,7 @@ def moe_combine(y_sorted: torch.Tensor, pair_pos: torch.Tensor, weights: torch.T
     _lib.check(rc, "nkb_moe_combine")
     _launches += 1
     return out
+
+
+from . import mixers  # noqa: E402  (uses the helpers above)
+from .mixers import (MapsSpec, Proj, gated_act, gated_residual, hgrn2, maps_append, maps_attention)  # noqa: E402,F401

@@ -24,6 +24,7 @@ ROOT = Path(__file__).resolve().parents[2]
 SRC_DIR = ROOT / "csrc" / "kernels"
 OBJ_DIR = ROOT / "build" / "kernels"
 LIB_PATH = Path(__file__).resolve().parent / "libnkipy_b200_kernels.so"
+SUBSET_PATH = LIB_PATH.with_name("libnkipy_b200_serving.so")
 # digest of every source, header and flag the library was built from; `_lib.lib()` refuses to load a
 # library whose stamp does not match the sources (the ctypes signatures are declared from the sources,
 # so a stale binary would receive shifted arguments)
@@ -42,7 +43,13 @@ NVCC_FLAGS = [
 # fast-math turns exp2f / division into their approximate forms, which is what the
 # GEMM epilogue and the attention softmax want; the normalisation and sampling
 # files keep IEEE division and sqrt.
-NO_FAST_MATH = {"sampling.cu", "elementwise.cu", "decode_layer.cu"}
+NO_FAST_MATH = {"sampling.cu", "elementwise.cu", "decode_layer.cu", "gated_residual.cu", "recurrent.cu", "attn_maps.cu",
+                "gemm_simt.cu"}
+
+
+# what a single-GPU decoder of models/hybrid.py launches
+SERVING_SOURCES = ("host_glue.cu", "gemm_tcgen05.cu", "gemm_2cta.cu", "gemm_simt.cu", "elementwise.cu", "sampling.cu",
+                   "gated_residual.cu", "recurrent.cu", "attn_maps.cu", "attn_maps_prefill.cu")
 
 
 def _nvcc() -> str:
@@ -104,12 +111,21 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         return _build_locked(force, verbose)
 
 
-def _build_locked(force: bool, verbose: bool) -> Path:
+def build_subset() -> Path:
+    """Compile (if stale) and link only `SERVING_SOURCES`; returns the library's path.  Objects are shared with the
+    full build."""
+    with _build_lock():
+        objs, _ = _compile([SRC_DIR / n for n in SERVING_SOURCES], False, False)
+        _link(objs, SUBSET_PATH, OBJ_DIR / "link_serving.stamp", False)
+    return SUBSET_PATH
+
+
+def _compile(srcs, force: bool, verbose: bool):
+    """Objects of the given sources, compiled in parallel where their digest changed."""
     nvcc = _nvcc()
     OBJ_DIR.mkdir(parents=True, exist_ok=True)
-    digest = source_digest()
     jobs = []
-    for src in sources():
+    for src in srcs:
         flags = [f for f in NVCC_FLAGS if not (f == "--use_fast_math" and src.name in NO_FAST_MATH)]
         obj = OBJ_DIR / f"{src.stem}.{_digest(src, flags)}.o"
         jobs.append((src, obj, flags))
@@ -130,18 +146,27 @@ def _build_locked(force: bool, verbose: bool) -> Path:
 
     with ThreadPoolExecutor(max_workers=min(8, len(jobs) or 1)) as pool:
         rebuilt = list(pool.map(compile_one, jobs))
-    objs = [str(o) for _, o, _ in jobs]
+    return [str(o) for _, o, _ in jobs], rebuilt
+
+
+def _link(objs, path: Path, stamp_file: Path, force: bool) -> None:
     stamp = hashlib.sha256("".join(objs).encode()).hexdigest()[:16]
-    stamp_file = OBJ_DIR / "link.stamp"
-    if force or not LIB_PATH.exists() or not stamp_file.exists() or stamp_file.read_text() != stamp:
-        # link under a temporary name and move it into place: a process that has the old file mapped keeps it
-        tmp_lib = LIB_PATH.with_name(f".{LIB_PATH.name}.tmp{os.getpid()}")
-        cmd = [nvcc, "-shared", "-o", str(tmp_lib), *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
-        res = subprocess.run(cmd, capture_output=True, text=True)
-        if res.returncode != 0:
-            raise RuntimeError(f"link failed:\n{' '.join(cmd)}\n{res.stdout}\n{res.stderr}")
-        os.replace(tmp_lib, LIB_PATH)
-        stamp_file.write_text(stamp)
+    if not force and path.exists() and stamp_file.exists() and stamp_file.read_text() == stamp:
+        return
+    # link under a temporary name and move it into place: a process that has the old file mapped keeps it
+    tmp_lib = path.with_name(f".{path.name}.tmp{os.getpid()}")
+    cmd = [_nvcc(), "-shared", "-o", str(tmp_lib), *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
+    res = subprocess.run(cmd, capture_output=True, text=True)
+    if res.returncode != 0:
+        raise RuntimeError(f"link failed:\n{' '.join(cmd)}\n{res.stdout}\n{res.stderr}")
+    os.replace(tmp_lib, path)
+    stamp_file.write_text(stamp)
+
+
+def _build_locked(force: bool, verbose: bool) -> Path:
+    digest = source_digest()
+    objs, rebuilt = _compile(sources(), force, verbose)
+    _link(objs, LIB_PATH, OBJ_DIR / "link.stamp", force)
     STAMP_PATH.write_text(digest)
     if verbose:
         for msg in rebuilt:

@@ -17,8 +17,24 @@ LIB_PATH = Path(__file__).resolve().parent / "libnkipy_b200_kernels.so"
 
 _lib = None
 _initialised = False
+_subset = False
 
 _P = c_void_p
+
+
+class ProjArg(ctypes.Structure):
+    """One slice of a projection's result (csrc/kernels/proj_src.h)."""
+    _fields_ = [("ptr", c_void_p), ("ld", c_longlong), ("split_stride", c_longlong), ("splits", c_int), ("bf16", c_int)]
+
+
+class MapsArg(ctypes.Structure):
+    """Sizes and constants of attention with several score maps (csrc/kernels/attn_maps.h)."""
+    _fields_ = [(n, c_int) for n in ("maps", "heads", "kv_heads", "dim", "dim_p", "vdim", "vdim_p")] + \
+               [(n, c_float) for n in ("scale", "softcap", "lam", "out_scale", "eps")]
+
+
+_PP = ctypes.POINTER(ProjArg)
+_PM = ctypes.POINTER(MapsArg)
 _SIGNATURES = {
     "nkb_init": (c_int, []),
     "nkb_status": (c_int, [c_int]),
@@ -26,10 +42,26 @@ _SIGNATURES = {
     "nkb_gemm_bf16": (
         c_int,
         [_P, _P, _P, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_int, c_int, c_int, c_longlong,
-         c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, _P],
+         c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P],
     ),
     "nkb_gemm_bf16_2cta": (c_int, [_P, _P, _P, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, _P, _P, c_int,
-                                   c_int, _P]),
+                                   c_int, c_int, _P]),
+    "nkb_gemm_simt": (c_int, [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong,
+                              _P]),
+    "nkb_gated_residual": (c_int, [_P, _P, _P, c_int, c_int, c_float, c_int, _PP, _PP, ctypes.POINTER(_P), _P, _P, _P,
+                                   c_int, ctypes.POINTER(_P), ctypes.POINTER(_P), c_int, c_int, c_int, c_int, c_float,
+                                   _P]),
+    "nkb_gated_act": (c_int, [_PP, _PP, _P, c_int, c_int, c_int, c_int, _P]),
+    "nkb_hgrn2_scan": (c_int, [_PP, _PP, _PP, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
+                               _P, c_float, _P]),
+    "nkb_hgrn2_step": (c_int, [_PP, _PP, _PP, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, c_float,
+                               _P]),
+    "nkb_maps_append": (c_int, [_PM, _PP, _PP, _PP, _P, c_int, c_int, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P]),
+    "nkb_maps_attn_simple": (c_int, [_PM, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P]),
+    "nkb_maps_decode_scratch_floats": (c_longlong, [_PM, c_int, c_int]),
+    "nkb_maps_attn_decode": (c_int, [_PM, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P]),
+    "nkb_maps_attn_prefill": (c_int, [_PM, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
+                                      _P]),
     "nkb_gemm_bf16_grouped": (
         c_int,
         [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_int, c_int, _P, c_longlong,
@@ -105,12 +137,25 @@ def available() -> bool:
     return LIB_PATH.exists()
 
 
+def use_serving_subset() -> None:
+    """For a process that only serves a single-GPU decoder: when the library has to be built first, build and load
+    only the kernels such a model launches (`_build.SERVING_SOURCES`).  A library that is up to date is used as is."""
+    global _subset
+    _subset = True
+
+
 def lib():
     """Load the shared library (once) and declare its signatures."""
     global _lib
     if _lib is not None:
         return _lib
     from . import _build
+
+    if _subset and _build.is_stale():
+        try:
+            return _declare(_build.build_subset())
+        except RuntimeError as e:
+            raise KernelLibraryError(f"the serving kernels could not be built: {e}")
 
     # The signatures below are declared from the sources in the tree, so the binary must have been built
     # from exactly those sources: a stale library would be handed shifted arguments.
@@ -125,7 +170,12 @@ def lib():
                 f"{LIB_PATH} is missing or was built from other sources than csrc/kernels: "
                 "run `python -m nkipy_b200.ops._build` (needs nvcc) first"
             )
-    handle = ctypes.CDLL(str(LIB_PATH))
+    return _declare(LIB_PATH)
+
+
+def _declare(path):
+    global _lib
+    handle = ctypes.CDLL(str(path))
     for name, (res, args) in _SIGNATURES.items():
         try:
             fn = getattr(handle, name)

@@ -1,0 +1,351 @@
+"""Operators of decoders whose layers mix attention and linear recurrences around an fp32 residual stream.
+
+    gated_residual   embedding or residual + gated branches (+ additions ahead of a repeated block), and the
+                     group-wise RMS norms of the sum, in one launch
+    gated_act        act(gate) * up
+    hgrn2            linear attention with a per-channel forget gate; state in slots, fp32
+    maps_append      interleaved partial RoPE of queries / keys with several score maps, paged-cache append
+    maps_attention   attention with several score maps over shared values (differential attention), score soft cap
+    linear_simt      products on the CUDA cores: 32-bit models, operands TMA cannot describe
+
+All of them take the projections they consume as `Proj` slices, so a decode-sized batch hands over split-K partial
+sums and a prefill-sized one finished bf16 without a copy in between.  CUDA tensors run the kernels of
+csrc/kernels/{gated_residual,recurrent,attn_maps,attn_maps_prefill,gemm_simt}.cu; CPU tensors run the PyTorch
+statement of the same op.
+"""
+
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+from typing import List, NamedTuple, Optional, Sequence, Tuple
+
+import torch
+import torch.nn.functional as F
+
+from . import _lib
+from . import _count_launch, _decode_scratch, _gather_kv, _native, _ptr, _stream, pick_kv_splits
+
+# name -> (kernel code, PyTorch function)
+ACTIVATIONS = {"silu": (0, F.silu), "gelu_tanh": (1, lambda z: F.gelu(z, approximate="tanh"))}
+
+
+class Proj(NamedTuple):
+    """Columns [col, col + width) of a projection's result: fp32 split-K partials [S, T, N], or bf16 / fp32 [T, N]."""
+    t: torch.Tensor
+    col: int
+    width: int
+
+    def value(self) -> torch.Tensor:
+        """The finished slice in fp32, [T, width]."""
+        x = self.t[..., self.col:self.col + self.width].float()
+        return x.sum(0) if x.dim() == 3 else x
+
+    def arg(self) -> _lib.ProjArg:
+        t = self.t
+        if t.stride(-1) != 1 or t.dtype not in (torch.float32, torch.bfloat16):
+            raise ValueError("a projection slice needs unit column stride and fp32 or bf16 values")
+        split = t.dim() == 3
+        return _lib.ProjArg(t.data_ptr() + self.col * t.element_size(), t.stride(-2), t.stride(0) if split else 0,
+                            t.shape[0] if split else 1, 1 if t.dtype == torch.bfloat16 else 0)
+
+
+def _ref(p: Proj):
+    return ctypes.byref(p.arg())
+
+
+def _ptr_array(ts: Sequence[Optional[torch.Tensor]]):
+    return (ctypes.c_void_p * max(len(ts), 1))(*[_ptr(t) for t in ts])
+
+
+def linear_simt(x: torch.Tensor, w: torch.Tensor, *, gated: bool = False, act: str = "silu",
+                fp32_out: bool = False) -> torch.Tensor:
+    """``x @ w.T`` with fp32 accumulation on the CUDA cores; x and w both fp32 or both bf16."""
+    M, K = x.shape
+    N = w.shape[0]
+    f32 = x.dtype == torch.float32
+    if x.dtype != w.dtype:
+        raise TypeError(f"operands of different types: {x.dtype} and {w.dtype}")
+    out = torch.empty((M, N), dtype=torch.float32 if f32 or fp32_out or gated else torch.bfloat16, device=x.device)
+    rc = _lib.lib().nkb_gemm_simt(x.data_ptr(), 0 if f32 else 1, w.data_ptr(), 0 if f32 else 1, out.data_ptr(),
+                                  0 if out.dtype == torch.float32 else 1, M, N, K, x.stride(0), w.stride(0), N, _stream())
+    _lib.check(rc, "nkb_gemm_simt")
+    _count_launch()
+    if gated:
+        return gated_act(Proj(out, 0, N // 2), Proj(out, N // 2, N // 2), act, dtype=x.dtype)
+    return out
+
+
+def group_rmsnorm_ref(x: torch.Tensor, w: torch.Tensor, groups: int, eps: float) -> torch.Tensor:
+    y = x.float().reshape(*x.shape[:-1], groups, x.shape[-1] // groups)
+    y = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps)
+    return y.reshape(x.shape) * w.float()
+
+
+def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Tuple[Proj, Proj, torch.Tensor]] = (), *,
+                   ids: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None, scale: float = 1.0,
+                   add_mat: Optional[torch.Tensor] = None, add_row: Optional[torch.Tensor] = None,
+                   norms: Sequence[torch.Tensor] = (), groups: int = 1, eps: float = 1e-6,
+                   dtype: torch.dtype = torch.bfloat16) -> Tuple[torch.Tensor, List[torch.Tensor]]:
+    """One residual update of an fp32 stream and the norms that read it.
+
+        r = x  (or table[ids] * scale)
+        r += sum over branches (y, g, b) of sigmoid(g + b) * y;   r += add_mat;   r += add_row
+        h_j = w_j * (r divided, in `groups` equal parts, by sqrt(mean(part^2) + eps))
+
+    x [T, W] fp32; b, add_row and the norm weights fp32 [W]; add_mat fp32 [T, W].  Returns (r, [h_j in `dtype`])."""
+    if x is not None:
+        rows, width = x.shape
+        dev = x.device
+    else:
+        rows, width = ids.numel(), table.shape[1]
+        dev = table.device
+    r = torch.empty((rows, width), dtype=torch.float32, device=dev)
+    outs = [torch.empty((rows, width), dtype=dtype, device=dev) for _ in norms]
+    if not _native(r):
+        acc = x.clone() if x is not None else table[ids.long().clamp(0, table.shape[0] - 1)].float() * scale
+        if branches:
+            acc = acc + sum(y.value() * torch.sigmoid(g.value() + b) for y, g, b in branches)
+        if add_mat is not None:
+            acc = acc + add_mat
+        if add_row is not None:
+            acc = acc + add_row
+        r.copy_(acc)
+        for o, w in zip(outs, norms):
+            o.copy_(group_rmsnorm_ref(acc, w, groups, eps).to(dtype))
+        return r, outs
+    for t in [x, add_mat, add_row, *norms, *[b for _, _, b in branches]]:
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
+            raise TypeError("gated_residual wants contiguous fp32 residuals, biases and norm weights")
+    n = len(branches)
+    ya = (_lib.ProjArg * 2)(*[y.arg() for y, _, _ in branches])
+    ga = (_lib.ProjArg * 2)(*[g.arg() for _, g, _ in branches])
+    rc = _lib.lib().nkb_gated_residual(
+        _ptr(x), _ptr(ids), _ptr(table), 1 if table is not None and table.dtype == torch.bfloat16 else 0,
+        table.shape[0] if table is not None else 0, float(scale), n, ya, ga, _ptr_array([b for _, _, b in branches]),
+        _ptr(add_row), _ptr(add_mat), r.data_ptr(), len(outs), _ptr_array(list(norms)), _ptr_array(outs),
+        1 if dtype == torch.bfloat16 else 0, rows, width, int(groups), float(eps), _stream())
+    _lib.check(rc, "nkb_gated_residual")
+    _count_launch()
+    return r, outs
+
+
+def gated_act(gate: Proj, up: Proj, act: str = "silu", dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
+    """``act(gate) * up`` -> [T, width] in `dtype`."""
+    rows = gate.t.shape[-2]
+    out = torch.empty((rows, gate.width), dtype=dtype, device=gate.t.device)
+    if not _native(out):
+        out.copy_((ACTIVATIONS[act][1](gate.value()) * up.value()).to(dtype))
+        return out
+    rc = _lib.lib().nkb_gated_act(_ref(gate), _ref(up), out.data_ptr(), 1 if dtype == torch.bfloat16 else 0, rows,
+                                  gate.width, ACTIVATIONS[act][0], _stream())
+    _lib.check(rc, "nkb_gated_act")
+    _count_launch()
+    return out
+
+
+# --------------------------------------------------------------------------- linear recurrence
+def hgrn2_state_shape(heads: int, dim: int, vdim: int) -> Tuple[int, int, int]:
+    """State of one sequence: [heads, vdim, dim rounded up to whole 16-byte pieces]."""
+    return heads, vdim, (dim + 3) // 4 * 4
+
+
+def hgrn2(q: Proj, f: Proj, v: Proj, f_bias: torch.Tensor, lower: torch.Tensor, norm_w: torch.Tensor,
+          state: torch.Tensor, context_lens: torch.Tensor, *, heads: int, dim: int, vdim: int, eps: float,
+          q_start: Optional[torch.Tensor] = None, q_lens: Optional[torch.Tensor] = None,
+          rows: Optional[torch.Tensor] = None, dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
+    """Gated linear recurrence over the new tokens of every sequence; returns the normed heads [T, heads * vdim].
+
+        f = lower + (1 - lower) sigmoid(f + f_bias);   S <- diag(f) S + (1 - f) v^T;   o = S^T silu(q)
+        o <- norm_w * o / sqrt(mean(o^2) + eps)   per head
+
+    state [slots, heads, vdim, dim_p] fp32 is read and written in place at slot rows[b] (rows None: b).
+    context_lens counts the new tokens; a sequence whose tokens are all new starts from a zero state, one with a
+    negative length is skipped.  q_lens None: one new token per sequence (a decode step)."""
+    T = q.t.shape[-2]
+    out = torch.empty((T, heads * vdim), dtype=dtype, device=state.device)
+    if not _native(state):
+        qa = F.silu(q.value()).reshape(T, heads, dim)
+        low = lower.float()
+        fa = (low + (1 - low) * torch.sigmoid(f.value() + f_bias.float())).reshape(T, heads, dim)
+        va = v.value().reshape(T, heads, vdim)
+        o = torch.zeros((T, heads, vdim))
+        for b in range(context_lens.shape[0]):
+            n = 1 if q_lens is None else int(q_lens[b])
+            t0 = b if q_lens is None else int(q_start[b])
+            ctx, slot = int(context_lens[b]), b if rows is None else int(rows[b])
+            if n <= 0 or ctx < n:
+                continue
+            S = torch.zeros((heads, vdim, dim)) if ctx == n else state[slot, :, :, :dim].clone()
+            for t in range(t0, t0 + n):
+                ft, vt = fa[t][:, None, :], va[t][:, :, None]
+                S = ft * (S - vt) + vt
+                o[t] = torch.einsum("hvd,hd->hv", S, qa[t])
+            state[slot, :, :, :dim] = S
+        if q_lens is not None and dtype == torch.bfloat16:
+            o = o.to(dtype).float()
+        o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float()
+        out.copy_(o.reshape(T, heads * vdim).to(dtype))
+        return out
+    if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != hgrn2_state_shape(
+            heads, dim, vdim):
+        raise ValueError("state must be contiguous fp32 [slots, heads, vdim, dim_p]")
+    for t in (f_bias, lower, norm_w):
+        if t.dtype != torch.float32 or not t.is_contiguous():
+            raise TypeError("hgrn2 wants fp32 gate bias, lower bound and norm weight")
+    L, bf = _lib.lib(), 1 if dtype == torch.bfloat16 else 0
+    B = context_lens.shape[0]
+    if q_lens is None:
+        if T != B:
+            raise ValueError("a step has one token per sequence")
+        rc = L.nkb_hgrn2_step(_ref(q), _ref(f), _ref(v), f_bias.data_ptr(), lower.data_ptr(), state.data_ptr(),
+                              _ptr(rows), context_lens.data_ptr(), out.data_ptr(), bf, B, heads, dim, vdim,
+                              norm_w.data_ptr(), float(eps), _stream())
+        _lib.check(rc, "nkb_hgrn2_step")
+        _count_launch()
+        return out
+    rc = L.nkb_hgrn2_scan(_ref(q), _ref(f), _ref(v), f_bias.data_ptr(), lower.data_ptr(), state.data_ptr(), _ptr(rows),
+                          q_start.data_ptr(), q_lens.data_ptr(), context_lens.data_ptr(), out.data_ptr(), bf, B, T,
+                          heads, dim, vdim, norm_w.data_ptr(), float(eps), _stream())
+    _lib.check(rc, "nkb_hgrn2_scan")
+    _count_launch(2)
+    return out
+
+
+# --------------------------------------------------------------------------- attention with score maps
+def _tiled(n: int, sizes: Sequence[int]) -> int:
+    for s in sizes:
+        if n <= s:
+            return s
+    return (n + 1) // 2 * 2
+
+
+@dataclass
+class MapsSpec:
+    """Sizes and constants of attention with `maps` score maps per head over shared values.  Two maps are combined as
+    ``a0 - lam * a1``, root-mean-square normed over the head and multiplied by `out_scale`; softcap <= 0: none.
+    dim_p / vdim_p are the padded sizes of queries / keys (per map) and values in the cache; the tiled bf16 kernels
+    take 32 or 64 and 64 or 128, other sizes are only rounded to even and use the general kernel."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    maps: int = 1
+    softcap: float = 0.0
+    lam: float = 0.0
+    out_scale: float = 1.0
+    eps: float = 1e-6
+    tiled: bool = True
+
+    @property
+    def dim_p(self) -> int:
+        return _tiled(self.dim, (32, 64) if self.tiled else ())
+
+    @property
+    def vdim_p(self) -> int:
+        return _tiled(self.vdim, (64, 128) if self.tiled else ())
+
+    def arg(self) -> _lib.MapsArg:
+        return _lib.MapsArg(self.maps, self.heads, self.kv_heads, self.dim, self.dim_p, self.vdim, self.vdim_p,
+                            float(self.scale), float(self.softcap), float(self.lam), float(self.out_scale),
+                            float(self.eps))
+
+
+def maps_append(spec: MapsSpec, q: Proj, k: Proj, v: Proj, cos_sin: torch.Tensor, positions: torch.Tensor,
+                slots: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor) -> torch.Tensor:
+    """Rotate queries and keys (pairs (2i, 2i + 1) of the first cos_sin.shape[1] dimensions of every map), write keys
+    and values to their cache slots (negative slot: not stored), return the queries [T, heads, maps * dim_p]."""
+    T = q.t.shape[-2]
+    H, G, M, d, dp = spec.heads, spec.kv_heads, spec.maps, spec.dim, spec.dim_p
+    bs = k_cache.shape[2]
+    q_out = torch.empty((T, H, M * dp), dtype=k_cache.dtype, device=k_cache.device)
+    rd = cos_sin.shape[1]
+    if not _native(k_cache):
+        cs = cos_sin[positions.long().clamp(0, cos_sin.shape[0] - 1)]
+        c, s = cs[:, None, None, :rd // 2], cs[:, None, None, rd // 2:]
+
+        def rot(x, n):
+            x = F.pad(x.reshape(T, n, M, d), (0, dp - d))
+            u, w = x[..., 0:rd:2].clone(), x[..., 1:rd:2].clone()
+            x[..., 0:rd:2] = u * c - w * s
+            x[..., 1:rd:2] = w * c + u * s
+            return x.reshape(T, n, M * dp).to(k_cache.dtype)
+
+        q_out.copy_(rot(q.value(), H))
+        sl = slots.long()
+        keep = sl >= 0
+        blk, off = sl[keep] // bs, sl[keep] % bs
+        k_cache[blk, :, off] = rot(k.value(), G)[keep]
+        v_cache[blk, :, off] = F.pad(v.value().reshape(T, G, spec.vdim), (0, spec.vdim_p - spec.vdim))[keep].to(v_cache.dtype)
+        return q_out
+    a = spec.arg()
+    rc = _lib.lib().nkb_maps_append(ctypes.byref(a), _ref(q), _ref(k), _ref(v), cos_sin.data_ptr(), rd, cos_sin.shape[0],
+                                    positions.data_ptr(), slots.data_ptr(), q_out.data_ptr(), k_cache.data_ptr(),
+                                    v_cache.data_ptr(), 1 if k_cache.dtype == torch.bfloat16 else 0, T, bs, _stream())
+    _lib.check(rc, "nkb_maps_append")
+    _count_launch()
+    return q_out
+
+
+def maps_attention(spec: MapsSpec, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                   block_table: torch.Tensor, context_lens: torch.Tensor, *, q_start: Optional[torch.Tensor] = None,
+                   q_lens: Optional[torch.Tensor] = None, max_q_len: int = 1, num_splits: int = 0) -> torch.Tensor:
+    """Causal attention of the new tokens over the paged cache (which already holds them); returns the combined heads
+    [T, heads * vdim].  q_lens None: one new token per sequence (decode); otherwise sequence b owns rows
+    q_start[b] .. q_start[b] + q_lens[b], the last of which sits at position context_lens[b] - 1."""
+    T, H = q.shape[0], spec.heads
+    bs = k_cache.shape[2]
+    B = block_table.shape[0]
+    out = torch.empty((T, H * spec.vdim), dtype=k_cache.dtype, device=k_cache.device)
+    if not _native(k_cache):
+        M, dp = spec.maps, spec.dim_p
+        res = torch.zeros((T, H, spec.vdim))
+        rep = H // spec.kv_heads
+        for b in range(B):
+            n = 1 if q_lens is None else int(q_lens[b])
+            t0 = b if q_lens is None else int(q_start[b])
+            ctx = int(context_lens[b])
+            if n <= 0 or ctx < n:
+                continue
+            k = _gather_kv(k_cache, block_table[b], ctx).float().reshape(ctx, spec.kv_heads, M, dp)
+            v = _gather_kv(v_cache, block_table[b], ctx).float()[..., :spec.vdim]
+            k, v = k.repeat_interleave(rep, 1), v.repeat_interleave(rep, 1)
+            s = torch.einsum("qhmd,khmd->hmqk", q[t0:t0 + n].float().reshape(n, H, M, dp), k) * spec.scale
+            if spec.softcap > 0:
+                s = spec.softcap * torch.tanh(s / spec.softcap)
+            vis = torch.arange(ctx)[None, :] <= (ctx - n + torch.arange(n))[:, None]
+            a = torch.einsum("hmqk,khv->qhmv", s.masked_fill(~vis, float("-inf")).softmax(-1), v)
+            o = a[:, :, 0]
+            if M == 2:
+                o = o - spec.lam * a[:, :, 1]
+                o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + spec.eps) * spec.out_scale
+            res[t0:t0 + n] = o
+        out.copy_(res.reshape(T, -1).to(out.dtype))
+        return out
+    L, a = _lib.lib(), spec.arg()
+    ref = ctypes.byref(a)
+    bf = k_cache.dtype == torch.bfloat16
+    common = (q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr())
+    rc = -5
+    if bf and q_lens is None:
+        group = H // spec.kv_heads
+        if num_splits <= 0:
+            num_splits = pick_kv_splits(B * spec.kv_heads * ((group + 7) // 8), block_table.shape[1])
+        need = L.nkb_maps_decode_scratch_floats(ref, B, num_splits)
+        scratch = _decode_scratch(q.device, need) if need else None
+        rc = L.nkb_maps_attn_decode(ref, *common, context_lens.data_ptr(), out.data_ptr(), _ptr(scratch), B, bs,
+                                    k_cache.shape[0], block_table.stride(0), num_splits, _stream())
+    elif bf:
+        rc = L.nkb_maps_attn_prefill(ref, *common, q_start.data_ptr(), q_lens.data_ptr(), context_lens.data_ptr(),
+                                     out.data_ptr(), B, T, int(max_q_len), bs, k_cache.shape[0], block_table.stride(0),
+                                     _stream())
+    if rc == -5:
+        if q_lens is None:
+            q_start = torch.arange(B, dtype=torch.int32, device=q.device)
+            q_lens = torch.ones((B,), dtype=torch.int32, device=q.device)
+        rc = L.nkb_maps_attn_simple(ref, *common, q_start.data_ptr(), q_lens.data_ptr(), context_lens.data_ptr(),
+                                    out.data_ptr(), 1 if bf else 0, B, T, bs, block_table.stride(0), _stream())
+    _lib.check(rc, "maps_attention")
+    _count_launch()
+    return out
