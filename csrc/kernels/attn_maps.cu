@@ -29,7 +29,16 @@ struct MapsAppendParams {
   const int* slots;
   void *q_out, *k_cache, *v_cache;
   int rot_dims, max_pos, tokens;
+  int vec;                  // sizes and alignments allow four elements at a time
 };
+
+template <typename T>
+__device__ __forceinline__ void store4(T* dst, float4 x) {
+  if constexpr (sizeof(T) == 2)
+    *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(x.x, x.y), pack_bf16x2(x.z, x.w));
+  else
+    *reinterpret_cast<float4*>(dst) = x;
+}
 
 template <typename T>
 __global__ void __launch_bounds__(256) maps_append_kernel(const __grid_constant__ MapsAppendParams p) {
@@ -39,8 +48,7 @@ __global__ void __launch_bounds__(256) maps_append_kernel(const __grid_constant_
   griddep_wait();
   griddep_launch();
   if (gw >= (long long)p.tokens * units) return;
-  const long long t = gw / units;
-  const int u = int(gw % units);
+  const int t = int(unsigned(gw) / unsigned(units)), u = int(unsigned(gw) % unsigned(units));
   const bool is_q = u < p.a.heads, is_v = u >= p.a.heads + p.a.kv_heads;
   const int slot = p.slots[t];
   if (!is_q && slot < 0) return;
@@ -48,16 +56,35 @@ __global__ void __launch_bounds__(256) maps_append_kernel(const __grid_constant_
   if (is_v) {
     const int h = u - p.a.heads - p.a.kv_heads;
     T* dst = reinterpret_cast<T*>(p.v_cache) + ((blk * p.a.kv_heads + h) * kMapsPage + off) * p.a.vdim_p;
+    if (p.vec) {
+      for (int c = lane * 4; c < p.a.vdim; c += 128) store4<T>(dst + c, proj_load4(p.v, t, h * p.a.vdim + c));
+      return;
+    }
     for (int c = lane; c < p.a.vdim; c += 32) dst[c] = cast_out<T>(proj_load(p.v, t, h * p.a.vdim + c));
     return;
   }
   const int h = is_q ? u : u - p.a.heads;
   const int kw = p.a.maps * p.a.dim_p;
-  T* dst = is_q ? reinterpret_cast<T*>(p.q_out) + (t * p.a.heads + h) * kw
+  T* dst = is_q ? reinterpret_cast<T*>(p.q_out) + ((long long)t * p.a.heads + h) * kw
                 : reinterpret_cast<T*>(p.k_cache) + ((blk * p.a.kv_heads + h) * kMapsPage + off) * kw;
   const NkbProj& src = is_q ? p.q : p.k;
   const int pos = min(max(p.positions[t], 0), p.max_pos - 1);
   const float* cs = p.cos_sin + (long long)pos * p.rot_dims;
+  const int quarter = p.a.dim_p / 4;
+  if (p.vec) {
+    // four consecutive elements (two pairs) per lane
+    for (int i = lane; i < p.a.maps * quarter; i += 32) {
+      const int m = i / quarter, c = (i % quarter) * 4;
+      float4 x = c < p.a.dim ? proj_load4(src, t, (h * p.a.maps + m) * p.a.dim + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < p.rot_dims) {
+        const float2 co = *reinterpret_cast<const float2*>(cs + (c >> 1));
+        const float2 si = *reinterpret_cast<const float2*>(cs + (p.rot_dims >> 1) + (c >> 1));
+        x = make_float4(x.x * co.x - x.y * si.x, x.y * co.x + x.x * si.x, x.z * co.y - x.w * si.y, x.w * co.y + x.z * si.y);
+      }
+      store4<T>(dst + m * p.a.dim_p + c, x);
+    }
+    return;
+  }
   const int half = p.a.dim_p / 2;
   for (int i = lane; i < p.a.maps * half; i += 32) {
     const int m = i / half, c = (i % half) * 2;         // pair (c, c + 1) of map m
@@ -526,7 +553,11 @@ extern "C" int nkb_maps_append(const NkbMapsArgs* a, const NkbProj* q, const Nkb
   p.cos_sin = cos_sin; p.positions = positions; p.slots = slots;
   p.q_out = q_out; p.k_cache = k_cache; p.v_cache = v_cache;
   p.rot_dims = rot_dims; p.max_pos = max_pos; p.tokens = tokens;
+  const auto al16 = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
+  p.vec = ((a->dim | a->dim_p | a->vdim | a->vdim_p | rot_dims) & 3) == 0 && proj_vec4_ok(*q) && proj_vec4_ok(*k) &&
+          proj_vec4_ok(*v) && al16(cos_sin) && al16(q_out) && al16(k_cache) && al16(v_cache);
   const long long warps = (long long)tokens * (a->heads + 2 * a->kv_heads);
+  if (warps > 0x7fffffffll) return -2;
   const dim3 grid(unsigned((warps + 7) / 8));
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return bf16 ? launch_pdl(maps_append_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, p)

@@ -37,14 +37,30 @@ struct GatedResidualParams {
 };
 
 template <int V>
-struct VecF {
-  float v[V];
-};
+__device__ __forceinline__ void load_vec(float (&a)[V], const float* p) {
+  if constexpr (V == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    a[0] = x.x; a[1] = x.y; a[2] = x.z; a[3] = x.w;
+  } else {
+    a[0] = *p;
+  }
+}
+template <int V>
+__device__ __forceinline__ void proj_vec(float (&a)[V], const NkbProj& s, long long row, int c) {
+  if constexpr (V == 4) {
+    const float4 x = proj_load4(s, row, c);
+    a[0] = x.x; a[1] = x.y; a[2] = x.z; a[3] = x.w;
+  } else {
+    a[0] = proj_load(s, row, c);
+  }
+}
 
-template <int V, typename OutT>
-__global__ void __launch_bounds__(256) gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
+// PACKED: every projection is bf16 and aligned (prefill), which keeps the kernel at few registers and many CTAs per SM
+template <int V, bool PACKED, typename OutT>
+__global__ void __launch_bounds__(PACKED ? 256 : 1024, PACKED ? 6 : 1)
+gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
   extern __shared__ float row_s[];                 // [width] then [groups]
-  __shared__ float red[8];
+  __shared__ float red[32];
   float* inv_s = row_s + p.width;
   const long long t = blockIdx.x;
   const int nv = p.width / V;
@@ -54,14 +70,9 @@ __global__ void __launch_bounds__(256) gated_residual_kernel(const __grid_consta
   const int id = p.ids ? min(max(p.ids[t], 0), p.vocab - 1) : 0;
   for (int i = threadIdx.x; i < nv; i += blockDim.x) {
     const int c = i * V;
-    float a[V];
+    float a[V], s[V];
     if (p.x_in) {
-      if constexpr (V == 4) {
-        const float4 x = *reinterpret_cast<const float4*>(p.x_in + t * p.width + c);
-        a[0] = x.x; a[1] = x.y; a[2] = x.z; a[3] = x.w;
-      } else {
-        a[0] = p.x_in[t * p.width + c];
-      }
+      load_vec<V>(a, p.x_in + t * p.width + c);
     } else {
 #pragma unroll
       for (int j = 0; j < V; ++j) {
@@ -70,38 +81,56 @@ __global__ void __launch_bounds__(256) gated_residual_kernel(const __grid_consta
                                        : reinterpret_cast<const float*>(p.table)[o]);
       }
     }
-    float s[V];
 #pragma unroll
     for (int j = 0; j < V; ++j) s[j] = 0.f;
+    if constexpr (PACKED) {
+      uint2 y[2], g[2];
 #pragma unroll
-    for (int b = 0; b < 2; ++b) {
-      if (b < p.branches) {
-        float y[V], g[V];
-        if constexpr (V == 4) {
-          const float4 yy = proj_load4(p.y[b], t, c), gg = proj_load4(p.g[b], t, c);
-          const float4 bb = *reinterpret_cast<const float4*>(p.gbias[b] + c);
-          y[0] = yy.x; y[1] = yy.y; y[2] = yy.z; y[3] = yy.w;
-          g[0] = gg.x + bb.x; g[1] = gg.y + bb.y; g[2] = gg.z + bb.z; g[3] = gg.w + bb.w;
-        } else {
-          y[0] = proj_load(p.y[b], t, c);
-          g[0] = proj_load(p.g[b], t, c) + p.gbias[b][c];
+      for (int b = 0; b < 2; ++b)
+        if (b < p.branches) {
+          y[b] = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.y[b].ptr) + t * p.y[b].ld + c);
+          g[b] = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.g[b].ptr) + t * p.g[b].ld + c);
         }
 #pragma unroll
-        for (int j = 0; j < V; ++j) s[j] += y[j] * sigmoid_f(g[j]);
-      }
+      for (int b = 0; b < 2; ++b)
+        if (b < p.branches) {
+          const float4 bias = *reinterpret_cast<const float4*>(p.gbias[b] + c);
+          const float2 y0 = unpack_bf16x2(y[b].x), y1 = unpack_bf16x2(y[b].y);
+          const float2 g0 = unpack_bf16x2(g[b].x), g1 = unpack_bf16x2(g[b].y);
+          s[0] += y0.x * sigmoid_f(g0.x + bias.x);
+          s[1] += y0.y * sigmoid_f(g0.y + bias.y);
+          s[2] += y1.x * sigmoid_f(g1.x + bias.z);
+          s[3] += y1.y * sigmoid_f(g1.y + bias.w);
+        }
+    } else {
+      float y[2][V], g[2][V];
+#pragma unroll
+      for (int b = 0; b < 2; ++b)
+        if (b < p.branches) {
+          proj_vec<V>(y[b], p.y[b], t, c);
+          proj_vec<V>(g[b], p.g[b], t, c);
+        }
+#pragma unroll
+      for (int b = 0; b < 2; ++b)
+        if (b < p.branches) {
+          float bias[V];
+          load_vec<V>(bias, p.gbias[b] + c);
+#pragma unroll
+          for (int j = 0; j < V; ++j) s[j] += y[b][j] * sigmoid_f(g[b][j] + bias[j]);
+        }
     }
 #pragma unroll
     for (int j = 0; j < V; ++j) {
       a[j] += s[j];
       if (p.add_mat) a[j] += p.add_mat[t * p.width + c + j];
       if (p.add_row) a[j] += p.add_row[c + j];
-      row_s[c + j] = a[j];
     }
-    if (p.x_out) {
-      if constexpr (V == 4)
-        *reinterpret_cast<float4*>(p.x_out + t * p.width + c) = make_float4(a[0], a[1], a[2], a[3]);
-      else
-        p.x_out[t * p.width + c] = a[0];
+    if constexpr (V == 4) {
+      *reinterpret_cast<float4*>(row_s + c) = make_float4(a[0], a[1], a[2], a[3]);
+      if (p.x_out) *reinterpret_cast<float4*>(p.x_out + t * p.width + c) = make_float4(a[0], a[1], a[2], a[3]);
+    } else {
+      row_s[c] = a[0];
+      if (p.x_out) p.x_out[t * p.width + c] = a[0];
     }
   }
   if (p.norms == 0) return;
@@ -140,8 +169,9 @@ __global__ void __launch_bounds__(256) gated_residual_kernel(const __grid_consta
     const int c = i * V;
     const float inv = inv_s[c / gsz];              // V > 1 only when a group is a multiple of V
     float a[V];
+    load_vec<V>(a, row_s + c);
 #pragma unroll
-    for (int j = 0; j < V; ++j) a[j] = row_s[c + j] * inv;
+    for (int j = 0; j < V; ++j) a[j] *= inv;
 #pragma unroll
     for (int n = 0; n < 2; ++n) {
       if (n < p.norms) {
@@ -225,14 +255,23 @@ extern "C" int nkb_gated_residual(const float* x_in, const int* ids, const void*
   p.add_row = add_row; p.add_mat = add_mat; p.x_out = x_out;
   p.width = width; p.groups = groups; p.eps = eps;
   const size_t smem = size_t(width + groups) * sizeof(float);
-  const int threads = (vec ? width / 4 : width) > 128 ? 256 : 128;
+  bool packed = vec && branches > 0;
+  for (int i = 0; i < branches; ++i) packed = packed && y[i].bf16 && g[i].bf16;
+  // few rows: one vector per thread, so that every load of a row is in flight at once
+  const int nv = vec ? width / 4 : width, most = packed || rows > 2 * 148 ? 256 : 1024;
+  const int threads = nv >= most ? most : (nv < 64 ? 64 : (nv + 31) / 32 * 32);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (smem > 48 * 1024) return -2;
+  using bf = __nv_bfloat16;
+  const dim3 grid(rows), block(threads);
+  if (packed)
+    return out_bf16 ? launch_pdl(gated_residual_kernel<4, true, bf>, grid, block, smem, s, p)
+                    : launch_pdl(gated_residual_kernel<4, true, float>, grid, block, smem, s, p);
   if (vec)
-    return out_bf16 ? launch_pdl(gated_residual_kernel<4, __nv_bfloat16>, dim3(rows), dim3(threads), smem, s, p)
-                    : launch_pdl(gated_residual_kernel<4, float>, dim3(rows), dim3(threads), smem, s, p);
-  return out_bf16 ? launch_pdl(gated_residual_kernel<1, __nv_bfloat16>, dim3(rows), dim3(threads), smem, s, p)
-                  : launch_pdl(gated_residual_kernel<1, float>, dim3(rows), dim3(threads), smem, s, p);
+    return out_bf16 ? launch_pdl(gated_residual_kernel<4, false, bf>, grid, block, smem, s, p)
+                    : launch_pdl(gated_residual_kernel<4, false, float>, grid, block, smem, s, p);
+  return out_bf16 ? launch_pdl(gated_residual_kernel<1, false, bf>, grid, block, smem, s, p)
+                  : launch_pdl(gated_residual_kernel<1, false, float>, grid, block, smem, s, p);
 }
 
 extern "C" int nkb_gated_act(const NkbProj* gate, const NkbProj* up, void* out, int out_bf16, int rows, int inter,

@@ -32,7 +32,8 @@ static inline bool proj_vec4_ok(const NkbProj& s) {
   const uintptr_t a = reinterpret_cast<uintptr_t>(s.ptr);
   return (a & (s.bf16 ? 7 : 15)) == 0 && (s.ld & 3) == 0 && (s.split_stride & 3) == 0;
 }
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+// the reciprocal is the approximate one (two units in the last place): an IEEE division costs more than the exponential
+__device__ __forceinline__ float sigmoid_f(float z) { return __fdividef(1.f, 1.f + expf(-z)); }
 
 template <typename T>
 __device__ __forceinline__ T cast_out(float v);

@@ -62,7 +62,7 @@ class _TimedLib:
 
     _LAUNCHERS = ("nkb_gemm", "nkb_tp_", "nkb_moe", "nkb_argmax", "nkb_rmsnorm", "nkb_add_rmsnorm", "nkb_silu",
                   "nkb_embedding", "nkb_rope", "nkb_decode_advance", "nkb_sample", "nkb_router", "nkb_paged_attn_decode",
-                  "nkb_flash", "nkb_ag_gemm", "nkb_decode_gemm", "nkb_lmhead")
+                  "nkb_flash", "nkb_ag_gemm", "nkb_decode_gemm", "nkb_lmhead", "nkb_gated", "nkb_hgrn2", "nkb_maps")
 
     def __init__(self, real):
         object.__setattr__(self, "_real", real)
@@ -84,7 +84,8 @@ class _TimedLib:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--model", default="llama3-8b", choices=["llama3-8b", "qwen3-30b-a3b"])
+    ap.add_argument("--model", default="llama3-8b", choices=["llama3-8b", "qwen3-30b-a3b", "tolenex"])
+    ap.add_argument("--prefill", action="store_true", help="time one packed prefill of the batch instead of a decode step")
     ap.add_argument("--shard-of", type=int, default=1, help="run the per-rank shard of an N-way TP model on one GPU")
     ap.add_argument("--layers", type=int, default=None)
     ap.add_argument("--batch", type=int, default=None)
@@ -98,8 +99,7 @@ def main(argv=None) -> int:
     from ..parallel.comm import TPGroup
     from . import config as C
     from .engine import GenerationEngine
-    from .transformer import TransformerLM
-    from .weights import random_weights
+    from . import registry
 
     tp = TPGroup.from_env()
     dev = tp.device
@@ -107,10 +107,13 @@ def main(argv=None) -> int:
     proxy = _TimedLib(_lib.lib())
     _lib._lib = proxy
 
-    cfg = C.llama3_8b() if args.model == "llama3-8b" else C.qwen3_30b_a3b()
-    batch = args.batch or (64 if args.model == "llama3-8b" else 128)
-    prompt_len = args.prompt_len or (1024 if args.model == "llama3-8b" else 512)
-    if args.layers:
+    moe = args.model == "qwen3-30b-a3b"
+    cfg = C.qwen3_30b_a3b() if moe else C.llama3_8b()
+    if args.model == "tolenex":
+        cfg = C.tolenex_shape(4096, layers=args.layers or 32, heads=32, kv_heads=8, ff=14336)
+    batch = args.batch or (128 if moe else 64)
+    prompt_len = args.prompt_len or (512 if moe else 1024)
+    if args.layers and cfg.layers is None:
         cfg = cfg.scaled(num_layers=args.layers)
     n = args.shard_of
     if n > 1:
@@ -118,29 +121,41 @@ def main(argv=None) -> int:
             raise SystemExit("--shard-of is a single-GPU mode")
         cfg = cfg.shard_shapes(n)
     torch.manual_seed(0)
-    weights = random_weights(cfg, tp.rank, tp.world_size, device=dev, seed=0, std=0.02)
-    model = TransformerLM(cfg, weights, tp, device=dev, force_fused=n > 1)
+    arch = registry.for_config(cfg)
+    weights = arch.random(cfg, tp.rank, tp.world_size, dev, 0, "ep")
+    model = arch.model(cfg, weights, tp, device=dev, **(dict(force_fused=True) if n > 1 else {}))
     del weights
     eng = GenerationEngine(model, max_batch=batch, max_seq_len=prompt_len + 64 + 8 * args.steps,
                            use_cuda_graph=False)
     g = torch.Generator().manual_seed(0)
     seqs = eng.add_requests(torch.randint(0, cfg.vocab_size, (batch, prompt_len), generator=g).tolist())
     eng.prefill(seqs)
-    eng.prepare_decode(32 + 8 * args.steps)
-    for _ in range(3):
-        eng.decode_step_device()
-    eng.advance_host_state(3)
+    if args.prefill:
+        args.steps = 1
+        eng.release(seqs)
+        seqs = eng.add_requests(torch.randint(0, cfg.vocab_size, (batch, prompt_len), generator=g).tolist())
+    else:
+        eng.prepare_decode(32 + 8 * args.steps)
+        for _ in range(3):
+            eng.decode_step_device()
+        eng.advance_host_state(3)
     torch.cuda.synchronize()
     tp.barrier()
     proxy.enabled = True
     per_step = []
     for _ in range(args.steps):
         proxy.records = []
-        eng.decode_step_device()
+        if args.prefill:
+            eng.prefill(seqs)
+        else:
+            eng.decode_step_device()
         torch.cuda.synchronize()
         per_step.append(proxy.records)
     proxy.enabled = False
-    eng.advance_host_state(args.steps)
+    if args.prefill:
+        eng.prepare_decode(32)
+    else:
+        eng.advance_host_state(args.steps)
     ops.raise_on_device_error()
 
     agg = collections.OrderedDict()
