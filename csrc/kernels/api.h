@@ -166,9 +166,10 @@ int nkb_gated_act(const NkbProj* gate, const NkbProj* up, void* out, int out_bf1
 int nkb_gemm_simt(const void* x, int x_bf16, const void* w, int w_bf16, void* out, int out_bf16, int m, int n, int k,
                   long long ldx, long long ldw, long long ldo, void* stream);
 // gated linear recurrence (recurrent.cu)
+long long nkb_hgrn2_scan_scratch(int heads, int dim, int vdim);
 int nkb_hgrn2_scan(const NkbProj* q, const NkbProj* f, const NkbProj* v, const float* f_bias, const float* lower,
                    float* state, const int* slot_ids, const int* q_start, const int* q_lens, const int* context_lens,
-                   void* out, int out_bf16, int batch, int tokens, int heads, int dim, int vdim, const float* norm_w,
+                   float* scratch, void* out, int out_bf16, int batch, int tokens, int heads, int dim, int vdim, const float* norm_w,
                    float eps, void* stream);
 int nkb_hgrn2_step(const NkbProj* q, const NkbProj* f, const NkbProj* v, const float* f_bias, const float* lower,
                    float* state, const int* slot_ids, const int* context_lens, void* out, int out_bf16, int batch,

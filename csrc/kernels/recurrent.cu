@@ -9,19 +9,19 @@
 // 16-byte pieces); a sequence whose first new token has position 0 starts from zero, whatever the slot held.
 //
 // Two kernels:
-//   scan   any number of new tokens per sequence.  A CTA owns some columns of one head of one sequence for all of its
+//   scan   any number of new tokens per sequence.  A kernel of its own turns the projections into fp32 queries, gates and
+//          value differences once per head.  A CTA then owns some columns of one head of one sequence for all of its
 //          tokens; sixteen lanes share a set of columns, each holding every sixteenth group of four channels of them in
-//          registers, so a token costs one packed subtract and two packed multiply-adds per two state elements, and the
-//          gates and queries read from shared memory serve all of a lane's columns.  Sixteen partial sums (tokens x
-//          columns) are exchanged together: a transposing butterfly of fifteen shuffles leaves each of the sixteen
-//          lanes with one finished value.  The next tile of tokens is fetched while the current one is multiplied.
+//          registers, so a token costs two packed multiply-adds per two state elements, and the gates and queries read from
+//          shared memory serve all of a lane's columns.  Sixteen partial sums (tokens x columns) are exchanged together: a
+//          transposing butterfly of fifteen shuffles leaves each of the sixteen lanes with one finished value.  The next
+//          tile of tokens is copied while the current one is multiplied.
 //   step   one new token per sequence (decode).  A CTA owns a head of a sequence, streams its state through
 //          registers once (the whole state of a 128 x 128 head is in flight at once), and applies the per-head
 //          norm of the result itself.
 #include "common.cuh"
 #include "proj_src.cuh"
 #include "api.h"
-#include <type_traits>
 
 namespace nkb {
 
@@ -40,24 +40,6 @@ struct RecurrentParams {
   int heads, dim, dim_p, vdim;
 };
 
-// four consecutive channels of a token as fetched: bf16 values stay packed until they are needed
-template <int V>
-struct RawGroup {
-  float4 v;
-  __device__ __forceinline__ void clear() { v = make_float4(0.f, 0.f, 0.f, 0.f); }
-  __device__ __forceinline__ float4 get() const { return v; }
-};
-constexpr int kPackedBf16 = 2;     // V of the packed form: aligned bf16 values
-template <>
-struct RawGroup<kPackedBf16> {
-  uint2 v;
-  __device__ __forceinline__ void clear() { v = make_uint2(0u, 0u); }
-  __device__ __forceinline__ float4 get() const {
-    const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y);
-    return make_float4(a.x, a.y, b.x, b.y);
-  }
-};
-
 template <int V>
 __device__ __forceinline__ float4 load_group(const NkbProj& s, long long row, int head_col, int c, int dim) {
   if constexpr (V == 4) return proj_load4(s, row, head_col + c);
@@ -68,13 +50,6 @@ __device__ __forceinline__ float4 load_group(const NkbProj& s, long long row, in
   if (c + 3 < dim) r.w = proj_load(s, row, head_col + c + 3);
   return r;
 }
-template <int V>
-__device__ __forceinline__ void fetch_group(RawGroup<V>& r, const NkbProj& s, long long row, int head_col, int c, int dim) {
-  if constexpr (V == kPackedBf16)
-    r.v = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(s.ptr) + row * s.ld + head_col + c);
-  else
-    r.v = load_group<V>(s, row, head_col, c, dim);
-}
 __device__ __forceinline__ float query_act(float u, bool on) { return on ? u * sigmoid_f(u) : 0.f; }
 __device__ __forceinline__ float forget_gate(float z, float bias, float lower, bool on) {
   return on ? lower + (1.f - lower) * sigmoid_f(z + bias) : 1.f;
@@ -82,27 +57,74 @@ __device__ __forceinline__ float forget_gate(float z, float bias, float lower, b
 
 constexpr int kScanThreads = 128;
 constexpr int kScanLanes = 16;     // lanes that share the columns of a half warp
-constexpr int kScanTokens = 8;     // tokens per tile
 
-__device__ __forceinline__ float2 fsub2(float2 a, float2 b) {
-  uint64_t rd;
-  asm("sub.f32x2 %0, %1, %2;" : "=l"(rd) : "l"(reinterpret_cast<uint64_t&>(a)), "l"(reinterpret_cast<uint64_t&>(b)));
-  return reinterpret_cast<float2&>(rd);
+// Per-token inputs of the scan in fp32, computed once per head instead of once per column slice:
+//   q_act [tokens, heads, dp], f_act [tokens, heads, dp]   silu(u) and the forget gate; channels past dim: 0 and 1
+//   dv    [tokens, heads, vp]                              v_t - v_(t+1), with v_(t+1) = 0 for a sequence's last new token
+template <int V>
+__global__ void __launch_bounds__(256)
+hgrn2_gates_kernel(const __grid_constant__ RecurrentParams p, float* __restrict__ q_act, float* __restrict__ f_act,
+                   float* __restrict__ dv, int dp, int vp, int batch) {
+  griddep_wait();
+  griddep_launch();
+  const long long t = blockIdx.x;
+  bool end = false;
+  for (int b = threadIdx.x; b < batch; b += blockDim.x) end = end || (t == (long long)p.q_start[b] + p.q_lens[b] - 1);
+  const bool last = __syncthreads_or(end) != 0 || blockIdx.x + 1 == gridDim.x;
+  const int gq = dp / 4, gv = vp / 4;
+  for (int i = threadIdx.x; i < p.heads * gq; i += blockDim.x) {
+    const int head = i / gq, c = (i % gq) * 4, hq = head * p.dim;
+    float4 u = make_float4(0.f, 0.f, 0.f, 0.f), z = u;
+    if (c < p.dim) {
+      u = load_group<V>(p.q, t, hq, c, p.dim);
+      z = load_group<V>(p.f, t, hq, c, p.dim);
+    }
+    const float uv[4] = {u.x, u.y, u.z, u.w}, zv[4] = {z.x, z.y, z.z, z.w};
+    float qo[4], fo[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const bool on = c + e < p.dim;
+      qo[e] = query_act(uv[e], on);
+      fo[e] = on ? forget_gate(zv[e], p.f_bias[hq + c + e], p.lower[hq + c + e], true) : 1.f;
+    }
+    const long long o = (t * p.heads + head) * dp + c;
+    *reinterpret_cast<float4*>(q_act + o) = make_float4(qo[0], qo[1], qo[2], qo[3]);
+    *reinterpret_cast<float4*>(f_act + o) = make_float4(fo[0], fo[1], fo[2], fo[3]);
+  }
+  for (int i = threadIdx.x; i < p.heads * gv; i += blockDim.x) {
+    const int head = i / gv, c = (i % gv) * 4, hv = head * p.vdim;
+    float4 x = load_group<V>(p.v, t, hv, c, p.vdim);
+    if (!last) {
+      const float4 y = load_group<V>(p.v, t + 1, hv, c, p.vdim);
+      x = make_float4(x.x - y.x, x.y - y.y, x.z - y.z, x.w - y.w);
+    }
+    *reinterpret_cast<float4*>(dv + (t * p.heads + head) * vp + c) = x;
+  }
 }
 
-// CL: channels per lane (dim <= 16 CL), NC: columns per lane
-template <int CL, int NC, int V, typename OutT>
+// 16 bytes global -> shared, zeros when `on` is false
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool on) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
+// CL: channels per lane (dim <= 16 CL), NC: columns per lane.  The registers hold D = S - v of the next token, which
+// takes one multiply-add per element and token (D <- f D + dv) where S takes two operations; v's share of the output,
+// v_(t+1) sum(q), is added when the output is written, and D of a sequence's last new token is its state.
+template <int CL, int NC, typename OutT>
 __global__ void __launch_bounds__(kScanThreads, CL <= 8 ? 4 : 1)
-hgrn2_scan_kernel(const __grid_constant__ RecurrentParams p) {
-  constexpr int TT = kScanTokens, DP = kScanLanes * CL, COLS = 8 * NC;   // COLS: columns of the CTA
-  constexpr int NG = TT * DP / 4 / kScanThreads > 0 ? TT * DP / 4 / kScanThreads : 1;
-  constexpr int NVG = TT * COLS / 4;                // groups of four values per tile
-  constexpr int NV = (NVG + kScanThreads - 1) / kScanThreads;
+hgrn2_scan_kernel(const __grid_constant__ RecurrentParams p, const float* __restrict__ q_act,
+                  const float* __restrict__ f_act, const float* __restrict__ dv, int vp) {
+  constexpr int TT = CL <= 8 ? 16 : 8;              // tokens per tile
+  constexpr int DP = kScanLanes * CL, COLS = 8 * NC;
   constexpr int TB = kScanLanes / NC;               // tokens whose sums are exchanged together
+  constexpr int NO = TT * COLS / kScanThreads;      // outputs of a thread per tile
   __shared__ __align__(16) float qs[2][TT][DP];
   __shared__ __align__(16) float fs[2][TT][DP];
-  __shared__ __align__(16) float2 vs[2][TT][COLS];  // every value twice, as a packed pair
+  __shared__ __align__(16) float ds[2][TT][COLS];
   __shared__ float os[TT][COLS];
+  __shared__ float qsum[TT];
   const int head = blockIdx.y, b = blockIdx.z, col0 = blockIdx.x * COLS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane & 15;
   const int cl0 = (warp * 2 + (lane >> 4)) * NC;    // first of this lane's columns within the CTA
@@ -110,94 +132,84 @@ hgrn2_scan_kernel(const __grid_constant__ RecurrentParams p) {
   griddep_launch();
   const int n = p.q_lens[b], ctx = p.context_lens[b];
   if (n <= 0 || ctx < n) return;
-  const int row0 = p.q_start[b];
+  const long long row0 = p.q_start[b];
   const int slot = p.slot_ids ? p.slot_ids[b] : b;
   const bool fresh = ctx == n;
+  const int hv = head * p.vdim;
   float* st = p.state + (((long long)slot * p.heads + head) * p.vdim + col0 + cl0) * p.dim_p;
 
-  // channels of this lane: groups of four, group j at (j * 16 + g) * 4
-  float2 S[NC][CL / 2];
+  auto fetch = [&](int buf, int t0) {
 #pragma unroll
-  for (int k = 0; k < NC; ++k)
+    for (int i = 0; i < TT * DP / 4 / kScanThreads; ++i) {
+      const int idx = threadIdx.x + i * kScanThreads, tok = idx / (DP / 4), c = idx % (DP / 4) * 4;
+      const bool on = t0 + tok < n;
+      const long long o = ((row0 + (on ? t0 + tok : 0)) * p.heads + head) * DP + c;
+      cp_async16(&qs[buf][tok][c], q_act + o, on);
+      cp_async16(&fs[buf][tok][c], f_act + o, on);
+    }
+#pragma unroll
+    for (int i = 0; i < (TT * COLS / 4 + kScanThreads - 1) / kScanThreads; ++i) {
+      const int idx = threadIdx.x + i * kScanThreads, tok = idx / (COLS / 4), c = idx % (COLS / 4) * 4;
+      if (idx < TT * COLS / 4) {
+        const bool on = t0 + tok < n && col0 + c < vp;
+        const long long o = on ? ((row0 + t0 + tok) * p.heads + head) * vp + col0 + c : 0;
+        cp_async16(&ds[buf][tok][c], dv + o, on);
+      }
+    }
+    cp_async_commit();
+  };
+  fetch(0, 0);
+
+  // channels of this lane: groups of four, group j at (j * 16 + g) * 4
+  float2 D[NC][CL / 2];
+#pragma unroll
+  for (int k = 0; k < NC; ++k) {
+    const bool ok = col0 + cl0 + k < p.vdim;
+    const float v0 = ok ? proj_load(p.v, row0, hv + col0 + cl0 + k) : 0.f;
 #pragma unroll
     for (int j = 0; j < CL / 4; ++j) {
       const int c = (j * kScanLanes + g) * 4;
       float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (!fresh && col0 + cl0 + k < p.vdim && c < p.dim_p)
-        x = *reinterpret_cast<const float4*>(st + (long long)k * p.dim_p + c);
-      S[k][2 * j] = make_float2(x.x, x.y);
-      S[k][2 * j + 1] = make_float2(x.z, x.w);
+      if (!fresh && ok && c < p.dim_p) x = *reinterpret_cast<const float4*>(st + (long long)k * p.dim_p + c);
+      D[k][2 * j] = make_float2(x.x - v0, x.y - v0);
+      D[k][2 * j + 1] = make_float2(x.z - v0, x.w - v0);
     }
-
-  RawGroup<V> rq[NG], rf[NG], rv[NV];
-  const int hq = head * p.dim, hv = head * p.vdim;
-  // a thread fetches the same four channels of several tokens
-  constexpr int kTokStep = kScanThreads / (DP / 4);
-  const int lc = (threadIdx.x % (DP / 4)) * 4, ltok = threadIdx.x / (DP / 4);
-  float fb[4], fl[4];
-#pragma unroll
-  for (int e = 0; e < 4; ++e) {
-    fb[e] = lc + e < p.dim ? p.f_bias[hq + lc + e] : 0.f;
-    fl[e] = lc + e < p.dim ? p.lower[hq + lc + e] : 0.f;
   }
-  auto fetch = [&](int t0) {
-#pragma unroll
-    for (int i = 0; i < NG; ++i) {
-      const int tok = ltok + i * kTokStep;
-      rq[i].clear();
-      rf[i].clear();
-      if (tok < TT && t0 + tok < n && lc < p.dim) {
-        fetch_group<V>(rq[i], p.q, row0 + t0 + tok, hq, lc, p.dim);
-        fetch_group<V>(rf[i], p.f, row0 + t0 + tok, hq, lc, p.dim);
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < NV; ++i) {
-      const int idx = threadIdx.x + i * kScanThreads, tok = idx / (COLS / 4), c = col0 + idx % (COLS / 4) * 4;
-      rv[i].clear();
-      if (idx < NVG && t0 + tok < n && c < p.vdim) fetch_group<V>(rv[i], p.v, row0 + t0 + tok, hv, c, p.vdim);
-    }
-  };
-  // activations of the fetched tile into shared memory; a token past the end keeps the state (f = 1, q = 0)
-  auto publish = [&](int buf, int t0) {
-#pragma unroll
-    for (int i = 0; i < NG; ++i) {
-      const int tok = ltok + i * kTokStep;
-      if (tok < TT) {
-        const bool on = t0 + tok < n;
-        const float4 u = rq[i].get(), z = rf[i].get();
-        float4 q, f;
-        q.x = query_act(u.x, on && lc < p.dim);
-        q.y = query_act(u.y, on && lc + 1 < p.dim);
-        q.z = query_act(u.z, on && lc + 2 < p.dim);
-        q.w = query_act(u.w, on && lc + 3 < p.dim);
-        f.x = forget_gate(z.x, fb[0], fl[0], on && lc < p.dim);
-        f.y = forget_gate(z.y, fb[1], fl[1], on && lc + 1 < p.dim);
-        f.z = forget_gate(z.z, fb[2], fl[2], on && lc + 2 < p.dim);
-        f.w = forget_gate(z.w, fb[3], fl[3], on && lc + 3 < p.dim);
-        *reinterpret_cast<float4*>(&qs[buf][tok][lc]) = q;
-        *reinterpret_cast<float4*>(&fs[buf][tok][lc]) = f;
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < NV; ++i) {
-      const int idx = threadIdx.x + i * kScanThreads;
-      if (idx < NVG) {
-        const float4 x = rv[i].get();
-        float4* dst = reinterpret_cast<float4*>(&vs[buf][idx / (COLS / 4)][idx % (COLS / 4) * 4]);
-        dst[0] = make_float4(x.x, x.x, x.y, x.y);
-        dst[1] = make_float4(x.z, x.z, x.w, x.w);
-      }
-    }
-  };
-  fetch(0);
-  publish(0, 0);
-  __syncthreads();
+
   int buf = 0;
 #pragma unroll 1
   for (int t0 = 0; t0 < n; t0 += TT, buf ^= 1) {
-    const bool more = t0 + TT < n;
-    if (more) fetch(t0 + TT);
+    cp_async_wait_all();
+    __syncthreads();                                 // the tile is there; nobody reads the other buffer or os any more
+    if (t0 + TT < n) {
+      fetch(buf ^ 1, t0 + TT);
+    } else {
+      // tokens past the end keep D: gate one (query and dv are zero-filled)
+      for (int i = threadIdx.x; i < (t0 + TT - n) * DP; i += kScanThreads) fs[buf][n - t0 + i / DP][i % DP] = 1.f;
+      __syncthreads();
+    }
+    // v of the token after each of this thread's outputs, as fetched: a conversion here would wait for the load
+    uint32_t vn[NO];
+#pragma unroll
+    for (int i = 0; i < NO; ++i) {
+      const int idx = threadIdx.x + i * kScanThreads, tok = idx / COLS, c = col0 + idx % COLS;
+      vn[i] = 0u;
+      if (t0 + tok + 1 < n && c < p.vdim) {
+        const long long r = row0 + t0 + tok + 1;
+        if (p.v.bf16)
+          vn[i] = reinterpret_cast<const uint16_t*>(p.v.ptr)[r * p.v.ld + hv + c];
+        else
+          vn[i] = __float_as_uint(proj_load(p.v, r, hv + c));
+      }
+    }
+#pragma unroll
+    for (int tok = warp; tok < TT; tok += kScanThreads / 32) {
+      float a = 0.f;
+#pragma unroll
+      for (int i = 0; i < DP / 32; ++i) a += qs[buf][tok][lane + 32 * i];
+      a = warp_sum(a);
+      if (lane == 0) qsum[tok] = a;
+    }
 #pragma unroll 1
     for (int h = 0; h < TT; h += TB) {
       if (t0 + h >= n) break;
@@ -212,14 +224,25 @@ hgrn2_scan_kernel(const __grid_constant__ RecurrentParams p) {
           f2[2 * j] = make_float2(f.x, f.y); f2[2 * j + 1] = make_float2(f.z, f.w);
           q2[2 * j] = make_float2(q.x, q.y); q2[2 * j + 1] = make_float2(q.z, q.w);
         }
+        float d[NC];
+        if constexpr (NC >= 4) {
+#pragma unroll
+          for (int k = 0; k < NC; k += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(&ds[buf][h + tt][cl0 + k]);
+            d[k] = x.x; d[k + 1] = x.y; d[k + 2] = x.z; d[k + 3] = x.w;
+          }
+        } else {
+#pragma unroll
+          for (int k = 0; k < NC; ++k) d[k] = ds[buf][h + tt][cl0 + k];
+        }
 #pragma unroll
         for (int k = 0; k < NC; ++k) {
-          const float2 v2 = vs[buf][h + tt][cl0 + k];
+          const float2 d2 = make_float2(d[k], d[k]);
           float2 o = make_float2(0.f, 0.f);
 #pragma unroll
           for (int j = 0; j < CL / 2; ++j) {
-            S[k][j] = ffma2(f2[j], fsub2(S[k][j], v2), v2);
-            o = ffma2(q2[j], S[k][j], o);
+            D[k][j] = ffma2(f2[j], D[k][j], d2);
+            o = ffma2(q2[j], D[k][j], o);
           }
           po[tt * NC + k] = o.x + o.y;
         }
@@ -235,16 +258,15 @@ hgrn2_scan_kernel(const __grid_constant__ RecurrentParams p) {
       }
       os[h + g / NC][cl0 + g % NC] = po[0];
     }
-    if (more) publish(buf ^ 1, t0 + TT);
     __syncthreads();
     OutT* out = reinterpret_cast<OutT*>(p.out);
 #pragma unroll
-    for (int i = 0; i < TT * COLS / kScanThreads; ++i) {
+    for (int i = 0; i < NO; ++i) {
       const int idx = threadIdx.x + i * kScanThreads, tok = idx / COLS, c = col0 + idx % COLS;
       if (t0 + tok < n && c < p.vdim)
-        out[(long long)(row0 + t0 + tok) * p.heads * p.vdim + hv + c] = cast_out<OutT>(os[tok][idx % COLS]);
+        out[(row0 + t0 + tok) * p.heads * p.vdim + hv + c] = cast_out<OutT>(
+            fmaf(__uint_as_float(p.v.bf16 ? vn[i] << 16 : vn[i]), qsum[tok], os[tok][idx % COLS]));
     }
-    __syncthreads();
   }
 #pragma unroll
   for (int k = 0; k < NC; ++k)
@@ -253,12 +275,13 @@ hgrn2_scan_kernel(const __grid_constant__ RecurrentParams p) {
       const int c = (j * kScanLanes + g) * 4;
       if (col0 + cl0 + k < p.vdim && c < p.dim_p)
         *reinterpret_cast<float4*>(st + (long long)k * p.dim_p + c) =
-            make_float4(S[k][2 * j].x, S[k][2 * j].y, S[k][2 * j + 1].x, S[k][2 * j + 1].y);
+            make_float4(D[k][2 * j].x, D[k][2 * j].y, D[k][2 * j + 1].x, D[k][2 * j + 1].y);
     }
 }
 
-// x[t, h, :] / sqrt(mean(x[t, h, :]^2) + eps) * w, in place; one warp per (token, head)
-template <typename T>
+// x[t, h, :] / sqrt(mean(x[t, h, :]^2) + eps) * w, in place; one warp per (token, head).  VEC: vdim is a multiple of 4
+// and at most 128, so that a lane holds its four elements in registers.
+template <bool VEC, typename T>
 __global__ void __launch_bounds__(256) head_rmsnorm_kernel(T* __restrict__ x, const float* __restrict__ w, long long n,
                                                            int vdim, float eps) {
   griddep_wait();
@@ -267,6 +290,31 @@ __global__ void __launch_bounds__(256) head_rmsnorm_kernel(T* __restrict__ x, co
   const int lane = threadIdx.x & 31;
   if (i >= n) return;
   T* r = x + i * vdim;
+  if constexpr (VEC) {
+    const int c = lane * 4;
+    const bool on = c < vdim;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (on) {
+      if constexpr (sizeof(T) == 2) {
+        const uint2 u = *reinterpret_cast<const uint2*>(r + c);
+        const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+        v = make_float4(a.x, a.y, b.x, b.y);
+      } else {
+        v = *reinterpret_cast<const float4*>(r + c);
+      }
+    }
+    const float ss = warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w);
+    const float inv = 1.f / sqrtf(ss / float(vdim) + eps);
+    if (on) {
+      const float4 ww = *reinterpret_cast<const float4*>(w + c);
+      v = make_float4(v.x * inv * ww.x, v.y * inv * ww.y, v.z * inv * ww.z, v.w * inv * ww.w);
+      if constexpr (sizeof(T) == 2)
+        *reinterpret_cast<uint2*>(r + c) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+      else
+        *reinterpret_cast<float4*>(r + c) = v;
+    }
+    return;
+  }
   float ss = 0.f;
   for (int c = lane; c < vdim; c += 32) {
     const float v = cast_in<T>(r[c]);
@@ -274,6 +322,13 @@ __global__ void __launch_bounds__(256) head_rmsnorm_kernel(T* __restrict__ x, co
   }
   const float inv = 1.f / sqrtf(warp_sum(ss) / float(vdim) + eps);
   for (int c = lane; c < vdim; c += 32) r[c] = cast_out<T>(cast_in<T>(r[c]) * inv * w[c]);
+}
+template <typename T>
+static int launch_head_rmsnorm(void* x, const float* w, long long rows, int vdim, float eps, cudaStream_t s) {
+  const bool vec = vdim % 4 == 0 && vdim <= 128 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) == 0;
+  const dim3 grid(unsigned((rows + 7) / 8));
+  return vec ? launch_pdl(head_rmsnorm_kernel<true, T>, grid, dim3(256), 0, s, reinterpret_cast<T*>(x), w, rows, vdim, eps)
+             : launch_pdl(head_rmsnorm_kernel<false, T>, grid, dim3(256), 0, s, reinterpret_cast<T*>(x), w, rows, vdim, eps);
 }
 
 constexpr int kStepThreads = 256;
@@ -369,22 +424,30 @@ hgrn2_step_kernel(const __grid_constant__ RecurrentParams p) {
   for (int c = threadIdx.x; c < p.vdim; c += kStepThreads) out[c] = cast_out<OutT>(os[c] * inv * p.norm_w[c]);
 }
 
-template <int CL, int NC, int V>
-static int launch_scan_nc(const RecurrentParams& p, int batch, int out_bf16, cudaStream_t s) {
+struct ScanInputs {
+  const float *q_act, *f_act, *dv;
+  int vp;
+};
+template <int CL, int NC>
+static int launch_scan_nc(const RecurrentParams& p, const ScanInputs& in, int batch, int out_bf16, cudaStream_t s) {
   const dim3 grid((p.vdim + 8 * NC - 1) / (8 * NC), p.heads, batch);
-  return out_bf16 ? launch_pdl(hgrn2_scan_kernel<CL, NC, V, __nv_bfloat16>, grid, dim3(kScanThreads), 0, s, p)
-                  : launch_pdl(hgrn2_scan_kernel<CL, NC, V, float>, grid, dim3(kScanThreads), 0, s, p);
+  return out_bf16 ? launch_pdl(hgrn2_scan_kernel<CL, NC, __nv_bfloat16>, grid, dim3(kScanThreads), 0, s, p, in.q_act,
+                               in.f_act, in.dv, in.vp)
+                  : launch_pdl(hgrn2_scan_kernel<CL, NC, float>, grid, dim3(kScanThreads), 0, s, p, in.q_act, in.f_act,
+                               in.dv, in.vp);
 }
-// More columns per lane mean fewer shared-memory reads per state element, fewer mean more CTAs: take the most columns
-// that still give (nearly) every SM a CTA.
-template <int CL, int V>
-static int launch_scan(const RecurrentParams& p, int batch, int out_bf16, cudaStream_t s) {
+// More columns per lane mean fewer shared-memory reads per state element, fewer mean more warps to hide latency with:
+// eight columns from about two CTAs per SM on, two when even four would leave SMs with a single CTA (measured on one,
+// two, four and eight sequences of 32 heads of 128 x 128).
+template <int CL>
+static int launch_scan(const RecurrentParams& p, const ScanInputs& in, int batch, int out_bf16, cudaStream_t s) {
   const auto ctas = [&](int cols) { return (long long)batch * p.heads * ((p.vdim + cols - 1) / cols); };
   if constexpr (CL <= 8)
-    if (ctas(64) >= 120) return launch_scan_nc<CL, 8, V>(p, batch, out_bf16, s);
-  if (ctas(32) >= 120) return launch_scan_nc<CL, 4, V>(p, batch, out_bf16, s);
-  return launch_scan_nc<CL, 2, V>(p, batch, out_bf16, s);
+    if (ctas(64) >= 2 * 148) return launch_scan_nc<CL, 8>(p, in, batch, out_bf16, s);
+  if (ctas(32) >= 200) return launch_scan_nc<CL, 4>(p, in, batch, out_bf16, s);
+  return launch_scan_nc<CL, 2>(p, in, batch, out_bf16, s);
 }
+static int scan_channels(int dim) { return dim <= 64 ? 64 : (dim <= 128 ? 128 : 256); }
 template <int CH>
 static int launch_step(const RecurrentParams& p, int batch, int out_bf16, cudaStream_t s) {
   const dim3 grid(p.heads, batch);
@@ -407,33 +470,40 @@ static int recurrent_params(RecurrentParams& p, const NkbProj* q, const NkbProj*
   return 0;
 }
 
+// floats of scratch one token of a scan needs
+extern "C" long long nkb_hgrn2_scan_scratch(int heads, int dim, int vdim) {
+  return (long long)heads * (2 * scan_channels(dim) + (vdim + 3) / 4 * 4);
+}
+
+// scratch: tokens * nkb_hgrn2_scan_scratch(...) floats, 16-byte aligned.  Every row of the packed batch belongs to one
+// of the sequences.
 extern "C" int nkb_hgrn2_scan(const NkbProj* q, const NkbProj* f, const NkbProj* v, const float* f_bias,
                               const float* lower, float* state, const int* slot_ids, const int* q_start,
-                              const int* q_lens, const int* context_lens, void* out, int out_bf16, int batch, int tokens,
-                              int heads, int dim, int vdim, const float* norm_w, float eps, void* stream) {
+                              const int* q_lens, const int* context_lens, float* scratch, void* out, int out_bf16,
+                              int batch, int tokens, int heads, int dim, int vdim, const float* norm_w, float eps,
+                              void* stream) {
   if (batch <= 0 || tokens <= 0) return 0;
-  if (batch > 65535 || heads > 65535) return -2;
+  if (batch > 65535 || heads > 65535 || !scratch || (reinterpret_cast<uintptr_t>(scratch) & 15)) return -2;
   RecurrentParams p{};
   if (int rc = recurrent_params(p, q, f, v, f_bias, lower, state, slot_ids, context_lens, out, heads, dim, vdim)) return rc;
   p.q_start = q_start;
   p.q_lens = q_lens;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const bool vec = dim % 4 == 0 && vdim % 4 == 0 && proj_vec4_ok(*q) && proj_vec4_ok(*f) && proj_vec4_ok(*v);
-  const int form = !vec ? 1 : (q->bf16 && f->bf16 && v->bf16 ? kPackedBf16 : 4);
-  const auto scan = [&](auto cl) {
-    constexpr int CL = decltype(cl)::value;
-    return form == 1 ? launch_scan<CL, 1>(p, batch, out_bf16, s)
-                     : (form == 4 ? launch_scan<CL, 4>(p, batch, out_bf16, s) : launch_scan<CL, kPackedBf16>(p, batch, out_bf16, s));
-  };
-  const int rc = dim <= 64 ? scan(std::integral_constant<int, 4>{})
-                           : (dim <= 128 ? scan(std::integral_constant<int, 8>{}) : scan(std::integral_constant<int, 16>{}));
+  const int dp = scan_channels(dim), vp = (vdim + 3) / 4 * 4;
+  float* q_act = scratch;
+  float* f_act = q_act + (long long)tokens * heads * dp;
+  float* dv = f_act + (long long)tokens * heads * dp;
+  int rc = vec ? launch_pdl(hgrn2_gates_kernel<4>, dim3(tokens), dim3(256), 0, s, p, q_act, f_act, dv, dp, vp, batch)
+               : launch_pdl(hgrn2_gates_kernel<1>, dim3(tokens), dim3(256), 0, s, p, q_act, f_act, dv, dp, vp, batch);
+  if (rc) return rc;
+  const ScanInputs in{q_act, f_act, dv, vp};
+  rc = dp == 64 ? launch_scan<4>(p, in, batch, out_bf16, s)
+                : (dp == 128 ? launch_scan<8>(p, in, batch, out_bf16, s) : launch_scan<16>(p, in, batch, out_bf16, s));
   if (rc || !norm_w) return rc;
   const long long rows = (long long)tokens * heads;
-  const dim3 grid(unsigned((rows + 7) / 8));
-  return out_bf16 ? launch_pdl(head_rmsnorm_kernel<__nv_bfloat16>, grid, dim3(256), 0, s,
-                               reinterpret_cast<__nv_bfloat16*>(out), norm_w, rows, vdim, eps)
-                  : launch_pdl(head_rmsnorm_kernel<float>, grid, dim3(256), 0, s, reinterpret_cast<float*>(out), norm_w,
-                               rows, vdim, eps);
+  return out_bf16 ? launch_head_rmsnorm<__nv_bfloat16>(out, norm_w, rows, vdim, eps, s)
+                  : launch_head_rmsnorm<float>(out, norm_w, rows, vdim, eps, s);
 }
 
 extern "C" int nkb_hgrn2_step(const NkbProj* q, const NkbProj* f, const NkbProj* v, const float* f_bias,

@@ -71,7 +71,7 @@ class _TimedLib:
 
     def __getattr__(self, name):
         fn = getattr(self._real, name)
-        if not name.startswith(self._LAUNCHERS) or name.endswith(("_splits", "_floats")):
+        if not name.startswith(self._LAUNCHERS) or name.endswith(("_splits", "_floats", "_scratch")):
             return fn
         return _TimedFn(self, name, fn)
 

@@ -64,7 +64,7 @@ def build_prompts(args, cfg: ModelConfig, tokenizer) -> List[List[int]]:
 def shrink(cfg: ModelConfig) -> ModelConfig:
     """Same architecture features, toy sizes."""
     if cfg.layers is not None:
-        return tolenex_shape(256, layers=len(cfg.layers), heads=4, kv_heads=2, ff=512, vocab=2048, dim=32, vdim=64,
+        return tolenex_shape(256, layers=len(cfg.layers), heads=4, kv_heads=1, ff=512, vocab=2048, dim=32, vdim=64,
                              groups=cfg.norm_groups, loop=cfg.loop, embedding_scale=cfg.embedding_scale)
     over = dict(vocab_size=2048, hidden_size=256, num_heads=4, num_kv_heads=2, head_dim=64, intermediate_size=512,
                 max_position=min(cfg.max_position, 4096))

@@ -52,7 +52,8 @@ _SIGNATURES = {
                                    c_int, ctypes.POINTER(_P), ctypes.POINTER(_P), c_int, c_int, c_int, c_int, c_float,
                                    _P]),
     "nkb_gated_act": (c_int, [_PP, _PP, _P, c_int, c_int, c_int, c_int, _P]),
-    "nkb_hgrn2_scan": (c_int, [_PP, _PP, _PP, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
+    "nkb_hgrn2_scan_scratch": (c_longlong, [c_int, c_int, c_int]),
+    "nkb_hgrn2_scan": (c_int, [_PP, _PP, _PP, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
                                _P, c_float, _P]),
     "nkb_hgrn2_step": (c_int, [_PP, _PP, _PP, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, c_float,
                                _P]),

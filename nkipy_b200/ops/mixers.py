@@ -204,11 +204,12 @@ def hgrn2(q: Proj, f: Proj, v: Proj, f_bias: torch.Tensor, lower: torch.Tensor, 
         _lib.check(rc, "nkb_hgrn2_step")
         _count_launch()
         return out
+    scratch = torch.empty((T * L.nkb_hgrn2_scan_scratch(heads, dim, vdim),), dtype=torch.float32, device=state.device)
     rc = L.nkb_hgrn2_scan(_ref(q), _ref(f), _ref(v), f_bias.data_ptr(), lower.data_ptr(), state.data_ptr(), _ptr(rows),
-                          q_start.data_ptr(), q_lens.data_ptr(), context_lens.data_ptr(), out.data_ptr(), bf, B, T,
-                          heads, dim, vdim, norm_w.data_ptr(), float(eps), _stream())
+                          q_start.data_ptr(), q_lens.data_ptr(), context_lens.data_ptr(), scratch.data_ptr(),
+                          out.data_ptr(), bf, B, T, heads, dim, vdim, norm_w.data_ptr(), float(eps), _stream())
     _lib.check(rc, "nkb_hgrn2_scan")
-    _count_launch(2)
+    _count_launch(3)
     return out
 
 
