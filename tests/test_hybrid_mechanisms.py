@@ -21,6 +21,15 @@ in_dtypes = pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], id
 TOL = {torch.float32: 2e-5, torch.bfloat16: 2e-2}
 
 
+@pytest.fixture(autouse=True, scope="module")
+def _one_thread():
+    """The small tensors of these tests gain nothing from threads and lose a lot when several test processes share cores."""
+    n = torch.get_num_threads()
+    torch.set_num_threads(1)
+    yield
+    torch.set_num_threads(n)
+
+
 def rnd(*shape, seed=0, std=1.0):
     return torch.randn(shape, generator=torch.Generator().manual_seed(seed)) * std
 

@@ -25,6 +25,15 @@ on_devices = pytest.mark.parametrize("device", DEVICES)
 in_dtypes = pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], ids=["f32", "bf16"])
 TOL = {torch.float32: 1e-4, torch.bfloat16: 8e-2}
 
+
+@pytest.fixture(autouse=True, scope="module")
+def _one_thread():
+    """The small tensors of these tests gain nothing from threads and lose a lot when several test processes share cores."""
+    n = torch.get_num_threads()
+    torch.set_num_threads(1)
+    yield
+    torch.set_num_threads(n)
+
 # name -> small_config arguments; sizes, orders and branches differ between them
 MODELS = {
     "mixed": dict(layers="rara", loop=(1, 3, 3)),
