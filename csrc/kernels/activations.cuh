@@ -1,0 +1,19 @@
+// Elementwise activations by code (the table ACTIVATIONS of nkipy_b200/ops/mixers.py).
+#pragma once
+#include "proj_src.cuh"
+
+namespace nkb {
+enum { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_RELU2 = 2, ACT_TANH = 3, ACT_SIGMOID = 4, ACT_NONE = 5, ACT_COUNT = 6 };
+
+// GELU in its tanh form is written with the exponential: (1 + tanh u) / 2 = 1 / (1 + exp(-2 u))
+__device__ __forceinline__ float apply_act(float z, int kind) {
+  switch (kind) {
+    case ACT_SILU: return z / (1.f + expf(-z));
+    case ACT_GELU_TANH: return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+    case ACT_RELU2: { const float r = fmaxf(z, 0.f); return r * r; }
+    case ACT_TANH: return tanhf(z);
+    case ACT_SIGMOID: return 1.f / (1.f + expf(-z));
+    default: return z;
+  }
+}
+}  // namespace nkb

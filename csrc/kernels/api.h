@@ -6,6 +6,7 @@
 #include <cuda.h>
 #include <stdint.h>
 #include "attn_maps.h"
+#include "linear_attn.h"
 #include "proj_src.h"
 
 namespace nkb {
@@ -71,8 +72,8 @@ int nkb_gemm_bf16_grouped(const void* weights, const void* x_sorted, void* out, 
                           float act_alpha, int block_n, const int* tile_list, const int* tile_count, int max_tiles,
                           const void* arrive, unsigned int arrive_target, void* stream);
 int nkb_moe_dispatch(const int* experts, int tokens, int top_k, int expert_lo, int num_local, const void* x, int hidden,
-                     void* x_sorted, int* counts, int* offsets, int* cursors, int* pair_pos, int bn_a, int* tiles_a,
-                     int* ntiles_a, int bn_b, int* tiles_b, int* ntiles_b, void* stream);
+                     void* x_sorted, int* counts, int* offsets, int* cursors, int* pair_pos, int* row_token, int bn_a,
+                     int* tiles_a, int* ntiles_a, int bn_b, int* tiles_b, int* ntiles_b, void* stream);
 // expert-parallel token all-to-all (moe_a2a.cu)
 int nkb_moe_a2a_dispatch(const void* x, const int* experts, int tokens, int top_k, int hidden, int num_experts,
                          int n_ranks, int rank, unsigned int epoch, void* const* cnt, void* const* cnt_flag,
@@ -134,7 +135,8 @@ int nkb_argmax(const void* logits, int is_fp32, int* out_ids, float* out_vals, i
 int nkb_sample(const void* logits, int is_fp32, int* out_ids, int rows, int vocab, long long ld, float temperature,
                int top_k, float top_p, unsigned long long seed, unsigned long long step, void* stream);
 int nkb_router_topk(const void* logits, int is_fp32, int splits, long long split_stride, const void* bias,
-                    float* weights, int* experts, int tokens, int num_experts, int top_k, int mode, void* stream);
+                    float* weights, int* experts, int tokens, int num_experts, int top_k, int mode, int groups, int keep,
+                    float scale, void* stream);
 
 int nkb_paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                           const int* context_lens, void* out, float* scratch, int batch, int q_len, int nq, int nkv,
@@ -157,14 +159,28 @@ int nkb_flash_attn_prefill(const void* q, const void* k_cache, const void* v_cac
 
 // layers with an fp32 residual stream (gated_residual.cu)
 int nkb_gated_residual(const float* x_in, const int* ids, const void* table, int table_bf16, int vocab, float scale,
-                       int branches, const NkbProj* y, const NkbProj* g, const float* const* gbias, const float* add_row,
-                       const float* add_mat, float* x_out, int norms, const float* const* w, void* const* out,
-                       int out_bf16, int rows, int width, int groups, float eps, void* stream);
+                       int branches, const NkbBranch* br, const float* add_row, const float* add_mat, float* x_out,
+                       int norms, const float* const* w, void* const* out, int out_bf16, int rows, int width, int groups,
+                       float eps, void* stream);
 int nkb_gated_act(const NkbProj* gate, const NkbProj* up, void* out, int out_bf16, int rows, int inter, int kind,
                   void* stream);
 // CUDA-core GEMM for 32-bit models and untileable sizes (gemm_simt.cu)
 int nkb_gemm_simt(const void* x, int x_bf16, const void* w, int w_bf16, void* out, int out_bf16, int m, int n, int k,
                   long long ldx, long long ldw, long long ldo, void* stream);
+int nkb_gemm_simt_grouped(const void* x, int x_bf16, const void* w, int w_bf16, void* out, int out_bf16,
+                          const int* offsets, const int* row_token, int groups, int max_rows, int n, int k,
+                          long long ldx, long long ldo, void* stream);
+// linear attention with per-channel decay and what surrounds it (linear_attn.cu)
+int nkb_linattn_scan(const NkbLinAttn* args, void* stream);
+int nkb_linattn_step(const NkbLinAttn* args, void* stream);
+int nkb_low_rank(const NkbProj* x, int act, const void* w, int w_bf16, float* out, int tokens, int rank, int n,
+                 void* stream);
+int nkb_token_mix(const void* h, int bf16, const float* mu, float* state, const int* slot_ids, const int* q_start,
+                  const int* q_lens, const int* context_lens, void* out, int batch, int tokens, int width, int mixes,
+                  void* stream);
+int nkb_gate_heads(const void* x, int x_bf16, long long ld_token, long long ld_head, const NkbProj* gate, int gate_act,
+                   const float* norm_w, int norm_stride, float eps, float scale, void* out, int out_bf16,
+                   long long out_ld, int tokens, int heads, int width, void* stream);
 // gated linear recurrence (recurrent.cu)
 long long nkb_hgrn2_scan_scratch(int heads, int dim, int vdim);
 int nkb_hgrn2_scan(const NkbProj* q, const NkbProj* f, const NkbProj* v, const float* f_bias, const float* lower,
@@ -178,6 +194,9 @@ int nkb_hgrn2_step(const NkbProj* q, const NkbProj* f, const NkbProj* v, const f
 int nkb_maps_append(const NkbMapsArgs* a, const NkbProj* q, const NkbProj* k, const NkbProj* v, const float* cos_sin,
                     int rot_dims, int max_pos, const int* positions, const int* slots, void* q_out, void* k_cache,
                     void* v_cache, int bf16, int tokens, int block_size, void* stream);
+int nkb_row_norm_append(const NkbMapsArgs* a, const NkbProj* q, const NkbProj* k, const NkbProj* v, const float* q_norm,
+                        const float* k_norm, const int* slots, void* q_out, void* k_cache, void* v_cache, int bf16,
+                        int tokens, int block_size, void* stream);
 int nkb_maps_attn_simple(const NkbMapsArgs* a, const void* q, const void* k_cache, const void* v_cache,
                          const int* block_table, const int* q_start, const int* q_lens, const int* context_lens,
                          void* out, int bf16, int batch, int total_q, int block_size, int max_blocks_per_seq,

@@ -1,6 +1,7 @@
 // Attention with several score maps over shared values (attn_maps.h), everything but the tensor-core prefill:
 //   append   interleaved partial rotary embedding of queries and keys from the fused projection, keys and values
 //            into their slots of the paged cache
+//   row norm append   the same for one map without rotation, queries and keys normed over all heads of the token together
 //   decode   one new token per sequence, bf16: the two maps of up to eight query heads are the sixteen rows of
 //            one MMA fragment (rows 0-7 map 0, rows 8-15 map 1).  A key row holds both maps' keys side by side, so with
 //            the query of map 0 only in the first half of the contraction and that of map 1 only in the second, one
@@ -102,6 +103,108 @@ __global__ void __launch_bounds__(256) maps_append_kernel(const __grid_constant_
   }
 }
 
+// One CTA per token: RMS norms over the whole query and the whole key projection (weights of their full widths), queries
+// out with zeroed padding, keys and values into the cache.
+struct RowNormAppendParams {
+  NkbProj q, k, v;
+  NkbMapsArgs a;
+  const float *q_norm, *k_norm;
+  const int* slots;
+  void *q_out, *k_cache, *v_cache;
+};
+
+template <int V, typename T>
+__device__ __forceinline__ void store_v(T* dst, const float (&x)[V]) {
+  if constexpr (V == 4) {
+    store4<T>(dst, make_float4(x[0], x[1], x[2], x[3]));
+  } else {
+    *dst = cast_out<T>(x[0]);
+  }
+}
+template <int V>
+__device__ __forceinline__ void load_v(float (&x)[V], const NkbProj& s, long long row, int c) {
+  if constexpr (V == 4) {
+    const float4 r = proj_load4(s, row, c);
+    x[0] = r.x; x[1] = r.y; x[2] = r.z; x[3] = r.w;
+  } else {
+    x[0] = proj_load(s, row, c);
+  }
+}
+
+template <int V, typename T>
+__global__ void __launch_bounds__(256) row_norm_append_kernel(const __grid_constant__ RowNormAppendParams p) {
+  extern __shared__ __align__(16) float rn_s[];   // q row, k row
+  __shared__ float red[2][8];
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int nq = p.a.heads * p.a.dim, nk = p.a.kv_heads * p.a.dim, nv = p.a.kv_heads * p.a.vdim;
+  griddep_wait();
+  griddep_launch();
+  const int slot = p.slots[t];
+  const long long blk = slot < 0 ? 0 : slot / kMapsPage, off = slot < 0 ? 0 : slot % kMapsPage;
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x * V; c < nq; c += 256 * V) {
+    float x[V];
+    load_v<V>(x, p.q, t, c);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      sq += x[j] * x[j];
+      rn_s[c + j] = x[j];
+    }
+  }
+  for (int c = threadIdx.x * V; c < nk; c += 256 * V) {
+    float x[V];
+    load_v<V>(x, p.k, t, c);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      sk += x[j] * x[j];
+      rn_s[nq + c + j] = x[j];
+    }
+  }
+  if (slot >= 0) {
+    T* vc = reinterpret_cast<T*>(p.v_cache);
+    for (int c = threadIdx.x * V; c < nv; c += 256 * V) {
+      float x[V];
+      load_v<V>(x, p.v, t, c);
+      const int h = c / p.a.vdim, d = c % p.a.vdim;
+      store_v<V, T>(vc + ((blk * p.a.kv_heads + h) * kMapsPage + off) * p.a.vdim_p + d, x);
+    }
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if (lane == 0) {
+    red[0][warp] = sq;
+    red[1][warp] = sk;
+  }
+  __syncthreads();
+  float tq = 0.f, tk = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) {
+    tq += red[0][w];
+    tk += red[1][w];
+  }
+  const float iq = 1.f / sqrtf(tq / float(nq) + p.a.eps), ik = 1.f / sqrtf(tk / float(nk) + p.a.eps);
+  T* qo = reinterpret_cast<T*>(p.q_out) + (long long)t * p.a.heads * p.a.dim_p;
+  for (int i = threadIdx.x * V; i < p.a.heads * p.a.dim_p; i += 256 * V) {
+    const int h = i / p.a.dim_p, d = i % p.a.dim_p;
+    float x[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const int c = h * p.a.dim + d + j;
+      x[j] = d + j < p.a.dim ? rn_s[c] * iq * p.q_norm[c] : 0.f;
+    }
+    store_v<V, T>(qo + i, x);
+  }
+  if (slot < 0) return;
+  T* kc = reinterpret_cast<T*>(p.k_cache);
+  for (int c = threadIdx.x * V; c < nk; c += 256 * V) {
+    const int h = c / p.a.dim, d = c % p.a.dim;
+    float x[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[j] = rn_s[nq + c + j] * ik * p.k_norm[c + j];
+    store_v<V, T>(kc + ((blk * p.a.kv_heads + h) * kMapsPage + off) * p.a.dim_p + d, x);
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ simple
 struct MapsSimpleParams {
   NkbMapsArgs a;
@@ -149,11 +252,12 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) maps_simple_kernel(const __
 #pragma unroll
   for (int i = 0; i < kSimpleCols; ++i) o[0][i] = o[1][i] = 0.f;
   const int pages = pos / kMapsPage + 1;
-  for (int pg = warp; pg < pages; pg += kSimpleWarps) {
+  const int lo = p.a.window > 0 ? max(0, pos - p.a.window + 1) : 0;      // first visible position
+  for (int pg = lo / kMapsPage + warp; pg < pages; pg += kSimpleWarps) {
     const long long blk = table[pg];
     const T* kr = reinterpret_cast<const T*>(p.k_cache) + ((blk * p.a.kv_heads + g) * kMapsPage + lane) * kw;
     const T* vb = reinterpret_cast<const T*>(p.v_cache) + (blk * p.a.kv_heads + g) * kMapsPage * VP;
-    const bool vis = pg * kMapsPage + lane <= pos;
+    const bool vis = pg * kMapsPage + lane <= pos && pg * kMapsPage + lane >= lo;
     const int nvis = min(kMapsPage, pos + 1 - pg * kMapsPage);
     float pr[2] = {0.f, 0.f};
 #pragma unroll
@@ -564,6 +668,30 @@ extern "C" int nkb_maps_append(const NkbMapsArgs* a, const NkbProj* q, const Nkb
               : launch_pdl(maps_append_kernel<float>, grid, dim3(256), 0, s, p);
 }
 
+extern "C" int nkb_row_norm_append(const NkbMapsArgs* a, const NkbProj* q, const NkbProj* k, const NkbProj* v,
+                                   const float* q_norm, const float* k_norm, const int* slots, void* q_out, void* k_cache,
+                                   void* v_cache, int bf16, int tokens, int block_size, void* stream) {
+  if (tokens <= 0) return 0;
+  if (!maps_ok(*a) || a->maps != 1 || block_size != kMapsPage) return -2;
+  RowNormAppendParams p{};
+  p.q = *q; p.k = *k; p.v = *v; p.a = *a;
+  p.q_norm = q_norm; p.k_norm = k_norm; p.slots = slots;
+  p.q_out = q_out; p.k_cache = k_cache; p.v_cache = v_cache;
+  const size_t smem = size_t(a->heads + a->kv_heads) * a->dim * sizeof(float);
+  if (smem > 48 * 1024 - 128) return -2;
+  const auto al16 = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
+  const bool vec = ((a->dim | a->dim_p | a->vdim | a->vdim_p) & 3) == 0 && proj_vec4_ok(*q) && proj_vec4_ok(*k) &&
+                   proj_vec4_ok(*v) && al16(q_out) && al16(k_cache) && al16(v_cache);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid(tokens), block(256);
+  using bf = __nv_bfloat16;
+  if (vec)
+    return bf16 ? launch_pdl(row_norm_append_kernel<4, bf>, grid, block, smem, s, p)
+                : launch_pdl(row_norm_append_kernel<4, float>, grid, block, smem, s, p);
+  return bf16 ? launch_pdl(row_norm_append_kernel<1, bf>, grid, block, smem, s, p)
+              : launch_pdl(row_norm_append_kernel<1, float>, grid, block, smem, s, p);
+}
+
 extern "C" int nkb_maps_attn_simple(const NkbMapsArgs* a, const void* q, const void* k_cache, const void* v_cache,
                                     const int* block_table, const int* q_start, const int* q_lens,
                                     const int* context_lens, void* out, int bf16, int batch, int total_q, int block_size,
@@ -596,7 +724,7 @@ extern "C" int nkb_maps_attn_decode(const NkbMapsArgs* a, const void* q, const v
                                     void* stream) {
   if (batch <= 0) return 0;
   if (!maps_ok(*a) || block_size != kMapsPage || batch > 65535) return -2;
-  if (a->maps != 2 || (a->dim_p != 32 && a->dim_p != 64) || (a->vdim_p != 64 && a->vdim_p != 128)) return -5;
+  if (a->maps != 2 || a->window > 0 || (a->dim_p != 32 && a->dim_p != 64) || (a->vdim_p != 64 && a->vdim_p != 128)) return -5;
   if (!status_word() && nkb_init() != 0) return -1;
   MapsDecodeParams p{};
   p.a = *a;

@@ -58,11 +58,6 @@ __device__ __forceinline__ bool mp_wait(uint64_t* bar, uint32_t parity, volatile
   return mp_wait_slow(bar, parity, abort_flag, status, code);
 }
 
-__device__ __forceinline__ float2 fmul2(float2 a, float2 b) {
-  uint64_t rd;
-  asm("mul.f32x2 %0, %1, %2;" : "=l"(rd) : "l"(reinterpret_cast<uint64_t&>(a)), "l"(reinterpret_cast<uint64_t&>(b)));
-  return reinterpret_cast<float2&>(rd);
-}
 __device__ __forceinline__ float2 dup2(float x) { return make_float2(x, x); }
 
 // DP: padded size of one map's query / key (32 or 64), VD: padded value size (64 or 128)
@@ -470,7 +465,7 @@ extern "C" int nkb_maps_attn_prefill(const NkbMapsArgs* a, const void* q, const 
                                      const int* context_lens, void* out, int batch, int total_q, int max_q_len,
                                      int block_size, int num_blocks, int max_blocks_per_seq, void* stream) {
   if (batch <= 0 || total_q <= 0) return 0;
-  if (a->maps != 2 || (a->dim_p != 32 && a->dim_p != 64) || (a->vdim_p != 64 && a->vdim_p != 128)) return -5;
+  if (a->maps != 2 || a->window > 0 || (a->dim_p != 32 && a->dim_p != 64) || (a->vdim_p != 64 && a->vdim_p != 128)) return -5;
   if (block_size != kMpPage || a->kv_heads < 1 || a->heads % a->kv_heads || batch > 65535 || a->heads > 65535) return -2;
   if (!status_word() && nkb_init() != 0) return -1;
   MapsPrefillParams p{};

@@ -479,6 +479,11 @@ __device__ __forceinline__ float2 ffma2(float2 a, float2 b, float2 c) {
       : "l"(reinterpret_cast<uint64_t&>(a)), "l"(reinterpret_cast<uint64_t&>(b)), "l"(reinterpret_cast<uint64_t&>(c)));
   return reinterpret_cast<float2&>(rd);
 }
+__device__ __forceinline__ float2 fmul2(float2 a, float2 b) {
+  uint64_t rd;
+  asm("mul.f32x2 %0, %1, %2;" : "=l"(rd) : "l"(reinterpret_cast<uint64_t&>(a)), "l"(reinterpret_cast<uint64_t&>(b)));
+  return reinterpret_cast<float2&>(rd);
+}
 __device__ __forceinline__ float2 fadd2(float2 a, float2 b) {
   uint64_t rd;
   asm("add.f32x2 %0, %1, %2;" : "=l"(rd) : "l"(reinterpret_cast<uint64_t&>(a)), "l"(reinterpret_cast<uint64_t&>(b)));

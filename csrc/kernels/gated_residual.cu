@@ -1,16 +1,18 @@
 // The elementwise ends of a layer whose residual stream stays in fp32:
 //
 //   embedding        x = table[id] * scale
-//   gated residual   x <- x + sum_i sigmoid(gate_i + gate_bias_i) * branch_i   (+ a per-model vector) (+ a
-//                    per-token matrix, both used ahead of a repeated block of layers)
+//   residual         x <- x + sum_i branch_i   (+ a per-model vector) (+ a per-token matrix, both used ahead of a
+//                    repeated block of layers); a branch is scaled, gated by sigmoid(gate_i + gate_bias_i), or the
+//                    weighted sum of the token's expert rows (NkbBranch)
 //   group norms      out_j = w_j * x / sqrt(mean over the element's group of x^2 + eps), up to two weightings
 //                    of one normalised row (layers whose two sublayers read the same residual)
 //
 // in one launch per layer: a CTA owns a token row, keeps it in shared memory between the sum and the norm, and
-// takes the branches and gates as split-K partial sums, bf16 or fp32 (proj_src.h).  Also here: the gated
-// activation act(gate) * up over the same forms.
+// takes the branches and gates as split-K partial sums, bf16 or fp32 (proj_src.h).  Also here: the activations
+// act(gate) * up and act(x) over the same forms.
 #include "common.cuh"
 #include "proj_src.cuh"
+#include "activations.cuh"
 #include "api.h"
 
 namespace nkb {
@@ -24,8 +26,7 @@ struct GatedResidualParams {
   float scale;
   int vocab, table_bf16;
   int branches;
-  NkbProj y[2], g[2];
-  const float* gbias[2];
+  NkbBranch br[2];
   const float* add_row;           // [width] or nullptr
   const float* add_mat;           // [tokens, width] fp32 or nullptr
   float* x_out;                   // may be nullptr
@@ -53,6 +54,24 @@ __device__ __forceinline__ void proj_vec(float (&a)[V], const NkbProj& s, long l
   } else {
     a[0] = proj_load(s, row, c);
   }
+}
+
+template <int V>
+__device__ __forceinline__ void pair_rows(float (&s)[V], const NkbBranch& br, long long t, int c) {
+  float a[V];
+#pragma unroll
+  for (int j = 0; j < V; ++j) a[j] = 0.f;
+#pragma unroll 4
+  for (int i = 0; i < br.top_k; ++i) {
+    const int pos = br.pair_pos[t * br.top_k + i];
+    const float w = br.pair_w[t * br.top_k + i];
+    float r[V];
+    proj_vec<V>(r, br.y, max(pos, 0), c);
+#pragma unroll
+    for (int j = 0; j < V; ++j) a[j] = pos >= 0 ? fmaf(w, r[j], a[j]) : a[j];
+  }
+#pragma unroll
+  for (int j = 0; j < V; ++j) s[j] = fmaf(br.scale, a[j], s[j]);
 }
 
 // PACKED: every projection is bf16 and aligned (prefill), which keeps the kernel at few registers and many CTAs per SM
@@ -87,36 +106,56 @@ gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
       uint2 y[2], g[2];
 #pragma unroll
       for (int b = 0; b < 2; ++b)
-        if (b < p.branches) {
-          y[b] = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.y[b].ptr) + t * p.y[b].ld + c);
-          g[b] = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.g[b].ptr) + t * p.g[b].ld + c);
+        if (b < p.branches && !p.br[b].pair_pos) {
+          y[b] = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.br[b].y.ptr) + t * p.br[b].y.ld + c);
+          if (p.br[b].g.ptr)
+            g[b] = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.br[b].g.ptr) + t * p.br[b].g.ld + c);
         }
 #pragma unroll
       for (int b = 0; b < 2; ++b)
         if (b < p.branches) {
-          const float4 bias = *reinterpret_cast<const float4*>(p.gbias[b] + c);
+          if (p.br[b].pair_pos) {
+            pair_rows<V>(s, p.br[b], t, c);
+            continue;
+          }
           const float2 y0 = unpack_bf16x2(y[b].x), y1 = unpack_bf16x2(y[b].y);
-          const float2 g0 = unpack_bf16x2(g[b].x), g1 = unpack_bf16x2(g[b].y);
-          s[0] += y0.x * sigmoid_f(g0.x + bias.x);
-          s[1] += y0.y * sigmoid_f(g0.y + bias.y);
-          s[2] += y1.x * sigmoid_f(g1.x + bias.z);
-          s[3] += y1.y * sigmoid_f(g1.y + bias.w);
+          if (p.br[b].g.ptr) {
+            const float4 bias = *reinterpret_cast<const float4*>(p.br[b].gbias + c);
+            const float2 g0 = unpack_bf16x2(g[b].x), g1 = unpack_bf16x2(g[b].y);
+            s[0] += y0.x * sigmoid_f(g0.x + bias.x);
+            s[1] += y0.y * sigmoid_f(g0.y + bias.y);
+            s[2] += y1.x * sigmoid_f(g1.x + bias.z);
+            s[3] += y1.y * sigmoid_f(g1.y + bias.w);
+          } else {
+            const float w = p.br[b].scale;
+            s[0] = fmaf(w, y0.x, s[0]);
+            s[1] = fmaf(w, y0.y, s[1]);
+            s[2] = fmaf(w, y1.x, s[2]);
+            s[3] = fmaf(w, y1.y, s[3]);
+          }
         }
     } else {
       float y[2][V], g[2][V];
 #pragma unroll
       for (int b = 0; b < 2; ++b)
-        if (b < p.branches) {
-          proj_vec<V>(y[b], p.y[b], t, c);
-          proj_vec<V>(g[b], p.g[b], t, c);
+        if (b < p.branches && !p.br[b].pair_pos) {
+          proj_vec<V>(y[b], p.br[b].y, t, c);
+          if (p.br[b].g.ptr) proj_vec<V>(g[b], p.br[b].g, t, c);
         }
 #pragma unroll
       for (int b = 0; b < 2; ++b)
         if (b < p.branches) {
-          float bias[V];
-          load_vec<V>(bias, p.gbias[b] + c);
+          if (p.br[b].pair_pos) {
+            pair_rows<V>(s, p.br[b], t, c);
+          } else if (p.br[b].g.ptr) {
+            float bias[V];
+            load_vec<V>(bias, p.br[b].gbias + c);
 #pragma unroll
-          for (int j = 0; j < V; ++j) s[j] += y[b][j] * sigmoid_f(g[b][j] + bias[j]);
+            for (int j = 0; j < V; ++j) s[j] += y[b][j] * sigmoid_f(g[b][j] + bias[j]);
+          } else {
+#pragma unroll
+            for (int j = 0; j < V; ++j) s[j] = fmaf(p.br[b].scale, y[b][j], s[j]);
+          }
         }
     }
 #pragma unroll
@@ -188,12 +227,7 @@ gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
   }
 }
 
-// kind 0: SiLU, 1: GELU in its tanh form, written with the exponential: (1 + tanh u) / 2 = 1 / (1 + exp(-2 u))
-__device__ __forceinline__ float gate_act(float z, int kind) {
-  if (kind == 0) return z / (1.f + expf(-z));
-  return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
-}
-
+// act(gate) * up, or act(gate) alone when up.ptr is null
 template <int V, typename OutT>
 __global__ void __launch_bounds__(256) gated_act_kernel(const __grid_constant__ NkbProj gate,
                                                         const __grid_constant__ NkbProj up, OutT* __restrict__ out,
@@ -207,15 +241,16 @@ __global__ void __launch_bounds__(256) gated_act_kernel(const __grid_constant__ 
     const int c = int(i % nv) * V;
     float g[V], u[V];
     if constexpr (V == 4) {
-      const float4 a = proj_load4(gate, r, c), b = proj_load4(up, r, c);
+      const float4 a = proj_load4(gate, r, c);
+      const float4 b = up.ptr ? proj_load4(up, r, c) : make_float4(1.f, 1.f, 1.f, 1.f);
       g[0] = a.x; g[1] = a.y; g[2] = a.z; g[3] = a.w;
       u[0] = b.x; u[1] = b.y; u[2] = b.z; u[3] = b.w;
     } else {
       g[0] = proj_load(gate, r, c);
-      u[0] = proj_load(up, r, c);
+      u[0] = up.ptr ? proj_load(up, r, c) : 1.f;
     }
 #pragma unroll
-    for (int j = 0; j < V; ++j) g[j] = gate_act(g[j], kind) * u[j];
+    for (int j = 0; j < V; ++j) g[j] = apply_act(g[j], kind) * u[j];
     OutT* o = out + r * inter + c;
     if constexpr (V == 4 && sizeof(OutT) == 2) {
       *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16x2(g[0], g[1]), pack_bf16x2(g[2], g[3]));
@@ -233,10 +268,10 @@ using namespace nkb;
 static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
 extern "C" int nkb_gated_residual(const float* x_in, const int* ids, const void* table, int table_bf16, int vocab,
-                                  float scale, int branches, const NkbProj* y, const NkbProj* g,
-                                  const float* const* gbias, const float* add_row, const float* add_mat, float* x_out,
-                                  int norms, const float* const* w, void* const* out, int out_bf16, int rows, int width,
-                                  int groups, float eps, void* stream) {
+                                  float scale, int branches, const NkbBranch* br, const float* add_row,
+                                  const float* add_mat, float* x_out, int norms, const float* const* w,
+                                  void* const* out, int out_bf16, int rows, int width, int groups, float eps,
+                                  void* stream) {
   if (rows <= 0) return 0;
   if (width <= 0 || width > 12000 || groups < 1 || groups > kGrMaxGroups || width % groups) return -2;
   if (branches < 0 || branches > 2 || norms < 0 || norms > 2 || (!x_in && (!ids || !table || vocab < 1))) return -2;
@@ -245,8 +280,8 @@ extern "C" int nkb_gated_residual(const float* x_in, const int* ids, const void*
   p.branches = branches; p.norms = norms;
   bool vec = width % 4 == 0 && (width / groups) % 4 == 0 && (!x_in || aligned16(x_in)) && (!x_out || aligned16(x_out));
   for (int b = 0; b < branches; ++b) {
-    p.y[b] = y[b]; p.g[b] = g[b]; p.gbias[b] = gbias[b];
-    vec = vec && proj_vec4_ok(y[b]) && proj_vec4_ok(g[b]) && aligned16(gbias[b]);
+    p.br[b] = br[b];
+    vec = vec && proj_vec4_ok(br[b].y) && proj_vec4_ok(br[b].g) && aligned16(br[b].gbias);
   }
   for (int n = 0; n < norms; ++n) {
     p.w[n] = w[n]; p.out[n] = out[n];
@@ -256,7 +291,7 @@ extern "C" int nkb_gated_residual(const float* x_in, const int* ids, const void*
   p.width = width; p.groups = groups; p.eps = eps;
   const size_t smem = size_t(width + groups) * sizeof(float);
   bool packed = vec && branches > 0;
-  for (int i = 0; i < branches; ++i) packed = packed && y[i].bf16 && g[i].bf16;
+  for (int i = 0; i < branches; ++i) packed = packed && br[i].y.bf16 && (br[i].g.bf16 || !br[i].g.ptr);
   // few rows: one vector per thread, so that every load of a row is in flight at once
   const int nv = vec ? width / 4 : width, most = packed || rows > 2 * 148 ? 256 : 1024;
   const int threads = nv >= most ? most : (nv < 64 ? 64 : (nv + 31) / 32 * 32);
@@ -277,7 +312,7 @@ extern "C" int nkb_gated_residual(const float* x_in, const int* ids, const void*
 extern "C" int nkb_gated_act(const NkbProj* gate, const NkbProj* up, void* out, int out_bf16, int rows, int inter,
                              int kind, void* stream) {
   if (rows <= 0 || inter <= 0) return 0;
-  if (kind < 0 || kind > 1) return -2;
+  if (kind < 0 || kind >= ACT_COUNT) return -2;
   const bool vec = inter % 4 == 0 && proj_vec4_ok(*gate) && proj_vec4_ok(*up) && aligned16(out);
   const long long n = (long long)rows * (vec ? inter / 4 : inter);
   const int blocks = int((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);

@@ -32,7 +32,7 @@ struct Gemm2Args {            // <= 128 bytes (see GemmArgs)
   int group_m;                // row tiles that share one sweep over the column tiles (L2 reuse)
   int gated;                  // B holds [gate; up] rows: the pair's first CTA loads gate rows, the second up rows
   int gate_off;               // row offset of the up half in B
-  int act;                    // gated: 0 = SiLU, 1 = GELU (tanh form)
+  int act;                    // gated: 0 = SiLU, 1 = GELU (tanh form); plain: 2 = squared ReLU
   long long ldo;
   void* out;
   const __nv_bfloat16* bias;
@@ -243,6 +243,13 @@ gemm2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CU
             if (cbase + j < args.n)
               v[j] = __float_as_uint(__uint_as_float(v[j]) + __bfloat162float(args.bias[cbase + j]));
         }
+        if (args.act == 2) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            const float r = fmaxf(__uint_as_float(v[j]), 0.f);
+            v[j] = __float_as_uint(r * r);
+          }
+        }
         const long long off = (long long)row * args.ldo + cbase;
         if (cbase + 32 <= args.n && ((off & 7) == 0)) {
           uint32_t pk[16];
@@ -305,11 +312,12 @@ static int g_pairs_last = 0;
 extern "C" int nkb_gemm_2cta_pairs() { return g_pairs_last; }
 
 // gated != 0: B holds [gate; up] (2 x n rows, the up half starting at row gate_off) and out[m, n] =
-// silu(A gate^T) * (A up^T); bias / residual are not applied in that mode.
+// silu(A gate^T) * (A up^T); bias / residual are not applied in that mode.  act 1: GELU in place of SiLU; 2 (not gated):
+// the square of the positive part of (A B^T + bias).
 extern "C" int nkb_gemm_bf16_2cta(const void* A, const void* B, void* out, int m, int n, int k, long long lda,
                                   long long ldb, long long ldo, const void* bias, const void* residual, int gated,
                                   int gate_off, int act, void* stream) {
-  if (act < 0 || act > 1) return -2;
+  if (act < 0 || act > 2 || (act == 2 && gated)) return -2;
   if (!status_word() && nkb_init() != 0) return -1;
   if (m <= 0 || n <= 0 || k <= 0) return -2;
   if ((k & 7) || (lda & 7) || (ldb & 7)) return -2;

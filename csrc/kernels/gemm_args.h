@@ -23,7 +23,7 @@ struct GemmArgs {
   int out_fp32;
   int bias_on_rows;
   int stages;
-  int act;              // gated epilogue: 0 = SiLU, 1 = GELU (tanh form)
+  int act;              // gated epilogue: 0 = SiLU, 1 = GELU (tanh form); plain: 2 = squared ReLU
   int weights_operand;  // 0 = A, 1 = B holds immutable weights (may be fetched before the dependency wait), -1 none
   long long ldo;
   long long split_stride;

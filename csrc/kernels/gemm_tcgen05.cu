@@ -169,7 +169,8 @@ extern "C" int nkb_gemm_bf16(const void* A, const void* B, void* out, int rows, 
                              const void* residual, int block_n, int max_ctas, int weights_operand, int ctas_per_sm,
                              int act, void* stream) {
   if (!status_word() && nkb_init() != 0) return -1;
-  if (act < 0 || act > 1) return -2;
+  if (act < 0 || act > 2) return -2;
+  if (act == 2 && (gated || transpose_out || splits > 1)) return -2;   // in the general epilogue of finished values only
   if (rows <= 0 || cols <= 0 || k <= 0) return -2;
   if ((k & 7) || (lda & 7) || (ldb & 7)) return -2;
   if (splits > 1 && !out_fp32) return -2;

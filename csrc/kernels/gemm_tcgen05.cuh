@@ -613,6 +613,13 @@ __device__ __forceinline__ bool gemm_bf16_body(const CUtensorMap& tmA, const CUt
                 v[j] = __float_as_uint(__uint_as_float(v[j]) + __bfloat162float(args.bias[cbase + j]));
           }
         }
+        if (args.act == 2) {       // plain product: square of the positive part
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            const float r = fmaxf(__uint_as_float(v[j]), 0.f);
+            v[j] = __float_as_uint(r * r);
+          }
+        }
         if constexpr (PUSH) {
           // stage the chunk (token j, feature quad * 32 + lane), then the four warps store it to every rank as
           // 16-byte pieces, 256 contiguous bytes per token.  cbase and cols_end are CTA-uniform, so the four

@@ -79,7 +79,8 @@ __global__ void moe_tiles_kernel(const int* __restrict__ offsets, int num_local,
 // Small batches (decode): one block counts, scans, assigns every pair its sorted position and
 // builds both tile schedules, replacing the count / scan / tile kernels and the memset.
 __global__ void moe_plan_small_kernel(const int* __restrict__ experts, int pairs, int expert_lo, int num_local,
-                                      int* __restrict__ offsets, int* __restrict__ pair_pos, int bn_a,
+                                      int* __restrict__ offsets, int* __restrict__ pair_pos,
+                                      int* __restrict__ row_token, int top_k, int bn_a,
                                       int* __restrict__ tiles_a, int* __restrict__ ntiles_a, int bn_b,
                                       int* __restrict__ tiles_b, int* __restrict__ ntiles_b) {
   griddep_wait();
@@ -121,7 +122,9 @@ __global__ void moe_plan_small_kernel(const int* __restrict__ experts, int pairs
   // deterministic order inside an expert is not needed: every pair's output row is independent
   for (int i = t; i < pairs; i += 1024) {
     const int e = experts[i] - expert_lo;
-    pair_pos[i] = (e >= 0 && e < num_local) ? off[e] + atomicAdd(&cnt[e], 1) : -1;
+    const int pos = (e >= 0 && e < num_local) ? off[e] + atomicAdd(&cnt[e], 1) : -1;
+    pair_pos[i] = pos;
+    if (row_token && pos >= 0) row_token[pos] = i / top_k;
   }
 }
 
@@ -143,7 +146,7 @@ __global__ void moe_gather_kernel(const int* __restrict__ pair_pos, int top_k, c
 __global__ void moe_scatter_kernel(const int* __restrict__ experts, int pairs, int top_k, int expert_lo,
                                    int num_local, const int* __restrict__ offsets, int* __restrict__ cursors,
                                    const __nv_bfloat16* __restrict__ x, int hidden, __nv_bfloat16* __restrict__ x_sorted,
-                                   int* __restrict__ pair_pos) {
+                                   int* __restrict__ pair_pos, int* __restrict__ row_token) {
   griddep_wait();
   griddep_launch();
   __shared__ int s_pos;
@@ -153,8 +156,10 @@ __global__ void moe_scatter_kernel(const int* __restrict__ experts, int pairs, i
     int pos = -1;
     if (e >= 0 && e < num_local) pos = offsets[e] + atomicAdd(&cursors[e], 1);
     pair_pos[pair] = pos;
+    if (row_token && pos >= 0) row_token[pos] = pair / top_k;
     s_pos = pos;
   }
+  if (!x) return;
   __syncthreads();
   const int pos = s_pos;
   if (pos < 0) return;
@@ -199,19 +204,20 @@ using namespace nkb;
 
 // experts [tokens * top_k] int32 (global expert ids).  Workspace (device, int32): counts[num_local],
 // offsets[num_local + 1], cursors[num_local], pair_pos[tokens * top_k].  x_sorted must hold
-// tokens * top_k rows.  After the call offsets / pair_pos / x_sorted are valid on the stream.
+// tokens * top_k rows.  After the call offsets / pair_pos / x_sorted are valid on the stream.  x == nullptr: the rows are
+// not gathered (any width); row_token [tokens * top_k], when given, names the token of every sorted row instead.
 extern "C" int nkb_moe_dispatch(const int* experts, int tokens, int top_k, int expert_lo, int num_local, const void* x,
                                 int hidden, void* x_sorted, int* counts, int* offsets, int* cursors, int* pair_pos,
-                                int bn_a, int* tiles_a, int* ntiles_a, int bn_b, int* tiles_b, int* ntiles_b,
+                                int* row_token, int bn_a, int* tiles_a, int* ntiles_a, int bn_b, int* tiles_b, int* ntiles_b,
                                 void* stream) {
   if (tokens <= 0) return 0;
-  if (num_local > 1024 || (hidden & 7) || bn_a <= 0 || bn_b <= 0) return -2;
+  if (num_local > 1024 || (x && (hidden & 7)) || (!x && !row_token) || bn_a <= 0 || bn_b <= 0) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const int pairs = tokens * top_k;
   if (pairs <= 8192) {
     int rc = launch_pdl(moe_plan_small_kernel, dim3(1), dim3(1024), 0, s, experts, pairs, expert_lo, num_local, offsets,
-                        pair_pos, bn_a, tiles_a, ntiles_a, bn_b, tiles_b, ntiles_b);
-    if (rc) return rc;
+                        pair_pos, row_token, top_k, bn_a, tiles_a, ntiles_a, bn_b, tiles_b, ntiles_b);
+    if (rc || !x) return rc;
     return launch_pdl(moe_gather_kernel, dim3(pairs), dim3(128), 0, s, (const int*)pair_pos, top_k,
                       (const __nv_bfloat16*)x, hidden, (__nv_bfloat16*)x_sorted);
   }
@@ -226,7 +232,7 @@ extern "C" int nkb_moe_dispatch(const int* experts, int tokens, int top_k, int e
                   bn_b, tiles_b, ntiles_b);
   if (rc) return rc;
   return launch_pdl(moe_scatter_kernel, dim3(pairs), dim3(128), 0, s, experts, pairs, top_k, expert_lo, num_local,
-                    (const int*)offsets, cursors, (const __nv_bfloat16*)x, hidden, (__nv_bfloat16*)x_sorted, pair_pos);
+                    (const int*)offsets, cursors, (const __nv_bfloat16*)x, hidden, (__nv_bfloat16*)x_sorted, pair_pos, row_token);
 }
 
 extern "C" int nkb_moe_combine(const void* y_sorted, const int* pair_pos, const float* weights, int tokens, int top_k,

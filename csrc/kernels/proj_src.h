@@ -11,3 +11,14 @@ struct NkbProj {
   int splits;               // 1 for finished values
   int bf16;                 // 1 = bf16 values, 0 = fp32
 };
+
+// One addend of a residual update: scale * y, with a gate sigmoid(g + gbias) on it when g.ptr is set, or (pair_pos set) the
+// weighted sum of a token's top_k rows of y, pair_w[t, j] * y[pair_pos[t, j]] (routed experts).
+struct NkbBranch {
+  NkbProj y, g;
+  const float* gbias;
+  const int* pair_pos;
+  const float* pair_w;
+  int top_k;
+  float scale;
+};

@@ -224,11 +224,14 @@ __global__ void __launch_bounds__(1024) sample_kernel(const void* __restrict__ l
 // MoE router: one warp per token, num_experts <= 1024.
 //   mode 0: softmax over all experts -> top-k -> divide by the selected sum
 //   mode 1: top-k on raw logits -> softmax over the selected
+// groups > 0 (mode 0): experts form `groups` equal runs of neighbours; only the experts of the `keep` runs with the
+// largest single score take part.  The weights are multiplied by `scale`.
 // ---------------------------------------------------------------------------
 // logits may be bf16 / fp32 [tokens, E] or fp32 split-K partials [splits, tokens, E] (summed here, plus bias)
 __global__ void router_topk_kernel(const void* __restrict__ logits, int is_fp32, int splits, long long split_stride,
                                    const __nv_bfloat16* __restrict__ bias, float* __restrict__ weights,
-                                   int* __restrict__ experts, int tokens, int num_experts, int top_k, int mode) {
+                                   int* __restrict__ experts, int tokens, int num_experts, int top_k, int mode,
+                                   int groups, int keep, float scale) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   griddep_wait();
@@ -258,8 +261,33 @@ __global__ void router_topk_kernel(const void* __restrict__ logits, int is_fp32,
     float s = 0.f;
 #pragma unroll
     for (int j = 0; j < kPer; ++j)
-      if (j < per && v[j] > -FLT_MAX) s += __expf(v[j] - mx);
+      if (j < per && v[j] > -FLT_MAX) s += expf(v[j] - mx);
     denom = warp_sum(s);
+  }
+  if (groups > 0) {
+    // `keep` passes over the groups' best scores: the best remaining expert names the next group
+    const int n = num_experts / groups;
+    unsigned open_bits = 0u;                     // this lane's experts (bit j) whose group is kept
+    for (int r = 0; r < keep; ++r) {
+      float best = -FLT_MAX;
+      int bi = 0x7fffffff;
+#pragma unroll
+      for (int j = 0; j < kPer; ++j)
+        if (j < per && !((open_bits >> j) & 1u)) argmax_combine(best, bi, v[j], j * 32 + lane);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        float ov = __shfl_xor_sync(0xffffffffu, best, o);
+        int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        argmax_combine(best, bi, ov, oi);
+      }
+      const int g = bi / n;
+#pragma unroll
+      for (int j = 0; j < kPer; ++j)
+        if (j < per && (j * 32 + lane) / n == g) open_bits |= 1u << j;
+    }
+#pragma unroll
+    for (int j = 0; j < kPer; ++j)
+      if (!((open_bits >> j) & 1u)) v[j] = -FLT_MAX;
   }
   float sel_sum = 0.f;
   float my_w = 0.f;
@@ -277,7 +305,7 @@ __global__ void router_topk_kernel(const void* __restrict__ logits, int is_fp32,
       argmax_combine(best, bi, ov, oi);
     }
     // mode 0 weight = softmax prob; mode 1 weight = exp(logit - max selected) (first pick is the max)
-    const float wgt = (mode == 0) ? __expf(best - mx) / denom : __expf(best - mx);
+    const float wgt = (mode == 0) ? expf(best - mx) / denom : expf(best - mx);
     sel_sum += wgt;
     if (lane == r % 32 && r / 32 == 0) { my_w = wgt; my_e = bi; }
     if ((bi & 31) == lane) {
@@ -287,7 +315,7 @@ __global__ void router_topk_kernel(const void* __restrict__ logits, int is_fp32,
     }
   }
   if (lane < top_k) {
-    weights[(long long)warp * top_k + lane] = my_w / sel_sum;
+    weights[(long long)warp * top_k + lane] = my_w / (sel_sum + 1e-20f) * scale;
     experts[(long long)warp * top_k + lane] = my_e;
   }
 }
@@ -312,15 +340,17 @@ extern "C" int nkb_sample(const void* logits, int is_fp32, int* out_ids, int row
 }
 
 extern "C" int nkb_router_topk(const void* logits, int is_fp32, int splits, long long split_stride, const void* bias,
-                               float* weights, int* experts, int tokens, int num_experts, int top_k, int mode,
-                               void* stream) {
+                               float* weights, int* experts, int tokens, int num_experts, int top_k, int mode, int groups,
+                               int keep, float scale, void* stream) {
   if (tokens <= 0) return 0;
   if (num_experts > 1024 || top_k > 32 || top_k > num_experts) return -2;
+  if (groups > 0 && (mode != 0 || num_experts % groups || keep < 1 || keep > groups || top_k > num_experts / groups * keep))
+    return -2;
   const int threads = 128;
   const int blocks = (tokens * 32 + threads - 1) / threads;
   if (splits < 1) splits = 1;
   if (splits > 1 && !is_fp32) return -2;
   return launch_pdl(router_topk_kernel, dim3(blocks), dim3(threads), 0, reinterpret_cast<cudaStream_t>(stream), logits,
                     is_fp32, splits, split_stride, (const __nv_bfloat16*)bias, weights, experts, tokens, num_experts,
-                    top_k, mode);
+                    top_k, mode, groups, keep, scale);
 }

@@ -53,10 +53,71 @@ class RecurrenceSpec:
 
 
 @dataclass(frozen=True)
+class LinearAttentionSpec:
+    """Gated linear attention: `dim` key channels by `vdim` values per head, decays sigmoid(z)^(1 / tau) from a low-rank z
+    (rank 0: as the weights have it)."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float = 16.0
+    rank: int = 0
+    kind = "gla"
+
+
+@dataclass(frozen=True)
+class TimeMixSpec:
+    """RWKV-style time mixing: every projection reads its own mix of the token and the one before it, `dim` by `dim` states
+    with data-dependent decays and a bonus for the current token."""
+    heads: int
+    dim: int
+    rank: int = 0
+    kind = "rwkv"
+
+
+@dataclass(frozen=True)
+class WindowAttentionSpec:
+    """Grouped-query attention without rotation over the last `window` tokens (0: all), queries and keys normed over all
+    heads together, sigmoid gate on the heads."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int
+    kind = "window"
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Attention and time mixing side by side on the same input, summed with constant weights."""
+    left: WindowAttentionSpec
+    right: TimeMixSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+    kind = "parallel"
+
+
+@dataclass(frozen=True)
+class ExpertsSpec:
+    """Routed SiLU-gated feed-forwards of width `ff`: softmax over all experts, the `top` best of the `keep` best of
+    `groups` equal groups (0: all), weights normalised and multiplied by `scale`."""
+    experts: int
+    top: int
+    ff: int
+    groups: int = 0
+    keep: int = 0
+    scale: float = 1.0
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[MapsAttentionSpec, RecurrenceSpec]
-    ff: int = 0                      # 0: no feed-forward
+    """block "gated": mixer and gated feed-forward beside each other, a sigmoid gate on both results; "pre-norm": the
+    mixer, then the feed-forward (plain `act`, or `experts`), each added to the residual."""
+    mixer: Union[MapsAttentionSpec, RecurrenceSpec, LinearAttentionSpec, ParallelSpec]
+    ff: int = 0                      # 0: no dense feed-forward
     act: str = "gelu_tanh"
+    block: str = "gated"
+    experts: Optional[ExpertsSpec] = None
 
 
 @dataclass(frozen=True)
@@ -107,6 +168,8 @@ class ModelConfig:
     loop: Optional[LoopSpec] = None
     embedding_scale: float = 1.0
     norm_groups: int = 1
+    norm_offset: float = 0.0              # added to the stored weights of the layer and final norms
+    tie_embeddings: bool = False          # logits from the embedding table
 
     @property
     def q_size(self) -> int:
@@ -154,15 +217,9 @@ class ModelConfig:
     def param_count(self) -> int:
         h = self.hidden_size
         if self.layers is not None:
-            n = 2 * self.vocab_size * h + h + (self.loop.times * h if self.loop else 0)
-            for l in self.layers:
-                m = l.mixer
-                if m.kind == "hgrn2":
-                    n += h * m.heads * (2 * m.dim + 2 * m.vdim) + 2 * m.heads * m.dim + m.vdim
-                else:
-                    n += h * (2 * m.dim * (m.heads + m.kv_heads) + m.vdim * (m.heads + m.kv_heads)) + 4 * m.dim
-                n += h + h * h + h + ((3 * l.ff + h + 2) * h if l.ff else 0)
-            return n
+            from .weights import hybrid_weight_shapes
+
+            return sum(math.prod(shape) for shape in hybrid_weight_shapes(self).values())
         attn = h * (self.q_size + 2 * self.kv_size) + self.q_size * h
         if self.is_moe:
             ffn = self.num_experts * 3 * h * self.moe_intermediate_size + h * self.num_experts
@@ -283,6 +340,61 @@ def tolenex_shape(width: int, *, layers: int, heads: int, kv_heads: int, ff: int
         specs.append(LayerSpec(mixer, ff))
     base = dict(name="tolenex", vocab_size=vocab, hidden_size=width, num_layers=layers, rms_eps=1e-5,
                 norm_groups=groups, layers=specs, loop=loop, embedding_scale=1.0, max_position=0)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+def mumilorn_config(raw: dict, **kw) -> ModelConfig:
+    """`ModelConfig` of a Mumilorn config.json."""
+
+    def mixer_of(kind, m):
+        if kind == "gla":
+            return LinearAttentionSpec(m["heads"], m["dim"], m["vdim"], m["tau"])
+        if kind == "parallel":
+            a, r = m["left"], m["right"]
+            return ParallelSpec(
+                WindowAttentionSpec(a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["scale"], a["mask"]["size"]),
+                TimeMixSpec(r["heads"], r["dim"]), m["left_scale"], m["right_scale"])
+        raise ValueError(f"unknown layer type {kind!r}")
+
+    layers = []
+    for l in raw["layers"]:
+        mlp, ff, experts = l.get("mlp"), 0, None
+        if mlp is not None:
+            if mlp["kind"] == "dense":
+                ff = mlp["ff"]
+            elif mlp["kind"] == "moe":
+                r = mlp["router"]
+                g = r.get("groups") or {}
+                experts = ExpertsSpec(r["experts"], r["top"], mlp["expert"]["ff"], g.get("count", 0), g.get("keep", 0),
+                                      r["scale"])
+            else:
+                raise ValueError(f"unknown feed-forward kind {mlp['kind']!r}")
+        layers.append(LayerSpec(mixer_of(l["type"], l["mixer"]), ff, "relu2", "pre-norm", experts))
+    base = dict(name="mumilorn", vocab_size=raw["vocab"], hidden_size=raw["width"], num_layers=len(layers),
+                rms_eps=raw["norm"]["eps"], layers=layers, norm_offset=1.0, tie_embeddings=True, max_position=0)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+def mumilorn_shape(width: int, *, layers: int, heads: int, kv_heads: int, ff: int, vocab: int = 32000, dim: int = 128,
+                   window: int = 1024, rank: int = 64, parallel_every: int = 2, experts: int = 0, top: int = 0,
+                   expert_ff: int = 0, groups: int = 0, keep: int = 0, moe_every: int = 2, **kw) -> ModelConfig:
+    """A Mumilorn configuration of regular shape: every `parallel_every`-th layer has the parallel mixer, the others gated
+    linear attention; with experts, every `moe_every`-th feed-forward is routed."""
+    specs = []
+    for i in range(layers):
+        if i % parallel_every == parallel_every - 1:
+            mixer = ParallelSpec(WindowAttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, window),
+                                 TimeMixSpec(heads, dim, rank), 0.7, 0.7)
+        else:
+            mixer = LinearAttentionSpec(heads, dim, dim, 16.0, rank)
+        if experts and i % moe_every == moe_every - 1:
+            specs.append(LayerSpec(mixer, 0, "relu2", "pre-norm", ExpertsSpec(experts, top, expert_ff, groups, keep, 1.0)))
+        else:
+            specs.append(LayerSpec(mixer, ff, "relu2", "pre-norm"))
+    base = dict(name="mumilorn", vocab_size=vocab, hidden_size=width, num_layers=layers, rms_eps=1e-6, layers=specs,
+                norm_offset=1.0, tie_embeddings=True, max_position=0)
     base.update(kw)
     return ModelConfig(**base)
 

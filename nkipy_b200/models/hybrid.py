@@ -1,15 +1,14 @@
-"""Decoder whose layers are listed one by one: attention with score maps or a linear recurrence, each beside a dense
-feed-forward, around an fp32 residual stream (the Tolenex design).
+"""Decoders whose layers are listed one by one: each layer has its own token mixer (models/mixers.py) and feed-forward,
+around an fp32 residual stream.  Two kinds of layer:
 
-A layer reads the residual once and updates it once:
+    gated (Tolenex)       h1 = norm1(x), h2 = norm2(x)
+                          x <- x + sigmoid(W_g1 h1 + b1) * mixer(h1) + sigmoid(W_g2 h2 + b2) * feed_forward(h2)
+    pre-norm (Mumilorn)   x <- x + mixer(norm1(x)),   then   x <- x + feed_forward(norm2(x))
 
-    h1 = norm1(x), h2 = norm2(x)
-    x <- x + sigmoid(W_g1 h1 + b1) * mixer(h1) + sigmoid(W_g2 h2 + b2) * feed_forward(h2)
-
-so everything between two residual updates hangs on two input projections (queries / keys / values / gate of the
-mixer; gate / up / gate of the feed-forward) and two output projections, and one kernel per layer sums the
-gated branches, applies what precedes a repeated pass of a looped block and norms the result twice
-(`ops.gated_residual`).  The model plugs into the same engine, paged cache and decode graph as `TransformerLM`.
+A layer is a list of stages; a stage reads norms of the residual and returns the branches that are added to it.  One
+kernel per stage (`ops.gated_residual`) sums the branches, applies what precedes a repeated pass of a looped block and
+norms the result for the next stage.  The model plugs into the same engine, paged cache and decode graph as
+`TransformerLM`.
 
 Batches of at most 128 tokens (decode steps, small mixed steps) run their projections as split-K GEMMs whose fp32
 partial sums the next kernel adds up; larger ones as tiled GEMMs with bf16 results and the activation in
@@ -26,51 +25,118 @@ from typing import Dict, List, Optional
 import torch
 
 from .. import ops
-from ..ops import MapsSpec, Proj
-from ..ops.mixers import hgrn2_state_shape
+from ..ops import Branch, Proj
 from ..parallel.comm import TPGroup
 from .config import LayerSpec, ModelConfig, RopeSpec, rope_frequencies
-from .kv_cache import KVLayer, PagedKVCache, StateLayer
+from .kv_cache import PagedKVCache
+from .mixers import MIXERS, Tensors
+from .moe import RoutedExperts
 from .transformer import pick_splits
 
 SMALL_BATCH = 128
 
 
-class HybridLayer:
-    """Device weights of one layer, input projections stacked: w_in1 = [mixer inputs; gate 1], w_in2 = [gate; up; gate 2]."""
+class Stage:
+    """norms: weights of the residual's norms it reads; run(h, entry, cache, batch) -> branches."""
+    __slots__ = ("norms", "run")
 
-    def __init__(self, cfg: ModelConfig, spec: LayerSpec, index: int, get, dtype: torch.dtype):
-        p = f"l{index}."
-        m = spec.mixer
-        f32 = lambda name: get(name).float().contiguous()
-        mat = lambda *names: torch.cat([get(n).to(dtype) for n in names]).contiguous()
-        self.spec = spec
-        self.norms = [f32(p + "norm1")] + ([f32(p + "norm2")] if spec.ff else [])
-        if m.kind == "hgrn2":
-            self.w_in1 = mat(p + "mix.q", p + "mix.f", p + "mix.v", p + "rg1")
-            self.widths = [m.heads * m.dim, m.heads * m.dim, m.heads * m.vdim]
-            self.f_bias, self.lower, self.head_norm = f32(p + "mix.f.b"), f32(p + "mix.lower"), f32(p + "mix.norm")
-        else:
-            self.w_in1 = mat(p + "mix.q", p + "mix.k", p + "mix.v", p + "rg1")
-            self.widths = [m.heads * 2 * m.dim, m.kv_heads * 2 * m.dim, m.kv_heads * m.vdim]
-            dot = lambda a, b: float(torch.exp((get(p + "mix." + a).double() * get(p + "mix." + b).double()).sum()))
-            lam = dot("lq1", "lk1") - dot("lq2", "lk2") + m.diff
-            self.maps = MapsSpec(m.heads, m.kv_heads, m.dim, m.vdim, m.scale, maps=2, softcap=m.softcap, lam=lam,
-                                 out_scale=1.0 - m.diff, eps=cfg.rms_eps, tiled=dtype == torch.bfloat16)
-        self.w_o = mat(p + "mix.o")
-        self.gate_bias = [f32(p + "rg1.b")]
+    def __init__(self, norms, run):
+        self.norms, self.run = norms, run
+
+
+class GatedLayer:
+    """Mixer and gated feed-forward beside each other.  Input projections stacked: w_in1 = [mixer inputs; gate 1],
+    w_in2 = [gate; up; gate 2]."""
+
+    def __init__(self, model: "HybridLM", spec: LayerSpec, t: Tensors):
+        cfg = model.cfg
+        self.model, self.spec, self.width = model, spec, cfg.hidden_size
+        self.mixer = MIXERS[spec.mixer.kind](spec.mixer, t.under("mix."), cfg.rms_eps)
+        self.w_in1 = torch.cat([self.mixer.w_in, t.mat("rg1")]).contiguous()
+        self.mixer.w_in = None
+        self.gate_bias = [t.f32("rg1.b")]
+        norms = [t.f32("norm1", cfg.norm_offset)]
         if spec.ff:
-            self.w_in2 = mat(p + "mlp.gate", p + "mlp.up", p + "rg2")
-            self.w_down = mat(p + "mlp.down")
-            self.gate_bias.append(f32(p + "rg2.b"))
-        if sum(self.widths) + cfg.hidden_size != self.w_in1.shape[0]:
-            raise ValueError(f"layer {index}: projection sizes do not fit the configuration")
+            norms.append(t.f32("norm2", cfg.norm_offset))
+            self.w_in2 = t.mat("mlp.gate", "mlp.up", "rg2")
+            self.w_down = t.mat("mlp.down")
+            self.gate_bias.append(t.f32("rg2.b"))
+        if sum(self.mixer.widths) + cfg.hidden_size != self.w_in1.shape[0]:
+            raise ValueError("projection sizes do not fit the configuration")
+        self.stages = [Stage(norms, self._run)]
 
-    def cache_layer(self):
-        m = self.spec.mixer
-        if m.kind == "hgrn2":
-            return StateLayer(hgrn2_state_shape(m.heads, m.dim, m.vdim))
-        return KVLayer(m.kv_heads, self.maps.maps * self.maps.dim_p, self.maps.vdim_p)
+    def weights(self):
+        return [self.w_in1, self.mixer.w_o] + ([self.w_in2, self.w_down] if self.spec.ff else [])
+
+    def _feed_forward(self, h: torch.Tensor):
+        """(down projection, gate slice) of the feed-forward branch."""
+        ff, width, m = self.spec.ff, self.width, self.model
+        if x_small(h):
+            y = m.project(h, self.w_in2)
+            act = ops.gated_act(Proj(y, 0, ff), Proj(y, ff, ff), self.spec.act, dtype=h.dtype)
+            gate = Proj(y, 2 * ff, width)
+        else:
+            act = ops.linear(h, self.w_in2[:2 * ff], gated=True, act=self.spec.act, swap=False)
+            gate = Proj(ops.linear(h, self.w_in2[2 * ff:], swap=False), 0, width)
+        return Proj(m.project(act, self.w_down), 0, width), gate
+
+    def _run(self, h, entry, cache, b) -> List[Branch]:
+        m, width = self.model, self.width
+        y = m.project(h[0], self.w_in1)
+        mixed = self.mixer.run(m, y, h[0], entry, cache, b)
+        branches = [Branch(Proj(m.project(mixed, self.mixer.w_o), 0, width), Proj(y, sum(self.mixer.widths), width),
+                           self.gate_bias[0])]
+        if self.spec.ff:
+            branches.append(Branch(*self._feed_forward(h[1]), self.gate_bias[1]))
+        return branches
+
+
+class DenseMLP:
+    """down(act(up h))."""
+
+    def __init__(self, act: str, t: Tensors):
+        self.act, self.up, self.down = act, t.mat("up"), t.mat("down")
+
+    def weights(self):
+        return [self.up, self.down]
+
+    def run(self, model: "HybridLM", h: torch.Tensor) -> Branch:
+        if x_small(h):
+            a = ops.activation(Proj(model.project(h, self.up), 0, self.up.shape[0]), self.act, dtype=h.dtype)
+        else:
+            a = ops.linear(h, self.up, swap=False, out_act=self.act)
+        return Branch(Proj(model.project(a, self.down), 0, h.shape[1]))
+
+
+class PreNormLayer:
+    """Mixer, then feed-forward (dense or routed), each on its own norm of the residual."""
+
+    def __init__(self, model: "HybridLM", spec: LayerSpec, t: Tensors):
+        cfg = model.cfg
+        self.model, self.width = model, cfg.hidden_size
+        self.mixer = MIXERS[spec.mixer.kind](spec.mixer, t.under("mix."), cfg.rms_eps)
+        self.mlp = None
+        if spec.experts is not None:
+            self.mlp = RoutedExperts(spec.experts, t.under("mlp."))
+        elif spec.ff:
+            self.mlp = DenseMLP(spec.act, t.under("mlp."))
+        if self.mixer.w_in is not None and sum(self.mixer.widths) != self.mixer.w_in.shape[0]:
+            raise ValueError("projection sizes do not fit the configuration")
+        self.stages = [Stage([t.f32("norm1", cfg.norm_offset)], self._mix)]
+        if self.mlp is not None:
+            self.stages.append(Stage([t.f32("norm2", cfg.norm_offset)], lambda h, *_: [self.mlp.run(model, h[0])]))
+
+    def weights(self):
+        ws = [self.mixer.w_in, self.mixer.w_o, getattr(getattr(self.mixer, "right", None), "w_each", None)]
+        return [w for w in ws if w is not None] + (self.mlp.weights() if self.mlp is not None else [])
+
+    def _mix(self, h, entry, cache, b) -> List[Branch]:
+        m = self.model
+        y = m.project(h[0], self.mixer.w_in) if self.mixer.w_in is not None else None
+        return [Branch(Proj(m.project(self.mixer.run(m, y, h[0], entry, cache, b), self.mixer.w_o), 0, self.width))]
+
+
+LAYERS = {"gated": GatedLayer, "pre-norm": PreNormLayer}
 
 
 class HybridLM:
@@ -88,39 +154,45 @@ class HybridLM:
         self.device = torch.device(device if device is not None else weights["embed"].device)
         get = lambda name: weights[name].to(self.device)
         self.embed = get("embed").to(dtype).contiguous()
-        self.head = get("head").to(dtype).contiguous()
-        self.final_norm = get("final.norm").float().contiguous()
-        self.layers: List[HybridLayer] = [HybridLayer(cfg, s, i, get, dtype) for i, s in enumerate(cfg.layers)]
+        self.head = self.embed if cfg.tie_embeddings else get("head").to(dtype).contiguous()
+        self.final_norm = (get("final.norm").float() + cfg.norm_offset).contiguous()
+        self.layers = [LAYERS[s.block](self, s, Tensors(get, f"l{i}.", dtype)) for i, s in enumerate(cfg.layers)]
         self.runs = cfg.layer_runs()
+        self.entry = []                      # first cache entry of every run
+        n = 0
+        for i, _ in self.runs:
+            self.entry.append(n)
+            n += len(self.layers[i].mixer.entries())
         self.loop_step = get("loop.step").float().contiguous() if cfg.loop else None
         self._rope: Dict[RopeSpec, torch.Tensor] = {}
+        self._offsets: Dict[tuple, torch.Tensor] = {}
 
     # ------------------------------------------------------------------ cache
     def new_cache(self, num_blocks: int, max_batch: int, max_seq_len: int,
                   enable_prefix_sharing: bool = True) -> PagedKVCache:
         max_blocks = (max_seq_len + self.cfg.block_size - 1) // self.cfg.block_size
         self._extend_rope(max_blocks * self.cfg.block_size)
-        return PagedKVCache.for_layers([self.layers[i].cache_layer() for i, _ in self.runs], num_blocks, max_batch,
-                                       max_blocks, self.device, self.dtype, enable_prefix_sharing)
+        entries = [e for i, _ in self.runs for e in self.layers[i].mixer.entries()]
+        return PagedKVCache.for_layers(entries, num_blocks, max_batch, max_blocks, self.device, self.dtype,
+                                       enable_prefix_sharing)
 
     def _extend_rope(self, positions: int) -> None:
         """cos / sin tables [positions, dims] of every rotation the layers use."""
-        for layer in self.layers:
-            if layer.spec.mixer.kind != "attention":
-                continue
-            rope = layer.spec.mixer.rope
-            if rope not in self._rope or self._rope[rope].shape[0] < positions:
+        for layer in self.cfg.layers:
+            rope = getattr(layer.mixer, "rope", None)
+            if rope is not None and (rope not in self._rope or self._rope[rope].shape[0] < positions):
                 freq, mult = rope_frequencies(rope)
                 self._rope[rope] = ops.rope_table(rope.dims, positions, inv_freq=freq, scaling=mult, device=self.device)
 
+    def rope_table(self, rope: RopeSpec) -> torch.Tensor:
+        return self._rope[rope]
+
     def weight_bytes(self) -> int:
-        ts = [self.embed, self.head]
-        for l in self.layers:
-            ts += [l.w_in1, l.w_o] + ([l.w_in2, l.w_down] if l.spec.ff else [])
+        ts = [self.embed, self.head] + [t for l in self.layers for t in l.weights()]
         return sum(t.numel() * t.element_size() for t in ts)
 
     # ------------------------------------------------------------------ layers
-    def _project(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    def project(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
         """fp32 (split-K partials) for small batches, bf16 for large ones, fp32 for 32-bit models."""
         if x.dtype == torch.float32:
             return ops.linear(x, w)
@@ -129,43 +201,31 @@ class HybridLM:
             return ops.linear(x, w, splits=splits) if splits > 1 else ops.linear(x, w, fp32_out=True)
         return ops.linear(x, w, swap=False)
 
-    def _feed_forward(self, layer: HybridLayer, h: torch.Tensor):
-        """(down projection, gate slice) of the feed-forward branch."""
-        ff, width = layer.spec.ff, self.cfg.hidden_size
-        if x_small(h):
-            y = self._project(h, layer.w_in2)
-            act = ops.gated_act(Proj(y, 0, ff), Proj(y, ff, ff), layer.spec.act, dtype=h.dtype)
-            gate = Proj(y, 2 * ff, width)
-        else:
-            act = ops.linear(h, layer.w_in2[:2 * ff], gated=True, act=layer.spec.act, swap=False)
-            gate = Proj(ops.linear(h, layer.w_in2[2 * ff:], swap=False), 0, width)
-        return Proj(self._project(act, layer.w_down), 0, width), gate
-
-    def _mixer(self, layer: HybridLayer, y: torch.Tensor, run: int, cache: PagedKVCache, b: "Batch") -> torch.Tensor:
-        m = layer.spec.mixer
-        c1, c2 = layer.widths[0], layer.widths[0] + layer.widths[1]
-        first, second, third = Proj(y, 0, c1), Proj(y, c1, layer.widths[1]), Proj(y, c2, layer.widths[2])
-        if m.kind == "hgrn2":
-            return ops.hgrn2(first, second, third, layer.f_bias, layer.lower, layer.head_norm, cache.state[run],
-                             b.context_lens, heads=m.heads, dim=m.dim, vdim=m.vdim, eps=self.cfg.rms_eps,
-                             q_start=b.q_start, q_lens=b.q_lens, rows=b.rows, dtype=self.dtype)
-        q = ops.maps_append(layer.maps, first, second, third, self._rope[m.rope], b.positions, b.slots, cache.k[run],
-                            cache.v[run])
-        return ops.maps_attention(layer.maps, q, cache.k[run], cache.v[run], b.block_table, b.context_lens,
-                                  q_start=b.q_start, q_lens=b.q_lens, max_q_len=b.max_q_len)
+    def project_each(self, x: torch.Tensor, w: torch.Tensor) -> List[Proj]:
+        """x[i] @ w[i].T for x [M, T, K], w [M, N, K]: one grouped product for small bf16 batches."""
+        M, T, K = x.shape
+        N = w.shape[1]
+        if x_small(x[0]) and x.dtype == torch.bfloat16 and K % 8 == 0:
+            if (M, T) not in self._offsets:
+                self._offsets[M, T] = torch.arange(0, M * T + 1, T, dtype=torch.int32, device=x.device)
+            y = ops.grouped_linear(x.reshape(M * T, K), w, self._offsets[M, T], max_rows_per_group=T)
+            return [Proj(y[i * T:(i + 1) * T], 0, N) for i in range(M)]
+        return [Proj(self.project(x[i], w[i]), 0, N) for i in range(M)]
 
     def _forward(self, ids: torch.Tensor, cache: PagedKVCache, b: "Batch", return_hidden: bool = False):
-        cfg, width = self.cfg, self.cfg.hidden_size
+        cfg = self.cfg
         norm = dict(groups=cfg.norm_groups, eps=cfg.rms_eps, dtype=self.dtype)
         start = cfg.loop.start if cfg.loop else -1
+        plan = [(r, s) for r, (i, _) in enumerate(self.runs) for s in range(len(self.layers[i].stages))]
 
-        def ahead(r):
-            """What is added to the residual before run r, and the norms that read it."""
-            if r == len(self.runs):
+        def ahead(n):
+            """What is added to the residual before stage n of the plan, and the norms that read it."""
+            if n == len(plan):
                 return dict(norms=[self.final_norm])
+            r, s = plan[n]
             i, t = self.runs[r]
-            pre = dict(norms=self.layers[i].norms)
-            if t >= 0 and i == start:
+            pre = dict(norms=self.layers[i].stages[s].norms)
+            if s == 0 and t >= 0 and i == start:
                 pre["add_row"] = self.loop_step[t]
                 if t > 0:
                     pre["add_mat"] = embedded
@@ -178,17 +238,12 @@ class HybridLM:
         if "add_row" in first:
             x, h = ops.gated_residual(x, **first, **norm)
         taps = []
-        for r, (i, _) in enumerate(self.runs):
-            layer = self.layers[i]
-            y1 = self._project(h[0], layer.w_in1)
-            mixed = self._mixer(layer, y1, r, cache, b)
-            branches = [(Proj(self._project(mixed, layer.w_o), 0, width), Proj(y1, sum(layer.widths), width),
-                         layer.gate_bias[0])]
-            if layer.spec.ff:
-                branches.append((*self._feed_forward(layer, h[1]), layer.gate_bias[1]))
-            if return_hidden:
+        for n, (r, s) in enumerate(plan):
+            stages = self.layers[self.runs[r][0]].stages
+            branches = stages[s].run(h, self.entry[r], cache, b)
+            if return_hidden and s == len(stages) - 1:
                 taps.append(ops.gated_residual(x, branches)[0])
-            x, h = ops.gated_residual(x, branches, **ahead(r + 1), **norm)
+            x, h = ops.gated_residual(x, branches, **ahead(n + 1), **norm)
         return (h[0], taps) if return_hidden else h[0]
 
     # ------------------------------------------------------------------ the engine's entry points

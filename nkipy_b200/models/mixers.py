@@ -1,0 +1,186 @@
+"""Token mixers of the layer-by-layer decoders (models/hybrid.py).
+
+A mixer owns the rows it puts into its layer's input projection (`w_in`), its entries of the cache (paged keys and values
+or per-sequence states), its output projection (`w_o`), and the step in between: `run` takes the input projection's result
+and returns the operand of the output projection.  A new kind of layer is a new class here beside a spec in config.py.
+"""
+
+from __future__ import annotations
+
+from typing import List
+
+import torch
+
+from .. import ops
+from ..ops import Decay, MapsSpec, Proj
+from ..ops.linear_attention import linear_state_shape
+from ..ops.mixers import hgrn2_state_shape
+from .kv_cache import KVLayer, StateLayer
+
+
+class Tensors:
+    """The tensors under one prefix, in the forms the layers keep: fp32 vectors and stacked matrices of the model's type."""
+
+    def __init__(self, get, prefix: str, dtype: torch.dtype):
+        self.get, self.prefix, self.dtype = get, prefix, dtype
+
+    def under(self, prefix: str) -> "Tensors":
+        return Tensors(self.get, self.prefix + prefix, self.dtype)
+
+    def raw(self, name: str) -> torch.Tensor:
+        return self.get(self.prefix + name)
+
+    def f32(self, name: str, offset: float = 0.0) -> torch.Tensor:
+        return (self.raw(name).float() + offset).contiguous()
+
+    def mat(self, *names: str) -> torch.Tensor:
+        return torch.cat([self.raw(n).to(self.dtype) for n in names]).contiguous()
+
+    def stack(self, *names: str) -> torch.Tensor:
+        return torch.stack([self.raw(n).to(self.dtype) for n in names]).contiguous()
+
+
+def columns(y: torch.Tensor, widths: List[int]) -> List[Proj]:
+    out, c = [], 0
+    for w in widths:
+        out.append(Proj(y, c, w))
+        c += w
+    return out
+
+
+class Hgrn2Mixer:
+    """Linear recurrence with a forget gate."""
+
+    def __init__(self, spec, t: Tensors, eps: float):
+        self.spec, self.eps = spec, eps
+        self.w_in, self.w_o = t.mat("q", "f", "v"), t.mat("o")
+        self.widths = [spec.heads * spec.dim, spec.heads * spec.dim, spec.heads * spec.vdim]
+        self.f_bias, self.lower, self.norm = t.f32("f.b"), t.f32("lower"), t.f32("norm")
+
+    def entries(self):
+        return [StateLayer(hgrn2_state_shape(self.spec.heads, self.spec.dim, self.spec.vdim))]
+
+    def run(self, model, y, h, entry, cache, b):
+        m = self.spec
+        return ops.hgrn2(*columns(y, self.widths), self.f_bias, self.lower, self.norm, cache.state[entry], b.context_lens,
+                         heads=m.heads, dim=m.dim, vdim=m.vdim, eps=self.eps, q_start=b.q_start, q_lens=b.q_lens,
+                         rows=b.rows, dtype=model.dtype)
+
+
+class MapsMixer:
+    """Differential attention: two score maps per head, interleaved partial rotation."""
+
+    def __init__(self, spec, t: Tensors, eps: float):
+        self.spec = spec
+        self.w_in, self.w_o = t.mat("q", "k", "v"), t.mat("o")
+        self.widths = [spec.heads * 2 * spec.dim, spec.kv_heads * 2 * spec.dim, spec.kv_heads * spec.vdim]
+        dot = lambda a, b: float(torch.exp((t.raw(a).double() * t.raw(b).double()).sum()))
+        lam = dot("lq1", "lk1") - dot("lq2", "lk2") + spec.diff
+        self.maps = MapsSpec(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.scale, maps=2, softcap=spec.softcap,
+                             lam=lam, out_scale=1.0 - spec.diff, eps=eps, tiled=t.dtype == torch.bfloat16)
+
+    def entries(self):
+        return [KVLayer(self.spec.kv_heads, self.maps.maps * self.maps.dim_p, self.maps.vdim_p)]
+
+    def run(self, model, y, h, entry, cache, b):
+        q = ops.maps_append(self.maps, *columns(y, self.widths), model.rope_table(self.spec.rope), b.positions, b.slots,
+                            cache.k[entry], cache.v[entry])
+        return ops.maps_attention(self.maps, q, cache.k[entry], cache.v[entry], b.block_table, b.context_lens,
+                                  q_start=b.q_start, q_lens=b.q_lens, max_q_len=b.max_q_len)
+
+
+class LinearAttentionMixer:
+    """Gated linear attention."""
+
+    def __init__(self, spec, t: Tensors, eps: float):
+        self.spec, self.eps = spec, eps
+        self.w_in, self.w_o = t.mat("q", "k", "v", "g", "a1"), t.mat("o")
+        c, n = spec.heads * spec.dim, spec.heads * spec.vdim
+        self.w_decay, self.decay_bias, self.norm = t.mat("a2"), t.f32("a2.b"), t.f32("norm")
+        self.widths = [c, c, n, n, self.w_decay.shape[1]]
+
+    def entries(self):
+        return [StateLayer(linear_state_shape(self.spec.heads, self.spec.dim, self.spec.vdim))]
+
+    def run(self, model, y, h, entry, cache, b):
+        m = self.spec
+        q, k, v, g, a = columns(y, self.widths)
+        decay = Decay("sigmoid_root", a, self.w_decay, self.decay_bias, tau=m.tau)
+        return ops.linear_attention(q, k, v, decay, g, self.norm, cache.state[entry], b.context_lens, heads=m.heads,
+                                    dim=m.dim, vdim=m.vdim, eps=self.eps, q_scale=m.dim ** -0.5, q_start=b.q_start,
+                                    q_lens=b.q_lens, rows=b.rows, dtype=model.dtype)
+
+
+class WindowAttentionMixer:
+    """Grouped-query attention over a sliding window, queries and keys normed over all heads, sigmoid-gated heads."""
+
+    def __init__(self, spec, t: Tensors, eps: float, scale: float = 1.0):
+        self.spec, self.scale = spec, scale
+        self.w_in, self.w_o = t.mat("q", "k", "v", "g"), t.mat("o")
+        self.widths = [spec.heads * spec.dim, spec.kv_heads * spec.dim, spec.kv_heads * spec.vdim, spec.heads * spec.vdim]
+        self.q_norm, self.k_norm = t.f32("q.norm"), t.f32("k.norm")
+        self.maps = MapsSpec(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.scale, maps=1, eps=eps,
+                             window=spec.window, tiled=t.dtype == torch.bfloat16)
+
+    def entries(self):
+        return [KVLayer(self.spec.kv_heads, self.maps.dim_p, self.maps.vdim_p)]
+
+    def run(self, model, y, h, entry, cache, b, out=None):
+        q, k, v, g = columns(y, self.widths)
+        kc, vc = cache.k[entry], cache.v[entry]
+        q = ops.row_norm_append(self.maps, q, k, v, self.q_norm, self.k_norm, b.slots, kc, vc)
+        o = ops.heads_attention(self.maps, q, kc, vc, b.block_table, b.context_lens, q_start=b.q_start, q_lens=b.q_lens,
+                                max_q_len=b.max_q_len)
+        return ops.gate_heads(o, g, "sigmoid", scale=self.scale, out=out)
+
+
+class TimeMixMixer:
+    """RWKV-style time mixing.  Its projections read mixes of neighbouring tokens and not h, so it has no rows in the
+    layer's input projection."""
+
+    def __init__(self, spec, t: Tensors, eps: float, scale: float = 1.0):
+        self.spec, self.eps, self.scale = spec, eps, scale
+        self.w_in, self.widths, self.w_o = None, [], t.mat("o")
+        self.w_each, self.w_narrow, self.w_decay = t.stack("r", "k", "v", "g"), t.mat("w1"), t.mat("w2")
+        self.mu = torch.stack([t.f32("mu." + n) for n in "rkvgw"]).contiguous()
+        self.decay_bias, self.bonus, self.norm = t.f32("w0"), t.f32("u").reshape(-1).contiguous(), t.f32("norm")
+
+    def entries(self):
+        return [StateLayer(linear_state_shape(self.spec.heads, self.spec.dim, self.spec.dim)), StateLayer((self.mu.shape[1],))]
+
+    def run(self, model, y, h, entry, cache, b, out=None):
+        m = self.spec
+        x = ops.token_mix(h, self.mu, cache.state[entry + 1], b.context_lens, q_start=b.q_start, q_lens=b.q_lens,
+                          rows=b.rows)
+        r, k, v, g = model.project_each(x[:4], self.w_each)
+        narrow = model.project(x[4], self.w_narrow)
+        decay = Decay("double_exp", Proj(narrow, 0, self.w_narrow.shape[0]), self.w_decay, self.decay_bias, act="tanh")
+        return ops.linear_attention(r, k, v, decay, g, self.norm, cache.state[entry], b.context_lens, heads=m.heads,
+                                    dim=m.dim, vdim=m.dim, eps=self.eps, bonus=self.bonus, scale=self.scale,
+                                    q_start=b.q_start, q_lens=b.q_lens, rows=b.rows, dtype=model.dtype, out=out)
+
+
+class ParallelMixer:
+    """Two mixers on the same input.  Their constant weights are applied to the operands of the output projections, which
+    then are one product over the joined operands."""
+
+    def __init__(self, spec, t: Tensors, eps: float):
+        self.left = WindowAttentionMixer(spec.left, t.under("left."), eps, spec.left_scale)
+        self.right = TimeMixMixer(spec.right, t.under("right."), eps, spec.right_scale)
+        self.w_in, self.widths = self.left.w_in, self.left.widths
+        self.split = self.left.w_o.shape[1]
+        self.w_o = torch.cat([self.left.w_o, self.right.w_o], 1).contiguous()
+        self.left.w_o = self.right.w_o = None
+
+    def entries(self):
+        return self.left.entries() + self.right.entries()
+
+    def run(self, model, y, h, entry, cache, b):
+        out = torch.empty((h.shape[0], self.w_o.shape[1]), dtype=model.dtype, device=h.device)
+        self.left.run(model, y, h, entry, cache, b, out=out[:, :self.split])
+        self.right.run(model, None, h, entry + 1, cache, b, out=out[:, self.split:])
+        return out
+
+
+MIXERS = {"hgrn2": Hgrn2Mixer, "attention": MapsMixer, "gla": LinearAttentionMixer, "window": WindowAttentionMixer,
+          "rwkv": TimeMixMixer, "parallel": ParallelMixer}

@@ -17,6 +17,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
+from ..ops import Branch, Proj
 from ..parallel.comm import TPGroup
 from .config import ModelConfig
 
@@ -30,8 +31,7 @@ class MoEBlock:
         self.expert_lo = tp.rank * self.num_local if moe_parallel == "ep" else 0
 
     def route(self, lw, x: torch.Tensor):
-        # one 128-row weight tile: split the contraction so several SMs share the work
-        logits = ops.linear(x, lw.router, splits=max(2, min(16, x.shape[1] // 256)))
+        logits = ops.linear(x, lw.router, splits=route_splits(x.shape[1]))
         return ops.router_topk(logits, self.cfg.top_k, self.cfg.router_mode, bias=lw.router_bias)
 
     def _experts(self, lw, x: torch.Tensor):
@@ -85,3 +85,39 @@ class MoEBlock:
         weights, experts = self.route(lw, x_local)
         return a2a.forward(x_local, experts, weights, lw.gate_up, lw.down, gate_up_bias=lw.gate_up_bias,
                            down_bias=lw.down_bias, act_limit=cfg.swiglu_limit, act_alpha=cfg.swiglu_alpha)
+
+
+def route_splits(width: int) -> int:
+    """Split-K factor of a router's product: its few outputs are one weight tile, so several SMs share the contraction."""
+    return max(2, min(16, width // 256))
+
+
+class RoutedExperts:
+    """Routed feed-forward of one layer of a layer-by-layer decoder (`config.ExpertsSpec`, one rank).  The weighted sum of
+    the experts' rows is left to the residual kernel (`ops.Branch`).  bf16 sizes with 16-byte rows run the grouped
+    tcgen05 products, everything else the grouped products on the CUDA cores."""
+
+    def __init__(self, spec, t):
+        self.spec = spec
+        self.router = t.mat("router")
+        self.gate_up = torch.stack([t.mat(f"e{e}.gate", f"e{e}.up") for e in range(spec.experts)]).contiguous()
+        self.down = t.stack(*[f"e{e}.down" for e in range(spec.experts)])
+        self.tiled = t.dtype == torch.bfloat16 and self.down.shape[1] % 8 == 0 and spec.ff % 8 == 0
+
+    def weights(self):
+        return [self.router, self.gate_up, self.down]
+
+    def run(self, model, h: torch.Tensor) -> Branch:
+        s, (T, W) = self.spec, h.shape
+        logits = ops.linear(h, self.router, splits=route_splits(W)) if h.dtype == torch.bfloat16 else ops.linear(h, self.router)
+        weights, experts = ops.router_topk(logits, s.top, groups=s.groups, keep=s.keep, scale=s.scale)
+        plan = ops.moe_dispatch(h, experts, 0, s.experts, gather=self.tiled)
+        if self.tiled:
+            act = ops.grouped_linear(plan.x_sorted, self.gate_up, plan.offsets, max_rows_per_group=T, gated=True,
+                                     tiles=plan.tiles)
+            y = ops.grouped_linear(act, self.down, plan.offsets, max_rows_per_group=T, tiles=plan.tiles)
+        else:
+            gu = ops.grouped_linear_simt(plan, h, self.gate_up, False)
+            act = ops.gated_act(Proj(gu, 0, s.ff), Proj(gu, s.ff, s.ff), "silu", dtype=h.dtype)
+            y = ops.grouped_linear_simt(plan, act, self.down, True)
+        return Branch(Proj(y, 0, W), pair_pos=plan.pair_pos, pair_w=weights)

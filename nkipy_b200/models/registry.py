@@ -59,6 +59,13 @@ def _transformer(config) -> Architecture:
                                                                    moe_parallel=moe))
 
 
+def _hybrid(config) -> Architecture:
+    return Architecture(
+        config, HybridLM,
+        lambda cfg, sd, rank, world, moe: {k: sd[k] for k in sd.keys()},
+        lambda cfg, rank, world, device, seed, moe: hybrid_random_weights(cfg, device=device, seed=seed))
+
+
 _MOE = {"num_experts_per_tok": "top_k", "intermediate_size": ""}
 
 ARCHITECTURES: Dict[str, Architecture] = {
@@ -68,10 +75,8 @@ ARCHITECTURES: Dict[str, Architecture] = {
                                                    moe_intermediate_size="moe_intermediate_size")),
     "GptOssForCausalLM": _transformer(_hf_config(C.gpt_oss_20b, **{**_MOE, "intermediate_size": "moe_intermediate_size"},
                                                  num_local_experts="num_experts", sliding_window="sliding_window")),
-    "Tolenex": Architecture(
-        C.tolenex_config, HybridLM,
-        lambda cfg, sd, rank, world, moe: {k: sd[k] for k in sd.keys()},
-        lambda cfg, rank, world, device, seed, moe: hybrid_random_weights(cfg, device=device, seed=seed)),
+    "Tolenex": _hybrid(C.tolenex_config),
+    "Mumilorn": _hybrid(C.mumilorn_config),
 }
 
 
@@ -84,7 +89,9 @@ def architecture_of(raw: dict) -> Architecture:
 
 def for_config(cfg: C.ModelConfig) -> Architecture:
     """The architecture entry that runs a configuration made in code."""
-    return ARCHITECTURES["Tolenex"] if cfg.layers is not None else ARCHITECTURES["LlamaForCausalLM"]
+    if cfg.layers is None:
+        return ARCHITECTURES["LlamaForCausalLM"]
+    return ARCHITECTURES["Mumilorn" if cfg.name == "mumilorn" else "Tolenex"]
 
 
 def read_config(folder: str):

@@ -154,43 +154,76 @@ def random_weights(cfg: ModelConfig, rank: int = 0, world: int = 1, device="cpu"
     return out
 
 
+def _mixer_shapes(m, W: int) -> Dict[str, tuple]:
+    """Tensors of a token mixer (models/mixers.py) by their names under '<layer>.mix.'."""
+    if m.kind == "parallel":
+        return {**{"left." + k: v for k, v in _mixer_shapes(m.left, W).items()},
+                **{"right." + k: v for k, v in _mixer_shapes(m.right, W).items()}}
+    if m.kind == "rwkv":
+        c, rank = m.heads * m.dim, m.rank or 16
+        return {**{f"mu.{n}": (W,) for n in "rkvgw"}, **{n: (c, W) for n in "rkvg"}, "w1": (rank, W), "w2": (c, rank),
+                "w0": (c,), "u": (m.heads, m.dim), "norm": (c,), "o": (W, c)}
+    out = m.heads * m.vdim
+    if m.kind == "window":
+        q, k = m.heads * m.dim, m.kv_heads * m.dim
+        return {"q": (q, W), "k": (k, W), "v": (m.kv_heads * m.vdim, W), "q.norm": (q,), "k.norm": (k,), "g": (out, W),
+                "o": (W, out)}
+    if m.kind == "gla":
+        c, rank = m.heads * m.dim, m.rank or 16
+        return {"q": (c, W), "k": (c, W), "v": (out, W), "g": (out, W), "a1": (rank, W), "a2": (c, rank), "a2.b": (c,),
+                "norm": (m.vdim,), "o": (W, out)}
+    if m.kind == "hgrn2":
+        c = m.heads * m.dim
+        return {"q": (c, W), "f": (c, W), "f.b": (c,), "lower": (c,), "v": (out, W), "norm": (m.vdim,), "o": (W, out)}
+    return {"q": (2 * m.heads * m.dim, W), "k": (2 * m.kv_heads * m.dim, W), "v": (m.kv_heads * m.vdim, W), "o": (W, out),
+            **{n: (m.dim,) for n in ("lq1", "lk1", "lq2", "lk2")}}
+
+
 def hybrid_weight_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
     """Name -> shape of every tensor of a layer-by-layer configuration (models/hybrid.py), matrices [out, in]."""
     W, V = cfg.hidden_size, cfg.vocab_size
-    out: Dict[str, tuple] = {"embed": (V, W), "head": (V, W), "final.norm": (W,)}
+    out: Dict[str, tuple] = {"embed": (V, W), "final.norm": (W,)}
+    if not cfg.tie_embeddings:
+        out["head"] = (V, W)
     if cfg.loop:
         out["loop.step"] = (cfg.loop.times, W)
     for i, layer in enumerate(cfg.layers):
-        p, m = f"l{i}.", layer.mixer
-        shapes = {"norm1": (W,), "rg1": (W, W), "rg1.b": (W,), "mix.o": (W, m.heads * m.vdim)}
-        if m.kind == "hgrn2":
-            c = m.heads * m.dim
-            shapes.update({"mix.q": (c, W), "mix.f": (c, W), "mix.f.b": (c,), "mix.lower": (c,),
-                           "mix.v": (m.heads * m.vdim, W), "mix.norm": (m.vdim,)})
-        else:
-            shapes.update({"mix.q": (2 * m.heads * m.dim, W), "mix.k": (2 * m.kv_heads * m.dim, W),
-                           "mix.v": (m.kv_heads * m.vdim, W)})
-            shapes.update({f"mix.{n}": (m.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
+        shapes = {"norm1": (W,), **{"mix." + k: v for k, v in _mixer_shapes(layer.mixer, W).items()}}
+        if layer.block == "gated":
+            shapes.update({"rg1": (W, W), "rg1.b": (W,)})
+        if layer.ff or layer.experts:
+            shapes["norm2"] = (W,)
         if layer.ff:
-            shapes.update({"norm2": (W,), "mlp.gate": (layer.ff, W), "mlp.up": (layer.ff, W),
-                           "mlp.down": (W, layer.ff), "rg2": (W, W), "rg2.b": (W,)})
-        out.update({p + k: v for k, v in shapes.items()})
+            shapes.update({"mlp.up": (layer.ff, W), "mlp.down": (W, layer.ff)})
+            if layer.block == "gated":
+                shapes.update({"mlp.gate": (layer.ff, W), "rg2": (W, W), "rg2.b": (W,)})
+        if layer.experts:
+            x = layer.experts
+            shapes["mlp.router"] = (x.experts, W)
+            for e in range(x.experts):
+                shapes.update({f"mlp.e{e}.gate": (x.ff, W), f"mlp.e{e}.up": (x.ff, W), f"mlp.e{e}.down": (W, x.ff)})
+        out.update({f"l{i}." + k: v for k, v in shapes.items()})
     return out
 
 
 def hybrid_random_weights(cfg: ModelConfig, device="cpu", seed: int = 0, std: float = 0.02,
                           dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
-    """Random-init weights of a layer-by-layer configuration: N(0, std), norm weights 1, lower bounds of the
-    forget gates uniform in [0, 0.9)."""
+    """Random-init weights of a layer-by-layer configuration: N(0, std), norms that multiply by 1, lower bounds of the
+    forget gates and mixes of neighbouring tokens uniform in [0, 0.9), slow decays."""
     out: Dict[str, torch.Tensor] = {}
     for n, (name, shape) in enumerate(hybrid_weight_shapes(cfg).items()):
-        if name.endswith(("norm1", "norm2", ".norm")):
+        leaf = name.rsplit(".", 1)[-1]
+        if leaf in ("norm1", "norm2") or name == "final.norm":
+            out[name] = torch.full(shape, 1.0 - cfg.norm_offset, dtype=dtype, device=device)
+        elif leaf == "norm":
             out[name] = torch.ones(shape, dtype=dtype, device=device)
-        elif name.endswith(".lower"):
+        elif leaf == "lower" or ".mu." in name:
             g = torch.Generator(device=device).manual_seed(seed * 100003 + n)
             out[name] = (0.9 * torch.rand(shape, generator=g, device=device)).to(dtype)
         else:
             out[name] = _normal(shape, std, seed * 100003 + n, device, dtype)
+            if leaf == "w0":
+                out[name] -= 4.0             # exp(-exp(-4)): a memory of some fifty tokens
     return out
 
 

@@ -29,7 +29,9 @@ from ._lib import KernelLibraryError, device_status, raise_on_device_error
 __all__ = [
     "linear", "decode_linear", "qkv_rope_append", "reduce_partials", "rmsnorm", "add_rmsnorm", "silu_mul", "embedding", "rope_kv_append",
     "argmax", "sample", "decode_advance", "router_topk", "moe_dispatch", "grouped_linear", "moe_combine", "paged_attn_decode", "flash_attn_prefill", "rope_table",
-    "MapsSpec", "Proj", "gated_act", "gated_residual", "hgrn2", "maps_append", "maps_attention",
+    "Branch", "MapsSpec", "Proj", "activation", "gate_heads", "gated_act", "gated_residual", "hgrn2", "maps_append",
+    "heads_attention", "maps_attention", "row_norm_append",
+    "Decay", "linear_attention", "low_rank", "token_mix",
     "KernelLibraryError", "device_status", "raise_on_device_error", "native_available", "launch_count",
     "reset_launch_count",
 ]
@@ -104,6 +106,7 @@ def linear(
     ctas_per_sm: Optional[int] = None,
     act: str = "silu",
     fp32_out: bool = False,
+    out_act: Optional[str] = None,
 ) -> torch.Tensor:
     """``y = x @ w.T`` with optional fused epilogue.
 
@@ -112,6 +115,7 @@ def linear(
     gated: w is ``[2*I, K]`` holding gate rows then up rows; returns
            ``act(x @ gate.T) * (x @ up.T)`` of shape [M, I], act "silu" or "gelu_tanh".
     fp32_out: finished values in fp32 instead of bf16 (not with gated).
+    out_act: "relu2" applies the square of the positive part to a plain product (finished bf16 values).
     splits > 1: split-K; returns fp32 partial sums ``[S, M, N]`` (S may be smaller
            than requested) for a fused reduction (`add_rmsnorm`, `rope_kv_append`,
            `reduce_partials`).  bias is added to partial 0.
@@ -137,6 +141,8 @@ def linear(
             y = y + bias.float()
         if splits > 1:
             return y.unsqueeze(0)
+        if out_act is not None:
+            y = mixers.ACTIVATIONS[out_act][1](y)
         if residual is not None:
             y = y + residual.float()
         y = y.to(torch.float32 if fp32_out or x.dtype == torch.float32 else torch.bfloat16)
@@ -147,15 +153,20 @@ def linear(
     global _launches
     if x.stride(1) != 1 or w.stride(1) != 1:
         raise ValueError("linear needs K-contiguous operands")
-    if x.dtype == torch.float32 or (K | x.stride(0) | w.stride(0)) & 7:
+    if out_act not in (None, "relu2") or (out_act and (gated or residual is not None or fp32_out)):
+        raise ValueError("out_act is relu2, for finished plain products")
+    if x.dtype == torch.float32 or (K | x.stride(0) | w.stride(0)) & 7 or (x.data_ptr() | w.data_ptr()) & 15:
         if bias is not None or residual is not None or out is not None:
             raise ValueError("the CUDA-core GEMM has no bias, residual or out argument")
-        return mixers.linear_simt(x, w, gated=gated, act=act, fp32_out=fp32_out or splits > 1)
+        y = mixers.linear_simt(x, w, gated=gated, act=act, fp32_out=fp32_out or splits > 1 or out_act is not None)
+        return y if out_act is None else mixers.activation(Proj(y, 0, N), out_act, dtype=x.dtype)
     _check_bf16(x, w, bias, residual)
     if fp32_out and gated:
         raise ValueError("fp32_out is for plain products")
     if swap is None:
         swap = M <= 128
+    if out_act is not None and (swap or splits > 1):
+        raise ValueError("out_act wants finished values in the prefill orientation (swap=False)")
     L = _lib.lib()
     if splits > 1:
         eff = L.nkb_gemm_effective_splits(K, splits)
@@ -172,12 +183,13 @@ def linear(
         out_view = out
         out_fp32, split_stride = 1 if fp32_out else 0, 0
     ldo = out_view.stride(-2) if out_view.dim() >= 2 else N
+    act_code = mixers.ACTIVATIONS[act][0] if gated else (mixers.ACTIVATIONS[out_act][0] if out_act else 0)
     if (not swap and splits <= 1 and not fp32_out and M >= 512 and N >= 256 and _USE_2CTA and (ldo & 7) == 0
             and not (gated and (bias is not None or residual is not None))):
         # prefill-sized: CTA pairs on 256 x 256 tiles (csrc/kernels/gemm_2cta.cu)
         rc = L.nkb_gemm_bf16_2cta(x.data_ptr(), w.data_ptr(), out_view.data_ptr(), M, N, K, x.stride(0), w.stride(0),
-                                  ldo, _ptr(bias), _ptr(residual), 1 if gated else 0, N if gated else 0,
-                                  mixers.ACTIVATIONS[act][0], _stream())
+                                  ldo, _ptr(bias), _ptr(residual), 1 if gated else 0, N if gated else 0, act_code,
+                                  _stream())
         if rc != -5:
             _lib.check(rc, "nkb_gemm_bf16_2cta")
             _launches += 1
@@ -198,7 +210,7 @@ def linear(
         a.data_ptr(), b.data_ptr(), out_view.data_ptr(), rows, cols, K, lda, ldb, ldo, transpose_out, out_fp32,
         eff if splits > 1 else 1, split_stride, gate_mode, N if gated else 0, _ptr(bias), bias_on_rows,
         _ptr(residual), block_n, max_ctas, (0 if swap else 1) if weights_static else -1,
-        (2 if (swap and not gated) else 1) if ctas_per_sm is None else ctas_per_sm, mixers.ACTIVATIONS[act][0], _stream(),
+        (2 if (swap and not gated) else 1) if ctas_per_sm is None else ctas_per_sm, act_code, _stream(),
     )
     _lib.check(rc, "nkb_gemm_bf16")
     _launches += 1
@@ -687,11 +699,13 @@ def sample(logits: torch.Tensor, temperature: float = 1.0, top_k: int = 0, top_p
     return out_ids
 
 
-def router_topk(logits: torch.Tensor, top_k: int, mode: str = "softmax_topk",
-                bias: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+def router_topk(logits: torch.Tensor, top_k: int, mode: str = "softmax_topk", bias: Optional[torch.Tensor] = None, *,
+                groups: int = 0, keep: int = 0, scale: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
     """MoE routing.  mode "softmax_topk": softmax over all experts, top-k, renormalise
     (Qwen3); "topk_softmax": top-k raw logits, softmax over them (gpt-oss).  logits are bf16 /
     fp32 ``[T, E]`` or fp32 split-K partials ``[S, T, E]`` (summed here); bias [E] is added first.
+    groups > 0 (softmax_topk): experts form that many equal runs of neighbours and only those of the `keep` runs with
+    the largest single score can be chosen.  The weights are multiplied by `scale`.
     Returns (weights fp32 [T, k], experts int32 [T, k])."""
     partial = logits.dim() == 3
     T, E = logits.shape[-2], logits.shape[-1]
@@ -701,12 +715,17 @@ def router_topk(logits: torch.Tensor, top_k: int, mode: str = "softmax_topk",
             lf = lf + bias.float()
         if mode == "softmax_topk":
             p = torch.softmax(lf, dim=-1)
-            w, e = p.topk(top_k, dim=-1)
-            w = w / w.sum(-1, keepdim=True)
+            pick = p
+            if groups > 0:
+                best = p.reshape(T, groups, E // groups).amax(-1).topk(keep, dim=-1).indices
+                on = torch.zeros((T, groups), dtype=torch.bool).scatter_(1, best, True)
+                pick = p.masked_fill(~on.repeat_interleave(E // groups, dim=1), -1.0)
+            w, e = pick.topk(top_k, dim=-1)
+            w = w / (w.sum(-1, keepdim=True) + 1e-20)
         else:
             v, e = lf.topk(top_k, dim=-1)
             w = torch.softmax(v, dim=-1)
-        return w, e.to(torch.int32)
+        return w * scale, e.to(torch.int32)
     global _launches
     w = torch.empty((T, top_k), dtype=torch.float32, device=logits.device)
     e = torch.empty((T, top_k), dtype=torch.int32, device=logits.device)
@@ -716,7 +735,7 @@ def router_topk(logits: torch.Tensor, top_k: int, mode: str = "softmax_topk",
     splits = logits.shape[0] if partial else 1
     rc = _lib.lib().nkb_router_topk(logits.data_ptr(), is_fp32, splits, logits.stride(0) if partial else 0, _ptr(bias),
                                     w.data_ptr(), e.data_ptr(), T, E, top_k, 0 if mode == "softmax_topk" else 1,
-                                    _stream())
+                                    int(groups), int(keep), float(scale), _stream())
     _lib.check(rc, "nkb_router_topk")
     _launches += 1
     return w, e
@@ -971,10 +990,11 @@ def flash_attn_prefill(
 # --------------------------------------------------------------------------- mixture of experts
 class MoEPlan:
     """Result of `moe_dispatch`: expert-sorted rows plus the device-side schedules of the grouped GEMMs."""
-    __slots__ = ("x_sorted", "offsets", "pair_pos", "tiles", "max_rows")
+    __slots__ = ("x_sorted", "offsets", "pair_pos", "tiles", "max_rows", "row_token")
 
-    def __init__(self, x_sorted, offsets, pair_pos, tiles, max_rows):
+    def __init__(self, x_sorted, offsets, pair_pos, tiles, max_rows, row_token=None):
         self.x_sorted, self.offsets, self.pair_pos, self.tiles, self.max_rows = x_sorted, offsets, pair_pos, tiles, max_rows
+        self.row_token = row_token
 
     def __iter__(self):          # (x_sorted, offsets, pair_pos) unpacking
         return iter((self.x_sorted, self.offsets, self.pair_pos))
@@ -987,12 +1007,13 @@ def moe_tile_widths(tokens: int):
     return 64, 128
 
 
-def moe_dispatch(x: torch.Tensor, experts: torch.Tensor, expert_lo: int, num_local: int) -> MoEPlan:
+def moe_dispatch(x: torch.Tensor, experts: torch.Tensor, expert_lo: int, num_local: int, gather: bool = True) -> MoEPlan:
     """Sort the (token, expert) pairs routed to local experts [expert_lo, expert_lo + num_local) by
     expert and gather their token rows.  x [T, H] bf16, experts [T, k] int32 (global ids).
     Returns a `MoEPlan` (unpacks to x_sorted [T * k, H], offsets int32 [num_local + 1], pair_pos int32
     [T * k]); rows past offsets[-1] of x_sorted are unspecified, pair_pos is -1 for pairs of other
-    ranks' experts."""
+    ranks' experts.  gather False: x_sorted is x itself and `row_token` names the token of every sorted row (any type and
+    width, for `grouped_linear_simt`)."""
     T, H = x.shape
     k = experts.shape[1]
     pairs = T * k
@@ -1007,13 +1028,23 @@ def moe_dispatch(x: torch.Tensor, experts: torch.Tensor, expert_lo: int, num_loc
         counts = torch.bincount(flat[local], minlength=num_local)
         offsets = torch.zeros((num_local + 1,), dtype=torch.int32)
         offsets[1:] = counts.cumsum(0).to(torch.int32)
+        row_token = torch.zeros((pairs,), dtype=torch.int32)
+        row_token[:n_local] = (order[:n_local] // k).to(torch.int32)
+        if not gather:
+            return MoEPlan(x, offsets, pair_pos, None, T, row_token)
         x_sorted = torch.zeros((pairs, H), dtype=x.dtype)
         x_sorted[:n_local] = x[(order[:n_local] // k)]
-        return MoEPlan(x_sorted, offsets, pair_pos, None, T)
+        return MoEPlan(x_sorted, offsets, pair_pos, None, T, row_token)
     global _launches
     bn_a, bn_b = moe_tile_widths(T)
     cap_a, cap_b = num_local + pairs // bn_a + 1, num_local + pairs // bn_b + 1
-    x_sorted = torch.empty((pairs, H), dtype=x.dtype, device=dev)
+    if gather:
+        _check_bf16(x)
+        x_sorted = torch.empty((pairs, H), dtype=x.dtype, device=dev)
+        row_token = None
+    else:
+        x_sorted = x
+        row_token = torch.empty((pairs,), dtype=torch.int32, device=dev)
     work = torch.empty((3 * num_local + 1 + pairs + 2 * cap_a + 2 * cap_b + 2,), dtype=torch.int32, device=dev)
     o = 0
     counts = work[o:o + num_local]; o += num_local
@@ -1025,15 +1056,15 @@ def moe_dispatch(x: torch.Tensor, experts: torch.Tensor, expert_lo: int, num_loc
     ntiles = work[o:o + 2]
     if experts.dtype != torch.int32:
         experts = experts.to(torch.int32)
-    rc = _lib.lib().nkb_moe_dispatch(experts.data_ptr(), T, k, int(expert_lo), int(num_local), x.data_ptr(), H,
-                                     x_sorted.data_ptr(), counts.data_ptr(), offsets.data_ptr(), cursors.data_ptr(),
-                                     pair_pos.data_ptr(), bn_a, tiles_a.data_ptr(), ntiles.data_ptr(), bn_b,
+    rc = _lib.lib().nkb_moe_dispatch(experts.data_ptr(), T, k, int(expert_lo), int(num_local),
+                                     x.data_ptr() if gather else None, H, x_sorted.data_ptr(), counts.data_ptr(),
+                                     offsets.data_ptr(), cursors.data_ptr(), pair_pos.data_ptr(), _ptr(row_token), bn_a, tiles_a.data_ptr(), ntiles.data_ptr(), bn_b,
                                      tiles_b.data_ptr(), ntiles.data_ptr() + 4, _stream())
     _lib.check(rc, "nkb_moe_dispatch")
     _launches += 2 if pairs <= 8192 else 5
     tiles = {bn_a: (tiles_a, ntiles[0:1], cap_a)}
     tiles.setdefault(bn_b, (tiles_b, ntiles[1:2], cap_b))
-    return MoEPlan(x_sorted, offsets, pair_pos, tiles, T)
+    return MoEPlan(x_sorted, offsets, pair_pos, tiles, T, row_token)
 
 
 def grouped_linear(x_sorted: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, *, max_rows_per_group: int,
@@ -1091,6 +1122,29 @@ def grouped_linear(x_sorted: torch.Tensor, w: torch.Tensor, offsets: torch.Tenso
     return out
 
 
+def grouped_linear_simt(plan: MoEPlan, x: torch.Tensor, w: torch.Tensor, sorted_rows: bool) -> torch.Tensor:
+    """fp32 ``y[r] = x[row] @ w[g(r)].T`` on the CUDA cores, for the expert-sorted rows of a plan: row r of x when
+    sorted_rows, its token's row (`row_token`) otherwise.  x and w [G, N, K] both fp32 or both bf16, any sizes."""
+    G, N, K = w.shape
+    P = plan.pair_pos.numel()
+    out = torch.empty((P, N), dtype=torch.float32, device=x.device)
+    if not _native(x):
+        rows = x if sorted_rows else x[plan.row_token.long()]
+        off = plan.offsets.tolist()
+        for g in range(G):
+            out[off[g]:off[g + 1]] = rows[off[g]:off[g + 1]].float() @ w[g].float().T
+        return out
+    if x.dtype != w.dtype or not w.is_contiguous():
+        raise TypeError("grouped_linear_simt wants operands of one type and contiguous weights")
+    bf = 1 if x.dtype == torch.bfloat16 else 0
+    rc = _lib.lib().nkb_gemm_simt_grouped(
+        x.data_ptr(), bf, w.data_ptr(), bf, out.data_ptr(), 0, plan.offsets.data_ptr(),
+        None if sorted_rows else plan.row_token.data_ptr(), G, int(plan.max_rows), N, K, x.stride(0), N, _stream())
+    _lib.check(rc, "nkb_gemm_simt_grouped")
+    _count_launch()
+    return out
+
+
 def moe_combine(y_sorted: torch.Tensor, pair_pos: torch.Tensor, weights: torch.Tensor, tokens: int) -> torch.Tensor:
     """``out[t] = sum_j weights[t, j] * y_sorted[pair_pos[t * k + j]]`` over local pairs -> bf16 [T, H]."""
     k = weights.shape[1]
@@ -1112,4 +1166,6 @@ def moe_combine(y_sorted: torch.Tensor, pair_pos: torch.Tensor, weights: torch.T
 
 
 from . import mixers  # noqa: E402  (uses the helpers above)
-from .mixers import (MapsSpec, Proj, gated_act, gated_residual, hgrn2, maps_append, maps_attention)  # noqa: E402,F401
+from .mixers import (Branch, MapsSpec, Proj, activation, gate_heads, gated_act, gated_residual,  # noqa: E402,F401
+                     heads_attention, hgrn2, maps_append, maps_attention, row_norm_append)
+from .linear_attention import Decay, linear_attention, low_rank, token_mix  # noqa: E402,F401

@@ -30,7 +30,23 @@ class ProjArg(ctypes.Structure):
 class MapsArg(ctypes.Structure):
     """Sizes and constants of attention with several score maps (csrc/kernels/attn_maps.h)."""
     _fields_ = [(n, c_int) for n in ("maps", "heads", "kv_heads", "dim", "dim_p", "vdim", "vdim_p")] + \
-               [(n, c_float) for n in ("scale", "softcap", "lam", "out_scale", "eps")]
+               [(n, c_float) for n in ("scale", "softcap", "lam", "out_scale", "eps")] + [("window", c_int)]
+
+
+class BranchArg(ctypes.Structure):
+    """One addend of a residual update (csrc/kernels/proj_src.h)."""
+    _fields_ = [("y", ProjArg), ("g", ProjArg), ("gbias", c_void_p), ("pair_pos", c_void_p), ("pair_w", c_void_p),
+                ("top_k", c_int), ("scale", c_float)]
+
+
+class LinAttnArg(ctypes.Structure):
+    """Arguments of the linear-attention kernels (csrc/kernels/linear_attn.h)."""
+    _fields_ = [(n, ProjArg) for n in ("q", "k", "v", "z", "g")] + \
+               [(n, c_void_p) for n in ("w2", "z_bias", "bonus", "norm_w", "state", "slot_ids", "q_start", "q_lens",
+                                        "context_lens", "heads_out", "out")] + [("out_ld", c_longlong)] + \
+               [(n, c_int) for n in ("w2_bf16", "rank", "z_act", "decay", "norm_stride", "gate_act", "bf16", "batch",
+                                     "tokens", "heads", "dim", "vdim")] + \
+               [(n, c_float) for n in ("q_scale", "inv_tau", "out_scale", "eps")]
 
 
 _PP = ctypes.POINTER(ProjArg)
@@ -48,7 +64,16 @@ _SIGNATURES = {
                                    c_int, c_int, _P]),
     "nkb_gemm_simt": (c_int, [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong,
                               _P]),
-    "nkb_gated_residual": (c_int, [_P, _P, _P, c_int, c_int, c_float, c_int, _PP, _PP, ctypes.POINTER(_P), _P, _P, _P,
+    "nkb_gemm_simt_grouped": (c_int, [_P, c_int, _P, c_int, _P, c_int, _P, _P, c_int, c_int, c_int, c_int, c_longlong,
+                                      c_longlong, _P]),
+    "nkb_linattn_scan": (c_int, [ctypes.POINTER(LinAttnArg), _P]),
+    "nkb_linattn_step": (c_int, [ctypes.POINTER(LinAttnArg), _P]),
+    "nkb_low_rank": (c_int, [_PP, c_int, _P, c_int, _P, c_int, c_int, c_int, _P]),
+    "nkb_token_mix": (c_int, [_P, c_int, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P]),
+    "nkb_gate_heads": (c_int, [_P, c_int, c_longlong, c_longlong, _PP, c_int, _P, c_int, c_float, c_float, _P, c_int,
+                               c_longlong, c_int, c_int, c_int, _P]),
+    "nkb_row_norm_append": (c_int, [_PM, _PP, _PP, _PP, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P]),
+    "nkb_gated_residual": (c_int, [_P, _P, _P, c_int, c_int, c_float, c_int, ctypes.POINTER(BranchArg), _P, _P, _P,
                                    c_int, ctypes.POINTER(_P), ctypes.POINTER(_P), c_int, c_int, c_int, c_int, c_float,
                                    _P]),
     "nkb_gated_act": (c_int, [_PP, _PP, _P, c_int, c_int, c_int, c_int, _P]),
@@ -75,8 +100,8 @@ _SIGNATURES = {
     "nkb_moe_a2a_combine": (c_int, [_P, _P, c_int, c_int, c_int, c_int, c_int, ctypes.c_uint, ctypes.POINTER(_P),
                                     ctypes.POINTER(_P), ctypes.POINTER(_P), ctypes.POINTER(_P), ctypes.POINTER(_P),
                                     ctypes.POINTER(_P), _P, _P]),
-    "nkb_moe_dispatch": (c_int, [_P, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, _P, _P, _P, c_int, _P, _P, c_int,
-                                 _P, _P, _P]),
+    "nkb_moe_dispatch": (c_int, [_P, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, _P, _P, _P, _P, c_int, _P, _P,
+                                 c_int, _P, _P, _P]),
     "nkb_moe_combine": (c_int, [_P, _P, _P, c_int, c_int, c_int, _P, _P]),
     "nkb_gemm_effective_splits": (c_int, [c_int, c_int]),
     "nkb_decode_gemm_splits": (c_int, [c_int, c_int, c_int]),
@@ -110,7 +135,8 @@ _SIGNATURES = {
     "nkb_argmax": (c_int, [_P, c_int, _P, _P, c_int, c_int, c_longlong, _P]),
     "nkb_sample": (c_int, [_P, c_int, _P, c_int, c_int, c_longlong, c_float, c_int, c_float, c_ulonglong,
                            c_ulonglong, _P]),
-    "nkb_router_topk": (c_int, [_P, c_int, c_int, c_longlong, _P, _P, _P, c_int, c_int, c_int, c_int, _P]),
+    "nkb_router_topk": (c_int, [_P, c_int, c_int, c_longlong, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
+                                c_float, _P]),
     "nkb_paged_attn_decode": (
         c_int,
         [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P,

@@ -1,11 +1,14 @@
 """Operators of decoders whose layers mix attention and linear recurrences around an fp32 residual stream.
 
-    gated_residual   embedding or residual + gated branches (+ additions ahead of a repeated block), and the
-                     group-wise RMS norms of the sum, in one launch
-    gated_act        act(gate) * up
+    gated_residual   embedding or residual + branches (gated, scaled or routed; + additions ahead of a repeated block),
+                     and the group-wise RMS norms of the sum, in one launch
+    gated_act        act(gate) * up; `activation` for act(x) alone
+    gate_heads       scale * act(gate) * norm(head), the norm optional
     hgrn2            linear attention with a per-channel forget gate; state in slots, fp32
+    row_norm_append  queries and keys normed over all their heads, paged-cache append
     maps_append      interleaved partial RoPE of queries / keys with several score maps, paged-cache append
-    maps_attention   attention with several score maps over shared values (differential attention), score soft cap
+    heads_attention  attention with several score maps over shared values (differential attention), score soft cap;
+                     with one map plain grouped-query attention, also through a sliding window
     linear_simt      products on the CUDA cores: 32-bit models, operands TMA cannot describe
 
 All of them take the projections they consume as `Proj` slices, so a decode-sized batch hands over split-K partial
@@ -24,10 +27,13 @@ import torch
 import torch.nn.functional as F
 
 from . import _lib
-from . import _count_launch, _decode_scratch, _gather_kv, _native, _ptr, _stream, pick_kv_splits
+from . import (_count_launch, _decode_scratch, _gather_kv, _native, _ptr, _stream, flash_attn_prefill,
+               paged_attn_decode, pick_kv_splits)
 
 # name -> (kernel code, PyTorch function)
-ACTIVATIONS = {"silu": (0, F.silu), "gelu_tanh": (1, lambda z: F.gelu(z, approximate="tanh"))}
+ACTIVATIONS = {"silu": (0, F.silu), "gelu_tanh": (1, lambda z: F.gelu(z, approximate="tanh")),
+               "relu2": (2, lambda z: F.relu(z).square()), "tanh": (3, torch.tanh), "sigmoid": (4, torch.sigmoid),
+               "none": (5, lambda z: z)}
 
 
 class Proj(NamedTuple):
@@ -48,6 +54,35 @@ class Proj(NamedTuple):
         split = t.dim() == 3
         return _lib.ProjArg(t.data_ptr() + self.col * t.element_size(), t.stride(-2), t.stride(0) if split else 0,
                             t.shape[0] if split else 1, 1 if t.dtype == torch.bfloat16 else 0)
+
+
+class Branch(NamedTuple):
+    """One addend of a residual update: scale * y; with gate and bias, sigmoid(gate + bias) * y; with pair_pos [T * k] and
+    pair_w [T, k], scale * sum_j pair_w[t, j] * y[pair_pos[t * k + j]] (routed experts)."""
+    y: Proj
+    gate: Optional[Proj] = None
+    bias: Optional[torch.Tensor] = None
+    scale: float = 1.0
+    pair_pos: Optional[torch.Tensor] = None
+    pair_w: Optional[torch.Tensor] = None
+
+    def value(self) -> torch.Tensor:
+        if self.pair_pos is not None:
+            T, k = self.pair_w.shape
+            rows = self.y.value()[self.pair_pos.reshape(T, k).long().clamp(min=0)]
+            w = self.pair_w * (self.pair_pos.reshape(T, k) >= 0)
+            return self.scale * (rows * w[..., None]).sum(1)
+        if self.gate is not None:
+            return self.y.value() * torch.sigmoid(self.gate.value() + self.bias)
+        return self.scale * self.y.value()
+
+    def arg(self) -> _lib.BranchArg:
+        none = _lib.ProjArg(None, 0, 0, 1, 0)
+        if self.gate is not None and (self.scale != 1.0 or self.pair_pos is not None):
+            raise ValueError("a gated branch has neither a scale nor routed rows")
+        return _lib.BranchArg(self.y.arg(), none if self.gate is None else self.gate.arg(), _ptr(self.bias),
+                              _ptr(self.pair_pos), _ptr(self.pair_w), 0 if self.pair_w is None else self.pair_w.shape[1],
+                              float(self.scale))
 
 
 def _ref(p: Proj):
@@ -82,7 +117,7 @@ def group_rmsnorm_ref(x: torch.Tensor, w: torch.Tensor, groups: int, eps: float)
     return y.reshape(x.shape) * w.float()
 
 
-def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Tuple[Proj, Proj, torch.Tensor]] = (), *,
+def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Branch] = (), *,
                    ids: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None, scale: float = 1.0,
                    add_mat: Optional[torch.Tensor] = None, add_row: Optional[torch.Tensor] = None,
                    norms: Sequence[torch.Tensor] = (), groups: int = 1, eps: float = 1e-6,
@@ -90,10 +125,11 @@ def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Tuple[Proj, Pro
     """One residual update of an fp32 stream and the norms that read it.
 
         r = x  (or table[ids] * scale)
-        r += sum over branches (y, g, b) of sigmoid(g + b) * y;   r += add_mat;   r += add_row
+        r += sum over branches (see `Branch`);   r += add_mat;   r += add_row
         h_j = w_j * (r divided, in `groups` equal parts, by sqrt(mean(part^2) + eps))
 
-    x [T, W] fp32; b, add_row and the norm weights fp32 [W]; add_mat fp32 [T, W].  Returns (r, [h_j in `dtype`])."""
+    x [T, W] fp32; gate biases, add_row and the norm weights fp32 [W]; add_mat fp32 [T, W].  Returns (r, [h_j in `dtype`])."""
+    branches = [b if isinstance(b, Branch) else Branch(*b) for b in branches]
     if x is not None:
         rows, width = x.shape
         dev = x.device
@@ -105,7 +141,7 @@ def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Tuple[Proj, Pro
     if not _native(r):
         acc = x.clone() if x is not None else table[ids.long().clamp(0, table.shape[0] - 1)].float() * scale
         if branches:
-            acc = acc + sum(y.value() * torch.sigmoid(g.value() + b) for y, g, b in branches)
+            acc = acc + sum(b.value() for b in branches)
         if add_mat is not None:
             acc = acc + add_mat
         if add_row is not None:
@@ -114,16 +150,14 @@ def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Tuple[Proj, Pro
         for o, w in zip(outs, norms):
             o.copy_(group_rmsnorm_ref(acc, w, groups, eps).to(dtype))
         return r, outs
-    for t in [x, add_mat, add_row, *norms, *[b for _, _, b in branches]]:
+    for t in [x, add_mat, add_row, *norms, *[b.bias for b in branches]]:
         if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
             raise TypeError("gated_residual wants contiguous fp32 residuals, biases and norm weights")
     n = len(branches)
-    ya = (_lib.ProjArg * 2)(*[y.arg() for y, _, _ in branches])
-    ga = (_lib.ProjArg * 2)(*[g.arg() for _, g, _ in branches])
+    ba = (_lib.BranchArg * 2)(*[b.arg() for b in branches])
     rc = _lib.lib().nkb_gated_residual(
         _ptr(x), _ptr(ids), _ptr(table), 1 if table is not None and table.dtype == torch.bfloat16 else 0,
-        table.shape[0] if table is not None else 0, float(scale), n, ya, ga, _ptr_array([b for _, _, b in branches]),
-        _ptr(add_row), _ptr(add_mat), r.data_ptr(), len(outs), _ptr_array(list(norms)), _ptr_array(outs),
+        table.shape[0] if table is not None else 0, float(scale), n, ba, _ptr(add_row), _ptr(add_mat), r.data_ptr(), len(outs), _ptr_array(list(norms)), _ptr_array(outs),
         1 if dtype == torch.bfloat16 else 0, rows, width, int(groups), float(eps), _stream())
     _lib.check(rc, "nkb_gated_residual")
     _count_launch()
@@ -140,6 +174,47 @@ def gated_act(gate: Proj, up: Proj, act: str = "silu", dtype: torch.dtype = torc
     rc = _lib.lib().nkb_gated_act(_ref(gate), _ref(up), out.data_ptr(), 1 if dtype == torch.bfloat16 else 0, rows,
                                   gate.width, ACTIVATIONS[act][0], _stream())
     _lib.check(rc, "nkb_gated_act")
+    _count_launch()
+    return out
+
+
+def activation(x: Proj, act: str, dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
+    """``act(x)`` -> [T, width] in `dtype`."""
+    rows = x.t.shape[-2]
+    out = torch.empty((rows, x.width), dtype=dtype, device=x.t.device)
+    if not _native(out):
+        out.copy_(ACTIVATIONS[act][1](x.value()).to(dtype))
+        return out
+    none = _lib.ProjArg(None, 0, 0, 1, 0)
+    rc = _lib.lib().nkb_gated_act(_ref(x), ctypes.byref(none), out.data_ptr(), 1 if dtype == torch.bfloat16 else 0, rows,
+                                  x.width, ACTIVATIONS[act][0], _stream())
+    _lib.check(rc, "nkb_gated_act")
+    _count_launch()
+    return out
+
+
+def gate_heads(x: torch.Tensor, gate: Proj, act: str, *, norm_w: Optional[torch.Tensor] = None, eps: float = 1e-6,
+               scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``scale * act(gate) * x`` for heads x [T, H, n] (any strides of tokens and heads); with norm_w (fp32, [n] shared by the
+    heads or [H * n]) every head is first divided by its root mean square and multiplied by the weight.  Returns
+    [T, H * n], written to `out` (a slice of columns) when given."""
+    T, H, n = x.shape
+    if out is None:
+        out = torch.empty((T, H * n), dtype=x.dtype, device=x.device)
+    if not _native(x):
+        y = x.float()
+        if norm_w is not None:
+            y = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float().reshape(-1, n)
+        out.copy_((scale * ACTIVATIONS[act][1](gate.value()) * y.reshape(T, H * n)).to(out.dtype))
+        return out
+    if x.stride(2) != 1 or out.stride(1) != 1 or x.dtype != out.dtype:
+        raise ValueError("gate_heads wants unit column strides and one type")
+    stride = 0 if norm_w is None or norm_w.numel() == n else n
+    rc = _lib.lib().nkb_gate_heads(
+        x.data_ptr(), 1 if x.dtype == torch.bfloat16 else 0, x.stride(0), x.stride(1), _ref(gate), ACTIVATIONS[act][0],
+        _ptr(norm_w), stride, float(eps), float(scale), out.data_ptr(), 1 if out.dtype == torch.bfloat16 else 0,
+        out.stride(0), T, H, n, _stream())
+    _lib.check(rc, "nkb_gate_heads")
     _count_launch()
     return out
 
@@ -226,7 +301,9 @@ class MapsSpec:
     """Sizes and constants of attention with `maps` score maps per head over shared values.  Two maps are combined as
     ``a0 - lam * a1``, root-mean-square normed over the head and multiplied by `out_scale`; softcap <= 0: none.
     dim_p / vdim_p are the padded sizes of queries / keys (per map) and values in the cache; the tiled bf16 kernels
-    take 32 or 64 and 64 or 128, other sizes are only rounded to even and use the general kernel."""
+    take 32 or 64 and 64 or 128, other sizes are only rounded to even and use the general kernel.  With one map the tiled
+    kernels are those of plain attention, which take one size of 64 or 128 for both.  window > 0 (one map): a query sees
+    itself and the window - 1 tokens before it."""
     heads: int
     kv_heads: int
     dim: int
@@ -238,19 +315,61 @@ class MapsSpec:
     out_scale: float = 1.0
     eps: float = 1e-6
     tiled: bool = True
+    window: int = 0
+
+    @property
+    def plain(self) -> bool:
+        """Whether the kernels of plain attention serve this (one map, sizes they take)."""
+        return self.tiled and self.maps == 1 and self.softcap <= 0 and max(self.dim, self.vdim) <= 128
 
     @property
     def dim_p(self) -> int:
+        if self.plain:
+            return 64 if max(self.dim, self.vdim) <= 64 else 128
         return _tiled(self.dim, (32, 64) if self.tiled else ())
 
     @property
     def vdim_p(self) -> int:
+        if self.plain:
+            return self.dim_p
         return _tiled(self.vdim, (64, 128) if self.tiled else ())
 
     def arg(self) -> _lib.MapsArg:
         return _lib.MapsArg(self.maps, self.heads, self.kv_heads, self.dim, self.dim_p, self.vdim, self.vdim_p,
                             float(self.scale), float(self.softcap), float(self.lam), float(self.out_scale),
-                            float(self.eps))
+                            float(self.eps), int(self.window))
+
+
+def row_norm_append(spec: MapsSpec, q: Proj, k: Proj, v: Proj, q_norm: torch.Tensor, k_norm: torch.Tensor,
+                    slots: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor) -> torch.Tensor:
+    """RMS norms of a token's whole query and whole key projection (fp32 weights of those widths, spec.eps), keys and
+    values written to their cache slots (negative slot: not stored); returns the queries [T, heads, dim_p]."""
+    T = q.t.shape[-2]
+    H, G, d, dp = spec.heads, spec.kv_heads, spec.dim, spec.dim_p
+    bs = k_cache.shape[2]
+    q_out = torch.empty((T, H, dp), dtype=k_cache.dtype, device=k_cache.device)
+    if not _native(k_cache):
+        def norm(x, w, n):
+            x = x.value()
+            x = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + spec.eps) * w
+            return F.pad(x.reshape(T, n, d), (0, dp - d)).to(k_cache.dtype)
+
+        q_out.copy_(norm(q, q_norm, H))
+        sl = slots.long()
+        keep = sl >= 0
+        blk, off = sl[keep] // bs, sl[keep] % bs
+        k_cache[blk, :, off] = norm(k, k_norm, G)[keep]
+        v_cache[blk, :, off] = F.pad(v.value().reshape(T, G, spec.vdim), (0, spec.vdim_p - spec.vdim))[keep].to(v_cache.dtype)
+        return q_out
+    if q_norm.dtype != torch.float32 or k_norm.dtype != torch.float32:
+        raise TypeError("row_norm_append wants fp32 norm weights")
+    a = spec.arg()
+    rc = _lib.lib().nkb_row_norm_append(ctypes.byref(a), _ref(q), _ref(k), _ref(v), q_norm.data_ptr(), k_norm.data_ptr(),
+                                        slots.data_ptr(), q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
+                                        1 if k_cache.dtype == torch.bfloat16 else 0, T, bs, _stream())
+    _lib.check(rc, "nkb_row_norm_append")
+    _count_launch()
+    return q_out
 
 
 def maps_append(spec: MapsSpec, q: Proj, k: Proj, v: Proj, cos_sin: torch.Tensor, positions: torch.Tensor,
@@ -289,16 +408,32 @@ def maps_append(spec: MapsSpec, q: Proj, k: Proj, v: Proj, cos_sin: torch.Tensor
     return q_out
 
 
-def maps_attention(spec: MapsSpec, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+def maps_attention(*args, **kw) -> torch.Tensor:
+    """`heads_attention` with the heads side by side, [T, heads * vdim]."""
+    return heads_attention(*args, **kw).flatten(1)
+
+
+def heads_attention(spec: MapsSpec, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                    block_table: torch.Tensor, context_lens: torch.Tensor, *, q_start: Optional[torch.Tensor] = None,
                    q_lens: Optional[torch.Tensor] = None, max_q_len: int = 1, num_splits: int = 0) -> torch.Tensor:
     """Causal attention of the new tokens over the paged cache (which already holds them); returns the combined heads
-    [T, heads * vdim].  q_lens None: one new token per sequence (decode); otherwise sequence b owns rows
+    [T, heads, vdim] (strided when the cache's values are padded).  q_lens None: one new token per sequence (decode); otherwise sequence b owns rows
     q_start[b] .. q_start[b] + q_lens[b], the last of which sits at position context_lens[b] - 1."""
     T, H = q.shape[0], spec.heads
     bs = k_cache.shape[2]
     B = block_table.shape[0]
-    out = torch.empty((T, H * spec.vdim), dtype=k_cache.dtype, device=k_cache.device)
+    if spec.window > 0 and spec.maps != 1:
+        raise ValueError("a sliding window is for one score map")
+    if _native(k_cache) and spec.plain:
+        qf = q.reshape(T, -1)
+        if q_lens is None:
+            o = paged_attn_decode(qf, k_cache, v_cache, block_table, context_lens, spec.scale, window=spec.window,
+                                  num_splits=num_splits)
+        else:
+            o = flash_attn_prefill(qf, k_cache, v_cache, block_table, q_start, q_lens, context_lens, spec.scale,
+                                   max_q_len=max_q_len, window=spec.window)
+        return o.view(T, H, spec.vdim_p)[..., :spec.vdim]
+    out = torch.empty((T, H, spec.vdim), dtype=k_cache.dtype, device=k_cache.device)
     if not _native(k_cache):
         M, dp = spec.maps, spec.dim_p
         res = torch.zeros((T, H, spec.vdim))
@@ -315,14 +450,17 @@ def maps_attention(spec: MapsSpec, q: torch.Tensor, k_cache: torch.Tensor, v_cac
             s = torch.einsum("qhmd,khmd->hmqk", q[t0:t0 + n].float().reshape(n, H, M, dp), k) * spec.scale
             if spec.softcap > 0:
                 s = spec.softcap * torch.tanh(s / spec.softcap)
-            vis = torch.arange(ctx)[None, :] <= (ctx - n + torch.arange(n))[:, None]
+            pos = (ctx - n + torch.arange(n))[:, None]
+            vis = torch.arange(ctx)[None, :] <= pos
+            if spec.window > 0:
+                vis &= torch.arange(ctx)[None, :] > pos - spec.window
             a = torch.einsum("hmqk,khv->qhmv", s.masked_fill(~vis, float("-inf")).softmax(-1), v)
             o = a[:, :, 0]
             if M == 2:
                 o = o - spec.lam * a[:, :, 1]
                 o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + spec.eps) * spec.out_scale
             res[t0:t0 + n] = o
-        out.copy_(res.reshape(T, -1).to(out.dtype))
+        out.copy_(res.to(out.dtype))
         return out
     L, a = _lib.lib(), spec.arg()
     ref = ctypes.byref(a)
