@@ -92,11 +92,12 @@ def parse_args():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "eager", "eager-graph"],
                     help="eager-graph: the eager PyTorch decode step captured in a CUDA graph (static cache, position "
                          "on the device), so the comparison is not against Python launch overhead; dense models")
-    ap.add_argument("--model", default="llama3-8b", choices=["llama3-8b", "qwen3-30b-a3b", "gpt-oss-20b", "tolenex"],
-                    help="tolenex: prefill and decode of the layer-by-layer design beside a dense model of equal size")
+    ap.add_argument("--model", default="llama3-8b", choices=["llama3-8b", "qwen3-30b-a3b", "gpt-oss-20b", "tolenex", "mumilorn"],
+                    help="tolenex, mumilorn: prefill and decode of a layer-by-layer design beside the closest other model of "
+                         "equal size")
     ap.add_argument("--sizes", default="2048x5632x16,4096x14336x8",
-                    help="tolenex: width x feed-forward x layers of the compared models")
-    ap.add_argument("--points", default="64x1024,8x4096,1x2048", help="tolenex: batch x prompt length")
+                    help="layer-by-layer designs: width x feed-forward x layers of the compared models")
+    ap.add_argument("--points", default="64x1024,8x4096,1x2048", help="layer-by-layer designs: batch x prompt length")
     ap.add_argument("--batch", type=int, default=None)
     ap.add_argument("--prompt-len", type=int, default=None)
     ap.add_argument("--layers", type=int, default=None, help="debug only: fewer layers (result marked invalid)")
@@ -296,14 +297,14 @@ def main():
         # (examples/models/gpt_oss/peagle/README.md:101-102: 31.5 / 34.7 tok/s base decode on trn2 at TP = 4)
         return C.gpt_oss_20b(), args.batch or 1, args.prompt_len or 128, f"tp{world}-ep{world}"
 
-    cfg, batch, prompt_len, parallelism = shape_of("llama3-8b" if args.model == "tolenex" else args.model)
+    cfg, batch, prompt_len, parallelism = shape_of("llama3-8b" if args.model in LAYERED else args.model)
     debug = False
     if args.layers:
         cfg = cfg.scaled(num_layers=args.layers)
         debug = True
     K, W = args.steps, max(args.warmup, 3)
 
-    if args.model == "tolenex":
+    if args.model in LAYERED:
         return compare_designs(args, tp)
     torch.manual_seed(0)
     weights = random_weights(cfg, tp.rank, world, device=dev, seed=0, std=0.02)
@@ -381,25 +382,37 @@ def main():
     return 0
 
 
-def compare_designs(args, tp):
-    """Prefill and decode throughput of the layer-by-layer design (alternating recurrence and score-map attention
-    layers) and of the dense decoder with the same width, feed-forward, heads, layers and vocabulary.  One JSON line per
-    size and (batch, prompt length)."""
+LAYERED = ("tolenex", "mumilorn")
+
+
+def compared_models(design, width, ff, layers, vocab):
+    """Name -> configuration of a layer-by-layer design and of the models it is put beside: the same width, feed-forward,
+    heads, layers and vocabulary."""
     from nkipy_b200.models import config as C
 
+    heads = width // 128
+    kv = max(1, heads // 4)
+    tolenex = C.tolenex_shape(width, layers=layers, heads=heads, kv_heads=kv, ff=ff, vocab=vocab)
+    if design == "tolenex":
+        return {"tolenex": tolenex,
+                "dense": C.llama3_8b(vocab_size=vocab, hidden_size=width, num_layers=layers, num_heads=heads,
+                                     num_kv_heads=kv, intermediate_size=ff)}
+    shape = dict(layers=layers, heads=heads, kv_heads=kv, ff=ff, vocab=vocab)
+    return {"mumilorn": C.mumilorn_shape(width, **shape),
+            "mumilorn-moe": C.mumilorn_shape(width, **shape, experts=32, top=4, expert_ff=ff // 8, groups=8, keep=4),
+            "tolenex": tolenex}
+
+
+def compare_designs(args, tp):
+    """Prefill and decode throughput of a layer-by-layer design and of the closest other model of equal size.  One JSON
+    line per model, size and (batch, prompt length)."""
     if tp.world_size != 1:
-        raise SystemExit("--model tolenex runs on one GPU")
+        raise SystemExit(f"--model {args.model} runs on one GPU")
     K, W = args.steps, max(args.warmup, 3)
     vocab = 32000
     for size in args.sizes.split(","):
         width, ff, layers = (int(x) for x in size.split("x"))
-        heads = width // 128
-        kv = max(1, heads // 4)
-        models = {
-            "tolenex": C.tolenex_shape(width, layers=layers, heads=heads, kv_heads=kv, ff=ff, vocab=vocab),
-            "dense": C.llama3_8b(vocab_size=vocab, hidden_size=width, num_layers=layers, num_heads=heads,
-                                 num_kv_heads=kv, intermediate_size=ff),
-        }
+        models = compared_models(args.model, width, ff, layers, vocab)
         for point in args.points.split(","):
             batch, prompt = (int(x) for x in point.split("x"))
             for name, cfg in models.items():
@@ -409,7 +422,7 @@ def compare_designs(args, tp):
                     "ms_per_step": round(r["ms_per_step"], 4), "e2e_tokens_per_s": round(r["e2e_value"], 1),
                     "prefill_tokens_per_s": round(batch * prompt / r["prefill_s"], 1), "prefill_s": round(r["prefill_s"], 4),
                     "launches_per_step": r["launches_per_step"], "params_m": round(cfg.param_count() / 1e6, 1),
-                    "config": {"width": width, "ff": ff, "layers": layers, "heads": heads, "kv_heads": kv, "vocab": vocab,
+                    "config": {"width": width, "ff": ff, "layers": layers, "heads": width // 128, "vocab": vocab,
                                "batch": batch, "prompt_len": prompt},
                     "steps": K, "warmup": W, "dtype": "bf16", "data": "synthetic", "clocks": r["clocks"]}), flush=True)
     return 0

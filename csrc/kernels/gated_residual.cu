@@ -74,9 +74,12 @@ __device__ __forceinline__ void pair_rows(float (&s)[V], const NkbBranch& br, lo
   for (int j = 0; j < V; ++j) s[j] = fmaf(br.scale, a[j], s[j]);
 }
 
+// What the branches of a launch are: all gated, all plain (scaled), or any mixture with routed ones.
+enum { BR_GATED = 0, BR_PLAIN = 1, BR_ANY = 2 };
+
 // PACKED: every projection is bf16 and aligned (prefill), which keeps the kernel at few registers and many CTAs per SM
-template <int V, bool PACKED, typename OutT>
-__global__ void __launch_bounds__(PACKED ? 256 : 1024, PACKED ? 6 : 1)
+template <int V, bool PACKED, int MODE, typename OutT>
+__global__ void __launch_bounds__(PACKED ? 256 : 1024, PACKED ? (MODE == BR_ANY ? 4 : 6) : 1)
 gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
   extern __shared__ float row_s[];                 // [width] then [groups]
   __shared__ float red[32];
@@ -102,24 +105,39 @@ gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
     }
 #pragma unroll
     for (int j = 0; j < V; ++j) s[j] = 0.f;
-    if constexpr (PACKED) {
+    if constexpr (MODE == BR_ANY) {
+#pragma unroll 1
+      for (int b = 0; b < p.branches; ++b) {
+        if (p.br[b].pair_pos) {
+          pair_rows<V>(s, p.br[b], t, c);
+          continue;
+        }
+        float y[V], w[V];
+        proj_vec<V>(y, p.br[b].y, t, c);
+#pragma unroll
+        for (int j = 0; j < V; ++j) w[j] = p.br[b].scale;
+        if (p.br[b].g.ptr) {
+          proj_vec<V>(w, p.br[b].g, t, c);
+#pragma unroll
+          for (int j = 0; j < V; ++j) w[j] = sigmoid_f(w[j] + p.br[b].gbias[c + j]);
+        }
+#pragma unroll
+        for (int j = 0; j < V; ++j) s[j] = fmaf(w[j], y[j], s[j]);
+      }
+    } else if constexpr (PACKED) {
       uint2 y[2], g[2];
 #pragma unroll
       for (int b = 0; b < 2; ++b)
-        if (b < p.branches && !p.br[b].pair_pos) {
+        if (b < p.branches) {
           y[b] = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.br[b].y.ptr) + t * p.br[b].y.ld + c);
-          if (p.br[b].g.ptr)
+          if constexpr (MODE == BR_GATED)
             g[b] = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.br[b].g.ptr) + t * p.br[b].g.ld + c);
         }
 #pragma unroll
       for (int b = 0; b < 2; ++b)
         if (b < p.branches) {
-          if (p.br[b].pair_pos) {
-            pair_rows<V>(s, p.br[b], t, c);
-            continue;
-          }
           const float2 y0 = unpack_bf16x2(y[b].x), y1 = unpack_bf16x2(y[b].y);
-          if (p.br[b].g.ptr) {
+          if constexpr (MODE == BR_GATED) {
             const float4 bias = *reinterpret_cast<const float4*>(p.br[b].gbias + c);
             const float2 g0 = unpack_bf16x2(g[b].x), g1 = unpack_bf16x2(g[b].y);
             s[0] += y0.x * sigmoid_f(g0.x + bias.x);
@@ -138,16 +156,14 @@ gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
       float y[2][V], g[2][V];
 #pragma unroll
       for (int b = 0; b < 2; ++b)
-        if (b < p.branches && !p.br[b].pair_pos) {
+        if (b < p.branches) {
           proj_vec<V>(y[b], p.br[b].y, t, c);
-          if (p.br[b].g.ptr) proj_vec<V>(g[b], p.br[b].g, t, c);
+          if constexpr (MODE == BR_GATED) proj_vec<V>(g[b], p.br[b].g, t, c);
         }
 #pragma unroll
       for (int b = 0; b < 2; ++b)
         if (b < p.branches) {
-          if (p.br[b].pair_pos) {
-            pair_rows<V>(s, p.br[b], t, c);
-          } else if (p.br[b].g.ptr) {
+          if constexpr (MODE == BR_GATED) {
             float bias[V];
             load_vec<V>(bias, p.br[b].gbias + c);
 #pragma unroll
@@ -267,6 +283,20 @@ using namespace nkb;
 
 static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
+template <int MODE>
+static int launch_residual(const GatedResidualParams& p, bool packed, bool vec, int out_bf16, dim3 grid, dim3 block,
+                           size_t smem, cudaStream_t s) {
+  using bf = __nv_bfloat16;
+  if (packed)
+    return out_bf16 ? launch_pdl(gated_residual_kernel<4, true, MODE, bf>, grid, block, smem, s, p)
+                    : launch_pdl(gated_residual_kernel<4, true, MODE, float>, grid, block, smem, s, p);
+  if (vec)
+    return out_bf16 ? launch_pdl(gated_residual_kernel<4, false, MODE, bf>, grid, block, smem, s, p)
+                    : launch_pdl(gated_residual_kernel<4, false, MODE, float>, grid, block, smem, s, p);
+  return out_bf16 ? launch_pdl(gated_residual_kernel<1, false, MODE, bf>, grid, block, smem, s, p)
+                  : launch_pdl(gated_residual_kernel<1, false, MODE, float>, grid, block, smem, s, p);
+}
+
 extern "C" int nkb_gated_residual(const float* x_in, const int* ids, const void* table, int table_bf16, int vocab,
                                   float scale, int branches, const NkbBranch* br, const float* add_row,
                                   const float* add_mat, float* x_out, int norms, const float* const* w,
@@ -297,16 +327,19 @@ extern "C" int nkb_gated_residual(const float* x_in, const int* ids, const void*
   const int threads = nv >= most ? most : (nv < 64 ? 64 : (nv + 31) / 32 * 32);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (smem > 48 * 1024) return -2;
-  using bf = __nv_bfloat16;
   const dim3 grid(rows), block(threads);
-  if (packed)
-    return out_bf16 ? launch_pdl(gated_residual_kernel<4, true, bf>, grid, block, smem, s, p)
-                    : launch_pdl(gated_residual_kernel<4, true, float>, grid, block, smem, s, p);
-  if (vec)
-    return out_bf16 ? launch_pdl(gated_residual_kernel<4, false, bf>, grid, block, smem, s, p)
-                    : launch_pdl(gated_residual_kernel<4, false, float>, grid, block, smem, s, p);
-  return out_bf16 ? launch_pdl(gated_residual_kernel<1, false, bf>, grid, block, smem, s, p)
-                  : launch_pdl(gated_residual_kernel<1, false, float>, grid, block, smem, s, p);
+  int mode = BR_GATED;
+  if (branches > 0) {
+    int gated = 0, routed = 0;
+    for (int i = 0; i < branches; ++i) {
+      gated += br[i].g.ptr != nullptr;
+      routed += br[i].pair_pos != nullptr;
+    }
+    mode = routed || (gated && gated < branches) ? BR_ANY : (gated ? BR_GATED : BR_PLAIN);
+  }
+  if (mode == BR_GATED) return launch_residual<BR_GATED>(p, packed, vec, out_bf16, grid, block, smem, s);
+  if (mode == BR_PLAIN) return launch_residual<BR_PLAIN>(p, packed, vec, out_bf16, grid, block, smem, s);
+  return launch_residual<BR_ANY>(p, packed, vec, out_bf16, grid, block, smem, s);
 }
 
 extern "C" int nkb_gated_act(const NkbProj* gate, const NkbProj* up, void* out, int out_bf16, int rows, int inter,

@@ -21,8 +21,14 @@
 
 namespace nkb {
 
-// z already includes its bias.  sigmoid(z)^t = exp(-t * log(1 + exp(-z))), the logarithm in its stable form.
+// z already includes its bias.  sigmoid(z)^t = exp(-t * log(1 + exp(-z))), the logarithm in its stable form.  FAST uses the
+// hardware's approximate exponential and logarithm (a few units in the last place of fp32), which bf16 inputs do not notice.
+template <bool FAST>
 __device__ __forceinline__ float decay_of(float z, int kind, float inv_tau) {
+  if constexpr (FAST) {
+    if (kind == NKB_DECAY_DOUBLE_EXP) return __expf(-__expf(z));
+    return __expf(-inv_tau * (fmaxf(-z, 0.f) + __logf(1.f + __expf(-fabsf(z)))));
+  }
   if (kind == NKB_DECAY_DOUBLE_EXP) return expf(-expf(z));
   return expf(-inv_tau * (fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))));
 }
@@ -219,17 +225,16 @@ __global__ void __launch_bounds__(kScanThreads, CL <= 8 ? 4 : 1) linattn_scan_ke
   __nv_bfloat16(*kr)[DP] = qr + TT;
   __nv_bfloat16(*vr)[COLS] = reinterpret_cast<__nv_bfloat16(*)[COLS]>(kr + TT);
   __shared__ float bon[TT][BW];
+  __shared__ __align__(16) float zbs[DP], uus[BONUS ? DP : 4];
   const int head = blockIdx.y, b = blockIdx.z, col0 = blockIdx.x * COLS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane & 15;
   const int cl0 = (warp * 2 + (lane >> 4)) * NC;    // first of this lane's columns within the CTA
   const int hq = head * p.dim, hv = head * p.vdim, dim_p = (p.dim + 3) / 4 * 4;
   // the channels this thread prepares are the same in every pass over a tile
   const int pc = (threadIdx.x % QW) * 4;
-  float zb[4], uu[4];
-#pragma unroll
-  for (int e = 0; e < 4; ++e) {
-    zb[e] = pc + e < p.dim ? p.z_bias[hq + pc + e] : 0.f;
-    uu[e] = BONUS && pc + e < p.dim ? p.bonus[hq + pc + e] : 0.f;
+  for (int c = threadIdx.x; c < DP; c += kScanThreads) {
+    zbs[c] = c < p.dim ? p.z_bias[hq + c] : 0.f;
+    if (BONUS) uus[c] = c < p.dim ? p.bonus[hq + c] : 0.f;
   }
   griddep_wait();
   griddep_launch();
@@ -291,14 +296,15 @@ __global__ void __launch_bounds__(kScanThreads, CL <= 8 ? 4 : 1) linattn_scan_ke
         for (int e = 0; e < 4; ++e) {
           q[e] = qv[e] * p.q_scale;
           k[e] = kv[e];
-          a[e] = decay_of(zv[e] + zb[e], p.decay, p.inv_tau);
+          a[e] = decay_of<ASYNC>(zv[e] + zbs[pc + e], p.decay, p.inv_tau);
         }
       }
       *reinterpret_cast<float4*>(&qs[tok][pc]) = make_float4(q[0], q[1], q[2], q[3]);
       *reinterpret_cast<float4*>(&ks[tok][pc]) = make_float4(k[0], k[1], k[2], k[3]);
       *reinterpret_cast<float4*>(&as[tok][pc]) = make_float4(a[0], a[1], a[2], a[3]);
       if constexpr (BONUS) {
-        float s = q[0] * uu[0] * k[0] + q[1] * uu[1] * k[1] + q[2] * uu[2] * k[2] + q[3] * uu[3] * k[3];
+        const float4 u4 = *reinterpret_cast<const float4*>(&uus[pc]);
+        float s = q[0] * u4.x * k[0] + q[1] * u4.y * k[1] + q[2] * u4.z * k[2] + q[3] * u4.w * k[3];
 #pragma unroll
         for (int w = (QW < 32 ? QW : 32) / 2; w > 0; w >>= 1) s += __shfl_xor_sync(0xffffffffu, s, w);
         if (threadIdx.x % (QW < 32 ? QW : 32) == 0) bon[tok][BW > 1 ? (threadIdx.x % QW) / 32 : 0] = s;
@@ -422,6 +428,12 @@ __global__ void __launch_bounds__(kScanThreads, CL <= 8 ? 4 : 1) linattn_scan_ke
 }
 
 // ------------------------------------------------------------------------------------------------ gate heads
+// the two gates in use, without the switch over all activations where a kernel is bound by issue slots
+__device__ __forceinline__ float apply_gate(float z, int kind) {
+  if (kind == ACT_SILU || kind == ACT_SIGMOID) return (kind == ACT_SILU ? z : 1.f) * __fdividef(1.f, 1.f + __expf(-z));
+  return apply_act(z, kind);
+}
+
 struct GateHeadsParams {
   const void* x;            // token t, head h: x + t * ld_token + h * ld_head
   long long ld_token, ld_head;
@@ -494,6 +506,69 @@ __global__ void __launch_bounds__(256) gate_heads_kernel(const __grid_constant__
                             apply_act(proj_load(p.g, t, h * p.width + c), p.gate_act));
 }
 
+// bf16 heads of a multiple of eight elements, at most 256: L lanes share a head, a lane holds eight consecutive elements.
+template <int L>
+__global__ void __launch_bounds__(256) gate_heads8_kernel(const __grid_constant__ GateHeadsParams p) {
+  using bf = __nv_bfloat16;
+  const int per = 256 / L, lane = threadIdx.x & (L - 1), c = lane * 8;
+  const bool on = c < p.width;
+  griddep_wait();
+  griddep_launch();
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const long long i = (blockIdx.x * 2ll + u) * per + threadIdx.x / L;
+    if (i - threadIdx.x / L >= p.rows) return;              // uniform
+    const bool live = i < p.rows && on;
+    const long long t = live ? int(i) / p.heads : 0;
+    const int h = live ? int(i) % p.heads : 0;
+    float x[8], g[8];
+    if (live) {
+      const uint4 r = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(p.x) + t * p.ld_token + h * p.ld_head + c);
+      const int col = h * p.width + c;
+      if (p.g.bf16) {
+        const uint4 q = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(p.g.ptr) + t * p.g.ld + col);
+        const uint32_t qw[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 f = unpack_bf16x2(qw[e]);
+          g[2 * e] = f.x;
+          g[2 * e + 1] = f.y;
+        }
+      } else {
+        const float4 lo = proj_load4(p.g, t, col), hi = proj_load4(p.g, t, col + 4);
+        g[0] = lo.x; g[1] = lo.y; g[2] = lo.z; g[3] = lo.w;
+        g[4] = hi.x; g[5] = hi.y; g[6] = hi.z; g[7] = hi.w;
+      }
+      const uint32_t rw[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 f = unpack_bf16x2(rw[e]);
+        x[2 * e] = f.x;
+        x[2 * e + 1] = f.y;
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] = g[e] = 0.f;
+    }
+    float inv = p.scale;
+    if (p.norm_w) {
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
+#pragma unroll
+      for (int w = L / 2; w > 0; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
+      inv *= 1.f / sqrtf(ss / float(p.width) + p.eps);
+    }
+    if (live) {
+      const float* w = p.norm_w ? p.norm_w + (long long)h * p.norm_stride + c : nullptr;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] *= inv * (w ? w[e] : 1.f) * apply_gate(g[e], p.gate_act);
+      *reinterpret_cast<uint4*>(reinterpret_cast<bf*>(p.out) + t * p.out_ld + (long long)h * p.width + c) =
+          make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
+    }
+  }
+}
+
 static bool al(const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
 
 static int launch_gate_heads(const GateHeadsParams& p, int x_bf16, int out_bf16, cudaStream_t s) {
@@ -503,6 +578,14 @@ static int launch_gate_heads(const GateHeadsParams& p, int x_bf16, int out_bf16,
                    (!p.norm_w || (al(p.norm_w, 16) && p.norm_stride % 4 == 0));
   const dim3 grid(unsigned((p.rows + 7) / 8)), block(256);
   using bf = __nv_bfloat16;
+  if (x_bf16 && out_bf16 && p.width % 8 == 0 && p.width <= 256 && p.rows < (1ll << 30) && p.ld_token % 8 == 0 &&
+      p.ld_head % 8 == 0 && p.out_ld % 8 == 0 && al(p.x, 16) && al(p.out, 16) && proj_vec4_ok(p.g) &&
+      (!p.g.bf16 || (al(p.g.ptr, 16) && p.g.ld % 8 == 0))) {
+    const auto blocks = [&](int lanes) { return dim3(unsigned((p.rows + 512 / lanes - 1) / (512 / lanes))); };
+    if (p.width <= 64) return launch_pdl(gate_heads8_kernel<8>, blocks(8), block, 0, s, p);
+    if (p.width <= 128) return launch_pdl(gate_heads8_kernel<16>, blocks(16), block, 0, s, p);
+    return launch_pdl(gate_heads8_kernel<32>, blocks(32), block, 0, s, p);
+  }
   if (x_bf16 && out_bf16)
     return vec ? launch_pdl(gate_heads_kernel<true, bf, bf>, grid, block, 0, s, p)
                : launch_pdl(gate_heads_kernel<false, bf, bf>, grid, block, 0, s, p);
@@ -595,7 +678,7 @@ __global__ void __launch_bounds__(kStepThreads) linattn_step_kernel(const __grid
       }
 #pragma unroll
       for (int w = P / 2; w > 0; w >>= 1) z += __shfl_xor_sync(0xffffffffu, z, w);
-      if (part == 0 && c < D8) as[c] = c < p.dim ? decay_of(z + p.z_bias[hq + c], p.decay, p.inv_tau) : 1.f;
+      if (part == 0 && c < D8) as[c] = c < p.dim ? decay_of<sizeof(OutT) == 2>(z + p.z_bias[hq + c], p.decay, p.inv_tau) : 1.f;
       __syncthreads();
     }
 #pragma unroll

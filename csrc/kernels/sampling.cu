@@ -228,6 +228,8 @@ __global__ void __launch_bounds__(1024) sample_kernel(const void* __restrict__ l
 // largest single score take part.  The weights are multiplied by `scale`.
 // ---------------------------------------------------------------------------
 // logits may be bf16 / fp32 [tokens, E] or fp32 split-K partials [splits, tokens, E] (summed here, plus bias)
+// kPer: experts per lane
+template <int kPer>
 __global__ void router_topk_kernel(const void* __restrict__ logits, int is_fp32, int splits, long long split_stride,
                                    const __nv_bfloat16* __restrict__ bias, float* __restrict__ weights,
                                    int* __restrict__ experts, int tokens, int num_experts, int top_k, int mode,
@@ -237,7 +239,6 @@ __global__ void router_topk_kernel(const void* __restrict__ logits, int is_fp32,
   griddep_wait();
   griddep_launch();
   if (warp >= tokens) return;
-  constexpr int kPer = 32;
   float v[kPer];
   const int per = (num_experts + 31) / 32;
   float mx = -FLT_MAX;
@@ -246,6 +247,7 @@ __global__ void router_topk_kernel(const void* __restrict__ logits, int is_fp32,
     const int e = j * 32 + lane;
     if (j < per && e < num_experts) {
       float a = load_logit(logits, is_fp32, (long long)warp * num_experts + e);
+#pragma unroll 8
       for (int s = 1; s < splits; ++s)
         a += reinterpret_cast<const float*>(logits)[s * split_stride + (long long)warp * num_experts + e];
       if (bias) a += __bfloat162float(bias[e]);
@@ -350,7 +352,14 @@ extern "C" int nkb_router_topk(const void* logits, int is_fp32, int splits, long
   const int blocks = (tokens * 32 + threads - 1) / threads;
   if (splits < 1) splits = 1;
   if (splits > 1 && !is_fp32) return -2;
-  return launch_pdl(router_topk_kernel, dim3(blocks), dim3(threads), 0, reinterpret_cast<cudaStream_t>(stream), logits,
-                    is_fp32, splits, split_stride, (const __nv_bfloat16*)bias, weights, experts, tokens, num_experts,
-                    top_k, mode, groups, keep, scale);
+  const auto go = [&](auto kernel) {
+    return launch_pdl(kernel, dim3(blocks), dim3(threads), 0, reinterpret_cast<cudaStream_t>(stream), logits, is_fp32, splits,
+                      split_stride, (const __nv_bfloat16*)bias, weights, experts, tokens, num_experts, top_k, mode, groups, keep,
+                      scale);
+  };
+  if (num_experts <= 32) return go(router_topk_kernel<1>);
+  if (num_experts <= 64) return go(router_topk_kernel<2>);
+  if (num_experts <= 128) return go(router_topk_kernel<4>);
+  if (num_experts <= 256) return go(router_topk_kernel<8>);
+  return go(router_topk_kernel<32>);
 }

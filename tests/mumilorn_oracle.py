@@ -164,3 +164,56 @@ def forward(raw, weights, ids):
                 x = x + experts(h, under(w, "mlp."), m)
         taps.append(x)
     return pre_norm(x, W["final.norm"], eps) @ W["embed"].T, taps
+
+
+# ----------------------------------------------------------------------------- small models for the tests
+def small_config(width=96, vocab=160, layers="gpg", mlps="dmd", heads=4, kv_heads=2, dim=24, vdim=40, window=21, scale=None,
+                 lheads=3, ldim=20, lvdim=28, tau=8.0, rheads=2, rdim=24, left_scale=0.6, right_scale=1.3, ff=112, experts=6,
+                 top=2, eff=40, groups=(3, 2), rscale=1.7, eps=1e-5):
+    """config.json contents: layers 'g' gated linear attention, 'p' parallel; mlps 'd' dense, 'm' routed, '-' none."""
+    specs = []
+    for c, f in zip(layers, mlps):
+        if c == "g":
+            kind, m = "gla", {"heads": lheads, "dim": ldim, "vdim": lvdim, "tau": tau}
+        else:
+            kind = "parallel"
+            m = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": window},
+                          "scale": scale or dim ** -0.5},
+                 "right": {"heads": rheads, "dim": rdim}, "left_scale": left_scale, "right_scale": right_scale}
+        mlp = {"d": {"kind": "dense", "ff": ff}, "-": None,
+               "m": {"kind": "moe", "expert": {"ff": eff},
+                     "router": {"experts": experts, "top": top, "scale": rscale,
+                                "groups": {"count": groups[0], "keep": groups[1]} if groups else None}}}[f]
+        specs.append({"type": kind, "mixer": m, "mlp": mlp})
+    return {"architecture": "Mumilorn", "layers": specs, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def small_weights(raw, shapes, seed=0):
+    """bf16 tensors of the given name -> shape map, scaled so that every mechanism has a visible effect: slow decays with a
+    few fast channels, scores of several units, mixes over the whole range, strong bonus, decided routers."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in shapes.items():
+        x, leaf = torch.randn(shape, generator=g), name.rsplit(".", 1)[-1]
+        if leaf in ("norm1", "norm2") or name == "final.norm":
+            x = 0.3 * x
+        elif name.endswith(("q.norm", "k.norm")):
+            x = 1.6 + 0.4 * x
+        elif leaf == "norm":
+            x = 1 + 0.3 * x
+        elif ".mu." in name:
+            x = torch.rand(shape, generator=g)
+        elif leaf == "w0":
+            x = -2.5 + 1.5 * x
+        elif leaf == "b":
+            x = 1 + 1.5 * x
+        elif leaf == "u":
+            x = 1.5 * x
+        elif leaf == "router":
+            x = x * 4 / shape[-1] ** 0.5
+        elif leaf in ("w2", "a2"):
+            x = x / shape[-1] ** 0.5
+        elif len(shape) == 2 and name != "embed":
+            x = x / shape[-1] ** 0.5
+        out[name] = x.to(torch.bfloat16)
+    return out
