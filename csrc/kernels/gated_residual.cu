@@ -56,19 +56,38 @@ __device__ __forceinline__ void proj_vec(float (&a)[V], const NkbProj& s, long l
   }
 }
 
+constexpr int kMaxTop = 32;
+
+// Sum of a token's routed rows, four at a time so that their loads are in flight together; pos / w: the token's pairs.
 template <int V>
-__device__ __forceinline__ void pair_rows(float (&s)[V], const NkbBranch& br, long long t, int c) {
+__device__ __forceinline__ void pair_rows(float (&s)[V], const NkbBranch& br, const int* pos, const float* w, int c) {
   float a[V];
 #pragma unroll
   for (int j = 0; j < V; ++j) a[j] = 0.f;
-#pragma unroll 4
-  for (int i = 0; i < br.top_k; ++i) {
-    const int pos = br.pair_pos[t * br.top_k + i];
-    const float w = br.pair_w[t * br.top_k + i];
-    float r[V];
-    proj_vec<V>(r, br.y, max(pos, 0), c);
+  if (V == 4 && br.y.bf16) {
+    const __nv_bfloat16* y = reinterpret_cast<const __nv_bfloat16*>(br.y.ptr) + c;
+#pragma unroll 1
+    for (int i0 = 0; i0 < br.top_k; i0 += 4) {
+      uint2 r[4];
 #pragma unroll
-    for (int j = 0; j < V; ++j) a[j] = pos >= 0 ? fmaf(w, r[j], a[j]) : a[j];
+      for (int i = 0; i < 4; ++i)
+        r[i] = i0 + i < br.top_k ? *reinterpret_cast<const uint2*>(y + pos[i0 + i] * br.y.ld) : make_uint2(0u, 0u);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 lo = unpack_bf16x2(r[i].x), hi = unpack_bf16x2(r[i].y);
+        const float x[4] = {lo.x, lo.y, hi.x, hi.y}, wi = i0 + i < br.top_k ? w[i0 + i] : 0.f;
+#pragma unroll
+        for (int j = 0; j < V; ++j) a[j] = fmaf(wi, x[j & 3], a[j]);
+      }
+    }
+  } else {
+#pragma unroll 1
+    for (int i = 0; i < br.top_k; ++i) {
+      float r[V];
+      proj_vec<V>(r, br.y, pos[i], c);
+#pragma unroll
+      for (int j = 0; j < V; ++j) a[j] = fmaf(w[i], r[j], a[j]);
+    }
   }
 #pragma unroll
   for (int j = 0; j < V; ++j) s[j] = fmaf(br.scale, a[j], s[j]);
@@ -79,7 +98,7 @@ enum { BR_GATED = 0, BR_PLAIN = 1, BR_ANY = 2 };
 
 // PACKED: every projection is bf16 and aligned (prefill), which keeps the kernel at few registers and many CTAs per SM
 template <int V, bool PACKED, int MODE, typename OutT>
-__global__ void __launch_bounds__(PACKED ? 256 : 1024, PACKED ? (MODE == BR_ANY ? 4 : 6) : 1)
+__global__ void __launch_bounds__(PACKED ? 256 : 1024, PACKED ? (MODE == BR_ANY ? 5 : 6) : 1)
 gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
   extern __shared__ float row_s[];                 // [width] then [groups]
   __shared__ float red[32];
@@ -90,6 +109,18 @@ gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
   griddep_wait();
   griddep_launch();
   const int id = p.ids ? min(max(p.ids[t], 0), p.vocab - 1) : 0;
+  __shared__ int pos_s[MODE == BR_ANY ? 2 : 1][MODE == BR_ANY ? kMaxTop : 1];
+  __shared__ float pw_s[MODE == BR_ANY ? 2 : 1][MODE == BR_ANY ? kMaxTop : 1];
+  if constexpr (MODE == BR_ANY) {
+    // rows of pairs that are handled elsewhere count with weight zero (of a row that exists)
+    for (int b = 0; b < p.branches; ++b)
+      if (p.br[b].pair_pos && int(threadIdx.x) < p.br[b].top_k) {
+        const int pos = p.br[b].pair_pos[t * p.br[b].top_k + threadIdx.x];
+        pos_s[b][threadIdx.x] = max(pos, 0);
+        pw_s[b][threadIdx.x] = pos >= 0 ? p.br[b].pair_w[t * p.br[b].top_k + threadIdx.x] : 0.f;
+      }
+    __syncthreads();
+  }
   for (int i = threadIdx.x; i < nv; i += blockDim.x) {
     const int c = i * V;
     float a[V], s[V];
@@ -109,7 +140,7 @@ gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
 #pragma unroll 1
       for (int b = 0; b < p.branches; ++b) {
         if (p.br[b].pair_pos) {
-          pair_rows<V>(s, p.br[b], t, c);
+          pair_rows<V>(s, p.br[b], pos_s[b], pw_s[b], c);
           continue;
         }
         float y[V], w[V];
@@ -311,6 +342,7 @@ extern "C" int nkb_gated_residual(const float* x_in, const int* ids, const void*
   bool vec = width % 4 == 0 && (width / groups) % 4 == 0 && (!x_in || aligned16(x_in)) && (!x_out || aligned16(x_out));
   for (int b = 0; b < branches; ++b) {
     p.br[b] = br[b];
+    if (br[b].pair_pos && (br[b].top_k < 1 || br[b].top_k > kMaxTop || !br[b].pair_w || br[b].g.ptr)) return -2;
     vec = vec && proj_vec4_ok(br[b].y) && proj_vec4_ok(br[b].g) && aligned16(br[b].gbias);
   }
   for (int n = 0; n < norms; ++n) {

@@ -54,20 +54,51 @@ struct TokenMixParams {
   int batch, tokens, width, mixes;
 };
 constexpr int kMixTokens = 8;     // tokens of a CTA in prompts
-constexpr int kMaxMixes = 8;
+constexpr int kMaxMixes = 5;
 
-// A CTA owns a run of TB tokens and 256 V columns.  The first row of a portion reads what the last row writes, so the CTA
+// V consecutive elements in registers: 16 bytes of bf16 (V = 8), 16 bytes of fp32 (V = 4) or one element
+template <int V, typename T>
+__device__ __forceinline__ void load_run(float (&x)[V], const T* p) {
+  if constexpr (V == 8) {
+    const uint4 r = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = unpack_bf16x2(w[e]);
+      x[2 * e] = f.x;
+      x[2 * e + 1] = f.y;
+    }
+  } else if constexpr (V == 4) {
+    const float4 r = *reinterpret_cast<const float4*>(p);
+    x[0] = r.x; x[1] = r.y; x[2] = r.z; x[3] = r.w;
+  } else {
+    x[0] = cast_in<T>(*p);
+  }
+}
+template <int V, typename T>
+__device__ __forceinline__ void store_run(T* p, const float (&x)[V]) {
+  if constexpr (V == 8) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]),
+                                              pack_bf16x2(x[6], x[7]));
+  } else if constexpr (V == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+  } else {
+    *p = cast_out<T>(x[0]);
+  }
+}
+
+// A CTA owns a run of TB tokens and 128 V columns.  The first row of a portion reads what the last row writes, so the CTA
 // that holds a sequence's last row also mixes its first one (before it stores), and the first row's own CTA leaves it out.
 template <int V, int TB, typename T>
-__global__ void __launch_bounds__(256) token_mix_kernel(const __grid_constant__ TokenMixParams p) {
+__global__ void __launch_bounds__(128) token_mix_kernel(const __grid_constant__ TokenMixParams p) {
   __shared__ int first_of[TB], last_of[TB];     // sequence that starts / ends at each token of the run, or -1
   const int t0 = blockIdx.y * TB, nt = min(TB, p.tokens - t0);
-  const int c = (blockIdx.x * 256 + threadIdx.x) * V;
+  const int c = (blockIdx.x * 128 + threadIdx.x) * V;
   if (threadIdx.x < TB) first_of[threadIdx.x] = last_of[threadIdx.x] = -1;
   griddep_wait();
   griddep_launch();
   __syncthreads();
-  for (int b = threadIdx.x; b < p.batch; b += 256) {
+  for (int b = threadIdx.x; b < p.batch; b += 128) {
     const int s = p.q_lens ? p.q_start[b] : b, n = p.q_lens ? p.q_lens[b] : 1;
     if (n <= 0) continue;
     if (s >= t0 && s < t0 + nt) first_of[s - t0] = b;
@@ -75,24 +106,14 @@ __global__ void __launch_bounds__(256) token_mix_kernel(const __grid_constant__ 
   }
   __syncthreads();
   if (c >= p.width) return;
-  const T* h = reinterpret_cast<const T*>(p.h);
-  T* out = reinterpret_cast<T*>(p.out);
+  const T* h = reinterpret_cast<const T*>(p.h) + c;
+  T* out = reinterpret_cast<T*>(p.out) + c;
   float mu[kMaxMixes][V];
 #pragma unroll
   for (int m = 0; m < kMaxMixes; ++m)
     if (m < p.mixes)
 #pragma unroll
       for (int j = 0; j < V; ++j) mu[m][j] = p.mu[(long long)m * p.width + c + j];
-  auto load_row = [&](float (&x)[V], long long t) {
-    if constexpr (V == 4 && sizeof(T) == 2) {
-      const uint2 r = *reinterpret_cast<const uint2*>(h + t * p.width + c);
-      const float2 a = unpack_bf16x2(r.x), b = unpack_bf16x2(r.y);
-      x[0] = a.x; x[1] = a.y; x[2] = b.x; x[3] = b.y;
-    } else {
-#pragma unroll
-      for (int j = 0; j < V; ++j) x[j] = cast_in<T>(h[t * p.width + c + j]);
-    }
-  };
   auto emit = [&](long long t, const float (&prev)[V], const float (&x)[V]) {
 #pragma unroll
     for (int m = 0; m < kMaxMixes; ++m)
@@ -100,38 +121,38 @@ __global__ void __launch_bounds__(256) token_mix_kernel(const __grid_constant__ 
         float y[V];
 #pragma unroll
         for (int j = 0; j < V; ++j) y[j] = fmaf(prev[j] - x[j], mu[m][j], x[j]);
-        T* o = out + ((long long)m * p.tokens + t) * p.width + c;
-        if constexpr (V == 4 && sizeof(T) == 2) {
-          *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]));
-        } else {
-#pragma unroll
-          for (int j = 0; j < V; ++j) o[j] = cast_out<T>(y[j]);
-        }
+        store_run<V, T>(out + ((long long)m * p.tokens + t) * p.width, y);
       }
   };
   float prev[V], x[V];
 #pragma unroll
   for (int j = 0; j < V; ++j) prev[j] = 0.f;
-  if (t0 > 0 && first_of[0] < 0) load_row(prev, t0 - 1);
+  if (t0 > 0 && first_of[0] < 0) load_run<V, T>(prev, h + (t0 - 1ll) * p.width);
+  load_run<V, T>(x, h + (long long)t0 * p.width);
+#pragma unroll 1
   for (int i = 0; i < nt; ++i) {
     const long long t = t0 + i;
-    load_row(x, t);
+    float next[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) next[j] = 0.f;
+    if (i + 1 < nt) load_run<V, T>(next, h + (t + 1) * p.width);
     const int bl = last_of[i];
     if (bl >= 0) {
       const int n = p.q_lens ? p.q_lens[bl] : 1, ctx = p.context_lens[bl];
       const long long start = p.q_lens ? p.q_start[bl] : bl;
       const bool active = ctx >= n;
       float* st = p.state + (long long)(p.slot_ids ? p.slot_ids[bl] : bl) * p.width + c;
-      float carried[V], head[V];
-#pragma unroll
-      for (int j = 0; j < V; ++j) carried[j] = active && ctx > n ? st[j] : 0.f;
+      float head[V];
       if (n > 1) {
-        load_row(head, start);
-        emit(start, carried, head);
         emit(t, prev, x);
+        load_run<V, T>(head, h + start * p.width);
       } else {
-        emit(t, carried, x);
+#pragma unroll
+        for (int j = 0; j < V; ++j) head[j] = x[j];
       }
+#pragma unroll
+      for (int j = 0; j < V; ++j) prev[j] = active && ctx > n ? st[j] : 0.f;      // the row before the first one
+      emit(start, prev, head);
       if (active)
 #pragma unroll
         for (int j = 0; j < V; ++j) st[j] = x[j];
@@ -139,7 +160,10 @@ __global__ void __launch_bounds__(256) token_mix_kernel(const __grid_constant__ 
       emit(t, prev, x);
     }
 #pragma unroll
-    for (int j = 0; j < V; ++j) prev[j] = x[j];
+    for (int j = 0; j < V; ++j) {
+      prev[j] = x[j];
+      x[j] = next[j];
+    }
   }
 }
 
@@ -428,12 +452,6 @@ __global__ void __launch_bounds__(kScanThreads, CL <= 8 ? 4 : 1) linattn_scan_ke
 }
 
 // ------------------------------------------------------------------------------------------------ gate heads
-// the two gates in use, without the switch over all activations where a kernel is bound by issue slots
-__device__ __forceinline__ float apply_gate(float z, int kind) {
-  if (kind == ACT_SILU || kind == ACT_SIGMOID) return (kind == ACT_SILU ? z : 1.f) * __fdividef(1.f, 1.f + __expf(-z));
-  return apply_act(z, kind);
-}
-
 struct GateHeadsParams {
   const void* x;            // token t, head h: x + t * ld_token + h * ld_head
   long long ld_token, ld_head;
@@ -506,52 +524,60 @@ __global__ void __launch_bounds__(256) gate_heads_kernel(const __grid_constant__
                             apply_act(proj_load(p.g, t, h * p.width + c), p.gate_act));
 }
 
-// bf16 heads of a multiple of eight elements, at most 256: L lanes share a head, a lane holds eight consecutive elements.
-template <int L>
+// bf16 heads of a multiple of eight elements, at most 256: L lanes share a head, a lane holds eight consecutive elements of
+// two heads and loads all of them first.
+template <int L, int GATE, bool NORM>
 __global__ void __launch_bounds__(256) gate_heads8_kernel(const __grid_constant__ GateHeadsParams p) {
   using bf = __nv_bfloat16;
   const int per = 256 / L, lane = threadIdx.x & (L - 1), c = lane * 8;
   const bool on = c < p.width;
   griddep_wait();
   griddep_launch();
+  uint4 xr[2], gr[2], gr2[2];
+  int tok[2], hd[2];
 #pragma unroll
   for (int u = 0; u < 2; ++u) {
     const long long i = (blockIdx.x * 2ll + u) * per + threadIdx.x / L;
-    if (i - threadIdx.x / L >= p.rows) return;              // uniform
     const bool live = i < p.rows && on;
-    const long long t = live ? int(i) / p.heads : 0;
-    const int h = live ? int(i) % p.heads : 0;
-    float x[8], g[8];
+    tok[u] = live ? int(i) / p.heads : -1;
+    hd[u] = live ? int(i) % p.heads : 0;
+    xr[u] = gr[u] = gr2[u] = make_uint4(0u, 0u, 0u, 0u);
     if (live) {
-      const uint4 r = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(p.x) + t * p.ld_token + h * p.ld_head + c);
-      const int col = h * p.width + c;
+      const int col = hd[u] * p.width + c;
+      xr[u] = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(p.x) + tok[u] * p.ld_token + hd[u] * p.ld_head + c);
       if (p.g.bf16) {
-        const uint4 q = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(p.g.ptr) + t * p.g.ld + col);
-        const uint32_t qw[4] = {q.x, q.y, q.z, q.w};
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float2 f = unpack_bf16x2(qw[e]);
-          g[2 * e] = f.x;
-          g[2 * e + 1] = f.y;
-        }
+        gr[u] = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(p.g.ptr) + tok[u] * p.g.ld + col);
       } else {
-        const float4 lo = proj_load4(p.g, t, col), hi = proj_load4(p.g, t, col + 4);
-        g[0] = lo.x; g[1] = lo.y; g[2] = lo.z; g[3] = lo.w;
-        g[4] = hi.x; g[5] = hi.y; g[6] = hi.z; g[7] = hi.w;
+        const float4 lo = proj_load4(p.g, tok[u], col), hi = proj_load4(p.g, tok[u], col + 4);
+        gr[u] = make_uint4(__float_as_uint(lo.x), __float_as_uint(lo.y), __float_as_uint(lo.z), __float_as_uint(lo.w));
+        gr2[u] = make_uint4(__float_as_uint(hi.x), __float_as_uint(hi.y), __float_as_uint(hi.z), __float_as_uint(hi.w));
       }
-      const uint32_t rw[4] = {r.x, r.y, r.z, r.w};
+    }
+  }
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    float x[8], g[8];
+    const uint32_t rw[4] = {xr[u].x, xr[u].y, xr[u].z, xr[u].w};
+    const uint32_t gw[8] = {gr[u].x, gr[u].y, gr[u].z, gr[u].w, gr2[u].x, gr2[u].y, gr2[u].z, gr2[u].w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = unpack_bf16x2(rw[e]);
+      x[2 * e] = f.x;
+      x[2 * e + 1] = f.y;
+    }
+    if (p.g.bf16) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const float2 f = unpack_bf16x2(rw[e]);
-        x[2 * e] = f.x;
-        x[2 * e + 1] = f.y;
+        const float2 f = unpack_bf16x2(gw[e]);
+        g[2 * e] = f.x;
+        g[2 * e + 1] = f.y;
       }
     } else {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[e] = g[e] = 0.f;
+      for (int e = 0; e < 8; ++e) g[e] = __uint_as_float(gw[e]);
     }
     float inv = p.scale;
-    if (p.norm_w) {
+    if constexpr (NORM) {
       float ss = 0.f;
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
@@ -559,17 +585,38 @@ __global__ void __launch_bounds__(256) gate_heads8_kernel(const __grid_constant_
       for (int w = L / 2; w > 0; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
       inv *= 1.f / sqrtf(ss / float(p.width) + p.eps);
     }
-    if (live) {
-      const float* w = p.norm_w ? p.norm_w + (long long)h * p.norm_stride + c : nullptr;
+    if (tok[u] >= 0) {
+      if constexpr (NORM) {
+        const float* w = p.norm_w + (long long)hd[u] * p.norm_stride + c;
+        const float4 lo = *reinterpret_cast<const float4*>(w), hi = *reinterpret_cast<const float4*>(w + 4);
+        const float ww[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[e] *= inv * (w ? w[e] : 1.f) * apply_gate(g[e], p.gate_act);
-      *reinterpret_cast<uint4*>(reinterpret_cast<bf*>(p.out) + t * p.out_ld + (long long)h * p.width + c) =
+        for (int e = 0; e < 8; ++e) x[e] *= ww[e];
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        if constexpr (GATE == ACT_SILU) x[e] *= inv * g[e] * __fdividef(1.f, 1.f + __expf(-g[e]));
+        else if constexpr (GATE == ACT_SIGMOID) x[e] *= inv * __fdividef(1.f, 1.f + __expf(-g[e]));
+        else x[e] *= inv * apply_act(g[e], p.gate_act);
+      }
+      *reinterpret_cast<uint4*>(reinterpret_cast<bf*>(p.out) + tok[u] * p.out_ld + (long long)hd[u] * p.width + c) =
           make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
     }
   }
 }
 
 static bool al(const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
+
+template <int L>
+static int launch_gate_heads8(const GateHeadsParams& p, cudaStream_t s) {
+  const dim3 grid(unsigned((p.rows + 512 / L - 1) / (512 / L))), block(256);
+  if (p.norm_w) {
+    if (p.gate_act == ACT_SILU) return launch_pdl(gate_heads8_kernel<L, ACT_SILU, true>, grid, block, 0, s, p);
+    return launch_pdl(gate_heads8_kernel<L, ACT_NONE, true>, grid, block, 0, s, p);
+  }
+  if (p.gate_act == ACT_SIGMOID) return launch_pdl(gate_heads8_kernel<L, ACT_SIGMOID, false>, grid, block, 0, s, p);
+  return launch_pdl(gate_heads8_kernel<L, ACT_NONE, false>, grid, block, 0, s, p);
+}
 
 static int launch_gate_heads(const GateHeadsParams& p, int x_bf16, int out_bf16, cudaStream_t s) {
   const int xb = x_bf16 ? 8 : 16, ob = out_bf16 ? 8 : 16;
@@ -581,10 +628,11 @@ static int launch_gate_heads(const GateHeadsParams& p, int x_bf16, int out_bf16,
   if (x_bf16 && out_bf16 && p.width % 8 == 0 && p.width <= 256 && p.rows < (1ll << 30) && p.ld_token % 8 == 0 &&
       p.ld_head % 8 == 0 && p.out_ld % 8 == 0 && al(p.x, 16) && al(p.out, 16) && proj_vec4_ok(p.g) &&
       (!p.g.bf16 || (al(p.g.ptr, 16) && p.g.ld % 8 == 0))) {
-    const auto blocks = [&](int lanes) { return dim3(unsigned((p.rows + 512 / lanes - 1) / (512 / lanes))); };
-    if (p.width <= 64) return launch_pdl(gate_heads8_kernel<8>, blocks(8), block, 0, s, p);
-    if (p.width <= 128) return launch_pdl(gate_heads8_kernel<16>, blocks(16), block, 0, s, p);
-    return launch_pdl(gate_heads8_kernel<32>, blocks(32), block, 0, s, p);
+    if (!p.norm_w || (al(p.norm_w, 16) && p.norm_stride % 4 == 0)) {
+      if (p.width <= 64) return launch_gate_heads8<8>(p, s);
+      if (p.width <= 128) return launch_gate_heads8<16>(p, s);
+      return launch_gate_heads8<32>(p, s);
+    }
   }
   if (x_bf16 && out_bf16)
     return vec ? launch_pdl(gate_heads_kernel<true, bf, bf>, grid, block, 0, s, p)
@@ -604,10 +652,11 @@ __global__ void __launch_bounds__(kStepThreads) linattn_step_kernel(const __grid
   constexpr int D8 = 8 * CH;
   __shared__ __align__(16) float qs[D8], ks[D8], as[D8], us[BONUS ? D8 : 4];
   __shared__ float red[kStepThreads / 32];
-  extern __shared__ float dyn[];                    // v [vdim], o [vdim], low-rank input [rank]
+  extern __shared__ float dyn[];                    // v, o, norm weight times gate [vdim] each, low-rank input [rank]
   float* vs = dyn;
   float* os = dyn + p.vdim;
-  float* xs = os + p.vdim;
+  float* gs = os + p.vdim;
+  float* xs = gs + p.vdim;
   const int head = blockIdx.x, b = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane & 7;
   const int cl = warp * 4 + (lane >> 3);
@@ -639,7 +688,10 @@ __global__ void __launch_bounds__(kStepThreads) linattn_step_kernel(const __grid
     }
     if (b0 == 0) {
       for (int r = threadIdx.x; r < p.rank; r += kStepThreads) xs[r] = apply_act(proj_load(p.z, b, r), p.z_act);
-      for (int c = threadIdx.x; c < p.vdim; c += kStepThreads) vs[c] = proj_load(p.v, b, hv + c);
+      for (int c = threadIdx.x; c < p.vdim; c += kStepThreads) {
+        vs[c] = proj_load(p.v, b, hv + c);
+        gs[c] = p.norm_w[(long long)head * p.norm_stride + c] * apply_act(proj_load(p.g, b, hv + c), p.gate_act);
+      }
       for (int c = threadIdx.x; c < D8; c += kStepThreads) {
         const bool on = c < p.dim;
         const float q = on ? proj_load(p.q, b, hq + c) * p.q_scale : 0.f, k = on ? proj_load(p.k, b, hq + c) : 0.f;
@@ -728,9 +780,7 @@ __global__ void __launch_bounds__(kStepThreads) linattn_step_kernel(const __grid
 #pragma unroll
   for (int w = 0; w < kStepThreads / 32; ++w) tot += red[w];
   const float inv = p.out_scale / sqrtf(tot / float(p.vdim) + p.eps);
-  const float* nw = p.norm_w + (long long)head * p.norm_stride;
-  for (int c = threadIdx.x; c < p.vdim; c += kStepThreads)
-    out[c] = cast_out<OutT>(os[c] * inv * nw[c] * apply_act(proj_load(p.g, b, hv + c), p.gate_act));
+  for (int c = threadIdx.x; c < p.vdim; c += kStepThreads) out[c] = cast_out<OutT>(os[c] * inv * gs[c]);
 }
 
 template <int CL, int NC, bool BONUS, bool ASYNC, typename OutT>
@@ -769,7 +819,7 @@ static int launch_scan(const NkbLinAttn& p, bool async, cudaStream_t s) {
 template <int CH, bool BONUS>
 static int launch_step_form(const NkbLinAttn& p, cudaStream_t s) {
   const dim3 grid(p.heads, p.batch);
-  const size_t smem = size_t(2 * p.vdim + p.rank) * sizeof(float);
+  const size_t smem = size_t(3 * p.vdim + p.rank) * sizeof(float);
   return p.bf16 ? launch_pdl(linattn_step_kernel<CH, BONUS, __nv_bfloat16>, grid, dim3(kStepThreads), smem, s, p)
                 : launch_pdl(linattn_step_kernel<CH, BONUS, float>, grid, dim3(kStepThreads), smem, s, p);
 }
@@ -840,15 +890,15 @@ extern "C" int nkb_token_mix(const void* h, int bf16, const float* mu, float* st
   if (batch <= 0 || tokens <= 0) return 0;
   if (width < 1 || mixes < 1 || mixes > kMaxMixes || tokens > 65535 * kMixTokens || (q_lens == nullptr && tokens != batch)) return -2;
   TokenMixParams p{h, mu, state, slot_ids, q_start, q_lens, context_lens, out, batch, tokens, width, mixes};
-  const bool vec = width % 4 == 0 && al(h, bf16 ? 8 : 16) && al(out, bf16 ? 8 : 16);
+  const bool vec = width % (bf16 ? 8 : 4) == 0 && al(h, 16) && al(out, 16);
   const bool one = tokens <= 512;
-  const int cols = vec ? 1024 : 256;
-  const dim3 grid((width + cols - 1) / cols, one ? tokens : (tokens + kMixTokens - 1) / kMixTokens), block(256);
+  const int cols = 128 * (vec ? (bf16 ? 8 : 4) : 1);
+  const dim3 grid((width + cols - 1) / cols, one ? tokens : (tokens + kMixTokens - 1) / kMixTokens), block(128);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   using bf = __nv_bfloat16;
   if (bf16) {
-    if (vec) return one ? launch_pdl(token_mix_kernel<4, 1, bf>, grid, block, 0, s, p)
-                        : launch_pdl(token_mix_kernel<4, kMixTokens, bf>, grid, block, 0, s, p);
+    if (vec) return one ? launch_pdl(token_mix_kernel<8, 1, bf>, grid, block, 0, s, p)
+                        : launch_pdl(token_mix_kernel<8, kMixTokens, bf>, grid, block, 0, s, p);
     return one ? launch_pdl(token_mix_kernel<1, 1, bf>, grid, block, 0, s, p)
                : launch_pdl(token_mix_kernel<1, kMixTokens, bf>, grid, block, 0, s, p);
   }
