@@ -3,7 +3,8 @@
 #include "proj_src.cuh"
 
 namespace nkb {
-enum { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_RELU2 = 2, ACT_TANH = 3, ACT_SIGMOID = 4, ACT_NONE = 5, ACT_COUNT = 6 };
+enum { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_RELU2 = 2, ACT_TANH = 3, ACT_SIGMOID = 4, ACT_NONE = 5,
+       ACT_CLAMPED = 6 /* of a pair: gated_residual.cu */, ACT_COUNT = 7 };
 
 // GELU in its tanh form is written with the exponential: (1 + tanh u) / 2 = 1 / (1 + exp(-2 u))
 __device__ __forceinline__ float apply_act(float z, int kind) {

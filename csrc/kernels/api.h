@@ -6,6 +6,7 @@
 #include <cuda.h>
 #include <stdint.h>
 #include "attn_maps.h"
+#include "latent_attn.h"
 #include "linear_attn.h"
 #include "proj_src.h"
 
@@ -71,8 +72,8 @@ int nkb_gemm_bf16_grouped(const void* weights, const void* x_sorted, void* out, 
                           int gated, int gate_off, const void* bias, long long bias_group_stride, float act_limit,
                           float act_alpha, int block_n, const int* tile_list, const int* tile_count, int max_tiles,
                           const void* arrive, unsigned int arrive_target, void* stream);
-int nkb_moe_dispatch(const int* experts, int tokens, int top_k, int expert_lo, int num_local, const void* x, int hidden,
-                     void* x_sorted, int* counts, int* offsets, int* cursors, int* pair_pos, int* row_token, int bn_a,
+int nkb_moe_dispatch(const int* experts, int tokens, int top_k, int expert_lo, int num_local, const void* x, int x_f32,
+                     int hidden, const float* pair_w, void* x_sorted, int* counts, int* offsets, int* cursors, int* pair_pos, int* row_token, int bn_a,
                      int* tiles_a, int* ntiles_a, int bn_b, int* tiles_b, int* ntiles_b, void* stream);
 // expert-parallel token all-to-all (moe_a2a.cu)
 int nkb_moe_a2a_dispatch(const void* x, const int* experts, int tokens, int top_k, int hidden, int num_experts,
@@ -134,14 +135,15 @@ int nkb_argmax(const void* logits, int is_fp32, int* out_ids, float* out_vals, i
                void* stream);
 int nkb_sample(const void* logits, int is_fp32, int* out_ids, int rows, int vocab, long long ld, float temperature,
                int top_k, float top_p, unsigned long long seed, unsigned long long step, void* stream);
-int nkb_router_topk(const void* logits, int is_fp32, int splits, long long split_stride, const void* bias,
+int nkb_softcap(float* x, long long n, float cap, void* stream);
+int nkb_router_topk(const void* logits, int is_fp32, int splits, long long split_stride, long long ld, const void* bias,
                     float* weights, int* experts, int tokens, int num_experts, int top_k, int mode, int groups, int keep,
                     float scale, void* stream);
 
 int nkb_paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                           const int* context_lens, void* out, float* scratch, int batch, int q_len, int nq, int nkv,
                           int head_dim, int block_size, int num_blocks, int max_blocks_per_seq, float scale,
-                          int window, const float* sinks, int num_splits, void* stream);
+                          int window, int chunk, const float* sinks, int num_splits, void* stream);
 int nkb_paged_attn_decode_fused(const float* qkv_partials, int qkv_splits, long long qkv_split_stride,
                                 const void* qkv_bias, const int* positions, const int* slots, const float* cos_sin,
                                 const void* q_norm_w, const void* k_norm_w, float norm_eps, int max_pos, void* k_cache,
@@ -154,16 +156,16 @@ long long nkb_paged_attn_decode_scratch_floats(int batch, int q_len, int nq, int
 int nkb_flash_attn_prefill(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                            const int* q_start, const int* q_lens, const int* context_lens, void* out, int batch,
                            int total_q, int max_q_len, int nq, int nkv, int head_dim, int block_size, int num_blocks,
-                           int max_blocks_per_seq, float scale, int causal, int window, const float* sinks,
+                           int max_blocks_per_seq, float scale, int causal, int window, int chunk, const float* sinks,
                            void* stream);
 
 // layers with an fp32 residual stream (gated_residual.cu)
 int nkb_gated_residual(const float* x_in, const int* ids, const void* table, int table_bf16, int vocab, float scale,
-                       int branches, const NkbBranch* br, const float* add_row, const float* add_mat, float* x_out,
-                       int norms, const float* const* w, void* const* out, int out_bf16, int rows, int width, int groups,
-                       float eps, void* stream);
-int nkb_gated_act(const NkbProj* gate, const NkbProj* up, void* out, int out_bf16, int rows, int inter, int kind,
-                  void* stream);
+                       int branches, const NkbBranch* br, const float* add_row, const float* add_mat, float* x_out, int norms,
+                       int norm_kind, const float* const* w, const float* const* b, void* const* out, int out_bf16, int rows,
+                       int width, int groups, float eps, void* stream);
+int nkb_gated_act(const NkbProj* gate, const NkbProj* up, void* out, int out_bf16, int rows, int inter, int kind, float limit,
+                  float alpha, const int* up_rows, int up_limit, void* stream);
 // CUDA-core GEMM for 32-bit models and untileable sizes (gemm_simt.cu)
 int nkb_gemm_simt(const void* x, int x_bf16, const void* w, int w_bf16, void* out, int out_bf16, int m, int n, int k,
                   long long ldx, long long ldw, long long ldo, void* stream);
@@ -178,7 +180,8 @@ int nkb_low_rank(const NkbProj* x, int act, const void* w, int w_bf16, float* ou
 int nkb_token_mix(const void* h, int bf16, const float* mu, float* state, const int* slot_ids, const int* q_start,
                   const int* q_lens, const int* context_lens, void* out, int batch, int tokens, int width, int mixes,
                   void* stream);
-int nkb_gate_heads(const void* x, int x_bf16, long long ld_token, long long ld_head, const NkbProj* gate, int gate_act,
+int nkb_gate_heads(const void* x, int x_bf16, long long ld_token, long long ld_head, const NkbProj* gate, int head_gate,
+                   int gate_act,
                    const float* norm_w, int norm_stride, float eps, float scale, void* out, int out_bf16,
                    long long out_ld, int tokens, int heads, int width, void* stream);
 // gated linear recurrence (recurrent.cu)
@@ -197,6 +200,9 @@ int nkb_maps_append(const NkbMapsArgs* a, const NkbProj* q, const NkbProj* k, co
 int nkb_row_norm_append(const NkbMapsArgs* a, const NkbProj* q, const NkbProj* k, const NkbProj* v, const float* q_norm,
                         const float* k_norm, const int* slots, void* q_out, void* k_cache, void* v_cache, int bf16,
                         int tokens, int block_size, void* stream);
+int nkb_rope_norm_append(const NkbMapsArgs* a, const NkbProj* q, const NkbProj* k, const NkbProj* v, const float* bias,
+                         const float* cos_sin, int rot_dims, int max_pos, const int* positions, const int* slots, int norm,
+                         void* q_out, void* k_cache, void* v_cache, int bf16, int tokens, int block_size, void* stream);
 int nkb_maps_attn_simple(const NkbMapsArgs* a, const void* q, const void* k_cache, const void* v_cache,
                          const int* block_table, const int* q_start, const int* q_lens, const int* context_lens,
                          void* out, int bf16, int batch, int total_q, int block_size, int max_blocks_per_seq,
@@ -209,4 +215,17 @@ int nkb_maps_attn_prefill(const NkbMapsArgs* a, const void* q, const void* k_cac
                           const int* block_table, const int* q_start, const int* q_lens, const int* context_lens,
                           void* out, int batch, int total_q, int max_q_len, int block_size, int num_blocks,
                           int max_blocks_per_seq, void* stream);
+// latent attention (latent_attn.cu)
+int nkb_latent_append(const NkbLatentArgs* a, const NkbProj* q, const NkbProj* kv, const float* q_norm, const float* kv_norm,
+                      const float* cos_sin, int max_pos, const int* positions, const int* slots, void* q_out, void* cache,
+                      int bf16, int tokens, int block_size, void* stream);
+int nkb_latent_queries(const NkbLatentArgs* a, const NkbProj* q, const float* cos_sin, int max_pos, const int* positions,
+                       void* plain, long long plain_token, long long plain_head, int plain_pad, void* rotated,
+                       long long rot_token, long long rot_head, int rot_pad, int bf16, int tokens, void* stream);
+int nkb_latent_gather(const void* cache, const int* pages, int n_pages, int row, int rank, int rot, int rot_ld, void* c_out,
+                      void* r_out, int bf16, int block_size, void* stream);
+long long nkb_latent_scratch_floats(const NkbLatentArgs* a, int tokens, int num_splits);
+int nkb_latent_attn(const NkbLatentArgs* a, const void* q, const void* cache, const int* block_table, const int* q_start,
+                    const int* q_lens, const int* context_lens, void* out, float* scratch, int batch, int tokens,
+                    int block_size, int num_blocks, int max_blocks_per_seq, int num_splits, void* stream);
 }

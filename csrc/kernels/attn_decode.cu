@@ -27,6 +27,7 @@
 // and prefix sharing are new here.
 #include "common.cuh"
 #include "mma_frag.cuh"
+#include "attn_maps.h"
 #include "api.h"
 #include <math.h>
 
@@ -47,7 +48,7 @@ struct DecodeParams {
   unsigned int* counters;    // arrival counters of the split merge
   const float* sinks;
   int* status;
-  int batch, q_len, nq, nkv, group, max_blocks, num_splits, window;
+  int batch, q_len, nq, nkv, group, max_blocks, num_splits, window, chunk;
   float scale_log2;
   // Fused mode (qkv_partials != nullptr, q_len == 1): the kernel takes the split-K partials of the fused QKV
   // projection [splits][batch][(nq + 2 nkv) * D] instead of finished queries.  Every CTA builds its group's
@@ -206,8 +207,7 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_c
   const int ctx_paged = fused ? ctx - 1 : ctx;
 
   // ---- page range of this split
-  int first_tok = 0;
-  if (p.window > 0) first_tok = max(0, ctx - p.q_len - p.window + 1);
+  const int first_tok = nkb_first_visible(max(ctx - p.q_len, 0), p.window, p.chunk);
   const int page_lo = first_tok / kPage, page_hi = (ctx_paged + kPage - 1) / kPage;
   const int npages = max(page_hi - page_lo, 0);
   const int per_split = (npages + p.num_splits - 1) / p.num_splits;
@@ -327,8 +327,8 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_c
   const int qpos0 = ctx - p.q_len + (g < rows ? g / p.group : 0);
   const int qpos1 = ctx - p.q_len + (g + 8 < rows ? (g + 8) / p.group : 0);
   const int lim0 = fused ? qpos0 - 1 : qpos0, lim1 = fused ? qpos1 - 1 : qpos1;   // fused: the new token is not paged
-  const int low0 = p.window > 0 ? qpos0 - p.window + 1 : 0;
-  const int low1 = p.window > 0 ? qpos1 - p.window + 1 : 0;
+  const int low0 = nkb_first_visible(qpos0, p.window, p.chunk);
+  const int low1 = nkb_first_visible(qpos1, p.window, p.chunk);
 
   int stage = 0;
   uint32_t phase = 0;
@@ -588,7 +588,7 @@ extern "C" long long nkb_paged_attn_decode_scratch_floats(int batch, int q_len, 
 extern "C" int nkb_paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                                      const int* context_lens, void* out, float* scratch, int batch, int q_len, int nq,
                                      int nkv, int head_dim, int block_size, int num_blocks, int max_blocks_per_seq,
-                                     float scale, int window, const float* sinks, int num_splits, void* stream) {
+                                     float scale, int window, int chunk, const float* sinks, int num_splits, void* stream) {
   if (batch <= 0) return 0;
   if (block_size != kPage || nq % nkv != 0) return -2;
   const int group = nq / nkv;
@@ -606,7 +606,7 @@ extern "C" int nkb_paged_attn_decode(const void* q, const void* k_cache, const v
   p.sinks = sinks;
   p.status = status_word();
   p.batch = batch; p.q_len = q_len; p.nq = nq; p.nkv = nkv; p.group = group;
-  p.max_blocks = max_blocks_per_seq; p.num_splits = num_splits; p.window = window;
+  p.max_blocks = max_blocks_per_seq; p.num_splits = num_splits; p.window = window; p.chunk = chunk;
   p.scale_log2 = scale * 1.4426950408889634f;
   CUtensorMap tk, tv;
   const uint64_t dims[4] = {uint64_t(head_dim), uint64_t(kPage), uint64_t(nkv), uint64_t(num_blocks)};

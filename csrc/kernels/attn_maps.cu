@@ -2,6 +2,8 @@
 //   append   interleaved partial rotary embedding of queries and keys from the fused projection, keys and values
 //            into their slots of the paged cache
 //   row norm append   the same for one map without rotation, queries and keys normed over all heads of the token together
+//   rope norm append   the same for one map with projection biases, the rotation whose pairs are half a rotated part apart, and
+//            an RMS norm without weight over every head of queries and keys; without keys for layers that read another layer's
 //   decode   one new token per sequence, bf16: the two maps of up to eight query heads are the sixteen rows of
 //            one MMA fragment (rows 0-7 map 0, rows 8-15 map 1).  A key row holds both maps' keys side by side, so with
 //            the query of map 0 only in the first half of the contraction and that of map 1 only in the second, one
@@ -205,6 +207,107 @@ __global__ void __launch_bounds__(256) row_norm_append_kernel(const __grid_const
   }
 }
 
+// One warp per (token, head of queries / keys / values).
+struct RopeNormAppendParams {
+  NkbProj q, k, v;          // k.ptr null: queries only
+  NkbMapsArgs a;
+  const float* bias;        // [heads * dim (+ kv_heads * dim + kv_heads * vdim)] or null
+  const float* cos_sin;     // [max_pos, rot_dims]: cos of the rot_dims / 2 angles, then sin
+  const int *positions, *slots;
+  void *q_out, *k_cache, *v_cache;
+  int rot_dims, max_pos, tokens, norm;
+};
+
+template <int V>
+__device__ __forceinline__ void add_bias(float (&x)[V], const float* bias, int c) {
+  if (!bias) return;
+#pragma unroll
+  for (int j = 0; j < V; ++j) x[j] += bias[c + j];
+}
+
+template <int V, typename T>
+__global__ void __launch_bounds__(256) rope_norm_append_kernel(const __grid_constant__ RopeNormAppendParams p) {
+  const int units = p.a.heads + (p.k.ptr ? 2 * p.a.kv_heads : 0), dim = p.a.dim;
+  const long long gw = (blockIdx.x * 256ll + threadIdx.x) >> 5;
+  const int lane = threadIdx.x & 31;
+  griddep_wait();
+  griddep_launch();
+  if (gw >= (long long)p.tokens * units) return;
+  const int t = int(unsigned(gw) / unsigned(units)), u = int(unsigned(gw) % unsigned(units));
+  const bool is_q = u < p.a.heads, is_v = u >= p.a.heads + p.a.kv_heads;
+  const int slot = is_q ? 0 : p.slots[t];
+  if (slot < 0) return;
+  const long long blk = slot / kMapsPage, off = slot % kMapsPage;
+  if (is_v) {
+    const int h = u - p.a.heads - p.a.kv_heads;
+    const float* bias = p.bias ? p.bias + (p.a.heads + p.a.kv_heads) * dim + h * p.a.vdim : nullptr;
+    T* dst = reinterpret_cast<T*>(p.v_cache) + ((blk * p.a.kv_heads + h) * kMapsPage + off) * p.a.vdim_p;
+    for (int c = lane * V; c < p.a.vdim; c += 32 * V) {
+      float x[V];
+      load_v<V>(x, p.v, t, h * p.a.vdim + c);
+      add_bias<V>(x, bias, c);
+      store_v<V, T>(dst + c, x);
+    }
+    return;
+  }
+  const int h = is_q ? u : u - p.a.heads;
+  const NkbProj& src = is_q ? p.q : p.k;
+  const float* bias = p.bias ? p.bias + u * dim : nullptr;
+  T* dst = is_q ? reinterpret_cast<T*>(p.q_out) + ((long long)t * p.a.heads + h) * p.a.dim_p
+                : reinterpret_cast<T*>(p.k_cache) + ((blk * p.a.kv_heads + h) * kMapsPage + off) * p.a.dim_p;
+  const int pos = min(max(p.positions[t], 0), p.max_pos - 1), n = p.rot_dims / 2;
+  const float* cs = p.cos_sin + (long long)pos * p.rot_dims;
+  const auto load = [&](float (&x)[V], int c) {
+    load_v<V>(x, src, t, h * dim + c);
+    add_bias<V>(x, bias, c);
+  };
+  const auto finish = [&](float (&x)[V], const float (&y)[V], int c, float inv) {       // y: the other half's elements
+    if (c < 2 * n) {
+      const int i = c < n ? c : c - n;
+      const float sign = c < n ? -1.f : 1.f;
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] = x[j] * cs[i + j] + sign * y[j] * cs[n + i + j];
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[j] *= inv;
+    store_v<V, T>(dst + c, x);
+  };
+  // the rotation keeps a head's length, so the norm's sum is taken before it
+  float x[V], ss = 0.f;
+  if (dim <= 32 * V) {
+    // a lane holds its elements; those it is paired with lie n / V lanes away
+    const int c = lane * V;
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[j] = 0.f;
+    if (c < dim) load(x, c);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += x[j] * x[j];
+    const float inv = p.norm ? 1.f / sqrtf(warp_sum(ss) / float(dim) + p.a.eps) : 1.f;
+    const int from = c < n ? lane + n / V : (c < 2 * n ? lane - n / V : lane);
+    float y[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) y[j] = __shfl_sync(0xffffffffu, x[j], from);
+    if (c < p.a.dim_p) finish(x, y, c, inv);
+    const float zero[V] = {};
+    for (int z = c + 32 * V; z < p.a.dim_p; z += 32 * V) store_v<V, T>(dst + z, zero);
+    return;
+  }
+  for (int c = lane * V; c < dim; c += 32 * V) {
+    load(x, c);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += x[j] * x[j];
+  }
+  const float inv = p.norm ? 1.f / sqrtf(warp_sum(ss) / float(dim) + p.a.eps) : 1.f;
+  for (int c = lane * V; c < p.a.dim_p; c += 32 * V) {
+    float y[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[j] = y[j] = 0.f;
+    if (c < dim) load(x, c);
+    if (c < 2 * n) load(y, c < n ? c + n : c - n);
+    finish(x, y, c, inv);
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ simple
 struct MapsSimpleParams {
   NkbMapsArgs a;
@@ -215,19 +318,19 @@ struct MapsSimpleParams {
 };
 
 constexpr int kSimpleWarps = 4;
-constexpr int kSimpleCols = 8;       // value columns per lane: vdim_p <= 256
 
-template <typename T>
+// COLS: value columns per lane
+template <typename T, int MAPS, int COLS>
 __global__ void __launch_bounds__(kSimpleWarps * 32) maps_simple_kernel(const __grid_constant__ MapsSimpleParams p) {
-  extern __shared__ float sm[];      // q [2][dim_p], o [warps][2][vdim_p], m [warps][2], l [warps][2], red[warps]
+  extern __shared__ float sm[];      // q [MAPS][dim_p], o [warps][MAPS][vdim_p], m [warps][MAPS], l [warps][MAPS], red[warps]
   const int t = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int maps = p.a.maps, kw = maps * p.a.dim_p, VP = p.a.vdim_p;
+  const int kw = MAPS * p.a.dim_p, VP = p.a.vdim_p, v_ld = p.a.v_ld;
   float* q_s = sm;
-  float* o_s = q_s + 2 * p.a.dim_p;
-  float* m_s = o_s + kSimpleWarps * 2 * VP;
-  float* l_s = m_s + kSimpleWarps * 2;
-  float* red = l_s + kSimpleWarps * 2;
+  float* o_s = q_s + kw;
+  float* m_s = o_s + kSimpleWarps * MAPS * VP;
+  float* l_s = m_s + kSimpleWarps * MAPS;
+  float* red = l_s + kSimpleWarps * MAPS;
   griddep_wait();
   griddep_launch();
   int b = -1, pos = 0;
@@ -238,31 +341,35 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) maps_simple_kernel(const __
       pos = p.context_lens[i] - p.q_lens[i] + r;
     }
   }
-  T* out = reinterpret_cast<T*>(p.out) + ((long long)t * p.a.heads + h) * p.a.vdim;
+  T* out = reinterpret_cast<T*>(p.out) + t * p.a.o_token + h * p.a.o_head;
   if (b < 0 || pos < 0) {
     for (int c = threadIdx.x; c < p.a.vdim; c += blockDim.x) out[c] = cast_out<T>(0.f);
     return;
   }
-  const T* q = reinterpret_cast<const T*>(p.q) + ((long long)t * p.a.heads + h) * kw;
+  const T* q = reinterpret_cast<const T*>(p.q) + t * p.a.q_token + h * p.a.q_head;
   for (int c = threadIdx.x; c < kw; c += blockDim.x) q_s[c] = cast_in<T>(q[c]);
   __syncthreads();
   const int g = h / (p.a.heads / p.a.kv_heads);
   const int* table = p.block_table + (long long)b * p.max_blocks;
-  float o[2][kSimpleCols], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  float o[MAPS][COLS], m[MAPS], l[MAPS];
 #pragma unroll
-  for (int i = 0; i < kSimpleCols; ++i) o[0][i] = o[1][i] = 0.f;
+  for (int mp = 0; mp < MAPS; ++mp) {
+    m[mp] = -INFINITY;
+    l[mp] = 0.f;
+#pragma unroll
+    for (int i = 0; i < COLS; ++i) o[mp][i] = 0.f;
+  }
   const int pages = pos / kMapsPage + 1;
-  const int lo = p.a.window > 0 ? max(0, pos - p.a.window + 1) : 0;      // first visible position
+  const int lo = nkb_first_visible(pos, p.a.window, p.a.chunk);
   for (int pg = lo / kMapsPage + warp; pg < pages; pg += kSimpleWarps) {
     const long long blk = table[pg];
     const T* kr = reinterpret_cast<const T*>(p.k_cache) + ((blk * p.a.kv_heads + g) * kMapsPage + lane) * kw;
-    const T* vb = reinterpret_cast<const T*>(p.v_cache) + (blk * p.a.kv_heads + g) * kMapsPage * VP;
+    const T* vb = reinterpret_cast<const T*>(p.v_cache) + (blk * p.a.kv_heads + g) * kMapsPage * v_ld;
     const bool vis = pg * kMapsPage + lane <= pos && pg * kMapsPage + lane >= lo;
     const int nvis = min(kMapsPage, pos + 1 - pg * kMapsPage);
-    float pr[2] = {0.f, 0.f};
+    float pr[MAPS];
 #pragma unroll
-    for (int mp = 0; mp < 2; ++mp) {
-      if (mp >= maps) break;
+    for (int mp = 0; mp < MAPS; ++mp) {
       float s = 0.f;
       if (vis) {
         for (int c = 0; c < p.a.dim; ++c) s = fmaf(q_s[mp * p.a.dim_p + c], cast_in<T>(kr[mp * p.a.dim_p + c]), s);
@@ -271,59 +378,64 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) maps_simple_kernel(const __
       } else {
         s = -INFINITY;
       }
-      const float mn = fmaxf(m[mp], warp_max(s));
+      const float mn = fmaxf(m[mp], warp_max(s));            // finite: every page read holds a visible token
       const float alpha = expf(m[mp] - mn);
       pr[mp] = expf(s - mn);
       l[mp] = l[mp] * alpha + warp_sum(pr[mp]);
       m[mp] = mn;
 #pragma unroll
-      for (int i = 0; i < kSimpleCols; ++i) o[mp][i] *= alpha;
+      for (int i = 0; i < COLS; ++i) o[mp][i] *= alpha;
     }
     for (int j = 0; j < nvis; ++j) {
-      const float p0 = __shfl_sync(0xffffffffu, pr[0], j), p1 = __shfl_sync(0xffffffffu, pr[1], j);
+      float pj[MAPS];
 #pragma unroll
-      for (int i = 0; i < kSimpleCols; ++i) {
+      for (int mp = 0; mp < MAPS; ++mp) pj[mp] = __shfl_sync(0xffffffffu, pr[mp], j);
+#pragma unroll
+      for (int i = 0; i < COLS; ++i) {
         const int c = lane + 32 * i;
         if (c < VP) {
-          const float v = cast_in<T>(vb[j * VP + c]);
-          o[0][i] = fmaf(p0, v, o[0][i]);
-          o[1][i] = fmaf(p1, v, o[1][i]);
+          const float v = cast_in<T>(vb[j * v_ld + c]);
+#pragma unroll
+          for (int mp = 0; mp < MAPS; ++mp) o[mp][i] = fmaf(pj[mp], v, o[mp][i]);
         }
       }
     }
   }
 #pragma unroll
-  for (int mp = 0; mp < 2; ++mp) {
+  for (int mp = 0; mp < MAPS; ++mp) {
 #pragma unroll
-    for (int i = 0; i < kSimpleCols; ++i)
-      if (lane + 32 * i < VP) o_s[(warp * 2 + mp) * VP + lane + 32 * i] = o[mp][i];
+    for (int i = 0; i < COLS; ++i)
+      if (lane + 32 * i < VP) o_s[(warp * MAPS + mp) * VP + lane + 32 * i] = o[mp][i];
     if (lane == 0) {
-      m_s[warp * 2 + mp] = m[mp];
-      l_s[warp * 2 + mp] = l[mp];
+      m_s[warp * MAPS + mp] = m[mp];
+      l_s[warp * MAPS + mp] = l[mp];
     }
   }
   __syncthreads();
   float ss = 0.f;
   for (int c = threadIdx.x; c < p.a.vdim; c += blockDim.x) {
-    float a[2] = {0.f, 0.f};
+    float a[MAPS];
 #pragma unroll
-    for (int mp = 0; mp < 2; ++mp) {
-      if (mp >= maps) break;
+    for (int mp = 0; mp < MAPS; ++mp) {
       float mx = -INFINITY, acc = 0.f, den = 0.f;
-      for (int w = 0; w < kSimpleWarps; ++w) mx = fmaxf(mx, m_s[w * 2 + mp]);
+      for (int w = 0; w < kSimpleWarps; ++w) mx = fmaxf(mx, m_s[w * MAPS + mp]);
+      if (p.a.sinks) {
+        mx = fmaxf(mx, p.a.sinks[h]);
+        den = expf(p.a.sinks[h] - mx);
+      }
       for (int w = 0; w < kSimpleWarps; ++w) {
-        const float mw = m_s[w * 2 + mp];
+        const float mw = m_s[w * MAPS + mp];
         const float f = mw == -INFINITY ? 0.f : expf(mw - mx);
-        acc += f * o_s[(w * 2 + mp) * VP + c];
-        den += f * l_s[w * 2 + mp];
+        acc += f * o_s[(w * MAPS + mp) * VP + c];
+        den += f * l_s[w * MAPS + mp];
       }
       a[mp] = acc / den;
     }
-    const float r = maps == 2 ? a[0] - p.a.lambda * a[1] : a[0];
+    const float r = MAPS == 2 ? a[0] - p.a.lambda * a[MAPS - 1] : a[0];
     ss += r * r;
     o_s[c] = r;                      // warp 0's map 0 slot of this column: read above by this thread only
   }
-  if (maps == 2) {
+  if (MAPS == 2) {
     ss = warp_sum(ss);
     if (lane == 0) red[warp] = ss;
     __syncthreads();
@@ -692,22 +804,63 @@ extern "C" int nkb_row_norm_append(const NkbMapsArgs* a, const NkbProj* q, const
               : launch_pdl(row_norm_append_kernel<1, float>, grid, block, smem, s, p);
 }
 
+extern "C" int nkb_rope_norm_append(const NkbMapsArgs* a, const NkbProj* q, const NkbProj* k, const NkbProj* v,
+                                    const float* bias, const float* cos_sin, int rot_dims, int max_pos, const int* positions,
+                                    const int* slots, int norm, void* q_out, void* k_cache, void* v_cache, int bf16, int tokens,
+                                    int block_size, void* stream) {
+  if (tokens <= 0) return 0;
+  if (!maps_ok(*a) || a->maps != 1 || block_size != kMapsPage || rot_dims < 0 || rot_dims > a->dim || (rot_dims & 1) ||
+      max_pos < 1 || (k->ptr && !v->ptr))
+    return -2;
+  RopeNormAppendParams p{};
+  p.q = *q; p.k = *k; p.v = *v; p.a = *a;
+  p.bias = bias; p.cos_sin = cos_sin; p.positions = positions; p.slots = slots;
+  p.q_out = q_out; p.k_cache = k_cache; p.v_cache = v_cache;
+  p.rot_dims = rot_dims; p.max_pos = max_pos; p.tokens = tokens; p.norm = norm;
+  const auto al16 = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
+  const bool vec = ((a->dim | a->dim_p | a->vdim | a->vdim_p) & 3) == 0 && (rot_dims & 7) == 0 && proj_vec4_ok(*q) &&
+                   proj_vec4_ok(*k) && proj_vec4_ok(*v) && al16(q_out) && al16(k_cache) && al16(v_cache);
+  const long long warps = (long long)tokens * (a->heads + (k->ptr ? 2 * a->kv_heads : 0));
+  if (warps > 0x7fffffffll) return -2;
+  const dim3 grid(unsigned((warps + 7) / 8)), block(256);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  using bf = __nv_bfloat16;
+  if (vec)
+    return bf16 ? launch_pdl(rope_norm_append_kernel<4, bf>, grid, block, 0, s, p)
+                : launch_pdl(rope_norm_append_kernel<4, float>, grid, block, 0, s, p);
+  return bf16 ? launch_pdl(rope_norm_append_kernel<1, bf>, grid, block, 0, s, p)
+              : launch_pdl(rope_norm_append_kernel<1, float>, grid, block, 0, s, p);
+}
+
+template <typename T>
+static int launch_simple(const MapsSimpleParams& p, dim3 grid, size_t smem, cudaStream_t s) {
+  const dim3 block(kSimpleWarps * 32);
+  if (p.a.maps == 2)
+    return p.a.vdim_p <= 256 ? launch_pdl(maps_simple_kernel<T, 2, 8>, grid, block, smem, s, p) : -2;
+  if (p.a.vdim_p <= 256) return launch_pdl(maps_simple_kernel<T, 1, 8>, grid, block, smem, s, p);
+  if (p.a.vdim_p <= 1024) return launch_pdl(maps_simple_kernel<T, 1, 32>, grid, block, smem, s, p);
+  return -2;
+}
+
 extern "C" int nkb_maps_attn_simple(const NkbMapsArgs* a, const void* q, const void* k_cache, const void* v_cache,
                                     const int* block_table, const int* q_start, const int* q_lens,
                                     const int* context_lens, void* out, int bf16, int batch, int total_q, int block_size,
                                     int max_blocks_per_seq, void* stream) {
   if (batch <= 0 || total_q <= 0) return 0;
-  if (!maps_ok(*a) || block_size != kMapsPage || a->vdim_p > 32 * kSimpleCols || a->heads > 65535) return -2;
+  if (!maps_ok(*a) || block_size != kMapsPage || a->heads > 65535 || (a->sinks && a->maps != 1)) return -2;
   MapsSimpleParams p{};
   p.a = *a; p.q = q; p.k_cache = k_cache; p.v_cache = v_cache;
   p.block_table = block_table; p.q_start = q_start; p.q_lens = q_lens; p.context_lens = context_lens;
   p.out = out; p.batch = batch; p.max_blocks = max_blocks_per_seq;
-  const size_t smem = size_t(2 * a->dim_p + kSimpleWarps * (2 * a->vdim_p + 5)) * sizeof(float);
+  const int kw = a->maps * a->dim_p;
+  if (!p.a.q_token) { p.a.q_token = (long long)a->heads * kw; p.a.q_head = kw; }
+  if (!p.a.o_token) { p.a.o_token = (long long)a->heads * a->vdim; p.a.o_head = a->vdim; }
+  if (!p.a.v_ld) p.a.v_ld = a->vdim_p;
+  const size_t smem = size_t(kw + kSimpleWarps * (a->maps * a->vdim_p + 5)) * sizeof(float);
   if (smem > 48 * 1024) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const dim3 grid(total_q, a->heads);
-  return bf16 ? launch_pdl(maps_simple_kernel<__nv_bfloat16>, grid, dim3(kSimpleWarps * 32), smem, s, p)
-              : launch_pdl(maps_simple_kernel<float>, grid, dim3(kSimpleWarps * 32), smem, s, p);
+  return bf16 ? launch_simple<__nv_bfloat16>(p, grid, smem, s) : launch_simple<float>(p, grid, smem, s);
 }
 
 extern "C" long long nkb_maps_decode_scratch_floats(const NkbMapsArgs* a, int batch, int num_splits) {
@@ -724,7 +877,7 @@ extern "C" int nkb_maps_attn_decode(const NkbMapsArgs* a, const void* q, const v
                                     void* stream) {
   if (batch <= 0) return 0;
   if (!maps_ok(*a) || block_size != kMapsPage || batch > 65535) return -2;
-  if (a->maps != 2 || a->window > 0 || (a->dim_p != 32 && a->dim_p != 64) || (a->vdim_p != 64 && a->vdim_p != 128)) return -5;
+  if (a->maps != 2 || a->window > 0 || a->chunk > 0 || a->sinks || (a->dim_p != 32 && a->dim_p != 64) || (a->vdim_p != 64 && a->vdim_p != 128)) return -5;
   if (!status_word() && nkb_init() != 0) return -1;
   MapsDecodeParams p{};
   p.a = *a;

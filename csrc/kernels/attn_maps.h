@@ -4,11 +4,27 @@
 // maps the head's result is
 //     o = a_0 - lambda * a_1;     o <- out_scale * o / sqrt(mean(o^2) + eps)
 // and with one map it is a_0.  softcap > 0 replaces a score s by softcap * tanh(s / softcap); window > 0 limits a query to
-// itself and the window - 1 tokens before it.
+// itself and the window - 1 tokens before it, chunk > 0 to the tokens of its own chunk of that many positions; sinks holds
+// per head (one map) the logarithm of an addend of the softmax's denominator.
 #pragma once
 
 struct NkbMapsArgs {
   int maps, heads, kv_heads, dim, dim_p, vdim, vdim_p;
   float scale, softcap, lambda, out_scale, eps;
-  int window;
+  int window, chunk;
+  const float* sinks;                    // [heads] or null
+  // elements between tokens / heads of queries and results, 0: one token's heads side by side
+  long long q_token, q_head, o_token, o_head;
+  int v_ld;                              // elements between the values of two tokens, 0: vdim_p (values inside wider rows)
 };
+
+// First position a query at `pos` sees.
+static inline
+#ifdef __CUDACC__
+__host__ __device__
+#endif
+int nkb_first_visible(int pos, int window, int chunk) {
+  int lo = window > 0 && pos >= window ? pos - window + 1 : 0;
+  if (chunk > 0 && pos - pos % chunk > lo) lo = pos - pos % chunk;
+  return lo;
+}

@@ -43,6 +43,7 @@
 // examples/models/gpt_oss/kernels/attention.py:116-148, non-causal-free prefill
 // of examples/models/qwen3_embedding/kernels/attention.py.
 #include "common.cuh"
+#include "attn_maps.h"
 #include "api.h"
 #include <math.h>
 
@@ -64,7 +65,7 @@ struct PrefillParams {
   __nv_bfloat16* out;
   const float* sinks;
   int* status;
-  int nq, nkv, max_blocks, causal, window;
+  int nq, nkv, max_blocks, causal, window, chunk;
   float scale_log2;
 };
 
@@ -118,7 +119,7 @@ __device__ __forceinline__ TileRange tile_range(const PrefillParams& p, int row0
   r.pos0 = ctx - q_len + row0;                       // kv position of the tile's first query
   r.hi = (ctx + kKVTile - 1) / kKVTile;
   if (p.causal) r.hi = min(r.hi, (r.pos0 + r.rows - 1) / kKVTile + 1);
-  if (p.window > 0) r.lo = max(0, r.pos0 - p.window + 1) / kKVTile;
+  r.lo = nkb_first_visible(r.pos0, p.window, p.chunk) / kKVTile;
   if (r.hi < r.lo) r.hi = r.lo;
   return r;
 }
@@ -332,7 +333,7 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
     float m = -INFINITY, l = 0.f;
     int hi_pos = ctx - 1;
     if (p.causal) hi_pos = min(hi_pos, q_pos);
-    const int lo_pos = p.window > 0 ? q_pos - p.window + 1 : 0;
+    const int lo_pos = nkb_first_visible(q_pos, p.window, p.chunk);
     bool alive = true;
 
     for (int it = 0; it < n_tiles; ++it) {
@@ -528,7 +529,7 @@ extern "C" int nkb_flash_attn_prefill(const void* q, const void* k_cache, const 
                                       const int* q_start, const int* q_lens, const int* context_lens, void* out,
                                       int batch, int total_q, int max_q_len, int nq, int nkv, int head_dim,
                                       int block_size, int num_blocks, int max_blocks_per_seq, float scale, int causal,
-                                      int window, const float* sinks, void* stream) {
+                                      int window, int chunk, const float* sinks, void* stream) {
   if (batch <= 0 || total_q <= 0) return 0;
   if (block_size != kPfPage || nq % nkv != 0) return -2;
   if (!status_word() && nkb_init() != 0) return -1;
@@ -540,7 +541,7 @@ extern "C" int nkb_flash_attn_prefill(const void* q, const void* k_cache, const 
   p.out = reinterpret_cast<__nv_bfloat16*>(out);
   p.sinks = sinks;
   p.status = status_word();
-  p.nq = nq; p.nkv = nkv; p.max_blocks = max_blocks_per_seq; p.causal = causal; p.window = window;
+  p.nq = nq; p.nkv = nkv; p.max_blocks = max_blocks_per_seq; p.causal = causal; p.window = window; p.chunk = chunk;
   p.scale_log2 = scale * 1.4426950408889634f;
   CUtensorMap tq, tk, tv;
   {

@@ -132,5 +132,7 @@ extern "C" int nkb_gemm_simt_grouped(const void* x, int x_bf16, const void* w, i
     return launch_simt_grouped<float, float, float>(x, w, out, offsets, row_token, groups, max_rows, n, k, ldx, ldo, s);
   if (x_bf16 && w_bf16 && !out_bf16)
     return launch_simt_grouped<bf, bf, float>(x, w, out, offsets, row_token, groups, max_rows, n, k, ldx, ldo, s);
+  if (x_bf16 && w_bf16 && out_bf16)
+    return launch_simt_grouped<bf, bf, bf>(x, w, out, offsets, row_token, groups, max_rows, n, k, ldx, ldo, s);
   return -2;
 }

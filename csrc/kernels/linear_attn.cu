@@ -455,11 +455,11 @@ __global__ void __launch_bounds__(kScanThreads, CL <= 8 ? 4 : 1) linattn_scan_ke
 struct GateHeadsParams {
   const void* x;            // token t, head h: x + t * ld_token + h * ld_head
   long long ld_token, ld_head;
-  NkbProj g;                // [tokens, heads * width]
+  NkbProj g;                // [tokens, heads * width], or [tokens, heads]: one gate per head
   const float* norm_w;      // nullptr: the head is not normed; otherwise element h * norm_stride + j
   void* out;
   long long out_ld, rows;   // rows = tokens * heads
-  int gate_act, norm_stride, heads, width;
+  int gate_act, norm_stride, heads, width, head_gate;
   float eps, scale;
 };
 
@@ -493,7 +493,8 @@ __global__ void __launch_bounds__(256) gate_heads_kernel(const __grid_constant__
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f), gt = v, ww = make_float4(1.f, 1.f, 1.f, 1.f);
     if (on) {
       v = load4_as<XT>(x + c);
-      gt = proj_load4(p.g, t, h * p.width + c);
+      if (p.head_gate) gt.x = gt.y = gt.z = gt.w = proj_load(p.g, t, h);
+      else gt = proj_load4(p.g, t, h * p.width + c);
       if (w) ww = *reinterpret_cast<const float4*>(w + c);
     }
     float inv = p.scale;
@@ -521,12 +522,12 @@ __global__ void __launch_bounds__(256) gate_heads_kernel(const __grid_constant__
   }
   for (int c = lane; c < p.width; c += 32)
     out[c] = cast_out<OutT>(cast_in<XT>(x[c]) * inv * (w ? w[c] : 1.f) *
-                            apply_act(proj_load(p.g, t, h * p.width + c), p.gate_act));
+                            apply_act(proj_load(p.g, t, p.head_gate ? h : h * p.width + c), p.gate_act));
 }
 
 // bf16 heads of a multiple of eight elements, at most 256: L lanes share a head, a lane holds eight consecutive elements of
 // two heads and loads all of them first.
-template <int L, int GATE, bool NORM>
+template <int L, int GATE, bool NORM, bool HEAD = false>
 __global__ void __launch_bounds__(256) gate_heads8_kernel(const __grid_constant__ GateHeadsParams p) {
   using bf = __nv_bfloat16;
   const int per = 256 / L, lane = threadIdx.x & (L - 1), c = lane * 8;
@@ -534,6 +535,7 @@ __global__ void __launch_bounds__(256) gate_heads8_kernel(const __grid_constant_
   griddep_wait();
   griddep_launch();
   uint4 xr[2], gr[2], gr2[2];
+  float hg[2];
   int tok[2], hd[2];
 #pragma unroll
   for (int u = 0; u < 2; ++u) {
@@ -542,10 +544,13 @@ __global__ void __launch_bounds__(256) gate_heads8_kernel(const __grid_constant_
     tok[u] = live ? int(i) / p.heads : -1;
     hd[u] = live ? int(i) % p.heads : 0;
     xr[u] = gr[u] = gr2[u] = make_uint4(0u, 0u, 0u, 0u);
+    hg[u] = 0.f;
     if (live) {
       const int col = hd[u] * p.width + c;
       xr[u] = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(p.x) + tok[u] * p.ld_token + hd[u] * p.ld_head + c);
-      if (p.g.bf16) {
+      if constexpr (HEAD) {
+        hg[u] = proj_load(p.g, tok[u], hd[u]);
+      } else if (p.g.bf16) {
         gr[u] = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(p.g.ptr) + tok[u] * p.g.ld + col);
       } else {
         const float4 lo = proj_load4(p.g, tok[u], col), hi = proj_load4(p.g, tok[u], col + 4);
@@ -565,7 +570,10 @@ __global__ void __launch_bounds__(256) gate_heads8_kernel(const __grid_constant_
       x[2 * e] = f.x;
       x[2 * e + 1] = f.y;
     }
-    if (p.g.bf16) {
+    if constexpr (HEAD) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) g[e] = hg[u];
+    } else if (p.g.bf16) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const float2 f = unpack_bf16x2(gw[e]);
@@ -610,6 +618,11 @@ static bool al(const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p
 template <int L>
 static int launch_gate_heads8(const GateHeadsParams& p, cudaStream_t s) {
   const dim3 grid(unsigned((p.rows + 512 / L - 1) / (512 / L))), block(256);
+  if (p.head_gate) {
+    if (p.norm_w) return launch_pdl(gate_heads8_kernel<L, ACT_NONE, true, true>, grid, block, 0, s, p);
+    if (p.gate_act == ACT_SIGMOID) return launch_pdl(gate_heads8_kernel<L, ACT_SIGMOID, false, true>, grid, block, 0, s, p);
+    return launch_pdl(gate_heads8_kernel<L, ACT_NONE, false, true>, grid, block, 0, s, p);
+  }
   if (p.norm_w) {
     if (p.gate_act == ACT_SILU) return launch_pdl(gate_heads8_kernel<L, ACT_SILU, true>, grid, block, 0, s, p);
     return launch_pdl(gate_heads8_kernel<L, ACT_NONE, true>, grid, block, 0, s, p);
@@ -621,13 +634,13 @@ static int launch_gate_heads8(const GateHeadsParams& p, cudaStream_t s) {
 static int launch_gate_heads(const GateHeadsParams& p, int x_bf16, int out_bf16, cudaStream_t s) {
   const int xb = x_bf16 ? 8 : 16, ob = out_bf16 ? 8 : 16;
   const bool vec = p.width % 4 == 0 && p.width <= 128 && p.ld_token % 4 == 0 && p.ld_head % 4 == 0 && p.out_ld % 4 == 0 &&
-                   al(p.x, xb) && al(p.out, ob) && proj_vec4_ok(p.g) &&
+                   al(p.x, xb) && al(p.out, ob) && (p.head_gate || proj_vec4_ok(p.g)) &&
                    (!p.norm_w || (al(p.norm_w, 16) && p.norm_stride % 4 == 0));
   const dim3 grid(unsigned((p.rows + 7) / 8)), block(256);
   using bf = __nv_bfloat16;
   if (x_bf16 && out_bf16 && p.width % 8 == 0 && p.width <= 256 && p.rows < (1ll << 30) && p.ld_token % 8 == 0 &&
-      p.ld_head % 8 == 0 && p.out_ld % 8 == 0 && al(p.x, 16) && al(p.out, 16) && proj_vec4_ok(p.g) &&
-      (!p.g.bf16 || (al(p.g.ptr, 16) && p.g.ld % 8 == 0))) {
+      p.ld_head % 8 == 0 && p.out_ld % 8 == 0 && al(p.x, 16) && al(p.out, 16) && (p.head_gate || proj_vec4_ok(p.g)) &&
+      (p.head_gate || !p.g.bf16 || (al(p.g.ptr, 16) && p.g.ld % 8 == 0))) {
     if (!p.norm_w || (al(p.norm_w, 16) && p.norm_stride % 4 == 0)) {
       if (p.width <= 64) return launch_gate_heads8<8>(p, s);
       if (p.width <= 128) return launch_gate_heads8<16>(p, s);
@@ -909,11 +922,11 @@ extern "C" int nkb_token_mix(const void* h, int bf16, const float* mu, float* st
 }
 
 extern "C" int nkb_gate_heads(const void* x, int x_bf16, long long ld_token, long long ld_head, const NkbProj* gate,
-                              int gate_act, const float* norm_w, int norm_stride, float eps, float scale, void* out,
+                              int head_gate, int gate_act, const float* norm_w, int norm_stride, float eps, float scale, void* out,
                               int out_bf16, long long out_ld, int tokens, int heads, int width, void* stream) {
   if (tokens <= 0) return 0;
   if (heads < 1 || width < 1 || gate_act < 0 || gate_act >= ACT_COUNT) return -2;
   GateHeadsParams p{x, ld_token, ld_head, *gate, norm_w, out, out_ld, (long long)tokens * heads, gate_act, norm_stride,
-                    heads, width, eps, scale};
+                    heads, width, head_gate, eps, scale};
   return launch_gate_heads(p, x_bf16, out_bf16, reinterpret_cast<cudaStream_t>(stream));
 }

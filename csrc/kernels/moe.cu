@@ -128,25 +128,51 @@ __global__ void moe_plan_small_kernel(const int* __restrict__ experts, int pairs
   }
 }
 
+// The token row of a pair at its sorted position, multiplied by the pair's weight when there are weights (experts whose
+// weight scales the input).
+template <typename T>
+__device__ __forceinline__ void moe_copy_row(const T* __restrict__ x, int hidden, int token, int pos, const float* pair_w,
+                                             int pair, T* __restrict__ x_sorted) {
+  const float w = pair_w ? pair_w[pair] : 1.f;
+  const T* src = x + (long long)token * hidden;
+  T* dst = x_sorted + (long long)pos * hidden;
+  if constexpr (sizeof(T) == 4) {
+    for (int v = threadIdx.x; v < hidden; v += blockDim.x) dst[v] = pair_w ? w * src[v] : src[v];
+  } else if (hidden & 7) {
+    for (int v = threadIdx.x; v < hidden; v += blockDim.x) dst[v] = __float2bfloat16(w * __bfloat162float(src[v]));
+  } else {
+    for (int v = threadIdx.x; v < (hidden >> 3); v += blockDim.x) {
+      uint4 r = reinterpret_cast<const uint4*>(src)[v];
+      if (pair_w) {
+        uint32_t* rw = reinterpret_cast<uint32_t*>(&r);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 f = unpack_bf16x2(rw[e]);
+          rw[e] = pack_bf16x2(w * f.x, w * f.y);
+        }
+      }
+      reinterpret_cast<uint4*>(dst)[v] = r;
+    }
+  }
+}
+
 // one block per pair: copy the token row to its sorted position
-__global__ void moe_gather_kernel(const int* __restrict__ pair_pos, int top_k, const __nv_bfloat16* __restrict__ x,
-                                  int hidden, __nv_bfloat16* __restrict__ x_sorted) {
+template <typename T>
+__global__ void moe_gather_kernel(const int* __restrict__ pair_pos, int top_k, const T* __restrict__ x, int hidden,
+                                  const float* __restrict__ pair_w, T* __restrict__ x_sorted) {
   griddep_wait();
   griddep_launch();
   const int pair = blockIdx.x;
   const int pos = pair_pos[pair];
-  if (pos < 0) return;
-  const int token = pair / top_k;
-  const uint4* src = reinterpret_cast<const uint4*>(x + (long long)token * hidden);
-  uint4* dst = reinterpret_cast<uint4*>(x_sorted + (long long)pos * hidden);
-  for (int v = threadIdx.x; v < (hidden >> 3); v += blockDim.x) dst[v] = src[v];
+  if (pos >= 0) moe_copy_row<T>(x, hidden, pair / top_k, pos, pair_w, pair, x_sorted);
 }
 
 // one block per pair: claim a slot in its expert's segment and copy the token row there
+template <typename T>
 __global__ void moe_scatter_kernel(const int* __restrict__ experts, int pairs, int top_k, int expert_lo,
                                    int num_local, const int* __restrict__ offsets, int* __restrict__ cursors,
-                                   const __nv_bfloat16* __restrict__ x, int hidden, __nv_bfloat16* __restrict__ x_sorted,
-                                   int* __restrict__ pair_pos, int* __restrict__ row_token) {
+                                   const T* __restrict__ x, int hidden, const float* __restrict__ pair_w,
+                                   T* __restrict__ x_sorted, int* __restrict__ pair_pos, int* __restrict__ row_token) {
   griddep_wait();
   griddep_launch();
   __shared__ int s_pos;
@@ -161,12 +187,7 @@ __global__ void moe_scatter_kernel(const int* __restrict__ experts, int pairs, i
   }
   if (!x) return;
   __syncthreads();
-  const int pos = s_pos;
-  if (pos < 0) return;
-  const int token = pair / top_k;
-  const uint4* src = reinterpret_cast<const uint4*>(x + (long long)token * hidden);
-  uint4* dst = reinterpret_cast<uint4*>(x_sorted + (long long)pos * hidden);
-  for (int v = threadIdx.x; v < (hidden >> 3); v += blockDim.x) dst[v] = src[v];
+  if (s_pos >= 0) moe_copy_row<T>(x, hidden, pair / top_k, s_pos, pair_w, pair, x_sorted);
 }
 
 // out[t] = sum_j w[t, j] * y_sorted[pair_pos[t * k + j]]   over the pairs handled locally
@@ -205,21 +226,25 @@ using namespace nkb;
 // experts [tokens * top_k] int32 (global expert ids).  Workspace (device, int32): counts[num_local],
 // offsets[num_local + 1], cursors[num_local], pair_pos[tokens * top_k].  x_sorted must hold
 // tokens * top_k rows.  After the call offsets / pair_pos / x_sorted are valid on the stream.  x == nullptr: the rows are
-// not gathered (any width); row_token [tokens * top_k], when given, names the token of every sorted row instead.
+// not gathered (any width); row_token [tokens * top_k], when given, names the token of every sorted row instead.  pair_w
+// [tokens * top_k]: the gathered rows are multiplied by it.  x_f32: x and x_sorted are fp32.
 extern "C" int nkb_moe_dispatch(const int* experts, int tokens, int top_k, int expert_lo, int num_local, const void* x,
-                                int hidden, void* x_sorted, int* counts, int* offsets, int* cursors, int* pair_pos,
+                                int x_f32, int hidden, const float* pair_w, void* x_sorted, int* counts, int* offsets, int* cursors, int* pair_pos,
                                 int* row_token, int bn_a, int* tiles_a, int* ntiles_a, int bn_b, int* tiles_b, int* ntiles_b,
                                 void* stream) {
   if (tokens <= 0) return 0;
-  if (num_local > 1024 || (x && (hidden & 7)) || (!x && !row_token) || bn_a <= 0 || bn_b <= 0) return -2;
+  if (num_local > 1024 || (!x && !row_token) || bn_a <= 0 || bn_b <= 0) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const int pairs = tokens * top_k;
   if (pairs <= 8192) {
     int rc = launch_pdl(moe_plan_small_kernel, dim3(1), dim3(1024), 0, s, experts, pairs, expert_lo, num_local, offsets,
                         pair_pos, row_token, top_k, bn_a, tiles_a, ntiles_a, bn_b, tiles_b, ntiles_b);
     if (rc || !x) return rc;
-    return launch_pdl(moe_gather_kernel, dim3(pairs), dim3(128), 0, s, (const int*)pair_pos, top_k,
-                      (const __nv_bfloat16*)x, hidden, (__nv_bfloat16*)x_sorted);
+    if (x_f32)
+      return launch_pdl(moe_gather_kernel<float>, dim3(pairs), dim3(128), 0, s, (const int*)pair_pos, top_k,
+                        (const float*)x, hidden, pair_w, (float*)x_sorted);
+    return launch_pdl(moe_gather_kernel<__nv_bfloat16>, dim3(pairs), dim3(128), 0, s, (const int*)pair_pos, top_k,
+                      (const __nv_bfloat16*)x, hidden, pair_w, (__nv_bfloat16*)x_sorted);
   }
   cudaError_t e = cudaMemsetAsync(counts, 0, sizeof(int) * num_local, s);
   if (e != cudaSuccess) return int(e);
@@ -231,8 +256,12 @@ extern "C" int nkb_moe_dispatch(const int* experts, int tokens, int top_k, int e
   rc = launch_pdl(moe_tiles_kernel, dim3(1), dim3(1024), 0, s, (const int*)offsets, num_local, bn_a, tiles_a, ntiles_a,
                   bn_b, tiles_b, ntiles_b);
   if (rc) return rc;
-  return launch_pdl(moe_scatter_kernel, dim3(pairs), dim3(128), 0, s, experts, pairs, top_k, expert_lo, num_local,
-                    (const int*)offsets, cursors, (const __nv_bfloat16*)x, hidden, (__nv_bfloat16*)x_sorted, pair_pos, row_token);
+  if (x_f32)
+    return launch_pdl(moe_scatter_kernel<float>, dim3(pairs), dim3(128), 0, s, experts, pairs, top_k, expert_lo, num_local,
+                      (const int*)offsets, cursors, (const float*)x, hidden, pair_w, (float*)x_sorted, pair_pos, row_token);
+  return launch_pdl(moe_scatter_kernel<__nv_bfloat16>, dim3(pairs), dim3(128), 0, s, experts, pairs, top_k, expert_lo, num_local,
+                    (const int*)offsets, cursors, (const __nv_bfloat16*)x, hidden, pair_w, (__nv_bfloat16*)x_sorted, pair_pos,
+                    row_token);
 }
 
 extern "C" int nkb_moe_combine(const void* y_sorted, const int* pair_pos, const float* weights, int tokens, int top_k,

@@ -12,13 +12,15 @@ struct NkbProj {
   int bf16;                 // 1 = bf16 values, 0 = fp32
 };
 
-// One addend of a residual update: scale * y, with a gate sigmoid(g + gbias) on it when g.ptr is set, or (pair_pos set) the
-// weighted sum of a token's top_k rows of y, pair_w[t, j] * y[pair_pos[t, j]] (routed experts).
+// One addend of a residual update: scale * y, with a gate sigmoid(g + gbias) on it when g.ptr is set (token_gate: one g per
+// token, no bias), or (pair_pos set) the sum of a token's top_k rows of y, pair_w[t, j] * y[pair_pos[t, j]] (routed experts;
+// pair_w null: weights of one), or (norm_w set) norm_w * y / sqrt(mean(y^2) + eps).
 struct NkbBranch {
   NkbProj y, g;
   const float* gbias;
   const int* pair_pos;
   const float* pair_w;
-  int top_k;
+  const float* norm_w;
+  int top_k, token_gate;
   float scale;
 };

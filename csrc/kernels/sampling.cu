@@ -220,18 +220,38 @@ __global__ void __launch_bounds__(1024) sample_kernel(const void* __restrict__ l
   }
 }
 
+// x <- cap * tanh(x / cap), in place (logits)
+__global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, long long n, float cap) {
+  griddep_wait();
+  griddep_launch();
+  const long long stride = (long long)gridDim.x * blockDim.x, i0 = blockIdx.x * (long long)blockDim.x + threadIdx.x;
+  if ((n & 3) == 0) {
+    for (long long i = i0; i < n / 4; i += stride) {
+      float4 v = reinterpret_cast<float4*>(x)[i];
+      v.x = cap * tanhf(v.x / cap);
+      v.y = cap * tanhf(v.y / cap);
+      v.z = cap * tanhf(v.z / cap);
+      v.w = cap * tanhf(v.w / cap);
+      reinterpret_cast<float4*>(x)[i] = v;
+    }
+  } else {
+    for (long long i = i0; i < n; i += stride) x[i] = cap * tanhf(x[i] / cap);
+  }
+}
+
 // ---------------------------------------------------------------------------
 // MoE router: one warp per token, num_experts <= 1024.
 //   mode 0: softmax over all experts -> top-k -> divide by the selected sum
 //   mode 1: top-k on raw logits -> softmax over the selected
+//   mode 2: sigmoid of every logit -> top-k, the chosen scores as they are
 // groups > 0 (mode 0): experts form `groups` equal runs of neighbours; only the experts of the `keep` runs with the
 // largest single score take part.  The weights are multiplied by `scale`.
 // ---------------------------------------------------------------------------
-// logits may be bf16 / fp32 [tokens, E] or fp32 split-K partials [splits, tokens, E] (summed here, plus bias)
+// logits may be bf16 / fp32 [tokens, E] or fp32 split-K partials [splits, tokens, E] (summed here, plus bias), rows ld apart
 // kPer: experts per lane
 template <int kPer>
 __global__ void router_topk_kernel(const void* __restrict__ logits, int is_fp32, int splits, long long split_stride,
-                                   const __nv_bfloat16* __restrict__ bias, float* __restrict__ weights,
+                                   long long ld, const __nv_bfloat16* __restrict__ bias, float* __restrict__ weights,
                                    int* __restrict__ experts, int tokens, int num_experts, int top_k, int mode,
                                    int groups, int keep, float scale) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
@@ -246,10 +266,10 @@ __global__ void router_topk_kernel(const void* __restrict__ logits, int is_fp32,
   for (int j = 0; j < kPer; ++j) {
     const int e = j * 32 + lane;
     if (j < per && e < num_experts) {
-      float a = load_logit(logits, is_fp32, (long long)warp * num_experts + e);
+      float a = load_logit(logits, is_fp32, warp * ld + e);
 #pragma unroll 8
       for (int s = 1; s < splits; ++s)
-        a += reinterpret_cast<const float*>(logits)[s * split_stride + (long long)warp * num_experts + e];
+        a += reinterpret_cast<const float*>(logits)[s * split_stride + warp * ld + e];
       if (bias) a += __bfloat162float(bias[e]);
       v[j] = a;
     } else {
@@ -307,7 +327,7 @@ __global__ void router_topk_kernel(const void* __restrict__ logits, int is_fp32,
       argmax_combine(best, bi, ov, oi);
     }
     // mode 0 weight = softmax prob; mode 1 weight = exp(logit - max selected) (first pick is the max)
-    const float wgt = (mode == 0) ? expf(best - mx) / denom : expf(best - mx);
+    const float wgt = mode == 2 ? 1.f / (1.f + expf(-best)) : (mode == 0) ? expf(best - mx) / denom : expf(best - mx);
     sel_sum += wgt;
     if (lane == r % 32 && r / 32 == 0) { my_w = wgt; my_e = bi; }
     if ((bi & 31) == lane) {
@@ -317,7 +337,7 @@ __global__ void router_topk_kernel(const void* __restrict__ logits, int is_fp32,
     }
   }
   if (lane < top_k) {
-    weights[(long long)warp * top_k + lane] = my_w / (sel_sum + 1e-20f) * scale;
+    weights[(long long)warp * top_k + lane] = (mode == 2 ? my_w : my_w / (sel_sum + 1e-20f)) * scale;
     experts[(long long)warp * top_k + lane] = my_e;
   }
 }
@@ -341,11 +361,19 @@ extern "C" int nkb_sample(const void* logits, int is_fp32, int* out_ids, int row
                     out_ids, vocab, ld, temperature, top_k, top_p, seed, step);
 }
 
-extern "C" int nkb_router_topk(const void* logits, int is_fp32, int splits, long long split_stride, const void* bias,
+extern "C" int nkb_softcap(float* x, long long n, float cap, void* stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f) || (reinterpret_cast<uintptr_t>(x) & 15)) return -2;
+  const long long blocks = (n + 1023) / 1024;
+  return launch_pdl(softcap_kernel, dim3(unsigned(blocks < 148 * 8 ? blocks : 148 * 8)), dim3(256), 0,
+                    reinterpret_cast<cudaStream_t>(stream), x, n, cap);
+}
+
+extern "C" int nkb_router_topk(const void* logits, int is_fp32, int splits, long long split_stride, long long ld, const void* bias,
                                float* weights, int* experts, int tokens, int num_experts, int top_k, int mode, int groups,
                                int keep, float scale, void* stream) {
   if (tokens <= 0) return 0;
-  if (num_experts > 1024 || top_k > 32 || top_k > num_experts) return -2;
+  if (num_experts > 1024 || top_k > 32 || top_k > num_experts || mode < 0 || mode > 2 || ld < num_experts) return -2;
   if (groups > 0 && (mode != 0 || num_experts % groups || keep < 1 || keep > groups || top_k > num_experts / groups * keep))
     return -2;
   const int threads = 128;
@@ -354,7 +382,7 @@ extern "C" int nkb_router_topk(const void* logits, int is_fp32, int splits, long
   if (splits > 1 && !is_fp32) return -2;
   const auto go = [&](auto kernel) {
     return launch_pdl(kernel, dim3(blocks), dim3(threads), 0, reinterpret_cast<cudaStream_t>(stream), logits, is_fp32, splits,
-                      split_stride, (const __nv_bfloat16*)bias, weights, experts, tokens, num_experts, top_k, mode, groups, keep,
+                      split_stride, ld, (const __nv_bfloat16*)bias, weights, experts, tokens, num_experts, top_k, mode, groups, keep,
                       scale);
   };
   if (num_experts <= 32) return go(router_topk_kernel<1>);

@@ -20,13 +20,16 @@ from typing import List, Optional, Tuple, Union
 
 @dataclass(frozen=True)
 class RopeSpec:
-    """Rotary embedding of the first `dims` dimensions of a head, YaRN-scaled when factor is given."""
+    """Rotary embedding of the first `dims` dimensions of a head.  With a factor the frequencies are scaled: by YaRN, or with
+    `high` set by bands of wavelengths (Llama 3.1: kept below original / high, divided by the factor above original / low)."""
     base: float = 10000.0
     dims: int = 0
     factor: Optional[float] = None
     original: float = 0.0
     fast: float = 32.0
     slow: float = 1.0
+    low: float = 0.0
+    high: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -98,22 +101,68 @@ class ParallelSpec:
 
 
 @dataclass(frozen=True)
+class ChunkAttentionSpec:
+    """Grouped-query attention inside chunks of `chunk` positions: projection biases, half-split rotation, per-head norm of
+    queries and keys, one gate per head.  kv_from: the keys and values are those of that layer."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    chunk: int
+    rope: RopeSpec = RopeSpec()
+    kv_from: Optional[int] = None
+    kind = "chunk"
+
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    """Latent attention over the last `window` tokens with a sink and a gate per head: queries through a latent of q_rank, keys
+    and values from a cached latent of kv_rank and a shared rotated part of `rot` dimensions."""
+    heads: int
+    dim: int
+    rot: int
+    vdim: int
+    kv_rank: int
+    q_rank: int
+    scale: float
+    window: int
+    rope: RopeSpec = RopeSpec()
+    kind = "latent"
+
+
+@dataclass(frozen=True)
+class ClampedSpec:
+    """Gated feed-forward g sigmoid(1.702 g) (u + 1) with g at most `limit` and u within +-limit."""
+    ff: int
+    limit: float
+
+
+@dataclass(frozen=True)
 class ExpertsSpec:
-    """Routed SiLU-gated feed-forwards of width `ff`: softmax over all experts, the `top` best of the `keep` best of
-    `groups` equal groups (0: all), weights normalised and multiplied by `scale`."""
+    """Routed gated feed-forwards of width `ff`.  score "softmax": softmax over all experts, the `top` best of the `keep` best
+    of `groups` equal groups (0: all), weights normalised and multiplied by `scale`; "sigmoid": the `top` largest sigmoids,
+    not normalised.  limit 0: SiLU gate, otherwise the form of `ClampedSpec`.  scale_input: the weight multiplies an expert's
+    input instead of its output.  shared: a feed-forward of every token, with a sigmoid gate of its own."""
     experts: int
     top: int
     ff: int
     groups: int = 0
     keep: int = 0
     scale: float = 1.0
+    score: str = "softmax"
+    limit: float = 0.0
+    scale_input: bool = False
+    shared: Optional[ClampedSpec] = None
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     """block "gated": mixer and gated feed-forward beside each other, a sigmoid gate on both results; "pre-norm": the
-    mixer, then the feed-forward (plain `act`, or `experts`), each added to the residual."""
-    mixer: Union[MapsAttentionSpec, RecurrenceSpec, LinearAttentionSpec, ParallelSpec]
+    mixer, then the feed-forward (plain `act`, or `experts`), each added to the residual; "parallel": mixer and feed-forward
+    (gated `act`, or `experts`) on one norm, their sum added to the residual, then the per-layer token input."""
+    mixer: Union[MapsAttentionSpec, RecurrenceSpec, LinearAttentionSpec, ParallelSpec, ChunkAttentionSpec,
+                 LatentAttentionSpec]
     ff: int = 0                      # 0: no dense feed-forward
     act: str = "gelu_tanh"
     block: str = "gated"
@@ -170,6 +219,9 @@ class ModelConfig:
     norm_groups: int = 1
     norm_offset: float = 0.0              # added to the stored weights of the layer and final norms
     tie_embeddings: bool = False          # logits from the embedding table
+    layer_norm: bool = False              # layer norms with bias instead of RMS norms
+    token_side: int = 0                   # width of the per-layer token input (0: none)
+    logit_softcap: float = 0.0            # > 0: logits <- cap * tanh(logits / cap)
 
     @property
     def q_size(self) -> int:
@@ -278,8 +330,9 @@ def tiny(**kw) -> ModelConfig:
 
 
 def rope_frequencies(rope: RopeSpec):
-    """(frequencies [dims / 2], cos / sin multiplier) of a `RopeSpec`.  With a factor, the frequencies are blended
-    between base^(-2i/dims) and the same divided by the factor over the pairs whose wavelengths lie between
+    """(frequencies [dims / 2], cos / sin multiplier) of a `RopeSpec`.  With a factor and `high`, frequencies of wavelengths
+    above original / low are divided by the factor, those below original / high are kept and those in between are blended
+    linearly in original / wavelength.  With a factor alone, the frequencies are blended between base^(-2i/dims) and the same divided by the factor over the pairs whose wavelengths lie between
     original / fast and original / slow tokens (bounds rounded outwards to whole pairs)."""
     import torch
 
@@ -287,6 +340,10 @@ def rope_frequencies(rope: RopeSpec):
     freq = rope.base ** (-2.0 * i / max(rope.dims, 1))
     if rope.factor is None:
         return freq, 1.0
+    if rope.high:
+        turns = rope.original * freq / (2 * math.pi)
+        s = ((turns - rope.low) / (rope.high - rope.low)).clamp(0, 1)
+        return (1 - s) * freq / rope.factor + s * freq, 1.0
 
     def pair_of(turns):          # pair index whose angle makes `turns` full turns over the original length
         return rope.dims * math.log(rope.original / (2 * math.pi * turns)) / (2 * math.log(rope.base))
@@ -395,6 +452,79 @@ def mumilorn_shape(width: int, *, layers: int, heads: int, kv_heads: int, ff: in
             specs.append(LayerSpec(mixer, ff, "relu2", "pre-norm"))
     base = dict(name="mumilorn", vocab_size=vocab, hidden_size=width, num_layers=layers, rms_eps=1e-6, layers=specs,
                 norm_offset=1.0, tie_embeddings=True, max_position=0)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+def ligizen_config(raw: dict, **kw) -> ModelConfig:
+    """`ModelConfig` of a Ligizen config.json."""
+
+    def mixer_of(kind, m):
+        r = m["rot"]
+        sc = r.get("scaling") or {}
+        rope = RopeSpec(r["base"], r["dims"], sc.get("factor"), sc.get("original", 0), low=sc.get("low", 0.0),
+                        high=sc.get("high", 0.0))
+        if kind == "attention":
+            return ChunkAttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["scale"], m["mask"]["size"], rope,
+                                      m.get("kv_from"))
+        if kind == "latent_attention":
+            if r["dims"] != m["rot_dim"]:
+                raise ValueError("the whole rotated part of a latent attention is rotated")
+            return LatentAttentionSpec(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"], m["scale"],
+                                       m["mask"]["size"], rope)
+        raise ValueError(f"unknown layer type {kind!r}")
+
+    layers = []
+    for i, l in enumerate(raw["layers"]):
+        mlp, ff, experts = l.get("mlp"), 0, None
+        if mlp is not None:
+            if mlp["kind"] == "dense":
+                ff = mlp["ff"]
+            elif mlp["kind"] == "moe":
+                r, sh = mlp["router"], mlp.get("shared")
+                experts = ExpertsSpec(r["experts"], r["top"], mlp["expert"]["ff"], score="sigmoid",
+                                      limit=mlp["expert"]["limit"], scale_input=True,
+                                      shared=ClampedSpec(sh["ff"], sh["limit"]) if sh else None)
+            else:
+                raise ValueError(f"unknown feed-forward kind {mlp['kind']!r}")
+        mixer = mixer_of(l["type"], l["mixer"])
+        src = getattr(mixer, "kv_from", None)
+        if src is not None and not (0 <= src < i and layers[src].mixer.kind == "chunk" and layers[src].mixer.kv_from is None):
+            raise ValueError(f"layer {i} cannot read the keys of layer {src}")
+        layers.append(LayerSpec(mixer, ff, "silu", "parallel", experts))
+    base = dict(name="ligizen", vocab_size=raw["vocab"], hidden_size=raw["width"], num_layers=len(layers),
+                rms_eps=raw["norm"]["eps"], layers=layers, embedding_scale=raw["embedding"]["scale"], layer_norm=True,
+                token_side=(raw.get("token_side") or {}).get("dim", 0), logit_softcap=raw.get("logit_softcap") or 0.0,
+                max_position=0)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+def ligizen_shape(width: int, *, layers: int, heads: int, kv_heads: int, ff: int, vocab: int = 32000, dim: int = 128,
+                  window: int = 1024, chunk: int = 1024, latent_dim: int = 64, rot: int = 64, kv_rank: int = 512,
+                  q_rank: int = 1536, side: int = 256, experts: int = 0, top: int = 0, expert_ff: int = 0, moe_every: int = 2,
+                  share_every: int = 0, **kw) -> ModelConfig:
+    """A Ligizen configuration of regular shape: latent and chunked attention alternate; with experts, every `moe_every`-th
+    feed-forward is routed (with a shared expert); with share_every, every share_every-th chunked layer but the first reads
+    the keys and values of the chunked layer before it."""
+    rope = RopeSpec(500000.0, dim, 8.0, 8192, low=1.0, high=4.0)
+    specs, chunked, source = [], 0, None
+    for i in range(layers):
+        if i % 2 == 0:
+            mixer = LatentAttentionSpec(heads, latent_dim, rot, dim, kv_rank, q_rank, (latent_dim + rot) ** -0.5, window,
+                                        RopeSpec(10000.0, rot))
+        else:
+            chunked += 1
+            shares = share_every and chunked > 1 and chunked % share_every == 0
+            mixer = ChunkAttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, chunk, rope, source if shares else None)
+            source = source if shares else i
+        if experts and i % moe_every == moe_every - 1:
+            specs.append(LayerSpec(mixer, 0, "silu", "parallel", ExpertsSpec(
+                experts, top, expert_ff, score="sigmoid", limit=7.0, scale_input=True, shared=ClampedSpec(expert_ff, 7.0))))
+        else:
+            specs.append(LayerSpec(mixer, ff, "silu", "parallel"))
+    base = dict(name="ligizen", vocab_size=vocab, hidden_size=width, num_layers=layers, rms_eps=1e-5, layers=specs,
+                layer_norm=True, token_side=side, logit_softcap=50.0, max_position=0)
     base.update(kw)
     return ModelConfig(**base)
 

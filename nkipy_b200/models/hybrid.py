@@ -1,9 +1,10 @@
 """Decoders whose layers are listed one by one: each layer has its own token mixer (models/mixers.py) and feed-forward,
-around an fp32 residual stream.  Two kinds of layer:
+around an fp32 residual stream.  Three kinds of layer:
 
     gated (Tolenex)       h1 = norm1(x), h2 = norm2(x)
                           x <- x + sigmoid(W_g1 h1 + b1) * mixer(h1) + sigmoid(W_g2 h2 + b2) * feed_forward(h2)
     pre-norm (Mumilorn)   x <- x + mixer(norm1(x)),   then   x <- x + feed_forward(norm2(x))
+    parallel (Ligizen)    h = norm1(x);  x <- x + mixer(h) + feed_forward(h),  then  x <- x + norm(token input of x)
 
 A layer is a list of stages; a stage reads norms of the residual and returns the branches that are added to it.  One
 kernel per stage (`ops.gated_residual`) sums the branches, applies what precedes a repeated pass of a looped block and
@@ -25,7 +26,7 @@ from typing import Dict, List, Optional
 import torch
 
 from .. import ops
-from ..ops import Branch, Proj
+from ..ops import Branch, Norm, Proj
 from ..parallel.comm import TPGroup
 from .config import LayerSpec, ModelConfig, RopeSpec, rope_frequencies
 from .kv_cache import PagedKVCache
@@ -37,7 +38,7 @@ SMALL_BATCH = 128
 
 
 class Stage:
-    """norms: weights of the residual's norms it reads; run(h, entry, cache, batch) -> branches."""
+    """norms: the residual's norms it reads (weights of RMS norms, or `ops.Norm`); run(h, entry, cache, batch) -> branches."""
     __slots__ = ("norms", "run")
 
     def __init__(self, norms, run):
@@ -100,12 +101,33 @@ class DenseMLP:
     def weights(self):
         return [self.up, self.down]
 
-    def run(self, model: "HybridLM", h: torch.Tensor) -> Branch:
+    def run(self, model: "HybridLM", h: torch.Tensor) -> List[Branch]:
         if x_small(h):
             a = ops.activation(Proj(model.project(h, self.up), 0, self.up.shape[0]), self.act, dtype=h.dtype)
         else:
             a = ops.linear(h, self.up, swap=False, out_act=self.act)
-        return Branch(Proj(model.project(a, self.down), 0, h.shape[1]))
+        return [Branch(Proj(model.project(a, self.down), 0, h.shape[1]))]
+
+
+class GatedMLP:
+    """down(act(gate h) * up h).  `w_wide` holds [gate; up] as rows for the input projection of a layer whose sublayers share
+    their input."""
+
+    def __init__(self, act: str, t: Tensors):
+        self.act, self.w_wide, self.w_narrow, self.down = act, t.mat("gate", "up"), None, t.mat("down")
+
+    def weights(self):
+        return [self.w_wide, self.down]
+
+    def run(self, model: "HybridLM", h: torch.Tensor, wide: Optional[Proj] = None, narrow=None) -> List[Branch]:
+        if wide is None and x_small(h):
+            wide = Proj(model.project(h, self.w_wide), 0, self.w_wide.shape[0])
+        if wide is not None:
+            n = wide.width // 2
+            a = ops.gated_act(Proj(wide.t, wide.col, n), Proj(wide.t, wide.col + n, n), self.act, dtype=h.dtype)
+        else:
+            a = ops.linear(h, self.w_wide, gated=True, act=self.act, swap=False)
+        return [Branch(Proj(model.project(a, self.down), 0, h.shape[1]))]
 
 
 class PreNormLayer:
@@ -124,7 +146,7 @@ class PreNormLayer:
             raise ValueError("projection sizes do not fit the configuration")
         self.stages = [Stage([t.f32("norm1", cfg.norm_offset)], self._mix)]
         if self.mlp is not None:
-            self.stages.append(Stage([t.f32("norm2", cfg.norm_offset)], lambda h, *_: [self.mlp.run(model, h[0])]))
+            self.stages.append(Stage([t.f32("norm2", cfg.norm_offset)], lambda h, *_: self.mlp.run(model, h[0])))
 
     def weights(self):
         ws = [self.mixer.w_in, self.mixer.w_o, getattr(getattr(self.mixer, "right", None), "w_each", None)]
@@ -136,7 +158,71 @@ class PreNormLayer:
         return [Branch(Proj(m.project(self.mixer.run(m, y, h[0], entry, cache, b), self.mixer.w_o), 0, self.width))]
 
 
-LAYERS = {"gated": GatedLayer, "pre-norm": PreNormLayer}
+class ParallelLayer:
+    """Mixer and feed-forward on one norm of the residual, then the layer's token input: a low-rank product of the residual and
+    a row of a table that belongs to the token and the layer.
+
+    Small batches run one input projection [feed-forward's wide rows; mixer; feed-forward's narrow rows], each part filled up
+    to whole 16 bytes with zero rows; `spans` holds the rows of the parts."""
+
+    def __init__(self, model: "HybridLM", spec: LayerSpec, t: Tensors):
+        cfg = model.cfg
+        self.model, self.width = model, cfg.hidden_size
+        self.mixer = mixer = MIXERS[spec.mixer.kind](spec.mixer, t.under("mix."), cfg.rms_eps)
+        self.mlp = None
+        if spec.experts is not None:
+            self.mlp = RoutedExperts(spec.experts, t.under("mlp."))
+        elif spec.ff:
+            self.mlp = GatedMLP(spec.act, t.under("mlp."))
+        if sum(mixer.widths) != mixer.w_in.shape[0]:
+            raise ValueError("projection sizes do not fit the configuration")
+        parts = [getattr(self.mlp, "w_wide", None), mixer.w_in, getattr(self.mlp, "w_narrow", None)]
+        self.spans, rows, n = [], [], 0
+        for w in parts:
+            if w is None:
+                self.spans.append(None)
+                continue
+            self.spans.append((n, w.shape[0]))
+            pad = -w.shape[0] % 8
+            rows += [w] + ([w.new_zeros((pad, w.shape[1]))] if pad else [])
+            n += w.shape[0] + pad
+        self.w_in = torch.cat(rows).contiguous()
+        views = [None if s is None else self.w_in[s[0]:s[0] + s[1]] for s in self.spans]
+        start, rows = self.spans[1]
+        mixer.w_in = self.w_in[start:start + (rows + 7) // 8 * 8]
+        if self.mlp is not None:
+            self.mlp.w_wide, self.mlp.w_narrow = views[0], views[2]
+        self.stages = [Stage([model.norm(t, "norm1")], self._run)]
+        if cfg.token_side:
+            self.side_gate, self.side_proj, self.side_norm = t.mat("side.gate"), t.mat("side.proj"), t.f32("side.norm")
+            self.stages.append(Stage([Norm()], self._token_input))
+
+    def weights(self):
+        ws = [self.w_in, self.mixer.w_o, *getattr(self.mixer, "weights", list)()]
+        if self.mlp is not None:
+            ws += [w for w in self.mlp.weights() if w is not self.mlp.w_wide and w is not self.mlp.w_narrow]
+        return ws + ([self.side_gate, self.side_proj] if self.model.cfg.token_side else [])
+
+    def _run(self, h, entry, cache, b) -> List[Branch]:
+        m, h = self.model, h[0]
+        wide = narrow = None
+        if x_small(h):
+            y = m.project(h, self.w_in)
+            wide, mix, narrow = [None if s is None else Proj(y, *s) for s in self.spans]
+        else:
+            mix = Proj(m.project(h, self.mixer.w_in), 0, self.spans[1][1])
+        o = self.mixer.run(m, mix, h, entry, cache, b)
+        branches = [Branch(Proj(m.project(o, self.mixer.w_o), 0, self.width))]
+        return branches if self.mlp is None else branches + self.mlp.run(m, h, wide, narrow)
+
+    def _token_input(self, h, entry, cache, b) -> List[Branch]:
+        m, n = self.model, self.side_gate.shape[0]
+        z = Proj(m.project(h[0], self.side_gate), 0, n)
+        a = ops.gated_act(z, Proj(m.side_table, m.layers.index(self) * n, n), "gelu_tanh", dtype=m.dtype, up_rows=b.ids)
+        return [Branch(Proj(m.project(a, self.side_proj), 0, self.width), norm=self.side_norm)]
+
+
+LAYERS = {"gated": GatedLayer, "pre-norm": PreNormLayer, "parallel": ParallelLayer}
 
 
 class HybridLM:
@@ -155,17 +241,26 @@ class HybridLM:
         get = lambda name: weights[name].to(self.device)
         self.embed = get("embed").to(dtype).contiguous()
         self.head = self.embed if cfg.tie_embeddings else get("head").to(dtype).contiguous()
-        self.final_norm = (get("final.norm").float() + cfg.norm_offset).contiguous()
+        self.final_norm = self.norm(Tensors(get, "final.", dtype), "norm")
+        self.side_table = get("side.embed").to(dtype).contiguous() if cfg.token_side else None
         self.layers = [LAYERS[s.block](self, s, Tensors(get, f"l{i}.", dtype)) for i, s in enumerate(cfg.layers)]
         self.runs = cfg.layer_runs()
-        self.entry = []                      # first cache entry of every run
-        n = 0
+        self.entry = []                      # first cache entry of every run, or that of the layer whose keys it reads
+        n, first = 0, {}
         for i, _ in self.runs:
-            self.entry.append(n)
+            source = getattr(cfg.layers[i].mixer, "kv_from", None)
+            first[i] = n if source is None else first[source]
+            self.entry.append(first[i])
             n += len(self.layers[i].mixer.entries())
         self.loop_step = get("loop.step").float().contiguous() if cfg.loop else None
         self._rope: Dict[RopeSpec, torch.Tensor] = {}
         self._offsets: Dict[tuple, torch.Tensor] = {}
+
+    def norm(self, t: Tensors, name: str) -> Norm:
+        """The model's kind of norm, from the tensors of that name."""
+        if self.cfg.layer_norm:
+            return Norm(t.f32(name), t.f32(name + ".b"), center=True)
+        return Norm(t.f32(name, self.cfg.norm_offset))
 
     # ------------------------------------------------------------------ cache
     def new_cache(self, num_blocks: int, max_batch: int, max_seq_len: int,
@@ -188,7 +283,7 @@ class HybridLM:
         return self._rope[rope]
 
     def weight_bytes(self) -> int:
-        ts = [self.embed, self.head] + [t for l in self.layers for t in l.weights()]
+        ts = [self.embed, self.head] + ([] if self.side_table is None else [self.side_table]) + [t for l in self.layers for t in l.weights()]
         return sum(t.numel() * t.element_size() for t in ts)
 
     # ------------------------------------------------------------------ layers
@@ -242,7 +337,7 @@ class HybridLM:
             stages = self.layers[self.runs[r][0]].stages
             branches = stages[s].run(h, self.entry[r], cache, b)
             if return_hidden and s == len(stages) - 1:
-                taps.append(ops.gated_residual(x, branches)[0])
+                taps.append(ops.gated_residual(x, branches, eps=cfg.rms_eps)[0])
             x, h = ops.gated_residual(x, branches, **ahead(n + 1), **norm)
         return (h[0], taps) if return_hidden else h[0]
 
@@ -253,15 +348,16 @@ class HybridLM:
         rows[b] is the batch row (state slot) of sequence b.  Returns the final-normed hidden states [T, W] (and the
         residual stream after every layer run)."""
         return self._forward(ids, cache, Batch(positions, slots, block_table, context_lens, q_start, q_lens, max_q_len,
-                                               rows), return_hidden)
+                                               rows, ids), return_hidden)
 
     def decode_step(self, ids, positions, slots, cache, block_table, context_lens, return_hidden: bool = False):
         """One new token for every batch row; rows with a negative context length are inactive."""
-        return self._forward(ids, cache, Batch(positions, slots, block_table, context_lens), return_hidden)
+        return self._forward(ids, cache, Batch(positions, slots, block_table, context_lens, ids=ids), return_hidden)
 
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:
         """fp32 logits [rows, vocab]."""
-        return ops.linear(hidden, self.head, fp32_out=True)
+        z = ops.linear(hidden, self.head, fp32_out=True)
+        return ops.softcap(z, self.cfg.logit_softcap) if self.cfg.logit_softcap > 0 else z
 
     def greedy(self, hidden: torch.Tensor, out_ids: Optional[torch.Tensor] = None) -> torch.Tensor:
         return ops.argmax(self.logits(hidden), out_ids=out_ids)
@@ -271,13 +367,15 @@ class HybridLM:
 
 
 class Batch:
-    """Where the tokens of a step sit: cache slots, block tables, and how they are grouped into sequences (q_lens
+    """The tokens of a step, where they sit (cache slots, block tables) and how they are grouped into sequences (q_lens
     None: one per batch row)."""
-    __slots__ = ("positions", "slots", "block_table", "context_lens", "q_start", "q_lens", "max_q_len", "rows")
+    __slots__ = ("positions", "slots", "block_table", "context_lens", "q_start", "q_lens", "max_q_len", "rows", "ids")
 
-    def __init__(self, positions, slots, block_table, context_lens, q_start=None, q_lens=None, max_q_len=1, rows=None):
+    def __init__(self, positions, slots, block_table, context_lens, q_start=None, q_lens=None, max_q_len=1, rows=None,
+                 ids=None):
         self.positions, self.slots, self.block_table, self.context_lens = positions, slots, block_table, context_lens
         self.q_start, self.q_lens, self.max_q_len, self.rows = q_start, q_lens, max_q_len, rows
+        self.ids = ids
 
 
 def x_small(h: torch.Tensor) -> bool:

@@ -7,12 +7,12 @@ and returns the operand of the output projection.  A new kind of layer is a new 
 
 from __future__ import annotations
 
-from typing import List
+from typing import List, Union
 
 import torch
 
 from .. import ops
-from ..ops import Decay, MapsSpec, Proj
+from ..ops import Decay, LatentSpec, MapsSpec, Proj
 from ..ops.linear_attention import linear_state_shape
 from ..ops.mixers import hgrn2_state_shape
 from .kv_cache import KVLayer, StateLayer
@@ -40,10 +40,12 @@ class Tensors:
         return torch.stack([self.raw(n).to(self.dtype) for n in names]).contiguous()
 
 
-def columns(y: torch.Tensor, widths: List[int]) -> List[Proj]:
-    out, c = [], 0
+def columns(y: Union[torch.Tensor, Proj], widths: List[int]) -> List[Proj]:
+    """Slices of a projection's result (or of a slice of it) of the given widths, one after the other."""
+    t, c = (y.t, y.col) if isinstance(y, Proj) else (y, 0)
+    out = []
     for w in widths:
-        out.append(Proj(y, c, w))
+        out.append(Proj(t, c, w))
         c += w
     return out
 
@@ -134,6 +136,70 @@ class WindowAttentionMixer:
         return ops.gate_heads(o, g, "sigmoid", scale=self.scale, out=out)
 
 
+class ChunkAttentionMixer:
+    """Grouped-query attention inside chunks of positions, one gate per head.  With `kv_from` its cache entry is that of
+    another layer, whose keys and values it reads with its own queries."""
+
+    def __init__(self, spec, t: Tensors, eps: float):
+        self.spec = spec
+        own = spec.kv_from is None
+        names = ("q", "k", "v") if own else ("q",)
+        self.w_in, self.w_o = t.mat(*names, "g"), t.mat("o")
+        self.widths = [spec.heads * spec.dim, spec.kv_heads * spec.dim, spec.kv_heads * spec.vdim][:len(names)] + [spec.heads]
+        self.bias = torch.cat([t.f32(n + ".b") for n in names]).contiguous()
+        self.maps = MapsSpec(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.scale, maps=1, eps=eps, chunk=spec.chunk,
+                             tiled=t.dtype == torch.bfloat16)
+
+    def entries(self):
+        return [KVLayer(self.spec.kv_heads, self.maps.dim_p, self.maps.vdim_p)] if self.spec.kv_from is None else []
+
+    def run(self, model, y, h, entry, cache, b):
+        q, *kv, g = columns(y, self.widths)
+        kc, vc = cache.k[entry], cache.v[entry]
+        q = ops.rope_norm_append(self.maps, q, *(kv or (None, None)), self.bias, model.rope_table(self.spec.rope), b.positions,
+                                 b.slots, kc, vc)
+        o = ops.heads_attention(self.maps, q, kc, vc, b.block_table, b.context_lens, q_start=b.q_start, q_lens=b.q_lens,
+                                max_q_len=b.max_q_len)
+        return ops.gate_heads(o, g, "sigmoid")
+
+
+class LatentAttentionMixer:
+    """Latent attention with a sink and a gate per head.  Attention runs on the cached latents: the queries are folded through
+    the keys' up projection, and the values' up projection is applied to the mixtures of latents."""
+
+    def __init__(self, spec, t: Tensors, eps: float):
+        self.spec = spec
+        H, R = spec.heads, spec.kv_rank
+        self.w_in, self.w_o = t.mat("dq", "dkv", "g"), t.mat("o")
+        self.widths = [spec.q_rank, R + spec.rot, H]
+        self.w_uq = t.mat("uq")
+        self.w_uk = t.mat("uk").reshape(H, spec.dim, R).transpose(1, 2).contiguous()     # [H, R, dim]
+        self.w_uv = t.mat("uv").reshape(H, spec.vdim, R)
+        self.q_norm, self.kv_norm, self.sink = t.f32("dq.norm"), t.f32("dkv.norm"), t.f32("sink")
+        self.latent = LatentSpec(H, spec.dim, spec.rot, spec.vdim, R, spec.q_rank, spec.scale, spec.window, eps,
+                                 tiled=t.dtype == torch.bfloat16)
+
+    def weights(self):
+        return [self.w_uq, self.w_uk, self.w_uv]
+
+    def entries(self):
+        return [KVLayer(1, self.latent.row, 0)]
+
+    def run(self, model, y, h, entry, cache, b):
+        s, (q, kv, g) = self.latent, columns(y, self.widths)
+        table, rows = model.rope_table(self.spec.rope), cache.k[entry]
+        T = h.shape[0]
+        c = ops.latent_append(s, q, kv, self.q_norm, self.kv_norm, table, b.positions, b.slots, rows)
+        up = Proj(model.project(c, self.w_uq), 0, self.w_uq.shape[0])
+        plain = torch.empty((s.heads, T, s.dim), dtype=model.dtype, device=h.device)
+        q = torch.empty((s.heads, T, s.row), dtype=model.dtype, device=h.device)
+        ops.latent_queries(s, up, table, b.positions, plain.transpose(0, 1), q.transpose(0, 1)[..., s.rank:])
+        ops.head_linear(plain, self.w_uk, out=q[..., :s.rank])
+        o = ops.latent_attention(s, q, rows, b.block_table, b.context_lens, q_start=b.q_start, q_lens=b.q_lens,
+                                 sinks=self.sink)
+        return ops.gate_heads(ops.head_linear(o, self.w_uv).transpose(0, 1), g, "sigmoid")
+
+
 class TimeMixMixer:
     """RWKV-style time mixing.  Its projections read mixes of neighbouring tokens and not h, so it has no rows in the
     layer's input projection."""
@@ -183,4 +249,4 @@ class ParallelMixer:
 
 
 MIXERS = {"hgrn2": Hgrn2Mixer, "attention": MapsMixer, "gla": LinearAttentionMixer, "window": WindowAttentionMixer,
-          "rwkv": TimeMixMixer, "parallel": ParallelMixer}
+          "rwkv": TimeMixMixer, "parallel": ParallelMixer, "chunk": ChunkAttentionMixer, "latent": LatentAttentionMixer}

@@ -14,6 +14,8 @@ reference's sharding with the same code path (all experts local, narrower expert
 
 from __future__ import annotations
 
+from typing import List, Optional
+
 import torch
 
 from .. import ops
@@ -93,31 +95,57 @@ def route_splits(width: int) -> int:
 
 
 class RoutedExperts:
-    """Routed feed-forward of one layer of a layer-by-layer decoder (`config.ExpertsSpec`, one rank).  The weighted sum of
+    """Routed feed-forward of one layer of a layer-by-layer decoder (`config.ExpertsSpec`, one rank).  The (weighted) sum of
     the experts' rows is left to the residual kernel (`ops.Branch`).  bf16 sizes with 16-byte rows run the grouped
-    tcgen05 products, everything else the grouped products on the CUDA cores."""
+    tcgen05 products, everything else the grouped products on the CUDA cores.
+
+    Rows for the input projection of a layer whose sublayers share their input: `w_wide` the shared expert's [gate; up] (None
+    without one), `w_narrow` [router; shared gate]."""
 
     def __init__(self, spec, t):
         self.spec = spec
-        self.router = t.mat("router")
         self.gate_up = torch.stack([t.mat(f"e{e}.gate", f"e{e}.up") for e in range(spec.experts)]).contiguous()
         self.down = t.stack(*[f"e{e}.down" for e in range(spec.experts)])
         self.tiled = t.dtype == torch.bfloat16 and self.down.shape[1] % 8 == 0 and spec.ff % 8 == 0
+        self.w_wide, self.shared_down = None, None
+        self.w_narrow = t.mat("router")
+        if spec.shared:
+            self.w_wide, self.shared_down = t.mat("shared.gate", "shared.up"), t.mat("shared.down")
+            self.w_narrow = t.mat("router", "shared.sg")
 
     def weights(self):
-        return [self.router, self.gate_up, self.down]
+        return [w for w in (self.w_narrow, self.gate_up, self.down, self.w_wide, self.shared_down) if w is not None]
 
-    def run(self, model, h: torch.Tensor) -> Branch:
+    def run(self, model, h: torch.Tensor, wide: Optional[Proj] = None, narrow: Optional[Proj] = None) -> List[Branch]:
+        """wide / narrow: results of `w_wide` and `w_narrow` when the layer has them already."""
         s, (T, W) = self.spec, h.shape
-        logits = ops.linear(h, self.router, splits=route_splits(W)) if h.dtype == torch.bfloat16 else ops.linear(h, self.router)
-        weights, experts = ops.router_topk(logits, s.top, groups=s.groups, keep=s.keep, scale=s.scale)
-        plan = ops.moe_dispatch(h, experts, 0, s.experts, gather=self.tiled)
+        if narrow is None:
+            z = ops.linear(h, self.w_narrow, splits=route_splits(W)) if h.dtype == torch.bfloat16 else ops.linear(h, self.w_narrow)
+            narrow = Proj(z, 0, self.w_narrow.shape[0])
+        logits = Proj(narrow.t, narrow.col, s.experts)
+        if s.score == "sigmoid":
+            weights, experts = ops.router_topk(logits, s.top, "sigmoid_topk", scale=s.scale)
+        else:
+            weights, experts = ops.router_topk(logits, s.top, groups=s.groups, keep=s.keep, scale=s.scale)
+        gather = self.tiled or s.scale_input
+        plan = ops.moe_dispatch(h, experts, 0, s.experts, gather=gather, weights=weights if s.scale_input else None)
         if self.tiled:
             act = ops.grouped_linear(plan.x_sorted, self.gate_up, plan.offsets, max_rows_per_group=T, gated=True,
-                                     tiles=plan.tiles)
+                                     act_limit=s.limit, tiles=plan.tiles)
             y = ops.grouped_linear(act, self.down, plan.offsets, max_rows_per_group=T, tiles=plan.tiles)
         else:
-            gu = ops.grouped_linear_simt(plan, h, self.gate_up, False)
-            act = ops.gated_act(Proj(gu, 0, s.ff), Proj(gu, s.ff, s.ff), "silu", dtype=h.dtype)
+            gu = ops.grouped_linear_simt(plan, plan.x_sorted, self.gate_up, gather)
+            act = ops.gated_act(Proj(gu, 0, s.ff), Proj(gu, s.ff, s.ff), "clamped" if s.limit else "silu", dtype=h.dtype,
+                                limit=s.limit)
             y = ops.grouped_linear_simt(plan, act, self.down, True)
-        return Branch(Proj(y, 0, W), pair_pos=plan.pair_pos, pair_w=weights)
+        if s.scale_input:
+            out = [Branch(Proj(y, 0, W), pair_pos=plan.pair_pos, top_k=s.top)]
+        else:
+            out = [Branch(Proj(y, 0, W), pair_pos=plan.pair_pos, pair_w=weights)]
+        if s.shared:
+            n, limit = s.shared.ff, s.shared.limit
+            if wide is None:
+                wide = Proj(model.project(h, self.w_wide), 0, 2 * n)
+            act = ops.gated_act(Proj(wide.t, wide.col, n), Proj(wide.t, wide.col + n, n), "clamped", dtype=h.dtype, limit=limit)
+            out.append(Branch(Proj(model.project(act, self.shared_down), 0, W), Proj(narrow.t, narrow.col + s.experts, 1)))
+        return out

@@ -77,6 +77,7 @@ ARCHITECTURES: Dict[str, Architecture] = {
                                                  num_local_experts="num_experts", sliding_window="sliding_window")),
     "Tolenex": _hybrid(C.tolenex_config),
     "Mumilorn": _hybrid(C.mumilorn_config),
+    "Ligizen": _hybrid(C.ligizen_config),
 }
 
 
@@ -91,7 +92,7 @@ def for_config(cfg: C.ModelConfig) -> Architecture:
     """The architecture entry that runs a configuration made in code."""
     if cfg.layers is None:
         return ARCHITECTURES["LlamaForCausalLM"]
-    return ARCHITECTURES["Mumilorn" if cfg.name == "mumilorn" else "Tolenex"]
+    return ARCHITECTURES[{"mumilorn": "Mumilorn", "ligizen": "Ligizen"}.get(cfg.name, "Tolenex")]
 
 
 def read_config(folder: str):

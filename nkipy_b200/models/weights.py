@@ -164,6 +164,14 @@ def _mixer_shapes(m, W: int) -> Dict[str, tuple]:
         return {**{f"mu.{n}": (W,) for n in "rkvgw"}, **{n: (c, W) for n in "rkvg"}, "w1": (rank, W), "w2": (c, rank),
                 "w0": (c,), "u": (m.heads, m.dim), "norm": (c,), "o": (W, c)}
     out = m.heads * m.vdim
+    if m.kind == "chunk":
+        q, k, v = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim
+        own = {} if m.kv_from is not None else {"k": (k, W), "k.b": (k,), "v": (v, W), "v.b": (v,)}
+        return {"q": (q, W), "q.b": (q,), **own, "g": (m.heads, W), "o": (W, out)}
+    if m.kind == "latent":
+        return {"dq": (m.q_rank, W), "dq.norm": (m.q_rank,), "uq": (m.heads * (m.dim + m.rot), m.q_rank),
+                "dkv": (m.kv_rank + m.rot, W), "dkv.norm": (m.kv_rank,), "uk": (m.heads * m.dim, m.kv_rank),
+                "uv": (out, m.kv_rank), "sink": (m.heads,), "g": (m.heads, W), "o": (W, out)}
     if m.kind == "window":
         q, k = m.heads * m.dim, m.kv_heads * m.dim
         return {"q": (q, W), "k": (k, W), "v": (m.kv_heads * m.vdim, W), "q.norm": (q,), "k.norm": (k,), "g": (out, W),
@@ -187,21 +195,36 @@ def hybrid_weight_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
         out["head"] = (V, W)
     if cfg.loop:
         out["loop.step"] = (cfg.loop.times, W)
+    if cfg.layer_norm:
+        out["final.norm.b"] = (W,)
+    if cfg.token_side:
+        out["side.embed"] = (V, len(cfg.layers) * cfg.token_side)
     for i, layer in enumerate(cfg.layers):
         shapes = {"norm1": (W,), **{"mix." + k: v for k, v in _mixer_shapes(layer.mixer, W).items()}}
         if layer.block == "gated":
             shapes.update({"rg1": (W, W), "rg1.b": (W,)})
-        if layer.ff or layer.experts:
+        if cfg.layer_norm:
+            shapes["norm1.b"] = (W,)
+        if (layer.ff or layer.experts) and layer.block != "parallel":
             shapes["norm2"] = (W,)
         if layer.ff:
             shapes.update({"mlp.up": (layer.ff, W), "mlp.down": (W, layer.ff)})
+            if layer.block != "pre-norm":
+                shapes["mlp.gate"] = (layer.ff, W)
             if layer.block == "gated":
-                shapes.update({"mlp.gate": (layer.ff, W), "rg2": (W, W), "rg2.b": (W,)})
+                shapes.update({"rg2": (W, W), "rg2.b": (W,)})
         if layer.experts:
             x = layer.experts
             shapes["mlp.router"] = (x.experts, W)
             for e in range(x.experts):
                 shapes.update({f"mlp.e{e}.gate": (x.ff, W), f"mlp.e{e}.up": (x.ff, W), f"mlp.e{e}.down": (W, x.ff)})
+            if x.shared:
+                n = x.shared.ff
+                shapes.update({"mlp.shared.gate": (n, W), "mlp.shared.up": (n, W), "mlp.shared.down": (W, n),
+                               "mlp.shared.sg": (1, W)})
+        if cfg.token_side:
+            n = cfg.token_side
+            shapes.update({"side.gate": (n, W), "side.proj": (W, n), "side.norm": (W,)})
         out.update({f"l{i}." + k: v for k, v in shapes.items()})
     return out
 

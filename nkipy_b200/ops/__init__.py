@@ -29,8 +29,9 @@ from ._lib import KernelLibraryError, device_status, raise_on_device_error
 __all__ = [
     "linear", "decode_linear", "qkv_rope_append", "reduce_partials", "rmsnorm", "add_rmsnorm", "silu_mul", "embedding", "rope_kv_append",
     "argmax", "sample", "decode_advance", "router_topk", "moe_dispatch", "grouped_linear", "moe_combine", "paged_attn_decode", "flash_attn_prefill", "rope_table",
-    "Branch", "MapsSpec", "Proj", "activation", "gate_heads", "gated_act", "gated_residual", "hgrn2", "maps_append",
-    "heads_attention", "maps_attention", "row_norm_append",
+    "Branch", "MapsSpec", "Norm", "Proj", "activation", "gate_heads", "gated_act", "gated_residual", "hgrn2", "maps_append",
+    "heads_attention", "maps_attention", "row_norm_append", "rope_norm_append", "head_linear", "softcap",
+    "LatentSpec", "latent_append", "latent_attention", "latent_gather", "latent_queries",
     "Decay", "linear_attention", "low_rank", "token_mix",
     "KernelLibraryError", "device_status", "raise_on_device_error", "native_available", "launch_count",
     "reset_launch_count",
@@ -671,6 +672,17 @@ def argmax(logits: torch.Tensor, out_ids: Optional[torch.Tensor] = None,
     return out_ids
 
 
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """``cap * tanh(x / cap)`` of contiguous fp32 values, in place."""
+    if not _native(x):
+        return x.copy_(cap * torch.tanh(x / cap))
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise TypeError("softcap wants contiguous fp32 values")
+    _lib.check(_lib.lib().nkb_softcap(x.data_ptr(), x.numel(), float(cap), _stream()), "nkb_softcap")
+    _count_launch()
+    return x
+
+
 def sample(logits: torch.Tensor, temperature: float = 1.0, top_k: int = 0, top_p: float = 1.0, seed: int = 0,
            step: int = 0, out_ids: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Temperature / top-k / top-p sampling.  Candidates are limited to the 1024 most
@@ -699,14 +711,20 @@ def sample(logits: torch.Tensor, temperature: float = 1.0, top_k: int = 0, top_p
     return out_ids
 
 
-def router_topk(logits: torch.Tensor, top_k: int, mode: str = "softmax_topk", bias: Optional[torch.Tensor] = None, *,
+ROUTER_MODES = {"softmax_topk": 0, "topk_softmax": 1, "sigmoid_topk": 2}
+
+
+def router_topk(logits, top_k: int, mode: str = "softmax_topk", bias: Optional[torch.Tensor] = None, *,
                 groups: int = 0, keep: int = 0, scale: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
     """MoE routing.  mode "softmax_topk": softmax over all experts, top-k, renormalise
-    (Qwen3); "topk_softmax": top-k raw logits, softmax over them (gpt-oss).  logits are bf16 /
-    fp32 ``[T, E]`` or fp32 split-K partials ``[S, T, E]`` (summed here); bias [E] is added first.
+    (Qwen3); "topk_softmax": top-k raw logits, softmax over them (gpt-oss); "sigmoid_topk": the top-k sigmoids as they
+    are.  logits are bf16 / fp32 ``[T, E]``, fp32 split-K partials ``[S, T, E]`` (summed here) or a `Proj` slice of
+    either; bias [E] is added first.
     groups > 0 (softmax_topk): experts form that many equal runs of neighbours and only those of the `keep` runs with
     the largest single score can be chosen.  The weights are multiplied by `scale`.
     Returns (weights fp32 [T, k], experts int32 [T, k])."""
+    if isinstance(logits, Proj):
+        logits = logits.t[..., logits.col:logits.col + logits.width]
     partial = logits.dim() == 3
     T, E = logits.shape[-2], logits.shape[-1]
     if not _native(logits):
@@ -722,6 +740,9 @@ def router_topk(logits: torch.Tensor, top_k: int, mode: str = "softmax_topk", bi
                 pick = p.masked_fill(~on.repeat_interleave(E // groups, dim=1), -1.0)
             w, e = pick.topk(top_k, dim=-1)
             w = w / (w.sum(-1, keepdim=True) + 1e-20)
+        elif mode == "sigmoid_topk":
+            v, e = lf.topk(top_k, dim=-1)
+            w = torch.sigmoid(v)
         else:
             v, e = lf.topk(top_k, dim=-1)
             w = torch.softmax(v, dim=-1)
@@ -730,12 +751,12 @@ def router_topk(logits: torch.Tensor, top_k: int, mode: str = "softmax_topk", bi
     w = torch.empty((T, top_k), dtype=torch.float32, device=logits.device)
     e = torch.empty((T, top_k), dtype=torch.int32, device=logits.device)
     is_fp32 = 1 if logits.dtype == torch.float32 else 0
-    if not logits.is_contiguous():
-        logits = logits.contiguous()
+    if logits.stride(-1) != 1:
+        raise ValueError("router logits need unit column stride")
     splits = logits.shape[0] if partial else 1
-    rc = _lib.lib().nkb_router_topk(logits.data_ptr(), is_fp32, splits, logits.stride(0) if partial else 0, _ptr(bias),
-                                    w.data_ptr(), e.data_ptr(), T, E, top_k, 0 if mode == "softmax_topk" else 1,
-                                    int(groups), int(keep), float(scale), _stream())
+    rc = _lib.lib().nkb_router_topk(logits.data_ptr(), is_fp32, splits, logits.stride(0) if partial else 0,
+                                    logits.stride(-2), _ptr(bias), w.data_ptr(), e.data_ptr(), T, E, top_k,
+                                    ROUTER_MODES[mode], int(groups), int(keep), float(scale), _stream())
     _lib.check(rc, "nkb_router_topk")
     _launches += 1
     return w, e
@@ -750,7 +771,7 @@ def _gather_kv(cache: torch.Tensor, table_row: torch.Tensor, ctx: int) -> torch.
     return blocks.permute(0, 2, 1, 3).reshape(nblk * bs, cache.shape[1], cache.shape[3])[:ctx]
 
 
-def _ref_attention(q, k, v, scale, q_pos0, causal, window, sinks):
+def _ref_attention(q, k, v, scale, q_pos0, causal, window, sinks, chunk=0):
     """q [Lq, nq, D], k/v [Lk, nkv, D] fp32 -> [Lq, nq, D]; query i sits at kv position q_pos0 + i."""
     Lq, nq, D = q.shape
     Lk, nkv, _ = k.shape
@@ -765,6 +786,8 @@ def _ref_attention(q, k, v, scale, q_pos0, causal, window, sinks):
         mask &= kpos <= qpos
     if window and window > 0:
         mask &= kpos > qpos - window
+    if chunk > 0:
+        mask &= kpos >= qpos - qpos % chunk
     s = s.masked_fill(~mask[None], float("-inf"))
     if sinks is not None:
         s = torch.cat([s, sinks.float()[:, None, None].expand(nq, Lq, 1)], dim=-1)
@@ -811,6 +834,7 @@ def paged_attn_decode(
     *,
     q_len: int = 1,
     window: int = 0,
+    chunk: int = 0,
     sinks: Optional[torch.Tensor] = None,
     num_splits: int = 0,
     scratch: Optional[torch.Tensor] = None,
@@ -818,7 +842,8 @@ def paged_attn_decode(
 ) -> torch.Tensor:
     """Decode attention over the paged cache.  q ``[B * q_len, nq * D]`` (the q_len
     newest tokens of each sequence, already appended to the cache);
-    context_lens counts them.  Causal among the new tokens."""
+    context_lens counts them.  Causal among the new tokens; window > 0: a query sees itself and the window - 1 tokens
+    before it; chunk > 0: only the positions of its own chunk of that many."""
     nkv, bs, D = k_cache.shape[1], k_cache.shape[2], k_cache.shape[3]
     B = block_table.shape[0]
     nq = q.shape[-1] // D
@@ -831,7 +856,7 @@ def paged_attn_decode(
             ctx = int(context_lens[b])
             k = _gather_kv(k_cache, block_table[b], ctx).float()
             v = _gather_kv(v_cache, block_table[b], ctx).float()
-            res[b] = _ref_attention(qf[b], k, v, scale, ctx - q_len, True, window, sinks)
+            res[b] = _ref_attention(qf[b], k, v, scale, ctx - q_len, True, window, sinks, chunk)
         out.copy_(res.reshape(out.shape).to(out.dtype))
         return out
     global _launches
@@ -842,7 +867,7 @@ def paged_attn_decode(
         q_start = torch.arange(B, device=q.device, dtype=torch.int32) * q_len
         q_lens = torch.full((B,), q_len, device=q.device, dtype=torch.int32)
         return flash_attn_prefill(q, k_cache, v_cache, block_table, q_start, q_lens, context_lens, scale,
-                                  max_q_len=q_len, causal=True, window=window, sinks=sinks, out=out)
+                                  max_q_len=q_len, causal=True, window=window, chunk=chunk, sinks=sinks, out=out)
     L = _lib.lib()
     if num_splits <= 0:
         num_splits = pick_kv_splits(B * nkv, block_table.shape[1])
@@ -853,7 +878,7 @@ def paged_attn_decode(
     rc = L.nkb_paged_attn_decode(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), context_lens.data_ptr(),
         out.data_ptr(), _ptr(scratch), B, q_len, nq, nkv, D, bs, k_cache.shape[0], block_table.stride(0),
-        float(scale), int(window), _ptr(sinks), num_splits, _stream(),
+        float(scale), int(window), int(chunk), _ptr(sinks), num_splits, _stream(),
     )
     _lib.check(rc, "nkb_paged_attn_decode")
     _launches += 1
@@ -949,6 +974,7 @@ def flash_attn_prefill(
     max_q_len: int,
     causal: bool = True,
     window: int = 0,
+    chunk: int = 0,
     sinks: Optional[torch.Tensor] = None,
     out: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
@@ -971,7 +997,7 @@ def flash_attn_prefill(
                 continue
             k = _gather_kv(k_cache, block_table[b], ctx).float()
             v = _gather_kv(v_cache, block_table[b], ctx).float()
-            res[qs:qs + ql] = _ref_attention(qf[qs:qs + ql], k, v, scale, ctx - ql, causal, window, sinks)
+            res[qs:qs + ql] = _ref_attention(qf[qs:qs + ql], k, v, scale, ctx - ql, causal, window, sinks, chunk)
         out.copy_(res.reshape(out.shape).to(out.dtype))
         return out
     global _launches
@@ -979,7 +1005,7 @@ def flash_attn_prefill(
     rc = _lib.lib().nkb_flash_attn_prefill(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), q_start.data_ptr(),
         q_lens.data_ptr(), context_lens.data_ptr(), out.data_ptr(), B, total_q, int(max_q_len), nq, nkv, D, bs,
-        k_cache.shape[0], block_table.stride(0), float(scale), 1 if causal else 0, int(window), _ptr(sinks),
+        k_cache.shape[0], block_table.stride(0), float(scale), 1 if causal else 0, int(window), int(chunk), _ptr(sinks),
         _stream(),
     )
     _lib.check(rc, "nkb_flash_attn_prefill")
@@ -1007,9 +1033,11 @@ def moe_tile_widths(tokens: int):
     return 64, 128
 
 
-def moe_dispatch(x: torch.Tensor, experts: torch.Tensor, expert_lo: int, num_local: int, gather: bool = True) -> MoEPlan:
+def moe_dispatch(x: torch.Tensor, experts: torch.Tensor, expert_lo: int, num_local: int, gather: bool = True,
+                 weights: Optional[torch.Tensor] = None) -> MoEPlan:
     """Sort the (token, expert) pairs routed to local experts [expert_lo, expert_lo + num_local) by
-    expert and gather their token rows.  x [T, H] bf16, experts [T, k] int32 (global ids).
+    expert and gather their token rows.  x [T, H] bf16 or fp32, experts [T, k] int32 (global ids); weights [T, k] fp32:
+    gathered rows are multiplied by their pair's weight.
     Returns a `MoEPlan` (unpacks to x_sorted [T * k, H], offsets int32 [num_local + 1], pair_pos int32
     [T * k]); rows past offsets[-1] of x_sorted are unspecified, pair_pos is -1 for pairs of other
     ranks' experts.  gather False: x_sorted is x itself and `row_token` names the token of every sorted row (any type and
@@ -1033,13 +1061,17 @@ def moe_dispatch(x: torch.Tensor, experts: torch.Tensor, expert_lo: int, num_loc
         if not gather:
             return MoEPlan(x, offsets, pair_pos, None, T, row_token)
         x_sorted = torch.zeros((pairs, H), dtype=x.dtype)
-        x_sorted[:n_local] = x[(order[:n_local] // k)]
+        rows = x[(order[:n_local] // k)]
+        x_sorted[:n_local] = rows if weights is None else (rows.float() * weights.reshape(-1)[order[:n_local], None]).to(x.dtype)
         return MoEPlan(x_sorted, offsets, pair_pos, None, T, row_token)
     global _launches
     bn_a, bn_b = moe_tile_widths(T)
     cap_a, cap_b = num_local + pairs // bn_a + 1, num_local + pairs // bn_b + 1
+    if weights is not None and (not gather or weights.dtype != torch.float32 or not weights.is_contiguous()):
+        raise ValueError("weights are contiguous fp32 and scale gathered rows")
     if gather:
-        _check_bf16(x)
+        if not x.is_contiguous() or x.dtype not in (torch.bfloat16, torch.float32):
+            raise TypeError("gathered rows are contiguous bf16 or fp32")
         x_sorted = torch.empty((pairs, H), dtype=x.dtype, device=dev)
         row_token = None
     else:
@@ -1057,7 +1089,8 @@ def moe_dispatch(x: torch.Tensor, experts: torch.Tensor, expert_lo: int, num_loc
     if experts.dtype != torch.int32:
         experts = experts.to(torch.int32)
     rc = _lib.lib().nkb_moe_dispatch(experts.data_ptr(), T, k, int(expert_lo), int(num_local),
-                                     x.data_ptr() if gather else None, H, x_sorted.data_ptr(), counts.data_ptr(),
+                                     x.data_ptr() if gather else None, 1 if x.dtype == torch.float32 else 0, H,
+                                     _ptr(weights), x_sorted.data_ptr(), counts.data_ptr(),
                                      offsets.data_ptr(), cursors.data_ptr(), pair_pos.data_ptr(), _ptr(row_token), bn_a, tiles_a.data_ptr(), ntiles.data_ptr(), bn_b,
                                      tiles_b.data_ptr(), ntiles.data_ptr() + 4, _stream())
     _lib.check(rc, "nkb_moe_dispatch")
@@ -1078,7 +1111,8 @@ def grouped_linear(x_sorted: torch.Tensor, w: torch.Tensor, offsets: torch.Tenso
     G = w.shape[0]
     N = w.shape[1] // 2 if gated else w.shape[1]
     if not _native(x_sorted):
-        out = torch.zeros((R, N), dtype=torch.bfloat16)
+        if out is None:
+            out = torch.zeros((R, N), dtype=torch.bfloat16)
         off = offsets.tolist()
         for g in range(G):
             a, b = off[g], off[g + 1]
@@ -1114,7 +1148,7 @@ def grouped_linear(x_sorted: torch.Tensor, w: torch.Tensor, offsets: torch.Tenso
             block_n = 128
     rc = _lib.lib().nkb_gemm_bf16_grouped(
         w.data_ptr(), x_sorted.data_ptr(), out.data_ptr(), offsets.data_ptr(), G, N, K, R, int(max_rows_per_group),
-        x_sorted.stride(0), N, 1 if gated else 0, N if gated else 0, _ptr(bias),
+        x_sorted.stride(0), out.stride(0), 1 if gated else 0, N if gated else 0, _ptr(bias),
         bias.stride(0) if bias is not None else 0, float(act_limit), float(act_alpha), block_n, tl, tc,
         int(max_tiles), arrive, int(arrive_target), _stream())
     _lib.check(rc, "nkb_gemm_bf16_grouped")
@@ -1145,6 +1179,35 @@ def grouped_linear_simt(plan: MoEPlan, x: torch.Tensor, w: torch.Tensor, sorted_
     return out
 
 
+_HEAD_OFFSETS = {}
+
+
+def head_linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``x[h] @ w[h].T`` for every head: x [H, T, K], w [H, N, K] -> [H, T, N] in x's type; out: a [H, T, N] view whose heads
+    follow one another (rows may be wider than N)."""
+    H, T, K = x.shape
+    N = w.shape[1]
+    if out is None:
+        out = torch.empty((H, T, N), dtype=x.dtype, device=x.device)
+    if not _native(x):
+        return out.copy_(torch.einsum("htk,hnk->htn", x.float(), w.float()).to(out.dtype))
+    if not x.is_contiguous() or not w.is_contiguous() or out.stride(2) != 1 or out.stride(0) != T * out.stride(1):
+        raise ValueError("head_linear wants contiguous operands and heads that follow one another")
+    key = (x.device, H, T)
+    if key not in _HEAD_OFFSETS:
+        _HEAD_OFFSETS[key] = torch.arange(0, H * T + 1, T, dtype=torch.int32, device=x.device)
+    offsets, rows = _HEAD_OFFSETS[key], out.as_strided((H * T, N), (out.stride(1), 1))
+    if x.dtype == torch.bfloat16 and K % 8 == 0:
+        grouped_linear(x.reshape(H * T, K), w, offsets, max_rows_per_group=T, out=rows)
+        return out
+    bf = 1 if x.dtype == torch.bfloat16 else 0
+    rc = _lib.lib().nkb_gemm_simt_grouped(x.data_ptr(), bf, w.data_ptr(), bf, out.data_ptr(), bf, offsets.data_ptr(), None, H,
+                                          T, N, K, K, out.stride(1), _stream())
+    _lib.check(rc, "nkb_gemm_simt_grouped")
+    _count_launch()
+    return out
+
+
 def moe_combine(y_sorted: torch.Tensor, pair_pos: torch.Tensor, weights: torch.Tensor, tokens: int) -> torch.Tensor:
     """``out[t] = sum_j weights[t, j] * y_sorted[pair_pos[t * k + j]]`` over local pairs -> bf16 [T, H]."""
     k = weights.shape[1]
@@ -1166,6 +1229,8 @@ def moe_combine(y_sorted: torch.Tensor, pair_pos: torch.Tensor, weights: torch.T
 
 
 from . import mixers  # noqa: E402  (uses the helpers above)
-from .mixers import (Branch, MapsSpec, Proj, activation, gate_heads, gated_act, gated_residual,  # noqa: E402,F401
-                     heads_attention, hgrn2, maps_append, maps_attention, row_norm_append)
+from .mixers import (Branch, MapsSpec, Norm, Proj, activation, gate_heads, gated_act, gated_residual,  # noqa: E402,F401
+                     heads_attention, hgrn2, maps_append, maps_attention, rope_norm_append, row_norm_append)
+from .latent_attention import (LatentSpec, latent_append, latent_attention, latent_gather,  # noqa: E402,F401
+                               latent_queries)
 from .linear_attention import Decay, linear_attention, low_rank, token_mix  # noqa: E402,F401

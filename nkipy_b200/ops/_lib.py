@@ -30,13 +30,22 @@ class ProjArg(ctypes.Structure):
 class MapsArg(ctypes.Structure):
     """Sizes and constants of attention with several score maps (csrc/kernels/attn_maps.h)."""
     _fields_ = [(n, c_int) for n in ("maps", "heads", "kv_heads", "dim", "dim_p", "vdim", "vdim_p")] + \
-               [(n, c_float) for n in ("scale", "softcap", "lam", "out_scale", "eps")] + [("window", c_int)]
+               [(n, c_float) for n in ("scale", "softcap", "lam", "out_scale", "eps")] + \
+               [("window", c_int), ("chunk", c_int), ("sinks", c_void_p)] + \
+               [(n, c_longlong) for n in ("q_token", "q_head", "o_token", "o_head")] + [("v_ld", c_int)]
+
+
+class LatentArg(ctypes.Structure):
+    """Sizes and constants of latent attention (csrc/kernels/latent_attn.h)."""
+    _fields_ = [(n, c_int) for n in ("heads", "dim", "rot", "rank", "q_rank", "row")] + \
+               [("eps", c_float), ("scale", c_float), ("window", c_int), ("sinks", c_void_p)] + \
+               [(n, c_longlong) for n in ("q_token", "q_head", "o_token", "o_head")]
 
 
 class BranchArg(ctypes.Structure):
     """One addend of a residual update (csrc/kernels/proj_src.h)."""
     _fields_ = [("y", ProjArg), ("g", ProjArg), ("gbias", c_void_p), ("pair_pos", c_void_p), ("pair_w", c_void_p),
-                ("top_k", c_int), ("scale", c_float)]
+                ("norm_w", c_void_p), ("top_k", c_int), ("token_gate", c_int), ("scale", c_float)]
 
 
 class LinAttnArg(ctypes.Structure):
@@ -51,6 +60,7 @@ class LinAttnArg(ctypes.Structure):
 
 _PP = ctypes.POINTER(ProjArg)
 _PM = ctypes.POINTER(MapsArg)
+_PL = ctypes.POINTER(LatentArg)
 _SIGNATURES = {
     "nkb_init": (c_int, []),
     "nkb_status": (c_int, [c_int]),
@@ -70,13 +80,21 @@ _SIGNATURES = {
     "nkb_linattn_step": (c_int, [ctypes.POINTER(LinAttnArg), _P]),
     "nkb_low_rank": (c_int, [_PP, c_int, _P, c_int, _P, c_int, c_int, c_int, _P]),
     "nkb_token_mix": (c_int, [_P, c_int, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P]),
-    "nkb_gate_heads": (c_int, [_P, c_int, c_longlong, c_longlong, _PP, c_int, _P, c_int, c_float, c_float, _P, c_int,
+    "nkb_gate_heads": (c_int, [_P, c_int, c_longlong, c_longlong, _PP, c_int, c_int, _P, c_int, c_float, c_float, _P, c_int,
                                c_longlong, c_int, c_int, c_int, _P]),
     "nkb_row_norm_append": (c_int, [_PM, _PP, _PP, _PP, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P]),
+    "nkb_rope_norm_append": (c_int, [_PM, _PP, _PP, _PP, _P, _P, c_int, c_int, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int,
+                                     _P]),
+    "nkb_latent_append": (c_int, [_PL, _PP, _PP, _P, _P, _P, c_int, _P, _P, _P, _P, c_int, c_int, c_int, _P]),
+    "nkb_latent_queries": (c_int, [_PL, _PP, _P, c_int, _P, _P, c_longlong, c_longlong, c_int, _P, c_longlong, c_longlong,
+                                   c_int, c_int, c_int, _P]),
+    "nkb_latent_gather": (c_int, [_P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, c_int, _P]),
+    "nkb_latent_scratch_floats": (c_longlong, [_PL, c_int, c_int]),
+    "nkb_latent_attn": (c_int, [_PL, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
     "nkb_gated_residual": (c_int, [_P, _P, _P, c_int, c_int, c_float, c_int, ctypes.POINTER(BranchArg), _P, _P, _P,
-                                   c_int, ctypes.POINTER(_P), ctypes.POINTER(_P), c_int, c_int, c_int, c_int, c_float,
-                                   _P]),
-    "nkb_gated_act": (c_int, [_PP, _PP, _P, c_int, c_int, c_int, c_int, _P]),
+                                   c_int, c_int, ctypes.POINTER(_P), ctypes.POINTER(_P), ctypes.POINTER(_P), c_int, c_int,
+                                   c_int, c_int, c_float, _P]),
+    "nkb_gated_act": (c_int, [_PP, _PP, _P, c_int, c_int, c_int, c_int, c_float, c_float, _P, c_int, _P]),
     "nkb_hgrn2_scan_scratch": (c_longlong, [c_int, c_int, c_int]),
     "nkb_hgrn2_scan": (c_int, [_PP, _PP, _PP, _P, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
                                _P, c_float, _P]),
@@ -100,7 +118,7 @@ _SIGNATURES = {
     "nkb_moe_a2a_combine": (c_int, [_P, _P, c_int, c_int, c_int, c_int, c_int, ctypes.c_uint, ctypes.POINTER(_P),
                                     ctypes.POINTER(_P), ctypes.POINTER(_P), ctypes.POINTER(_P), ctypes.POINTER(_P),
                                     ctypes.POINTER(_P), _P, _P]),
-    "nkb_moe_dispatch": (c_int, [_P, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, _P, _P, _P, _P, c_int, _P, _P,
+    "nkb_moe_dispatch": (c_int, [_P, c_int, c_int, c_int, c_int, _P, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, c_int, _P, _P,
                                  c_int, _P, _P, _P]),
     "nkb_moe_combine": (c_int, [_P, _P, _P, c_int, c_int, c_int, _P, _P]),
     "nkb_gemm_effective_splits": (c_int, [c_int, c_int]),
@@ -135,12 +153,13 @@ _SIGNATURES = {
     "nkb_argmax": (c_int, [_P, c_int, _P, _P, c_int, c_int, c_longlong, _P]),
     "nkb_sample": (c_int, [_P, c_int, _P, c_int, c_int, c_longlong, c_float, c_int, c_float, c_ulonglong,
                            c_ulonglong, _P]),
-    "nkb_router_topk": (c_int, [_P, c_int, c_int, c_longlong, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
+    "nkb_softcap": (c_int, [_P, c_longlong, c_float, _P]),
+    "nkb_router_topk": (c_int, [_P, c_int, c_int, c_longlong, c_longlong, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
                                 c_float, _P]),
     "nkb_paged_attn_decode": (
         c_int,
-        [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P,
-         c_int, _P],
+        [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
+         _P, c_int, _P],
     ),
     "nkb_paged_attn_decode_fused": (
         c_int,
@@ -151,7 +170,7 @@ _SIGNATURES = {
     "nkb_flash_attn_prefill": (
         c_int,
         [_P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-         c_int, c_int, _P, _P],
+         c_int, c_int, c_int, _P, _P],
     ),
 }
 

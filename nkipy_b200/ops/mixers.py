@@ -1,14 +1,16 @@
 """Operators of decoders whose layers mix attention and linear recurrences around an fp32 residual stream.
 
-    gated_residual   embedding or residual + branches (gated, scaled or routed; + additions ahead of a repeated block),
-                     and the group-wise RMS norms of the sum, in one launch
-    gated_act        act(gate) * up; `activation` for act(x) alone
-    gate_heads       scale * act(gate) * norm(head), the norm optional
+    gated_residual   embedding or residual + branches (gated, scaled, routed or normed; + additions ahead of a repeated
+                     block), and the norms of the sum (group-wise RMS, layer norm, or a copy), in one launch
+    gated_act        act(gate) * up, also with clamped operands or rows of a table as up; `activation` for act(x) alone
+    gate_heads       scale * act(gate) * norm(head), the norm optional, one gate per element or per head
     hgrn2            linear attention with a per-channel forget gate; state in slots, fp32
     row_norm_append  queries and keys normed over all their heads, paged-cache append
+    rope_norm_append biases, half-split partial RoPE and per-head norm of queries and keys, paged-cache append
     maps_append      interleaved partial RoPE of queries / keys with several score maps, paged-cache append
     heads_attention  attention with several score maps over shared values (differential attention), score soft cap;
-                     with one map plain grouped-query attention, also through a sliding window
+                     with one map plain grouped-query attention, also through a sliding window, inside chunks and
+                     with sinks
     linear_simt      products on the CUDA cores: 32-bit models, operands TMA cannot describe
 
 All of them take the projections they consume as `Proj` slices, so a decode-sized batch hands over split-K partial
@@ -34,6 +36,7 @@ from . import (_count_launch, _decode_scratch, _gather_kv, _native, _ptr, _strea
 ACTIVATIONS = {"silu": (0, F.silu), "gelu_tanh": (1, lambda z: F.gelu(z, approximate="tanh")),
                "relu2": (2, lambda z: F.relu(z).square()), "tanh": (3, torch.tanh), "sigmoid": (4, torch.sigmoid),
                "none": (5, lambda z: z)}
+CLAMPED = 6                  # of a gate and up pair (`gated_act`)
 
 
 class Proj(NamedTuple):
@@ -57,32 +60,66 @@ class Proj(NamedTuple):
 
 
 class Branch(NamedTuple):
-    """One addend of a residual update: scale * y; with gate and bias, sigmoid(gate + bias) * y; with pair_pos [T * k] and
-    pair_w [T, k], scale * sum_j pair_w[t, j] * y[pair_pos[t * k + j]] (routed experts)."""
+    """One addend of a residual update: scale * y; with gate and bias, sigmoid(gate + bias) * y; with a gate of one column and no
+    bias, scale * sigmoid(gate) * y; with pair_pos [T * k] and pair_w [T, k] (None with top_k = k: ones),
+    scale * sum_j pair_w[t, j] * y[pair_pos[t * k + j]] (routed experts); with norm, scale * norm * y / sqrt(mean(y^2) + eps)."""
     y: Proj
     gate: Optional[Proj] = None
     bias: Optional[torch.Tensor] = None
     scale: float = 1.0
     pair_pos: Optional[torch.Tensor] = None
     pair_w: Optional[torch.Tensor] = None
+    top_k: int = 0
+    norm: Optional[torch.Tensor] = None
 
-    def value(self) -> torch.Tensor:
+    @property
+    def chosen(self) -> int:
+        return self.top_k if self.pair_w is None else self.pair_w.shape[1]
+
+    def value(self, eps: float) -> torch.Tensor:
         if self.pair_pos is not None:
-            T, k = self.pair_w.shape
-            rows = self.y.value()[self.pair_pos.reshape(T, k).long().clamp(min=0)]
-            w = self.pair_w * (self.pair_pos.reshape(T, k) >= 0)
+            pos = self.pair_pos.reshape(-1, self.chosen)
+            rows = self.y.value()[pos.long().clamp(min=0)]
+            w = (pos >= 0) if self.pair_w is None else self.pair_w * (pos >= 0)
             return self.scale * (rows * w[..., None]).sum(1)
+        y = self.y.value()
+        if self.norm is not None:
+            return self.scale * y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps) * self.norm
         if self.gate is not None:
-            return self.y.value() * torch.sigmoid(self.gate.value() + self.bias)
-        return self.scale * self.y.value()
+            g = self.gate.value()
+            return self.scale * y * torch.sigmoid(g if self.bias is None else g + self.bias)
+        return self.scale * y
 
     def arg(self) -> _lib.BranchArg:
         none = _lib.ProjArg(None, 0, 0, 1, 0)
-        if self.gate is not None and (self.scale != 1.0 or self.pair_pos is not None):
-            raise ValueError("a gated branch has neither a scale nor routed rows")
+        token_gate = self.gate is not None and self.bias is None
+        if token_gate and self.gate.width != 1:
+            raise ValueError("a gate without bias has one column")
+        if self.gate is not None and (self.pair_pos is not None or self.norm is not None or (not token_gate and self.scale != 1.0)):
+            raise ValueError("a gated branch has neither routed rows nor a norm, and a scale only with one gate per token")
         return _lib.BranchArg(self.y.arg(), none if self.gate is None else self.gate.arg(), _ptr(self.bias),
-                              _ptr(self.pair_pos), _ptr(self.pair_w), 0 if self.pair_w is None else self.pair_w.shape[1],
-                              float(self.scale))
+                              _ptr(self.pair_pos), _ptr(self.pair_w), _ptr(self.norm),
+                              0 if self.pair_pos is None else self.chosen, 1 if token_gate else 0, float(self.scale))
+
+
+class Norm(NamedTuple):
+    """What reads the residual: its RMS norm with a weight (a bare tensor means the same), with center its layer norm with
+    weight and bias, without a weight the residual itself."""
+    weight: Optional[torch.Tensor] = None
+    bias: Optional[torch.Tensor] = None
+    center: bool = False
+
+    @property
+    def kind(self) -> int:
+        return 2 if self.weight is None else (1 if self.center else 0)
+
+    def value(self, x: torch.Tensor, groups: int, eps: float) -> torch.Tensor:
+        if self.weight is None:
+            return x
+        if self.center:
+            d = x - x.mean(-1, keepdim=True)
+            return d / torch.sqrt(d.pow(2).mean(-1, keepdim=True) + eps) * self.weight + self.bias
+        return group_rmsnorm_ref(x, self.weight, groups, eps)
 
 
 def _ref(p: Proj):
@@ -120,16 +157,19 @@ def group_rmsnorm_ref(x: torch.Tensor, w: torch.Tensor, groups: int, eps: float)
 def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Branch] = (), *,
                    ids: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None, scale: float = 1.0,
                    add_mat: Optional[torch.Tensor] = None, add_row: Optional[torch.Tensor] = None,
-                   norms: Sequence[torch.Tensor] = (), groups: int = 1, eps: float = 1e-6,
+                   norms: Sequence = (), groups: int = 1, eps: float = 1e-6,
                    dtype: torch.dtype = torch.bfloat16) -> Tuple[torch.Tensor, List[torch.Tensor]]:
     """One residual update of an fp32 stream and the norms that read it.
 
         r = x  (or table[ids] * scale)
         r += sum over branches (see `Branch`);   r += add_mat;   r += add_row
-        h_j = w_j * (r divided, in `groups` equal parts, by sqrt(mean(part^2) + eps))
+        h_j = w_j * (r divided, in `groups` equal parts, by sqrt(mean(part^2) + eps)), or as `Norm` says (one kind per call)
 
     x [T, W] fp32; gate biases, add_row and the norm weights fp32 [W]; add_mat fp32 [T, W].  Returns (r, [h_j in `dtype`])."""
     branches = [b if isinstance(b, Branch) else Branch(*b) for b in branches]
+    norms = [n if isinstance(n, Norm) else Norm(n) for n in norms]
+    if len({n.kind for n in norms}) > 1:
+        raise ValueError("the norms of one residual update are of one kind")
     if x is not None:
         rows, width = x.shape
         dev = x.device
@@ -141,38 +181,47 @@ def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Branch] = (), *
     if not _native(r):
         acc = x.clone() if x is not None else table[ids.long().clamp(0, table.shape[0] - 1)].float() * scale
         if branches:
-            acc = acc + sum(b.value() for b in branches)
+            acc = acc + sum(b.value(eps) for b in branches)
         if add_mat is not None:
             acc = acc + add_mat
         if add_row is not None:
             acc = acc + add_row
         r.copy_(acc)
-        for o, w in zip(outs, norms):
-            o.copy_(group_rmsnorm_ref(acc, w, groups, eps).to(dtype))
+        for o, n in zip(outs, norms):
+            o.copy_(n.value(acc, groups, eps).to(dtype))
         return r, outs
-    for t in [x, add_mat, add_row, *norms, *[b.bias for b in branches]]:
+    weights, biases = [n.weight for n in norms], [n.bias for n in norms]
+    for t in [x, add_mat, add_row, *weights, *biases, *[b.bias for b in branches], *[b.norm for b in branches]]:
         if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
             raise TypeError("gated_residual wants contiguous fp32 residuals, biases and norm weights")
     n = len(branches)
-    ba = (_lib.BranchArg * 2)(*[b.arg() for b in branches])
+    ba = (_lib.BranchArg * max(n, 1))(*[b.arg() for b in branches])
     rc = _lib.lib().nkb_gated_residual(
         _ptr(x), _ptr(ids), _ptr(table), 1 if table is not None and table.dtype == torch.bfloat16 else 0,
-        table.shape[0] if table is not None else 0, float(scale), n, ba, _ptr(add_row), _ptr(add_mat), r.data_ptr(), len(outs), _ptr_array(list(norms)), _ptr_array(outs),
-        1 if dtype == torch.bfloat16 else 0, rows, width, int(groups), float(eps), _stream())
+        table.shape[0] if table is not None else 0, float(scale), n, ba, _ptr(add_row), _ptr(add_mat), r.data_ptr(), len(outs),
+        norms[0].kind if norms else 0, _ptr_array(weights), _ptr_array(biases), _ptr_array(outs), 1 if dtype == torch.bfloat16 else 0, rows, width, int(groups), float(eps), _stream())
     _lib.check(rc, "nkb_gated_residual")
     _count_launch()
     return r, outs
 
 
-def gated_act(gate: Proj, up: Proj, act: str = "silu", dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
-    """``act(gate) * up`` -> [T, width] in `dtype`."""
+def gated_act(gate: Proj, up: Proj, act: str = "silu", dtype: torch.dtype = torch.bfloat16, *, limit: float = 0.0,
+              alpha: float = 1.702, up_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``act(gate) * up`` -> [T, width] in `dtype`; act "clamped": ``g * sigmoid(alpha * g) * (u + 1)`` with gate at most `limit`
+    and up within +-limit.  up_rows [T] int32: up is a table, of which token t takes row up_rows[t]."""
     rows = gate.t.shape[-2]
     out = torch.empty((rows, gate.width), dtype=dtype, device=gate.t.device)
     if not _native(out):
-        out.copy_((ACTIVATIONS[act][1](gate.value()) * up.value()).to(dtype))
-        return out
+        g, u = gate.value(), up.value()
+        if up_rows is not None:
+            u = u[up_rows.long().clamp(0, u.shape[0] - 1)]
+        if act == "clamped":
+            g = g.clamp(max=limit)
+            return out.copy_((g * torch.sigmoid(alpha * g) * (u.clamp(-limit, limit) + 1)).to(dtype))
+        return out.copy_((ACTIVATIONS[act][1](g) * u).to(dtype))
+    kind = CLAMPED if act == "clamped" else ACTIVATIONS[act][0]
     rc = _lib.lib().nkb_gated_act(_ref(gate), _ref(up), out.data_ptr(), 1 if dtype == torch.bfloat16 else 0, rows,
-                                  gate.width, ACTIVATIONS[act][0], _stream())
+                                  gate.width, kind, float(limit), float(alpha), _ptr(up_rows), up.t.shape[-2], _stream())
     _lib.check(rc, "nkb_gated_act")
     _count_launch()
     return out
@@ -187,7 +236,7 @@ def activation(x: Proj, act: str, dtype: torch.dtype = torch.bfloat16) -> torch.
         return out
     none = _lib.ProjArg(None, 0, 0, 1, 0)
     rc = _lib.lib().nkb_gated_act(_ref(x), ctypes.byref(none), out.data_ptr(), 1 if dtype == torch.bfloat16 else 0, rows,
-                                  x.width, ACTIVATIONS[act][0], _stream())
+                                  x.width, ACTIVATIONS[act][0], 0.0, 0.0, None, 0, _stream())
     _lib.check(rc, "nkb_gated_act")
     _count_launch()
     return out
@@ -195,7 +244,8 @@ def activation(x: Proj, act: str, dtype: torch.dtype = torch.bfloat16) -> torch.
 
 def gate_heads(x: torch.Tensor, gate: Proj, act: str, *, norm_w: Optional[torch.Tensor] = None, eps: float = 1e-6,
                scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """``scale * act(gate) * x`` for heads x [T, H, n] (any strides of tokens and heads); with norm_w (fp32, [n] shared by the
+    """``scale * act(gate) * x`` for heads x [T, H, n] (any strides of tokens and heads), gate [T, H * n] or, one per head,
+    [T, H]; with norm_w (fp32, [n] shared by the
     heads or [H * n]) every head is first divided by its root mean square and multiplied by the weight.  Returns
     [T, H * n], written to `out` (a slice of columns) when given."""
     T, H, n = x.shape
@@ -205,14 +255,17 @@ def gate_heads(x: torch.Tensor, gate: Proj, act: str, *, norm_w: Optional[torch.
         y = x.float()
         if norm_w is not None:
             y = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float().reshape(-1, n)
-        out.copy_((scale * ACTIVATIONS[act][1](gate.value()) * y.reshape(T, H * n)).to(out.dtype))
+        g = ACTIVATIONS[act][1](gate.value()).reshape(T, H, -1)
+        out.copy_((scale * g * y).reshape(T, H * n).to(out.dtype))
         return out
     if x.stride(2) != 1 or out.stride(1) != 1 or x.dtype != out.dtype:
         raise ValueError("gate_heads wants unit column strides and one type")
+    if gate.width not in (H, H * n):
+        raise ValueError("one gate per element or per head")
     stride = 0 if norm_w is None or norm_w.numel() == n else n
     rc = _lib.lib().nkb_gate_heads(
-        x.data_ptr(), 1 if x.dtype == torch.bfloat16 else 0, x.stride(0), x.stride(1), _ref(gate), ACTIVATIONS[act][0],
-        _ptr(norm_w), stride, float(eps), float(scale), out.data_ptr(), 1 if out.dtype == torch.bfloat16 else 0,
+        x.data_ptr(), 1 if x.dtype == torch.bfloat16 else 0, x.stride(0), x.stride(1), _ref(gate),
+        1 if gate.width == H and n > 1 else 0, ACTIVATIONS[act][0], _ptr(norm_w), stride, float(eps), float(scale), out.data_ptr(), 1 if out.dtype == torch.bfloat16 else 0,
         out.stride(0), T, H, n, _stream())
     _lib.check(rc, "nkb_gate_heads")
     _count_launch()
@@ -303,7 +356,7 @@ class MapsSpec:
     dim_p / vdim_p are the padded sizes of queries / keys (per map) and values in the cache; the tiled bf16 kernels
     take 32 or 64 and 64 or 128, other sizes are only rounded to even and use the general kernel.  With one map the tiled
     kernels are those of plain attention, which take one size of 64 or 128 for both.  window > 0 (one map): a query sees
-    itself and the window - 1 tokens before it."""
+    itself and the window - 1 tokens before it.  chunk > 0 (one map): it sees the tokens of its own chunk of that many positions."""
     heads: int
     kv_heads: int
     dim: int
@@ -316,6 +369,7 @@ class MapsSpec:
     eps: float = 1e-6
     tiled: bool = True
     window: int = 0
+    chunk: int = 0
 
     @property
     def plain(self) -> bool:
@@ -337,7 +391,7 @@ class MapsSpec:
     def arg(self) -> _lib.MapsArg:
         return _lib.MapsArg(self.maps, self.heads, self.kv_heads, self.dim, self.dim_p, self.vdim, self.vdim_p,
                             float(self.scale), float(self.softcap), float(self.lam), float(self.out_scale),
-                            float(self.eps), int(self.window))
+                            float(self.eps), int(self.window), int(self.chunk), None, 0, 0, 0, 0, 0)
 
 
 def row_norm_append(spec: MapsSpec, q: Proj, k: Proj, v: Proj, q_norm: torch.Tensor, k_norm: torch.Tensor,
@@ -368,6 +422,55 @@ def row_norm_append(spec: MapsSpec, q: Proj, k: Proj, v: Proj, q_norm: torch.Ten
                                         slots.data_ptr(), q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
                                         1 if k_cache.dtype == torch.bfloat16 else 0, T, bs, _stream())
     _lib.check(rc, "nkb_row_norm_append")
+    _count_launch()
+    return q_out
+
+
+def half_rotate(x: torch.Tensor, cos_sin: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+    """x [T, n, d] fp32 with the first cos_sin.shape[1] dimensions rotated, dimension i paired with i + half."""
+    n = cos_sin.shape[1] // 2
+    cs = cos_sin[positions.long().clamp(0, cos_sin.shape[0] - 1)]
+    c, s = cs[:, None, :n], cs[:, None, n:]
+    u, v = x[..., :n], x[..., n:2 * n]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * n:]], -1)
+
+
+def rope_norm_append(spec: MapsSpec, q: Proj, k: Optional[Proj], v: Optional[Proj], bias: Optional[torch.Tensor],
+                     cos_sin: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, k_cache: torch.Tensor,
+                     v_cache: torch.Tensor, norm: bool = True) -> torch.Tensor:
+    """Add the biases (fp32 [q | k | v]), rotate the first cos_sin.shape[1] dimensions of every head of queries and keys (dimension
+    i paired with i + half), with `norm` divide every head by sqrt(mean(head^2) + spec.eps), write keys and values to their
+    cache slots (negative slot: not stored) and return the queries [T, heads, dim_p].  k and v None: only the queries."""
+    T = q.t.shape[-2]
+    H, G, d, dp = spec.heads, spec.kv_heads, spec.dim, spec.dim_p
+    bs = k_cache.shape[2]
+    q_out = torch.empty((T, H, dp), dtype=k_cache.dtype, device=k_cache.device)
+    if not _native(k_cache):
+        def head(x, n, first):
+            x = x.value() if bias is None else x.value() + bias[first:first + x.width]
+            x = half_rotate(x.reshape(T, n, d), cos_sin, positions)
+            if norm:
+                x = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + spec.eps)
+            return F.pad(x, (0, dp - d)).to(k_cache.dtype)
+
+        q_out.copy_(head(q, H, 0))
+        if k is not None:
+            sl = slots.long()
+            keep = sl >= 0
+            blk, off = sl[keep] // bs, sl[keep] % bs
+            k_cache[blk, :, off] = head(k, G, q.width)[keep]
+            x = v.value() if bias is None else v.value() + bias[q.width + k.width:]
+            v_cache[blk, :, off] = F.pad(x.reshape(T, G, spec.vdim), (0, spec.vdim_p - spec.vdim))[keep].to(v_cache.dtype)
+        return q_out
+    for t in (bias, cos_sin):
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
+            raise TypeError("rope_norm_append wants fp32 biases and angles")
+    a, none = spec.arg(), ctypes.byref(_lib.ProjArg(None, 0, 0, 1, 0))
+    rc = _lib.lib().nkb_rope_norm_append(
+        ctypes.byref(a), _ref(q), none if k is None else _ref(k), none if v is None else _ref(v), _ptr(bias),
+        cos_sin.data_ptr(), cos_sin.shape[1], cos_sin.shape[0], positions.data_ptr(), slots.data_ptr(), 1 if norm else 0,
+        q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), 1 if k_cache.dtype == torch.bfloat16 else 0, T, bs, _stream())
+    _lib.check(rc, "nkb_rope_norm_append")
     _count_launch()
     return q_out
 
@@ -415,23 +518,25 @@ def maps_attention(*args, **kw) -> torch.Tensor:
 
 def heads_attention(spec: MapsSpec, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                    block_table: torch.Tensor, context_lens: torch.Tensor, *, q_start: Optional[torch.Tensor] = None,
-                   q_lens: Optional[torch.Tensor] = None, max_q_len: int = 1, num_splits: int = 0) -> torch.Tensor:
+                   q_lens: Optional[torch.Tensor] = None, max_q_len: int = 1, num_splits: int = 0,
+                   sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of the new tokens over the paged cache (which already holds them); returns the combined heads
-    [T, heads, vdim] (strided when the cache's values are padded).  q_lens None: one new token per sequence (decode); otherwise sequence b owns rows
+    [T, heads, vdim] (strided when the cache's values are padded).  sinks [heads] fp32: logarithms of an addend of every
+    softmax's denominator.  q_lens None: one new token per sequence (decode); otherwise sequence b owns rows
     q_start[b] .. q_start[b] + q_lens[b], the last of which sits at position context_lens[b] - 1."""
     T, H = q.shape[0], spec.heads
     bs = k_cache.shape[2]
     B = block_table.shape[0]
-    if spec.window > 0 and spec.maps != 1:
-        raise ValueError("a sliding window is for one score map")
+    if (spec.window > 0 or spec.chunk > 0 or sinks is not None) and spec.maps != 1:
+        raise ValueError("windows, chunks and sinks are for one score map")
     if _native(k_cache) and spec.plain:
         qf = q.reshape(T, -1)
         if q_lens is None:
             o = paged_attn_decode(qf, k_cache, v_cache, block_table, context_lens, spec.scale, window=spec.window,
-                                  num_splits=num_splits)
+                                  chunk=spec.chunk, sinks=sinks, num_splits=num_splits)
         else:
             o = flash_attn_prefill(qf, k_cache, v_cache, block_table, q_start, q_lens, context_lens, spec.scale,
-                                   max_q_len=max_q_len, window=spec.window)
+                                   max_q_len=max_q_len, window=spec.window, chunk=spec.chunk, sinks=sinks)
         return o.view(T, H, spec.vdim_p)[..., :spec.vdim]
     out = torch.empty((T, H, spec.vdim), dtype=k_cache.dtype, device=k_cache.device)
     if not _native(k_cache):
@@ -454,7 +559,12 @@ def heads_attention(spec: MapsSpec, q: torch.Tensor, k_cache: torch.Tensor, v_ca
             vis = torch.arange(ctx)[None, :] <= pos
             if spec.window > 0:
                 vis &= torch.arange(ctx)[None, :] > pos - spec.window
-            a = torch.einsum("hmqk,khv->qhmv", s.masked_fill(~vis, float("-inf")).softmax(-1), v)
+            if spec.chunk > 0:
+                vis &= torch.arange(ctx)[None, :] >= pos - pos % spec.chunk
+            s = s.masked_fill(~vis, float("-inf"))
+            if sinks is not None:
+                s = torch.cat([s, sinks.float()[:, None, None, None].expand(H, M, n, 1)], -1)
+            a = torch.einsum("hmqk,khv->qhmv", s.softmax(-1)[..., :ctx], v)
             o = a[:, :, 0]
             if M == 2:
                 o = o - spec.lam * a[:, :, 1]
@@ -463,6 +573,7 @@ def heads_attention(spec: MapsSpec, q: torch.Tensor, k_cache: torch.Tensor, v_ca
         out.copy_(res.to(out.dtype))
         return out
     L, a = _lib.lib(), spec.arg()
+    a.sinks = _ptr(sinks)
     ref = ctypes.byref(a)
     bf = k_cache.dtype == torch.bfloat16
     common = (q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr())

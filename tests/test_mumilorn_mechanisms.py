@@ -497,7 +497,7 @@ def test_routed_experts(device, dtype, W, ff, E, top, tokens):
     spec = ExpertsSpec(E, top, ff, 0, 0, 1.4)
     block = RoutedExperts(spec, Tensors(lambda k: ws[k].to(device), "", dtype))
     h = rnd(tokens, W, seed=99).to(dtype)
-    got = ops.gated_residual(torch.zeros(tokens, W, device=device), [block.run(None, h.to(device))])[0].cpu()
+    got = ops.gated_residual(torch.zeros(tokens, W, device=device), block.run(None, h.to(device)))[0].cpu()
     some = range(tokens) if tokens < 100 else range(0, tokens, 97)
     m = {"router": {"top": top, "groups": None, "scale": 1.4}}
     want = O.experts(h[list(some)].double(), {k: v.double() for k, v in ws.items()}, m)
