@@ -224,6 +224,10 @@ int nkb_latent_queries(const NkbLatentArgs* a, const NkbProj* q, const float* co
                        long long rot_token, long long rot_head, int rot_pad, int bf16, int tokens, void* stream);
 int nkb_latent_gather(const void* cache, const int* pages, int n_pages, int row, int rank, int rot, int rot_ld, void* c_out,
                       void* r_out, int bf16, int block_size, void* stream);
+int nkb_latent_prefill(const void* q, const void* kv, const void* rotated, const int* q_start, const int* q_lens,
+                       const int* context_lens, const int* kv_base, void* out, int batch, int total_q, int max_q_len, int rows,
+                       int heads, int dim, int rot, int vdim, long long ld, long long rot_ld, int nk, int nv, float scale,
+                       int window, const float* sinks, void* stream);
 long long nkb_latent_scratch_floats(const NkbLatentArgs* a, int tokens, int num_splits);
 int nkb_latent_attn(const NkbLatentArgs* a, const void* q, const void* cache, const int* block_table, const int* q_start,
                     const int* q_lens, const int* context_lens, void* out, float* scratch, int batch, int tokens,

@@ -20,8 +20,13 @@
 // unchanged because both carry the same factor.  KV tiles past a query tile's causal diagonal or before
 // its window are skipped for that tile; the mask is only evaluated on tiles that cross either edge.
 // GQA needs no repeat of K/V: the query head picks its kv head.  Supports causal
-// masking with a cached prefix (q_len <= context_len), sliding windows and
+// masking with a cached prefix (q_len <= context_len), sliding windows, chunks and
 // attention-sink logits.
+//
+// Keys wider than values (latent attention): the sizes are counted in slabs of 64 columns, NK of queries and keys and NV of
+// values, KT tokens per KV tile (64 with three slabs, to fit shared memory).  In the ROWS form K and V are not paged: token j of
+// sequence b is row kv_base[b] + j of matrices with one column block per head, and the last slab of every head's keys
+// comes from a matrix that all heads share (the rotated key part).
 //
 // What the structure answers to (measured on B200 with a cycle trace of one CTA and an issue-rate probe):
 // * The tensor pipe runs a 128 x 128 x 16 MMA in 64 cycles from any operand source, but queues only a few of
@@ -51,10 +56,9 @@ namespace nkb {
 
 constexpr int kQTile = 128;          // rows of one MMA tile
 constexpr int kQPair = 2 * kQTile;   // query rows per CTA
-constexpr int kKVTile = 128;
 constexpr int kPfPage = 32;
 constexpr int kPfThreads = 384;      // warpgroup 0: TMA warp, two MMA warps, one idle; warpgroups 1, 2: softmax
-constexpr int kKVStages = 3;
+constexpr int kMaxKVStages = 4;
 constexpr float kRescaleStep = 8.f;  // log2 of the growth of the row maximum that triggers a rescale of O
 
 struct PrefillParams {
@@ -64,6 +68,7 @@ struct PrefillParams {
   const int* context_lens;
   __nv_bfloat16* out;
   const float* sinks;
+  const int* kv_base;                  // ROWS: row of position 0 of every sequence (may be negative)
   int* status;
   int nq, nkv, max_blocks, causal, window, chunk;
   float scale_log2;
@@ -71,7 +76,7 @@ struct PrefillParams {
 
 struct PrefillCtrl {
   uint64_t q_full;
-  uint64_t kv_full[kKVStages], kv_empty[kKVStages];
+  uint64_t kv_full[kMaxKVStages], kv_empty[kMaxKVStages];
   uint64_t s_full[2], s_empty[2];
   uint64_t p_full[2], o_full[2];
   uint64_t turn[2][4];
@@ -112,6 +117,7 @@ __device__ __forceinline__ bool pf_wait(uint64_t* bar, uint32_t parity, volatile
 struct TileRange {
   int lo, hi, pos0, rows;
 };
+template <int kKVTile>
 __device__ __forceinline__ TileRange tile_range(const PrefillParams& p, int row0, int q_len, int ctx) {
   TileRange r{0, 0, 0, 0};
   if (row0 >= q_len) return r;
@@ -124,15 +130,25 @@ __device__ __forceinline__ TileRange tile_range(const PrefillParams& p, int row0
   return r;
 }
 
-template <int D>
+template <int NK, int NV, int KT>
+struct PrefillSmem {
+  static constexpr int kHalf = kQTile * 128;          // [128 rows][64 bf16] swizzled slab = 16 KB
+  static constexpr int kKVHalf = KT * 128;            // slab of a K or V tile
+  static constexpr int kQBytes = NK * kHalf;          // one query tile
+  static constexpr int kStageBytes = (NK > NV ? NK : NV) * kKVHalf;
+  static constexpr int kPBytes = KT / 64 * kHalf;     // [128 rows][KT tokens]
+  static constexpr int kStages = NK == 3 ? 4 : 3;
+  static constexpr int kBytes = 2 * kQBytes + kStages * kStageBytes + 2 * kPBytes + int(sizeof(PrefillCtrl)) + 1024 + 64;
+};
+
+template <int NK, int NV, int KT, bool ROWS>
 __global__ void __launch_bounds__(kPfThreads, 1)
 flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                          const __grid_constant__ CUtensorMap tmV, const PrefillParams p) {
-  constexpr int NH = D / 64;
-  constexpr int kHalf = 128 * 128;          // [128 rows][64 bf16] swizzled slab = 16 KB
-  constexpr int kQBytes = NH * kHalf;       // one query tile
-  constexpr int kKVBytes = NH * kHalf;      // one K or V tile
-  constexpr int kPBytes = 2 * kHalf;        // [128 rows][128 tokens]
+                          const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmR,
+                          const PrefillParams p) {
+  using L = PrefillSmem<NK, NV, KT>;
+  constexpr int D = NV * 64, kKVTile = KT, kHalf = L::kHalf, kKVHalf = L::kKVHalf, kQBytes = L::kQBytes;
+  constexpr int kKVBytes = L::kStageBytes, kPBytes = L::kPBytes, kKVStages = L::kStages;
   constexpr uint32_t kTmemCols = 512;
   constexpr uint32_t kSCol = 0, kOCol = 256;   // S_t at kSCol + 128 t, O_t at kOCol + 128 t
 
@@ -145,8 +161,8 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
   const int ctx = p.context_lens[b];
   const int q_row0 = p.q_start[b] + qt * kQPair;        // row in the packed q / out arrays
   const int kvh = head / (p.nq / p.nkv);
-  const TileRange tr0 = tile_range(p, qt * kQPair, q_len, ctx);
-  const TileRange tr1 = tile_range(p, qt * kQPair + kQTile, q_len, ctx);
+  const TileRange tr0 = tile_range<KT>(p, qt * kQPair, q_len, ctx);
+  const TileRange tr1 = tile_range<KT>(p, qt * kQPair + kQTile, q_len, ctx);
   const bool two = tr1.rows > 0;
   // union of the two ranges; every tile of it is attended to by at least one query tile
   const int u_lo = tr0.lo, u_hi = two ? max(tr0.hi, tr1.hi) : tr0.hi;
@@ -164,6 +180,7 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
     tma_prefetch_desc(&tmQ);
     tma_prefetch_desc(&tmK);
     tma_prefetch_desc(&tmV);
+    if constexpr (ROWS) tma_prefetch_desc(&tmR);
     mbar_init(&ctrl->q_full, 1);
     for (int i = 0; i < kKVStages; ++i) {
       mbar_init(&ctrl->kv_full[i], 1);
@@ -197,11 +214,12 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
-        for (int h = 0; h < NH; ++h)
+        for (int h = 0; h < NK; ++h)
           tma_load_3d(q_s + t * kQBytes + h * kHalf, &tmQ, &ctrl->q_full, h * 64, head, q_row0 + t * kQTile);
     }
     __syncwarp();
-    const int* table = p.block_table + (long long)b * p.max_blocks;
+    const int* table = ROWS ? nullptr : p.block_table + (long long)b * p.max_blocks;
+    const int kv_row0 = ROWS ? p.kv_base[b] : 0;
     const int last_page = max((ctx + kPfPage - 1) / kPfPage - 1, 0);
     // Ring items in the order the issuers consume them: K(0), then per KV tile u: K(u+1), V(u).  Q K^T runs one
     // tile ahead of P V, so K(u+2) has the whole of iteration u to arrive.  Item `seq` lives in stage seq % 3.
@@ -215,18 +233,35 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       ++seq;
       bool ok = pf_wait(&ctrl->kv_empty[st], ph ^ 1u, abort_flag, p.status, ERR_WAIT_SMEM_EMPTY);
       if (!__all_sync(0xffffffffu, ok)) { live = false; return; }
-      int blk[4];
+      if constexpr (ROWS) {
+        if (lane == 0) {
+          uint8_t* dst = kv_s + st * kKVBytes;
+          const int row = kv_row0 + j * KT;
+          mbar_expect_tx(&ctrl->kv_full[st], (is_v ? NV : NK) * kKVHalf);
+          if (is_v) {
 #pragma unroll
-      for (int pi = 0; pi < 4; ++pi) blk[pi] = table[min(j * 4 + pi, last_page)];
-      if (lane == 0) {
-        const CUtensorMap* tm = is_v ? &tmV : &tmK;
-        uint8_t* dst = kv_s + st * kKVBytes;
-        mbar_expect_tx(&ctrl->kv_full[st], kKVBytes);
+            for (int h = 0; h < NV; ++h) tma_load_3d(dst + h * kKVHalf, &tmV, &ctrl->kv_full[st], h * 64, kvh, row);
+          } else {
 #pragma unroll
-        for (int pi = 0; pi < 4; ++pi)
+            for (int h = 0; h < NK - 1; ++h) tma_load_3d(dst + h * kKVHalf, &tmK, &ctrl->kv_full[st], h * 64, kvh, row);
+            tma_load_2d(dst + (NK - 1) * kKVHalf, &tmR, &ctrl->kv_full[st], 0, row);
+          }
+        }
+      } else {
+        constexpr int kPages = KT / kPfPage;
+        int blk[kPages];
 #pragma unroll
-          for (int h = 0; h < NH; ++h)
-            tma_load_4d(dst + h * kHalf + pi * (kPfPage * 128), tm, &ctrl->kv_full[st], h * 64, 0, kvh, blk[pi]);
+        for (int pi = 0; pi < kPages; ++pi) blk[pi] = table[min(j * kPages + pi, last_page)];
+        if (lane == 0) {
+          const CUtensorMap* tm = is_v ? &tmV : &tmK;
+          uint8_t* dst = kv_s + st * kKVBytes;
+          mbar_expect_tx(&ctrl->kv_full[st], kKVBytes);
+#pragma unroll
+          for (int pi = 0; pi < kPages; ++pi)
+#pragma unroll
+            for (int h = 0; h < NK; ++h)
+              tma_load_4d(dst + h * kKVHalf + pi * (kPfPage * 128), tm, &ctrl->kv_full[st], h * 64, 0, kvh, blk[pi]);
+        }
       }
       __syncwarp();
     };
@@ -248,7 +283,7 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
     const uint32_t kv_lo = uint32_t(make_smem_desc_sw128(smem_u32(kv_s), 0, 1024));
     const uint32_t p_lo = uint32_t(make_smem_desc_sw128(smem_u32(p_s + t * kPBytes), 0, 1024));
     const uint64_t hk = uint64_t(uint32_t(make_smem_desc_sw128(0, 0, 1024) >> 32)) << 32;   // SBO, version, swizzle
-    const uint32_t lbo_v = (uint32_t(kHalf) >> 4) << 16;                                    // low-word part of V's LBO
+    const uint32_t lbo_v = (uint32_t(kKVHalf) >> 4) << 16;                                  // low-word part of V's LBO
     const int a_lo = t == 0 ? tr0.lo - u_lo : (two ? tr1.lo - u_lo : 0);
     const int a_hi = t == 0 ? tr0.hi - u_lo : (two ? tr1.hi - u_lo : 0);
     const uint32_t s_tmem = tmem_base + kSCol + t * 128, o_tmem = tmem_base + kOCol + t * 128;
@@ -268,13 +303,12 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
           tc_fence_after();
           const uint32_t kvd = kv_lo + uint32_t(st * kKVBytes >> 4);
 #pragma unroll
-          for (int h = 0; h < NH; ++h) {
+          for (int h = 0; h < NK; ++h) {
             uint64_t da[4], db[4];
 #pragma unroll
             for (int k4 = 0; k4 < 4; ++k4) {
-              const uint32_t off = uint32_t(h * (kHalf >> 4) + k4 * 2);
-              da[k4] = hk | (q_lo + off);
-              db[k4] = hk | (kvd + off);
+              da[k4] = hk | (q_lo + uint32_t(h * (kHalf >> 4) + k4 * 2));
+              db[k4] = hk | (kvd + uint32_t(h * (kKVHalf >> 4) + k4 * 2));
             }
             umma4_ss(s_tmem, da, db, idesc_qk, h > 0 ? 1u : 0u);
           }
@@ -295,7 +329,7 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
           tc_fence_after();
           const uint32_t kvd = kv_lo + uint32_t(st * kKVBytes >> 4);
 #pragma unroll
-          for (int h = 0; h < 2; ++h) {
+          for (int h = 0; h < KT / 64; ++h) {
             uint64_t da[4], db[4];
 #pragma unroll
             for (int k4 = 0; k4 < 4; ++k4) {
@@ -503,22 +537,22 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
   }
 }
 
-template <int D>
-static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
+template <int NK, int NV, int KT, bool ROWS>
+static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tr,
                           const PrefillParams& p, int batch, int max_q_len, cudaStream_t s) {
-  constexpr int NH = D / 64;
-  constexpr int smem = NH * 16384 * (2 + kKVStages) + 2 * 2 * 16384 + int(sizeof(PrefillCtrl)) + 1024 + 64;
+  constexpr int smem = PrefillSmem<NK, NV, KT>::kBytes;
+  static_assert(smem <= 232448, "shared memory of a CTA");
   static bool attr_set[64] = {false};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -1;
   if (!attr_set[dev]) {
-    cudaError_t e =
-        cudaFuncSetAttribute(flash_attn_prefill_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(flash_attn_prefill_kernel<NK, NV, KT, ROWS>,
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return int(e);
     attr_set[dev] = true;
   }
   dim3 grid((max_q_len + kQPair - 1) / kQPair, p.nq, batch);
-  return launch_pdl(flash_attn_prefill_kernel<D>, grid, dim3(kPfThreads), size_t(smem), s, tq, tk, tv, p);
+  return launch_pdl(flash_attn_prefill_kernel<NK, NV, KT, ROWS>, grid, dim3(kPfThreads), size_t(smem), s, tq, tk, tv, tr, p);
 }
 
 }  // namespace nkb
@@ -559,7 +593,51 @@ extern "C" int nkb_flash_attn_prefill(const void* q, const void* k_cache, const 
     if (encode_tmap_bf16(&tv, v_cache, 4, dims, strides, box)) return -4;
   }
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (head_dim == 128) return launch_prefill<128>(tq, tk, tv, p, batch, max_q_len, s);
-  if (head_dim == 64) return launch_prefill<64>(tq, tk, tv, p, batch, max_q_len, s);
+  if (head_dim == 128) return launch_prefill<2, 2, 128, false>(tq, tk, tv, tk, p, batch, max_q_len, s);
+  if (head_dim == 64) return launch_prefill<1, 1, 128, false>(tq, tk, tv, tk, p, batch, max_q_len, s);
   return -2;
+}
+
+// Prefill attention over expanded latents: kv [rows, ld] holds every head's unrotated key (dim columns each) and then every
+// head's value (vdim columns each), rotated [rows, rot_ld] the key part all heads share; position j of sequence b is row
+// kv_base[b] + j.  q [total_q, heads, 64 nk] has a head's unrotated part in its first columns and the rotated one in its
+// last 64, zeros elsewhere; out is [total_q, heads, 64 nv].  Returns -5 for sizes it does not take.
+extern "C" int nkb_latent_prefill(const void* q, const void* kv, const void* rotated, const int* q_start, const int* q_lens,
+                                  const int* context_lens, const int* kv_base, void* out, int batch, int total_q, int max_q_len,
+                                  int rows, int heads, int dim, int rot, int vdim, long long ld, long long rot_ld, int nk, int nv,
+                                  float scale, int window, const float* sinks, void* stream) {
+  if (batch <= 0 || total_q <= 0) return 0;
+  if (dim < 1 || rot < 1 || vdim < 1 || dim > 64 * (nk - 1) || rot > 64 || vdim > 64 * nv || ((dim | vdim) & 7) || (ld & 7) ||
+      (rot_ld & 7) || rot_ld < rot || heads > 65535 || batch > 65535)
+    return -5;
+  if (rows < 1 || ld < (long long)heads * (dim + vdim)) return -2;
+  if (!status_word() && nkb_init() != 0) return -1;
+  PrefillParams p{};
+  p.q_start = q_start; p.q_lens = q_lens; p.context_lens = context_lens; p.kv_base = kv_base;
+  p.out = reinterpret_cast<__nv_bfloat16*>(out);
+  p.sinks = sinks;
+  p.status = status_word();
+  p.nq = heads; p.nkv = heads; p.causal = 1; p.window = window;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  const int kt = nk == 3 ? 64 : 128;
+  CUtensorMap tq, tk, tv, tr;
+  {
+    const uint64_t dims[3] = {uint64_t(nk) * 64, uint64_t(heads), uint64_t(total_q)};
+    const uint64_t strides[2] = {uint64_t(nk) * 128, uint64_t(nk) * 128 * heads};
+    const uint32_t box[3] = {64, 1, uint32_t(kQTile)};
+    if (encode_tmap_bf16(&tq, q, 3, dims, strides, box)) return -4;
+  }
+  const auto heads_map = [&](CUtensorMap* m, const void* base, int width) {
+    const uint64_t dims[3] = {uint64_t(width), uint64_t(heads), uint64_t(rows)};
+    const uint64_t strides[2] = {uint64_t(width) * 2, uint64_t(ld) * 2};
+    const uint32_t box[3] = {64, 1, uint32_t(kt)};
+    return encode_tmap_bf16(m, base, 3, dims, strides, box);
+  };
+  if (heads_map(&tk, kv, dim) || heads_map(&tv, reinterpret_cast<const __nv_bfloat16*>(kv) + (long long)heads * dim, vdim)) return -4;
+  if (encode_tmap_bf16_2d(&tr, rotated, rot, rows, rot_ld, 64, kt)) return -4;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (nk == 2 && nv == 1) return launch_prefill<2, 1, 128, true>(tq, tk, tv, tr, p, batch, max_q_len, s);
+  if (nk == 2 && nv == 2) return launch_prefill<2, 2, 128, true>(tq, tk, tv, tr, p, batch, max_q_len, s);
+  if (nk == 3 && nv == 2) return launch_prefill<3, 2, 64, true>(tq, tk, tv, tr, p, batch, max_q_len, s);
+  return -5;
 }

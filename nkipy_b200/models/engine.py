@@ -143,7 +143,8 @@ class GenerationEngine:
         ids_d, pos_d, slots_d = to(ids), to(pos), to(slots)
         qs_d, ql_d, ctx_d, rows_d = to(q_start, False), to(q_lens, False), to(ctx, False), to(rows, False)
         table = cache.block_table[rows_d.long()]
-        hidden = m.prefill(ids_d, pos_d, slots_d, cache, table, qs_d, ql_d, ctx_d, max(q_lens), rows=rows_d)
+        hidden = m.prefill(ids_d, pos_d, slots_d, cache, table, qs_d, ql_d, ctx_d, max(q_lens), rows=rows_d,
+                           spans=[(c, n) for _, c, n in parts])
         return hidden, (qs_d + ql_d - 1).long()
 
     def _portions(self, seqs: Sequence[SequenceState]):

@@ -29,7 +29,7 @@ from .. import ops
 from ..ops import Branch, Norm, Proj
 from ..parallel.comm import TPGroup
 from .config import LayerSpec, ModelConfig, RopeSpec, rope_frequencies
-from .kv_cache import PagedKVCache
+from .kv_cache import BLOCK_SIZE, PagedKVCache
 from .mixers import MIXERS, Tensors
 from .moe import RoutedExperts
 from .transformer import pick_splits
@@ -287,6 +287,11 @@ class HybridLM:
         return sum(t.numel() * t.element_size() for t in ts)
 
     # ------------------------------------------------------------------ layers
+    @staticmethod
+    def is_small(h: torch.Tensor) -> bool:
+        """Whether projections of h come as fp32 (split-K) sums, see `project`."""
+        return x_small(h)
+
     def project(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
         """fp32 (split-K partials) for small batches, bf16 for large ones, fp32 for 32-bit models."""
         if x.dtype == torch.float32:
@@ -343,12 +348,13 @@ class HybridLM:
 
     # ------------------------------------------------------------------ the engine's entry points
     def prefill(self, ids, positions, slots, cache, block_table, q_start, q_lens, context_lens, max_q_len,
-                return_hidden: bool = False, rows: Optional[torch.Tensor] = None):
+                return_hidden: bool = False, rows: Optional[torch.Tensor] = None, spans=None):
         """Packed step over the new tokens of several sequences (whole prompts, portions of prompts, single tokens);
-        rows[b] is the batch row (state slot) of sequence b.  Returns the final-normed hidden states [T, W] (and the
+        rows[b] is the batch row (state slot) of sequence b, spans its [first new position, context length) on the host (read
+        back from the device when not given and needed).  Returns the final-normed hidden states [T, W] (and the
         residual stream after every layer run)."""
         return self._forward(ids, cache, Batch(positions, slots, block_table, context_lens, q_start, q_lens, max_q_len,
-                                               rows, ids), return_hidden)
+                                               rows, ids, spans), return_hidden)
 
     def decode_step(self, ids, positions, slots, cache, block_table, context_lens, return_hidden: bool = False):
         """One new token for every batch row; rows with a negative context length are inactive."""
@@ -369,15 +375,36 @@ class HybridLM:
 class Batch:
     """The tokens of a step, where they sit (cache slots, block tables) and how they are grouped into sequences (q_lens
     None: one per batch row)."""
-    __slots__ = ("positions", "slots", "block_table", "context_lens", "q_start", "q_lens", "max_q_len", "rows", "ids")
+    __slots__ = ("positions", "slots", "block_table", "context_lens", "q_start", "q_lens", "max_q_len", "rows", "ids",
+                 "_spans", "_pages")
 
     def __init__(self, positions, slots, block_table, context_lens, q_start=None, q_lens=None, max_q_len=1, rows=None,
-                 ids=None):
+                 ids=None, spans=None):
         self.positions, self.slots, self.block_table, self.context_lens = positions, slots, block_table, context_lens
         self.q_start, self.q_lens, self.max_q_len, self.rows = q_start, q_lens, max_q_len, rows
-        self.ids = ids
+        self.ids, self._spans, self._pages = ids, spans, {}
+
+    def visible_pages(self, window: int):
+        """Cache pages that the new tokens see through a sliding window (0: all before them), sequence by sequence (int32 block
+        numbers), and per sequence the row its position 0 has when those pages' tokens follow one another."""
+        if window not in self._pages:
+            if self._spans is None:
+                self._spans = [(c - n, c) for c, n in zip(self.context_lens.tolist(), self.q_lens.tolist())]
+            seq, page, base, n = [], [], [], 0
+            for b, (first, end) in enumerate(self._spans):
+                lo = max(0, first - window + 1) // BLOCK_SIZE if window > 0 else 0
+                hi = (end + BLOCK_SIZE - 1) // BLOCK_SIZE
+                seq += [b] * (hi - lo)
+                page += range(lo, hi)
+                base.append((n - lo) * BLOCK_SIZE)
+                n += hi - lo
+            dev = self.block_table.device
+            at = torch.tensor([seq, page], dtype=torch.long).to(dev, non_blocking=True)
+            self._pages[window] = (self.block_table[at[0], at[1]].to(torch.int32).contiguous(),
+                                   torch.tensor(base, dtype=torch.int32).to(dev, non_blocking=True))
+        return self._pages[window]
 
 
 def x_small(h: torch.Tensor) -> bool:
-    """Whether the feed-forward's input projection leaves its activation to a kernel of its own."""
+    """Whether projections of h come as fp32 sums and leave what follows them to a kernel of its own."""
     return h.dtype == torch.float32 or h.shape[0] <= SMALL_BATCH

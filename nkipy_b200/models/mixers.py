@@ -164,8 +164,9 @@ class ChunkAttentionMixer:
 
 
 class LatentAttentionMixer:
-    """Latent attention with a sink and a gate per head.  Attention runs on the cached latents: the queries are folded through
-    the keys' up projection, and the values' up projection is applied to the mixtures of latents."""
+    """Latent attention with a sink and a gate per head.  Small batches attend to the cached latents: the queries are folded
+    through the keys' up projection, and the values' up projection is applied to the mixtures of latents.  Large ones expand the
+    keys and values of the visible tokens, which takes fewer operations per query."""
 
     def __init__(self, spec, t: Tensors, eps: float):
         self.spec = spec
@@ -173,14 +174,15 @@ class LatentAttentionMixer:
         self.w_in, self.w_o = t.mat("dq", "dkv", "g"), t.mat("o")
         self.widths = [spec.q_rank, R + spec.rot, H]
         self.w_uq = t.mat("uq")
-        self.w_uk = t.mat("uk").reshape(H, spec.dim, R).transpose(1, 2).contiguous()     # [H, R, dim]
-        self.w_uv = t.mat("uv").reshape(H, spec.vdim, R)
+        self.w_up = t.mat("uk", "uv")                                                    # [H dim + H vdim, R]
+        self.w_uk = self.w_up[:H * spec.dim].reshape(H, spec.dim, R).transpose(1, 2).contiguous()
+        self.w_uv = self.w_up[H * spec.dim:].reshape(H, spec.vdim, R)
         self.q_norm, self.kv_norm, self.sink = t.f32("dq.norm"), t.f32("dkv.norm"), t.f32("sink")
         self.latent = LatentSpec(H, spec.dim, spec.rot, spec.vdim, R, spec.q_rank, spec.scale, spec.window, eps,
                                  tiled=t.dtype == torch.bfloat16)
 
     def weights(self):
-        return [self.w_uq, self.w_uk, self.w_uv]
+        return [self.w_uq, self.w_up]
 
     def entries(self):
         return [KVLayer(1, self.latent.row, 0)]
@@ -191,6 +193,14 @@ class LatentAttentionMixer:
         T = h.shape[0]
         c = ops.latent_append(s, q, kv, self.q_norm, self.kv_norm, table, b.positions, b.slots, rows)
         up = Proj(model.project(c, self.w_uq), 0, self.w_uq.shape[0])
+        if b.q_lens is not None and not model.is_small(h) and s.slabs is not None:
+            q = torch.empty((T, s.heads, 64 * s.slabs[0]), dtype=model.dtype, device=h.device)
+            ops.latent_queries(s, up, table, b.positions, q[..., :-64], q[..., -64:])
+            pages, base = b.visible_pages(s.window)
+            c, r = ops.latent_gather(s, rows, pages, (s.rot + 7) // 8 * 8)
+            kv = model.project(c, self.w_up)
+            o = ops.latent_prefill(s, q, kv, r, base, b.q_start, b.q_lens, b.context_lens, b.max_q_len, self.sink)
+            return ops.gate_heads(o, g, "sigmoid")
         plain = torch.empty((s.heads, T, s.dim), dtype=model.dtype, device=h.device)
         q = torch.empty((s.heads, T, s.row), dtype=model.dtype, device=h.device)
         ops.latent_queries(s, up, table, b.positions, plain.transpose(0, 1), q.transpose(0, 1)[..., s.rank:])

@@ -408,11 +408,12 @@ class TransformerLM:
     # ------------------------------------------------------------------ prefill
     def prefill(self, ids: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, cache: PagedKVCache,
                 block_table: torch.Tensor, q_start: torch.Tensor, q_lens: torch.Tensor, context_lens: torch.Tensor,
-                max_q_len: int, return_hidden: bool = False, inputs=None, rows: Optional[torch.Tensor] = None):
+                max_q_len: int, return_hidden: bool = False, inputs=None, rows: Optional[torch.Tensor] = None,
+                spans=None):
         """Packed prefill of several sequences.  ids / positions / slots [T]; returns the
         final-normed hidden states [T, H] (and the per-layer residual streams when
         return_hidden is set, for speculative-decoding taps).  inputs: see `decode_step`.
-        rows (the sequences' batch rows) is for models with per-row state; unused here."""
+        rows (the sequences' batch rows) and spans (their new positions on the host) are for layer-by-layer models; unused here."""
         cfg = self.cfg
         tp1 = self.tp.world_size == 1
         if (not tp1 and not return_hidden and inputs is None and getattr(self.tp, "fused", None) is not None

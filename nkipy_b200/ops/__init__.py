@@ -31,7 +31,7 @@ __all__ = [
     "argmax", "sample", "decode_advance", "router_topk", "moe_dispatch", "grouped_linear", "moe_combine", "paged_attn_decode", "flash_attn_prefill", "rope_table",
     "Branch", "MapsSpec", "Norm", "Proj", "activation", "gate_heads", "gated_act", "gated_residual", "hgrn2", "maps_append",
     "heads_attention", "maps_attention", "row_norm_append", "rope_norm_append", "head_linear", "softcap",
-    "LatentSpec", "latent_append", "latent_attention", "latent_gather", "latent_queries",
+    "LatentSpec", "latent_append", "latent_attention", "latent_gather", "latent_prefill", "latent_queries",
     "Decay", "linear_attention", "low_rank", "token_mix",
     "KernelLibraryError", "device_status", "raise_on_device_error", "native_available", "launch_count",
     "reset_launch_count",
@@ -1232,5 +1232,5 @@ from . import mixers  # noqa: E402  (uses the helpers above)
 from .mixers import (Branch, MapsSpec, Norm, Proj, activation, gate_heads, gated_act, gated_residual,  # noqa: E402,F401
                      heads_attention, hgrn2, maps_append, maps_attention, rope_norm_append, row_norm_append)
 from .latent_attention import (LatentSpec, latent_append, latent_attention, latent_gather,  # noqa: E402,F401
-                               latent_queries)
+                               latent_prefill, latent_queries)
 from .linear_attention import Decay, linear_attention, low_rank, token_mix  # noqa: E402,F401

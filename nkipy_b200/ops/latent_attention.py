@@ -4,8 +4,9 @@
     latent_queries    up-projected queries split and rotated
     latent_attention  new tokens against the cached rows themselves (queries folded through the keys' up projection)
     latent_gather     cached rows of whole pages, as operands of the keys' and values' up projections
+    latent_prefill    new tokens against keys and values expanded from those rows
 
-CUDA tensors run csrc/kernels/latent_attn.cu (32-bit models and sizes its tensor-core kernel does not take: the general kernel
+CUDA tensors run csrc/kernels/latent_attn.cu and, for expanded keys, attn_prefill.cu (32-bit models and sizes its tensor-core kernel does not take: the general kernel
 of attn_maps.cu); CPU tensors run the PyTorch statement of the same op.
 """
 
@@ -49,6 +50,14 @@ class LatentSpec:
                 if self.rank <= 64 * vs and self.rank + self.rot <= 64 * ns:
                     return 64 * ns
         return (self.rank + self.rot + 7) // 8 * 8
+
+    @property
+    def slabs(self) -> Optional[Tuple[int, int]]:
+        """64-column slabs of expanded queries and keys (the last one rotated) and of values in the prefill kernel; None for
+        sizes it does not take."""
+        if not self.tiled or self.dim > 128 or self.rot > 64 or self.vdim > 128 or (self.dim | self.vdim | self.rank) % 8:
+            return None
+        return (2, 1 if self.vdim <= 64 else 2) if self.dim <= 64 else (3, 2)
 
     def arg(self) -> _lib.LatentArg:
         return _lib.LatentArg(self.heads, self.dim, self.rot, self.rank, self.q_rank, self.row, float(self.eps),
@@ -191,3 +200,44 @@ def latent_attention(spec: LatentSpec, q: torch.Tensor, cache: torch.Tensor, blo
     _lib.check(rc, "latent_attention")
     _count_launch()
     return out
+
+
+def latent_prefill(spec: LatentSpec, q: torch.Tensor, kv: torch.Tensor, rotated: torch.Tensor, kv_base: torch.Tensor,
+                   q_start: torch.Tensor, q_lens: torch.Tensor, context_lens: torch.Tensor, max_q_len: int,
+                   sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal attention over expanded rows: kv [rows, heads * dim | heads * vdim] and rotated [rows, >= rot] hold position j of
+    sequence b in row kv_base[b] + j; q [T, heads, 64 nk] has a head's unrotated part in front and its rotated part in the
+    last 64 columns.  Returns [T, heads, vdim] (strided)."""
+    T, H = q.shape[0], spec.heads
+    nk, nv = spec.slabs
+    out = torch.empty((T, H, 64 * nv), dtype=q.dtype, device=q.device)
+    if not _native(q):
+        out.zero_()
+        split = H * spec.dim
+        for b in range(q_lens.shape[0]):
+            n, t0, ctx, base = int(q_lens[b]), int(q_start[b]), int(context_lens[b]), int(kv_base[b])
+            lo = max(0, ctx - n - spec.window + 1) if spec.window > 0 else 0
+            rows = slice(base + lo, base + ctx)
+            x = q[t0:t0 + n].float()
+            k = kv[rows, :split].float().reshape(-1, H, spec.dim)
+            v = kv[rows, split:split + H * spec.vdim].float().reshape(-1, H, spec.vdim)
+            s = torch.einsum("qhd,khd->hqk", x[..., :spec.dim], k)
+            s = (s + torch.einsum("qhd,kd->hqk", x[..., -64:][..., :spec.rot], rotated[rows, :spec.rot].float())) * spec.scale
+            i, j = (ctx - n + torch.arange(n))[:, None], torch.arange(lo, ctx)[None, :]
+            vis = j <= i
+            if spec.window > 0:
+                vis &= j > i - spec.window
+            s = s.masked_fill(~vis, float("-inf"))
+            if sinks is not None:
+                s = torch.cat([s, sinks.float()[:, None, None].expand(H, n, 1)], -1)
+            out[t0:t0 + n, :, :spec.vdim] = torch.einsum("hqk,khn->qhn", s.softmax(-1)[..., :ctx - lo], v).to(out.dtype)
+        return out[..., :spec.vdim]
+    if not q.is_contiguous() or q.shape[2] != 64 * nk or q.dtype != torch.bfloat16 or kv.dtype != torch.bfloat16:
+        raise ValueError("latent_prefill wants contiguous bf16 queries of whole slabs")
+    rc = _lib.lib().nkb_latent_prefill(
+        q.data_ptr(), kv.data_ptr(), rotated.data_ptr(), q_start.data_ptr(), q_lens.data_ptr(), context_lens.data_ptr(),
+        kv_base.data_ptr(), out.data_ptr(), q_lens.shape[0], T, int(max_q_len), kv.shape[0], H, spec.dim, spec.rot, spec.vdim,
+        kv.stride(0), rotated.stride(0), nk, nv, float(spec.scale), int(spec.window), _ptr(sinks), _stream())
+    _lib.check(rc, "nkb_latent_prefill")
+    _count_launch()
+    return out[..., :spec.vdim]
