@@ -28,20 +28,34 @@ bool pdl_enabled();
 namespace nkb {
 // Launch with the programmatic-stream-serialization attribute (when enabled), so
 // the kernel's prologue overlaps the tail of its predecessor in the stream.
+// cluster_x > 1: that many CTAs along x form a cluster.
 template <typename... KArgs, typename... Args>
-inline int launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
-                      Args&&... args) {
+inline int launch_pdl_cluster(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+                              int cluster_x, Args&&... args) {
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = grid;
   cfg.blockDim = block;
   cfg.dynamicSmemBytes = smem;
   cfg.stream = stream;
-  cudaLaunchAttribute attr[1];
-  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  cudaLaunchAttribute attr[2];
+  int n = 0;
+  if (cluster_x > 1) {
+    attr[n].id = cudaLaunchAttributeClusterDimension;
+    attr[n].val.clusterDim.x = unsigned(cluster_x);
+    attr[n].val.clusterDim.y = 1;
+    attr[n++].val.clusterDim.z = 1;
+  }
+  if (pdl_enabled()) {
+    attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[n++].val.programmaticStreamSerializationAllowed = 1;
+  }
   cfg.attrs = attr;
-  cfg.numAttrs = pdl_enabled() ? 1 : 0;
+  cfg.numAttrs = n;
   return int(cudaLaunchKernelEx(&cfg, kernel, std::forward<Args>(args)...));
+}
+template <typename... KArgs, typename... Args>
+inline int launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args&&... args) {
+  return launch_pdl_cluster(kernel, grid, block, smem, stream, 1, std::forward<Args>(args)...);
 }
 }  // namespace nkb
 #endif
@@ -228,8 +242,6 @@ int nkb_latent_prefill(const void* q, const void* kv, const void* rotated, const
                        const int* context_lens, const int* kv_base, void* out, int batch, int total_q, int max_q_len, int rows,
                        int heads, int dim, int rot, int vdim, long long ld, long long rot_ld, int nk, int nv, float scale,
                        int window, const float* sinks, void* stream);
-long long nkb_latent_scratch_floats(const NkbLatentArgs* a, int tokens, int num_splits);
 int nkb_latent_attn(const NkbLatentArgs* a, const void* q, const void* cache, const int* block_table, const int* q_start,
-                    const int* q_lens, const int* context_lens, void* out, float* scratch, int batch, int tokens,
-                    int block_size, int num_blocks, int max_blocks_per_seq, int num_splits, void* stream);
+                    const int* q_lens, const int* context_lens, void* out, int batch, int tokens, int block_size, int num_blocks, int max_blocks_per_seq, int num_splits, void* stream);
 }

@@ -308,6 +308,98 @@ __global__ void __launch_bounds__(256) rope_norm_append_kernel(const __grid_cons
   }
 }
 
+// Prompts in bf16, sizes of whole 16-byte pieces, heads of at most 8 L elements: L lanes share a head of queries, keys or
+// values, a lane holds eight elements of kRopeUnits heads and loads all of them first.
+constexpr int kRopeUnits = 4;
+
+template <int L>
+__global__ void __launch_bounds__(256) rope_norm_append8_kernel(const __grid_constant__ RopeNormAppendParams p) {
+  using bf = __nv_bfloat16;
+  const int units = p.a.heads + (p.k.ptr ? 2 * p.a.kv_heads : 0), dim = p.a.dim, n = p.rot_dims / 2;
+  const int lane = threadIdx.x & (L - 1), c = lane * 8, groups = 256 / L;
+  griddep_wait();
+  griddep_launch();
+  const long long total = (long long)p.tokens * units, first = blockIdx.x * (long long)(groups * kRopeUnits) + threadIdx.x / L;
+  uint4 raw[kRopeUnits];
+  int tok[kRopeUnits], unit[kRopeUnits];
+#pragma unroll
+  for (int i = 0; i < kRopeUnits; ++i) {
+    const long long w = first + i * groups;
+    tok[i] = w < total ? int(unsigned(w) / unsigned(units)) : -1;
+    unit[i] = w < total ? int(unsigned(w) % unsigned(units)) : 0;
+    raw[i] = make_uint4(0u, 0u, 0u, 0u);
+    if (tok[i] < 0) continue;
+    const int u = unit[i];
+    const bool is_v = u >= p.a.heads + p.a.kv_heads;
+    const NkbProj& src = u < p.a.heads ? p.q : is_v ? p.v : p.k;
+    const int h = u < p.a.heads ? u : is_v ? u - p.a.heads - p.a.kv_heads : u - p.a.heads;
+    const int width = is_v ? p.a.vdim : dim;
+    if (c < width) raw[i] = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf*>(src.ptr) + tok[i] * src.ld + h * width + c);
+  }
+#pragma unroll
+  for (int i = 0; i < kRopeUnits; ++i) {
+    const int u = unit[i];
+    const bool live = tok[i] >= 0, is_q = u < p.a.heads, is_v = u >= p.a.heads + p.a.kv_heads;
+    const int slot = live && !is_q ? p.slots[tok[i]] : 0, width = is_v ? p.a.vdim : dim;
+    float x[8];
+    const uint32_t rw[4] = {raw[i].x, raw[i].y, raw[i].z, raw[i].w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = unpack_bf16x2(rw[e]);
+      x[2 * e] = f.x;
+      x[2 * e + 1] = f.y;
+    }
+    if (p.bias && live && c < width) {
+      const float* b = p.bias + (is_v ? (p.a.heads + p.a.kv_heads) * dim + (u - p.a.heads - p.a.kv_heads) * p.a.vdim : u * dim) + c;
+      const float4 lo = *reinterpret_cast<const float4*>(b), hi = *reinterpret_cast<const float4*>(b + 4);
+      x[0] += lo.x; x[1] += lo.y; x[2] += lo.z; x[3] += lo.w;
+      x[4] += hi.x; x[5] += hi.y; x[6] += hi.z; x[7] += hi.w;
+    }
+    float ss = 0.f, y[8];
+    const int from = c < n ? lane + n / 8 : (c < 2 * n ? lane - n / 8 : lane);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      ss += x[e] * x[e];
+      y[e] = __shfl_sync(0xffffffffu, x[e], from, L);
+    }
+#pragma unroll
+    for (int w = L / 2; w > 0; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
+    if (!live || slot < 0) continue;
+    const long long blk = slot / kMapsPage, off = slot % kMapsPage;
+    bf* dst;
+    int pad = p.a.dim_p;
+    if (is_v) {
+      dst = reinterpret_cast<bf*>(p.v_cache) + ((blk * p.a.kv_heads + u - p.a.heads - p.a.kv_heads) * kMapsPage + off) * p.a.vdim_p;
+      pad = p.a.vdim;
+    } else {
+      const float inv = p.norm ? 1.f / sqrtf(ss / float(dim) + p.a.eps) : 1.f;
+      if (c < 2 * n) {
+        const float* cs = p.cos_sin + (long long)min(max(p.positions[tok[i]], 0), p.max_pos - 1) * p.rot_dims + (c < n ? c : c - n);
+        const float sign = c < n ? -1.f : 1.f;
+        const float4 c0 = *reinterpret_cast<const float4*>(cs), c1 = *reinterpret_cast<const float4*>(cs + 4);
+        const float4 s0 = *reinterpret_cast<const float4*>(cs + n), s1 = *reinterpret_cast<const float4*>(cs + n + 4);
+        const float cv[8] = {c0.x, c0.y, c0.z, c0.w, c1.x, c1.y, c1.z, c1.w};
+        const float sv[8] = {s0.x, s0.y, s0.z, s0.w, s1.x, s1.y, s1.z, s1.w};
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = x[e] * cv[e] + sign * y[e] * sv[e];
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] *= inv;
+      dst = is_q ? reinterpret_cast<bf*>(p.q_out) + ((long long)tok[i] * p.a.heads + u) * p.a.dim_p
+                 : reinterpret_cast<bf*>(p.k_cache) + ((blk * p.a.kv_heads + u - p.a.heads) * kMapsPage + off) * p.a.dim_p;
+    }
+    if (c < pad)
+      *reinterpret_cast<uint4*>(dst + c) =
+          make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
+  }
+}
+
+template <int L>
+static int launch_rope_norm_append8(const RopeNormAppendParams& p, long long warps, cudaStream_t s) {
+  const long long per = 256 / L * kRopeUnits;
+  return launch_pdl(rope_norm_append8_kernel<L>, dim3(unsigned((warps + per - 1) / per)), dim3(256), 0, s, p);
+}
+
 // ------------------------------------------------------------------------------------------------ simple
 struct MapsSimpleParams {
   NkbMapsArgs a;
@@ -825,6 +917,14 @@ extern "C" int nkb_rope_norm_append(const NkbMapsArgs* a, const NkbProj* q, cons
   const dim3 grid(unsigned((warps + 7) / 8)), block(256);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   using bf = __nv_bfloat16;
+  const auto whole = [&](const NkbProj& x) { return !x.ptr || (x.bf16 && al16(x.ptr) && (x.ld & 7) == 0); };
+  const int wide = a->dim_p > a->vdim ? a->dim_p : a->vdim;
+  if (bf16 && ((a->dim | a->dim_p | a->vdim | a->vdim_p) & 7) == 0 && (rot_dims & 15) == 0 && wide <= 256 && whole(*q) && whole(*k) &&
+      whole(*v) && al16(q_out) && al16(k_cache) && al16(v_cache) && al16(bias) && al16(cos_sin)) {
+    if (wide <= 64) return launch_rope_norm_append8<8>(p, warps, s);
+    if (wide <= 128) return launch_rope_norm_append8<16>(p, warps, s);
+    return launch_rope_norm_append8<32>(p, warps, s);
+  }
   if (vec)
     return bf16 ? launch_pdl(rope_norm_append_kernel<4, bf>, grid, block, 0, s, p)
                 : launch_pdl(rope_norm_append_kernel<4, float>, grid, block, 0, s, p);

@@ -138,6 +138,102 @@ __global__ void __launch_bounds__(256) latent_append_kernel(const __grid_constan
   }
 }
 
+__device__ __forceinline__ void unpack8(float (&x)[8], uint4 r) {
+  const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const float2 f = unpack_bf16x2(w[e]);
+    x[2 * e] = f.x;
+    x[2 * e + 1] = f.y;
+  }
+}
+__device__ __forceinline__ uint4 pack8(const float (&x)[8]) {
+  return make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
+}
+__device__ __forceinline__ void load8(float (&x)[8], const float* p) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w;
+  x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+}
+// eight elements (four pairs) from column c of a rotated part of n pairs
+__device__ __forceinline__ void rotate8(float (&x)[8], int c, const float* cs, int n) {
+  const float4 co = *reinterpret_cast<const float4*>(cs + c / 2), si = *reinterpret_cast<const float4*>(cs + n + c / 2);
+  const float cv[4] = {co.x, co.y, co.z, co.w}, sv[4] = {si.x, si.y, si.z, si.w};
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float u = x[2 * j], w = x[2 * j + 1];
+    x[2 * j] = u * cv[j] - w * sv[j];
+    x[2 * j + 1] = w * cv[j] + u * sv[j];
+  }
+}
+
+// Prompts in bf16, sizes of whole 16-byte pieces: one warp per token, all of its loads in flight first.
+constexpr int kAppendQ = 8, kAppendK = 4;            // pieces of a latent per lane: q_rank <= 2048, rank <= 1024
+
+__global__ void __launch_bounds__(256) latent_append8_kernel(const __grid_constant__ LatentAppendParams p, int tokens) {
+  using bf = __nv_bfloat16;
+  const int t = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  griddep_wait();
+  griddep_launch();
+  if (t >= tokens) return;
+  const bf* qs = reinterpret_cast<const bf*>(p.q.ptr) + t * p.q.ld;
+  const bf* ks = reinterpret_cast<const bf*>(p.kv.ptr) + t * p.kv.ld;
+  const int slot = p.slots[t], pos = min(max(p.positions[t], 0), p.max_pos - 1);
+  uint4 q[kAppendQ], k[kAppendK], r = make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+  for (int i = 0; i < kAppendQ; ++i) {
+    const int c = (i * 32 + lane) * 8;
+    q[i] = c < p.a.q_rank ? *reinterpret_cast<const uint4*>(qs + c) : make_uint4(0u, 0u, 0u, 0u);
+  }
+#pragma unroll
+  for (int i = 0; i < kAppendK; ++i) {
+    const int c = (i * 32 + lane) * 8;
+    k[i] = c < p.a.rank ? *reinterpret_cast<const uint4*>(ks + c) : make_uint4(0u, 0u, 0u, 0u);
+  }
+  if (lane * 8 < p.a.rot) r = *reinterpret_cast<const uint4*>(ks + p.a.rank + lane * 8);
+  const auto squares = [](uint4 v) {
+    float x[8], s = 0.f;
+    unpack8(x, v);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s += x[j] * x[j];
+    return s;
+  };
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < kAppendQ; ++i) sq += squares(q[i]);
+#pragma unroll
+  for (int i = 0; i < kAppendK; ++i) sk += squares(k[i]);
+  const float iq = 1.f / sqrtf(warp_sum(sq) / float(p.a.q_rank) + p.a.eps);
+  const float ik = 1.f / sqrtf(warp_sum(sk) / float(p.a.rank) + p.a.eps);
+  const auto scaled = [](uint4 v, float inv, const float* w) {
+    float x[8], ww[8];
+    unpack8(x, v);
+    load8(ww, w);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) x[j] *= inv * ww[j];
+    return pack8(x);
+  };
+  bf* qo = reinterpret_cast<bf*>(p.q_out) + (long long)t * p.a.q_rank;
+#pragma unroll
+  for (int i = 0; i < kAppendQ; ++i) {
+    const int c = (i * 32 + lane) * 8;
+    if (c < p.a.q_rank) *reinterpret_cast<uint4*>(qo + c) = scaled(q[i], iq, p.q_norm + c);
+  }
+  if (slot < 0) return;
+  bf* row = reinterpret_cast<bf*>(p.cache) + (long long)slot * p.a.row;
+#pragma unroll
+  for (int i = 0; i < kAppendK; ++i) {
+    const int c = (i * 32 + lane) * 8;
+    if (c < p.a.rank) *reinterpret_cast<uint4*>(row + c) = scaled(k[i], ik, p.kv_norm + c);
+  }
+  if (lane * 8 < p.a.row - p.a.rank) {
+    float x[8];
+    unpack8(x, r);
+    if (lane * 8 < p.a.rot) rotate8(x, lane * 8, p.cos_sin + (long long)pos * p.a.rot, p.a.rot / 2);
+    *reinterpret_cast<uint4*>(row + p.a.rank + lane * 8) = pack8(x);
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ queries
 struct LatentQueryParams {
   NkbProj q;                // [tokens, heads * (dim + rot)]
@@ -175,6 +271,52 @@ __global__ void __launch_bounds__(256) latent_query_kernel(const __grid_constant
   }
 }
 
+// Prompts in bf16, sizes of whole 16-byte pieces: one CTA per token, kQueryUnroll pieces per thread in flight.
+constexpr int kQueryUnroll = 4;
+
+__global__ void __launch_bounds__(256) latent_query8_kernel(const __grid_constant__ LatentQueryParams p) {
+  using bf = __nv_bfloat16;
+  const long long t = blockIdx.x;
+  const int per = (p.plain_pad + p.rot_pad) / 8, n = p.a.heads * per;
+  griddep_wait();
+  griddep_launch();
+  const bf* src = reinterpret_cast<const bf*>(p.q.ptr) + t * p.q.ld;
+  bf* plain = reinterpret_cast<bf*>(p.plain) + t * p.plain_token;
+  bf* rotated = reinterpret_cast<bf*>(p.rotated) + t * p.rot_token;
+  const float* cs = p.cos_sin + (long long)min(max(p.positions[t], 0), p.max_pos - 1) * p.a.rot;
+  for (int i0 = threadIdx.x; i0 < n; i0 += 256 * kQueryUnroll) {
+    uint4 r[kQueryUnroll];
+    int hd[kQueryUnroll], col[kQueryUnroll];
+#pragma unroll
+    for (int u = 0; u < kQueryUnroll; ++u) {
+      const int i = i0 + u * 256;
+      hd[u] = i / per;
+      col[u] = (i % per) * 8;
+      r[u] = make_uint4(0u, 0u, 0u, 0u);
+      const bool rot = col[u] >= p.plain_pad;
+      const int c = rot ? col[u] - p.plain_pad : col[u];
+      if (i < n && c < (rot ? p.a.rot : p.a.dim))
+        r[u] = *reinterpret_cast<const uint4*>(src + hd[u] * (p.a.dim + p.a.rot) + (rot ? p.a.dim : 0) + c);
+    }
+#pragma unroll
+    for (int u = 0; u < kQueryUnroll; ++u) {
+      if (i0 + u * 256 >= n) break;
+      if (col[u] < p.plain_pad) {
+        *reinterpret_cast<uint4*>(plain + hd[u] * p.plain_head + col[u]) = r[u];
+        continue;
+      }
+      const int c = col[u] - p.plain_pad;
+      if (c < p.a.rot) {
+        float x[8];
+        unpack8(x, r[u]);
+        rotate8(x, c, cs, p.a.rot / 2);
+        r[u] = pack8(x);
+      }
+      *reinterpret_cast<uint4*>(rotated + hd[u] * p.rot_head + c) = r[u];
+    }
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ gather
 // One CTA per page: cached rows -> latents [.., rank] and rotated parts [.., rot_ld] (padding of the cache row included).
 template <typename T>
@@ -203,59 +345,74 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const T* __restrict_
 }
 
 // ------------------------------------------------------------------------------------------------ attention
-// One CTA of four warps per (split of the visible pages, 16 MT heads, new token).  A page's rows come in once by TMA (slabs of
-// 64 columns, 128-byte swizzle) and serve as keys and as values of all heads:
-//   scores   every warp contracts a quarter of the row's columns; the queries of its quarter stay in registers as MMA
-//            fragments.  The four partial products meet in shared memory.
-//   softmax  128 / (16 MT) threads per head sum the partials, mask, and keep the running maximum and denominator
-//   values   every warp multiplies the probabilities with a quarter of the latent's columns
-// Two block barriers per page.  Splits are merged by the CTA that arrives last, as in attn_decode.cu.
+// One CTA of 4 MT consumer warps and a TMA warp per (split of the visible pages, 16 MT heads, new token).  A page's rows come in once by TMA (slabs of
+// 64 columns, 128-byte swizzle) and serve as keys and as values of all heads.  A warp belongs to 16 heads and a quarter of the
+// columns (16 of every 64, so that all its addresses are a constant offset from one):
+//   scores   contracts its quarter of the row; the queries stay in registers as MMA fragments.  The four partial products
+//            of a head meet in shared memory.
+//   softmax  eight threads per head sum the partials, mask, and keep the running maximum and denominator
+//   values   multiplies the probabilities with its quarter of the latent
+// A page is mostly latency (loads of fragments, chains of products, exchanges), so the scores of page i + 1 are contracted
+// between the softmax and the values of page i: one barrier per page hands over both, with two buffers of each.  The ring
+// takes most of the shared memory, because a page arrives a microsecond and more after its load was issued.  The splits of a token are a cluster: each leaves its unnormalised sums in shared memory, and
+// each adds up a share of the heads from all of them.
 // NS: slabs of a row; VS: slabs of its latent.
-constexpr int kLatCounters = 16384;   // arrival counters in front of the split partials
+constexpr int kLatMaxSplits = 8;
 
 struct LatentMmaParams {
   NkbLatentArgs a;
   const __nv_bfloat16* q;
   const int *block_table, *q_start, *q_lens, *context_lens;
   __nv_bfloat16* out;
-  float* scratch;
-  unsigned int* counters;
   int* status;
   int batch, max_blocks, num_splits;
   float scale_log2;
 };
 
-template <int NS>
-struct LatentStages {
-  static constexpr int value = NS >= 8 ? 2 : 3;
-};
-
 template <int NS, int VS, int MT>
 struct LatentSmem {
-  static constexpr int kSlab = kLatPage * 128, kStage = NS * kSlab, kStages = LatentStages<NS>::value;
+  static constexpr int kSlab = kLatPage * 128, kStage = NS * kSlab, kStages = NS >= 9 ? 5 : 6;
   static constexpr int kRows = 16 * MT, kSLd = 36, kPLd = 40;      // leading dimensions of scores (fp32) and probabilities
   static constexpr int kScores = kStages * kStage;
-  static constexpr int kProbs = kScores + 4 * kRows * kSLd * 4;
-  static constexpr int kEnd = kProbs + kRows * kPLd * 2;
+  static constexpr int kScoreBytes = 4 * kRows * kSLd * 4, kProbBytes = kRows * kPLd * 2;
+  static constexpr int kProbs = kScores + 2 * kScoreBytes;
+  static constexpr int kEnd = kProbs + 2 * kProbBytes;
+  static constexpr int kOLd = VS * 64 + 8;                         // of the sums that splits exchange, in the ring's place
+  static_assert(kRows * kOLd * 4 <= kScores, "sums fit in the ring");
 };
 
+__device__ __forceinline__ float ld_cluster(uint32_t addr) {
+  float v;
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
+  return v;
+}
+__device__ __forceinline__ float4 ld_cluster4(uint32_t addr) {
+  float4 v;
+  asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr) : "memory");
+  return v;
+}
+
 template <int NS, int VS, int MT>
-__global__ void __launch_bounds__(128, 2)
+__global__ void __launch_bounds__(128 * MT + 32, 1)
 latent_mma_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ LatentMmaParams p) {
   using L = LatentSmem<NS, VS, MT>;
-  constexpr int kRows = L::kRows, VC = VS * 64, TPR = 128 / kRows, PER = kLatPage / TPR;
+  constexpr int kRows = L::kRows, VC = VS * 64, kThreads = 128 * MT, TPR = 8, PER = kLatPage / TPR;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  float* s_s = reinterpret_cast<float*>(smem + L::kScores);                       // [4][kRows][kSLd]
-  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(smem + L::kProbs);        // [kRows][kPLd]
-  __shared__ uint64_t bars[L::kStages];
-  __shared__ float al_s[kRows], m_s[kRows], l_s[kRows];
-  __shared__ int abort_flag, is_last;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
+  float* s_s = reinterpret_cast<float*>(smem + L::kScores);                       // [2][4][kRows][kSLd]
+  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(smem + L::kProbs);        // [2][kRows][kPLd]
+  __shared__ uint64_t full[L::kStages], empty[L::kStages];
+  __shared__ float al_s[2][kRows], m_s[kRows], l_s[kRows];
+  __shared__ float sc_s[kLatMaxSplits][kRows];
+  __shared__ int abort_flag;
+  const int mt = threadIdx.x >> 7, quarter = (threadIdx.x >> 5) & 3, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
   const int split = blockIdx.x, head0 = blockIdx.y * kRows, t = blockIdx.z;
   const int nh = min(kRows, p.a.heads - head0);
   if (threadIdx.x == 0) {
-    for (int s = 0; s < L::kStages; ++s) mbar_init(&bars[s], 1);
+    for (int s = 0; s < L::kStages; ++s) {
+      mbar_init(&full[s], 1);
+      mbar_init(&empty[s], 4 * MT);
+    }
     abort_flag = 0;
     mbar_fence_init();
     fence_proxy_async();
@@ -280,7 +437,7 @@ latent_mma_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant
   __nv_bfloat16* out = p.out + t * p.a.o_token + head0 * p.a.o_head;
   if (pos < 0) {
     if (split == 0)
-      for (int i = threadIdx.x; i < nh * p.a.rank; i += 128)
+      for (int i = threadIdx.x; i < nh * p.a.rank; i += blockDim.x)
         out[(i / p.a.rank) * p.a.o_head + i % p.a.rank] = __float2bfloat16(0.f);
     return;
   }
@@ -289,234 +446,249 @@ latent_mma_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant
   const int per_split = (npages + p.num_splits - 1) / p.num_splits;
   const int p0 = page_lo + split * per_split, n = max(0, min(page_lo + npages, p0 + per_split) - p0);
   const int* table = p.block_table + (long long)b * p.max_blocks;
-  auto issue = [&](int i) {
-    const int st = i % L::kStages, blk = table[p0 + i];
-    mbar_expect_tx(&bars[st], L::kStage);
+  const bool consumer = threadIdx.x < kThreads;
+  if (!consumer) {
+    int blk = n > 0 ? table[p0] : 0;
+    for (int i = 0; i < n; ++i) {
+      const int st = i % L::kStages, next = i + 1 < n ? table[p0 + i + 1] : 0;
+      const bool ok = mbar_wait(&empty[st], (uint32_t(i / L::kStages) & 1u) ^ 1u, &abort_flag, p.status, ERR_WAIT_SMEM_EMPTY);
+      if (!__all_sync(0xffffffffu, ok)) break;
+      if (lane == 0) {
+        mbar_expect_tx(&full[st], L::kStage);
 #pragma unroll
-    for (int s = 0; s < NS; ++s) tma_load_3d(smem + st * L::kStage + s * L::kSlab, &tmC, &bars[st], s * 64, 0, blk);
-  };
-  if (threadIdx.x == 0)
-    for (int i = 0; i < L::kStages && i < n; ++i) issue(i);
+        for (int s = 0; s < NS; ++s) tma_load_3d(smem + st * L::kStage + s * L::kSlab, &tmC, &full[st], s * 64, 0, blk);
+      }
+      __syncwarp();
+      blk = next;
+    }
+  }
 
-  uint32_t qf[MT][NS][4];
-#pragma unroll
-  for (int mt = 0; mt < MT; ++mt) {
+  uint32_t qf[NS][4];
+  if (consumer) {
     const int r0 = mt * 16 + g, r1 = r0 + 8;
     const __nv_bfloat16* q0 = p.q + t * p.a.q_token + (head0 + r0) * p.a.q_head;
     const __nv_bfloat16* q1 = q0 + 8 * p.a.q_head;
 #pragma unroll
     for (int k = 0; k < NS; ++k) {
-      const int c = (warp * NS + k) * 16 + 2 * tq;
-      qf[mt][k][0] = r0 < nh ? *reinterpret_cast<const uint32_t*>(q0 + c) : 0u;
-      qf[mt][k][1] = r1 < nh ? *reinterpret_cast<const uint32_t*>(q1 + c) : 0u;
-      qf[mt][k][2] = r0 < nh ? *reinterpret_cast<const uint32_t*>(q0 + c + 8) : 0u;
-      qf[mt][k][3] = r1 < nh ? *reinterpret_cast<const uint32_t*>(q1 + c + 8) : 0u;
+      const int c = (4 * k + quarter) * 16 + 2 * tq;
+      qf[k][0] = r0 < nh ? *reinterpret_cast<const uint32_t*>(q0 + c) : 0u;
+      qf[k][1] = r1 < nh ? *reinterpret_cast<const uint32_t*>(q1 + c) : 0u;
+      qf[k][2] = r0 < nh ? *reinterpret_cast<const uint32_t*>(q0 + c + 8) : 0u;
+      qf[k][3] = r1 < nh ? *reinterpret_cast<const uint32_t*>(q1 + c + 8) : 0u;
     }
   }
-  float o[MT][2 * VS][4];
+  float o[2 * VS][4];
 #pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-    for (int i = 0; i < 2 * VS; ++i) o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f;
+  for (int i = 0; i < 2 * VS; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   const int row = threadIdx.x / TPR, sub = threadIdx.x % TPR;
   float m = -INFINITY, l = 0.f;
+  // fragment addresses within a slab: keys (two groups of eight tokens by sixteen columns), values (transposed)
+  const uint32_t k_off = ((lane >> 4) * 8 + (lane & 7)) * 128 + (((2 * quarter + ((lane >> 3) & 1)) ^ (lane & 7)) << 4);
+  const uint32_t v_off = (lane & 15) * 128 + (((2 * quarter + (lane >> 4)) ^ (lane & 7)) << 4);
 
-  for (int i = 0; i < n; ++i) {
+  // partial scores of page i -> buffer i & 1; returns whether the page arrived
+  const auto scores = [&](int i) {
     const int st = i % L::kStages;
-    const bool ok = mbar_wait(&bars[st], uint32_t(i / L::kStages) & 1u, &abort_flag, p.status, ERR_WAIT_SMEM_FULL);
-    const uint32_t base = smem_u32(smem + st * L::kStage);
+    const bool ok = mbar_wait(&full[st], uint32_t(i / L::kStages) & 1u, &abort_flag, p.status, ERR_WAIT_SMEM_FULL);
+    const uint32_t base = smem_u32(smem + st * L::kStage) + k_off;
+    float s[4][4];
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      float s[MT][2][4];
+    for (int nt = 0; nt < 4; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
+    uint32_t kb[2][8];                // fragments of one step are loaded while the step before is multiplied
+    ldsm_x4(base, kb[0][0], kb[0][1], kb[0][2], kb[0][3]);
+    ldsm_x4(base + 2048, kb[0][4], kb[0][5], kb[0][6], kb[0][7]);
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-        for (int nt = 0; nt < 2; ++nt) s[mt][nt][0] = s[mt][nt][1] = s[mt][nt][2] = s[mt][nt][3] = 0.f;
-#pragma unroll
-      for (int k = 0; k < NS; ++k) {
-        // two groups of eight tokens by sixteen columns
-        const int tok = half * 16 + (lane >> 4) * 8 + (lane & 7), ch = 2 * (warp * NS + k) + ((lane >> 3) & 1);
-        uint32_t b0, b1, b2, b3;
-        ldsm_x4(base + (ch >> 3) * L::kSlab + tok * 128 + (((ch & 7) ^ (tok & 7)) << 4), b0, b1, b2, b3);
-#pragma unroll
-        for (int mt = 0; mt < MT; ++mt) {
-          mma_16816(s[mt][0], qf[mt][k], b0, b1);
-          mma_16816(s[mt][1], qf[mt][k], b2, b3);
-        }
+    for (int k = 0; k < NS; ++k) {
+      if (k + 1 < NS) {
+        uint32_t(&d)[8] = kb[(k + 1) & 1];
+        ldsm_x4(base + (k + 1) * L::kSlab, d[0], d[1], d[2], d[3]);
+        ldsm_x4(base + (k + 1) * L::kSlab + 2048, d[4], d[5], d[6], d[7]);
       }
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-          float* d = s_s + (warp * kRows + mt * 16 + g) * L::kSLd + half * 16 + nt * 8 + 2 * tq;
-          *reinterpret_cast<float2*>(d) = make_float2(s[mt][nt][0], s[mt][nt][1]);
-          *reinterpret_cast<float2*>(d + 8 * L::kSLd) = make_float2(s[mt][nt][2], s[mt][nt][3]);
-        }
+      for (int nt = 0; nt < 4; ++nt) mma_16816(s[nt], qf[k], kb[k & 1][2 * nt], kb[k & 1][2 * nt + 1]);
     }
-    if (!__syncthreads_and(ok)) break;
-    // every warp is done with the page before this one: its stage is free
-    if (threadIdx.x == 0 && i > 0 && i - 1 + L::kStages < n) issue(i - 1 + L::kStages);
-    float x[PER], mx = -INFINITY;
-    {
-      const float* sp = s_s + row * L::kSLd + sub * PER;
+    float* d = s_s + ((i & 1) * 4 + quarter) * kRows * L::kSLd + (mt * 16 + g) * L::kSLd + 2 * tq;
 #pragma unroll
-      for (int j = 0; j < PER; j += 4) {
-        float4 a = *reinterpret_cast<const float4*>(sp + j);
+    for (int nt = 0; nt < 4; ++nt) {
+      *reinterpret_cast<float2*>(d + nt * 8) = make_float2(s[nt][0], s[nt][1]);
+      *reinterpret_cast<float2*>(d + nt * 8 + 8 * L::kSLd) = make_float2(s[nt][2], s[nt][3]);
+    }
+    return ok;
+  };
+  if (consumer && n > 0) {
+    bool ok = bar_red_and(1, kThreads, scores(0));
+    for (int i = 0; i < n && ok; ++i) {
+      const int st = i % L::kStages, buf = i & 1;
+      {
+        static_assert(PER == 4, "one vector of scores per thread");
+        const float* sp = s_s + buf * 4 * kRows * L::kSLd + row * L::kSLd + sub * PER;
+        float4 a = *reinterpret_cast<const float4*>(sp);
 #pragma unroll
         for (int w = 1; w < 4; ++w) {
-          const float4 c = *reinterpret_cast<const float4*>(sp + w * kRows * L::kSLd + j);
+          const float4 c = *reinterpret_cast<const float4*>(sp + w * kRows * L::kSLd);
           a.x += c.x; a.y += c.y; a.z += c.z; a.w += c.w;
         }
-        x[j] = a.x; x[j + 1] = a.y; x[j + 2] = a.z; x[j + 3] = a.w;
+        float x[PER] = {a.x, a.y, a.z, a.w}, mx = -INFINITY;
+        const int tok0 = (p0 + i) * kLatPage + sub * PER;
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+          x[j] = tok0 + j >= lo && tok0 + j <= pos ? x[j] * p.scale_log2 : -INFINITY;
+          mx = fmaxf(mx, x[j]);
+        }
+#pragma unroll
+        for (int w = 1; w < TPR; w <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, w));
+        const float mn = fmaxf(m, mx), alpha = exp2f(m - mn);  // finite: every page holds a visible token
+        m = mn;
+        float sum = 0.f;
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+          x[j] = exp2f(x[j] - mn);
+          sum += x[j];
+        }
+        l = l * alpha + sum;                                   // this thread's share of the denominator
+        *reinterpret_cast<uint2*>(p_s + (buf * kRows + row) * L::kPLd + sub * PER) =
+            make_uint2(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]));
+        if (sub == 0) al_s[buf][row] = alpha;
       }
-      const int tok0 = (p0 + i) * kLatPage + sub * PER;
-#pragma unroll
-      for (int j = 0; j < PER; ++j) {
-        x[j] = tok0 + j >= lo && tok0 + j <= pos ? x[j] * p.scale_log2 : -INFINITY;
-        mx = fmaxf(mx, x[j]);
-      }
-    }
-#pragma unroll
-    for (int w = 1; w < TPR; w <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, w));
-    const float mn = fmaxf(m, mx), alpha = exp2f(m - mn);      // finite: every page holds a visible token
-    m = mn;
-    float sum = 0.f;
-#pragma unroll
-    for (int j = 0; j < PER; ++j) {
-      x[j] = exp2f(x[j] - mn);
-      sum += x[j];
-    }
-    l = l * alpha + sum;                                       // this thread's share of the denominator
-    __nv_bfloat16* pd = p_s + row * L::kPLd + sub * PER;
-#pragma unroll
-    for (int j = 0; j < PER; j += 4)
-      *reinterpret_cast<uint2*>(pd + j) = make_uint2(pack_bf16x2(x[j], x[j + 1]), pack_bf16x2(x[j + 2], x[j + 3]));
-    if (sub == 0) al_s[row] = alpha;
-    __syncthreads();
-    uint32_t pa[MT][2][4];
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt) {
-      const float a0 = al_s[mt * 16 + g], a1 = al_s[mt * 16 + g + 8];
-#pragma unroll
-      for (int u = 0; u < 2 * VS; ++u) {
-        o[mt][u][0] *= a0; o[mt][u][1] *= a0;
-        o[mt][u][2] *= a1; o[mt][u][3] *= a1;
-      }
+      bool next = true;
+      if (i + 1 < n) next = scores(i + 1);
+      ok = bar_red_and(1, kThreads, next);
+      if (!ok) break;
+      const uint32_t base = smem_u32(smem + st * L::kStage) + v_off;
+      uint32_t pa[2][4], vb[2][4];
 #pragma unroll
       for (int j = 0; j < 2; ++j)
-        ldsm_x4(smem_u32(p_s + (mt * 16 + (lane & 15)) * L::kPLd + 16 * j + (lane >> 4) * 8), pa[mt][j][0], pa[mt][j][1],
-                pa[mt][j][2], pa[mt][j][3]);
-    }
+        ldsm_x4(smem_u32(p_s + (buf * kRows + mt * 16 + (lane & 15)) * L::kPLd + 16 * j + (lane >> 4) * 8), pa[j][0], pa[j][1],
+                pa[j][2], pa[j][3]);
+      ldsm_x4_t(base, vb[0][0], vb[0][1], vb[0][2], vb[0][3]);
+      const float a0 = al_s[buf][mt * 16 + g], a1 = al_s[buf][mt * 16 + g + 8];
+      if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {   // most pages raise no maximum
 #pragma unroll
-    for (int j = 0; j < 2; ++j)
-#pragma unroll
-      for (int u = 0; u < VS; ++u) {
-        const int tok = 16 * j + ((lane >> 3) & 1) * 8 + (lane & 7), ch = 2 * (warp * VS + u) + (lane >> 4);
-        uint32_t v0, v1, v2, v3;
-        ldsm_x4_t(base + (ch >> 3) * L::kSlab + tok * 128 + (((ch & 7) ^ (tok & 7)) << 4), v0, v1, v2, v3);
-#pragma unroll
-        for (int mt = 0; mt < MT; ++mt) {
-          mma_16816(o[mt][2 * u], pa[mt][j], v0, v1);
-          mma_16816(o[mt][2 * u + 1], pa[mt][j], v2, v3);
+        for (int u = 0; u < 2 * VS; ++u) {
+          o[u][0] *= a0; o[u][1] *= a0;
+          o[u][2] *= a1; o[u][3] *= a1;
         }
       }
+#pragma unroll
+      for (int q = 0; q < 2 * VS; ++q) {
+        if (q + 1 < 2 * VS) {
+          uint32_t(&d)[4] = vb[(q + 1) & 1];
+          ldsm_x4_t(base + ((q + 1) % VS) * L::kSlab + ((q + 1) / VS) * 2048, d[0], d[1], d[2], d[3]);
+        }
+        const int u = q % VS, j = q / VS;
+        mma_16816(o[2 * u], pa[j], vb[q & 1][0], vb[q & 1][1]);
+        mma_16816(o[2 * u + 1], pa[j], vb[q & 1][2], vb[q & 1][3]);
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&empty[st]);
+    }
   }
   if (*(volatile int*)&abort_flag) {
     for (int i = 0; i < 200; ++i) __nanosleep(1000);
   }
 #pragma unroll
   for (int w = 1; w < TPR; w <<= 1) l += __shfl_xor_sync(0xffffffffu, l, w);
-  if (sub == 0) {
+  if (consumer && sub == 0) {
     m_s[row] = m;
     l_s[row] = l;
   }
   __syncthreads();
   const auto sink_log2 = [&](int r) { return p.a.sinks ? p.a.sinks[head0 + r] * 1.4426950408889634f : -INFINITY; };
   if (p.num_splits == 1) {
+    if (!consumer) return;
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
+    for (int e = 0; e < 2; ++e) {
+      const int r = mt * 16 + g + 8 * e;
+      if (r >= nh) continue;
+      const float sk = sink_log2(r), m2 = fmaxf(m_s[r], sk), sc = exp2f(m_s[r] - m2);
+      const float inv = sc / (l_s[r] * sc + exp2f(sk - m2));
+      __nv_bfloat16* dst = out + r * p.a.o_head;
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int r = mt * 16 + g + 8 * e;
-        if (r >= nh) continue;
-        const float sk = sink_log2(r), m2 = fmaxf(m_s[r], sk), sc = exp2f(m_s[r] - m2);
-        const float inv = sc / (l_s[r] * sc + exp2f(sk - m2));
-        __nv_bfloat16* dst = out + r * p.a.o_head;
-#pragma unroll
-        for (int u = 0; u < 2 * VS; ++u) {
-          const int c = warp * VS * 16 + u * 8 + 2 * tq;
-          const float v0 = o[mt][u][2 * e] * inv, v1 = o[mt][u][2 * e + 1] * inv;
-          if (c + 1 < p.a.rank && ((p.a.o_head | p.a.o_token) & 1) == 0) {
-            *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(v0, v1);
-          } else {
-            if (c < p.a.rank) dst[c] = __float2bfloat16(v0);
-            if (c + 1 < p.a.rank) dst[c + 1] = __float2bfloat16(v1);
-          }
+      for (int u = 0; u < 2 * VS; ++u) {
+        const int c = (u / 2 * 4 + quarter) * 16 + (u & 1) * 8 + 2 * tq;
+        const float v0 = o[u][2 * e] * inv, v1 = o[u][2 * e + 1] * inv;
+        if (c + 1 < p.a.rank && ((p.a.o_head | p.a.o_token) & 1) == 0) {
+          *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(v0, v1);
+        } else {
+          if (c < p.a.rank) dst[c] = __float2bfloat16(v0);
+          if (c + 1 < p.a.rank) dst[c + 1] = __float2bfloat16(v1);
         }
       }
+    }
     return;
   }
-  const long long unit = (long long)t * gridDim.y + blockIdx.y;
-  constexpr int kPart = kRows * VC + 2 * kRows;
-  float* part = p.scratch + (unit * p.num_splits + split) * kPart;
+  float* o_s = reinterpret_cast<float*>(smem);       // every page has been consumed (barrier above)
 #pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
+  for (int u = 0; u < 2 * VS; ++u) {
+    if (!consumer) break;
+    float* d = o_s + (mt * 16 + g) * L::kOLd + (u / 2 * 4 + quarter) * 16 + (u & 1) * 8 + 2 * tq;
+    *reinterpret_cast<float2*>(d) = make_float2(o[u][0], o[u][1]);
+    *reinterpret_cast<float2*>(d + 8 * L::kOLd) = make_float2(o[u][2], o[u][3]);
+  }
+  cluster_sync_all();
+  // this CTA's heads: r0 .. r0 + per - 1
+  const int splits = p.num_splits, per = kRows / splits, r0 = split * per;
+  if (int(threadIdx.x) < per) {
+    const int r = r0 + threadIdx.x;
+    const float sk = r < nh ? sink_log2(r) : -INFINITY;
+    float ms[kLatMaxSplits], ls[kLatMaxSplits], mf = sk, den = 0.f;
 #pragma unroll
-    for (int u = 0; u < 2 * VS; ++u) {
-      float* d = part + (mt * 16 + g) * VC + warp * VS * 16 + u * 8 + 2 * tq;
-      *reinterpret_cast<float2*>(d) = make_float2(o[mt][u][0], o[mt][u][1]);
-      *reinterpret_cast<float2*>(d + 8 * VC) = make_float2(o[mt][u][2], o[mt][u][3]);
-    }
-  if (int(threadIdx.x) < kRows) {
-    part[kRows * VC + threadIdx.x] = m_s[threadIdx.x];
-    part[kRows * VC + kRows + threadIdx.x] = l_s[threadIdx.x];
-  }
-  __threadfence();
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    unsigned int* ctr = p.counters + unit;
-    const unsigned int old = atomicAdd(ctr, 1u);
-    is_last = old == unsigned(p.num_splits - 1);
-    if (is_last) *ctr = 0u;
-  }
-  __syncthreads();
-  if (!is_last) return;
-  __threadfence();
-  const float* first = p.scratch + unit * p.num_splits * kPart;
-  if (int(threadIdx.x) < kRows) {
-    const int r = threadIdx.x;
-    float mf = r < nh ? sink_log2(r) : -INFINITY, den = 0.f;
-    for (int s = 0; s < p.num_splits; ++s) mf = fmaxf(mf, __ldcg(first + s * kPart + kRows * VC + r));
-    if (r < nh && p.a.sinks) den = exp2f(sink_log2(r) - mf);
-    for (int s = 0; s < p.num_splits; ++s) {
-      const float ms = __ldcg(first + s * kPart + kRows * VC + r);
-      if (ms > -INFINITY) den += exp2f(ms - mf) * __ldcg(first + s * kPart + kRows * VC + kRows + r);
-    }
-    m_s[r] = mf;
-    l_s[r] = den;
+    for (int s = 0; s < kLatMaxSplits; ++s)
+      if (s < splits) {
+        ms[s] = ld_cluster(map_to_cta(&m_s[r], s));
+        ls[s] = ld_cluster(map_to_cta(&l_s[r], s));
+      }
+#pragma unroll
+    for (int s = 0; s < kLatMaxSplits; ++s)
+      if (s < splits) mf = fmaxf(mf, ms[s]);
+#pragma unroll
+    for (int s = 0; s < kLatMaxSplits; ++s)
+      if (s < splits) {
+        ms[s] = ms[s] > -INFINITY ? exp2f(ms[s] - mf) : 0.f;
+        den += ms[s] * ls[s];
+      }
+    if (sk > -INFINITY) den += exp2f(sk - mf);
+#pragma unroll
+    for (int s = 0; s < kLatMaxSplits; ++s)
+      if (s < splits) sc_s[s][threadIdx.x] = ms[s] / den;
   }
   __syncthreads();
-  for (int i = threadIdx.x * 4; i < nh * VC; i += 512) {
+  uint32_t peer[kLatMaxSplits];
+#pragma unroll
+  for (int s = 0; s < kLatMaxSplits; ++s) peer[s] = s < splits ? map_to_cta(o_s, s) : 0u;
+#pragma unroll 2
+  for (int i = threadIdx.x * 4; consumer && i < per * VC; i += 4 * kThreads) {
     const int r = i / VC, c = i % VC;
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int s = 0; s < p.num_splits; ++s) {
-      const float* ps = first + s * kPart;
-      const float ms = __ldcg(ps + kRows * VC + r), sc = ms > -INFINITY ? exp2f(ms - m_s[r]) : 0.f;
-      const float4 x = __ldcg(reinterpret_cast<const float4*>(ps + i));
-      acc.x = fmaf(sc, x.x, acc.x); acc.y = fmaf(sc, x.y, acc.y); acc.z = fmaf(sc, x.z, acc.z); acc.w = fmaf(sc, x.w, acc.w);
-    }
-    const float inv = 1.f / l_s[r], v[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
-    __nv_bfloat16* dst = out + r * p.a.o_head + c;
+    float4 x[kLatMaxSplits];
 #pragma unroll
-    for (int e = 0; e < 4; ++e)
-      if (c + e < p.a.rank) dst[e] = __float2bfloat16(v[e]);
+    for (int s = 0; s < kLatMaxSplits; ++s)
+      if (s < splits) x[s] = ld_cluster4(peer[s] + ((r0 + r) * L::kOLd + c) * 4);
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int s = 0; s < kLatMaxSplits; ++s)
+      if (s < splits) {
+        const float sc = sc_s[s][r];
+        v[0] = fmaf(sc, x[s].x, v[0]); v[1] = fmaf(sc, x[s].y, v[1]);
+        v[2] = fmaf(sc, x[s].z, v[2]); v[3] = fmaf(sc, x[s].w, v[3]);
+      }
+    if (r0 + r >= nh) continue;
+    __nv_bfloat16* dst = out + (r0 + r) * p.a.o_head + c;
+    if (c + 3 < p.a.rank && ((p.a.o_head | p.a.o_token) & 3) == 0) {
+      *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (c + e < p.a.rank) dst[e] = __float2bfloat16(v[e]);
+    }
   }
+  cluster_sync_all();          // no CTA leaves while its sums are read
 }
 
 template <int NS, int VS, int MT>
 static int launch_latent(const CUtensorMap& tc, const LatentMmaParams& p, int tokens, cudaStream_t s) {
   using L = LatentSmem<NS, VS, MT>;
   constexpr int smem = L::kEnd + 1024;
+  static_assert(smem + 4096 <= 232448, "shared memory of a CTA");
   static bool attr_set[64] = {false};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -1;
@@ -526,7 +698,7 @@ static int launch_latent(const CUtensorMap& tc, const LatentMmaParams& p, int to
     attr_set[dev] = true;
   }
   const dim3 grid(p.num_splits, (p.a.heads + L::kRows - 1) / L::kRows, tokens);
-  return launch_pdl(latent_mma_kernel<NS, VS, MT>, grid, dim3(128), size_t(smem), s, tc, p);
+  return launch_pdl_cluster(latent_mma_kernel<NS, VS, MT>, grid, dim3(128 * MT + 32), size_t(smem), s, p.num_splits, tc, p);
 }
 template <int NS, int VS>
 static int launch_latent_heads(const CUtensorMap& tc, const LatentMmaParams& p, int tokens, cudaStream_t s) {
@@ -567,6 +739,10 @@ extern "C" int nkb_latent_append(const NkbLatentArgs* a, const NkbProj* q, const
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   using bf = __nv_bfloat16;
   const dim3 grid(tokens), block(256);
+  if (bf16 && q->bf16 && kv->bf16 && a->q_rank <= 256 * kAppendQ && a->rank <= 256 * kAppendK && a->row - a->rank <= 256 &&
+      ((a->q_rank | a->rank | a->rot | a->row) & 7) == 0 && ((q->ld | kv->ld) & 7) == 0 && al16(q->ptr) && al16(kv->ptr) &&
+      al16(q_out) && al16(cache) && al16(q_norm) && al16(kv_norm) && al16(cos_sin))
+    return launch_pdl(latent_append8_kernel, dim3((tokens + 7) / 8), block, 0, s, p, tokens);
   if (vec)
     return bf16 ? launch_pdl(latent_append_kernel<4, bf>, grid, block, smem, s, p)
                 : launch_pdl(latent_append_kernel<4, float>, grid, block, smem, s, p);
@@ -590,6 +766,9 @@ extern "C" int nkb_latent_queries(const NkbLatentArgs* a, const NkbProj* q, cons
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   using bf = __nv_bfloat16;
   const dim3 grid(unsigned((p.rows + 7) / 8)), block(256);
+  if (bf16 && q->bf16 && ((a->dim | a->rot | plain_pad | rot_pad) & 7) == 0 && (strides & 7) == 0 && (q->ld & 7) == 0 &&
+      al16(q->ptr) && al16(plain) && al16(rotated) && al16(cos_sin))
+    return launch_pdl(latent_query8_kernel, dim3(tokens), block, 0, s, p);
   if (vec)
     return bf16 ? launch_pdl(latent_query_kernel<4, bf>, grid, block, 0, s, p)
                 : launch_pdl(latent_query_kernel<4, float>, grid, block, 0, s, p);
@@ -612,38 +791,27 @@ extern "C" int nkb_latent_gather(const void* cache, const int* pages, int n_page
                     rot_ld, (float*)c_out, (float*)r_out);
 }
 
-extern "C" long long nkb_latent_scratch_floats(const NkbLatentArgs* a, int tokens, int num_splits) {
-  int vs = 0;
-  if (num_splits <= 1 || !latent_shape(*a, &vs)) return 0;
-  const int rows = a->heads <= 16 ? 16 : 32;
-  return kLatCounters + (long long)tokens * ((a->heads + rows - 1) / rows) * num_splits * (rows * vs * 64 + 2 * rows);
-}
-
 // Attention of new tokens, already in the cache, over the visible cached rows; queries and results as latents, bf16.  q_lens null:
-// token t belongs to sequence t.  Returns -5 for sizes it does not take.
+// token t belongs to sequence t.  num_splits is rounded down to 1, 2, 4 or 8.  Returns -5 for sizes it does not take.
 extern "C" int nkb_latent_attn(const NkbLatentArgs* a, const void* q, const void* cache, const int* block_table,
-                               const int* q_start, const int* q_lens, const int* context_lens, void* out, float* scratch,
-                               int batch, int tokens, int block_size, int num_blocks, int max_blocks_per_seq, int num_splits,
+                               const int* q_start, const int* q_lens, const int* context_lens, void* out, int batch,
+                               int tokens, int block_size, int num_blocks, int max_blocks_per_seq, int num_splits,
                                void* stream) {
   if (batch <= 0 || tokens <= 0) return 0;
   int vs = 0;
   const int ns = latent_shape(*a, &vs);
   if (!ns || a->row != ns * 64) return -5;
   if (!latent_ok(*a) || block_size != kLatPage || tokens > 65535 || (!q_lens && tokens != batch)) return -2;
-  if ((reinterpret_cast<uintptr_t>(q) & 3) || ((a->q_token | a->q_head) & 1) || (reinterpret_cast<uintptr_t>(out) & 3)) return -2;
+  if ((reinterpret_cast<uintptr_t>(q) & 3) || ((a->q_token | a->q_head) & 1) || (reinterpret_cast<uintptr_t>(out) & 7)) return -2;
   if (!status_word() && nkb_init() != 0) return -1;
   LatentMmaParams p{};
   p.a = *a;
-  const int rows = a->heads <= 16 ? 16 : 32;
-  if (num_splits < 1) num_splits = 1;
-  if (num_splits > 1 && (!scratch || (long long)tokens * ((a->heads + rows - 1) / rows) > kLatCounters)) return -2;
+  const int splits = num_splits >= 8 ? 8 : num_splits >= 4 ? 4 : num_splits >= 2 ? 2 : 1;
   p.q = reinterpret_cast<const __nv_bfloat16*>(q);
   p.block_table = block_table; p.q_start = q_start; p.q_lens = q_lens; p.context_lens = context_lens;
   p.out = reinterpret_cast<__nv_bfloat16*>(out);
-  p.scratch = num_splits > 1 ? scratch + kLatCounters : scratch;
-  p.counters = reinterpret_cast<unsigned int*>(scratch);
   p.status = status_word();
-  p.batch = batch; p.max_blocks = max_blocks_per_seq; p.num_splits = num_splits;
+  p.batch = batch; p.max_blocks = max_blocks_per_seq; p.num_splits = splits;
   p.scale_log2 = a->scale * 1.4426950408889634f;
   CUtensorMap tc;
   const uint64_t dims[3] = {uint64_t(a->row), uint64_t(kLatPage), uint64_t(num_blocks)};

@@ -501,7 +501,7 @@ def ligizen_config(raw: dict, **kw) -> ModelConfig:
 
 
 def ligizen_shape(width: int, *, layers: int, heads: int, kv_heads: int, ff: int, vocab: int = 32000, dim: int = 128,
-                  window: int = 1024, chunk: int = 1024, latent_dim: int = 64, rot: int = 64, kv_rank: int = 512,
+                  window: int = 1024, chunk: int = 1024, latent_dim: int = 128, rot: int = 64, kv_rank: int = 512,
                   q_rank: int = 1536, side: int = 256, experts: int = 0, top: int = 0, expert_ff: int = 0, moe_every: int = 2,
                   share_every: int = 0, **kw) -> ModelConfig:
     """A Ligizen configuration of regular shape: latent and chunked attention alternate; with experts, every `moe_every`-th

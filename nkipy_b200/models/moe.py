@@ -89,9 +89,10 @@ class MoEBlock:
                            down_bias=lw.down_bias, act_limit=cfg.swiglu_limit, act_alpha=cfg.swiglu_alpha)
 
 
-def route_splits(width: int) -> int:
-    """Split-K factor of a router's product: its few outputs are one weight tile, so several SMs share the contraction."""
-    return max(2, min(16, width // 256))
+def route_splits(width: int, tokens: int = 1) -> int:
+    """Split-K factor of a router's product: its few outputs are one weight tile, so several SMs share the contraction of a
+    row tile when there are few of those."""
+    return max(2, min(16, width // 256, 296 // max(tokens // 128, 1)))
 
 
 class RoutedExperts:
@@ -120,7 +121,7 @@ class RoutedExperts:
         """wide / narrow: results of `w_wide` and `w_narrow` when the layer has them already."""
         s, (T, W) = self.spec, h.shape
         if narrow is None:
-            z = ops.linear(h, self.w_narrow, splits=route_splits(W)) if h.dtype == torch.bfloat16 else ops.linear(h, self.w_narrow)
+            z = ops.linear(h, self.w_narrow, splits=route_splits(W, T)) if h.dtype == torch.bfloat16 else ops.linear(h, self.w_narrow)
             narrow = Proj(z, 0, self.w_narrow.shape[0])
         logits = Proj(narrow.t, narrow.col, s.experts)
         if s.score == "sigmoid":

@@ -91,8 +91,7 @@ _SIGNATURES = {
     "nkb_latent_gather": (c_int, [_P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, c_int, c_int, _P]),
     "nkb_latent_prefill": (c_int, [_P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                    c_longlong, c_longlong, c_int, c_int, c_float, c_int, _P, _P]),
-    "nkb_latent_scratch_floats": (c_longlong, [_PL, c_int, c_int]),
-    "nkb_latent_attn": (c_int, [_PL, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
+    "nkb_latent_attn": (c_int, [_PL, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
     "nkb_gated_residual": (c_int, [_P, _P, _P, c_int, c_int, c_float, c_int, ctypes.POINTER(BranchArg), _P, _P, _P,
                                    c_int, c_int, ctypes.POINTER(_P), ctypes.POINTER(_P), ctypes.POINTER(_P), c_int, c_int,
                                    c_int, c_int, c_float, _P]),

@@ -20,12 +20,11 @@ import torch
 import torch.nn.functional as F
 
 from . import _lib
-from . import _count_launch, _decode_scratch, _gather_kv, _native, _ptr, _stream, pick_kv_splits
+from . import _count_launch, _gather_kv, _native, _ptr, _stream
 from .mixers import Proj, _ref
 
 # (64-column slabs of a cached row, of its latent) the tensor-core kernel is built for
 _SHAPES = ((2, 1), (3, 2), (5, 4), (9, 8))
-_COUNTERS = 16384            # (token, group of heads) pairs whose splits can be merged
 
 
 @dataclass
@@ -62,6 +61,14 @@ class LatentSpec:
     def arg(self) -> _lib.LatentArg:
         return _lib.LatentArg(self.heads, self.dim, self.rot, self.rank, self.q_rank, self.row, float(self.eps),
                               float(self.scale), int(self.window), None, 0, 0, 0, 0)
+
+
+def _pick_splits(units: int, pages: int, sms: int = 148) -> int:
+    """CTAs (1, 2, 4 or 8) that share a token's pages: as many as leave each four pages while every SM has at most one."""
+    s = 1
+    while s < 8 and 2 * s * units <= sms and pages >= 8 * s:
+        s *= 2
+    return s
 
 
 def pair_rotate(x: torch.Tensor, cos_sin: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
@@ -179,14 +186,11 @@ def latent_attention(spec: LatentSpec, q: torch.Tensor, cache: torch.Tensor, blo
     if bf:
         a = spec.arg()
         a.sinks, a.q_token, a.q_head, a.o_token, a.o_head = _ptr(sinks), row, T * row, spec.rank, T * spec.rank
-        groups = (H + 31) // 32
         if num_splits <= 0:
             pages = block_table.shape[1] if spec.window <= 0 else min(block_table.shape[1], spec.window // bs + 2)
-            num_splits = pick_kv_splits(T * groups, pages) if T * groups <= _COUNTERS else 1
-        need = L.nkb_latent_scratch_floats(ctypes.byref(a), T, num_splits)
-        scratch = _decode_scratch(q.device, need) if need else None
+            num_splits = _pick_splits(T * ((H + 31) // 32), pages)
         rc = L.nkb_latent_attn(ctypes.byref(a), q.data_ptr(), cache.data_ptr(), block_table.data_ptr(), _ptr(q_start),
-                               _ptr(q_lens), context_lens.data_ptr(), out.data_ptr(), _ptr(scratch), B, T, bs, cache.shape[0],
+                               _ptr(q_lens), context_lens.data_ptr(), out.data_ptr(), B, T, bs, cache.shape[0],
                                block_table.stride(0), num_splits, _stream())
     if rc == -5:
         if q_lens is None:

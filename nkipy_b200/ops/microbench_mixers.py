@@ -4,10 +4,11 @@ from __future__ import annotations
 
 import torch
 
-from . import grouped_linear, linear, router_topk
+from . import grouped_linear, head_linear, linear, moe_dispatch, router_topk, softcap
+from .latent_attention import (LatentSpec, latent_append, latent_attention, latent_gather, latent_prefill, latent_queries)
 from .linear_attention import Decay, linear_attention, linear_state_shape, low_rank, token_mix
-from .mixers import (Branch, MapsSpec, Proj, activation, gate_heads, gated_act, gated_residual, heads_attention, hgrn2,
-                     hgrn2_state_shape, maps_append, maps_attention, row_norm_append)
+from .mixers import (Branch, MapsSpec, Norm, Proj, activation, gate_heads, gated_act, gated_residual, heads_attention, hgrn2,
+                     hgrn2_state_shape, maps_append, maps_attention, row_norm_append, rope_norm_append)
 
 H, G, D, V, W = 32, 8, 64, 128, 4096
 
@@ -305,6 +306,234 @@ def relu2(args, timer, sets_for):
                 shape=dict(tokens=T, ff=ff, splits=s))
 
 
+# latent attention: heads of 128 unrotated and 64 rotated dimensions, latents of 512 (keys, values) and 1536 (queries)
+LAT = dict(dim=128, rot=64, vdim=V, rank=512, q_rank=1536, scale=192 ** -0.5)
+
+
+def latent_decode(heads, window):
+    def case(args, timer, sets_for):
+        B, ctx, s = 64, 1056, LatentSpec(heads, window=window, **LAT)
+        pages, seen = (ctx + 31) // 32, min(window or ctx, ctx)
+        nb = B * pages
+        sets = sets_for(B * seen * s.row * 2, args.sets)
+        caches = [_bf16(nb, 1, 32, s.row) for _ in range(sets)]
+        table, lens = _i32(range(nb)).reshape(B, pages), torch.full((B,), ctx, device="cuda", dtype=torch.int32)
+        q, sinks = _bf16(heads, B, s.row), torch.zeros(heads, device="cuda")
+        fns = [lambda c=c: latent_attention(s, q, c, table, lens, sinks=sinks, num_splits=args.kv_splits) for c in caches]
+        return dict(case=f"latent-attn-decode-{heads}", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=B * seen * s.row * 2 + B * heads * (s.row + s.rank) * 2,
+                    flops=2.0 * B * heads * seen * (s.rank + s.rot + s.rank),
+                    shape=dict(batch=B, context=ctx, window=window, heads=heads, rank=s.rank, rot=s.rot, sets=sets))
+    return case
+
+
+def latent_pf(dim, window):
+    def case(args, timer, sets_for):
+        B, S, s = args.batch or 8, args.seq or 2048, LatentSpec(H, window=window, **{**LAT, "dim": dim})
+        T, nk = B * S, s.slabs[0]
+        q, kv, r = _bf16(T, H, 64 * nk), _bf16(T, H * (s.dim + s.vdim)), _bf16(T, s.rot)
+        start, lens, sinks = _i32(range(B)) * S, torch.full((B,), S, device="cuda", dtype=torch.int32), torch.zeros(H, device="cuda")
+        fns = [lambda: latent_prefill(s, q, kv, r, start, start, lens, lens, S, sinks)]
+        pairs = sum(min(i + 1, window or S) for i in range(S))
+        return dict(case=f"latent-attn-prefill-{dim}", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=(q.numel() + kv.numel() + r.numel() + T * H * V) * 2, flops=2.0 * B * H * pairs * (s.dim + s.rot + s.vdim),
+                    shape=dict(batch=B, seq=S, window=window, heads=H, dim=s.dim, rot=s.rot, vdim=s.vdim))
+    return case
+
+
+def chunk_pf(chunk):
+    def case(args, timer, sets_for):
+        B, S, s = args.batch or 8, args.seq or 2048, MapsSpec(H, G, V, V, V ** -0.5, maps=1, chunk=chunk)
+        nb = B * S // 32
+        k, v, q = _bf16(nb, G, 32, V), _bf16(nb, G, 32, V), _bf16(B * S, H, V)
+        table = _i32(range(nb)).reshape(B, S // 32)
+        start, lens = _i32(range(B)) * S, torch.full((B,), S, device="cuda", dtype=torch.int32)
+        fns = [lambda: heads_attention(s, q, k, v, table, lens, q_start=start, q_lens=lens, max_q_len=S)]
+        pairs = sum(i % chunk + 1 for i in range(S))
+        return dict(case="chunk-attn-prefill", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=(2 * q.numel() + k.numel() + v.numel()) * 2, flops=4.0 * B * H * pairs * V,
+                    shape=dict(batch=B, seq=S, chunk=chunk, heads=H, kv_heads=G, dim=V))
+    return case
+
+
+def chunk_decode(chunk):
+    def case(args, timer, sets_for):
+        B, ctx, s = 64, 2 * chunk, MapsSpec(H, G, V, V, V ** -0.5, maps=1, chunk=chunk)
+        pages = ctx // 32
+        nb = B * pages
+        sets = sets_for(B * chunk * G * 2 * V * 2, min(args.sets, 3))
+        caches = [(_bf16(nb, G, 32, V), _bf16(nb, G, 32, V)) for _ in range(sets)]
+        table, lens = _i32(range(nb)).reshape(B, pages), torch.full((B,), ctx, device="cuda", dtype=torch.int32)
+        q = _bf16(B, H, V)
+        fns = [lambda k=k, v=v: heads_attention(s, q, k, v, table, lens, num_splits=args.kv_splits) for k, v in caches]
+        return dict(case="chunk-attn-decode", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=B * chunk * G * 2 * V * 2, flops=4.0 * B * H * chunk * V,
+                    shape=dict(batch=B, context=ctx, chunk=chunk, heads=H, kv_heads=G, dim=V, sets=sets))
+    return case
+
+
+def latent_app(tokens, splits):
+    def case(args, timer, sets_for):
+        T, s = tokens, LatentSpec(H, window=1024, **LAT)
+        n = s.q_rank + s.rank + s.rot
+        y = torch.randn(splits, T, n + H, device="cuda") if splits else _bf16(T, n + H)
+        cache, slots = _bf16(max(T // 32, 1) + 8, 1, 32, s.row), _i32(range(T))
+        table, pos = torch.randn(4096, s.rot, device="cuda"), _i32(range(T)) % 4096
+        qn, kn = torch.ones(s.q_rank, device="cuda"), torch.ones(s.rank, device="cuda")
+        fns = [lambda: latent_append(s, Proj(y, 0, s.q_rank), Proj(y, s.q_rank, s.rank + s.rot), qn, kn, table, pos, slots, cache)]
+        return dict(case=f"latent-append-{T}", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=T * n * ((4 * splits if splits else 2) + 2), flops=0.0,
+                    shape=dict(tokens=T, q_rank=s.q_rank, rank=s.rank, rot=s.rot, splits=splits))
+    return case
+
+
+def latent_q(tokens, splits):
+    def case(args, timer, sets_for):
+        T, s = tokens, LatentSpec(H, window=1024, **LAT)
+        n = H * (s.dim + s.rot)
+        y = torch.randn(splits, T, n, device="cuda") if splits else _bf16(T, n)
+        table, pos = torch.randn(4096, s.rot, device="cuda"), _i32(range(T)) % 4096
+        if splits:
+            q = _bf16(H, T, s.row)
+            plain, rot = _bf16(H, T, s.dim).transpose(0, 1), q.transpose(0, 1)[..., s.rank:]
+        else:
+            q = _bf16(T, H, 64 * s.slabs[0])
+            plain, rot = q[..., :-64], q[..., -64:]
+        fns = [lambda: latent_queries(s, Proj(y, 0, n), table, pos, plain, rot)]
+        return dict(case=f"latent-queries-{T}", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=T * n * ((4 * splits if splits else 2) + 2), flops=0.0,
+                    shape=dict(tokens=T, heads=H, dim=s.dim, rot=s.rot, splits=splits))
+    return case
+
+
+def latent_rows(args, timer, sets_for):
+    P, s = 512, LatentSpec(H, window=1024, **LAT)
+    cache = _bf16(2 * P, 1, 32, s.row)
+    pages = torch.randperm(2 * P, device="cuda").to(torch.int32)[:P].contiguous()
+    fns = [lambda: latent_gather(s, cache, pages, s.rot)]
+    return dict(case="latent-gather-16384", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                bytes=4 * P * 32 * (s.rank + s.rot), flops=0.0, shape=dict(pages=P, rank=s.rank, rot=s.rot))
+
+
+def fold(k, n, name):
+    def case(args, timer, sets_for):
+        T = 64
+        sets = sets_for(H * n * k * 2, 32)
+        ws, x = [_bf16(H, n, k, scale=0.05) for _ in range(sets)], _bf16(H, T, k)
+        fns = [lambda w=w: head_linear(x, w) for w in ws]
+        return dict(case=name, us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=H * (n * k + T * (n + k)) * 2, flops=2.0 * H * T * n * k, shape=dict(tokens=T, heads=H, k=k, n=n, sets=sets))
+    return case
+
+
+def rope_append(tokens, splits):
+    def case(args, timer, sets_for):
+        T, s = tokens, MapsSpec(H, G, V, V, V ** -0.5, maps=1, chunk=1024)
+        nb, n = max(T // 32, 1) + 8, V * (H + 2 * G)
+        k, v = _bf16(nb, G, 32, V), _bf16(nb, G, 32, V)
+        y = torch.randn(splits, T, n + H, device="cuda") if splits else _bf16(T, n + H)
+        slots, bias = _i32(range(T)), torch.randn(n, device="cuda")
+        table, pos = torch.randn(4096, V, device="cuda"), _i32(range(T)) % 4096
+        fns = [lambda: rope_norm_append(s, Proj(y, 0, H * V), Proj(y, H * V, G * V), Proj(y, (H + G) * V, G * V), bias, table, pos,
+                                        slots, k, v)]
+        return dict(case=f"rope-norm-append-{T}", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=T * n * ((4 * splits if splits else 2) + 2), flops=0.0,
+                    shape=dict(tokens=T, heads=H, kv_heads=G, dim=V, splits=splits))
+    return case
+
+
+def head_gates(tokens):
+    def case(args, timer, sets_for):
+        T = tokens
+        x, g = _bf16(T, H, V), _bf16(T, H)
+        fns = [lambda: gate_heads(x, Proj(g, 0, H), "sigmoid")]
+        return dict(case=f"head-gates-{T}", us=timer(fns, args.iters, args.warmup, not args.no_graph), bytes=T * W * 4,
+                    flops=0.0, shape=dict(tokens=T, heads=H, width=V))
+    return case
+
+
+def side_residual(tokens, splits):
+    def case(args, timer, sets_for):
+        T = tokens
+        y = torch.randn(splits, T, W, device="cuda") if splits else _bf16(T, W)
+        x, n, b = torch.randn(T, W, device="cuda"), torch.ones(W, device="cuda"), torch.zeros(W, device="cuda")
+        fns = [lambda: gated_residual(x, [Branch(Proj(y, 0, W), norm=n)], norms=[Norm(n, b, True)], eps=1e-6)]
+        return dict(case=f"normed-residual-{tokens}", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=T * W * ((4 * splits if splits else 2) + 10), flops=0.0, shape=dict(tokens=T, width=W, splits=splits))
+    return case
+
+
+def parallel_residual(tokens, splits, routed):
+    def case(args, timer, sets_for):
+        T, k = tokens, 4
+        part = lambda: torch.randn(splits, T, W, device="cuda") if splits else _bf16(T, W)
+        x, br = torch.randn(T, W, device="cuda"), [Branch(Proj(part(), 0, W))]
+        per = 4 * splits if splits else 2
+        size = per
+        if routed:
+            rows, pos = _bf16(T * k, W), torch.randperm(T * k, device="cuda").to(torch.int32)
+            gate = torch.randn(2, T, 40, device="cuda")
+            br += [Branch(Proj(rows, 0, W), pair_pos=pos, top_k=k), Branch(Proj(part(), 0, W), Proj(gate, 32, 1))]
+            size += 2 * k + per
+        else:
+            br.append(Branch(Proj(part(), 0, W)))
+            size += per
+        fns = [lambda: gated_residual(x, br, norms=[Norm()])]
+        name = "shared-routed-residual" if routed else "parallel-residual"
+        return dict(case=f"{name}-{tokens}", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=T * W * (size + 10), flops=0.0, shape=dict(tokens=T, width=W, splits=splits, top=k if routed else 0))
+    return case
+
+
+def table_act(tokens, splits):
+    def case(args, timer, sets_for):
+        T, n, L, vocab = tokens, 256, 16, 32000
+        z = torch.randn(splits, T, n, device="cuda") if splits else _bf16(T, n)
+        table, ids = _bf16(vocab, L * n), torch.randint(0, vocab, (T,), device="cuda", dtype=torch.int32)
+        fns = [lambda i=i: gated_act(Proj(z, 0, n), Proj(table, i * n, n), "gelu_tanh", up_rows=ids) for i in range(4)]
+        return dict(case=f"table-act-{T}", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=T * n * ((4 * splits if splits else 2) + 4), flops=0.0, shape=dict(tokens=T, width=n, splits=splits))
+    return case
+
+
+def clamped_act(tokens, splits):
+    def case(args, timer, sets_for):
+        T, ff = tokens, 1792
+        y = torch.randn(splits, T, 2 * ff, device="cuda") if splits else _bf16(T, 2 * ff)
+        fns = [lambda: gated_act(Proj(y, 0, ff), Proj(y, ff, ff), "clamped", limit=7.0)]
+        return dict(case=f"clamped-act-{T}", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=T * ff * (2 * (4 * splits if splits else 2) + 2), flops=0.0, shape=dict(tokens=T, ff=ff, splits=splits))
+    return case
+
+
+def sigmoid_router(tokens, splits):
+    def case(args, timer, sets_for):
+        T, E = tokens, 32
+        z = torch.randn(splits, T, E + 8, device="cuda")
+        fns = [lambda: router_topk(Proj(z, 0, E), 4, "sigmoid_topk")]
+        return dict(case=f"sigmoid-router-{T}", us=timer(fns, args.iters, args.warmup, not args.no_graph), bytes=splits * T * E * 4,
+                    flops=0.0, shape=dict(tokens=T, experts=E, top=4, splits=splits))
+    return case
+
+
+def scaled_dispatch(tokens, scaled):
+    def case(args, timer, sets_for):
+        T, k, E = tokens, 4, 32
+        x, e = _bf16(T, W), torch.rand(T, E, device="cuda").topk(k, dim=-1).indices.to(torch.int32)
+        w = torch.rand(T, k, device="cuda") if scaled else None
+        fns = [lambda: moe_dispatch(x, e, 0, E, weights=w)]
+        return dict(case=f"{'scaled' if scaled else 'plain'}-dispatch-{T}", us=timer(fns, args.iters, args.warmup, not args.no_graph),
+                    bytes=T * W * 2 * (k + 1), flops=0.0, shape=dict(tokens=T, width=W, experts=E, top=k))
+    return case
+
+
+def cap(args, timer, sets_for):
+    z = torch.randn(64, 32000, device="cuda")
+    fns = [lambda: softcap(z, 30.0)]
+    return dict(case="softcap-64", us=timer(fns, args.iters, args.warmup, not args.no_graph), bytes=z.numel() * 8, flops=0.0,
+                shape=dict(rows=64, vocab=32000))
+
+
 CASES = {"maps-attn-decode": maps_decode, "maps-attn-prefill": maps_prefill(30.0),
          "maps-attn-prefill-large-scores": maps_prefill(30.0, 8.0, "maps-attn-prefill-large-scores"),
          "maps-attn-prefill-nocap": maps_prefill(0.0, 1.0, "maps-attn-prefill-nocap"), "maps-append": append,
@@ -317,4 +546,21 @@ CASES = {"maps-attn-decode": maps_decode, "maps-attn-prefill": maps_prefill(30.0
          "grouped-projections-64": each, "residual-64": plain_residual(64, 8), "residual-16384": plain_residual(16384, 0),
          "routed-residual-64": routed_residual(64), "routed-residual-16384": routed_residual(16384),
          "group-router-64": router(64), "group-router-16384": router(16384), "low-rank-64": decay_logits(64),
-         "low-rank-16384": decay_logits(16384), "gemm-prefill-relu2": relu2_gemm, "relu2-64": relu2}
+         "low-rank-16384": decay_logits(16384), "gemm-prefill-relu2": relu2_gemm, "relu2-64": relu2,
+         "latent-attn-decode-32": latent_decode(32, 1024), "latent-attn-decode-16": latent_decode(16, 1024),
+         "latent-attn-prefill-128": latent_pf(128, 1024), "latent-attn-prefill-64": latent_pf(64, 1024),
+         "chunk-attn-prefill": chunk_pf(1024), "chunk-attn-decode": chunk_decode(1024),
+         "latent-append-64": latent_app(64, 4), "latent-append-16384": latent_app(16384, 0), "latent-queries-64": latent_q(64, 4),
+         "latent-queries-16384": latent_q(16384, 0), "latent-gather-16384": latent_rows,
+         "fold-queries-64": fold(128, 512, "fold-queries-64"), "expand-values-64": fold(512, 128, "expand-values-64"),
+         "rope-norm-append-64": rope_append(64, 4), "rope-norm-append-16384": rope_append(16384, 0),
+         "head-gates-64": head_gates(64), "head-gates-16384": head_gates(16384), "normed-residual-64": side_residual(64, 4),
+         "normed-residual-16384": side_residual(16384, 0), "parallel-residual-64": parallel_residual(64, 8, False),
+         "parallel-residual-16384": parallel_residual(16384, 0, False),
+         "shared-routed-residual-64": parallel_residual(64, 8, True),
+         "shared-routed-residual-16384": parallel_residual(16384, 0, True), "table-act-64": table_act(64, 8),
+         "table-act-16384": table_act(16384, 0), "clamped-act-64": clamped_act(64, 4),
+         "clamped-act-16384": clamped_act(16384, 0), "sigmoid-router-64": sigmoid_router(64, 4),
+         "sigmoid-router-16384": sigmoid_router(16384, 2), "scaled-dispatch-64": scaled_dispatch(64, True),
+         "scaled-dispatch-16384": scaled_dispatch(16384, True), "plain-dispatch-64": scaled_dispatch(64, False),
+         "plain-dispatch-16384": scaled_dispatch(16384, False), "softcap-64": cap}

@@ -182,3 +182,60 @@ def forward(raw, weights, ids):
         taps.append(x)
     logits = layer_norm(x, W["final.norm"], W["final.norm.b"], eps) @ W["head"].T
     return softcap(logits, raw["logit_softcap"]), taps
+
+
+# ----------------------------------------------------------------------------- small models for the tests
+def small_config(width=96, vocab=160, layers="lcLk", mlps="dmsd", heads=4, kv_heads=2, dim=24, vdim=40, chunk=21, scale=None,
+                 rot=16, scaling=(8.0, 1.0, 4.0, 64), lheads=3, ldim=20, lrot=8, lvdim=24, rank=40, q_rank=56, window=27,
+                 lscale=None, ff=112, experts=6, top=2, eff=40, limit=1.2, sff=48, slimit=0.8, side=24, cap=20.0, escale=3.0,
+                 eps=1e-5):
+    """config.json contents.  Layers: 'l' latent attention, 'L' the same with other sizes, 'c' chunked attention, 'k' chunked
+    attention on the keys of the last 'c' (with a chunk of its own); mlps: 'd' dense, 'm' routed with a shared expert, 's'
+    routed without, '-' none."""
+    specs, source = [], None
+    for i, (c, f) in enumerate(zip(layers, mlps)):
+        if c in "lL":
+            kind, wide = "latent_attention", c == "L"
+            m = {"heads": lheads + 2 * wide, "dim": ldim, "rot_dim": lrot, "vdim": lvdim + 8 * wide, "kv_rank": rank + 16 * wide,
+                 "q_rank": q_rank, "mask": {"size": window + 10 * wide}, "scale": lscale or 2 * (ldim + lrot) ** -0.5,
+                 "rot": {"base": 3000.0, "dims": lrot}}
+        else:
+            kind = "attention"
+            m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": chunk + 6 * (c == "k")},
+                 "scale": scale or 2 * dim ** -0.5, "rot": {"base": 700.0, "dims": rot}}
+            if scaling:
+                m["rot"]["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+            if c == "k":
+                m["kv_from"] = source
+            else:
+                source = i
+        mlp = {"d": {"kind": "dense", "ff": ff}, "-": None}.get(f, {
+            "kind": "moe", "expert": {"ff": eff, "limit": limit}, "router": {"experts": experts, "top": top}})
+        if f == "m":
+            mlp["shared"] = {"ff": sff, "limit": slimit}
+        specs.append({"type": kind, "mixer": m, "mlp": mlp})
+    return {"architecture": "Ligizen", "embedding": {"scale": escale}, "layers": specs, "logit_softcap": cap,
+            "norm": {"eps": eps}, "token_side": {"dim": side}, "vocab": vocab, "width": width}
+
+
+def small_weights(raw, shapes, seed=0):
+    """bf16 tensors of the given name -> shape map, scaled so that every mechanism has a visible effect: scores of several
+    units, sinks that take a share, clamps that bite, decided routers, biases of the size of what they are added to."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in shapes.items():
+        x, leaf = torch.randn(shape, generator=g), name.rsplit(".", 1)[-1]
+        if name.endswith(".sink"):
+            x = 1 + x
+        elif leaf == "b":
+            x = 0.5 * x
+        elif leaf in ("norm1", "norm"):
+            x = 1 + 0.3 * x
+        elif leaf == "router":
+            x = x * 4 / shape[-1] ** 0.5
+        elif leaf in ("gate", "up") and ".side." not in name:
+            x = x * 1.5 / shape[-1] ** 0.5
+        elif len(shape) == 2 and name not in ("embed", "side.embed"):
+            x = x / shape[-1] ** 0.5
+        out[name] = x.to(torch.bfloat16)
+    return out
