@@ -84,23 +84,6 @@ struct PrefillCtrl {
   int abort;
 };
 
-// Four MMAs (k-steps) of one accumulator as one instruction sequence, descriptors prepared beforehand.
-__device__ __forceinline__ void umma4_ss(uint32_t d, const uint64_t (&a)[4], const uint64_t (&b)[4], uint32_t idesc,
-                                         uint32_t acc_first) {
-  asm volatile(
-      "{\n"
-      ".reg .pred p0, p1;\n"
-      "setp.ne.b32 p0, %10, 0;\n"
-      "setp.eq.b32 p1, %9, %9;\n"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %5, %9, p0;\n"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %2, %6, %9, p1;\n"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %3, %7, %9, p1;\n"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %4, %8, %9, p1;\n"
-      "}\n" ::"r"(d),
-      "l"(a[0]), "l"(a[1]), "l"(a[2]), "l"(a[3]), "l"(b[0]), "l"(b[1]), "l"(b[2]), "l"(b[3]), "r"(idesc), "r"(acc_first)
-      : "memory");
-}
-
 // Bounded barrier wait whose slow path (timer, abort flag) is one shared out-of-line function: the kernel has two
 // dozen waits and their inlined loops would push the hot code out of the instruction cache.
 __device__ __noinline__ bool pf_wait_slow(uint64_t* bar, uint32_t parity, volatile int* abort_flag, int* status,

@@ -281,6 +281,23 @@ __device__ __forceinline__ void umma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, ui
       "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate)
       : "memory");
 }
+// Four MMAs (k-steps) of one accumulator as one instruction sequence, descriptors prepared beforehand.
+__device__ __forceinline__ void umma4_ss(uint32_t d, const uint64_t (&a)[4], const uint64_t (&b)[4], uint32_t idesc,
+                                         uint32_t acc_first) {
+  asm volatile(
+      "{\n"
+      ".reg .pred p0, p1;\n"
+      "setp.ne.b32 p0, %10, 0;\n"
+      "setp.eq.b32 p1, %9, %9;\n"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %5, %9, p0;\n"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %2, %6, %9, p1;\n"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %3, %7, %9, p1;\n"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %4, %8, %9, p1;\n"
+      "}\n" ::"r"(d),
+      "l"(a[0]), "l"(a[1]), "l"(a[2]), "l"(a[3]), "l"(b[0]), "l"(b[1]), "l"(b[2]), "l"(b[3]), "r"(idesc), "r"(acc_first)
+      : "memory");
+}
+
 // Arrive on an mbarrier once all previously issued MMAs of this thread finished.
 __device__ __forceinline__ void umma_commit(uint64_t* bar) {
   asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar))

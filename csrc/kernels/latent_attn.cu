@@ -3,9 +3,8 @@
 //             shared key part rotated (pairs 2i, 2i + 1) into the token's cache row
 //   queries   the up-projected queries split into their unrotated and rotated parts, the latter rotated
 //   gather    cached rows of whole pages as two matrices, the operands of the up projections of keys and values
-//   attention any new tokens against the cached rows themselves, bf16: see latent_mma_kernel
+//   attention any new tokens against the cached rows themselves, bf16: see latent_attn_kernel
 #include "common.cuh"
-#include "mma_frag.cuh"
 #include "proj_src.cuh"
 #include "latent_attn.h"
 #include "attn_maps.h"
@@ -345,19 +344,20 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const T* __restrict_
 }
 
 // ------------------------------------------------------------------------------------------------ attention
-// One CTA of 4 MT consumer warps and a TMA warp per (split of the visible pages, 16 MT heads, new token).  A page's rows come in once by TMA (slabs of
-// 64 columns, 128-byte swizzle) and serve as keys and as values of all heads.  A warp belongs to 16 heads and a quarter of the
-// columns (16 of every 64, so that all its addresses are a constant offset from one):
-//   scores   contracts its quarter of the row; the queries stay in registers as MMA fragments.  The four partial products
-//            of a head meet in shared memory.
-//   softmax  eight threads per head sum the partials, mask, and keep the running maximum and denominator
-//   values   multiplies the probabilities with its quarter of the latent
-// A page is mostly latency (loads of fragments, chains of products, exchanges), so the scores of page i + 1 are contracted
-// between the softmax and the values of page i: one barrier per page hands over both, with two buffers of each.  The ring
-// takes most of the shared memory, because a page arrives a microsecond and more after its load was issued.  The splits of a token are a cluster: each leaves its unnormalised sums in shared memory, and
-// each adds up a share of the heads from all of them.
-// NS: slabs of a row; VS: slabs of its latent.
+// One CTA per (split of the visible pages, N heads, new token).  A page of 32 tokens comes in once by TMA (slabs of 64 columns,
+// 128-byte swizzle) and serves as keys and as values of all N heads:
+//   scores   S [heads, tokens] = Q C^T      Q the heads' queries, resident in tensor memory; C the page as it lies (K-major)
+//   values   O^T [latent, N] += C^T P^T     C^T the same page read MN-major, P the probabilities (K-major): transposed, so that
+//                                           the latent's columns and not the few heads are the 128-row side
+// so that every product reads the page's shared memory at most once.  Warp 0 loads; one thread of warp 1 issues S of the next
+// page ahead of O^T of this one; warp 4 holds a head per thread (lanes past N heads compute on whatever tensor memory holds
+// there, and nobody reads it).  A head's reference for its exponentials is only raised when its maximum has grown by more than
+// 2^8 since it was last set (see attn_prefill.cu); warps 4-7 then rescale O^T in tensor memory.
+// The splits of a token are a cluster: each leaves its unnormalised sums in shared memory, and each adds up a share of the
+// heads from all of them.  NS: slabs of a row; VS: slabs of its latent.
 constexpr int kLatMaxSplits = 8;
+constexpr float kLatRescaleStep = 8.f;
+enum { LAT_STEADY = 0, LAT_RAISE = 1, LAT_ABORT = 2 };
 
 struct LatentMmaParams {
   NkbLatentArgs a;
@@ -369,16 +369,20 @@ struct LatentMmaParams {
   float scale_log2;
 };
 
-template <int NS, int VS, int MT>
+template <int NS, int VS, int N>
 struct LatentSmem {
-  static constexpr int kSlab = kLatPage * 128, kStage = NS * kSlab, kStages = NS >= 9 ? 5 : 6;
-  static constexpr int kRows = 16 * MT, kSLd = 36, kPLd = 40;      // leading dimensions of scores (fp32) and probabilities
-  static constexpr int kScores = kStages * kStage;
-  static constexpr int kScoreBytes = 4 * kRows * kSLd * 4, kProbBytes = kRows * kPLd * 2;
-  static constexpr int kProbs = kScores + 2 * kScoreBytes;
-  static constexpr int kEnd = kProbs + 2 * kProbBytes;
+  static constexpr int kSlab = kLatPage * 128, kStage = NS * kSlab;
+  static constexpr int kStages = NS >= 5 ? 5 : 8;
+  static constexpr int kProb = N * 128;
+  static constexpr int kP = kStages * kStage;                      // two buffers
+  static constexpr int kEnd = kP + 2 * kProb;
   static constexpr int kOLd = VS * 64 + 8;                         // of the sums that splits exchange, in the ring's place
-  static_assert(kRows * kOLd * 4 <= kScores, "sums fit in the ring");
+  static constexpr int kTiles = (VS + 1) / 2;                      // 128-row tiles of O^T
+  // tensor memory: two buffers of S, the queries (two elements a column), O^T
+  static constexpr int kSCol = 0, kQCol = 2 * kLatPage, kOCol = kQCol + NS * 32;
+  static constexpr int kUsed = kOCol + kTiles * N;
+  static constexpr int kCols = kUsed <= 128 ? 128 : (kUsed <= 256 ? 256 : 512);
+  static_assert(N * kOLd * 4 <= kP && kUsed <= 512, "what splits exchange fits in the ring");
 };
 
 __device__ __forceinline__ float ld_cluster(uint32_t addr) {
@@ -391,36 +395,65 @@ __device__ __forceinline__ float4 ld_cluster4(uint32_t addr) {
   asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr) : "memory");
   return v;
 }
-
-template <int NS, int VS, int MT>
-__global__ void __launch_bounds__(128 * MT + 32, 1)
-latent_mma_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ LatentMmaParams p) {
-  using L = LatentSmem<NS, VS, MT>;
-  constexpr int kRows = L::kRows, VC = VS * 64, kThreads = 128 * MT, TPR = 8, PER = kLatPage / TPR;
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+template <int N>
+__device__ __forceinline__ void tmem_ld_cols(uint32_t addr, uint32_t (&r)[N]) {
+  if constexpr (N == 32) tmem_ld_32x32(addr, r);
+  else tmem_ld_32x16(addr, r);
+}
+template <int N>
+__device__ __forceinline__ void tmem_st_cols(uint32_t addr, const uint32_t (&r)[N]) {
+  if constexpr (N == 32) tmem_st_32x32(addr, r);
+  else tmem_st_32x16(addr, r);
+}
+template <int NS, int VS, int N>
+__global__ void __launch_bounds__(256, 1)
+latent_attn_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ LatentMmaParams p) {
+  using L = LatentSmem<NS, VS, N>;
+  constexpr int VC = VS * 64;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  float* s_s = reinterpret_cast<float*>(smem + L::kScores);                       // [2][4][kRows][kSLd]
-  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(smem + L::kProbs);        // [2][kRows][kPLd]
-  __shared__ uint64_t full[L::kStages], empty[L::kStages];
-  __shared__ float al_s[2][kRows], m_s[kRows], l_s[kRows];
-  __shared__ float sc_s[kLatMaxSplits][kRows];
-  __shared__ int abort_flag;
-  const int mt = threadIdx.x >> 7, quarter = (threadIdx.x >> 5) & 3, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
-  const int split = blockIdx.x, head0 = blockIdx.y * kRows, t = blockIdx.z;
-  const int nh = min(kRows, p.a.heads - head0);
+  uint8_t* p_s = smem + L::kP;
+  __shared__ uint64_t q_ready, kv_full[L::kStages], kv_empty[L::kStages], s_full[2], s_empty[2], p_full[2], p_empty[2];
+  __shared__ uint32_t tmem_s;
+  __shared__ __align__(16) float raise_s[N], m_s[N], l_s[N], sc_s[kLatMaxSplits][N];
+  __shared__ int abort_s, state_s[2];
+  const int warp = warp_idx_uniform(), lane = threadIdx.x & 31;
+  const int split = blockIdx.x, head0 = blockIdx.y * N, t = blockIdx.z;
+  const int nh = min(N, p.a.heads - head0);
   if (threadIdx.x == 0) {
+    tma_prefetch_desc(&tmC);
+    mbar_init(&q_ready, 1);
     for (int s = 0; s < L::kStages; ++s) {
-      mbar_init(&full[s], 1);
-      mbar_init(&empty[s], 4 * MT);
+      mbar_init(&kv_full[s], 1);
+      mbar_init(&kv_empty[s], 1);
     }
-    abort_flag = 0;
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&s_full[i], 1);
+      mbar_init(&s_empty[i], 1);
+      mbar_init(&p_full[i], 4);
+      mbar_init(&p_empty[i], 1);
+    }
+    abort_s = 0;
     mbar_fence_init();
     fence_proxy_async();
-    tma_prefetch_desc(&tmC);
   }
-  __syncthreads();
   griddep_wait();
+  // between the two: neither the kernel before this one nor the one after it can wait for tensor memory that this one holds
+  if (warp == 1) {
+    tmem_alloc(&tmem_s, L::kCols);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
   griddep_launch();
+  const uint32_t tmem = __shfl_sync(0xffffffffu, tmem_s, 0);
+  volatile int* abort_flag = &abort_s;
   int b = -1, pos = -1;
   if (!p.q_lens) {
     b = t;
@@ -437,200 +470,238 @@ latent_mma_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant
   __nv_bfloat16* out = p.out + t * p.a.o_token + head0 * p.a.o_head;
   if (pos < 0) {
     if (split == 0)
-      for (int i = threadIdx.x; i < nh * p.a.rank; i += blockDim.x)
+      for (int i = threadIdx.x; i < nh * p.a.rank; i += 256)
         out[(i / p.a.rank) * p.a.o_head + i % p.a.rank] = __float2bfloat16(0.f);
+    if (warp == 1) tmem_dealloc(tmem, L::kCols);
     return;
   }
   const int lo = nkb_first_visible(pos, p.a.window, 0);
   const int page_lo = lo / kLatPage, npages = pos / kLatPage + 1 - page_lo;
   const int per_split = (npages + p.num_splits - 1) / p.num_splits;
   const int p0 = page_lo + split * per_split, n = max(0, min(page_lo + npages, p0 + per_split) - p0);
-  const int* table = p.block_table + (long long)b * p.max_blocks;
-  const bool consumer = threadIdx.x < kThreads;
-  if (!consumer) {
-    int blk = n > 0 ? table[p0] : 0;
+
+  if (warp == 0) {
+    // ---------------------------------------------------------------- loads
+    const int* table = p.block_table + (long long)b * p.max_blocks;
+    int next = n > 0 ? table[p0] : 0;
     for (int i = 0; i < n; ++i) {
-      const int st = i % L::kStages, next = i + 1 < n ? table[p0 + i + 1] : 0;
-      const bool ok = mbar_wait(&empty[st], (uint32_t(i / L::kStages) & 1u) ^ 1u, &abort_flag, p.status, ERR_WAIT_SMEM_EMPTY);
+      const int st = i % L::kStages, blk = next;
+      if (i + 1 < n) next = table[p0 + i + 1];
+      const bool ok = mbar_wait(&kv_empty[st], (uint32_t(i / L::kStages) & 1u) ^ 1u, abort_flag, p.status, ERR_WAIT_SMEM_EMPTY);
       if (!__all_sync(0xffffffffu, ok)) break;
       if (lane == 0) {
-        mbar_expect_tx(&full[st], L::kStage);
+        uint8_t* dst = smem + st * L::kStage;
+        mbar_expect_tx(&kv_full[st], L::kStage);
 #pragma unroll
-        for (int s = 0; s < NS; ++s) tma_load_3d(smem + st * L::kStage + s * L::kSlab, &tmC, &full[st], s * 64, 0, blk);
+        for (int s = 0; s < NS; ++s) tma_load_3d(dst + s * L::kSlab, &tmC, &kv_full[st], s * 64, 0, blk);
       }
       __syncwarp();
-      blk = next;
     }
-  }
-
-  uint32_t qf[NS][4];
-  if (consumer) {
-    const int r0 = mt * 16 + g, r1 = r0 + 8;
-    const __nv_bfloat16* q0 = p.q + t * p.a.q_token + (head0 + r0) * p.a.q_head;
-    const __nv_bfloat16* q1 = q0 + 8 * p.a.q_head;
+  } else if (warp == 1) {
+    // ---------------------------------------------------------------- products
+    constexpr uint32_t idesc_s = make_idesc_bf16(128, kLatPage, 0, 0), idesc_o = make_idesc_bf16(128, N, 1, 0);
+    const uint64_t hk = uint64_t(uint32_t(make_smem_desc_sw128(0, 0, 1024) >> 32)) << 32;      // SBO, version, swizzle
+    const uint32_t c_lo = uint32_t(make_smem_desc_sw128(smem_u32(smem), 0, 1024));
+    const uint32_t p_lo = uint32_t(make_smem_desc_sw128(smem_u32(p_s), 0, 1024));
+    constexpr uint32_t lbo = (uint32_t(L::kSlab) >> 4) << 16;                                    // next 64 columns of C^T
+    if (n > 0 && elect_one()) {
+      bool ok = mbar_wait(&q_ready, 0, abort_flag, p.status, ERR_WAIT_SOFTMAX);
+      const auto scores = [&](int i) {
+        const int st = i % L::kStages, buf = i & 1;
+        ok = ok && mbar_wait(&kv_full[st], uint32_t(i / L::kStages) & 1u, abort_flag, p.status, ERR_WAIT_SMEM_FULL);
+        ok = ok && mbar_wait(&s_empty[buf], (uint32_t(i / 2) & 1u) ^ 1u, abort_flag, p.status, ERR_WAIT_TMEM_EMPTY);
+        if (!ok) return;
+        tc_fence_after();
 #pragma unroll
-    for (int k = 0; k < NS; ++k) {
-      const int c = (4 * k + quarter) * 16 + 2 * tq;
-      qf[k][0] = r0 < nh ? *reinterpret_cast<const uint32_t*>(q0 + c) : 0u;
-      qf[k][1] = r1 < nh ? *reinterpret_cast<const uint32_t*>(q1 + c) : 0u;
-      qf[k][2] = r0 < nh ? *reinterpret_cast<const uint32_t*>(q0 + c + 8) : 0u;
-      qf[k][3] = r1 < nh ? *reinterpret_cast<const uint32_t*>(q1 + c + 8) : 0u;
+        for (int k = 0; k < 4 * NS; ++k)
+          umma_f16_ts(tmem + L::kSCol + buf * kLatPage, tmem + L::kQCol + k * 8,
+                      hk | (c_lo + uint32_t((st * L::kStage + (k >> 2) * L::kSlab) >> 4) + (k & 3) * 2), idesc_s, k > 0 ? 1u : 0u);
+        umma_commit(&s_full[buf]);
+      };
+      scores(0);
+      for (int i = 0; i < n && ok; ++i) {
+        if (i + 1 < n) scores(i + 1);
+        const int st = i % L::kStages, buf = i & 1;
+        ok = ok && mbar_wait(&p_full[buf], uint32_t(i / 2) & 1u, abort_flag, p.status, ERR_WAIT_SOFTMAX);
+        if (!ok) break;
+        tc_fence_after();
+#pragma unroll
+        for (int m = 0; m < L::kTiles; ++m) {
+#pragma unroll
+          for (int k = 0; k < 2; ++k)              // sixteen tokens a step
+            umma_f16(tmem + L::kOCol + m * N, hk | ((c_lo + uint32_t((st * L::kStage + 2 * m * L::kSlab) >> 4) + k * 128) | lbo),
+                     hk | (p_lo + uint32_t(buf * L::kProb >> 4) + k * 2), idesc_o, i > 0 || k > 0 ? 1u : 0u);
+        }
+        umma_commit(&p_empty[buf]);
+        umma_commit(&kv_empty[st]);
+      }
     }
-  }
-  float o[2 * VS][4];
+    __syncwarp();
+  } else if (warp >= 4) {
+    // ---------------------------------------------------------------- softmax
+    const int quad = warp & 3, tok = quad * 32 + lane;
+    const uint32_t lanes = uint32_t(quad * 32) << 16;
+    const bool holds = quad == 0;                   // the warp with the heads
+    if (holds && n > 0) {
+      // queries of head `lane` -> tensor memory, half a row's slabs at a time so that their loads are in flight together
+      const uint4* q = reinterpret_cast<const uint4*>(p.q + t * p.a.q_token + (head0 + lane) * p.a.q_head);
+      constexpr int kHalf = (NS + 1) / 2;
 #pragma unroll
-  for (int i = 0; i < 2 * VS; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  const int row = threadIdx.x / TPR, sub = threadIdx.x % TPR;
-  float m = -INFINITY, l = 0.f;
-  // fragment addresses within a slab: keys (two groups of eight tokens by sixteen columns), values (transposed)
-  const uint32_t k_off = ((lane >> 4) * 8 + (lane & 7)) * 128 + (((2 * quarter + ((lane >> 3) & 1)) ^ (lane & 7)) << 4);
-  const uint32_t v_off = (lane & 15) * 128 + (((2 * quarter + (lane >> 4)) ^ (lane & 7)) << 4);
-
-  // partial scores of page i -> buffer i & 1; returns whether the page arrived
-  const auto scores = [&](int i) {
-    const int st = i % L::kStages;
-    const bool ok = mbar_wait(&full[st], uint32_t(i / L::kStages) & 1u, &abort_flag, p.status, ERR_WAIT_SMEM_FULL);
-    const uint32_t base = smem_u32(smem + st * L::kStage) + k_off;
-    float s[4][4];
+      for (int s0 = 0; s0 < NS; s0 += kHalf) {
+        uint32_t r[kHalf][32];
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
-    uint32_t kb[2][8];                // fragments of one step are loaded while the step before is multiplied
-    ldsm_x4(base, kb[0][0], kb[0][1], kb[0][2], kb[0][3]);
-    ldsm_x4(base + 2048, kb[0][4], kb[0][5], kb[0][6], kb[0][7]);
+        for (int s = 0; s < kHalf; ++s)
 #pragma unroll
-    for (int k = 0; k < NS; ++k) {
-      if (k + 1 < NS) {
-        uint32_t(&d)[8] = kb[(k + 1) & 1];
-        ldsm_x4(base + (k + 1) * L::kSlab, d[0], d[1], d[2], d[3]);
-        ldsm_x4(base + (k + 1) * L::kSlab + 2048, d[4], d[5], d[6], d[7]);
+          for (int c = 0; c < 8; ++c) {
+            const uint4 w = s0 + s < NS && lane < nh ? q[(s0 + s) * 8 + c] : make_uint4(0u, 0u, 0u, 0u);
+            r[s][4 * c] = w.x; r[s][4 * c + 1] = w.y; r[s][4 * c + 2] = w.z; r[s][4 * c + 3] = w.w;
+          }
+#pragma unroll
+        for (int s = 0; s < kHalf; ++s)
+          if (s0 + s < NS) tmem_st_32x32(tmem + L::kQCol + (s0 + s) * 32, r[s]);
       }
-#pragma unroll
-      for (int nt = 0; nt < 4; ++nt) mma_16816(s[nt], qf[k], kb[k & 1][2 * nt], kb[k & 1][2 * nt + 1]);
-    }
-    float* d = s_s + ((i & 1) * 4 + quarter) * kRows * L::kSLd + (mt * 16 + g) * L::kSLd + 2 * tq;
-#pragma unroll
-    for (int nt = 0; nt < 4; ++nt) {
-      *reinterpret_cast<float2*>(d + nt * 8) = make_float2(s[nt][0], s[nt][1]);
-      *reinterpret_cast<float2*>(d + nt * 8 + 8 * L::kSLd) = make_float2(s[nt][2], s[nt][3]);
-    }
-    return ok;
-  };
-  if (consumer && n > 0) {
-    bool ok = bar_red_and(1, kThreads, scores(0));
-    for (int i = 0; i < n && ok; ++i) {
-      const int st = i % L::kStages, buf = i & 1;
-      {
-        static_assert(PER == 4, "one vector of scores per thread");
-        const float* sp = s_s + buf * 4 * kRows * L::kSLd + row * L::kSLd + sub * PER;
-        float4 a = *reinterpret_cast<const float4*>(sp);
-#pragma unroll
-        for (int w = 1; w < 4; ++w) {
-          const float4 c = *reinterpret_cast<const float4*>(sp + w * kRows * L::kSLd);
-          a.x += c.x; a.y += c.y; a.z += c.z; a.w += c.w;
-        }
-        float x[PER] = {a.x, a.y, a.z, a.w}, mx = -INFINITY;
-        const int tok0 = (p0 + i) * kLatPage + sub * PER;
-#pragma unroll
-        for (int j = 0; j < PER; ++j) {
-          x[j] = tok0 + j >= lo && tok0 + j <= pos ? x[j] * p.scale_log2 : -INFINITY;
-          mx = fmaxf(mx, x[j]);
-        }
-#pragma unroll
-        for (int w = 1; w < TPR; w <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, w));
-        const float mn = fmaxf(m, mx), alpha = exp2f(m - mn);  // finite: every page holds a visible token
-        m = mn;
-        float sum = 0.f;
-#pragma unroll
-        for (int j = 0; j < PER; ++j) {
-          x[j] = exp2f(x[j] - mn);
-          sum += x[j];
-        }
-        l = l * alpha + sum;                                   // this thread's share of the denominator
-        *reinterpret_cast<uint2*>(p_s + (buf * kRows + row) * L::kPLd + sub * PER) =
-            make_uint2(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]));
-        if (sub == 0) al_s[buf][row] = alpha;
-      }
-      bool next = true;
-      if (i + 1 < n) next = scores(i + 1);
-      ok = bar_red_and(1, kThreads, next);
-      if (!ok) break;
-      const uint32_t base = smem_u32(smem + st * L::kStage) + v_off;
-      uint32_t pa[2][4], vb[2][4];
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-        ldsm_x4(smem_u32(p_s + (buf * kRows + mt * 16 + (lane & 15)) * L::kPLd + 16 * j + (lane >> 4) * 8), pa[j][0], pa[j][1],
-                pa[j][2], pa[j][3]);
-      ldsm_x4_t(base, vb[0][0], vb[0][1], vb[0][2], vb[0][3]);
-      const float a0 = al_s[buf][mt * 16 + g], a1 = al_s[buf][mt * 16 + g + 8];
-      if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {   // most pages raise no maximum
-#pragma unroll
-        for (int u = 0; u < 2 * VS; ++u) {
-          o[u][0] *= a0; o[u][1] *= a0;
-          o[u][2] *= a1; o[u][3] *= a1;
-        }
-      }
-#pragma unroll
-      for (int q = 0; q < 2 * VS; ++q) {
-        if (q + 1 < 2 * VS) {
-          uint32_t(&d)[4] = vb[(q + 1) & 1];
-          ldsm_x4_t(base + ((q + 1) % VS) * L::kSlab + ((q + 1) / VS) * 2048, d[0], d[1], d[2], d[3]);
-        }
-        const int u = q % VS, j = q / VS;
-        mma_16816(o[2 * u], pa[j], vb[q & 1][0], vb[q & 1][1]);
-        mma_16816(o[2 * u + 1], pa[j], vb[q & 1][2], vb[q & 1][3]);
-      }
+      tmem_st_wait();
+      tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(&empty[st]);
+      if (lane == 0) mbar_arrive(&q_ready);
     }
+    float l = 0.f, m = -INFINITY;                   // of head `lane`
+    bool alive = true;
+    for (int i = 0; i < n; ++i) {
+      const int buf = i & 1;
+      float x[kLatPage], mx = -INFINITY;
+      bool grow = false;
+      if (holds) {
+        alive = alive && mbar_wait(&s_full[buf], uint32_t(i / 2) & 1u, abort_flag, p.status, ERR_WAIT_TMEM_FULL);
+        alive = __all_sync(0xffffffffu, alive);
+        int state = LAT_ABORT;
+        if (alive) {
+          uint32_t r[kLatPage];
+          tc_fence_after();
+          tmem_ld_32x32(tmem + L::kSCol + buf * kLatPage, r);
+          tmem_ld_wait();
+          tc_fence_before();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&s_empty[buf]);
+          const int first = lo - (p0 + i) * kLatPage, last = pos - (p0 + i) * kLatPage;
+#pragma unroll
+          for (int j = 0; j < kLatPage; ++j) x[j] = __uint_as_float(r[j]) * p.scale_log2;
+          if (first > 0 || last < kLatPage - 1) {   // the same for all lanes
+#pragma unroll
+            for (int j = 0; j < kLatPage; ++j)
+              if (j < first || j > last) x[j] = -INFINITY;
+          }
+          float m4[4] = {x[0], x[1], x[2], x[3]};
+#pragma unroll
+          for (int j = 4; j < kLatPage; ++j) m4[j & 3] = fmaxf(m4[j & 3], x[j]);
+          mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));      // finite: every page holds a visible token
+          grow = lane < nh && (mx > m + kLatRescaleStep || m == -INFINITY);
+          if (i == 0) {                             // nothing to rescale
+            if (grow) m = mx;
+            grow = false;
+          }
+          state = __any_sync(0xffffffffu, grow) ? LAT_RAISE : LAT_STEADY;
+        }
+        if (lane == 0) state_s[buf] = state;
+      }
+      asm volatile("bar.sync 1, 128;" ::: "memory");
+      const int state = state_s[buf];
+      if (state == LAT_ABORT) break;
+      if (state == LAT_RAISE) {
+        if (holds) {
+          const float alpha = grow ? ex2(m - mx) : 1.f;
+          if (lane < N) raise_s[lane] = alpha;
+          if (grow) m = mx;
+          l *= alpha;
+        }
+        asm volatile("bar.sync 1, 128;" ::: "memory");
+        // O^T holds all of the page before this one
+        alive = alive && mbar_wait(&p_empty[buf ^ 1], uint32_t((i - 1) / 2) & 1u, abort_flag, p.status, ERR_WAIT_TMEM_FULL);
+        alive = __all_sync(0xffffffffu, alive);
+        tc_fence_after();
+#pragma unroll 1
+        for (int tile = 0; tile < L::kTiles; ++tile) {
+          uint32_t o[N];
+          tmem_ld_cols<N>(tmem + lanes + L::kOCol + tile * N, o);
+          tmem_ld_wait();
+#pragma unroll
+          for (int h = 0; h < N; ++h) o[h] = __float_as_uint(__uint_as_float(o[h]) * raise_s[h]);
+          tmem_st_cols<N>(tmem + lanes + L::kOCol + tile * N, o);
+        }
+        tmem_st_wait();
+      }
+      if (holds) {
+        const float base = m == -INFINITY ? 0.f : m;             // lanes without a head
+        float l4[4] = {0.f, 0.f, 0.f, 0.f};
+        uint32_t pk[kLatPage / 2];
+#pragma unroll
+        for (int j = 0; j < kLatPage; j += 2) {
+          const float e0 = ex2(x[j] - base), e1 = ex2(x[j + 1] - base);
+          l4[j & 2] += e0;
+          l4[(j & 2) + 1] += e1;
+          pk[j / 2] = pack_bf16x2(e0, e1);
+        }
+        l += (l4[0] + l4[1]) + (l4[2] + l4[3]);
+        if (i >= 2) {                               // the buffer's probabilities have been multiplied
+          alive = alive && mbar_wait(&p_empty[buf], uint32_t(i / 2 - 1) & 1u, abort_flag, p.status, ERR_WAIT_TMEM_FULL);
+          alive = __all_sync(0xffffffffu, alive);
+        }
+        if (lane < N) {
+          uint8_t* dst = p_s + buf * L::kProb + lane * 128;
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+            *reinterpret_cast<uint4*>(dst + ((c ^ (lane & 7)) << 4)) = make_uint4(pk[4 * c], pk[4 * c + 1], pk[4 * c + 2], pk[4 * c + 3]);
+        }
+        fence_proxy_async();
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_full[buf]);
+    }
+    // ---- all pages: O^T out of tensor memory
+    if (n > 0) {
+      alive = alive && mbar_wait(&p_empty[(n - 1) & 1], uint32_t((n - 1) / 2) & 1u, abort_flag, p.status, ERR_WAIT_TMEM_FULL);
+      alive = __all_sync(0xffffffffu, alive);
+      tc_fence_after();
+    }
+    if (holds && lane < N) {
+      m_s[lane] = lane < nh ? m : -INFINITY;
+      l_s[lane] = l;
+    }
+    float* o_s = reinterpret_cast<float*>(smem);                      // every page has been consumed
+#pragma unroll 1
+    for (int tile = 0; tile < L::kTiles; ++tile) {
+      uint32_t o[N];
+      if (n > 0) {
+        tmem_ld_cols<N>(tmem + lanes + L::kOCol + tile * N, o);
+        tmem_ld_wait();
+      } else {
+#pragma unroll
+        for (int h = 0; h < N; ++h) o[h] = 0u;
+      }
+      const int c = tile * 128 + tok;
+      if (c < VC) {
+#pragma unroll
+        for (int h = 0; h < N; ++h) o_s[h * L::kOLd + c] = __uint_as_float(o[h]);
+      }
+    }
+    tc_fence_before();
   }
-  if (*(volatile int*)&abort_flag) {
+  if (*abort_flag) {
     for (int i = 0; i < 200; ++i) __nanosleep(1000);
   }
-#pragma unroll
-  for (int w = 1; w < TPR; w <<= 1) l += __shfl_xor_sync(0xffffffffu, l, w);
-  if (consumer && sub == 0) {
-    m_s[row] = m;
-    l_s[row] = l;
-  }
   __syncthreads();
-  const auto sink_log2 = [&](int r) { return p.a.sinks ? p.a.sinks[head0 + r] * 1.4426950408889634f : -INFINITY; };
-  if (p.num_splits == 1) {
-    if (!consumer) return;
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int r = mt * 16 + g + 8 * e;
-      if (r >= nh) continue;
-      const float sk = sink_log2(r), m2 = fmaxf(m_s[r], sk), sc = exp2f(m_s[r] - m2);
-      const float inv = sc / (l_s[r] * sc + exp2f(sk - m2));
-      __nv_bfloat16* dst = out + r * p.a.o_head;
-#pragma unroll
-      for (int u = 0; u < 2 * VS; ++u) {
-        const int c = (u / 2 * 4 + quarter) * 16 + (u & 1) * 8 + 2 * tq;
-        const float v0 = o[u][2 * e] * inv, v1 = o[u][2 * e + 1] * inv;
-        if (c + 1 < p.a.rank && ((p.a.o_head | p.a.o_token) & 1) == 0) {
-          *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(v0, v1);
-        } else {
-          if (c < p.a.rank) dst[c] = __float2bfloat16(v0);
-          if (c + 1 < p.a.rank) dst[c + 1] = __float2bfloat16(v1);
-        }
-      }
-    }
-    return;
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, L::kCols);
   }
-  float* o_s = reinterpret_cast<float*>(smem);       // every page has been consumed (barrier above)
-#pragma unroll
-  for (int u = 0; u < 2 * VS; ++u) {
-    if (!consumer) break;
-    float* d = o_s + (mt * 16 + g) * L::kOLd + (u / 2 * 4 + quarter) * 16 + (u & 1) * 8 + 2 * tq;
-    *reinterpret_cast<float2*>(d) = make_float2(o[u][0], o[u][1]);
-    *reinterpret_cast<float2*>(d + 8 * L::kOLd) = make_float2(o[u][2], o[u][3]);
-  }
-  cluster_sync_all();
+  const float* o_s = reinterpret_cast<const float*>(smem);
+  if (p.num_splits > 1) cluster_sync_all();
   // this CTA's heads: r0 .. r0 + per - 1
-  const int splits = p.num_splits, per = kRows / splits, r0 = split * per;
+  const int splits = p.num_splits, per = N / splits, r0 = split * per;
   if (int(threadIdx.x) < per) {
     const int r = r0 + threadIdx.x;
-    const float sk = r < nh ? sink_log2(r) : -INFINITY;
+    const float sk = r < nh && p.a.sinks ? p.a.sinks[head0 + r] * 1.4426950408889634f : -INFINITY;
     float ms[kLatMaxSplits], ls[kLatMaxSplits], mf = sk, den = 0.f;
 #pragma unroll
     for (int s = 0; s < kLatMaxSplits; ++s)
@@ -657,7 +728,7 @@ latent_mma_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant
 #pragma unroll
   for (int s = 0; s < kLatMaxSplits; ++s) peer[s] = s < splits ? map_to_cta(o_s, s) : 0u;
 #pragma unroll 2
-  for (int i = threadIdx.x * 4; consumer && i < per * VC; i += 4 * kThreads) {
+  for (int i = threadIdx.x * 4; i < per * VC; i += 1024) {
     const int r = i / VC, c = i % VC;
     float4 x[kLatMaxSplits];
 #pragma unroll
@@ -681,28 +752,28 @@ latent_mma_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant
         if (c + e < p.a.rank) dst[e] = __float2bfloat16(v[e]);
     }
   }
-  cluster_sync_all();          // no CTA leaves while its sums are read
+  if (p.num_splits > 1) cluster_sync_all();          // no CTA leaves while its sums are read
 }
 
-template <int NS, int VS, int MT>
+template <int NS, int VS, int N>
 static int launch_latent(const CUtensorMap& tc, const LatentMmaParams& p, int tokens, cudaStream_t s) {
-  using L = LatentSmem<NS, VS, MT>;
+  using L = LatentSmem<NS, VS, N>;
   constexpr int smem = L::kEnd + 1024;
-  static_assert(smem + 4096 <= 232448, "shared memory of a CTA");
+  static_assert(smem + 3072 <= 232448, "shared memory of a CTA");
   static bool attr_set[64] = {false};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -1;
   if (!attr_set[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(latent_mma_kernel<NS, VS, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(latent_attn_kernel<NS, VS, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return int(e);
     attr_set[dev] = true;
   }
-  const dim3 grid(p.num_splits, (p.a.heads + L::kRows - 1) / L::kRows, tokens);
-  return launch_pdl_cluster(latent_mma_kernel<NS, VS, MT>, grid, dim3(128 * MT + 32), size_t(smem), s, p.num_splits, tc, p);
+  const dim3 grid(p.num_splits, (p.a.heads + N - 1) / N, tokens);
+  return launch_pdl_cluster(latent_attn_kernel<NS, VS, N>, grid, dim3(256), size_t(smem), s, p.num_splits, tc, p);
 }
 template <int NS, int VS>
 static int launch_latent_heads(const CUtensorMap& tc, const LatentMmaParams& p, int tokens, cudaStream_t s) {
-  return p.a.heads <= 16 ? launch_latent<NS, VS, 1>(tc, p, tokens, s) : launch_latent<NS, VS, 2>(tc, p, tokens, s);
+  return p.a.heads <= 16 ? launch_latent<NS, VS, 16>(tc, p, tokens, s) : launch_latent<NS, VS, 32>(tc, p, tokens, s);
 }
 
 // Slabs of a row and of its latent that the kernel is built for; 0 when it does not take the sizes.
@@ -802,12 +873,12 @@ extern "C" int nkb_latent_attn(const NkbLatentArgs* a, const void* q, const void
   const int ns = latent_shape(*a, &vs);
   if (!ns || a->row != ns * 64) return -5;
   if (!latent_ok(*a) || block_size != kLatPage || tokens > 65535 || (!q_lens && tokens != batch)) return -2;
-  if ((reinterpret_cast<uintptr_t>(q) & 3) || ((a->q_token | a->q_head) & 1) || (reinterpret_cast<uintptr_t>(out) & 7)) return -2;
+  if (!al16(q) || ((a->q_token | a->q_head) & 7) || (reinterpret_cast<uintptr_t>(out) & 7)) return -2;
   if (!status_word() && nkb_init() != 0) return -1;
   LatentMmaParams p{};
   p.a = *a;
-  const int splits = num_splits >= 8 ? 8 : num_splits >= 4 ? 4 : num_splits >= 2 ? 2 : 1;
   p.q = reinterpret_cast<const __nv_bfloat16*>(q);
+  const int splits = num_splits >= 8 ? 8 : num_splits >= 4 ? 4 : num_splits >= 2 ? 2 : 1;
   p.block_table = block_table; p.q_start = q_start; p.q_lens = q_lens; p.context_lens = context_lens;
   p.out = reinterpret_cast<__nv_bfloat16*>(out);
   p.status = status_word();
