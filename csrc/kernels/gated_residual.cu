@@ -389,6 +389,49 @@ __global__ void __launch_bounds__(256) gated_act_kernel(const __grid_constant__ 
   }
 }
 
+// Prompts: bf16 gate and up in whole 16-byte pieces, two pieces per thread in flight.
+__global__ void __launch_bounds__(256) gated_act8_kernel(const __grid_constant__ NkbProj gate, const __grid_constant__ NkbProj up,
+                                                         __nv_bfloat16* __restrict__ out, int pieces, int per_row, int kind,
+                                                         float limit, float alpha) {
+  griddep_wait();
+  griddep_launch();
+  uint4 g[2], u[2];
+  int row[2], col[2];
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const int i = (blockIdx.x * 2 + k) * 256 + threadIdx.x;
+    row[k] = i < pieces ? i / per_row : -1;
+    col[k] = i < pieces ? i % per_row * 8 : 0;
+    g[k] = u[k] = make_uint4(0u, 0u, 0u, 0u);
+    if (row[k] >= 0) {
+      g[k] = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(gate.ptr) + row[k] * gate.ld + col[k]);
+      u[k] = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(up.ptr) + row[k] * up.ld + col[k]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    if (row[k] < 0) continue;
+    const uint32_t gw[4] = {g[k].x, g[k].y, g[k].z, g[k].w}, uw[4] = {u[k].x, u[k].y, u[k].z, u[k].w};
+    uint32_t r[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 a = unpack_bf16x2(gw[e]), b = unpack_bf16x2(uw[e]);
+      float x[2] = {a.x, a.y}, y[2] = {b.x, b.y};
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        if (kind == ACT_CLAMPED) {
+          x[j] = fminf(x[j], limit);
+          x[j] *= sigmoid_f(alpha * x[j]) * (fminf(fmaxf(y[j], -limit), limit) + 1.f);
+        } else {
+          x[j] = apply_act(x[j], kind) * y[j];
+        }
+      }
+      r[e] = pack_bf16x2(x[0], x[1]);
+    }
+    *reinterpret_cast<uint4*>(out + (long long)row[k] * per_row * 8 + col[k]) = make_uint4(r[0], r[1], r[2], r[3]);
+  }
+}
+
 }  // namespace nkb
 
 using namespace nkb;
@@ -474,6 +517,11 @@ extern "C" int nkb_gated_act(const NkbProj* gate, const NkbProj* up, void* out, 
     return launch_pdl(kernel, dim3(blocks), dim3(256), 0, s, *gate, *up, o, rows, inter, kind, limit, alpha, up_rows, up_limit);
   };
   using bf = __nv_bfloat16;
+  const long long pieces = (long long)rows * (inter / 8);
+  if (out_bf16 && gate->bf16 && up->ptr && up->bf16 && !up_rows && inter % 8 == 0 && ((gate->ld | up->ld) & 7) == 0 &&
+      aligned16(gate->ptr) && aligned16(up->ptr) && aligned16(out) && pieces < (1ll << 30))
+    return launch_pdl(gated_act8_kernel, dim3(unsigned((pieces + 511) / 512)), dim3(256), 0, s, *gate, *up, reinterpret_cast<bf*>(out),
+                      int(pieces), inter / 8, kind, limit, alpha);
   if (out_bf16)
     return vec ? launch(gated_act_kernel<4, bf>, reinterpret_cast<bf*>(out)) : launch(gated_act_kernel<1, bf>, reinterpret_cast<bf*>(out));
   return vec ? launch(gated_act_kernel<4, float>, reinterpret_cast<float*>(out))
