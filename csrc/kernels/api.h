@@ -195,8 +195,7 @@ int nkb_token_mix(const void* h, int bf16, const float* mu, float* state, const 
                   const int* q_lens, const int* context_lens, void* out, int batch, int tokens, int width, int mixes,
                   void* stream);
 int nkb_gate_heads(const void* x, int x_bf16, long long ld_token, long long ld_head, const NkbProj* gate, int head_gate,
-                   int gate_act,
-                   const float* norm_w, int norm_stride, float eps, float scale, void* out, int out_bf16,
+                   int gate_act, const float* norm_w, int norm_stride, float eps, float scale, void* out, int out_bf16,
                    long long out_ld, int tokens, int heads, int width, void* stream);
 // gated linear recurrence (recurrent.cu)
 long long nkb_hgrn2_scan_scratch(int heads, int dim, int vdim);
@@ -243,5 +242,6 @@ int nkb_latent_prefill(const void* q, const void* kv, const void* rotated, const
                        int heads, int dim, int rot, int vdim, long long ld, long long rot_ld, int nk, int nv, float scale,
                        int window, const float* sinks, void* stream);
 int nkb_latent_attn(const NkbLatentArgs* a, const void* q, const void* cache, const int* block_table, const int* q_start,
-                    const int* q_lens, const int* context_lens, void* out, int batch, int tokens, int block_size, int num_blocks, int max_blocks_per_seq, int num_splits, void* stream);
+                    const int* q_lens, const int* context_lens, void* out, int batch, int tokens, int block_size,
+                    int num_blocks, int max_blocks_per_seq, int num_splits, void* stream);
 }

@@ -70,7 +70,7 @@ def shrink(cfg: ModelConfig) -> ModelConfig:
     if cfg.name == "ligizen":
         routed = any(l.experts for l in cfg.layers)
         return ligizen_shape(256, layers=len(cfg.layers), heads=4, kv_heads=2, ff=512, vocab=2048, dim=32, window=64, chunk=48,
-                             latent_dim=32, rot=16, kv_rank=64, q_rank=96, side=32, share_every=2,
+                             latent_dim=40, rot=8, kv_rank=48, q_rank=96, side=32, share_every=2,
                              **(dict(experts=8, top=2, expert_ff=64) if routed else {}))
     if cfg.layers is not None:
         return tolenex_shape(256, layers=len(cfg.layers), heads=4, kv_heads=1, ff=512, vocab=2048, dim=32, vdim=64,

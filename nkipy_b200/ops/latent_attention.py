@@ -6,8 +6,8 @@
     latent_gather     cached rows of whole pages, as operands of the keys' and values' up projections
     latent_prefill    new tokens against keys and values expanded from those rows
 
-CUDA tensors run csrc/kernels/latent_attn.cu and, for expanded keys, attn_prefill.cu (32-bit models and sizes its tensor-core kernel does not take: the general kernel
-of attn_maps.cu); CPU tensors run the PyTorch statement of the same op.
+CUDA tensors run csrc/kernels/latent_attn.cu and, for expanded keys, attn_prefill.cu (32-bit models and sizes the tensor-core
+kernel does not take: the general kernel of attn_maps.cu); CPU tensors run the PyTorch statement of the same op.
 """
 
 from __future__ import annotations

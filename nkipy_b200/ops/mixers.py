@@ -199,7 +199,8 @@ def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Branch] = (), *
     rc = _lib.lib().nkb_gated_residual(
         _ptr(x), _ptr(ids), _ptr(table), 1 if table is not None and table.dtype == torch.bfloat16 else 0,
         table.shape[0] if table is not None else 0, float(scale), n, ba, _ptr(add_row), _ptr(add_mat), r.data_ptr(), len(outs),
-        norms[0].kind if norms else 0, _ptr_array(weights), _ptr_array(biases), _ptr_array(outs), 1 if dtype == torch.bfloat16 else 0, rows, width, int(groups), float(eps), _stream())
+        norms[0].kind if norms else 0, _ptr_array(weights), _ptr_array(biases), _ptr_array(outs),
+        1 if dtype == torch.bfloat16 else 0, rows, width, int(groups), float(eps), _stream())
     _lib.check(rc, "nkb_gated_residual")
     _count_launch()
     return r, outs
@@ -265,8 +266,8 @@ def gate_heads(x: torch.Tensor, gate: Proj, act: str, *, norm_w: Optional[torch.
     stride = 0 if norm_w is None or norm_w.numel() == n else n
     rc = _lib.lib().nkb_gate_heads(
         x.data_ptr(), 1 if x.dtype == torch.bfloat16 else 0, x.stride(0), x.stride(1), _ref(gate),
-        1 if gate.width == H and n > 1 else 0, ACTIVATIONS[act][0], _ptr(norm_w), stride, float(eps), float(scale), out.data_ptr(), 1 if out.dtype == torch.bfloat16 else 0,
-        out.stride(0), T, H, n, _stream())
+        1 if gate.width == H and n > 1 else 0, ACTIVATIONS[act][0], _ptr(norm_w), stride, float(eps), float(scale),
+        out.data_ptr(), 1 if out.dtype == torch.bfloat16 else 0, out.stride(0), T, H, n, _stream())
     _lib.check(rc, "nkb_gate_heads")
     _count_launch()
     return out

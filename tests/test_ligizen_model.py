@@ -36,8 +36,8 @@ def _one_thread():
 # name -> small_config arguments; sizes, orders and branches differ between them
 MODELS = {
     "mixed": dict(),
-    "chunk-first": dict(layers="ckl", mlps="msd", width=128, heads=2, kv_heads=2, dim=32, vdim=32, rot=32, chunk=5, lheads=4,
-                        ldim=32, lrot=16, lvdim=32, rank=64, q_rank=48, window=7, experts=4, top=3, side=16),
+    "chunk-first": dict(layers="ckl", mlps="msd", width=128, heads=2, kv_heads=2, dim=32, vdim=32, rot=32, chunk=5, lheads=2,
+                        ldim=40, lrot=24, lvdim=48, rank=72, q_rank=48, window=7, experts=4, top=3, side=16),
     "no-ff": dict(layers="lc", mlps="--", width=64, heads=3, kv_heads=1, dim=64, vdim=72, rot=24, chunk=33, scaling=None,
                   lheads=1, ldim=64, lrot=64, lvdim=72, rank=128, window=33, vocab=96, escale=1.0),
     "latent": dict(layers="lL", mlps="d-", lheads=18, ldim=72, lrot=24, lvdim=80, rank=136, q_rank=64, window=64, eps=1e-3),
@@ -138,8 +138,8 @@ def test_long_prompt_and_long_decoding(name, device, dtype, window, chunk):
 @in_dtypes
 @pytest.mark.parametrize("size", [1, 2, 31, 32, 33])
 def test_window_and_chunk_edges_in_the_whole_model(device, dtype, size):
-    """Sharp scores, so that a window or a chunk that is one token off changes the logits; also in the very first tokens."""
-    sharp = dict(window=size, chunk=size, scale=0.3, lscale=0.4)
+    """Scores of a size at which a window or a chunk that is one token off changes most logits; also in the very first tokens."""
+    sharp = dict(window=size, chunk=size, scale=0.3, lscale=0.15)
     c = Case("chunk-first", device, dtype, **sharp)
     ids = c.tokens(70, 11)
     want = c.want(ids)
@@ -329,8 +329,8 @@ def test_config_reader():
 
 @on_devices
 def test_regular_shapes_and_random_weights_run(device):
-    cfg = C.ligizen_shape(128, layers=6, heads=4, kv_heads=2, ff=256, vocab=300, dim=32, window=40, chunk=48, latent_dim=32,
-                          rot=16, kv_rank=64, q_rank=96, side=32, experts=8, top=2, expert_ff=64, share_every=2)
+    cfg = C.ligizen_shape(128, layers=6, heads=4, kv_heads=2, ff=256, vocab=300, dim=32, window=40, chunk=48, latent_dim=40,
+                          rot=8, kv_rank=48, q_rank=96, side=32, experts=8, top=2, expert_ff=64, share_every=2)
     assert registry.for_config(cfg) is registry.ARCHITECTURES["Ligizen"]
     assert [getattr(l.mixer, "kv_from", None) for l in cfg.layers] == [None, None, None, 1, None, None]
     cfg = runner.shrink(cfg) if device == "cpu" else cfg
