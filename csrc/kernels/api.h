@@ -6,8 +6,10 @@
 #include <cuda.h>
 #include <stdint.h>
 #include "attn_maps.h"
+#include "head_recurrence.h"
 #include "latent_attn.h"
 #include "linear_attn.h"
+#include "post_residual.h"
 #include "proj_src.h"
 
 namespace nkb {
@@ -71,11 +73,11 @@ void nkb_set_pdl(int enabled);
 int nkb_gemm_bf16(const void* A, const void* B, void* out, int rows, int cols, int k, long long lda, long long ldb,
                   long long ldo, int transpose_out, int out_fp32, int splits, long long split_stride, int gated,
                   int gate_off, const void* bias, int bias_on_rows, const void* residual, int block_n, int max_ctas,
-                  int weights_operand, int ctas_per_sm, int act, void* stream);
+                  int weights_operand, int ctas_per_sm, int act, float act_a, float act_b, void* stream);
 int nkb_gemm_effective_splits(int k, int splits);
 int nkb_gemm_bf16_2cta(const void* A, const void* B, void* out, int m, int n, int k, long long lda, long long ldb,
                        long long ldo, const void* bias, const void* residual, int gated, int gate_off, int act,
-                       void* stream);
+                       float act_a, float act_b, void* stream);
 int nkb_gemm_bf16_push(const void* weights, const void* x, int features, int tokens, int k, long long ldw,
                        long long ldx, long long ldo, int splits, const void* bias, int block_n, void* const* peer_out,
                        void* const* peer_flag, int n_peers, int rank, void* done_counter, void* mc_out, void* mc_flag,
@@ -157,7 +159,7 @@ int nkb_router_topk(const void* logits, int is_fp32, int splits, long long split
 int nkb_paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                           const int* context_lens, void* out, float* scratch, int batch, int q_len, int nq, int nkv,
                           int head_dim, int block_size, int num_blocks, int max_blocks_per_seq, float scale,
-                          int window, int chunk, const float* sinks, int num_splits, void* stream);
+                          int window, int chunk, const float* sinks, const NkbScoreMods* mods, int num_splits, void* stream);
 int nkb_paged_attn_decode_fused(const float* qkv_partials, int qkv_splits, long long qkv_split_stride,
                                 const void* qkv_bias, const int* positions, const int* slots, const float* cos_sin,
                                 const void* q_norm_w, const void* k_norm_w, float norm_eps, int max_pos, void* k_cache,
@@ -171,7 +173,7 @@ int nkb_flash_attn_prefill(const void* q, const void* k_cache, const void* v_cac
                            const int* q_start, const int* q_lens, const int* context_lens, void* out, int batch,
                            int total_q, int max_q_len, int nq, int nkv, int head_dim, int block_size, int num_blocks,
                            int max_blocks_per_seq, float scale, int causal, int window, int chunk, const float* sinks,
-                           void* stream);
+                           const NkbScoreMods* mods, void* stream);
 
 // layers with an fp32 residual stream (gated_residual.cu)
 int nkb_gated_residual(const float* x_in, const int* ids, const void* table, int table_bf16, int vocab, float scale,
@@ -189,6 +191,16 @@ int nkb_gemm_simt_grouped(const void* x, int x_bf16, const void* w, int w_bf16, 
 // linear attention with per-channel decay and what surrounds it (linear_attn.cu)
 int nkb_linattn_scan(const NkbLinAttn* args, void* stream);
 int nkb_linattn_step(const NkbLinAttn* args, void* stream);
+// recurrences with one decay per head behind a short convolution (head_recurrence.cu)
+int nkb_short_conv(const NkbProj* x, const float* w, const float* b, float* state, const int* slot_ids, const int* q_start,
+                   const int* q_lens, const int* context_lens, void* out, int bf16, int batch, int tokens, int channels, int taps,
+                   int act, void* stream);
+int nkb_head_rec_scan(const NkbHeadRec* args, void* stream);
+int nkb_head_rec_step(const NkbHeadRec* args, void* stream);
+int nkb_gated_group_norm(const void* y, int y_bf16, const NkbProj* gate, int gate_act, const float* w, float eps, void* out,
+                         int out_bf16, int tokens, int width, int parts, void* stream);
+// residual updates through a norm, weighted averages of earlier results (post_residual.cu)
+int nkb_post_residual(const NkbPostResidual* args, void* stream);
 int nkb_low_rank(const NkbProj* x, int act, const void* w, int w_bf16, float* out, int tokens, int rank, int n,
                  void* stream);
 int nkb_token_mix(const void* h, int bf16, const float* mu, float* state, const int* slot_ids, const int* q_start,
@@ -215,7 +227,7 @@ int nkb_row_norm_append(const NkbMapsArgs* a, const NkbProj* q, const NkbProj* k
                         int tokens, int block_size, void* stream);
 int nkb_rope_norm_append(const NkbMapsArgs* a, const NkbProj* q, const NkbProj* k, const NkbProj* v, const float* bias,
                          const float* cos_sin, int rot_dims, int max_pos, const int* positions, const int* slots, int norm,
-                         void* q_out, void* k_cache, void* v_cache, int bf16, int tokens, int block_size, void* stream);
+                         int pairs, void* q_out, void* k_cache, void* v_cache, int bf16, int tokens, int block_size, void* stream);
 int nkb_maps_attn_simple(const NkbMapsArgs* a, const void* q, const void* k_cache, const void* v_cache,
                          const int* block_table, const int* q_start, const int* q_lens, const int* context_lens,
                          void* out, int bf16, int batch, int total_q, int block_size, int max_blocks_per_seq,

@@ -68,6 +68,7 @@ struct DecodeParams {
   __nv_bfloat16* v_cache;
   float norm_eps;
   int qkv_splits, max_pos;
+  NkbScoreMods mods;         // MODS only (not fused)
 };
 
 // One head row of the fused QKV output for token `tok`, in two steps so that a warp can have the loads of two
@@ -170,7 +171,21 @@ struct FusedRow {
   }
 };
 
-template <int D, int kDecWarps>
+// A scaled score in units of ln 2: the optional cap (tanh written with the exponential, absolute error of an ulp or two of the
+// cap), then the term that grows with the distance.
+__device__ __forceinline__ float modified_score(float s, const DecodeParams& p, float inv_cap, float dist_a, float dist_b, int dist) {
+  constexpr float kLog2e = 1.4426950408889634f;
+  s *= p.scale_log2;
+  if (p.mods.softcap > 0.f) {
+    const float cap2 = p.mods.softcap * kLog2e;
+    s = cap2 - 2.f * cap2 * __fdividef(1.f, exp2f(2.f * s * inv_cap) + 1.f);
+  }
+  if (p.mods.dist_a) s = fmaf(-dist_a, __log2f(fmaf(dist_b, float(dist), 1.f)), s);
+  return s;
+}
+
+// MODS: scores are capped, lose a term that grows with the distance, or the first tokens stay visible outside the window.
+template <int D, int kDecWarps, bool MODS>
 __global__ void __launch_bounds__(kDecWarps * 32)
 paged_attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                          const DecodeParams p) {
@@ -209,10 +224,15 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_c
   // ---- page range of this split
   const int first_tok = nkb_first_visible(max(ctx - p.q_len, 0), p.window, p.chunk);
   const int page_lo = first_tok / kPage, page_hi = (ctx_paged + kPage - 1) / kPage;
-  const int npages = max(page_hi - page_lo, 0);
+  // pages of kept first tokens come ahead of the window's (those that are not among them): walk position x is page page_at(x)
+  // (without MODS the walk counts pages themselves)
+  const int kept = MODS ? min((p.mods.keep_first + kPage - 1) / kPage, page_lo) : 0;
+  const int walk0 = MODS ? 0 : page_lo, shift = page_lo - kept;
+  const auto page_at = [&](int x) { return !MODS || x < kept ? x : x + shift; };
+  const int npages = kept + max(page_hi - page_lo, 0);
   const int per_split = (npages + p.num_splits - 1) / p.num_splits;
-  const int p0 = page_lo + split * per_split;
-  const int p1 = min(page_hi, p0 + per_split);
+  const int p0 = walk0 + split * per_split;
+  const int p1 = min(walk0 + npages, p0 + per_split);
   const int* table = p.block_table + (long long)b * p.max_blocks;
 
   float o[D / 8][4];
@@ -221,9 +241,9 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_c
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
 
   uint8_t* my_smem = smem + warp * kDecStages * kStageBytes;
-  auto issue = [&](int page, int stage) {
+  auto issue = [&](int at, int stage) {
     if (lane == 0) {
-      const int blk = table[page];
+      const int blk = table[page_at(at)];
       uint8_t* dst = my_smem + stage * kStageBytes;
       mbar_expect_tx(&bars[warp][stage], kStageBytes);
 #pragma unroll
@@ -329,6 +349,17 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_c
   const int lim0 = fused ? qpos0 - 1 : qpos0, lim1 = fused ? qpos1 - 1 : qpos1;   // fused: the new token is not paged
   const int low0 = nkb_first_visible(qpos0, p.window, p.chunk);
   const int low1 = nkb_first_visible(qpos1, p.window, p.chunk);
+  float inv_cap = 0.f, da0 = 0.f, da1 = 0.f, db0 = 0.f, db1 = 0.f;
+  if constexpr (MODS) {
+    inv_cap = p.mods.softcap > 0.f ? 1.f / p.mods.softcap : 0.f;
+    if (p.mods.dist_a) {
+      const int h0 = kvh * p.group + (g < rows ? g % p.group : 0), h1 = kvh * p.group + (g + 8 < rows ? (g + 8) % p.group : 0);
+      da0 = p.mods.dist_a[h0];
+      db0 = p.mods.dist_b[h0];
+      da1 = p.mods.dist_a[h1];
+      db1 = p.mods.dist_b[h1];
+    }
+  }
 
   int stage = 0;
   uint32_t phase = 0;
@@ -361,10 +392,19 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_c
     for (int nt = 0; nt < 4; ++nt) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const int tok = pg * kPage + nt * 8 + 2 * t + e;
-        float v0 = s[nt][e] * p.scale_log2, v1 = s[nt][2 + e] * p.scale_log2;
-        if (tok > lim0 || tok < low0) v0 = -INFINITY;
-        if (tok > lim1 || tok < low1) v1 = -INFINITY;
+        const int tok = page_at(pg) * kPage + nt * 8 + 2 * t + e;
+        float v0, v1;
+        if constexpr (MODS) {
+          v0 = modified_score(s[nt][e], p, inv_cap, da0, db0, qpos0 - tok);
+          v1 = modified_score(s[nt][2 + e], p, inv_cap, da1, db1, qpos1 - tok);
+          if (tok > lim0 || (tok < low0 && tok >= p.mods.keep_first)) v0 = -INFINITY;
+          if (tok > lim1 || (tok < low1 && tok >= p.mods.keep_first)) v1 = -INFINITY;
+        } else {
+          v0 = s[nt][e] * p.scale_log2;
+          v1 = s[nt][2 + e] * p.scale_log2;
+          if (tok > lim0 || tok < low0) v0 = -INFINITY;
+          if (tok > lim1 || tok < low1) v1 = -INFINITY;
+        }
         s[nt][e] = v0;
         s[nt][2 + e] = v1;
         mx0 = fmaxf(mx0, v0);
@@ -533,7 +573,7 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_c
   }
 }
 
-template <int D, int kDecWarps>
+template <int D, int kDecWarps, bool MODS>
 static int launch_decode(const CUtensorMap& tk, const CUtensorMap& tv, const DecodeParams& p, cudaStream_t s) {
   constexpr int kStageBytes = 2 * (D / 64) * kPage * 128;
   constexpr int smem = kDecWarps * kDecStages * kStageBytes + 1024;
@@ -545,30 +585,31 @@ static int launch_decode(const CUtensorMap& tk, const CUtensorMap& tv, const Dec
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -1;
   if (!attr_set[dev]) {
     cudaError_t e =
-        cudaFuncSetAttribute(paged_attn_decode_kernel<D, kDecWarps>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        cudaFuncSetAttribute(paged_attn_decode_kernel<D, kDecWarps, MODS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return int(e);
     attr_set[dev] = true;
   }
   dim3 grid(p.num_splits, p.nkv, p.batch);
-  return launch_pdl(paged_attn_decode_kernel<D, kDecWarps>, grid, dim3(kDecWarps * 32), size_t(smem), s, tk, tv, p);
+  return launch_pdl(paged_attn_decode_kernel<D, kDecWarps, MODS>, grid, dim3(kDecWarps * 32), size_t(smem), s, tk, tv, p);
 }
 
 // Warps per CTA: every warp streams its own pages through a private 3-stage ring (48 KB at D = 128), so an SM
 // holds four warps' rings whatever the CTA size.  The grid should fit the resident slots in one wave (a second,
 // partly filled wave costs as much as a full one): four-warp CTAs while there is at most one CTA per SM, two-warp
 // CTAs up to two per SM, one-warp CTAs (four per SM) beyond.
+template <bool MODS = false>
 static int dispatch_decode(int head_dim, long long ctas, int sms, const CUtensorMap& tk, const CUtensorMap& tv,
                            const DecodeParams& p, cudaStream_t s) {
   const int warps = ctas <= sms ? 4 : (ctas <= 2LL * sms ? 2 : 1);
   if (head_dim == 128) {
-    if (warps == 4) return launch_decode<128, 4>(tk, tv, p, s);
-    if (warps == 2) return launch_decode<128, 2>(tk, tv, p, s);
-    return launch_decode<128, 1>(tk, tv, p, s);
+    if (warps == 4) return launch_decode<128, 4, MODS>(tk, tv, p, s);
+    if (warps == 2) return launch_decode<128, 2, MODS>(tk, tv, p, s);
+    return launch_decode<128, 1, MODS>(tk, tv, p, s);
   }
   if (head_dim == 64) {
-    if (warps == 4) return launch_decode<64, 4>(tk, tv, p, s);
-    if (warps == 2) return launch_decode<64, 2>(tk, tv, p, s);
-    return launch_decode<64, 1>(tk, tv, p, s);
+    if (warps == 4) return launch_decode<64, 4, MODS>(tk, tv, p, s);
+    if (warps == 2) return launch_decode<64, 2, MODS>(tk, tv, p, s);
+    return launch_decode<64, 1, MODS>(tk, tv, p, s);
   }
   return -2;
 }
@@ -588,11 +629,13 @@ extern "C" long long nkb_paged_attn_decode_scratch_floats(int batch, int q_len, 
 extern "C" int nkb_paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                                      const int* context_lens, void* out, float* scratch, int batch, int q_len, int nq,
                                      int nkv, int head_dim, int block_size, int num_blocks, int max_blocks_per_seq,
-                                     float scale, int window, int chunk, const float* sinks, int num_splits, void* stream) {
+                                     float scale, int window, int chunk, const float* sinks, const NkbScoreMods* mods, int num_splits,
+                                     void* stream) {
   if (batch <= 0) return 0;
   if (block_size != kPage || nq % nkv != 0) return -2;
   const int group = nq / nkv;
   if (q_len * group > 16) return -2;
+  if (mods && (mods->keep_first < 0 || (mods->keep_first > 0 && chunk > 0) || !mods->dist_a != !mods->dist_b)) return -2;
   if (num_splits < 1) num_splits = 1;
   if (num_splits > 1 && (!scratch || (long long)batch * nkv > kDecCounters)) return -2;
   if (!status_word() && nkb_init() != 0) return -1;
@@ -607,6 +650,7 @@ extern "C" int nkb_paged_attn_decode(const void* q, const void* k_cache, const v
   p.status = status_word();
   p.batch = batch; p.q_len = q_len; p.nq = nq; p.nkv = nkv; p.group = group;
   p.max_blocks = max_blocks_per_seq; p.num_splits = num_splits; p.window = window; p.chunk = chunk;
+  if (mods) p.mods = *mods;
   p.scale_log2 = scale * 1.4426950408889634f;
   CUtensorMap tk, tv;
   const uint64_t dims[4] = {uint64_t(head_dim), uint64_t(kPage), uint64_t(nkv), uint64_t(num_blocks)};
@@ -616,7 +660,8 @@ extern "C" int nkb_paged_attn_decode(const void* q, const void* k_cache, const v
   if (encode_tmap_bf16(&tk, k_cache, 4, dims, strides, box)) return -4;
   if (encode_tmap_bf16(&tv, v_cache, 4, dims, strides, box)) return -4;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return dispatch_decode(head_dim, (long long)batch * nkv * num_splits, num_sms(), tk, tv, p, s);
+  const long long ctas = (long long)batch * nkv * num_splits;
+  return mods ? dispatch_decode<true>(head_dim, ctas, num_sms(), tk, tv, p, s) : dispatch_decode(head_dim, ctas, num_sms(), tk, tv, p, s);
 }
 
 // Decode attention that starts from the split-K partials of the fused QKV projection: bias, QK-norm, RoPE and the

@@ -2,8 +2,9 @@
 //   append   interleaved partial rotary embedding of queries and keys from the fused projection, keys and values
 //            into their slots of the paged cache
 //   row norm append   the same for one map without rotation, queries and keys normed over all heads of the token together
-//   rope norm append   the same for one map with projection biases, the rotation whose pairs are half a rotated part apart, and
-//            an RMS norm without weight over every head of queries and keys; without keys for layers that read another layer's
+//   rope norm append   the same for one map with projection biases, rotated or not (pairs half a rotated part apart, or next to
+//            each other), with or without an RMS norm without weight over every head of queries and keys; without keys for
+//            layers that read another layer's
 //   decode   one new token per sequence, bf16: the two maps of up to eight query heads are the sixteen rows of
 //            one MMA fragment (rows 0-7 map 0, rows 8-15 map 1).  A key row holds both maps' keys side by side, so with
 //            the query of map 0 only in the first half of the contraction and that of map 1 only in the second, one
@@ -216,6 +217,7 @@ struct RopeNormAppendParams {
   const int *positions, *slots;
   void *q_out, *k_cache, *v_cache;
   int rot_dims, max_pos, tokens, norm;
+  int pairs;                // rotation of pairs (2i, 2i + 1) instead of (i, i + rot_dims / 2)
 };
 
 template <int V>
@@ -261,8 +263,21 @@ __global__ void __launch_bounds__(256) rope_norm_append_kernel(const __grid_cons
     load_v<V>(x, src, t, h * dim + c);
     add_bias<V>(x, bias, c);
   };
-  const auto finish = [&](float (&x)[V], const float (&y)[V], int c, float inv) {       // y: the other half's elements
-    if (c < 2 * n) {
+  const auto finish = [&](float (&x)[V], const float (&y)[V], int c, float inv) {       // y: the elements x is paired with
+    if (p.pairs) {
+      if (c < 2 * n) {
+        if constexpr (V == 4) {
+          const float2 co = *reinterpret_cast<const float2*>(cs + (c >> 1)), si = *reinterpret_cast<const float2*>(cs + n + (c >> 1));
+          const float r0 = x[0] * co.x - x[1] * si.x, r2 = x[2] * co.y - x[3] * si.y;
+          x[1] = x[1] * co.x + x[0] * si.x;
+          x[3] = x[3] * co.y + x[2] * si.y;
+          x[0] = r0;
+          x[2] = r2;
+        } else {
+          x[0] = x[0] * cs[c >> 1] + ((c & 1) ? y[0] : -y[0]) * cs[n + (c >> 1)];
+        }
+      }
+    } else if (c < 2 * n) {
       const int i = c < n ? c : c - n;
       const float sign = c < n ? -1.f : 1.f;
 #pragma unroll
@@ -283,7 +298,7 @@ __global__ void __launch_bounds__(256) rope_norm_append_kernel(const __grid_cons
 #pragma unroll
     for (int j = 0; j < V; ++j) ss += x[j] * x[j];
     const float inv = p.norm ? 1.f / sqrtf(warp_sum(ss) / float(dim) + p.a.eps) : 1.f;
-    const int from = c < n ? lane + n / V : (c < 2 * n ? lane - n / V : lane);
+    const int from = p.pairs ? (V == 1 ? lane ^ 1 : lane) : c < n ? lane + n / V : (c < 2 * n ? lane - n / V : lane);
     float y[V];
 #pragma unroll
     for (int j = 0; j < V; ++j) y[j] = __shfl_sync(0xffffffffu, x[j], from);
@@ -303,7 +318,7 @@ __global__ void __launch_bounds__(256) rope_norm_append_kernel(const __grid_cons
 #pragma unroll
     for (int j = 0; j < V; ++j) x[j] = y[j] = 0.f;
     if (c < dim) load(x, c);
-    if (c < 2 * n) load(y, c < n ? c + n : c - n);
+    if (c < 2 * n) load(y, p.pairs ? (V == 1 ? c ^ 1 : c) : c < n ? c + n : c - n);
     finish(x, y, c, inv);
   }
 }
@@ -356,7 +371,7 @@ __global__ void __launch_bounds__(256) rope_norm_append8_kernel(const __grid_con
       x[4] += hi.x; x[5] += hi.y; x[6] += hi.z; x[7] += hi.w;
     }
     float ss = 0.f, y[8];
-    const int from = c < n ? lane + n / 8 : (c < 2 * n ? lane - n / 8 : lane);
+    const int from = p.pairs ? lane : c < n ? lane + n / 8 : (c < 2 * n ? lane - n / 8 : lane);
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       ss += x[e] * x[e];
@@ -373,7 +388,17 @@ __global__ void __launch_bounds__(256) rope_norm_append8_kernel(const __grid_con
       pad = p.a.vdim;
     } else {
       const float inv = p.norm ? 1.f / sqrtf(ss / float(dim) + p.a.eps) : 1.f;
-      if (c < 2 * n) {
+      if (p.pairs && c < 2 * n) {
+        const float* cs = p.cos_sin + (long long)min(max(p.positions[tok[i]], 0), p.max_pos - 1) * p.rot_dims + (c >> 1);
+        const float4 co = *reinterpret_cast<const float4*>(cs), si = *reinterpret_cast<const float4*>(cs + n);
+        const float cv[4] = {co.x, co.y, co.z, co.w}, sv[4] = {si.x, si.y, si.z, si.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float r = x[2 * e] * cv[e] - x[2 * e + 1] * sv[e];
+          x[2 * e + 1] = x[2 * e + 1] * cv[e] + x[2 * e] * sv[e];
+          x[2 * e] = r;
+        }
+      } else if (c < 2 * n) {
         const float* cs = p.cos_sin + (long long)min(max(p.positions[tok[i]], 0), p.max_pos - 1) * p.rot_dims + (c < n ? c : c - n);
         const float sign = c < n ? -1.f : 1.f;
         const float4 c0 = *reinterpret_cast<const float4*>(cs), c1 = *reinterpret_cast<const float4*>(cs + 4);
@@ -452,12 +477,16 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) maps_simple_kernel(const __
     for (int i = 0; i < COLS; ++i) o[mp][i] = 0.f;
   }
   const int pages = pos / kMapsPage + 1;
-  const int lo = nkb_first_visible(pos, p.a.window, p.a.chunk);
-  for (int pg = lo / kMapsPage + warp; pg < pages; pg += kSimpleWarps) {
+  const int lo = nkb_first_visible(pos, p.a.window, p.a.chunk), page_lo = lo / kMapsPage;
+  const int keep = p.a.keep_first, kept = min((keep + kMapsPage - 1) / kMapsPage, page_lo);   // pages of kept tokens before the window
+  const float da = p.a.dist_a ? p.a.dist_a[h] : 0.f, db = p.a.dist_a ? p.a.dist_b[h] : 0.f;
+  for (int i = warp; i < kept + pages - page_lo; i += kSimpleWarps) {
+    const int pg = i < kept ? i : i - kept + page_lo;
     const long long blk = table[pg];
     const T* kr = reinterpret_cast<const T*>(p.k_cache) + ((blk * p.a.kv_heads + g) * kMapsPage + lane) * kw;
     const T* vb = reinterpret_cast<const T*>(p.v_cache) + (blk * p.a.kv_heads + g) * kMapsPage * v_ld;
-    const bool vis = pg * kMapsPage + lane <= pos && pg * kMapsPage + lane >= lo;
+    const int key = pg * kMapsPage + lane;
+    const bool vis = key <= pos && (key >= lo || key < keep);
     const int nvis = min(kMapsPage, pos + 1 - pg * kMapsPage);
     float pr[MAPS];
 #pragma unroll
@@ -467,6 +496,7 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) maps_simple_kernel(const __
         for (int c = 0; c < p.a.dim; ++c) s = fmaf(q_s[mp * p.a.dim_p + c], cast_in<T>(kr[mp * p.a.dim_p + c]), s);
         s *= p.a.scale;
         if (p.a.softcap > 0.f) s = p.a.softcap * tanhf(s / p.a.softcap);
+        if (p.a.dist_a) s -= da * log1pf(db * float(pos - key));
       } else {
         s = -INFINITY;
       }
@@ -898,20 +928,22 @@ extern "C" int nkb_row_norm_append(const NkbMapsArgs* a, const NkbProj* q, const
 
 extern "C" int nkb_rope_norm_append(const NkbMapsArgs* a, const NkbProj* q, const NkbProj* k, const NkbProj* v,
                                     const float* bias, const float* cos_sin, int rot_dims, int max_pos, const int* positions,
-                                    const int* slots, int norm, void* q_out, void* k_cache, void* v_cache, int bf16, int tokens,
+                                    const int* slots, int norm, int pairs, void* q_out, void* k_cache, void* v_cache, int bf16, int tokens,
                                     int block_size, void* stream) {
   if (tokens <= 0) return 0;
   if (!maps_ok(*a) || a->maps != 1 || block_size != kMapsPage || rot_dims < 0 || rot_dims > a->dim || (rot_dims & 1) ||
-      max_pos < 1 || (k->ptr && !v->ptr))
+      max_pos < 1 || (k->ptr && !v->ptr) || (rot_dims > 0 && !cos_sin))
     return -2;
   RopeNormAppendParams p{};
   p.q = *q; p.k = *k; p.v = *v; p.a = *a;
   p.bias = bias; p.cos_sin = cos_sin; p.positions = positions; p.slots = slots;
   p.q_out = q_out; p.k_cache = k_cache; p.v_cache = v_cache;
-  p.rot_dims = rot_dims; p.max_pos = max_pos; p.tokens = tokens; p.norm = norm;
+  p.rot_dims = rot_dims; p.max_pos = max_pos; p.tokens = tokens; p.norm = norm; p.pairs = pairs;
   const auto al16 = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
-  const bool vec = ((a->dim | a->dim_p | a->vdim | a->vdim_p) & 3) == 0 && (rot_dims & 7) == 0 && proj_vec4_ok(*q) &&
-                   proj_vec4_ok(*k) && proj_vec4_ok(*v) && al16(q_out) && al16(k_cache) && al16(v_cache);
+  // whole vectors on one side of the rotation's end (and, with halves, of its middle); angles in aligned runs
+  const int half = pairs ? 1 : 2;
+  const bool vec = ((a->dim | a->dim_p | a->vdim | a->vdim_p) & 3) == 0 && rot_dims % (4 * half) == 0 && proj_vec4_ok(*q) &&
+                   proj_vec4_ok(*k) && proj_vec4_ok(*v) && al16(cos_sin) && al16(q_out) && al16(k_cache) && al16(v_cache);
   const long long warps = (long long)tokens * (a->heads + (k->ptr ? 2 * a->kv_heads : 0));
   if (warps > 0x7fffffffll) return -2;
   const dim3 grid(unsigned((warps + 7) / 8)), block(256);
@@ -919,7 +951,7 @@ extern "C" int nkb_rope_norm_append(const NkbMapsArgs* a, const NkbProj* q, cons
   using bf = __nv_bfloat16;
   const auto whole = [&](const NkbProj& x) { return !x.ptr || (x.bf16 && al16(x.ptr) && (x.ld & 7) == 0); };
   const int wide = a->dim_p > a->vdim ? a->dim_p : a->vdim;
-  if (bf16 && ((a->dim | a->dim_p | a->vdim | a->vdim_p) & 7) == 0 && (rot_dims & 15) == 0 && wide <= 256 && whole(*q) && whole(*k) &&
+  if (bf16 && ((a->dim | a->dim_p | a->vdim | a->vdim_p) & 7) == 0 && rot_dims % (8 * half) == 0 && wide <= 256 && whole(*q) && whole(*k) &&
       whole(*v) && al16(q_out) && al16(k_cache) && al16(v_cache) && al16(bias) && al16(cos_sin)) {
     if (wide <= 64) return launch_rope_norm_append8<8>(p, warps, s);
     if (wide <= 128) return launch_rope_norm_append8<16>(p, warps, s);
@@ -947,7 +979,9 @@ extern "C" int nkb_maps_attn_simple(const NkbMapsArgs* a, const void* q, const v
                                     const int* context_lens, void* out, int bf16, int batch, int total_q, int block_size,
                                     int max_blocks_per_seq, void* stream) {
   if (batch <= 0 || total_q <= 0) return 0;
-  if (!maps_ok(*a) || block_size != kMapsPage || a->heads > 65535 || (a->sinks && a->maps != 1)) return -2;
+  if (!maps_ok(*a) || block_size != kMapsPage || a->heads > 65535 || ((a->sinks || a->dist_a || a->keep_first > 0) && a->maps != 1) ||
+      a->keep_first < 0 || !a->dist_a != !a->dist_b)
+    return -2;
   MapsSimpleParams p{};
   p.a = *a; p.q = q; p.k_cache = k_cache; p.v_cache = v_cache;
   p.block_table = block_table; p.q_start = q_start; p.q_lens = q_lens; p.context_lens = context_lens;
@@ -977,7 +1011,7 @@ extern "C" int nkb_maps_attn_decode(const NkbMapsArgs* a, const void* q, const v
                                     void* stream) {
   if (batch <= 0) return 0;
   if (!maps_ok(*a) || block_size != kMapsPage || batch > 65535) return -2;
-  if (a->maps != 2 || a->window > 0 || a->chunk > 0 || a->sinks || (a->dim_p != 32 && a->dim_p != 64) || (a->vdim_p != 64 && a->vdim_p != 128)) return -5;
+  if (a->maps != 2 || a->window > 0 || a->chunk > 0 || a->sinks || a->dist_a || (a->dim_p != 32 && a->dim_p != 64) || (a->vdim_p != 64 && a->vdim_p != 128)) return -5;
   if (!status_word() && nkb_init() != 0) return -1;
   MapsDecodeParams p{};
   p.a = *a;

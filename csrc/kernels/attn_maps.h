@@ -4,8 +4,9 @@
 // maps the head's result is
 //     o = a_0 - lambda * a_1;     o <- out_scale * o / sqrt(mean(o^2) + eps)
 // and with one map it is a_0.  softcap > 0 replaces a score s by softcap * tanh(s / softcap); window > 0 limits a query to
-// itself and the window - 1 tokens before it, chunk > 0 to the tokens of its own chunk of that many positions; sinks holds
-// per head (one map) the logarithm of an addend of the softmax's denominator.
+// itself and the window - 1 tokens before it (and the first keep_first tokens), chunk > 0 to the tokens of its own chunk of that
+// many positions; sinks holds per head (one map) the logarithm of an addend of the softmax's denominator.  dist_a and dist_b, per
+// head (one map): after the cap a score loses dist_a * ln(1 + dist_b * distance).
 #pragma once
 
 struct NkbMapsArgs {
@@ -16,9 +17,18 @@ struct NkbMapsArgs {
   // elements between tokens / heads of queries and results, 0: one token's heads side by side
   long long q_token, q_head, o_token, o_head;
   int v_ld;                              // elements between the values of two tokens, 0: vdim_p (values inside wider rows)
+  int keep_first;                        // with a window: the first tokens every query sees
+  const float *dist_a, *dist_b;          // [heads] or null
 };
 
-// First position a query at `pos` sees.
+// What the kernels of plain attention (attn_prefill.cu, attn_decode.cu) do to a score beyond scaling it.
+struct NkbScoreMods {
+  float softcap;                         // <= 0: none
+  int keep_first;
+  const float *dist_a, *dist_b;
+};
+
+// First position a query at `pos` sees (kept first tokens aside).
 static inline
 #ifdef __CUDACC__
 __host__ __device__

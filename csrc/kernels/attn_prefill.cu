@@ -72,6 +72,7 @@ struct PrefillParams {
   int* status;
   int nq, nkv, max_blocks, causal, window, chunk;
   float scale_log2;
+  NkbScoreMods mods;                   // MODS only
 };
 
 struct PrefillCtrl {
@@ -124,7 +125,9 @@ struct PrefillSmem {
   static constexpr int kBytes = 2 * kQBytes + kStages * kStageBytes + 2 * kPBytes + int(sizeof(PrefillCtrl)) + 1024 + 64;
 };
 
-template <int NK, int NV, int KT, bool ROWS>
+// MODS: scores are capped, lose a term that grows with the distance, or the first tokens stay visible outside the window.  The cap is
+// the one of attn_maps_prefill.cu (an odd polynomial where all scores of a row are small, the exponential form otherwise).
+template <int NK, int NV, int KT, bool ROWS, bool MODS>
 __global__ void __launch_bounds__(kPfThreads, 1)
 flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                           const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmR,
@@ -145,11 +148,22 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
   const int q_row0 = p.q_start[b] + qt * kQPair;        // row in the packed q / out arrays
   const int kvh = head / (p.nq / p.nkv);
   const TileRange tr0 = tile_range<KT>(p, qt * kQPair, q_len, ctx);
-  const TileRange tr1 = tile_range<KT>(p, qt * kQPair + kQTile, q_len, ctx);
+  TileRange tr1 = tile_range<KT>(p, qt * kQPair + kQTile, q_len, ctx);
   const bool two = tr1.rows > 0;
   // union of the two ranges; every tile of it is attended to by at least one query tile
   const int u_lo = tr0.lo, u_hi = two ? max(tr0.hi, tr1.hi) : tr0.hi;
-  const int n_union = u_hi - u_lo;
+  // KV tiles of kept first tokens come ahead of the union (those that are not in it).  Where they reach into it, the second query
+  // tile walks all of the union: a tile it sees nothing of is masked.
+  int kept = 0;
+  if constexpr (MODS) {
+    kept = (p.mods.keep_first + KT - 1) / KT;
+    if (kept > u_lo) {
+      kept = u_lo;
+      if (two) tr1.lo = u_lo;
+    }
+  }
+  const int n_union = kept + u_hi - u_lo;
+  const auto tile_at = [&](int x) { return MODS && x < kept ? x : x - kept + u_lo; };     // KV tile of walk position x
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -210,7 +224,7 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
     bool live = true;
     auto load = [&](bool is_v, int x) {
       if (!live) return;
-      const int j = u_lo + x;
+      const int j = tile_at(x);
       const int st = seq % kKVStages;
       const uint32_t ph = uint32_t(seq / kKVStages) & 1u;
       ++seq;
@@ -267,8 +281,11 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
     const uint32_t p_lo = uint32_t(make_smem_desc_sw128(smem_u32(p_s + t * kPBytes), 0, 1024));
     const uint64_t hk = uint64_t(uint32_t(make_smem_desc_sw128(0, 0, 1024) >> 32)) << 32;   // SBO, version, swizzle
     const uint32_t lbo_v = (uint32_t(kKVHalf) >> 4) << 16;                                  // low-word part of V's LBO
-    const int a_lo = t == 0 ? tr0.lo - u_lo : (two ? tr1.lo - u_lo : 0);
-    const int a_hi = t == 0 ? tr0.hi - u_lo : (two ? tr1.hi - u_lo : 0);
+    // walk positions of this query tile: the kept tiles and [a_lo, a_hi)
+    const int a_lo = kept + (t == 0 ? tr0.lo - u_lo : (two ? tr1.lo - u_lo : 0));
+    const int a_hi = kept + (t == 0 ? tr0.hi - u_lo : (two ? tr1.hi - u_lo : 0));
+    const auto attends = [&](int x) { return (MODS && x < kept) || (x >= a_lo && x < a_hi); };
+    const auto turn_of = [&](int x) { return uint32_t(MODS && x < kept ? x : x - a_lo + kept); };
     const uint32_t s_tmem = tmem_base + kSCol + t * 128, o_tmem = tmem_base + kOCol + t * 128;
     if ((t == 0 || two) && elect_one()) {
       bool ok = pf_wait(&ctrl->q_full, 0, abort_flag, p.status, ERR_WAIT_SMEM_FULL);
@@ -279,8 +296,8 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         const int item = seq++, st = item % kKVStages;
         ok = pf_wait(&ctrl->kv_full[st], uint32_t(item / kKVStages) & 1u, abort_flag, p.status, ERR_WAIT_SMEM_FULL);
         if (!ok) return;
-        if (x >= a_lo && x < a_hi) {
-          const uint32_t lit = uint32_t(x - a_lo);
+        if (attends(x)) {
+          const uint32_t lit = turn_of(x);
           ok = pf_wait(&ctrl->s_empty[t], (lit & 1u) ^ 1u, abort_flag, p.status, ERR_WAIT_TMEM_EMPTY);
           if (!ok) return;
           tc_fence_after();
@@ -305,8 +322,8 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         const int item = seq++, st = item % kKVStages;
         ok = pf_wait(&ctrl->kv_full[st], uint32_t(item / kKVStages) & 1u, abort_flag, p.status, ERR_WAIT_SMEM_FULL);
         if (!ok) return;
-        if (x >= a_lo && x < a_hi) {
-          const uint32_t lit = uint32_t(x - a_lo);
+        if (attends(x)) {
+          const uint32_t lit = turn_of(x);
           ok = pf_wait(&ctrl->p_full[t], lit & 1u, abort_flag, p.status, ERR_WAIT_SOFTMAX);
           if (!ok) return;
           tc_fence_after();
@@ -345,16 +362,25 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
     const uint32_t s_addr = tmem_base + lane_off + kSCol + t * 128;
     const uint32_t o_addr = tmem_base + lane_off + kOCol + t * 128;
     uint8_t* my_p = p_s + t * kPBytes + r * 128;
-    const int n_tiles = tr.hi - tr.lo;
-    const int n_other = t == 0 ? (two ? tr1.hi - tr1.lo : 0) : tr0.hi - tr0.lo;   // KV tiles of the other query tile
+    const int n_tiles = (tr.rows > 0 ? kept : 0) + tr.hi - tr.lo;
+    // KV tiles of the other query tile
+    const int n_other = t == 0 ? (two ? kept + tr1.hi - tr1.lo : 0) : kept + tr0.hi - tr0.lo;
     float m = -INFINITY, l = 0.f;
     int hi_pos = ctx - 1;
     if (p.causal) hi_pos = min(hi_pos, q_pos);
     const int lo_pos = nkb_first_visible(q_pos, p.window, p.chunk);
     bool alive = true;
+    constexpr float kLog2e = 1.4426950408889634f;
+    const bool capped = MODS && p.mods.softcap > 0.f, distant = MODS && p.mods.dist_a != nullptr;
+    const float k_y = capped ? p.scale_log2 / (kLog2e * p.mods.softcap) : 0.f;   // raw score -> argument of tanh
+    const float cap2 = p.mods.softcap * kLog2e;
+    const float poly_raw = capped ? 0.6f / fmaxf(fabsf(k_y), 1e-30f) : 0.f;
+    const float dist_a = distant ? p.mods.dist_a[head] : 0.f, dist_b = distant ? p.mods.dist_b[head] : 0.f;
+    // raw scores become exponents of two in the exponential's multiply-add, or (MODS) before it
+    const float to_log2 = MODS ? 1.f : p.scale_log2;
 
     for (int it = 0; it < n_tiles; ++it) {
-      const int kv0 = (tr.lo + it) * kKVTile;
+      const int kv0 = (MODS && it < kept ? it : tr.lo + it - kept) * kKVTile;
       bool ok = pf_wait(&ctrl->s_full[t], uint32_t(it) & 1u, abort_flag, p.status, ERR_WAIT_TMEM_FULL);
       if (!__all_sync(0xffffffffu, ok)) { alive = false; break; }
       tc_fence_after();
@@ -366,13 +392,59 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       __syncwarp();
       if (lane == 0) mbar_arrive(&ctrl->s_empty[t]);   // the scores are in registers: S_t may be overwritten
 
+      if constexpr (MODS) {
+        if (capped) {
+          float am4[4];
+#pragma unroll
+          for (int i = 0; i < 4; ++i) am4[i] = fmaxf(fabsf(__uint_as_float(v[2 * i])), fabsf(__uint_as_float(v[2 * i + 1])));
+#pragma unroll
+          for (int i = 8; i < kKVTile; i += 2)
+            am4[(i >> 1) & 3] = fmax3(am4[(i >> 1) & 3], fabsf(__uint_as_float(v[i])), fabsf(__uint_as_float(v[i + 1])));
+          const float am = fmaxf(fmaxf(am4[0], am4[1]), fmaxf(am4[2], am4[3]));
+          if (__all_sync(0xffffffffu, am <= poly_raw)) {
+            // y * P(y^2), P(u) ~ tanh(sqrt(u)) / sqrt(u) on [0, 0.36]
+            const float2 ky2 = make_float2(k_y, k_y), c2 = make_float2(cap2, cap2);
+            const auto dup = [](float x) { return make_float2(x, x); };
+#pragma unroll
+            for (int i = 0; i < kKVTile; i += 2) {
+              const float2 y = fmul2(make_float2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), ky2);
+              const float2 u = fmul2(y, y);
+              float2 q = ffma2(u, dup(-0.005856427870f), dup(0.020757475450f));
+              q = ffma2(q, u, dup(-0.053769921786f));
+              q = ffma2(q, u, dup(0.133317047022f));
+              q = ffma2(q, u, dup(-0.333332839718f));
+              q = ffma2(q, u, dup(0.999999997563f));
+              const float2 w = fmul2(fmul2(y, c2), q);
+              v[i] = __float_as_uint(w.x);
+              v[i + 1] = __float_as_uint(w.y);
+            }
+          } else {
+            const float k_e = 2.f * kLog2e * k_y;
+#pragma unroll
+            for (int i = 0; i < kKVTile; ++i) {
+              const float e = exp2f(__uint_as_float(v[i]) * k_e);
+              v[i] = __float_as_uint(fmaf(-2.f * cap2, __fdividef(1.f, e + 1.f), cap2));
+            }
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < kKVTile; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * p.scale_log2);
+        }
+        if (distant) {
+          // dist_a ln(1 + dist_b d) in units of ln 2; keys after the query (negative distances) are masked below
+          const float d0 = fmaf(dist_b, float(q_pos - kv0), 1.f);
+#pragma unroll
+          for (int i = 0; i < kKVTile; ++i)
+            v[i] = __float_as_uint(fmaf(-dist_a, __log2f(fmaf(-dist_b, float(i), d0)), __uint_as_float(v[i])));
+        }
+      }
       // the mask only on tiles that cross the causal diagonal, the end of the context or the window edge
-      const bool edge = kv0 + kKVTile - 1 > hi_pos || kv0 < lo_pos;
+      const bool edge = kv0 + kKVTile - 1 > hi_pos || (kv0 < lo_pos && (!MODS || kv0 + kKVTile > p.mods.keep_first));
       if (__any_sync(0xffffffffu, edge)) {
-        const int hi_rel = hi_pos - kv0, lo_rel = lo_pos - kv0;
+        const int hi_rel = hi_pos - kv0, lo_rel = lo_pos - kv0, keep_rel = MODS ? p.mods.keep_first - kv0 : 0;
 #pragma unroll
         for (int i = 0; i < kKVTile; ++i)
-          if (i > hi_rel || i < lo_rel) v[i] = 0xff800000u;   // -inf
+          if (i > hi_rel || (i < lo_rel && (!MODS || i >= keep_rel))) v[i] = 0xff800000u;   // -inf
       }
       // four independent chains of three-input maxima instead of one 128-long dependent chain
       float mx4[4];
@@ -382,7 +454,7 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       for (int i = 8; i < kKVTile; i += 2)
         mx4[(i >> 1) & 3] = fmax3(mx4[(i >> 1) & 3], __uint_as_float(v[i]), __uint_as_float(v[i + 1]));
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-      mx *= p.scale_log2;
+      mx *= to_log2;
 
       bool p_free = it == 0;     // the P_t buffer may be overwritten (P V of the previous tile has finished)
       if (it == 0) {
@@ -411,7 +483,7 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         }
       }
       const float base = (m == -INFINITY) ? 0.f : m;
-      const float2 sc2 = make_float2(p.scale_log2, p.scale_log2), nb2 = make_float2(-base, -base);
+      const float2 sc2 = make_float2(to_log2, to_log2), nb2 = make_float2(-base, -base);
       float2 sum2[4];
 #pragma unroll
       for (int i = 0; i < 4; ++i) sum2[i] = make_float2(0.f, 0.f);
@@ -520,7 +592,7 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
   }
 }
 
-template <int NK, int NV, int KT, bool ROWS>
+template <int NK, int NV, int KT, bool ROWS, bool MODS = false>
 static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tr,
                           const PrefillParams& p, int batch, int max_q_len, cudaStream_t s) {
   constexpr int smem = PrefillSmem<NK, NV, KT>::kBytes;
@@ -529,13 +601,13 @@ static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CU
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -1;
   if (!attr_set[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(flash_attn_prefill_kernel<NK, NV, KT, ROWS>,
+    cudaError_t e = cudaFuncSetAttribute(flash_attn_prefill_kernel<NK, NV, KT, ROWS, MODS>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return int(e);
     attr_set[dev] = true;
   }
   dim3 grid((max_q_len + kQPair - 1) / kQPair, p.nq, batch);
-  return launch_pdl(flash_attn_prefill_kernel<NK, NV, KT, ROWS>, grid, dim3(kPfThreads), size_t(smem), s, tq, tk, tv, tr, p);
+  return launch_pdl(flash_attn_prefill_kernel<NK, NV, KT, ROWS, MODS>, grid, dim3(kPfThreads), size_t(smem), s, tq, tk, tv, tr, p);
 }
 
 }  // namespace nkb
@@ -546,9 +618,11 @@ extern "C" int nkb_flash_attn_prefill(const void* q, const void* k_cache, const 
                                       const int* q_start, const int* q_lens, const int* context_lens, void* out,
                                       int batch, int total_q, int max_q_len, int nq, int nkv, int head_dim,
                                       int block_size, int num_blocks, int max_blocks_per_seq, float scale, int causal,
-                                      int window, int chunk, const float* sinks, void* stream) {
+                                      int window, int chunk, const float* sinks, const NkbScoreMods* mods, void* stream) {
   if (batch <= 0 || total_q <= 0) return 0;
   if (block_size != kPfPage || nq % nkv != 0) return -2;
+  if (mods && (mods->keep_first < 0 || (mods->keep_first > 0 && chunk > 0) || !mods->dist_a != !mods->dist_b || (!causal && mods->dist_a)))
+    return -2;
   if (!status_word() && nkb_init() != 0) return -1;
   PrefillParams p{};
   p.block_table = block_table;
@@ -576,6 +650,12 @@ extern "C" int nkb_flash_attn_prefill(const void* q, const void* k_cache, const 
     if (encode_tmap_bf16(&tv, v_cache, 4, dims, strides, box)) return -4;
   }
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (mods) {
+    p.mods = *mods;
+    if (head_dim == 128) return launch_prefill<2, 2, 128, false, true>(tq, tk, tv, tk, p, batch, max_q_len, s);
+    if (head_dim == 64) return launch_prefill<1, 1, 128, false, true>(tq, tk, tv, tk, p, batch, max_q_len, s);
+    return -2;
+  }
   if (head_dim == 128) return launch_prefill<2, 2, 128, false>(tq, tk, tv, tk, p, batch, max_q_len, s);
   if (head_dim == 64) return launch_prefill<1, 1, 128, false>(tq, tk, tv, tk, p, batch, max_q_len, s);
   return -2;

@@ -345,7 +345,8 @@ gated_residual_kernel(const __grid_constant__ GatedResidualParams p) {
 }
 
 // act(gate) * up, or act(gate) alone when up.ptr is null; up_rows: row up_rows[t] of up (a table of up_limit rows) instead
-// of row t; ACT_CLAMPED: g sigmoid(alpha g) (u + 1) of g = min(gate, limit), u = clamp(up, -limit, limit)
+// of row t; ACT_CLAMPED: g sigmoid(alpha g) (u + 1) of g = min(gate, limit), u = clamp(up, -limit, limit); ACT_XIELU: its
+// parameters are limit and alpha
 template <int V, typename OutT>
 __global__ void __launch_bounds__(256) gated_act_kernel(const __grid_constant__ NkbProj gate,
                                                         const __grid_constant__ NkbProj up, OutT* __restrict__ out,
@@ -375,6 +376,9 @@ __global__ void __launch_bounds__(256) gated_act_kernel(const __grid_constant__ 
         const float gc = fminf(g[j], limit), uc = fminf(fmaxf(u[j], -limit), limit);
         g[j] = gc / (1.f + expf(-alpha * gc)) * (uc + 1.f);
       }
+    } else if (kind == ACT_XIELU) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) g[j] = xielu(g[j], limit, alpha) * u[j];
     } else {
 #pragma unroll
       for (int j = 0; j < V; ++j) g[j] = apply_act(g[j], kind) * u[j];
@@ -518,7 +522,7 @@ extern "C" int nkb_gated_act(const NkbProj* gate, const NkbProj* up, void* out, 
   };
   using bf = __nv_bfloat16;
   const long long pieces = (long long)rows * (inter / 8);
-  if (out_bf16 && gate->bf16 && up->ptr && up->bf16 && !up_rows && inter % 8 == 0 && ((gate->ld | up->ld) & 7) == 0 &&
+  if (out_bf16 && kind != ACT_XIELU && gate->bf16 && up->ptr && up->bf16 && !up_rows && inter % 8 == 0 && ((gate->ld | up->ld) & 7) == 0 &&
       aligned16(gate->ptr) && aligned16(up->ptr) && aligned16(out) && pieces < (1ll << 30))
     return launch_pdl(gated_act8_kernel, dim3(unsigned((pieces + 511) / 512)), dim3(256), 0, s, *gate, *up, reinterpret_cast<bf*>(out),
                       int(pieces), inter / 8, kind, limit, alpha);

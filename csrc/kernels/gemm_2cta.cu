@@ -32,7 +32,8 @@ struct Gemm2Args {            // <= 128 bytes (see GemmArgs)
   int group_m;                // row tiles that share one sweep over the column tiles (L2 reuse)
   int gated;                  // B holds [gate; up] rows: the pair's first CTA loads gate rows, the second up rows
   int gate_off;               // row offset of the up half in B
-  int act;                    // gated: 0 = SiLU, 1 = GELU (tanh form); plain: 2 = squared ReLU
+  int act;                    // gated: 0 = SiLU, 1 = GELU (tanh form); plain: 2 = squared ReLU, 7 = xIELU of act_a, act_b
+  float act_a, act_b;
   long long ldo;
   void* out;
   const __nv_bfloat16* bias;
@@ -243,7 +244,10 @@ gemm2_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CU
             if (cbase + j < args.n)
               v[j] = __float_as_uint(__uint_as_float(v[j]) + __bfloat162float(args.bias[cbase + j]));
         }
-        if (args.act == 2) {
+        if (args.act == 7) {       // xIELU
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(xielu_f(__uint_as_float(v[j]), args.act_a, args.act_b));
+        } else if (args.act == 2) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const float r = fmaxf(__uint_as_float(v[j]), 0.f);
@@ -313,11 +317,11 @@ extern "C" int nkb_gemm_2cta_pairs() { return g_pairs_last; }
 
 // gated != 0: B holds [gate; up] (2 x n rows, the up half starting at row gate_off) and out[m, n] =
 // silu(A gate^T) * (A up^T); bias / residual are not applied in that mode.  act 1: GELU in place of SiLU; 2 (not gated):
-// the square of the positive part of (A B^T + bias).
+// the square of the positive part of (A B^T + bias); 7 (not gated): xIELU with the parameters act_a, act_b.
 extern "C" int nkb_gemm_bf16_2cta(const void* A, const void* B, void* out, int m, int n, int k, long long lda,
                                   long long ldb, long long ldo, const void* bias, const void* residual, int gated,
-                                  int gate_off, int act, void* stream) {
-  if (act < 0 || act > 2 || (act == 2 && gated)) return -2;
+                                  int gate_off, int act, float act_a, float act_b, void* stream) {
+  if (act < 0 || (act > 2 && act != 7) || (act >= 2 && gated)) return -2;
   if (!status_word() && nkb_init() != 0) return -1;
   if (m <= 0 || n <= 0 || k <= 0) return -2;
   if ((k & 7) || (lda & 7) || (ldb & 7)) return -2;
@@ -329,6 +333,8 @@ extern "C" int nkb_gemm_bf16_2cta(const void* A, const void* B, void* out, int m
   a.gated = gated ? 1 : 0;
   a.gate_off = gate_off;
   a.act = act;
+  a.act_a = act_a;
+  a.act_b = act_b;
   if (gated && (bias || residual)) return -2;
   a.kb_total = (k + kBlockK - 1) / kBlockK;
   a.bias_on_cols = 1;

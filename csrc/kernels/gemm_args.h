@@ -23,7 +23,7 @@ struct GemmArgs {
   int out_fp32;
   int bias_on_rows;
   int stages;
-  int act;              // gated epilogue: 0 = SiLU, 1 = GELU (tanh form); plain: 2 = squared ReLU
+  int act;              // gated epilogue: 0 = SiLU, 1 = GELU (tanh form); plain: 2 = squared ReLU, 7 = xIELU of act_a, act_b
   int weights_operand;  // 0 = A, 1 = B holds immutable weights (may be fetched before the dependency wait), -1 none
   long long ldo;
   long long split_stride;
@@ -31,6 +31,7 @@ struct GemmArgs {
   const __nv_bfloat16* bias;
   const __nv_bfloat16* residual;
   int* status;
+  float act_a, act_b;
 };
 static_assert(sizeof(GemmArgs) <= 128, "GemmArgs grew past the fast kernel-parameter size");
 

@@ -167,10 +167,10 @@ extern "C" int nkb_gemm_bf16(const void* A, const void* B, void* out, int rows, 
                              long long ldb, long long ldo, int transpose_out, int out_fp32, int splits,
                              long long split_stride, int gated, int gate_off, const void* bias, int bias_on_rows,
                              const void* residual, int block_n, int max_ctas, int weights_operand, int ctas_per_sm,
-                             int act, void* stream) {
+                             int act, float act_a, float act_b, void* stream) {
   if (!status_word() && nkb_init() != 0) return -1;
-  if (act < 0 || act > 2) return -2;
-  if (act == 2 && (gated || transpose_out || splits > 1)) return -2;   // in the general epilogue of finished values only
+  if (act < 0 || (act > 2 && act != 7)) return -2;
+  if (act >= 2 && (gated || transpose_out || splits > 1)) return -2;   // in the general epilogue of finished values only
   if (rows <= 0 || cols <= 0 || k <= 0) return -2;
   if ((k & 7) || (lda & 7) || (ldb & 7)) return -2;
   if (splits > 1 && !out_fp32) return -2;
@@ -189,6 +189,8 @@ extern "C" int nkb_gemm_bf16(const void* A, const void* B, void* out, int rows, 
   args.num_col_tiles = (cols + block_n - 1) / block_n;
   args.gated = gated;
   args.act = act;
+  args.act_a = act_a;
+  args.act_b = act_b;
   args.gate_off = gate_off;
   args.transpose_out = transpose_out;
   args.out_fp32 = out_fp32;

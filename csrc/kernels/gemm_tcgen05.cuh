@@ -103,6 +103,9 @@ __device__ __forceinline__ WorkItem decode_work(const GemmArgs& a, const GroupAr
 }
 
 __device__ __forceinline__ float silu_f(float g) { return g / (1.f + __expf(-g)); }
+__device__ __forceinline__ float xielu_f(float z, float a, float b) {
+  return fmaf(0.5f, z, z > 0.f ? a * z * z : b * (__expf(z) - 1.f - z));
+}
 // tanh-form GELU with the exponential: (1 + tanh(w)) / 2 = 1 / (1 + exp(-2 w))
 __device__ __forceinline__ float gelu_tanh_f(float g) {
   return g / (1.f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g)));
@@ -613,7 +616,10 @@ __device__ __forceinline__ bool gemm_bf16_body(const CUtensorMap& tmA, const CUt
                 v[j] = __float_as_uint(__uint_as_float(v[j]) + __bfloat162float(args.bias[cbase + j]));
           }
         }
-        if (args.act == 2) {       // plain product: square of the positive part
+        if (args.act == 7) {       // xIELU
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(xielu_f(__uint_as_float(v[j]), args.act_a, args.act_b));
+        } else if (args.act == 2) {       // plain product: square of the positive part
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const float r = fmaxf(__uint_as_float(v[j]), 0.f);

@@ -132,6 +132,63 @@ class LatentAttentionSpec:
 
 
 @dataclass(frozen=True)
+class GroupedAttentionSpec:
+    """Grouped-query attention.  rope (None: no rotation): interleaved rotation of the first rope.dims dimensions; softcap > 0:
+    scores are capped; window > 0: the last `window` tokens and the first `keep_first` ones (0: all); distance: a score loses
+    r1 ln(1 + r2 distance), two numbers per head; sink, gate: one per head; bias: biases of all four projections.  kv_from: the
+    keys and values are those of that layer."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    softcap: float = 0.0
+    rope: Optional[RopeSpec] = None
+    window: int = 0
+    keep_first: int = 0
+    distance: bool = False
+    sink: bool = False
+    gate: bool = False
+    bias: bool = False
+    kv_from: Optional[int] = None
+    kind = "grouped"
+
+
+@dataclass(frozen=True)
+class DeltaSpec:
+    """Gated delta rule: `dim` by `vdim` states with one decay per head, short convolutions of `conv` taps on queries, keys and
+    values; query / key heads are shared by heads / kv_heads heads."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    kind = "delta"
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec:
+    """Mamba-2: `state` by `vdim` states with a scalar decay per head, input and read-out vectors in `groups`, a short convolution of
+    `conv` taps, gated results normed in `norm_groups` equal parts."""
+    heads: int
+    groups: int
+    state: int
+    vdim: int
+    conv: int
+    norm_groups: int = 1
+    kind = "ssd"
+
+
+@dataclass(frozen=True)
+class BlendSpec:
+    """Attention and a state-space mixer side by side on the same input; the mean of their results, each RMS-normed over the model's
+    width."""
+    left: GroupedAttentionSpec
+    right: StateSpaceSpec
+    kind = "blend"
+
+
+@dataclass(frozen=True)
 class ClampedSpec:
     """Gated feed-forward g sigmoid(1.702 g) (u + 1) with g at most `limit` and u within +-limit."""
     ff: int
@@ -159,10 +216,11 @@ class ExpertsSpec:
 @dataclass(frozen=True)
 class LayerSpec:
     """block "gated": mixer and gated feed-forward beside each other, a sigmoid gate on both results; "pre-norm": the
-    mixer, then the feed-forward (plain `act`, or `experts`), each added to the residual; "parallel": mixer and feed-forward
-    (gated `act`, or `experts`) on one norm, their sum added to the residual, then the per-layer token input."""
+    mixer, then the feed-forward (plain `act`, or `experts`), each added to the residual; "sandwich": the same with a norm after
+    each of the two as well; "parallel": mixer and feed-forward (gated `act`, or `experts`) on one norm, their sum added to
+    the residual, then the per-layer token input."""
     mixer: Union[MapsAttentionSpec, RecurrenceSpec, LinearAttentionSpec, ParallelSpec, ChunkAttentionSpec,
-                 LatentAttentionSpec]
+                 LatentAttentionSpec, GroupedAttentionSpec, DeltaSpec, BlendSpec]
     ff: int = 0                      # 0: no dense feed-forward
     act: str = "gelu_tanh"
     block: str = "gated"
@@ -220,6 +278,8 @@ class ModelConfig:
     norm_offset: float = 0.0              # added to the stored weights of the layer and final norms
     tie_embeddings: bool = False          # logits from the embedding table
     layer_norm: bool = False              # layer norms with bias instead of RMS norms
+    tanh_norm: bool = False               # tanh(alpha x) * w + b instead of RMS norms
+    depth_average: bool = False           # after a layer: weighted sum of the embedding output and all layers' results
     token_side: int = 0                   # width of the per-layer token input (0: none)
     logit_softcap: float = 0.0            # > 0: logits <- cap * tanh(logits / cap)
 
@@ -525,6 +585,69 @@ def ligizen_shape(width: int, *, layers: int, heads: int, kv_heads: int, ff: int
             specs.append(LayerSpec(mixer, ff, "silu", "parallel"))
     base = dict(name="ligizen", vocab_size=vocab, hidden_size=width, num_layers=layers, rms_eps=1e-5, layers=specs,
                 layer_norm=True, token_side=side, logit_softcap=50.0, max_position=0)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+def redodra_config(raw: dict, **kw) -> ModelConfig:
+    """`ModelConfig` of a Redodra config.json."""
+
+    def attention(m, **fields):
+        r, mask = m.get("rot"), m.get("mask") or {}
+        return GroupedAttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["scale"], m.get("softcap") or 0.0,
+                                    RopeSpec(r["base"], r["dims"]) if r else None, mask.get("size", 0),
+                                    mask.get("keep_first", 0), kv_from=m.get("kv_from"), **fields)
+
+    def mixer_of(kind, m):
+        if kind == "attention":
+            return attention(m, sink=True, gate=True)
+        if kind == "delta":
+            return DeltaSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"])
+        if kind == "parallel":
+            r = m["right"]
+            return BlendSpec(attention(m["left"], distance=True, bias=True),
+                             StateSpaceSpec(r["heads"], r["groups"], r["state"], r["vdim"], r["conv"], r["norm_groups"]))
+        raise ValueError(f"unknown layer type {kind!r}")
+
+    layers = []
+    for i, l in enumerate(raw["layers"]):
+        mlp = l.get("mlp")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise ValueError(f"unknown feed-forward kind {mlp['kind']!r}")
+        mixer = mixer_of(l["type"], l["mixer"])
+        src = getattr(mixer, "kv_from", None)
+        if src is not None and not (0 <= src < i and layers[src].mixer.kind == "grouped" and layers[src].mixer.kv_from is None):
+            raise ValueError(f"layer {i} cannot read the keys of layer {src}")
+        layers.append(LayerSpec(mixer, mlp["ff"] if mlp is not None else 0, "xielu", "sandwich"))
+    base = dict(name="redodra", vocab_size=raw["vocab"], hidden_size=raw["width"], num_layers=len(layers),
+                rms_eps=raw["norm"]["eps"], layers=layers, tanh_norm=True, depth_average=True, max_position=0)
+    base.update(kw)
+    return ModelConfig(**base)
+
+
+def redodra_shape(width: int, *, layers: int, heads: int, kv_heads: int, ff: int, vocab: int = 32000, dim: int = 128,
+                  window: int = 1024, keep_first: int = 4, state: int = 128, groups: int = 8, conv: int = 4,
+                  share_every: int = 0, **kw) -> ModelConfig:
+    """A Redodra configuration of regular shape: layers of the delta rule, the parallel mixer and attention take turns (delta rule and
+    parallel mixer twice as often as attention); with share_every, every share_every-th attention layer but the first reads the
+    keys and values of the attention layer before it."""
+    specs, attended, source = [], 0, None
+    for i in range(layers):
+        if i % 5 in (0, 2):
+            mixer = DeltaSpec(heads, heads, dim, dim, conv)
+        elif i % 5 in (1, 3):
+            mixer = BlendSpec(GroupedAttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, 30.0, None, window, keep_first,
+                                                   distance=True, bias=True),
+                              StateSpaceSpec(heads, groups, state, dim, conv, groups))
+        else:
+            attended += 1
+            shares = share_every and attended > 1 and attended % share_every == 0
+            mixer = GroupedAttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, 30.0, RopeSpec(500000.0, dim), sink=True,
+                                         gate=True, kv_from=source if shares else None)
+            source = source if shares else i
+        specs.append(LayerSpec(mixer, ff, "xielu", "sandwich"))
+    base = dict(name="redodra", vocab_size=vocab, hidden_size=width, num_layers=layers, rms_eps=1e-5, layers=specs,
+                tanh_norm=True, depth_average=True, max_position=0)
     base.update(kw)
     return ModelConfig(**base)
 

@@ -1,14 +1,16 @@
 """Decoders whose layers are listed one by one: each layer has its own token mixer (models/mixers.py) and feed-forward,
-around an fp32 residual stream.  Three kinds of layer:
+around an fp32 residual stream.  Four kinds of layer:
 
     gated (Tolenex)       h1 = norm1(x), h2 = norm2(x)
                           x <- x + sigmoid(W_g1 h1 + b1) * mixer(h1) + sigmoid(W_g2 h2 + b2) * feed_forward(h2)
     pre-norm (Mumilorn)   x <- x + mixer(norm1(x)),   then   x <- x + feed_forward(norm2(x))
+    sandwich (Redodra)    x <- x + norm1b(mixer(norm1(x))),   then   x <- x + norm2b(feed_forward(norm2(x)))
     parallel (Ligizen)    h = norm1(x);  x <- x + mixer(h) + feed_forward(h),  then  x <- x + norm(token input of x)
 
 A layer is a list of stages; a stage reads norms of the residual and returns the branches that are added to it.  One
 kernel per stage (`ops.gated_residual`) sums the branches, applies what precedes a repeated pass of a looped block and
-norms the result for the next stage.  The model plugs into the same engine, paged cache and decode graph as
+norms the result for the next stage.  With `depth_average` what leaves a layer is a weighted sum of the embedding output and all
+layers' results so far, which that kernel computes as well.  The model plugs into the same engine, paged cache and decode graph as
 `TransformerLM`.
 
 Batches of at most 128 tokens (decode steps, small mixed steps) run their projections as split-K GEMMs whose fp32
@@ -27,10 +29,11 @@ import torch
 
 from .. import ops
 from ..ops import Branch, Norm, Proj
+from ..ops.mixers import History
 from ..parallel.comm import TPGroup
 from .config import LayerSpec, ModelConfig, RopeSpec, rope_frequencies
 from .kv_cache import BLOCK_SIZE, PagedKVCache
-from .mixers import MIXERS, Tensors
+from .mixers import MIXERS, Tensors, padded_rows
 from .moe import RoutedExperts
 from .transformer import pick_splits
 
@@ -38,11 +41,12 @@ SMALL_BATCH = 128
 
 
 class Stage:
-    """norms: the residual's norms it reads (weights of RMS norms, or `ops.Norm`); run(h, entry, cache, batch) -> branches."""
-    __slots__ = ("norms", "run")
+    """norms: the residual's norms it reads (weights of RMS norms, or `ops.Norm`); run(h, entry, cache, batch) -> branches;
+    post: what their sum passes before it is added."""
+    __slots__ = ("norms", "run", "post")
 
-    def __init__(self, norms, run):
-        self.norms, self.run = norms, run
+    def __init__(self, norms, run, post: Optional[Norm] = None):
+        self.norms, self.run, self.post = norms, run, post
 
 
 class GatedLayer:
@@ -93,10 +97,13 @@ class GatedLayer:
 
 
 class DenseMLP:
-    """down(act(up h))."""
+    """down(act(up h)); xIELU's two parameters are the tensor `act`, through softplus."""
 
     def __init__(self, act: str, t: Tensors):
         self.act, self.up, self.down = act, t.mat("up"), t.mat("down")
+        if act == "xielu":
+            p, q = torch.nn.functional.softplus(t.raw("act").double(), threshold=100.0).tolist()
+            self.act = ops.Act("xielu", p, 0.5 + q)
 
     def weights(self):
         return [self.up, self.down]
@@ -156,6 +163,31 @@ class PreNormLayer:
         m = self.model
         y = m.project(h[0], self.mixer.w_in) if self.mixer.w_in is not None else None
         return [Branch(Proj(m.project(self.mixer.run(m, y, h[0], entry, cache, b), self.mixer.w_o), 0, self.width))]
+
+
+class SandwichLayer:
+    """Mixer, then feed-forward, each with a norm of the residual ahead of it and a norm of its result behind it."""
+
+    def __init__(self, model: "HybridLM", spec: LayerSpec, t: Tensors):
+        cfg = model.cfg
+        self.model, self.width = model, cfg.hidden_size
+        self.mixer = mixer = MIXERS[spec.mixer.kind](spec.mixer, t.under("mix."), cfg.rms_eps)
+        if sum(mixer.widths) != mixer.w_in.shape[0]:
+            raise ValueError("projection sizes do not fit the configuration")
+        mixer.w_in = padded_rows(mixer.w_in)
+        self.mlp = DenseMLP(spec.act, t.under("mlp.")) if spec.ff else None
+        self.stages = [Stage([model.norm(t, "norm1")], self._mix, model.norm(t, "norm1b"))]
+        if self.mlp is not None:
+            self.stages.append(Stage([model.norm(t, "norm2")], lambda h, *_: self.mlp.run(model, h[0]), model.norm(t, "norm2b")))
+
+    def weights(self):
+        ws = [self.mixer.w_in, self.mixer.w_o, *getattr(self.mixer, "weights", list)()]
+        return [w for w in ws if w is not None] + (self.mlp.weights() if self.mlp is not None else [])
+
+    def _mix(self, h, entry, cache, b) -> List[Branch]:
+        m = self.model
+        o = self.mixer.run(m, m.project(h[0], self.mixer.w_in), h[0], entry, cache, b)
+        return o if isinstance(o, list) else [Branch(Proj(m.project(o, self.mixer.w_o), 0, self.width))]
 
 
 class ParallelLayer:
@@ -222,7 +254,7 @@ class ParallelLayer:
         return [Branch(Proj(m.project(a, self.side_proj), 0, self.width), norm=self.side_norm)]
 
 
-LAYERS = {"gated": GatedLayer, "pre-norm": PreNormLayer, "parallel": ParallelLayer}
+LAYERS = {"gated": GatedLayer, "pre-norm": PreNormLayer, "sandwich": SandwichLayer, "parallel": ParallelLayer}
 
 
 class HybridLM:
@@ -252,12 +284,17 @@ class HybridLM:
             first[i] = n if source is None else first[source]
             self.entry.append(first[i])
             n += len(self.layers[i].mixer.entries())
+        if cfg.depth_average and cfg.loop:
+            raise ValueError("a depth average is over layers that run once")
+        self.averages = [get(f"l{i}.dwa").float().contiguous() for i in range(len(cfg.layers))] if cfg.depth_average else None
         self.loop_step = get("loop.step").float().contiguous() if cfg.loop else None
         self._rope: Dict[RopeSpec, torch.Tensor] = {}
         self._offsets: Dict[tuple, torch.Tensor] = {}
 
     def norm(self, t: Tensors, name: str) -> Norm:
         """The model's kind of norm, from the tensors of that name."""
+        if self.cfg.tanh_norm:
+            return Norm(t.f32(name), t.f32(name + ".b"), alpha=float(t.raw(name + ".alpha")))
         if self.cfg.layer_norm:
             return Norm(t.f32(name), t.f32(name + ".b"), center=True)
         return Norm(t.f32(name, self.cfg.norm_offset))
@@ -273,8 +310,8 @@ class HybridLM:
 
     def _extend_rope(self, positions: int) -> None:
         """cos / sin tables [positions, dims] of every rotation the layers use."""
-        for layer in self.cfg.layers:
-            rope = getattr(layer.mixer, "rope", None)
+        specs = [m for layer in self.cfg.layers for m in (layer.mixer, getattr(layer.mixer, "left", None))]
+        for rope in (getattr(m, "rope", None) for m in specs):
             if rope is not None and (rope not in self._rope or self._rope[rope].shape[0] < positions):
                 freq, mult = rope_frequencies(rope)
                 self._rope[rope] = ops.rope_table(rope.dims, positions, inv_freq=freq, scaling=mult, device=self.device)
@@ -332,8 +369,11 @@ class HybridLM:
             return pre
 
         first = ahead(0)
+        rows = None                          # results that later layers average: the embedding output, then every layer's
+        if cfg.depth_average:
+            rows = torch.empty((len(self.runs), ids.numel(), cfg.hidden_size), dtype=torch.float32, device=self.embed.device)
         x, h = ops.gated_residual(None, ids=ids, table=self.embed, scale=cfg.embedding_scale,
-                                  norms=[] if "add_row" in first else first["norms"], **norm)
+                                  norms=[] if "add_row" in first else first["norms"], out=None if rows is None else rows[0], **norm)
         embedded = x
         if "add_row" in first:
             x, h = ops.gated_residual(x, **first, **norm)
@@ -341,9 +381,13 @@ class HybridLM:
         for n, (r, s) in enumerate(plan):
             stages = self.layers[self.runs[r][0]].stages
             branches = stages[s].run(h, self.entry[r], cache, b)
-            if return_hidden and s == len(stages) - 1:
-                taps.append(ops.gated_residual(x, branches, eps=cfg.rms_eps)[0])
-            x, h = ops.gated_residual(x, branches, **ahead(n + 1), **norm)
+            how = dict(post=stages[s].post)
+            if s == len(stages) - 1:
+                if rows is not None:
+                    how["history"] = History(rows, r + 1, self.averages[r], store=r + 1 < len(rows))
+                if return_hidden:
+                    taps.append(ops.gated_residual(x, branches, eps=cfg.rms_eps, **how)[0])
+            x, h = ops.gated_residual(x, branches, **ahead(n + 1), **how, **norm)
         return (h[0], taps) if return_hidden else h[0]
 
     # ------------------------------------------------------------------ the engine's entry points

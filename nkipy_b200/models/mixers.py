@@ -2,7 +2,8 @@
 
 A mixer owns the rows it puts into its layer's input projection (`w_in`), its entries of the cache (paged keys and values
 or per-sequence states), its output projection (`w_o`), and the step in between: `run` takes the input projection's result
-and returns the operand of the output projection.  A new kind of layer is a new class here beside a spec in config.py.
+and returns the operand of the output projection, or, where a mixer has no single output projection (`w_o` None), the branches
+of the residual.  A new kind of layer is a new class here beside a spec in config.py.
 """
 
 from __future__ import annotations
@@ -12,7 +13,7 @@ from typing import List, Union
 import torch
 
 from .. import ops
-from ..ops import Decay, LatentSpec, MapsSpec, Proj
+from ..ops import Branch, Decay, HeadRecurrence, LatentSpec, MapsSpec, Proj, ShortConv
 from ..ops.linear_attention import linear_state_shape
 from ..ops.mixers import hgrn2_state_shape
 from .kv_cache import KVLayer, StateLayer
@@ -48,6 +49,12 @@ def columns(y: Union[torch.Tensor, Proj], widths: List[int]) -> List[Proj]:
         out.append(Proj(t, c, w))
         c += w
     return out
+
+
+def padded_rows(w: torch.Tensor, to: int = 8) -> torch.Tensor:
+    """w [N, K] filled up with zero rows to a multiple of `to`."""
+    n = -w.shape[0] % to
+    return torch.cat([w, w.new_zeros((n, w.shape[1]))]).contiguous() if n else w
 
 
 class Hgrn2Mixer:
@@ -258,5 +265,107 @@ class ParallelMixer:
         return out
 
 
+class GroupedAttentionMixer:
+    """Grouped-query attention with the options of `GroupedAttentionSpec`."""
+
+    def __init__(self, spec, t: Tensors, eps: float):
+        self.spec = s = spec
+        names = ("q", "k", "v") if s.kv_from is None else ("q",)
+        self.w_in, self.w_o = t.mat(*names, *(("g",) if s.gate else ())), t.mat("o")
+        self.widths = [s.heads * s.dim, s.kv_heads * s.dim, s.kv_heads * s.vdim][:len(names)] + ([s.heads] if s.gate else [])
+        self.bias = torch.cat([t.f32(n + ".b") for n in names]).contiguous() if s.bias else None
+        self.o_bias = t.f32("o.b") if s.bias else None
+        self.sink = t.f32("sink") if s.sink else None
+        dist = (t.f32("r1"), t.f32("r2")) if s.distance else (None, None)
+        self.maps = MapsSpec(s.heads, s.kv_heads, s.dim, s.vdim, s.scale, maps=1, softcap=s.softcap, eps=eps, window=s.window,
+                             keep_first=s.keep_first if s.window > 0 else 0, dist_a=dist[0], dist_b=dist[1],
+                             tiled=t.dtype == torch.bfloat16)
+
+    def entries(self):
+        return [KVLayer(self.spec.kv_heads, self.maps.dim_p, self.maps.vdim_p)] if self.spec.kv_from is None else []
+
+    def run(self, model, y, h, entry, cache, b):
+        q, *kv = columns(y, self.widths)
+        g = kv.pop() if self.spec.gate else None
+        kc, vc, rope = cache.k[entry], cache.v[entry], self.spec.rope
+        q = ops.rope_norm_append(self.maps, q, *(kv or (None, None)), self.bias, model.rope_table(rope) if rope else None,
+                                 b.positions, b.slots, kc, vc, norm=False, interleaved=True)
+        o = ops.heads_attention(self.maps, q, kc, vc, b.block_table, b.context_lens, q_start=b.q_start, q_lens=b.q_lens,
+                                max_q_len=b.max_q_len, sinks=self.sink)
+        return o.flatten(1) if g is None else ops.gate_heads(o, g, "sigmoid")
+
+
+class DeltaMixer:
+    """Gated delta rule."""
+
+    def __init__(self, spec, t: Tensors, eps: float):
+        c, n, H = spec.kv_heads * spec.dim, spec.heads * spec.vdim, spec.heads
+        self.w_in, self.w_o = t.mat("q", "k", "v", "g", "b", "a"), t.mat("o")
+        self.widths = [2 * c + n, n, H, H]
+        self.conv = ShortConv(torch.cat([t.f32(x + ".conv") for x in "qkv"]).t().contiguous())
+        self.norm = t.f32("norm")
+        self.rule = HeadRecurrence(H, spec.kv_heads, spec.dim, spec.vdim, 0, c, 2 * c, torch.exp(t.f32("A_log")), t.f32("dt_bias"),
+                                   delta=True, q_scale=spec.dim ** -0.5, eps=eps)
+
+    def entries(self):
+        return [StateLayer(self.rule.state_shape), StateLayer(self.conv.state_shape)]
+
+    def run(self, model, y, h, entry, cache, b):
+        x, gate, strength, decay = columns(y, self.widths)
+        return ops.head_recurrence(self.rule, x, self.conv, decay, strength, gate, self.norm, cache.state[entry],
+                                   cache.state[entry + 1], b.context_lens, q_start=b.q_start, q_lens=b.q_lens, rows=b.rows,
+                                   dtype=model.dtype)
+
+
+class StateSpaceMixer:
+    """Mamba-2."""
+
+    def __init__(self, spec, t: Tensors, eps: float):
+        n, c = spec.heads * spec.vdim, spec.groups * spec.state
+        self.w_in, self.w_o = t.mat("in"), t.mat("o")
+        self.widths, self.parts = [n, n + 2 * c, spec.heads], spec.norm_groups
+        self.conv = ShortConv(t.f32("conv").t().contiguous(), t.f32("conv.b"))
+        self.norm = t.f32("norm")
+        self.rule = HeadRecurrence(spec.heads, spec.groups, spec.state, spec.vdim, n + c, n, 0, torch.exp(t.f32("A_log")),
+                                   t.f32("dt_bias"), delta=False, skip=t.f32("D"), eps=eps)
+
+    def entries(self):
+        return [StateLayer(self.rule.state_shape), StateLayer(self.conv.state_shape)]
+
+    def run(self, model, y, h, entry, cache, b):
+        gate, x, dt = columns(y, self.widths)
+        return ops.head_recurrence(self.rule, x, self.conv, dt, None, gate, self.norm, cache.state[entry], cache.state[entry + 1],
+                                   b.context_lens, parts=self.parts, q_start=b.q_start, q_lens=b.q_lens, rows=b.rows,
+                                   dtype=model.dtype)
+
+
+class BlendMixer:
+    """Two mixers on the same input, each with its own output projection; the mean of their results, RMS-normed over the width.
+    Their rows of the input projection are one matrix, each part filled up to whole 16 bytes with zero rows."""
+
+    def __init__(self, spec, t: Tensors, eps: float):
+        self.left = GroupedAttentionMixer(spec.left, t.under("left."), eps)
+        self.right = StateSpaceMixer(spec.right, t.under("right."), eps)
+        self.norms = [t.f32("left.out"), t.f32("right.out")]
+        left = padded_rows(self.left.w_in)
+        self.w_in, self.w_o = torch.cat([left, self.right.w_in]).contiguous(), None
+        self.widths = [left.shape[0], self.right.w_in.shape[0]]
+        self.left.w_in = self.right.w_in = None
+
+    def weights(self):
+        return [self.left.w_o, self.right.w_o]
+
+    def entries(self):
+        return self.left.entries() + self.right.entries()
+
+    def run(self, model, y, h, entry, cache, b):
+        left, right = columns(y, self.widths)
+        outs = [(self.left, self.left.run(model, left, h, entry, cache, b)),
+                (self.right, self.right.run(model, right, h, entry + len(self.left.entries()), cache, b))]
+        return [Branch(Proj(model.project(o, m.w_o), 0, m.w_o.shape[0]), scale=0.5, norm=n, shift=getattr(m, "o_bias", None))
+                for (m, o), n in zip(outs, self.norms)]
+
+
 MIXERS = {"hgrn2": Hgrn2Mixer, "attention": MapsMixer, "gla": LinearAttentionMixer, "window": WindowAttentionMixer,
-          "rwkv": TimeMixMixer, "parallel": ParallelMixer, "chunk": ChunkAttentionMixer, "latent": LatentAttentionMixer}
+          "rwkv": TimeMixMixer, "parallel": ParallelMixer, "chunk": ChunkAttentionMixer, "latent": LatentAttentionMixer,
+          "grouped": GroupedAttentionMixer, "delta": DeltaMixer, "ssd": StateSpaceMixer, "blend": BlendMixer}

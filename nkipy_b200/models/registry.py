@@ -78,6 +78,7 @@ ARCHITECTURES: Dict[str, Architecture] = {
     "Tolenex": _hybrid(C.tolenex_config),
     "Mumilorn": _hybrid(C.mumilorn_config),
     "Ligizen": _hybrid(C.ligizen_config),
+    "Redodra": _hybrid(C.redodra_config),
 }
 
 
@@ -92,7 +93,7 @@ def for_config(cfg: C.ModelConfig) -> Architecture:
     """The architecture entry that runs a configuration made in code."""
     if cfg.layers is None:
         return ARCHITECTURES["LlamaForCausalLM"]
-    return ARCHITECTURES[{"mumilorn": "Mumilorn", "ligizen": "Ligizen"}.get(cfg.name, "Tolenex")]
+    return ARCHITECTURES[{"mumilorn": "Mumilorn", "ligizen": "Ligizen", "redodra": "Redodra"}.get(cfg.name, "Tolenex")]
 
 
 def read_config(folder: str):

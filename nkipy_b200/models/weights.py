@@ -156,14 +156,33 @@ def random_weights(cfg: ModelConfig, rank: int = 0, world: int = 1, device="cpu"
 
 def _mixer_shapes(m, W: int) -> Dict[str, tuple]:
     """Tensors of a token mixer (models/mixers.py) by their names under '<layer>.mix.'."""
-    if m.kind == "parallel":
+    if m.kind in ("parallel", "blend"):
+        out = {"left.out": (W,), "right.out": (W,)} if m.kind == "blend" else {}
         return {**{"left." + k: v for k, v in _mixer_shapes(m.left, W).items()},
-                **{"right." + k: v for k, v in _mixer_shapes(m.right, W).items()}}
+                **{"right." + k: v for k, v in _mixer_shapes(m.right, W).items()}, **out}
     if m.kind == "rwkv":
         c, rank = m.heads * m.dim, m.rank or 16
         return {**{f"mu.{n}": (W,) for n in "rkvgw"}, **{n: (c, W) for n in "rkvg"}, "w1": (rank, W), "w2": (c, rank),
                 "w0": (c,), "u": (m.heads, m.dim), "norm": (c,), "o": (W, c)}
     out = m.heads * m.vdim
+    if m.kind == "ssd":
+        channels = out + 2 * m.groups * m.state
+        return {"in": (out + channels + m.heads, W), "conv": (channels, m.conv), "conv.b": (channels,), "dt_bias": (m.heads,),
+                "A_log": (m.heads,), "D": (m.heads,), "norm": (out,), "o": (W, out)}
+    if m.kind == "delta":
+        c = m.kv_heads * m.dim
+        return {"q": (c, W), "q.conv": (c, m.conv), "k": (c, W), "k.conv": (c, m.conv), "v": (out, W), "v.conv": (out, m.conv),
+                "b": (m.heads, W), "a": (m.heads, W), "A_log": (m.heads,), "dt_bias": (m.heads,), "norm": (m.vdim,),
+                "g": (out, W), "o": (W, out)}
+    if m.kind == "grouped":
+        rows = {"q": m.heads * m.dim}
+        if m.kv_from is None:
+            rows.update(k=m.kv_heads * m.dim, v=m.kv_heads * m.vdim)
+        shapes = {**{k: (n, W) for k, n in rows.items()}, "o": (W, out)}
+        if m.bias:
+            shapes.update({k + ".b": (n,) for k, n in {**rows, "o": W}.items()})
+        per_head = (("r1", "r2") if m.distance else ()) + (("sink",) if m.sink else ())
+        return {**shapes, **{k: (m.heads,) for k in per_head}, **({"g": (m.heads, W)} if m.gate else {})}
     if m.kind == "chunk":
         q, k, v = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim
         own = {} if m.kv_from is not None else {"k": (k, W), "k.b": (k,), "v": (v, W), "v.b": (v,)}
@@ -195,21 +214,28 @@ def hybrid_weight_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
         out["head"] = (V, W)
     if cfg.loop:
         out["loop.step"] = (cfg.loop.times, W)
-    if cfg.layer_norm:
-        out["final.norm.b"] = (W,)
+    norm = lambda name: {name: (W,), **({name + ".b": (W,)} if cfg.layer_norm or cfg.tanh_norm else {}),
+                         **({name + ".alpha": ()} if cfg.tanh_norm else {})}
+    out.update(norm("final.norm"))
     if cfg.token_side:
         out["side.embed"] = (V, len(cfg.layers) * cfg.token_side)
     for i, layer in enumerate(cfg.layers):
-        shapes = {"norm1": (W,), **{"mix." + k: v for k, v in _mixer_shapes(layer.mixer, W).items()}}
+        shapes = {**norm("norm1"), **{"mix." + k: v for k, v in _mixer_shapes(layer.mixer, W).items()}}
+        if layer.block == "sandwich":
+            shapes.update(norm("norm1b"))
+        if cfg.depth_average:
+            shapes["dwa"] = (i + 2,)
         if layer.block == "gated":
             shapes.update({"rg1": (W, W), "rg1.b": (W,)})
-        if cfg.layer_norm:
-            shapes["norm1.b"] = (W,)
         if (layer.ff or layer.experts) and layer.block != "parallel":
-            shapes["norm2"] = (W,)
+            shapes.update(norm("norm2"))
+            if layer.block == "sandwich":
+                shapes.update(norm("norm2b"))
         if layer.ff:
             shapes.update({"mlp.up": (layer.ff, W), "mlp.down": (W, layer.ff)})
-            if layer.block != "pre-norm":
+            if layer.act == "xielu":
+                shapes["mlp.act"] = (2,)
+            if layer.block not in ("pre-norm", "sandwich"):
                 shapes["mlp.gate"] = (layer.ff, W)
             if layer.block == "gated":
                 shapes.update({"rg2": (W, W), "rg2.b": (W,)})
@@ -232,14 +258,18 @@ def hybrid_weight_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
 def hybrid_random_weights(cfg: ModelConfig, device="cpu", seed: int = 0, std: float = 0.02,
                           dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
     """Random-init weights of a layer-by-layer configuration: N(0, std), norms that multiply by 1, lower bounds of the
-    forget gates and mixes of neighbouring tokens uniform in [0, 0.9), slow decays."""
+    forget gates and mixes of neighbouring tokens uniform in [0, 0.9), slow decays, depth averages near their last term."""
     out: Dict[str, torch.Tensor] = {}
     for n, (name, shape) in enumerate(hybrid_weight_shapes(cfg).items()):
         leaf = name.rsplit(".", 1)[-1]
-        if leaf in ("norm1", "norm2") or name == "final.norm":
+        if leaf in ("norm1", "norm2", "norm1b", "norm2b") or name == "final.norm":
             out[name] = torch.full(shape, 1.0 - cfg.norm_offset, dtype=dtype, device=device)
-        elif leaf == "norm":
+        elif leaf in ("norm", "out", "alpha", "D", "r1"):
             out[name] = torch.ones(shape, dtype=dtype, device=device)
+        elif leaf == "r2":
+            out[name] = torch.full(shape, 0.1, dtype=dtype, device=device)
+        elif leaf == "conv":
+            out[name] = _normal(shape, shape[1] ** -0.5, seed * 100003 + n, device, dtype)
         elif leaf == "lower" or ".mu." in name:
             g = torch.Generator(device=device).manual_seed(seed * 100003 + n)
             out[name] = (0.9 * torch.rand(shape, generator=g, device=device)).to(dtype)
@@ -247,6 +277,10 @@ def hybrid_random_weights(cfg: ModelConfig, device="cpu", seed: int = 0, std: fl
             out[name] = _normal(shape, std, seed * 100003 + n, device, dtype)
             if leaf == "w0":
                 out[name] -= 4.0             # exp(-exp(-4)): a memory of some fifty tokens
+            elif leaf in ("A_log", "dt_bias"):
+                out[name] -= 2.0
+            elif leaf == "dwa":
+                out[name][-1] += 1.0
     return out
 
 

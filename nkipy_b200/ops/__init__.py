@@ -18,8 +18,10 @@ from __future__ import annotations
 
 import os
 
+import ctypes
 import math
-from typing import Optional, Tuple
+from dataclasses import dataclass
+from typing import Optional, Tuple, Union
 
 import torch
 
@@ -33,6 +35,7 @@ __all__ = [
     "heads_attention", "maps_attention", "row_norm_append", "rope_norm_append", "head_linear", "softcap",
     "LatentSpec", "latent_append", "latent_attention", "latent_gather", "latent_prefill", "latent_queries",
     "Decay", "linear_attention", "low_rank", "token_mix",
+    "Act", "ScoreMods", "HeadRecurrence", "ShortConv", "head_recurrence", "gated_group_norm", "short_conv",
     "KernelLibraryError", "device_status", "raise_on_device_error", "native_available", "launch_count",
     "reset_launch_count",
 ]
@@ -107,7 +110,7 @@ def linear(
     ctas_per_sm: Optional[int] = None,
     act: str = "silu",
     fp32_out: bool = False,
-    out_act: Optional[str] = None,
+    out_act: Optional[Union[str, "mixers.Act"]] = None,
 ) -> torch.Tensor:
     """``y = x @ w.T`` with optional fused epilogue.
 
@@ -116,7 +119,8 @@ def linear(
     gated: w is ``[2*I, K]`` holding gate rows then up rows; returns
            ``act(x @ gate.T) * (x @ up.T)`` of shape [M, I], act "silu" or "gelu_tanh".
     fp32_out: finished values in fp32 instead of bf16 (not with gated).
-    out_act: "relu2" applies the square of the positive part to a plain product (finished bf16 values).
+    out_act: activation of a plain product (finished bf16 values): "relu2", the square of the positive part, or xIELU
+           with its parameters (`mixers.Act`).
     splits > 1: split-K; returns fp32 partial sums ``[S, M, N]`` (S may be smaller
            than requested) for a fused reduction (`add_rmsnorm`, `rope_kv_append`,
            `reduce_partials`).  bias is added to partial 0.
@@ -143,7 +147,7 @@ def linear(
         if splits > 1:
             return y.unsqueeze(0)
         if out_act is not None:
-            y = mixers.ACTIVATIONS[out_act][1](y)
+            y = mixers.activate(y, out_act)
         if residual is not None:
             y = y + residual.float()
         y = y.to(torch.float32 if fp32_out or x.dtype == torch.float32 else torch.bfloat16)
@@ -154,8 +158,9 @@ def linear(
     global _launches
     if x.stride(1) != 1 or w.stride(1) != 1:
         raise ValueError("linear needs K-contiguous operands")
-    if out_act not in (None, "relu2") or (out_act and (gated or residual is not None or fp32_out)):
-        raise ValueError("out_act is relu2, for finished plain products")
+    epi = mixers.Act.of(out_act) if out_act is not None else mixers.Act("silu")
+    if out_act is not None and (epi.name not in ("relu2", "xielu") or gated or residual is not None or fp32_out):
+        raise ValueError("out_act is relu2 or xielu, for finished plain products")
     if x.dtype == torch.float32 or (K | x.stride(0) | w.stride(0)) & 7 or (x.data_ptr() | w.data_ptr()) & 15:
         if bias is not None or residual is not None or out is not None:
             raise ValueError("the CUDA-core GEMM has no bias, residual or out argument")
@@ -184,12 +189,12 @@ def linear(
         out_view = out
         out_fp32, split_stride = 1 if fp32_out else 0, 0
     ldo = out_view.stride(-2) if out_view.dim() >= 2 else N
-    act_code = mixers.ACTIVATIONS[act][0] if gated else (mixers.ACTIVATIONS[out_act][0] if out_act else 0)
+    act_code = mixers.ACTIVATIONS[act][0] if gated else (epi.code if out_act is not None else 0)
     if (not swap and splits <= 1 and not fp32_out and M >= 512 and N >= 256 and _USE_2CTA and (ldo & 7) == 0
             and not (gated and (bias is not None or residual is not None))):
         # prefill-sized: CTA pairs on 256 x 256 tiles (csrc/kernels/gemm_2cta.cu)
         rc = L.nkb_gemm_bf16_2cta(x.data_ptr(), w.data_ptr(), out_view.data_ptr(), M, N, K, x.stride(0), w.stride(0),
-                                  ldo, _ptr(bias), _ptr(residual), 1 if gated else 0, N if gated else 0, act_code,
+                                  ldo, _ptr(bias), _ptr(residual), 1 if gated else 0, N if gated else 0, act_code, epi.a, epi.b,
                                   _stream())
         if rc != -5:
             _lib.check(rc, "nkb_gemm_bf16_2cta")
@@ -211,7 +216,7 @@ def linear(
         a.data_ptr(), b.data_ptr(), out_view.data_ptr(), rows, cols, K, lda, ldb, ldo, transpose_out, out_fp32,
         eff if splits > 1 else 1, split_stride, gate_mode, N if gated else 0, _ptr(bias), bias_on_rows,
         _ptr(residual), block_n, max_ctas, (0 if swap else 1) if weights_static else -1,
-        (2 if (swap and not gated) else 1) if ctas_per_sm is None else ctas_per_sm, act_code, _stream(),
+        (2 if (swap and not gated) else 1) if ctas_per_sm is None else ctas_per_sm, act_code, epi.a, epi.b, _stream(),
     )
     _lib.check(rc, "nkb_gemm_bf16")
     _launches += 1
@@ -763,6 +768,38 @@ def router_topk(logits, top_k: int, mode: str = "softmax_topk", bias: Optional[t
 
 
 # --------------------------------------------------------------------------- attention
+@dataclass
+class ScoreMods:
+    """What attention does to a score beyond scaling it: softcap > 0: softcap * tanh(s / softcap), then dist_a * ln(1 + dist_b *
+    distance) is taken off (fp32 [query heads] each).  keep_first: with a window, tokens that stay visible outside it."""
+    softcap: float = 0.0
+    keep_first: int = 0
+    dist_a: Optional[torch.Tensor] = None
+    dist_b: Optional[torch.Tensor] = None
+
+    def __bool__(self) -> bool:
+        return self.softcap > 0 or self.keep_first > 0 or self.dist_a is not None
+
+    def arg(self):
+        for t in (self.dist_a, self.dist_b):
+            if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
+                raise TypeError("distance terms are contiguous fp32")
+        return _lib.ScoreModsArg(float(self.softcap), int(self.keep_first), _ptr(self.dist_a), _ptr(self.dist_b))
+
+    def apply(self, s: torch.Tensor, dist: torch.Tensor) -> torch.Tensor:
+        """Scaled scores [heads, ..., queries, keys] with dist [queries, keys]."""
+        if self.softcap > 0:
+            s = self.softcap * torch.tanh(s / self.softcap)
+        if self.dist_a is not None:
+            shape = (-1,) + (1,) * (s.dim() - 1)
+            s = s - self.dist_a.float().reshape(shape) * torch.log1p(self.dist_b.float().reshape(shape) * dist.clamp(min=0))
+        return s
+
+
+def _mods_ref(mods: Optional[ScoreMods]):
+    return ctypes.byref(mods.arg()) if mods else None
+
+
 def _gather_kv(cache: torch.Tensor, table_row: torch.Tensor, ctx: int) -> torch.Tensor:
     """[ctx, nkv, D] view of one sequence's cached K or V (reference path)."""
     bs = cache.shape[2]
@@ -771,7 +808,7 @@ def _gather_kv(cache: torch.Tensor, table_row: torch.Tensor, ctx: int) -> torch.
     return blocks.permute(0, 2, 1, 3).reshape(nblk * bs, cache.shape[1], cache.shape[3])[:ctx]
 
 
-def _ref_attention(q, k, v, scale, q_pos0, causal, window, sinks, chunk=0):
+def _ref_attention(q, k, v, scale, q_pos0, causal, window, sinks, chunk=0, mods=None):
     """q [Lq, nq, D], k/v [Lk, nkv, D] fp32 -> [Lq, nq, D]; query i sits at kv position q_pos0 + i."""
     Lq, nq, D = q.shape
     Lk, nkv, _ = k.shape
@@ -781,11 +818,13 @@ def _ref_attention(q, k, v, scale, q_pos0, causal, window, sinks, chunk=0):
     s = torch.einsum("qhd,khd->hqk", q, kk) * scale
     qpos = q_pos0 + torch.arange(Lq, device=q.device)[:, None]
     kpos = torch.arange(Lk, device=q.device)[None, :]
+    if mods:
+        s = mods.apply(s, qpos - kpos)
     mask = torch.ones((Lq, Lk), dtype=torch.bool, device=q.device)
     if causal:
         mask &= kpos <= qpos
     if window and window > 0:
-        mask &= kpos > qpos - window
+        mask &= (kpos > qpos - window) | (kpos < (mods.keep_first if mods else 0))
     if chunk > 0:
         mask &= kpos >= qpos - qpos % chunk
     s = s.masked_fill(~mask[None], float("-inf"))
@@ -836,6 +875,7 @@ def paged_attn_decode(
     window: int = 0,
     chunk: int = 0,
     sinks: Optional[torch.Tensor] = None,
+    mods: Optional[ScoreMods] = None,
     num_splits: int = 0,
     scratch: Optional[torch.Tensor] = None,
     out: Optional[torch.Tensor] = None,
@@ -843,7 +883,7 @@ def paged_attn_decode(
     """Decode attention over the paged cache.  q ``[B * q_len, nq * D]`` (the q_len
     newest tokens of each sequence, already appended to the cache);
     context_lens counts them.  Causal among the new tokens; window > 0: a query sees itself and the window - 1 tokens
-    before it; chunk > 0: only the positions of its own chunk of that many."""
+    before it; chunk > 0: only the positions of its own chunk of that many; mods: see `ScoreMods`."""
     nkv, bs, D = k_cache.shape[1], k_cache.shape[2], k_cache.shape[3]
     B = block_table.shape[0]
     nq = q.shape[-1] // D
@@ -856,7 +896,7 @@ def paged_attn_decode(
             ctx = int(context_lens[b])
             k = _gather_kv(k_cache, block_table[b], ctx).float()
             v = _gather_kv(v_cache, block_table[b], ctx).float()
-            res[b] = _ref_attention(qf[b], k, v, scale, ctx - q_len, True, window, sinks, chunk)
+            res[b] = _ref_attention(qf[b], k, v, scale, ctx - q_len, True, window, sinks, chunk, mods)
         out.copy_(res.reshape(out.shape).to(out.dtype))
         return out
     global _launches
@@ -867,7 +907,7 @@ def paged_attn_decode(
         q_start = torch.arange(B, device=q.device, dtype=torch.int32) * q_len
         q_lens = torch.full((B,), q_len, device=q.device, dtype=torch.int32)
         return flash_attn_prefill(q, k_cache, v_cache, block_table, q_start, q_lens, context_lens, scale,
-                                  max_q_len=q_len, causal=True, window=window, chunk=chunk, sinks=sinks, out=out)
+                                  max_q_len=q_len, causal=True, window=window, chunk=chunk, sinks=sinks, mods=mods, out=out)
     L = _lib.lib()
     if num_splits <= 0:
         num_splits = pick_kv_splits(B * nkv, block_table.shape[1])
@@ -878,7 +918,7 @@ def paged_attn_decode(
     rc = L.nkb_paged_attn_decode(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), context_lens.data_ptr(),
         out.data_ptr(), _ptr(scratch), B, q_len, nq, nkv, D, bs, k_cache.shape[0], block_table.stride(0),
-        float(scale), int(window), int(chunk), _ptr(sinks), num_splits, _stream(),
+        float(scale), int(window), int(chunk), _ptr(sinks), _mods_ref(mods), num_splits, _stream(),
     )
     _lib.check(rc, "nkb_paged_attn_decode")
     _launches += 1
@@ -976,12 +1016,13 @@ def flash_attn_prefill(
     window: int = 0,
     chunk: int = 0,
     sinks: Optional[torch.Tensor] = None,
+    mods: Optional[ScoreMods] = None,
     out: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """Blockwise prefill attention.  q ``[total_q, nq * D]`` packs the new tokens of
     all sequences (sequence b owns rows q_start[b] .. q_start[b] + q_lens[b]); K/V
     of the whole context (cached prefix + new tokens) are read from the paged
-    cache.  Query i of a sequence sits at position context_len - q_len + i."""
+    cache.  Query i of a sequence sits at position context_len - q_len + i.  mods: see `ScoreMods`."""
     nkv, bs, D = k_cache.shape[1], k_cache.shape[2], k_cache.shape[3]
     B = block_table.shape[0]
     total_q = q.shape[0]
@@ -997,7 +1038,7 @@ def flash_attn_prefill(
                 continue
             k = _gather_kv(k_cache, block_table[b], ctx).float()
             v = _gather_kv(v_cache, block_table[b], ctx).float()
-            res[qs:qs + ql] = _ref_attention(qf[qs:qs + ql], k, v, scale, ctx - ql, causal, window, sinks, chunk)
+            res[qs:qs + ql] = _ref_attention(qf[qs:qs + ql], k, v, scale, ctx - ql, causal, window, sinks, chunk, mods)
         out.copy_(res.reshape(out.shape).to(out.dtype))
         return out
     global _launches
@@ -1006,7 +1047,7 @@ def flash_attn_prefill(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), q_start.data_ptr(),
         q_lens.data_ptr(), context_lens.data_ptr(), out.data_ptr(), B, total_q, int(max_q_len), nq, nkv, D, bs,
         k_cache.shape[0], block_table.stride(0), float(scale), 1 if causal else 0, int(window), int(chunk), _ptr(sinks),
-        _stream(),
+        _mods_ref(mods), _stream(),
     )
     _lib.check(rc, "nkb_flash_attn_prefill")
     _launches += 1
@@ -1229,8 +1270,10 @@ def moe_combine(y_sorted: torch.Tensor, pair_pos: torch.Tensor, weights: torch.T
 
 
 from . import mixers  # noqa: E402  (uses the helpers above)
-from .mixers import (Branch, MapsSpec, Norm, Proj, activation, gate_heads, gated_act, gated_residual,  # noqa: E402,F401
+from .mixers import (Act, Branch, MapsSpec, Norm, Proj, activation, gate_heads, gated_act, gated_residual,  # noqa: E402,F401
                      heads_attention, hgrn2, maps_append, maps_attention, rope_norm_append, row_norm_append)
 from .latent_attention import (LatentSpec, latent_append, latent_attention, latent_gather,  # noqa: E402,F401
                                latent_prefill, latent_queries)
 from .linear_attention import Decay, linear_attention, low_rank, token_mix  # noqa: E402,F401
+from .head_recurrence import (HeadRecurrence, ShortConv, gated_group_norm, head_recurrence,  # noqa: E402,F401
+                              short_conv)

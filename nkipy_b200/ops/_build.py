@@ -44,13 +44,13 @@ NVCC_FLAGS = [
 # GEMM epilogue and the attention softmax want; the normalisation and sampling
 # files keep IEEE division and sqrt.
 NO_FAST_MATH = {"sampling.cu", "elementwise.cu", "decode_layer.cu", "gated_residual.cu", "recurrent.cu", "attn_maps.cu",
-                "gemm_simt.cu", "linear_attn.cu", "latent_attn.cu"}
+                "gemm_simt.cu", "linear_attn.cu", "latent_attn.cu", "head_recurrence.cu", "post_residual.cu"}
 
 
 # what a single-GPU decoder of models/hybrid.py launches
 SERVING_SOURCES = ("host_glue.cu", "gemm_tcgen05.cu", "gemm_2cta.cu", "gemm_simt.cu", "elementwise.cu", "sampling.cu",
                    "gated_residual.cu", "recurrent.cu", "attn_maps.cu", "attn_maps_prefill.cu", "linear_attn.cu",
-                   "latent_attn.cu", "attn_decode.cu", "attn_prefill.cu", "moe.cu")
+                   "latent_attn.cu", "head_recurrence.cu", "post_residual.cu", "attn_decode.cu", "attn_prefill.cu", "moe.cu")
 
 
 def _nvcc() -> str:

@@ -32,7 +32,13 @@ class MapsArg(ctypes.Structure):
     _fields_ = [(n, c_int) for n in ("maps", "heads", "kv_heads", "dim", "dim_p", "vdim", "vdim_p")] + \
                [(n, c_float) for n in ("scale", "softcap", "lam", "out_scale", "eps")] + \
                [("window", c_int), ("chunk", c_int), ("sinks", c_void_p)] + \
-               [(n, c_longlong) for n in ("q_token", "q_head", "o_token", "o_head")] + [("v_ld", c_int)]
+               [(n, c_longlong) for n in ("q_token", "q_head", "o_token", "o_head")] + \
+               [("v_ld", c_int), ("keep_first", c_int), ("dist_a", c_void_p), ("dist_b", c_void_p)]
+
+
+class ScoreModsArg(ctypes.Structure):
+    """What plain attention does to a score beyond scaling it (csrc/kernels/attn_maps.h)."""
+    _fields_ = [("softcap", c_float), ("keep_first", c_int), ("dist_a", c_void_p), ("dist_b", c_void_p)]
 
 
 class LatentArg(ctypes.Structure):
@@ -58,6 +64,32 @@ class LinAttnArg(ctypes.Structure):
                [(n, c_float) for n in ("q_scale", "inv_tau", "out_scale", "eps")]
 
 
+class HeadRecArg(ctypes.Structure):
+    """Arguments of recurrences with one decay per head (csrc/kernels/head_recurrence.h)."""
+    _fields_ = [(n, ProjArg) for n in ("x", "a", "b", "g")] + \
+               [(n, c_void_p) for n in ("conv_w", "conv_b", "conv_state", "rate", "dt_bias", "skip", "norm_w", "state", "slot_ids",
+                                        "q_start", "q_lens", "context_lens", "out")] + \
+               [(n, c_int) for n in ("taps", "channels", "q_col", "k_col", "v_col", "gate_act", "bf16", "batch", "tokens", "heads",
+                                     "groups", "dim", "vdim")] + [(n, c_float) for n in ("q_scale", "eps", "unit_eps")]
+
+
+class TanhNormArg(ctypes.Structure):
+    _fields_ = [("w", c_void_p), ("b", c_void_p), ("alpha", c_float), ("out", c_void_p)]
+
+
+class PostBranchArg(ctypes.Structure):
+    _fields_ = [("y", ProjArg), ("shift", c_void_p), ("norm_w", c_void_p), ("scale", c_float)]
+
+
+class PostResidualArg(ctypes.Structure):
+    """Arguments of a residual update through a norm (csrc/kernels/post_residual.h)."""
+    _fields_ = [("x_in", c_void_p), ("ids", c_void_p), ("table", c_void_p), ("br", PostBranchArg * 2), ("post", TanhNormArg),
+                ("norm", TanhNormArg * 2), ("history", c_void_p), ("coef", c_void_p), ("result", c_void_p), ("x_out", c_void_p),
+                ("history_stride", c_longlong)] + \
+               [(n, c_int) for n in ("vocab", "table_bf16", "branches", "norms", "past", "out_bf16", "rows", "width")] + \
+               [("table_scale", c_float), ("eps", c_float)]
+
+
 _PP = ctypes.POINTER(ProjArg)
 _PM = ctypes.POINTER(MapsArg)
 _PL = ctypes.POINTER(LatentArg)
@@ -68,10 +100,10 @@ _SIGNATURES = {
     "nkb_gemm_bf16": (
         c_int,
         [_P, _P, _P, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_int, c_int, c_int, c_longlong,
-         c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, _P],
+         c_int, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_float, _P],
     ),
     "nkb_gemm_bf16_2cta": (c_int, [_P, _P, _P, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, _P, _P, c_int,
-                                   c_int, c_int, _P]),
+                                   c_int, c_int, c_float, c_float, _P]),
     "nkb_gemm_simt": (c_int, [_P, c_int, _P, c_int, _P, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong,
                               _P]),
     "nkb_gemm_simt_grouped": (c_int, [_P, c_int, _P, c_int, _P, c_int, _P, _P, c_int, c_int, c_int, c_int, c_longlong,
@@ -83,8 +115,13 @@ _SIGNATURES = {
     "nkb_gate_heads": (c_int, [_P, c_int, c_longlong, c_longlong, _PP, c_int, c_int, _P, c_int, c_float, c_float, _P, c_int,
                                c_longlong, c_int, c_int, c_int, _P]),
     "nkb_row_norm_append": (c_int, [_PM, _PP, _PP, _PP, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P]),
-    "nkb_rope_norm_append": (c_int, [_PM, _PP, _PP, _PP, _P, _P, c_int, c_int, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int,
-                                     _P]),
+    "nkb_rope_norm_append": (c_int, [_PM, _PP, _PP, _PP, _P, _P, c_int, c_int, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int,
+                                     c_int, _P]),
+    "nkb_short_conv": (c_int, [_PP, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P]),
+    "nkb_head_rec_scan": (c_int, [ctypes.POINTER(HeadRecArg), _P]),
+    "nkb_head_rec_step": (c_int, [ctypes.POINTER(HeadRecArg), _P]),
+    "nkb_gated_group_norm": (c_int, [_P, c_int, _PP, c_int, _P, c_float, _P, c_int, c_int, c_int, c_int, _P]),
+    "nkb_post_residual": (c_int, [ctypes.POINTER(PostResidualArg), _P]),
     "nkb_latent_append": (c_int, [_PL, _PP, _PP, _P, _P, _P, c_int, _P, _P, _P, _P, c_int, c_int, c_int, _P]),
     "nkb_latent_queries": (c_int, [_PL, _PP, _P, c_int, _P, _P, c_longlong, c_longlong, c_int, _P, c_longlong, c_longlong,
                                    c_int, c_int, c_int, _P]),
@@ -160,7 +197,7 @@ _SIGNATURES = {
     "nkb_paged_attn_decode": (
         c_int,
         [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
-         _P, c_int, _P],
+         _P, ctypes.POINTER(ScoreModsArg), c_int, _P],
     ),
     "nkb_paged_attn_decode_fused": (
         c_int,
@@ -171,7 +208,7 @@ _SIGNATURES = {
     "nkb_flash_attn_prefill": (
         c_int,
         [_P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-         c_int, c_int, c_int, _P, _P],
+         c_int, c_int, c_int, _P, ctypes.POINTER(ScoreModsArg), _P],
     ),
 }
 

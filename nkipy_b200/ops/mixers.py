@@ -1,21 +1,23 @@
 """Operators of decoders whose layers mix attention and linear recurrences around an fp32 residual stream.
 
-    gated_residual   embedding or residual + branches (gated, scaled, routed or normed; + additions ahead of a repeated
-                     block), and the norms of the sum (group-wise RMS, layer norm, or a copy), in one launch
+    gated_residual   embedding or residual + branches (gated, scaled, routed or normed, also through a norm of their sum; +
+                     additions ahead of a repeated block, or an average with earlier results), and the norms of the
+                     sum (group-wise RMS, layer norm, tanh, or a copy), in one launch
     gated_act        act(gate) * up, also with clamped operands or rows of a table as up; `activation` for act(x) alone
     gate_heads       scale * act(gate) * norm(head), the norm optional, one gate per element or per head
     hgrn2            linear attention with a per-channel forget gate; state in slots, fp32
     row_norm_append  queries and keys normed over all their heads, paged-cache append
-    rope_norm_append biases, half-split partial RoPE and per-head norm of queries and keys, paged-cache append
+    rope_norm_append biases, partial RoPE (half-split or interleaved, or none) and per-head norm of queries and keys,
+                     paged-cache append
     maps_append      interleaved partial RoPE of queries / keys with several score maps, paged-cache append
     heads_attention  attention with several score maps over shared values (differential attention), score soft cap;
-                     with one map plain grouped-query attention, also through a sliding window, inside chunks and
-                     with sinks
+                     with one map plain grouped-query attention, also through a sliding window (with kept first
+                     tokens), inside chunks, with sinks and with a distance term
     linear_simt      products on the CUDA cores: 32-bit models, operands TMA cannot describe
 
 All of them take the projections they consume as `Proj` slices, so a decode-sized batch hands over split-K partial
 sums and a prefill-sized one finished bf16 without a copy in between.  CUDA tensors run the kernels of
-csrc/kernels/{gated_residual,recurrent,attn_maps,attn_maps_prefill,gemm_simt}.cu; CPU tensors run the PyTorch
+csrc/kernels/{gated_residual,post_residual,recurrent,attn_maps,attn_maps_prefill,gemm_simt}.cu; CPU tensors run the PyTorch
 statement of the same op.
 """
 
@@ -23,13 +25,13 @@ from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
-from typing import List, NamedTuple, Optional, Sequence, Tuple
+from typing import List, NamedTuple, Optional, Sequence, Tuple, Union
 
 import torch
 import torch.nn.functional as F
 
 from . import _lib
-from . import (_count_launch, _decode_scratch, _gather_kv, _native, _ptr, _stream, flash_attn_prefill,
+from . import (ScoreMods, _count_launch, _decode_scratch, _gather_kv, _native, _ptr, _stream, flash_attn_prefill,
                paged_attn_decode, pick_kv_splits)
 
 # name -> (kernel code, PyTorch function)
@@ -37,6 +39,31 @@ ACTIVATIONS = {"silu": (0, F.silu), "gelu_tanh": (1, lambda z: F.gelu(z, approxi
                "relu2": (2, lambda z: F.relu(z).square()), "tanh": (3, torch.tanh), "sigmoid": (4, torch.sigmoid),
                "none": (5, lambda z: z)}
 CLAMPED = 6                  # of a gate and up pair (`gated_act`)
+XIELU = 7                    # with two parameters (`Act`)
+
+
+def xielu(z: torch.Tensor, a: float, b: float) -> torch.Tensor:
+    return torch.where(z > 0, a * z * z, b * (torch.expm1(z) - z)) + z / 2
+
+
+class Act(NamedTuple):
+    """An activation with its parameters: "xielu" is a z^2 + z / 2 above zero and b (exp(z) - 1 - z) + z / 2 below."""
+    name: str
+    a: float = 0.0
+    b: float = 0.0
+
+    @staticmethod
+    def of(act: Union[str, "Act"]) -> "Act":
+        return act if isinstance(act, Act) else Act(act)
+
+    @property
+    def code(self) -> int:
+        return XIELU if self.name == "xielu" else ACTIVATIONS[self.name][0]
+
+
+def activate(z: torch.Tensor, act: Union[str, Act]) -> torch.Tensor:
+    act = Act.of(act)
+    return xielu(z, act.a, act.b) if act.name == "xielu" else ACTIVATIONS[act.name][1](z)
 
 
 class Proj(NamedTuple):
@@ -62,7 +89,8 @@ class Proj(NamedTuple):
 class Branch(NamedTuple):
     """One addend of a residual update: scale * y; with gate and bias, sigmoid(gate + bias) * y; with a gate of one column and no
     bias, scale * sigmoid(gate) * y; with pair_pos [T * k] and pair_w [T, k] (None with top_k = k: ones),
-    scale * sum_j pair_w[t, j] * y[pair_pos[t * k + j]] (routed experts); with norm, scale * norm * y / sqrt(mean(y^2) + eps)."""
+    scale * sum_j pair_w[t, j] * y[pair_pos[t * k + j]] (routed experts); with norm, scale * norm * y / sqrt(mean(y^2) + eps).
+    shift (fp32 [width], a projection's bias) is added to y first, in plain and normed branches."""
     y: Proj
     gate: Optional[Proj] = None
     bias: Optional[torch.Tensor] = None
@@ -71,6 +99,12 @@ class Branch(NamedTuple):
     pair_w: Optional[torch.Tensor] = None
     top_k: int = 0
     norm: Optional[torch.Tensor] = None
+    shift: Optional[torch.Tensor] = None
+
+    @property
+    def simple(self) -> bool:
+        """Whether it is only scaled or normed."""
+        return self.gate is None and self.pair_pos is None
 
     @property
     def chosen(self) -> int:
@@ -82,7 +116,7 @@ class Branch(NamedTuple):
             rows = self.y.value()[pos.long().clamp(min=0)]
             w = (pos >= 0) if self.pair_w is None else self.pair_w * (pos >= 0)
             return self.scale * (rows * w[..., None]).sum(1)
-        y = self.y.value()
+        y = self.y.value() if self.shift is None else self.y.value() + self.shift
         if self.norm is not None:
             return self.scale * y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps) * self.norm
         if self.gate is not None:
@@ -104,22 +138,37 @@ class Branch(NamedTuple):
 
 class Norm(NamedTuple):
     """What reads the residual: its RMS norm with a weight (a bare tensor means the same), with center its layer norm with
-    weight and bias, without a weight the residual itself."""
+    weight and bias, with alpha tanh(alpha * x) * weight + bias (no mean or variance), without a weight the residual itself."""
     weight: Optional[torch.Tensor] = None
     bias: Optional[torch.Tensor] = None
     center: bool = False
+    alpha: Optional[float] = None
 
     @property
     def kind(self) -> int:
-        return 2 if self.weight is None else (1 if self.center else 0)
+        return 2 if self.weight is None else (3 if self.alpha is not None else 1 if self.center else 0)
 
     def value(self, x: torch.Tensor, groups: int, eps: float) -> torch.Tensor:
         if self.weight is None:
             return x
+        if self.alpha is not None:
+            return torch.tanh(self.alpha * x) * self.weight + self.bias
         if self.center:
             d = x - x.mean(-1, keepdim=True)
             return d / torch.sqrt(d.pow(2).mean(-1, keepdim=True) + eps) * self.weight + self.bias
         return group_rmsnorm_ref(x, self.weight, groups, eps)
+
+    def arg(self, out: Optional[torch.Tensor] = None) -> _lib.TanhNormArg:
+        return _lib.TanhNormArg(_ptr(self.weight), _ptr(self.bias), float(self.alpha or 0.0), _ptr(out))
+
+
+class History(NamedTuple):
+    """Earlier results that a residual update averages with its own: sum_j coef[j] * rows[j] over j < past, + coef[past] * r.
+    rows fp32 [n, T, W]; coef fp32 [past + 1]; store: r also goes to rows[past]."""
+    rows: torch.Tensor
+    past: int
+    coef: torch.Tensor
+    store: bool = True
 
 
 def _ref(p: Proj):
@@ -157,15 +206,18 @@ def group_rmsnorm_ref(x: torch.Tensor, w: torch.Tensor, groups: int, eps: float)
 def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Branch] = (), *,
                    ids: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None, scale: float = 1.0,
                    add_mat: Optional[torch.Tensor] = None, add_row: Optional[torch.Tensor] = None,
-                   norms: Sequence = (), groups: int = 1, eps: float = 1e-6,
-                   dtype: torch.dtype = torch.bfloat16) -> Tuple[torch.Tensor, List[torch.Tensor]]:
+                   norms: Sequence = (), groups: int = 1, eps: float = 1e-6, dtype: torch.dtype = torch.bfloat16,
+                   post: Optional[Norm] = None, history: Optional[History] = None,
+                   out: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, List[torch.Tensor]]:
     """One residual update of an fp32 stream and the norms that read it.
 
         r = x  (or table[ids] * scale)
-        r += sum over branches (see `Branch`);   r += add_mat;   r += add_row
+        r += sum over branches (see `Branch`), with `post` (a tanh norm) its value of that sum;   r += add_mat;   r += add_row
+        r = average with earlier results (see `History`)
         h_j = w_j * (r divided, in `groups` equal parts, by sqrt(mean(part^2) + eps)), or as `Norm` says (one kind per call)
 
-    x [T, W] fp32; gate biases, add_row and the norm weights fp32 [W]; add_mat fp32 [T, W].  Returns (r, [h_j in `dtype`])."""
+    x [T, W] fp32; gate biases, add_row and the norm weights fp32 [W]; add_mat fp32 [T, W].  Returns (r, [h_j in `dtype`]), r in
+    `out` when given."""
     branches = [b if isinstance(b, Branch) else Branch(*b) for b in branches]
     norms = [n if isinstance(n, Norm) else Norm(n) for n in norms]
     if len({n.kind for n in norms}) > 1:
@@ -176,20 +228,28 @@ def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Branch] = (), *
     else:
         rows, width = ids.numel(), table.shape[1]
         dev = table.device
-    r = torch.empty((rows, width), dtype=torch.float32, device=dev)
+    r = out if out is not None else torch.empty((rows, width), dtype=torch.float32, device=dev)
     outs = [torch.empty((rows, width), dtype=dtype, device=dev) for _ in norms]
     if not _native(r):
         acc = x.clone() if x is not None else table[ids.long().clamp(0, table.shape[0] - 1)].float() * scale
         if branches:
-            acc = acc + sum(b.value(eps) for b in branches)
+            s = sum(b.value(eps) for b in branches)
+            acc = acc + (s if post is None else post.value(s, 1, eps))
         if add_mat is not None:
             acc = acc + add_mat
         if add_row is not None:
             acc = acc + add_row
+        if history is not None:
+            if history.store:
+                history.rows[history.past].copy_(acc)
+            acc = acc * history.coef[-1] + torch.einsum("n,ntw->tw", history.coef[:-1], history.rows[:history.past])
         r.copy_(acc)
         for o, n in zip(outs, norms):
             o.copy_(n.value(acc, groups, eps).to(dtype))
         return r, outs
+    if (post is not None or history is not None or any(n.kind == 3 for n in norms) or any(b.shift is not None for b in branches)
+            or sum(b.norm is not None for b in branches) > 1):
+        return _post_residual(x, branches, ids, table, scale, add_mat, add_row, norms, groups, eps, dtype, post, history, r, outs)
     weights, biases = [n.weight for n in norms], [n.bias for n in norms]
     for t in [x, add_mat, add_row, *weights, *biases, *[b.bias for b in branches], *[b.norm for b in branches]]:
         if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
@@ -203,6 +263,45 @@ def gated_residual(x: Optional[torch.Tensor], branches: Sequence[Branch] = (), *
         1 if dtype == torch.bfloat16 else 0, rows, width, int(groups), float(eps), _stream())
     _lib.check(rc, "nkb_gated_residual")
     _count_launch()
+    return r, outs
+
+
+def _post_residual(x, branches, ids, table, scale, add_mat, add_row, norms, groups, eps, dtype, post, history, r, outs):
+    """The forms of `gated_residual` that csrc/kernels/post_residual.cu computes."""
+    if len(branches) > 2 or not all(b.simple for b in branches):
+        raise ValueError("a norm or an average after the sum takes at most two branches, scaled or normed")
+    if post is not None and post.kind not in (2, 3):
+        raise ValueError("the norm of the branches is a tanh norm")
+    later = (norms and norms[0].kind in (0, 1)) or add_mat is not None or add_row is not None
+    inner = [] if later else norms
+    coef = None if history is None else history.coef
+    for t in [x, coef, r, *[v for n in [post or Norm(), *inner] for v in (n.weight, n.bias)],
+              *[v for b in branches for v in (b.norm, b.shift)]]:
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
+            raise TypeError("gated_residual wants contiguous fp32 residuals, biases and norm weights")
+    a = _lib.PostResidualArg()
+    a.x_in, a.ids, a.table, a.x_out = _ptr(x), _ptr(ids), _ptr(table), r.data_ptr()
+    for i, b in enumerate(branches):
+        a.br[i] = _lib.PostBranchArg(b.y.arg(), _ptr(b.shift), _ptr(b.norm), float(b.scale))
+    a.post = (post or Norm()).arg()
+    for i, (n, o) in enumerate(zip(inner, outs)):
+        a.norm[i] = n.arg(o)
+    if history is not None:
+        rows = history.rows
+        if rows.dtype != torch.float32 or not rows[0].is_contiguous() or coef.numel() != history.past + 1:
+            raise ValueError("a history is fp32 rows and one coefficient per result")
+        a.history, a.history_stride, a.past, a.coef = rows.data_ptr(), rows.stride(0), history.past, coef.data_ptr()
+        a.result = rows[history.past].data_ptr() if history.store else None
+    if table is not None:
+        a.vocab, a.table_bf16 = table.shape[0], 1 if table.dtype == torch.bfloat16 else 0
+    a.branches, a.norms, a.out_bf16 = len(branches), len(inner), 1 if dtype == torch.bfloat16 else 0
+    a.rows, a.width = r.shape
+    a.table_scale, a.eps = float(scale), float(eps)
+    _lib.check(_lib.lib().nkb_post_residual(ctypes.byref(a), _stream()), "nkb_post_residual")
+    _count_launch()
+    if later:
+        out, hs = gated_residual(r, add_mat=add_mat, add_row=add_row, norms=norms, groups=groups, eps=eps, dtype=dtype)
+        return r.copy_(out), hs
     return r, outs
 
 
@@ -228,16 +327,17 @@ def gated_act(gate: Proj, up: Proj, act: str = "silu", dtype: torch.dtype = torc
     return out
 
 
-def activation(x: Proj, act: str, dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
+def activation(x: Proj, act: Union[str, Act], dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
     """``act(x)`` -> [T, width] in `dtype`."""
+    act = Act.of(act)
     rows = x.t.shape[-2]
     out = torch.empty((rows, x.width), dtype=dtype, device=x.t.device)
     if not _native(out):
-        out.copy_(ACTIVATIONS[act][1](x.value()).to(dtype))
+        out.copy_(activate(x.value(), act).to(dtype))
         return out
     none = _lib.ProjArg(None, 0, 0, 1, 0)
     rc = _lib.lib().nkb_gated_act(_ref(x), ctypes.byref(none), out.data_ptr(), 1 if dtype == torch.bfloat16 else 0, rows,
-                                  x.width, ACTIVATIONS[act][0], 0.0, 0.0, None, 0, _stream())
+                                  x.width, act.code, act.a, act.b, None, 0, _stream())
     _lib.check(rc, "nkb_gated_act")
     _count_launch()
     return out
@@ -357,7 +457,9 @@ class MapsSpec:
     dim_p / vdim_p are the padded sizes of queries / keys (per map) and values in the cache; the tiled bf16 kernels
     take 32 or 64 and 64 or 128, other sizes are only rounded to even and use the general kernel.  With one map the tiled
     kernels are those of plain attention, which take one size of 64 or 128 for both.  window > 0 (one map): a query sees
-    itself and the window - 1 tokens before it.  chunk > 0 (one map): it sees the tokens of its own chunk of that many positions."""
+    itself and the window - 1 tokens before it, and the first keep_first ones.  chunk > 0 (one map): it sees the tokens of its own
+    chunk of that many positions.  dist_a, dist_b (one map, fp32 [heads]): after the cap a score loses dist_a * ln(1 + dist_b *
+    distance)."""
     heads: int
     kv_heads: int
     dim: int
@@ -371,11 +473,18 @@ class MapsSpec:
     tiled: bool = True
     window: int = 0
     chunk: int = 0
+    keep_first: int = 0
+    dist_a: Optional[torch.Tensor] = None
+    dist_b: Optional[torch.Tensor] = None
 
     @property
     def plain(self) -> bool:
         """Whether the kernels of plain attention serve this (one map, sizes they take)."""
-        return self.tiled and self.maps == 1 and self.softcap <= 0 and max(self.dim, self.vdim) <= 128
+        return self.tiled and self.maps == 1 and max(self.dim, self.vdim) <= 128
+
+    @property
+    def mods(self) -> ScoreMods:
+        return ScoreMods(self.softcap, self.keep_first, self.dist_a, self.dist_b)
 
     @property
     def dim_p(self) -> int:
@@ -392,7 +501,8 @@ class MapsSpec:
     def arg(self) -> _lib.MapsArg:
         return _lib.MapsArg(self.maps, self.heads, self.kv_heads, self.dim, self.dim_p, self.vdim, self.vdim_p,
                             float(self.scale), float(self.softcap), float(self.lam), float(self.out_scale),
-                            float(self.eps), int(self.window), int(self.chunk), None, 0, 0, 0, 0, 0)
+                            float(self.eps), int(self.window), int(self.chunk), None, 0, 0, 0, 0, 0, int(self.keep_first),
+                            _ptr(self.dist_a), _ptr(self.dist_b))
 
 
 def row_norm_append(spec: MapsSpec, q: Proj, k: Proj, v: Proj, q_norm: torch.Tensor, k_norm: torch.Tensor,
@@ -436,12 +546,22 @@ def half_rotate(x: torch.Tensor, cos_sin: torch.Tensor, positions: torch.Tensor)
     return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * n:]], -1)
 
 
+def pair_rotate(x: torch.Tensor, cos_sin: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+    """x [T, n, d] fp32 with the first cos_sin.shape[1] dimensions rotated, dimension 2i paired with 2i + 1."""
+    n = cos_sin.shape[1] // 2
+    cs = cos_sin[positions.long().clamp(0, cos_sin.shape[0] - 1)]
+    c, s = cs[:, None, :n], cs[:, None, n:]
+    u, v = x[..., :2 * n:2], x[..., 1:2 * n:2]
+    return torch.cat([torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2), x[..., 2 * n:]], -1)
+
+
 def rope_norm_append(spec: MapsSpec, q: Proj, k: Optional[Proj], v: Optional[Proj], bias: Optional[torch.Tensor],
-                     cos_sin: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, k_cache: torch.Tensor,
-                     v_cache: torch.Tensor, norm: bool = True) -> torch.Tensor:
-    """Add the biases (fp32 [q | k | v]), rotate the first cos_sin.shape[1] dimensions of every head of queries and keys (dimension
-    i paired with i + half), with `norm` divide every head by sqrt(mean(head^2) + spec.eps), write keys and values to their
-    cache slots (negative slot: not stored) and return the queries [T, heads, dim_p].  k and v None: only the queries."""
+                     cos_sin: Optional[torch.Tensor], positions: torch.Tensor, slots: torch.Tensor, k_cache: torch.Tensor,
+                     v_cache: torch.Tensor, norm: bool = True, interleaved: bool = False) -> torch.Tensor:
+    """Add the biases (fp32 [q | k | v]), rotate the first cos_sin.shape[1] dimensions (cos_sin None: none) of every head of queries
+    and keys (dimension i paired with i + half, interleaved: 2i with 2i + 1), with `norm` divide every head by
+    sqrt(mean(head^2) + spec.eps), write keys and values to their cache slots (negative slot: not stored) and return the
+    queries [T, heads, dim_p].  k and v None: only the queries."""
     T = q.t.shape[-2]
     H, G, d, dp = spec.heads, spec.kv_heads, spec.dim, spec.dim_p
     bs = k_cache.shape[2]
@@ -449,7 +569,9 @@ def rope_norm_append(spec: MapsSpec, q: Proj, k: Optional[Proj], v: Optional[Pro
     if not _native(k_cache):
         def head(x, n, first):
             x = x.value() if bias is None else x.value() + bias[first:first + x.width]
-            x = half_rotate(x.reshape(T, n, d), cos_sin, positions)
+            x = x.reshape(T, n, d)
+            if cos_sin is not None:
+                x = (pair_rotate if interleaved else half_rotate)(x, cos_sin, positions)
             if norm:
                 x = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + spec.eps)
             return F.pad(x, (0, dp - d)).to(k_cache.dtype)
@@ -469,7 +591,8 @@ def rope_norm_append(spec: MapsSpec, q: Proj, k: Optional[Proj], v: Optional[Pro
     a, none = spec.arg(), ctypes.byref(_lib.ProjArg(None, 0, 0, 1, 0))
     rc = _lib.lib().nkb_rope_norm_append(
         ctypes.byref(a), _ref(q), none if k is None else _ref(k), none if v is None else _ref(v), _ptr(bias),
-        cos_sin.data_ptr(), cos_sin.shape[1], cos_sin.shape[0], positions.data_ptr(), slots.data_ptr(), 1 if norm else 0,
+        _ptr(cos_sin), *((0, 1) if cos_sin is None else (cos_sin.shape[1], cos_sin.shape[0])), positions.data_ptr(),
+        slots.data_ptr(), 1 if norm else 0, 1 if interleaved else 0,
         q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), 1 if k_cache.dtype == torch.bfloat16 else 0, T, bs, _stream())
     _lib.check(rc, "nkb_rope_norm_append")
     _count_launch()
@@ -528,16 +651,16 @@ def heads_attention(spec: MapsSpec, q: torch.Tensor, k_cache: torch.Tensor, v_ca
     T, H = q.shape[0], spec.heads
     bs = k_cache.shape[2]
     B = block_table.shape[0]
-    if (spec.window > 0 or spec.chunk > 0 or sinks is not None) and spec.maps != 1:
-        raise ValueError("windows, chunks and sinks are for one score map")
+    if (spec.window > 0 or spec.chunk > 0 or sinks is not None or spec.dist_a is not None) and spec.maps != 1:
+        raise ValueError("windows, chunks, sinks and distance terms are for one score map")
     if _native(k_cache) and spec.plain:
         qf = q.reshape(T, -1)
         if q_lens is None:
             o = paged_attn_decode(qf, k_cache, v_cache, block_table, context_lens, spec.scale, window=spec.window,
-                                  chunk=spec.chunk, sinks=sinks, num_splits=num_splits)
+                                  chunk=spec.chunk, sinks=sinks, mods=spec.mods, num_splits=num_splits)
         else:
             o = flash_attn_prefill(qf, k_cache, v_cache, block_table, q_start, q_lens, context_lens, spec.scale,
-                                   max_q_len=max_q_len, window=spec.window, chunk=spec.chunk, sinks=sinks)
+                                   max_q_len=max_q_len, window=spec.window, chunk=spec.chunk, sinks=sinks, mods=spec.mods)
         return o.view(T, H, spec.vdim_p)[..., :spec.vdim]
     out = torch.empty((T, H, spec.vdim), dtype=k_cache.dtype, device=k_cache.device)
     if not _native(k_cache):
@@ -554,14 +677,14 @@ def heads_attention(spec: MapsSpec, q: torch.Tensor, k_cache: torch.Tensor, v_ca
             v = _gather_kv(v_cache, block_table[b], ctx).float()[..., :spec.vdim]
             k, v = k.repeat_interleave(rep, 1), v.repeat_interleave(rep, 1)
             s = torch.einsum("qhmd,khmd->hmqk", q[t0:t0 + n].float().reshape(n, H, M, dp), k) * spec.scale
-            if spec.softcap > 0:
-                s = spec.softcap * torch.tanh(s / spec.softcap)
             pos = (ctx - n + torch.arange(n))[:, None]
-            vis = torch.arange(ctx)[None, :] <= pos
+            key = torch.arange(ctx)[None, :]
+            s = spec.mods.apply(s, pos - key)
+            vis = key <= pos
             if spec.window > 0:
-                vis &= torch.arange(ctx)[None, :] > pos - spec.window
+                vis &= (key > pos - spec.window) | (key < spec.keep_first)
             if spec.chunk > 0:
-                vis &= torch.arange(ctx)[None, :] >= pos - pos % spec.chunk
+                vis &= key >= pos - pos % spec.chunk
             s = s.masked_fill(~vis, float("-inf"))
             if sinks is not None:
                 s = torch.cat([s, sinks.float()[:, None, None, None].expand(H, M, n, 1)], -1)
