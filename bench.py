@@ -92,8 +92,8 @@ def parse_args():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "eager", "eager-graph"],
                     help="eager-graph: the eager PyTorch decode step captured in a CUDA graph (static cache, position "
                          "on the device), so the comparison is not against Python launch overhead; dense models")
-    ap.add_argument("--model", default="llama3-8b", choices=["llama3-8b", "qwen3-30b-a3b", "gpt-oss-20b", "tolenex", "mumilorn", "ligizen"],
-                    help="tolenex, mumilorn, ligizen: prefill and decode of a layer-by-layer design beside the closest other model of "
+    ap.add_argument("--model", default="llama3-8b", choices=["llama3-8b", "qwen3-30b-a3b", "gpt-oss-20b", "tolenex", "mumilorn", "ligizen", "redodra"],
+                    help="tolenex, mumilorn, ligizen, redodra: prefill and decode of a layer-by-layer design beside the closest other model of "
                          "equal size")
     ap.add_argument("--sizes", default="2048x5632x16,4096x14336x8",
                     help="layer-by-layer designs: width x feed-forward x layers of the compared models")
@@ -382,7 +382,7 @@ def main():
     return 0
 
 
-LAYERED = ("tolenex", "mumilorn", "ligizen")
+LAYERED = ("tolenex", "mumilorn", "ligizen", "redodra")
 
 
 def compared_models(design, width, ff, layers, vocab):
@@ -402,6 +402,8 @@ def compared_models(design, width, ff, layers, vocab):
                 "mumilorn-moe": C.mumilorn_shape(width, **shape, experts=32, top=4, expert_ff=ff // 8, groups=8, keep=4)}
     if design == "mumilorn":
         return {**mumilorn, "tolenex": tolenex}
+    if design == "redodra":
+        return {"redodra": C.redodra_shape(width, **shape), "mumilorn": mumilorn["mumilorn"]}
     return {"ligizen": C.ligizen_shape(width, **shape),
             "ligizen-moe": C.ligizen_shape(width, **shape, experts=32, top=4, expert_ff=ff // 8), **mumilorn}
 

@@ -64,7 +64,7 @@ class _TimedLib:
                   "nkb_embedding", "nkb_rope", "nkb_decode_advance", "nkb_sample", "nkb_router", "nkb_paged_attn_decode",
                   "nkb_flash", "nkb_ag_gemm", "nkb_decode_gemm", "nkb_lmhead", "nkb_gated", "nkb_hgrn2", "nkb_maps",
                   "nkb_linattn", "nkb_low_rank", "nkb_token_mix", "nkb_gate_heads", "nkb_row_norm",
-                  "nkb_latent", "nkb_softcap")
+                  "nkb_latent", "nkb_softcap", "nkb_post", "nkb_short_conv", "nkb_head_rec")
 
     def __init__(self, real):
         object.__setattr__(self, "_real", real)
@@ -86,7 +86,7 @@ class _TimedLib:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--model", default="llama3-8b", choices=["llama3-8b", "qwen3-30b-a3b", "tolenex", "mumilorn", "ligizen"])
+    ap.add_argument("--model", default="llama3-8b", choices=["llama3-8b", "qwen3-30b-a3b", "tolenex", "mumilorn", "ligizen", "redodra"])
     ap.add_argument("--prefill", action="store_true", help="time one packed prefill of the batch instead of a decode step")
     ap.add_argument("--shard-of", type=int, default=1, help="run the per-rank shard of an N-way TP model on one GPU")
     ap.add_argument("--layers", type=int, default=None)
@@ -119,6 +119,8 @@ def main(argv=None) -> int:
     if args.model == "ligizen":
         cfg = C.ligizen_shape(4096, layers=args.layers or 32, heads=32, kv_heads=8, ff=14336, experts=32, top=4, expert_ff=1792,
                               moe_every=4)
+    if args.model == "redodra":
+        cfg = C.redodra_shape(4096, layers=args.layers or 30, heads=32, kv_heads=8, ff=14336)
     batch = args.batch or (128 if moe else 64)
     prompt_len = args.prompt_len or (512 if moe else 1024)
     if args.layers and cfg.layers is None:

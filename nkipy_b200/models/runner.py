@@ -16,7 +16,7 @@ from typing import List, Optional
 import torch
 
 from ..parallel.comm import TPGroup
-from .config import ModelConfig, ligizen_shape, mumilorn_shape, tolenex_shape
+from .config import ModelConfig, ligizen_shape, mumilorn_shape, redodra_shape, tolenex_shape
 from .engine import GenerationEngine, Sampling
 from .weights import load_shard
 
@@ -72,6 +72,9 @@ def shrink(cfg: ModelConfig) -> ModelConfig:
         return ligizen_shape(256, layers=len(cfg.layers), heads=4, kv_heads=2, ff=512, vocab=2048, dim=32, window=64, chunk=48,
                              latent_dim=40, rot=8, kv_rank=48, q_rank=96, side=32, share_every=2,
                              **(dict(experts=8, top=2, expert_ff=64) if routed else {}))
+    if cfg.name == "redodra":
+        return redodra_shape(256, layers=len(cfg.layers), heads=4, kv_heads=2, ff=512, vocab=2048, dim=32, window=64, keep_first=3,
+                             state=16, groups=2, share_every=2)
     if cfg.layers is not None:
         return tolenex_shape(256, layers=len(cfg.layers), heads=4, kv_heads=1, ff=512, vocab=2048, dim=32, vdim=64,
                              groups=cfg.norm_groups, loop=cfg.loop, embedding_scale=cfg.embedding_scale)

@@ -21,7 +21,7 @@ import torch
 
 from . import (add_rmsnorm, decode_linear, flash_attn_prefill, grouped_linear, linear, moe_combine, moe_dispatch,
                paged_attn_decode, router_topk)
-from . import microbench_mixers
+from . import microbench_mixers, microbench_sandwich
 
 _FALLBACK = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
 
@@ -399,7 +399,8 @@ CASES = {
     "moe-ep-block-tp1": case_moe_push,
     "add-rmsnorm": case_addnorm,
 }
-CASES.update({name: (lambda a, fn=fn: fn(a, _time, _sets_for)) for name, fn in microbench_mixers.CASES.items()})
+CASES.update({name: (lambda a, fn=fn: fn(a, _time, _sets_for))
+              for name, fn in {**microbench_mixers.CASES, **microbench_sandwich.CASES}.items()})
 
 
 def main(argv=None):

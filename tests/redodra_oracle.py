@@ -205,3 +205,59 @@ def forward(raw, weights, ids):
         x = depth_average(W[p + "dwa"], results)
         taps.append(x)
     return norm(x, "final.norm") @ W["head"].T, taps
+
+
+# ----------------------------------------------------------------------------- small models for the tests
+def small_config(width=88, vocab=150, layers="dpakp", mlps="dd-dd", ff=104, heads=4, kv_heads=2, dim=24, vdim=40, rot=16, base=900.0,
+                 cap=9.0, scale=None, dheads=4, dkv=2, ddim=16, dvdim=24, dconv=3, lheads=6, lkv=2, ldim=20, lvdim=28, window=19,
+                 first=5, lcap=7.0, lscale=None, rheads=6, groups=3, state=12, rvdim=20, rconv=4, parts=2, eps=1e-4):
+    """config.json contents.  Layers: 'd' delta rule, 'D' the same with other sizes, 'p' attention beside the state-space mixer, 'a'
+    attention, 'k' attention on the keys of the last 'a'; mlps: 'd' dense, '-' none."""
+    specs, source = [], None
+    for i, (c, f) in enumerate(zip(layers, mlps)):
+        if c in "dD":
+            kind, n = "delta", c == "D"
+            m = {"heads": dheads * (1 + n), "kv_heads": dkv, "dim": ddim + 8 * n, "vdim": dvdim, "conv": dconv + n}
+        elif c == "p":
+            kind = "parallel"
+            m = {"left": {"heads": lheads, "kv_heads": lkv, "dim": ldim, "vdim": lvdim, "scale": lscale or 1.5 * ldim ** -0.5,
+                          "softcap": lcap, "mask": {"size": window, "keep_first": first}},
+                 "right": {"heads": rheads, "groups": groups, "state": state, "vdim": rvdim, "conv": rconv, "norm_groups": parts}}
+        else:
+            kind = "attention"
+            m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale or 1.5 * dim ** -0.5, "softcap": cap,
+                 "rot": {"base": base, "dims": rot}}
+            if c == "k":
+                m["kv_from"] = source
+            else:
+                source = i
+        specs.append({"type": kind, "mixer": m, "mlp": {"kind": "dense", "ff": ff} if f == "d" else None})
+    return {"architecture": "Redodra", "layers": specs, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def small_weights(raw, shapes, seed=0):
+    """bf16 tensors of the given name -> shape map, scaled so that every mechanism has a visible effect: scores of several
+    units, sinks that take a share, decays from fast to slow, averages that mix all depths."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in shapes.items():
+        x, leaf = torch.randn(shape, generator=g), name.rsplit(".", 1)[-1]
+        if name.endswith(".mix.sink"):
+            x = 1 + x
+        elif leaf in ("r1", "r2"):
+            x = torch.rand(shape, generator=g) * (0.8 if leaf == "r1" else 0.3) + 0.1
+        elif leaf == "alpha":
+            x = 0.5 + 0.5 * torch.rand(shape, generator=g)
+        elif leaf in ("A_log", "dt_bias"):
+            x = x - 1
+        elif leaf == "dwa":
+            x = 0.3 * x
+            x[-1] += 1
+        elif leaf == "conv":
+            x = x / shape[-1] ** 0.5
+        elif len(shape) == 1 and leaf != "act":
+            x = 0.4 * x + (leaf in ("norm1", "norm2", "norm1b", "norm2b", "norm", "out", "D"))
+        elif len(shape) == 2 and name != "embed":
+            x = x * (2.0 if leaf in ("q", "k") else 1.2) / shape[-1] ** 0.5
+        out[name] = x.to(torch.bfloat16)
+    return out
