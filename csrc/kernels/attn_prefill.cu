@@ -73,6 +73,7 @@ struct PrefillParams {
   int nq, nkv, max_blocks, causal, window, chunk;
   float scale_log2;
   NkbScoreMods mods;                   // MODS only
+  int dist_far;                        // > 0: the terms up to this distance are a table in shared memory
 };
 
 struct PrefillCtrl {
@@ -121,12 +122,19 @@ struct PrefillSmem {
   static constexpr int kQBytes = NK * kHalf;          // one query tile
   static constexpr int kStageBytes = (NK > NV ? NK : NV) * kKVHalf;
   static constexpr int kPBytes = KT / 64 * kHalf;     // [128 rows][KT tokens]
-  static constexpr int kStages = NK == 3 ? 4 : 3;
+  static constexpr int kStages = NK == 3 || KT == 64 ? 4 : 3;
   static constexpr int kBytes = 2 * kQBytes + kStages * kStageBytes + 2 * kPBytes + int(sizeof(PrefillCtrl)) + 1024 + 64;
+  // Table of the distance term: element j of a copy belongs to distance far - j.  Tiles that a query tile walks hold distances from
+  // -(126 + KT) to window + KT + 253.  Copy c starts c elements later, so that four scores of any row are one aligned access;
+  // its pitch spreads the copies over the banks.
+  static __host__ __device__ constexpr int far_of(int window) { return window + KT + 256; }
+  static __host__ __device__ constexpr int pitch_of(int far) { return (far + KT + 128 + 4 + 31) / 32 * 32 + 8; }
 };
 
-// MODS: scores are capped, lose a term that grows with the distance, or the first tokens stay visible outside the window.  The cap is
-// the one of attn_maps_prefill.cu (an odd polynomial where all scores of a row are small, the exponential form otherwise).
+// MODS: scores are capped, lose a term that grows with the distance, or the first tokens stay visible outside the window.
+// The special-function unit is the bottleneck of the softmax, so that it should see no more than one operation per score: the cap is
+// an odd polynomial where all scores of a row stay below 0.35 or 1.1 of it (fits at Chebyshev nodes, relative errors 4e-8 and 2e-8;
+// beyond, the exponential form), and the distance term is read from a table wherever a window bounds the distances.
 template <int NK, int NV, int KT, bool ROWS, bool MODS>
 __global__ void __launch_bounds__(kPfThreads, 1)
 flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
@@ -197,6 +205,19 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
   if (warp == 1) {
     tmem_alloc(&ctrl->tmem_base, kTmemCols);
     tmem_relinquish();
+  }
+  if constexpr (MODS) {
+    if (p.dist_far > 0) {
+      const float da = p.mods.dist_a[head], db = p.mods.dist_b[head];
+      float* tab = reinterpret_cast<float*>(ctrl + 1);
+      const int pitch = L::pitch_of(p.dist_far);
+      for (int j = threadIdx.x; j < pitch + 3; j += kPfThreads) {
+        const float x = -da * __log2f(fmaf(db, float(max(p.dist_far - j, 0)), 1.f));
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+          if (j >= c && j - c < pitch) tab[c * pitch + j - c] = x;
+      }
+    }
   }
   tc_fence_before();
   __syncthreads();
@@ -374,7 +395,17 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
     const bool capped = MODS && p.mods.softcap > 0.f, distant = MODS && p.mods.dist_a != nullptr;
     const float k_y = capped ? p.scale_log2 / (kLog2e * p.mods.softcap) : 0.f;   // raw score -> argument of tanh
     const float cap2 = p.mods.softcap * kLog2e;
-    const float poly_raw = capped ? 0.6f / fmaxf(fabsf(k_y), 1e-30f) : 0.f;
+    // the polynomial's coefficients take the scales in (which must not underflow)
+    const float poly_raw = capped && fabsf(k_y) > 1e-4f ? 0.35f / fabsf(k_y) : -1.f;
+    const float wide_raw = capped ? 1.1f / fmaxf(fabsf(k_y), 1e-30f) : 0.f;
+    const float k2 = k_y * k_y, c0 = 0.999999965517f * cap2 * k_y, c1 = -0.333324263276f * cap2 * k_y * k2;
+    const float c2 = 0.132958838057f * cap2 * k_y * k2 * k2, c3 = -0.048962819976f * cap2 * k_y * k2 * k2 * k2;
+    const int far = MODS ? p.dist_far : 0, first_j = far - q_pos;        // table element of key 0
+    const float* dist_row = nullptr;
+    if (MODS && far > 0) {
+      const int copy = first_j & 3;                                       // tiles start at multiples of four
+      dist_row = reinterpret_cast<const float*>(ctrl + 1) + copy * L::pitch_of(far) + (first_j - copy);
+    }
     const float dist_a = distant ? p.mods.dist_a[head] : 0.f, dist_b = distant ? p.mods.dist_b[head] : 0.f;
     // raw scores become exponents of two in the exponential's multiply-add, or (MODS) before it
     const float to_log2 = MODS ? 1.f : p.scale_log2;
@@ -402,19 +433,28 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
             am4[(i >> 1) & 3] = fmax3(am4[(i >> 1) & 3], fabsf(__uint_as_float(v[i])), fabsf(__uint_as_float(v[i + 1])));
           const float am = fmaxf(fmaxf(am4[0], am4[1]), fmaxf(am4[2], am4[3]));
           if (__all_sync(0xffffffffu, am <= poly_raw)) {
-            // y * P(y^2), P(u) ~ tanh(sqrt(u)) / sqrt(u) on [0, 0.36]
-            const float2 ky2 = make_float2(k_y, k_y), c2 = make_float2(cap2, cap2);
+            const float2 d0 = make_float2(c0, c0), d1 = make_float2(c1, c1), d2 = make_float2(c2, c2), d3 = make_float2(c3, c3);
+#pragma unroll
+            for (int i = 0; i < kKVTile; i += 2) {
+              const float2 y = make_float2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), u = fmul2(y, y);
+              const float2 w = fmul2(y, ffma2(ffma2(ffma2(u, d3, d2), u, d1), u, d0));
+              v[i] = __float_as_uint(w.x);
+              v[i + 1] = __float_as_uint(w.y);
+            }
+          } else if (__all_sync(0xffffffffu, am <= wide_raw)) {
+            const float2 ky2 = make_float2(k_y, k_y), cc = make_float2(cap2, cap2);
             const auto dup = [](float x) { return make_float2(x, x); };
 #pragma unroll
             for (int i = 0; i < kKVTile; i += 2) {
-              const float2 y = fmul2(make_float2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), ky2);
-              const float2 u = fmul2(y, y);
-              float2 q = ffma2(u, dup(-0.005856427870f), dup(0.020757475450f));
-              q = ffma2(q, u, dup(-0.053769921786f));
-              q = ffma2(q, u, dup(0.133317047022f));
-              q = ffma2(q, u, dup(-0.333332839718f));
-              q = ffma2(q, u, dup(0.999999997563f));
-              const float2 w = fmul2(fmul2(y, c2), q);
+              const float2 y = fmul2(make_float2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), ky2), u = fmul2(y, y);
+              float2 q = ffma2(u, dup(-0.000275233992f), dup(0.002002967295f));
+              q = ffma2(q, u, dup(-0.007526384788f));
+              q = ffma2(q, u, dup(0.021194377645f));
+              q = ffma2(q, u, dup(-0.053775426680f));
+              q = ffma2(q, u, dup(0.133305659147f));
+              q = ffma2(q, u, dup(-0.333331798889f));
+              q = ffma2(q, u, dup(0.999999985913f));
+              const float2 w = fmul2(fmul2(y, cc), q);
               v[i] = __float_as_uint(w.x);
               v[i + 1] = __float_as_uint(w.y);
             }
@@ -430,7 +470,18 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
 #pragma unroll
           for (int i = 0; i < kKVTile; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * p.scale_log2);
         }
-        if (distant) {
+        if (dist_row && it >= kept) {
+#pragma unroll
+          for (int i = 0; i < kKVTile; i += 4) {
+            const float4 d = *reinterpret_cast<const float4*>(dist_row + kv0 + i);
+            const float2 a = fadd2(make_float2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), make_float2(d.x, d.y));
+            const float2 b = fadd2(make_float2(__uint_as_float(v[i + 2]), __uint_as_float(v[i + 3])), make_float2(d.z, d.w));
+            v[i] = __float_as_uint(a.x);
+            v[i + 1] = __float_as_uint(a.y);
+            v[i + 2] = __float_as_uint(b.x);
+            v[i + 3] = __float_as_uint(b.y);
+          }
+        } else if (distant) {
           // dist_a ln(1 + dist_b d) in units of ln 2; keys after the query (negative distances) are masked below
           const float d0 = fmaf(dist_b, float(q_pos - kv0), 1.f);
 #pragma unroll
@@ -594,15 +645,24 @@ flash_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
 
 template <int NK, int NV, int KT, bool ROWS, bool MODS = false>
 static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tr,
-                          const PrefillParams& p, int batch, int max_q_len, cudaStream_t s) {
-  constexpr int smem = PrefillSmem<NK, NV, KT>::kBytes;
-  static_assert(smem <= 232448, "shared memory of a CTA");
+                          PrefillParams p, int batch, int max_q_len, cudaStream_t s) {
+  using L = PrefillSmem<NK, NV, KT>;
+  constexpr int most = 232448;
+  static_assert(L::kBytes <= most && sizeof(PrefillCtrl) % 16 == 0, "shared memory of a CTA");
+  int smem = L::kBytes;
+  if (MODS && p.mods.dist_a && p.window > 0 && p.window <= 4096) {
+    const int far = L::far_of(p.window), bytes = smem + 16 * L::pitch_of(far);
+    if (bytes <= most) {
+      p.dist_far = far;
+      smem = bytes;
+    }
+  }
   static bool attr_set[64] = {false};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -1;
   if (!attr_set[dev]) {
     cudaError_t e = cudaFuncSetAttribute(flash_attn_prefill_kernel<NK, NV, KT, ROWS, MODS>,
-                                         cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize, MODS ? most : smem);
     if (e != cudaSuccess) return int(e);
     attr_set[dev] = true;
   }
@@ -652,7 +712,8 @@ extern "C" int nkb_flash_attn_prefill(const void* q, const void* k_cache, const 
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (mods) {
     p.mods = *mods;
-    if (head_dim == 128) return launch_prefill<2, 2, 128, false, true>(tq, tk, tv, tk, p, batch, max_q_len, s);
+    // tiles of 64 tokens: fewer scores in registers at once, and room for the table beside heads of 128
+    if (head_dim == 128) return launch_prefill<2, 2, 64, false, true>(tq, tk, tv, tk, p, batch, max_q_len, s);
     if (head_dim == 64) return launch_prefill<1, 1, 128, false, true>(tq, tk, tv, tk, p, batch, max_q_len, s);
     return -2;
   }

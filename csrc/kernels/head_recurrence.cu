@@ -34,35 +34,63 @@ struct ShortConvParams {
   float* state;
   const int *slot_ids, *q_start, *q_lens, *context_lens;
   void* out;                // [tokens, channels]
-  int batch, tokens, channels, taps, act;
+  int batch, tokens, channels, taps, act, run;      // run: tokens of a CTA
 };
-constexpr int kConvTokens = 16;
+constexpr int kConvTokens = 64;     // at most
 constexpr int kMaxTaps = 8;
 
+// V channels of a row: as they lie in memory (bf16 in one piece), and as numbers
 template <int V>
-__device__ __forceinline__ void load_chan(float (&x)[V], const NkbProj& s, long long row, int c) {
-  if constexpr (V == 8) {
-    const uint4 r = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(s.ptr) + row * s.ld + c);
+struct ChanRaw {
+  float x;
+  __device__ __forceinline__ void load(const NkbProj& s, long long row, int c) { x = proj_load(s, row, c); }
+  __device__ __forceinline__ void get(float (&o)[V]) const { o[0] = x; }
+};
+template <>
+struct ChanRaw<4> {
+  uint2 r;
+  __device__ __forceinline__ void load(const NkbProj& s, long long row, int c) {
+    r = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(s.ptr) + row * s.ld + c);
+  }
+  __device__ __forceinline__ void get(float (&o)[4]) const {
+    const float2 a = unpack_bf16x2(r.x), b = unpack_bf16x2(r.y);
+    o[0] = a.x; o[1] = a.y; o[2] = b.x; o[3] = b.y;
+  }
+};
+template <>
+struct ChanRaw<8> {
+  uint4 r;
+  __device__ __forceinline__ void load(const NkbProj& s, long long row, int c) {
+    r = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(s.ptr) + row * s.ld + c);
+  }
+  __device__ __forceinline__ void get(float (&o)[8]) const {
     const uint32_t w[4] = {r.x, r.y, r.z, r.w};
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const float2 f = unpack_bf16x2(w[e]);
-      x[2 * e] = f.x;
-      x[2 * e + 1] = f.y;
+      o[2 * e] = f.x;
+      o[2 * e + 1] = f.y;
     }
-  } else {
-    x[0] = proj_load(s, row, c);
   }
+};
+
+// z sigmoid(z) with the approximate exponential and reciprocal, for results that are stored in bf16
+__device__ __forceinline__ float silu_fast(float z) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-1.4426950408889634f * z));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return z * r;
 }
 
-// A CTA owns TB tokens and 128 V channels; V = 8: finished bf16 values in whole 16-byte pieces.  seq_of: the token's sequence.
+// A CTA owns a run of tokens and 128 V channels; V = 4: finished bf16 values in aligned pieces of four.  Four tokens are loaded while
+// the four before them are computed.  seq_of: the token's sequence.
 template <int V, int TAPS, typename OutT>
 __global__ void __launch_bounds__(128) short_conv_kernel(const __grid_constant__ ShortConvParams p) {
-  constexpr int TB = kConvTokens, H = TAPS > 1 ? TAPS - 1 : 1;
-  __shared__ int seq_of[TB];
-  const int t0 = blockIdx.y * TB, nt = min(TB, p.tokens - t0);
+  constexpr int H = TAPS > 1 ? TAPS - 1 : 1, AHEAD = 4;
+  __shared__ int seq_of[kConvTokens];
+  const int t0 = blockIdx.y * p.run, nt = min(p.run, p.tokens - t0);
   const int c = (blockIdx.x * 128 + threadIdx.x) * V;
-  if (threadIdx.x < TB) seq_of[threadIdx.x] = -1;
+  if (threadIdx.x < kConvTokens) seq_of[threadIdx.x] = -1;
   float w[TAPS][V], bias[V];
   if (c < p.channels) {
 #pragma unroll
@@ -74,6 +102,12 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const __grid_constant__
   }
   griddep_wait();
   griddep_launch();
+  ChanRaw<V> cur[AHEAD], next[AHEAD];
+  const auto fetch = [&](ChanRaw<V> (&r)[AHEAD], int i0) {
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) r[k].load(p.x, t0 + min(i0 + k, nt - 1), c);
+  };
+  if (c < p.channels) fetch(cur, 0);
   __syncthreads();
   for (int b = threadIdx.x; b < p.batch; b += 128) {
     const int s = p.q_start[b], e = s + p.q_lens[b];
@@ -89,56 +123,65 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const __grid_constant__
     for (int e = 0; e < V; ++e) past[l][e] = 0.f;
   int seq = -1;
 #pragma unroll 1
-  for (int i = 0; i < nt; ++i) {
-    const long long t = t0 + i;
-    float x[V];
-    load_chan<V>(x, p.x, t, c);
-    const int b = seq_of[i];
-    if (b >= 0 && b != seq) {                        // what precedes the first of this CTA's tokens of the sequence
-      const int first = p.q_start[b], n = p.q_lens[b], ctx = p.context_lens[b];
-      const float* st = p.state + (long long)(p.slot_ids ? p.slot_ids[b] : b) * TAPS * p.channels + c;
+  for (int i0 = 0; i0 < nt; i0 += AHEAD) {
+    fetch(next, i0 + AHEAD);                         // (past the end: the last token again)
 #pragma unroll
-      for (int l = 0; l < TAPS - 1; ++l) {
-        const long long from = t - 1 - l;
-        const int pos = ctx - n + int(from - first);
-        if (from >= first) {
-          load_chan<V>(past[l], p.x, from, c);
-        } else {
+    for (int k = 0; k < AHEAD; ++k) {
+      const int i = i0 + k;
+      if (i >= nt) break;
+      const long long t = t0 + i;
+      float x[V];
+      cur[k].get(x);
+      const int b = seq_of[i];
+      if (b >= 0 && b != seq) {                      // what precedes the first of this CTA's tokens of the sequence
+        const int first = p.q_start[b], n = p.q_lens[b], ctx = p.context_lens[b];
+        const float* st = p.state + (long long)(p.slot_ids ? p.slot_ids[b] : b) * TAPS * p.channels + c;
 #pragma unroll
-          for (int e = 0; e < V; ++e) past[l][e] = ctx >= n && pos >= 0 ? st[(long long)(pos % TAPS) * p.channels + e] : 0.f;
+        for (int l = 0; l < TAPS - 1; ++l) {
+          const long long from = t - 1 - l;
+          const int pos = ctx - n + int(from - first);
+          if (from >= first) {
+            ChanRaw<V> r;
+            r.load(p.x, from, c);
+            r.get(past[l]);
+          } else {
+#pragma unroll
+            for (int e = 0; e < V; ++e) past[l][e] = ctx >= n && pos >= 0 ? st[(long long)(pos % TAPS) * p.channels + e] : 0.f;
+          }
         }
       }
+      seq = b;
+      float y[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        y[e] = fmaf(w[TAPS - 1][e], x[e], bias[e]);
+#pragma unroll
+        for (int l = 0; l < TAPS - 1; ++l) y[e] = fmaf(w[TAPS - 2 - l][e], past[l][e], y[e]);
+      }
+      if (sizeof(OutT) == 2 && p.act == ACT_SILU) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[e] = silu_fast(y[e]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[e] = apply_act(y[e], p.act);
+      }
+      OutT* o = out + t * p.channels + c;
+      if constexpr (V == 4) {
+        *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]));
+      } else {
+        o[0] = cast_out<OutT>(y[0]);
+      }
+#pragma unroll
+      for (int l = TAPS - 2; l > 0; --l)
+#pragma unroll
+        for (int e = 0; e < V; ++e) past[l][e] = past[l - 1][e];
+      if constexpr (TAPS > 1) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) past[0][e] = x[e];
+      }
     }
-    seq = b;
-    float y[V];
 #pragma unroll
-    for (int e = 0; e < V; ++e) {
-      y[e] = fmaf(w[TAPS - 1][e], x[e], bias[e]);
-#pragma unroll
-      for (int l = 0; l < TAPS - 1; ++l) y[e] = fmaf(w[TAPS - 2 - l][e], past[l][e], y[e]);
-    }
-    if (sizeof(OutT) == 2 && p.act == ACT_SILU) {
-#pragma unroll
-      for (int e = 0; e < V; ++e) y[e] *= __fdividef(1.f, 1.f + __expf(-y[e]));
-    } else {
-#pragma unroll
-      for (int e = 0; e < V; ++e) y[e] = apply_act(y[e], p.act);
-    }
-    OutT* o = out + t * p.channels + c;
-    if constexpr (V == 8) {
-      *reinterpret_cast<uint4*>(o) = make_uint4(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]), pack_bf16x2(y[4], y[5]),
-                                                pack_bf16x2(y[6], y[7]));
-    } else {
-      o[0] = cast_out<OutT>(y[0]);
-    }
-#pragma unroll
-    for (int l = TAPS - 2; l > 0; --l)
-#pragma unroll
-      for (int e = 0; e < V; ++e) past[l][e] = past[l - 1][e];
-    if constexpr (TAPS > 1) {
-#pragma unroll
-      for (int e = 0; e < V; ++e) past[0][e] = x[e];
-    }
+    for (int k = 0; k < AHEAD; ++k) cur[k] = next[k];
   }
 }
 
@@ -155,8 +198,12 @@ __global__ void __launch_bounds__(256) conv_state_kernel(const __grid_constant__
 }
 
 template <int V, typename OutT>
-static int launch_conv(const ShortConvParams& p, cudaStream_t s) {
-  const dim3 grid((p.channels + 128 * V - 1) / (128 * V), (p.tokens + kConvTokens - 1) / kConvTokens), block(128);
+static int launch_conv(ShortConvParams p, cudaStream_t s) {
+  // long runs (what precedes a run is read again), as long as the grid fills the device a few times over
+  const int cols = (p.channels + 128 * V - 1) / (128 * V);
+  p.run = kConvTokens;
+  while (p.run > 4 && (long long)cols * ((p.tokens + p.run - 1) / p.run) < 148 * 16) p.run /= 2;
+  const dim3 grid(cols, (p.tokens + p.run - 1) / p.run), block(128);
   switch (p.taps) {
     case 1: return launch_pdl(short_conv_kernel<V, 1, OutT>, grid, block, 0, s, p);
     case 2: return launch_pdl(short_conv_kernel<V, 2, OutT>, grid, block, 0, s, p);
@@ -699,74 +746,122 @@ struct GroupNormParams {
   NkbProj g;                // [tokens, width]
   const float* w;
   void* out;
-  int width, parts, gate_act;
+  long long units;          // parts of tokens
+  int width, parts, warps, gate_act;      // warps: of a unit
   float eps;
 };
 
-// One CTA per token; V elements per access (8: bf16 in 16-byte pieces).  A part is shared by whole warps.
-template <int V, typename YT, typename OutT>
+// A unit (one part of one token) belongs to 1, 2, 4 or 8 warps; V elements per access: 8 of bf16, 4 of fp32 or split sums, or one.
+// R > 0: a lane's R vectors stay in registers; R = 0: longer parts are read again for the result.
+template <int V, int R, typename YT, typename OutT>
 __global__ void __launch_bounds__(256) group_norm_kernel(const __grid_constant__ GroupNormParams p) {
-  extern __shared__ __align__(16) float gn_s[];     // [width]
   __shared__ float red[8];
-  const long long t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, size = p.width / p.parts;
-  const int wpp = p.parts >= 8 ? 1 : 8 / p.parts;   // warps per part
+  const long long unit = blockIdx.x * (long long)(8 / p.warps) + warp / p.warps;
+  const bool on = unit < p.units;
+  const long long t = on ? unit / p.parts : 0;
+  const int first = on ? int(unit % p.parts) * size : 0;
+  const int i0 = (warp % p.warps * 32 + lane) * V, step = p.warps * 32 * V;
   griddep_wait();
   griddep_launch();
   const YT* y = reinterpret_cast<const YT*>(p.y) + t * p.width;
   OutT* out = reinterpret_cast<OutT*>(p.out) + t * p.width;
-  const int sub = warp % wpp;
-  for (int q0 = 0; q0 < p.parts; q0 += 8 / wpp) {   // the same number of turns for every warp
-    const int part = q0 + warp / wpp, first = part * size;
-    float ss = 0.f;
-    if (part < p.parts)
-      for (int i = (sub * 32 + lane) * V; i < size; i += wpp * 32 * V) {
-        const int c = first + i;
-        float x[V], gt[V];
-        if constexpr (V == 8) {
-          load_chan<8>(gt, p.g, t, c);
-          const uint4 r = *reinterpret_cast<const uint4*>(y + c);
-          const uint32_t rw[4] = {r.x, r.y, r.z, r.w};
+  const auto load = [&](float (&x)[V], int c) {
+    float gt[V];
+    if constexpr (V == 8) {
+      ChanRaw<8> a, b;
+      a.r = *reinterpret_cast<const uint4*>(y + c);
+      b.load(p.g, t, c);
+      a.get(x);
+      b.get(gt);
+    } else if constexpr (V == 4) {
+      const float4 a = *reinterpret_cast<const float4*>(y + c), b = proj_load4(p.g, t, c);
+      x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w;
+      gt[0] = b.x; gt[1] = b.y; gt[2] = b.z; gt[3] = b.w;
+    } else {
+      x[0] = cast_in<YT>(y[c]);
+      gt[0] = proj_load(p.g, t, c);
+    }
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const float2 f = unpack_bf16x2(rw[e]);
-            x[2 * e] = f.x;
-            x[2 * e + 1] = f.y;
-          }
-        } else {
-          x[0] = cast_in<YT>(y[c]);
-          gt[0] = proj_load(p.g, t, c);
-        }
+    for (int e = 0; e < V; ++e) {
+      if (sizeof(OutT) == 2 && p.gate_act == ACT_SILU) x[e] *= silu_fast(gt[e]);
+      else x[e] *= apply_act(gt[e], p.gate_act);
+    }
+  };
+  const auto store = [&](const float (&x)[V], int c, float inv) {
+    float r[V];
+    if constexpr (V >= 4) {
 #pragma unroll
-        for (int e = 0; e < V; ++e) {
-          if (V == 8 && p.gate_act == ACT_SILU) x[e] *= gt[e] * __fdividef(1.f, 1.f + __expf(-gt[e]));
-          else x[e] *= apply_act(gt[e], p.gate_act);
-          ss = fmaf(x[e], x[e], ss);
-          gn_s[c + e] = x[e];
-        }
+      for (int e = 0; e < V; e += 4) {
+        const float4 w = *reinterpret_cast<const float4*>(p.w + c + e);
+        r[e] = x[e] * inv * w.x;
+        r[e + 1] = x[e + 1] * inv * w.y;
+        r[e + 2] = x[e + 2] * inv * w.z;
+        r[e + 3] = x[e + 3] * inv * w.w;
       }
-    ss = warp_sum(ss);
+    } else {
+      r[0] = x[0] * inv * p.w[c];
+    }
+    if constexpr (V == 8)
+      *reinterpret_cast<uint4*>(out + c) =
+          make_uint4(pack_bf16x2(r[0], r[1]), pack_bf16x2(r[2], r[3]), pack_bf16x2(r[4], r[5]), pack_bf16x2(r[6], r[7]));
+    else if constexpr (V == 4 && sizeof(OutT) == 2)
+      *reinterpret_cast<uint2*>(out + c) = make_uint2(pack_bf16x2(r[0], r[1]), pack_bf16x2(r[2], r[3]));
+    else if constexpr (V == 4)
+      *reinterpret_cast<float4*>(out + c) = make_float4(r[0], r[1], r[2], r[3]);
+    else
+      out[c] = cast_out<OutT>(r[0]);
+  };
+  float x[R > 0 ? R : 1][V], ss = 0.f;
+  if constexpr (R > 0) {
+#pragma unroll
+    for (int k = 0; k < R; ++k) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[k][e] = 0.f;
+      if (on && i0 + k * step < size) load(x[k], first + i0 + k * step);
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss = fmaf(x[k][e], x[k][e], ss);
+    }
+  } else if (on) {
+    for (int i = i0; i < size; i += step) {
+      load(x[0], first + i);
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss = fmaf(x[0][e], x[0][e], ss);
+    }
+  }
+  ss = warp_sum(ss);
+  if (p.warps > 1) {
     if (lane == 0) red[warp] = ss;
     __syncthreads();
-    if (part < p.parts) {
-      float tot = 0.f;
-      for (int w = 0; w < wpp; ++w) tot += red[warp / wpp * wpp + w];
-      const float inv = 1.f / sqrtf(tot / float(size) + p.eps);
-      for (int i = (sub * 32 + lane) * V; i < size; i += wpp * 32 * V) {
-        const int c = first + i;
-        float x[V];
-#pragma unroll
-        for (int e = 0; e < V; ++e) x[e] = gn_s[c + e] * inv * p.w[c + e];
-        if constexpr (V == 8) {
-          *reinterpret_cast<uint4*>(out + c) = make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]),
-                                                          pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
-        } else {
-          out[c] = cast_out<OutT>(x[0]);
-        }
-      }
-    }
-    __syncthreads();
+    ss = 0.f;
+    for (int w = 0; w < p.warps; ++w) ss += red[warp / p.warps * p.warps + w];
   }
+  if (!on) return;
+  const float inv = 1.f / sqrtf(ss / float(size) + p.eps);
+  if constexpr (R > 0) {
+#pragma unroll
+    for (int k = 0; k < R; ++k)
+      if (i0 + k * step < size) store(x[k], first + i0 + k * step, inv);
+  } else {
+    for (int i = i0; i < size; i += step) {
+      load(x[0], first + i);
+      store(x[0], first + i, inv);
+    }
+  }
+}
+
+template <int V, typename YT, typename OutT>
+static int launch_group_norm(GroupNormParams p, cudaStream_t s) {
+  const int size = p.width / p.parts, vectors = (size + V - 1) / V;
+  // one warp per unit while that leaves four vectors or less per lane, more for long parts or few units
+  p.warps = 1;
+  while (p.warps < 8 && (vectors > 128 * p.warps || (p.units * p.warps < 148 * 16 && vectors > 32 * p.warps))) p.warps *= 2;
+  const dim3 grid(unsigned((p.units + 8 / p.warps - 1) / (8 / p.warps))), block(256);
+  const int rounds = (vectors + 32 * p.warps - 1) / (32 * p.warps);
+  if (rounds <= 1) return launch_pdl(group_norm_kernel<V, 1, YT, OutT>, grid, block, 0, s, p);
+  if (rounds <= 2) return launch_pdl(group_norm_kernel<V, 2, YT, OutT>, grid, block, 0, s, p);
+  if (rounds <= 4) return launch_pdl(group_norm_kernel<V, 4, YT, OutT>, grid, block, 0, s, p);
+  return launch_pdl(group_norm_kernel<V, 0, YT, OutT>, grid, block, 0, s, p);
 }
 
 static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
@@ -786,13 +881,13 @@ extern "C" int nkb_short_conv(const NkbProj* x, const float* w, const float* b, 
                               const int* q_start, const int* q_lens, const int* context_lens, void* out, int bf16, int batch,
                               int tokens, int channels, int taps, int act, void* stream) {
   if (batch <= 0 || tokens <= 0) return 0;
-  if (channels < 1 || taps < 1 || taps > kMaxTaps || batch > 65535 || (tokens + kConvTokens - 1) / kConvTokens > 65535 || act < 0 ||
+  if (channels < 1 || taps < 1 || taps > kMaxTaps || batch > 65535 || tokens > 4 * 65535 || act < 0 ||
       act >= ACT_CLAMPED || !q_start || !q_lens)
     return -2;
-  ShortConvParams p{*x, w, b, state, slot_ids, q_start, q_lens, context_lens, out, batch, tokens, channels, taps, act};
+  ShortConvParams p{*x, w, b, state, slot_ids, q_start, q_lens, context_lens, out, batch, tokens, channels, taps, act, 0};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   int rc;
-  if (bf16 && x->bf16 && channels % 8 == 0 && x->ld % 8 == 0 && al16(x->ptr) && al16(out)) rc = launch_conv<8, __nv_bfloat16>(p, s);
+  if (bf16 && x->bf16 && channels % 4 == 0 && proj_vec4_ok(*x) && al16(out)) rc = launch_conv<4, __nv_bfloat16>(p, s);
   else rc = bf16 ? launch_conv<1, __nv_bfloat16>(p, s) : launch_conv<1, float>(p, s);
   if (rc) return rc;
   return launch_pdl(conv_state_kernel, dim3((channels + 255) / 256, batch), dim3(256), 0, s, p);
@@ -825,20 +920,16 @@ extern "C" int nkb_head_rec_step(const NkbHeadRec* a, void* stream) {
 extern "C" int nkb_gated_group_norm(const void* y, int y_bf16, const NkbProj* gate, int gate_act, const float* w, float eps,
                                     void* out, int out_bf16, int tokens, int width, int parts, void* stream) {
   if (tokens <= 0) return 0;
-  if (width < 1 || width > 24000 || parts < 1 || width % parts || gate_act < 0 || gate_act >= ACT_CLAMPED || !gate->ptr || !w) return -2;
-  GroupNormParams p{y, *gate, w, out, width, parts, gate_act, eps};
+  if (width < 1 || parts < 1 || width % parts || gate_act < 0 || gate_act >= ACT_CLAMPED || !gate->ptr || !w) return -2;
+  GroupNormParams p{y, *gate, w, out, (long long)tokens * parts, width, parts, 1, gate_act, eps};
+  if (p.units > 0x7fffffffll) return -2;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  const size_t smem = size_t(width) * sizeof(float);
-  auto launch = [&](auto kernel) {
-    if (smem > 40 * 1024) {
-      const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem));
-      if (e != cudaSuccess) return int(e);
-    }
-    return launch_pdl(kernel, dim3(tokens), dim3(256), smem, s, p);
-  };
   using bf = __nv_bfloat16;
-  if (y_bf16 && out_bf16 && gate->bf16 && (width / parts) % 8 == 0 && al16(y) && al16(out) && al16(gate->ptr) && gate->ld % 8 == 0)
-    return launch(group_norm_kernel<8, bf, bf>);
-  if (y_bf16) return out_bf16 ? launch(group_norm_kernel<1, bf, bf>) : -2;
-  return out_bf16 ? launch(group_norm_kernel<1, float, bf>) : launch(group_norm_kernel<1, float, float>);
+  const int size = width / parts;
+  if (y_bf16 && out_bf16 && gate->bf16 && size % 8 == 0 && al16(y) && al16(w) && al16(out) && al16(gate->ptr) && gate->ld % 8 == 0)
+    return launch_group_norm<8, bf, bf>(p, s);
+  if (!y_bf16 && size % 4 == 0 && al16(y) && al16(w) && al16(out) && proj_vec4_ok(*gate))
+    return out_bf16 ? launch_group_norm<4, float, bf>(p, s) : launch_group_norm<4, float, float>(p, s);
+  if (y_bf16) return out_bf16 ? launch_group_norm<1, bf, bf>(p, s) : -2;
+  return out_bf16 ? launch_group_norm<1, float, bf>(p, s) : launch_group_norm<1, float, float>(p, s);
 }

@@ -511,7 +511,7 @@ def test_inactive_rows_of_a_step_are_left_alone(device, dtype):
 
 @on_devices
 @in_dtypes
-@pytest.mark.parametrize("W,parts", [(96, 1), (96, 3), (70, 5), (2048, 8), (2048, 16), (2048, 1), (40, 40)])
+@pytest.mark.parametrize("W,parts", [(96, 1), (96, 3), (70, 5), (2048, 8), (2048, 16), (2048, 1), (40, 40), (12288, 1), (1056, 1)])
 def test_gated_group_norm(device, dtype, W, parts):
     y, w = rnd(5, W, seed=1).to(dtype), 1 + rnd(W, seed=2)
     y[1] *= 1e-2
