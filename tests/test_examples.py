@@ -51,6 +51,12 @@ def test_ligizen_example_cpu():
     assert "Decode tokens/sec" in out
 
 
+def test_redodra_example_cpu():
+    out = _run("examples/models/redodra/redodra.py", "--tiny", "--batch", "2", "--prompt-len", "12", "-n", "3",
+               "--max-seq-len", "96", "--dtype", "float32", "--layers", "5")
+    assert "Decode tokens/sec" in out
+
+
 def test_embedding_example_cpu():
     out = _run("examples/models/qwen3_embedding/example_retrieval.py", "--layers", "1", "--device", "cpu")
     cos = float(out.strip().splitlines()[-1].split()[-1])

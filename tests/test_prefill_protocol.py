@@ -40,27 +40,30 @@ class Barrier:
 
 
 class Sim:
-    def __init__(self, n0, n1, lo0, lo1, seed, lockstep=True):
+    def __init__(self, n0, n1, lo0, lo1, seed, lockstep=True, kept=0, stages=KV_STAGES):
         """Query tile t attends to KV tiles [lo_t, lo_t + n_t) of the CTA's union range (n1 = 0: no second tile).
         lockstep=False lets an issuer release the stage of a KV tile its query tile skips without waiting for the
-        load, which is how the kernel first was written."""
+        load, which is how the kernel first was written.  kept: tiles of kept first tokens, which both query tiles attend to,
+        come ahead of the union range.  stages: of the ring (four for tiles of 64 tokens)."""
         self.rng = random.Random(seed)
         self.lockstep = lockstep
         self.two = n1 > 0
-        self.a_lo = [lo0, lo1 if self.two else 0]
-        self.a_hi = [lo0 + n0, lo1 + n1 if self.two else 0]
+        self.kept, self.stages = kept, stages
+        self.a_lo = [kept + lo0, kept + lo1 if self.two else 0]      # walk positions, behind the kept tiles
+        self.a_hi = [kept + lo0 + n0, kept + lo1 + n1 if self.two else 0]
+        self.n_tiles = [kept + n0, kept + n1 if self.two else 0]
         self.n_union = max(self.a_hi[0], self.a_hi[1]) if self.two else self.a_hi[0]
-        assert min(self.a_lo[0], self.a_lo[1] if self.two else self.a_lo[0]) == 0
-        self.kv_full = [Barrier(1) for _ in range(KV_STAGES)]
-        self.kv_empty = [Barrier(2 if self.two else 1) for _ in range(KV_STAGES)]
+        assert min(self.a_lo[0], self.a_lo[1] if self.two else self.a_lo[0]) == kept
+        self.kv_full = [Barrier(1) for _ in range(stages)]
+        self.kv_empty = [Barrier(2 if self.two else 1) for _ in range(stages)]
         self.s_full = [Barrier(1), Barrier(1)]
         self.s_empty = [Barrier(4), Barrier(4)]
         self.p_full = [Barrier(4), Barrier(4)]
         self.o_full = [Barrier(1), Barrier(1)]
         self.turn = [[Barrier(1) for _ in range(4)] for _ in range(2)]
         # data tags
-        self.stage_tag = [None] * KV_STAGES          # ("K" | "V", x) once the load has landed
-        self.stage_readers = [0] * KV_STAGES         # MMAs in flight that read the stage
+        self.stage_tag = [None] * stages          # ("K" | "V", x) once the load has landed
+        self.stage_readers = [0] * stages         # MMAs in flight that read the stage
         self.s_tag = [None, None]                    # local iteration whose scores S_t holds
         self.s_unread = [0, 0]                       # softmax warps that have not read S_t yet
         self.p_tag = [[None] * 4, [None] * 4]        # per softmax warp: iteration whose probabilities it wrote
@@ -101,7 +104,7 @@ class Sim:
                 order.append(("K", u + 1))
             order.append(("V", u))
         for kind, x in order:
-            st, ph = seq % KV_STAGES, (seq // KV_STAGES) & 1
+            st, ph = seq % self.stages, (seq // self.stages) & 1
             seq += 1
             yield lambda st=st, ph=ph: self.kv_empty[st].test(ph ^ 1)
             assert self.stage_readers[st] == 0, "ring stage overwritten while an MMA still reads it"
@@ -118,7 +121,9 @@ class Sim:
         if t == 1 and not self.two:
             return
         seq = 0
-        a_lo, a_hi = self.a_lo[t], self.a_hi[t]
+        a_lo, a_hi, kept = self.a_lo[t], self.a_hi[t], self.kept
+        attends = lambda x: x < kept or a_lo <= x < a_hi
+        turn_of = lambda x: x if x < kept else x - a_lo + kept
 
         def read_stage(st, want):
             def start():
@@ -132,11 +137,11 @@ class Sim:
                 return
             item = seq
             seq += 1
-            st, par = item % KV_STAGES, (item // KV_STAGES) & 1
-            if self.lockstep or a_lo <= x < a_hi:
+            st, par = item % self.stages, (item // self.stages) & 1
+            if self.lockstep or attends(x):
                 yield lambda: self.kv_full[st].test(par)
-            if a_lo <= x < a_hi:
-                lit = x - a_lo
+            if attends(x):
+                lit = turn_of(x)
                 yield lambda: self.s_empty[t].test((lit & 1) ^ 1)
                 assert self.s_unread[t] == 0, "S_t overwritten before every softmax warp has read it"
 
@@ -154,11 +159,11 @@ class Sim:
             nonlocal seq
             item = seq
             seq += 1
-            st, par = item % KV_STAGES, (item // KV_STAGES) & 1
-            if self.lockstep or a_lo <= x < a_hi:
+            st, par = item % self.stages, (item // self.stages) & 1
+            if self.lockstep or attends(x):
                 yield lambda: self.kv_full[st].test(par)
-            if a_lo <= x < a_hi:
-                lit = x - a_lo
+            if attends(x):
+                lit = turn_of(x)
                 yield lambda: self.p_full[t].test(lit & 1)
 
                 def start(st=st, lit=lit):
@@ -182,8 +187,7 @@ class Sim:
             yield from do_v(u)
 
     def softmax(self, t, quad):
-        n = self.a_hi[t] - self.a_lo[t]
-        n_other = self.a_hi[1 - t] - self.a_lo[1 - t]
+        n, n_other = self.n_tiles[t], self.n_tiles[1 - t]
         for it in range(n):
             yield lambda it=it: self.s_full[t].test(it & 1)
             assert self.s_tag[t] == it, (self.s_tag[t], it)
@@ -264,6 +268,14 @@ def test_protocol_finishes_and_keeps_its_data_under_random_interleavings(n0, n1,
         Sim(n0, n1, lo0, lo1, seed).run()
 
 
+@pytest.mark.parametrize("kept", [1, 2, 3])
+@pytest.mark.parametrize("stages", [3, 4])
+@pytest.mark.parametrize("n0,n1,lo0,lo1", SHAPES)
+def test_protocol_with_kept_tiles_ahead_of_the_window(n0, n1, lo0, lo1, stages, kept):
+    for seed in range(20):
+        Sim(n0, n1, lo0, lo1, seed, kept=kept, stages=stages).run()
+
+
 def test_the_model_notices_a_broken_protocol():
     """The checks have teeth: a ring whose items come in an order the issuers do not consume hangs or hands the MMA
     the wrong tile."""
@@ -274,7 +286,7 @@ def test_the_model_notices_a_broken_protocol():
             for u in range(self.n_union):                 # K(u), V(u) instead of K(u+1), V(u)
                 order += [("K", u), ("V", u)]
             for kind, x in order:
-                st, ph = seq % KV_STAGES, (seq // KV_STAGES) & 1
+                st, ph = seq % self.stages, (seq // self.stages) & 1
                 seq += 1
                 yield lambda st=st, ph=ph: self.kv_empty[st].test(ph ^ 1)
 
